@@ -1,4 +1,5 @@
-"""ctypes binding of libcacheir_b200.so (the C ABI declared in include/cacheir_b200.h).
+"""ctypes binding of libcacheir_b200.so (the C ABI declared in include/cacheir_b200.h)
+and libcacheir_b200_hybrid.so (include/cacheir_b200_hybrid.h).
 
 There is no fallback: if the shared library is missing the import of any
 compute entry point raises, telling the user to build it.
@@ -10,6 +11,7 @@ from ctypes import c_char_p, c_float, c_int, c_longlong, c_size_t, c_void_p
 from pathlib import Path
 
 LIB_PATH = Path(__file__).resolve().parent / "lib" / "libcacheir_b200.so"
+HYBRID_LIB_PATH = LIB_PATH.with_name("libcacheir_b200_hybrid.so")
 
 # name -> (restype, argtypes); mirrors include/cacheir_b200.h one to one
 SIGNATURES: dict[str, tuple[object, list[object]]] = {
@@ -102,7 +104,74 @@ SIGNATURES: dict[str, tuple[object, list[object]]] = {
     "cacheir_b200_advance_positions": (c_int, [c_void_p, c_void_p, c_int, c_void_p]),
 }
 
+
+
+class DenseArgs(ctypes.Structure):
+    """cacheir_b200_dense_args"""
+
+    _fields_ = [("x", c_void_p), ("w", c_void_p), ("y", c_void_p),
+                ("T", c_int), ("N", c_int), ("K", c_int), ("batch", c_int),
+                ("w_batch_rows", c_int), ("x_batch_cols", c_int), ("y_batch_cols", c_int), ("epilogue", c_int),
+                ("w_stride", c_longlong), ("x_stride", c_longlong), ("y_stride", c_longlong),
+                ("act_cols", c_int), ("next_mode", c_int), ("vocab", c_int), ("table_col", c_int),
+                ("gate", c_void_p), ("gate_stride", c_longlong), ("residual", c_void_p), ("norm_w", c_void_p), ("norm_b", c_void_p),
+                ("next_w", c_void_p), ("next_b", c_void_p), ("next_out", c_void_p), ("norm_alpha", c_float), ("next_alpha", c_float),
+                ("ids", c_void_p), ("table", c_void_p), ("table_stride", c_longlong)]
+
+
+class LatentArgs(ctypes.Structure):
+    """cacheir_b200_latent_args"""
+
+    _fields_ = [("positions", c_void_p), ("row_seg", c_void_p), ("cu_rows", c_void_p), ("page_table", c_void_p),
+                ("rows", c_int), ("segments", c_int), ("max_pages", c_int), ("page_size", c_int), ("num_slots", c_int),
+                ("heads", c_int), ("dim", c_int), ("rot_dim", c_int), ("vdim", c_int), ("kv_rank", c_int), ("window", c_int),
+                ("scale", c_float), ("pool", c_void_p), ("dtype", c_int), ("decode", c_int)]
+
+
+class RecurrenceArgs(ctypes.Structure):
+    """cacheir_b200_recurrence_args"""
+
+    _fields_ = [("positions", c_void_p), ("cu_rows", c_void_p), ("slots", c_void_p), ("rows", c_int), ("segments", c_int),
+                ("heads", c_int), ("dim", c_int), ("vdim", c_int), ("q", c_void_p), ("k", c_void_p), ("v", c_void_p),
+                ("stride", c_longlong), ("decay_pow", c_void_p), ("state", c_void_p), ("num_slots", c_int), ("out", c_void_p),
+                ("dtype", c_int)]
+
+
+_NEXT = [c_int, c_void_p, c_void_p, c_float, c_void_p]      # next_mode next_w next_b next_alpha next_out
+# mirrors include/cacheir_b200_hybrid.h one to one
+HYBRID_SIGNATURES: dict[str, tuple[object, list[object]]] = {
+    "cacheir_b200_dense_supported": (c_int, [c_int, c_longlong, c_longlong, c_int, c_int]),
+    "cacheir_b200_dense_gemm": (c_int, [c_void_p, c_void_p]),
+    "cacheir_b200_dense_simple": (c_int, [c_void_p] * 3 + [c_int] * 7 + [c_longlong] * 3 + [c_int, c_int, c_void_p]),
+    "cacheir_b200_scaled_embedding": (c_int, [c_void_p] * 3 + [c_int, c_int, c_int, c_float] + _NEXT + [c_int, c_void_p]),
+    "cacheir_b200_dyt_rows": (c_int, [c_void_p] * 4 + [c_float, c_void_p, c_int, c_int, c_int, c_void_p]),
+    "cacheir_b200_residual_dyt": (c_int, [c_void_p] * 4 + [c_float, c_int, c_int] + _NEXT + [c_int, c_void_p]),
+    "cacheir_b200_residual_rms": (c_int, [c_void_p] * 3 + [c_float, c_int, c_int] + _NEXT + [c_int, c_void_p]),
+    "cacheir_b200_gated_rms": (c_int, [c_void_p, c_void_p, c_longlong, c_void_p, c_float, c_void_p, c_int, c_int, c_int, c_void_p]),
+    "cacheir_b200_geglu_pairs": (c_int, [c_void_p, c_void_p, c_int, c_int, c_int, c_void_p]),
+    "cacheir_b200_gelu_embed": (c_int, [c_void_p] * 3 + [c_longlong, c_int, c_void_p, c_int, c_int, c_int, c_int, c_void_p]),
+    "cacheir_b200_silu_cols": (c_int, [c_void_p, c_int, c_longlong, c_int, c_int, c_void_p]),
+    "cacheir_b200_latent_prepare": (
+        c_int, [c_void_p, c_void_p, c_longlong, c_void_p, c_float, c_void_p, c_longlong, c_void_p, c_longlong, c_int, c_void_p,
+                c_int, c_int, c_void_p]),
+    "cacheir_b200_latent_attention_simple": (
+        c_int, [c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_void_p]),
+    "cacheir_b200_latent_attention_supported": (c_int, [c_int] * 4),
+    "cacheir_b200_latent_attention_splits": (c_int, [c_int] * 5),
+    "cacheir_b200_latent_attention_workspace_bytes": (c_size_t, [c_int] * 4),
+    "cacheir_b200_latent_attention": (c_int, [c_void_p] * 4 + [c_int, c_void_p, c_size_t, c_void_p]),
+    "cacheir_b200_recurrence_simple": (c_int, [c_void_p, c_void_p]),
+    "cacheir_b200_recurrence_step": (c_int, [c_void_p, c_void_p]),
+    "cacheir_b200_recurrence_chunked_supported": (c_int, [c_int] * 3),
+    "cacheir_b200_recurrence_workspace_bytes": (c_size_t, [c_int] * 5),
+    "cacheir_b200_recurrence_chunked": (c_int, [c_void_p, c_void_p, c_size_t, c_void_p]),
+    "cacheir_b200_hybrid_device_status": (c_int, [c_int]),
+}
+# entry points of glue.cu and misc.cu, which both libraries carry
+SHARED_NAMES = ("cacheir_b200_version", "cacheir_b200_error_string", "cacheir_b200_argmax_rows", "cacheir_b200_advance_positions")
+
 _LIB: ctypes.CDLL | None = None
+_HYBRID_LIB: ctypes.CDLL | None = None
 
 
 class CacheIRB200Error(RuntimeError):
@@ -127,7 +196,35 @@ def load() -> ctypes.CDLL:
     return lib
 
 
+def load_hybrid() -> ctypes.CDLL:
+    """The library of the hybrid families, loaded once. Raises if it is not built."""
+    global _HYBRID_LIB
+    if _HYBRID_LIB is not None:
+        return _HYBRID_LIB
+    if not HYBRID_LIB_PATH.exists():
+        raise CacheIRB200Error(
+            f"{HYBRID_LIB_PATH} is missing: build it first (python -m cacheir_b200.build --group hybrid). "
+            "cacheir_b200 has no CPU or PyTorch fallback.")
+    lib = ctypes.CDLL(str(HYBRID_LIB_PATH))
+    table = dict(HYBRID_SIGNATURES, **{name: SIGNATURES[name] for name in SHARED_NAMES})
+    for name, (restype, argtypes) in table.items():
+        fn = getattr(lib, name)
+        fn.restype = restype
+        fn.argtypes = argtypes
+    _HYBRID_LIB = lib
+    return lib
+
+
+def load_shared() -> ctypes.CDLL:
+    """A library that has the entry points of SHARED_NAMES: the one in use, else whichever is built."""
+    if _LIB is not None:
+        return _LIB
+    if _HYBRID_LIB is not None or (HYBRID_LIB_PATH.exists() and not LIB_PATH.exists()):
+        return load_hybrid()
+    return load()
+
+
 def check(code: int, what: str) -> None:
     if code != 0:
-        text = load().cacheir_b200_error_string(int(code)).decode("utf-8", "replace")
+        text = load_shared().cacheir_b200_error_string(int(code)).decode("utf-8", "replace")
         raise CacheIRB200Error(f"{what} failed with status {code}: {text}")

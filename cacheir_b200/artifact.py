@@ -180,9 +180,10 @@ class CompileArtifact:
 
     @classmethod
     def from_dict(cls, data: dict[str, Any]) -> "CompileArtifact":
+        from .models import config_from_dict        # (the registry imports this module)
         return cls(
             version=data.get("version", "0.1"), target=data.get("target", "cuda"), quant=data.get("quant"),
-            model_path=data.get("model_path", ""), config=ModelConfig.from_dict(data["config"]),
+            model_path=data.get("model_path", ""), config=config_from_dict(data["config"]),
             graphs={mode: Graph.from_dict(g) for mode, g in data.get("graphs", {}).items()},
             metadata=dict(data.get("metadata", {})),
         )

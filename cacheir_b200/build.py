@@ -1,11 +1,14 @@
-"""Build libcacheir_b200.so in-tree with nvcc for sm_100a.
+"""Build the CUDA libraries in-tree with nvcc for sm_100a.
 
-Usage: python -m cacheir_b200.build [--force] [--verbose]
+Usage: python -m cacheir_b200.build [--force] [--verbose] [--group core|hybrid]
 
-The library is a plain C-ABI shared object (no torch, no pybind): every .cu
-under csrc/ is compiled to an object with -gencode arch=compute_100a,code=sm_100a
-and linked with the static CUDA runtime. Objects are rebuilt only when their
-source or a header is newer.
+Two plain C-ABI shared objects (no torch, no pybind), each a group of the .cu
+files under csrc/ compiled with -gencode arch=compute_100a,code=sm_100a and
+linked with the static CUDA runtime: `core` (libcacheir_b200.so, Llama-shaped
+models) and `hybrid` (libcacheir_b200_hybrid.so, latent attention + linear
+recurrences). A model family names the group it needs, so a fresh checkout
+compiles only that. Objects are rebuilt only when their source or a header is
+newer.
 """
 from __future__ import annotations
 
@@ -21,7 +24,11 @@ PKG_DIR = Path(__file__).resolve().parent
 CSRC = PKG_DIR / "csrc"
 INCLUDE = PKG_DIR.parent / "include"
 BUILD_DIR = PKG_DIR / "build"
-LIB_PATH = PKG_DIR / "lib" / "libcacheir_b200.so"
+LIB_DIR = PKG_DIR / "lib"
+LIB_PATHS = {"core": LIB_DIR / "libcacheir_b200.so", "hybrid": LIB_DIR / "libcacheir_b200_hybrid.so"}
+LIB_PATH = LIB_PATHS["core"]
+HYBRID_ONLY = ("dense_gemm", "hybrid_glue", "latent_attention", "linear_recurrence")
+SHARED = ("glue", "misc")            # in both libraries: argmax, position bookkeeping, error text
 
 NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a",
@@ -45,11 +52,18 @@ def _stale(target: Path, deps: list[Path]) -> bool:
     return any(dep.stat().st_mtime > mtime for dep in deps)
 
 
-def build(force: bool = False, verbose: bool = False) -> Path:
+def group_sources(group: str) -> list[Path]:
+    if group == "hybrid":
+        return sorted(CSRC / f"{name}.cu" for name in HYBRID_ONLY + SHARED)
+    return sorted(src for src in CSRC.glob("*.cu") if src.stem not in HYBRID_ONLY)
+
+
+def build(force: bool = False, verbose: bool = False, groups: tuple[str, ...] = ("core", "hybrid")) -> Path:
+    """Bring the libraries of `groups` up to date; returns the path of the first one."""
     nvcc = find_nvcc()
     BUILD_DIR.mkdir(parents=True, exist_ok=True)
-    LIB_PATH.parent.mkdir(parents=True, exist_ok=True)
-    sources = sorted(CSRC.glob("*.cu"))
+    LIB_DIR.mkdir(parents=True, exist_ok=True)
+    sources = sorted({src for group in groups for src in group_sources(group)})
     headers = sorted(CSRC.glob("*.cuh")) + sorted(INCLUDE.glob("*.h")) + [Path(__file__)]
     extra = ["-Xptxas", "-v"] if verbose else []
 
@@ -65,21 +79,27 @@ def build(force: bool = False, verbose: bool = False) -> Path:
         return obj
 
     with ThreadPoolExecutor(max_workers=min(8, os.cpu_count() or 1)) as pool:
-        objects = list(pool.map(compile_one, sources))
+        objects = dict(zip(sources, pool.map(compile_one, sources)))
 
-    if force or _stale(LIB_PATH, objects):
-        cmd = [nvcc, "-shared", "-gencode", "arch=compute_100a,code=sm_100a", "-cudart", "static",
-               "-o", str(LIB_PATH), *map(str, objects)]
-        proc = subprocess.run(cmd, capture_output=True, text=True)
-        if proc.returncode != 0:
-            sys.stderr.write(proc.stdout + proc.stderr)
-            raise RuntimeError("linking libcacheir_b200.so failed")
-    return LIB_PATH
+    for group in groups:
+        target, members = LIB_PATHS[group], [objects[src] for src in group_sources(group)]
+        if force or _stale(target, members):
+            part = target.with_suffix(".so.part")      # a reader never sees a half-written library
+            cmd = [nvcc, "-shared", "-gencode", "arch=compute_100a,code=sm_100a", "-cudart", "static",
+                   "-o", str(part), *map(str, members)]
+            proc = subprocess.run(cmd, capture_output=True, text=True)
+            if proc.returncode != 0:
+                sys.stderr.write(proc.stdout + proc.stderr)
+                raise RuntimeError(f"linking {target.name} failed")
+            os.replace(part, target)
+    return LIB_PATHS[groups[0]]
 
 
 if __name__ == "__main__":
     parser = argparse.ArgumentParser(description=__doc__)
     parser.add_argument("--force", action="store_true")
     parser.add_argument("--verbose", action="store_true", help="print ptxas register/smem usage")
+    parser.add_argument("--group", choices=sorted(LIB_PATHS), help="build one library only")
     args = parser.parse_args()
-    print(build(force=args.force, verbose=args.verbose))
+    for name in (args.group,) if args.group else ("core", "hybrid"):
+        print(build(force=args.force, verbose=args.verbose, groups=(name,)))

@@ -1,0 +1,357 @@
+// Row operators of the hybrid families that are not a GEMM epilogue: embedding into the 32-bit residual stream, Dynamic
+// Tanh, the RMS-normed residual add, the gated RMS norm behind a recurrence, and the stand-alone forms of the dense
+// kernel's epilogues (used in 32-bit runs and for extents the tensor-core kernel does not take).
+#include "hybrid_common.cuh"
+
+namespace cb200 {
+namespace {
+
+struct NextArgs {
+  int mode;
+  const float* w;
+  const float* b;
+  float alpha;
+  void* out;
+};
+
+template <typename T>
+__device__ __forceinline__ void leave_next(const NextArgs& nx, size_t idx, int c, float s) {
+  if (nx.mode == CACHEIR_B200_NEXT_DYT) Elem<T>::st(static_cast<T*>(nx.out) + idx, fmaf(tanhf(nx.alpha * s), nx.w[c], nx.b[c]));
+  else if (nx.mode == CACHEIR_B200_NEXT_COPY) Elem<T>::st(static_cast<T*>(nx.out) + idx, s);
+}
+
+template <typename T>
+__global__ void __launch_bounds__(256)
+scaled_embedding_kernel(const T* __restrict__ table, const int64_t* __restrict__ ids, float* __restrict__ x, int width, int vocab,
+                        float scale, NextArgs nx) {
+  const size_t row = blockIdx.x;
+  const int64_t id = min(max(ids[row], static_cast<int64_t>(0)), static_cast<int64_t>(vocab - 1));
+  for (int c = blockIdx.y * 256 + threadIdx.x; c < width; c += gridDim.y * 256) {
+    const float s = Elem<T>::ld(table + id * width + c) * scale;
+    x[row * width + c] = s;
+    leave_next<T>(nx, row * width + c, c, s);
+  }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(256)
+dyt_rows_kernel(const float* __restrict__ x, const int32_t* __restrict__ row_index, const float* __restrict__ w,
+                const float* __restrict__ b, float alpha, T* __restrict__ out, int width) {
+  const size_t row = blockIdx.x;
+  const size_t src = row_index ? static_cast<size_t>(max(row_index[row], 0)) : row;
+  for (int c = blockIdx.y * 256 + threadIdx.x; c < width; c += gridDim.y * 256)
+    Elem<T>::st(out + row * width + c, fmaf(tanhf(alpha * x[src * width + c]), w[c], b[c]));
+}
+
+template <typename T>
+__global__ void __launch_bounds__(256)
+residual_dyt_kernel(float* __restrict__ x, const T* __restrict__ y, const float* __restrict__ w, const float* __restrict__ b,
+                    float alpha, int width, NextArgs nx) {
+  const size_t row = blockIdx.x;
+  for (int c = blockIdx.y * 256 + threadIdx.x; c < width; c += gridDim.y * 256) {
+    const size_t i = row * width + c;
+    const float s = x[i] + fmaf(tanhf(alpha * Elem<T>::ld(y + i)), w[c], b[c]);
+    x[i] = s;
+    leave_next<T>(nx, i, c, s);
+  }
+}
+
+// VEC neighbouring elements per access, PT accesses per thread kept in registers between the two passes
+template <typename T, int VEC>
+__device__ __forceinline__ void load_vec(const T* p, float (&v)[VEC]) {
+  if constexpr (VEC == 4 && sizeof(T) == 2) {
+    const uint2 raw = *reinterpret_cast<const uint2*>(p);
+    v[0] = __uint_as_float(raw.x << 16); v[1] = __uint_as_float(raw.x & 0xffff0000u);
+    v[2] = __uint_as_float(raw.y << 16); v[3] = __uint_as_float(raw.y & 0xffff0000u);
+  } else if constexpr (VEC == 4) {
+    const float4 f = *reinterpret_cast<const float4*>(p);
+    v[0] = f.x; v[1] = f.y; v[2] = f.z; v[3] = f.w;
+  } else {
+    v[0] = Elem<T>::ld(p);
+  }
+}
+template <typename T, int VEC>
+__device__ __forceinline__ void store_vec(T* p, const float (&v)[VEC]) {
+  if constexpr (VEC == 4 && sizeof(T) == 2) {
+    uint2 raw;
+    raw.x = pack_bf16(v[0], v[1]);
+    raw.y = pack_bf16(v[2], v[3]);
+    *reinterpret_cast<uint2*>(p) = raw;
+  } else if constexpr (VEC == 4) {
+    *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+  } else {
+    Elem<T>::st(p, v[0]);
+  }
+}
+
+constexpr int kRowThreads = 512;
+
+template <typename T, int VEC>
+__global__ void __launch_bounds__(kRowThreads)
+residual_rms_kernel(float* __restrict__ x, const T* __restrict__ y, const float* __restrict__ w, float eps, int width, NextArgs nx) {
+  __shared__ float scratch[32];
+  const size_t row = blockIdx.x;
+  const T* yr = y + row * width;
+  float* xr = x + row * width;
+  float ss = 0.f;
+  for (int c = threadIdx.x * VEC; c < width; c += kRowThreads * VEC) {
+    float v[VEC];
+    load_vec<T, VEC>(yr + c, v);
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) ss = fmaf(v[i], v[i], ss);
+  }
+  const float inv = 1.f / sqrtf(block_sum_all(ss, scratch) / static_cast<float>(width) + eps);
+  for (int c = threadIdx.x * VEC; c < width; c += kRowThreads * VEC) {
+    float v[VEC], wv[VEC], s[VEC];
+    load_vec<T, VEC>(yr + c, v);
+    load_vec<float, VEC>(w + c, wv);
+    load_vec<float, VEC>(xr + c, s);
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) s[i] = fmaf(v[i] * inv, wv[i], s[i]);
+    store_vec<float, VEC>(xr + c, s);
+    if (nx.mode == CACHEIR_B200_NEXT_DYT) {
+      float nw[VEC], nb[VEC];
+      load_vec<float, VEC>(nx.w + c, nw);
+      load_vec<float, VEC>(nx.b + c, nb);
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) s[i] = fmaf(tanhf(nx.alpha * s[i]), nw[i], nb[i]);
+    }
+    if (nx.mode != CACHEIR_B200_NEXT_NONE) store_vec<T, VEC>(static_cast<T*>(nx.out) + row * width + c, s);
+  }
+}
+
+template <typename T, int VEC>
+__global__ void __launch_bounds__(kRowThreads)
+gated_rms_kernel(const T* __restrict__ o, const T* __restrict__ gate, long long gate_stride, const float* __restrict__ w, float eps,
+                 T* __restrict__ out, int cols) {
+  __shared__ float scratch[32];
+  const size_t row = blockIdx.x;
+  const T* orow = o + row * cols;
+  const T* grow = gate + row * gate_stride;
+  float ss = 0.f;
+  for (int c = threadIdx.x * VEC; c < cols; c += kRowThreads * VEC) {
+    float v[VEC];
+    load_vec<T, VEC>(orow + c, v);
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) ss = fmaf(v[i], v[i], ss);
+  }
+  const float inv = 1.f / sqrtf(block_sum_all(ss, scratch) / static_cast<float>(cols) + eps);
+  for (int c = threadIdx.x * VEC; c < cols; c += kRowThreads * VEC) {
+    float v[VEC], wv[VEC], g[VEC];
+    load_vec<T, VEC>(orow + c, v);
+    load_vec<T, VEC>(grow + c, g);
+    load_vec<float, VEC>(w + c, wv);
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) v[i] = v[i] * inv * wv[i] * sigmoid_exact(g[i]);
+    store_vec<T, VEC>(out + row * cols + c, v);
+  }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(256)
+geglu_pairs_kernel(const T* __restrict__ y, T* __restrict__ out, int ff) {
+  const size_t row = blockIdx.x;
+  for (int c = blockIdx.y * 256 + threadIdx.x; c < ff; c += gridDim.y * 256) {
+    const T* p = y + row * 2 * ff + 2 * c;
+    Elem<T>::st(out + row * ff + c, gelu_tanh(Elem<T>::ld(p)) * Elem<T>::ld(p + 1));
+  }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(256)
+gelu_embed_kernel(const T* __restrict__ g, const int64_t* __restrict__ ids, const T* __restrict__ table, long long table_stride,
+                  int table_col, T* __restrict__ out, int dim, int vocab) {
+  const size_t row = blockIdx.x;
+  const int64_t id = min(max(ids[row], static_cast<int64_t>(0)), static_cast<int64_t>(vocab - 1));
+  for (int c = threadIdx.x; c < dim; c += 256)
+    Elem<T>::st(out + row * dim + c, gelu_tanh(Elem<T>::ld(g + row * dim + c)) * Elem<T>::ld(table + id * table_stride + table_col + c));
+}
+
+template <typename T>
+__global__ void __launch_bounds__(256)
+silu_cols_kernel(T* __restrict__ y, long long stride, int cols) {
+  T* yr = y + static_cast<size_t>(blockIdx.x) * stride;
+  for (int c = blockIdx.y * 256 + threadIdx.x; c < cols; c += gridDim.y * 256) Elem<T>::st(yr + c, silu_exact(Elem<T>::ld(yr + c)));
+}
+
+// ---- plain tiled GEMM, float32 arithmetic: 64 tokens x 64 columns per CTA, 16 k at a time ---------------------------
+constexpr int kTile = 64, kTileK = 16;
+template <typename T, typename TY>
+__global__ void __launch_bounds__(256)
+dense_simple_kernel(const T* __restrict__ x, const T* __restrict__ w, TY* __restrict__ y, int rows, int N, int K, int w_batch_rows,
+                    int x_batch_cols, int y_batch_cols, long long ws, long long xs, long long ys) {
+  __shared__ float sx[kTileK][kTile + 4], sw[kTileK][kTile + 4];
+  const int z = blockIdx.z;
+  x += static_cast<long long>(z) * x_batch_cols;
+  w += static_cast<long long>(z) * w_batch_rows * ws;
+  y += static_cast<long long>(z) * y_batch_cols;
+  const int t0 = blockIdx.y * kTile, n0 = blockIdx.x * kTile;
+  const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
+  float acc[4][4] = {};
+  for (int k0 = 0; k0 < K; k0 += kTileK) {
+    for (int i = threadIdx.x; i < kTile * kTileK; i += 256) {
+      const int r = i / kTileK, k = i % kTileK;
+      sx[k][r] = (t0 + r < rows && k0 + k < K) ? Elem<T>::ld(x + (t0 + r) * xs + k0 + k) : 0.f;
+      sw[k][r] = (n0 + r < N && k0 + k < K) ? Elem<T>::ld(w + (n0 + r) * ws + k0 + k) : 0.f;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int k = 0; k < kTileK; ++k) {
+      float a[4], b[4];
+#pragma unroll
+      for (int i = 0; i < 4; ++i) { a[i] = sx[k][ty * 4 + i]; b[i] = sw[k][tx * 4 + i]; }
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(a[i], b[j], acc[i][j]);
+    }
+    __syncthreads();
+  }
+#pragma unroll
+  for (int i = 0; i < 4; ++i)
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const int t = t0 + ty * 4 + i, n = n0 + tx * 4 + j;
+      if (t < rows && n < N) Elem<TY>::st(y + t * ys + n, acc[i][j]);
+    }
+}
+
+// grid.y so that a small batch still spreads over the SMs
+inline dim3 row_grid(int rows, int cols) {
+  int y = 1;
+  while (rows * y < kNumSMs * 2 && y * 256 < cols) ++y;
+  return dim3(rows, y);
+}
+bool next_ok(int mode, const float* w, const float* b, const void* out) {
+  if (mode == CACHEIR_B200_NEXT_NONE) return true;
+  if (mode == CACHEIR_B200_NEXT_COPY) return out != nullptr;
+  return mode == CACHEIR_B200_NEXT_DYT && w && b && out;
+}
+
+}  // namespace
+}  // namespace cb200
+
+using namespace cb200;
+
+#define CB200_HYBRID_DTYPE(dtype, ...)                                                  \
+  switch (dtype) {                                                                      \
+    case CACHEIR_B200_F32: { using T = float; __VA_ARGS__; break; }                     \
+    case CACHEIR_B200_BF16: { using T = __nv_bfloat16; __VA_ARGS__; break; }            \
+    default: return CACHEIR_B200_EUNSUPPORTED;                                          \
+  }
+
+extern "C" int cacheir_b200_scaled_embedding(const void* table, const int64_t* ids, float* residual, int rows, int width, int vocab,
+                                             float scale, int next_mode, const float* next_w, const float* next_b, float next_alpha,
+                                             void* next_out, int dtype, void* stream) {
+  if (rows <= 0 || width <= 0) return 0;
+  if (!table || !ids || !residual || vocab <= 0 || !next_ok(next_mode, next_w, next_b, next_out)) return CACHEIR_B200_EINVAL;
+  const NextArgs nx{next_mode, next_w, next_b, next_alpha, next_out};
+  CB200_HYBRID_DTYPE(dtype, (scaled_embedding_kernel<T><<<row_grid(rows, width), 256, 0, as_stream(stream)>>>(
+                                static_cast<const T*>(table), ids, residual, width, vocab, scale, nx)));
+  return launch_status();
+}
+
+extern "C" int cacheir_b200_dyt_rows(const float* residual, const int32_t* row_index, const float* w, const float* b, float alpha,
+                                     void* out, int rows, int width, int dtype, void* stream) {
+  if (rows <= 0 || width <= 0) return 0;
+  if (!residual || !w || !b || !out) return CACHEIR_B200_EINVAL;
+  CB200_HYBRID_DTYPE(dtype, (dyt_rows_kernel<T><<<row_grid(rows, width), 256, 0, as_stream(stream)>>>(
+                                residual, row_index, w, b, alpha, static_cast<T*>(out), width)));
+  return launch_status();
+}
+
+extern "C" int cacheir_b200_residual_dyt(float* residual, const void* y, const float* w, const float* b, float alpha, int rows,
+                                         int width, int next_mode, const float* next_w, const float* next_b, float next_alpha,
+                                         void* next_out, int dtype, void* stream) {
+  if (rows <= 0 || width <= 0) return 0;
+  if (!residual || !y || !w || !b || !next_ok(next_mode, next_w, next_b, next_out)) return CACHEIR_B200_EINVAL;
+  const NextArgs nx{next_mode, next_w, next_b, next_alpha, next_out};
+  CB200_HYBRID_DTYPE(dtype, (residual_dyt_kernel<T><<<row_grid(rows, width), 256, 0, as_stream(stream)>>>(
+                                residual, static_cast<const T*>(y), w, b, alpha, width, nx)));
+  return launch_status();
+}
+
+extern "C" int cacheir_b200_residual_rms(float* residual, const void* y, const float* w, float eps, int rows, int width,
+                                         int next_mode, const float* next_w, const float* next_b, float next_alpha, void* next_out,
+                                         int dtype, void* stream) {
+  if (rows <= 0 || width <= 0) return 0;
+  if (!residual || !y || !w || !next_ok(next_mode, next_w, next_b, next_out)) return CACHEIR_B200_EINVAL;
+  const NextArgs nx{next_mode, next_w, next_b, next_alpha, next_out};
+  const bool vec = width % 4 == 0 && aligned_to(residual, 16) && aligned_to(y, 16) && aligned_to(w, 16) &&
+                   (next_mode == CACHEIR_B200_NEXT_NONE || aligned_to(next_out, 16)) &&
+                   (next_mode != CACHEIR_B200_NEXT_DYT || (aligned_to(next_w, 16) && aligned_to(next_b, 16)));
+  CB200_HYBRID_DTYPE(dtype, {
+    if (vec) residual_rms_kernel<T, 4><<<rows, kRowThreads, 0, as_stream(stream)>>>(residual, static_cast<const T*>(y), w, eps, width, nx);
+    else residual_rms_kernel<T, 1><<<rows, kRowThreads, 0, as_stream(stream)>>>(residual, static_cast<const T*>(y), w, eps, width, nx);
+  });
+  return launch_status();
+}
+
+extern "C" int cacheir_b200_gated_rms(const void* o, const void* gate, long long gate_stride, const float* w, float eps, void* out,
+                                      int rows, int cols, int dtype, void* stream) {
+  if (rows <= 0 || cols <= 0) return 0;
+  if (!o || !gate || !w || !out) return CACHEIR_B200_EINVAL;
+  const bool vec = cols % 4 == 0 && gate_stride % 4 == 0 && aligned_to(o, 16) && aligned_to(gate, 16) && aligned_to(w, 16) && aligned_to(out, 16);
+  CB200_HYBRID_DTYPE(dtype, {
+    if (vec) gated_rms_kernel<T, 4><<<rows, kRowThreads, 0, as_stream(stream)>>>(
+        static_cast<const T*>(o), static_cast<const T*>(gate), gate_stride, w, eps, static_cast<T*>(out), cols);
+    else gated_rms_kernel<T, 1><<<rows, kRowThreads, 0, as_stream(stream)>>>(
+        static_cast<const T*>(o), static_cast<const T*>(gate), gate_stride, w, eps, static_cast<T*>(out), cols);
+  });
+  return launch_status();
+}
+
+extern "C" int cacheir_b200_geglu_pairs(const void* y, void* out, int rows, int ff, int dtype, void* stream) {
+  if (rows <= 0 || ff <= 0) return 0;
+  if (!y || !out) return CACHEIR_B200_EINVAL;
+  CB200_HYBRID_DTYPE(dtype, (geglu_pairs_kernel<T><<<row_grid(rows, ff), 256, 0, as_stream(stream)>>>(
+                                static_cast<const T*>(y), static_cast<T*>(out), ff)));
+  return launch_status();
+}
+
+extern "C" int cacheir_b200_gelu_embed(const void* g, const int64_t* ids, const void* table, long long table_stride, int table_col,
+                                       void* out, int rows, int dim, int vocab, int dtype, void* stream) {
+  if (rows <= 0 || dim <= 0) return 0;
+  if (!g || !ids || !table || !out || vocab <= 0) return CACHEIR_B200_EINVAL;
+  CB200_HYBRID_DTYPE(dtype, (gelu_embed_kernel<T><<<rows, 256, 0, as_stream(stream)>>>(
+                                static_cast<const T*>(g), ids, static_cast<const T*>(table), table_stride, table_col,
+                                static_cast<T*>(out), dim, vocab)));
+  return launch_status();
+}
+
+extern "C" int cacheir_b200_silu_cols(void* y, int rows, long long stride, int cols, int dtype, void* stream) {
+  if (rows <= 0 || cols <= 0) return 0;
+  if (!y) return CACHEIR_B200_EINVAL;
+  CB200_HYBRID_DTYPE(dtype, (silu_cols_kernel<T><<<row_grid(rows, cols), 256, 0, as_stream(stream)>>>(static_cast<T*>(y), stride, cols)));
+  return launch_status();
+}
+
+extern "C" int cacheir_b200_dense_simple(const void* x, const void* w, void* y, int rows, int N, int K, int batch, int w_batch_rows,
+                                         int x_batch_cols, int y_batch_cols, long long w_stride, long long x_stride,
+                                         long long y_stride, int dtype, int y_dtype, void* stream) {
+  if (rows <= 0 || N <= 0) return 0;
+  if (K <= 0 || !x || !w || !y || batch < 1) return CACHEIR_B200_EINVAL;
+  const dim3 grid((N + kTile - 1) / kTile, (rows + kTile - 1) / kTile, batch);
+  if (grid.y > 65535 || grid.z > 65535) return CACHEIR_B200_ELIMIT;
+  cudaStream_t st = as_stream(stream);
+#define CB200_SIMPLE(T, TY)                                                                                              \
+  dense_simple_kernel<T, TY><<<grid, 256, 0, st>>>(static_cast<const T*>(x), static_cast<const T*>(w), static_cast<TY*>(y), rows, N, \
+                                                   K, w_batch_rows, x_batch_cols, y_batch_cols, w_stride, x_stride, y_stride)
+  if (dtype == CACHEIR_B200_F32 && y_dtype == CACHEIR_B200_F32) CB200_SIMPLE(float, float);
+  else if (dtype == CACHEIR_B200_BF16 && y_dtype == CACHEIR_B200_F32) CB200_SIMPLE(__nv_bfloat16, float);
+  else if (dtype == CACHEIR_B200_BF16 && y_dtype == CACHEIR_B200_BF16) CB200_SIMPLE(__nv_bfloat16, __nv_bfloat16);
+  else return CACHEIR_B200_EUNSUPPORTED;
+#undef CB200_SIMPLE
+  return launch_status();
+}
+
+namespace cb200 {
+int dense_gemm_device_status(bool reset);
+int latent_attention_device_status(bool reset);
+}
+
+extern "C" int cacheir_b200_hybrid_device_status(int reset) {
+  const int gemm = dense_gemm_device_status(reset != 0);
+  const int attn = latent_attention_device_status(reset != 0);
+  return gemm != 0 ? gemm : attn;
+}

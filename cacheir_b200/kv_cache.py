@@ -54,7 +54,7 @@ class B200KVPageAllocator:
     _owner_counter = itertools.count(1)
 
     def __init__(self, *, page_size: int = 16, initial_slots: int = 64, max_slots: int | None = None,
-                 max_resident_pages: int | None = None):
+                 max_resident_pages: int | None = None, initial_states: int = 16, max_states: int | None = None):
         self.page_size = max(1, int(page_size))
         self.capacity = max(1, int(initial_slots))
         self.max_slots = max_slots
@@ -72,7 +72,16 @@ class B200KVPageAllocator:
         self.version = 0             # bumps whenever a page changes hands (allocate, retain, release)
         self.page_bytes: int | None = None
         self._pools: dict[int, dict[str, Any]] = {}
-        self._pool_spec: tuple[Any, Any, int, int] | None = None  # device, dtype, kv_heads, head_dim
+        self._pool_spec: tuple | None = None
+        self._pool_shapes: dict[int, dict[str, tuple[tuple[int, ...], Any]]] = {}   # layer -> tensor name -> (shape of a slot, dtype)
+        # recurrent state: one slot per live sequence, the same slot in every recurrent layer
+        self.state_capacity = max(1, int(initial_states) if max_states is None else min(int(initial_states), int(max_states)))
+        self.max_states = max_states
+        self._state_shapes: dict[int, tuple[int, ...]] = {}
+        self._states: dict[int, Any] = {}
+        self._free_states: list[int] = []
+        self._next_state = 0
+        self.state_owners: dict[int, str] = {}
 
     # ---- ids / refcounts ---------------------------------------------------------
     def new_owner(self) -> str:
@@ -118,6 +127,54 @@ class B200KVPageAllocator:
     def slots_in_use(self) -> int:
         return len(self._refcount)
 
+    def free_slots(self) -> int | None:
+        """Pages that can still be handed out (None: the pool may grow without bound)."""
+        return None if self.max_slots is None else self.max_slots - self.slots_in_use
+
+    # ---- recurrent state slots -----------------------------------------------------
+    @property
+    def has_state(self) -> bool:
+        return bool(self._state_shapes)
+
+    def free_states(self) -> int | None:
+        return None if self.max_states is None else self.max_states - len(self.state_owners)
+
+    def acquire_state(self, owner: str) -> int:
+        """A state slot for one sequence. Its contents are whatever the last owner left: the recurrence kernels start
+        from zero at position 0, so nothing is cleared here."""
+        if self._free_states:
+            slot = self._free_states.pop()
+        else:
+            slot = self._next_state
+            if self.max_states is not None and slot >= self.max_states:
+                raise KVPoolExhausted(f"recurrent state slots exhausted ({self.max_states})")
+            self._next_state += 1
+            if self._next_state > self.state_capacity:
+                self._grow_states(self._next_state)
+        self.state_owners[slot] = owner
+        self.version += 1
+        return slot
+
+    def release_state(self, slot: int) -> None:
+        del self.state_owners[slot]
+        self._free_states.append(slot)
+        self.version += 1
+
+    def state_for_layer(self, layer: int) -> Any | None:
+        return self._states.get(int(layer))
+
+    def _grow_states(self, needed: int) -> None:
+        new = max(needed, self.state_capacity * 2)
+        if self.max_states is not None:
+            new = max(needed, min(new, self.max_states))
+        old, self.state_capacity = self.state_capacity, new
+        for layer, state in list(self._states.items()):
+            grown = self._torch.zeros((new,) + self._state_shapes[layer], device=self._device, dtype=self._torch.float32)
+            grown[:old] = state
+            self._states[layer] = grown
+        if self._states:
+            self.generation += 1
+
     # ---- pools ---------------------------------------------------------------------
     def configure(self, *, torch: Any, device: Any, dtype: Any, num_layers: int, kv_heads: int, head_dim: int,
                   kv_dtype: str = "same") -> None:
@@ -128,31 +185,40 @@ class B200KVPageAllocator:
         self.kv_dtype = kv_dtype
         if kv_dtype == "int8":
             dtype = torch.uint8
-        spec = (str(device), str(dtype), int(kv_heads), int(head_dim))
+        row = (int(kv_heads), self.page_size, int(head_dim))
+        tensors = {"keys": (row, dtype), "values": (row, dtype)}
+        if kv_dtype == "int8":
+            tensors["scales"] = ((int(kv_heads), 2, self.page_size), torch.float16)
+        self.configure_layout(torch=torch, device=device, pools={layer: tensors for layer in range(num_layers)})
+
+    def configure_layout(self, *, torch: Any, device: Any, pools: dict[int, dict[str, tuple[tuple[int, ...], Any]]],
+                         states: dict[int, tuple[int, ...]] | None = None) -> None:
+        """Create the storage: per layer the named pool tensors (shape of one page slot, dtype) and, for recurrent
+        layers, a float32 state of the given shape per state slot."""
+        spec = (str(device), {layer: dict(t) for layer, t in pools.items()}, dict(states or {}))
         if self._pool_spec is not None:
-            if self._pool_spec[:4] != spec or len(self._pools) != num_layers:
+            if self._pool_spec != spec:
                 raise ValueError("a KV page allocator serves one model shape, dtype and device")
             return
         self._pool_spec = spec
-        self._torch, self._device, self._dtype = torch, device, dtype
-        self._kv_heads, self._head_dim = int(kv_heads), int(head_dim)
-        for layer in range(num_layers):
-            self._pools[layer] = self._new_pool(self.capacity)
+        self._torch, self._device = torch, device
+        self._pool_shapes = spec[1]
+        self._state_shapes = {layer: tuple(int(n) for n in shape) for layer, shape in spec[2].items()}
+        for layer in self._pool_shapes:
+            self._pools[layer] = self._new_pool(layer, self.capacity)
+        for layer, shape in self._state_shapes.items():
+            self._states[layer] = torch.zeros((self.state_capacity,) + shape, device=device, dtype=torch.float32)
         self.pool_grows += 1
         self.generation += 1
-        elem = torch.empty((), dtype=dtype).element_size()
-        self.page_bytes = 2 * self._kv_heads * self.page_size * self._head_dim * elem
-        if kv_dtype == "int8":
-            self.page_bytes += 2 * self._kv_heads * self.page_size * 2
+        largest = 0                                   # bytes of one page in one layer (the largest layer)
+        for tensors in self._pool_shapes.values():
+            largest = max(largest, sum(int(np.prod(shape)) * torch.empty((), dtype=dtype).element_size()
+                                       for shape, dtype in tensors.values()))
+        self.page_bytes = largest
 
-    def _new_pool(self, slots: int) -> dict[str, Any]:
-        shape = (slots, self._kv_heads, self.page_size, self._head_dim)
-        pool = {"keys": self._torch.zeros(shape, device=self._device, dtype=self._dtype),
-                "values": self._torch.zeros(shape, device=self._device, dtype=self._dtype)}
-        if getattr(self, "kv_dtype", "same") == "int8":
-            pool["scales"] = self._torch.zeros((slots, self._kv_heads, 2, self.page_size), device=self._device,
-                                               dtype=self._torch.float16)
-        return pool
+    def _new_pool(self, layer: int, slots: int) -> dict[str, Any]:
+        return {name: self._torch.zeros((slots,) + tuple(shape), device=self._device, dtype=dtype)
+                for name, (shape, dtype) in self._pool_shapes[layer].items()}
 
     def reserve_slots(self, slots: int) -> None:
         """Pre-size the pools so that no growth (and no pointer change) happens later."""
@@ -168,7 +234,7 @@ class B200KVPageAllocator:
         if not self._pools:
             return
         for layer, pool in self._pools.items():
-            grown = self._new_pool(new_capacity)
+            grown = self._new_pool(layer, new_capacity)
             for name in pool:
                 grown[name][:old] = pool[name]
             self._pools[layer] = grown
@@ -181,6 +247,12 @@ class B200KVPageAllocator:
     def stats(self) -> dict[str, object]:
         pools = []
         for layer, pool in sorted(self._pools.items()):
+            if "keys" not in pool:
+                first = next(iter(pool.values()))
+                pools.append({"layer": layer, "device": str(first.device), "dtype": str(first.dtype), "slots": self._next_slot,
+                              "capacity": int(first.shape[0]),
+                              "bytes": int(sum(t.numel() * t.element_size() for t in pool.values()))})
+                continue
             keys = pool["keys"]
             pools.append({
                 "layer": layer, "device": str(keys.device), "dtype": str(keys.dtype),
@@ -200,6 +272,8 @@ class B200KVPageAllocator:
             "pool_writes": self.pool_writes,
             "pool_grows": self.pool_grows,
             "persistent_pools": pools,
+            **({"state_slots": self.state_capacity, "states_in_use": len(self.state_owners),
+                "state_bytes": int(sum(t.numel() * 4 for t in self._states.values()))} if self._state_shapes else {}),
         }
 
 
@@ -213,6 +287,7 @@ class B200PagedKVCache:
     tokens: int = 0
     owner_id: str = ""
     epoch: int = 0          # bumps when the page list is replaced rather than extended
+    state_slot: int | None = None
 
     def __post_init__(self) -> None:
         self.page_size = self.allocator.page_size
@@ -221,6 +296,9 @@ class B200PagedKVCache:
 
     def clear(self) -> None:
         self.allocator.release_owner(self.owner_id)
+        if self.state_slot is not None:
+            self.allocator.release_state(self.state_slot)
+            self.state_slot = None
         self.pages = []
         self.tokens = 0
         self.epoch += 1
@@ -243,6 +321,8 @@ class B200PagedKVCache:
             self.tokens += 1
             self.allocator.pool_writes += self.num_layers
             return False
+        if self.state_slot is None and self.allocator.has_state and length > 0:
+            self.state_slot = self.allocator.acquire_state(self.owner_id)
         opened = False
         remaining = int(length)
         cursor = self.tokens
@@ -262,11 +342,17 @@ class B200PagedKVCache:
         self.allocator.pool_writes += int(length) * self.num_layers
         return opened
 
+    def pages_needed(self, length: int) -> int:
+        """New pages that `length` more tokens would open."""
+        return (self.tokens + int(length) + self.page_size - 1) // self.page_size - len(self.pages)
+
     def share_prefix(self, other: "B200PagedKVCache", tokens: int) -> int:
         """Alias the full pages covering the first `tokens` tokens of `other`
         (rounded down to whole pages). Returns the number of tokens shared."""
         if self.tokens != 0:
             raise RuntimeError("share_prefix needs an empty session")
+        if self.allocator.has_state:
+            raise RuntimeError("a recurrent state is a summary of its whole prefix: pages alone cannot be shared")
         n_pages = min(int(tokens), other.tokens) // self.page_size
         for page in other.pages[:n_pages]:
             self.pages.append(self.allocator.retain(owner=self.owner_id, page=page))

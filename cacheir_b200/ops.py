@@ -428,14 +428,14 @@ def argmax_rows(logits: torch.Tensor, out: torch.Tensor | None = None) -> torch.
     if not logits.is_contiguous():
         raise ValueError("argmax_rows expects contiguous logits")
     out = torch.empty((rows,), device=logits.device, dtype=torch.int64) if out is None else out
-    check(_lib.load().cacheir_b200_argmax_rows(logits.data_ptr(), out.data_ptr(), rows, vocab, dtype_code(logits.dtype),
+    check(_lib.load_shared().cacheir_b200_argmax_rows(logits.data_ptr(), out.data_ptr(), rows, vocab, dtype_code(logits.dtype),
                                                _stream()), "argmax_rows")
     return out
 
 
 def advance_positions(positions: torch.Tensor, seq_lens: torch.Tensor) -> None:
     _require_cuda(positions, seq_lens)
-    check(_lib.load().cacheir_b200_advance_positions(positions.data_ptr(), seq_lens.data_ptr(), seq_lens.numel(),
+    check(_lib.load_shared().cacheir_b200_advance_positions(positions.data_ptr(), seq_lens.data_ptr(), seq_lens.numel(),
                                                      _stream()), "advance_positions")
 
 

@@ -1,0 +1,343 @@
+"""Ragged steps: portions of prompts beside single decoded tokens as one pass through a lowered graph.
+
+`RaggedPlan` is the plan class of families whose layers need to know which rows belong to one sequence (linear
+recurrences, windowed attention over tiles of neighbouring tokens). It keeps `_DecodePlan`'s contract (static buffers,
+a flat launch list, CUDA-graph replay from the second step) and adds the segment arrays. A decode plan has one row per
+sequence and advances on the device; a portion plan has room for `rows` rows of `segments` sequences and takes its
+metadata in one copy per step. Residual stream float32; in bfloat16 runs each sublayer boundary (norm, residual add,
+next norm) is the epilogue of the GEMM in front of it.
+"""
+from __future__ import annotations
+
+from typing import Any, Callable
+
+import numpy as np
+import torch
+
+from . import hybrid_ops as H
+from . import ops
+
+# rows a portion plan is made for: one plan (and one CUDA graph) per bucket, not per portion length
+ROW_BUCKETS = (1, 2, 4, 8, 16, 32, 64, 128, 192, 256, 384, 512, 768, 1024, 1536, 2048, 3072, 4096)
+
+
+def bucket(n: int) -> int:
+    for b in ROW_BUCKETS:
+        if n <= b:
+            return b
+    return (n + 1023) // 1024 * 1024
+
+
+def rotate_half_table(positions: int, dims: int, base: float) -> np.ndarray:
+    """float32 [positions, dims/2, 2] (cos, sin) of p * base^(-2i/dims), evaluated in double precision."""
+    freq = float(base) ** (-2.0 * np.arange(dims // 2, dtype=np.float64) / dims)
+    angle = np.arange(positions, dtype=np.float64)[:, None] * freq[None, :]
+    return np.stack([np.cos(angle), np.sin(angle)], axis=-1).astype(np.float32)
+
+
+def make_plan_class(base: type) -> type:
+    """`RaggedPlan` over the runtime's plan class (the runtime module imports this one)."""
+
+    class RaggedPlan(base):
+        def __init__(self, engine: Any, rows: int, width: int, *, segments: int | None = None, logit_rows: int | None = None):
+            self.engine = engine
+            self.decode = segments is None
+            self.batch = rows
+            self.segments = rows if segments is None else segments
+            self.width = width
+            self.logit_rows = rows if logit_rows is None else logit_rows
+            self.pool_generation = engine.allocator.generation
+            dev = engine.device
+            # int32 metadata in one block, so that a portion step needs one copy
+            parts = {"lens": rows, "row_seg": rows, "cu_rows": self.segments + 1, "slots": self.segments, "logit_index": self.logit_rows,
+                     "table": self.segments * width}
+            offsets = np.cumsum([0] + [(n + 3) // 4 * 4 for n in parts.values()])
+            self._host_meta = torch.zeros((int(offsets[-1]),), dtype=torch.int32).pin_memory()
+            self._meta = torch.zeros((int(offsets[-1]),), device=dev, dtype=torch.int32)
+            device, host = {}, {}
+            for (name, n), off in zip(parts.items(), offsets):
+                device[name], host[name] = self._meta[off:off + n], self._host_meta[off:off + n]
+            self.seq_lens, self.host_lens = device["lens"], host["lens"]
+            self.page_table, self.host_table = device["table"].view(self.segments, width), host["table"].view(self.segments, width)
+            self._host = host
+            self._device_slots = device["slots"]
+            self.logit_index = None if self.decode else device["logit_index"]
+            self.ids = torch.zeros((rows,), device=dev, dtype=torch.int64)
+            self.host_ids = torch.zeros((rows,), dtype=torch.int64).pin_memory()
+            self.positions = torch.zeros((rows,), device=dev, dtype=torch.int32)
+            if self.decode:
+                device["row_seg"].copy_(torch.arange(rows, dtype=torch.int32))
+                device["cu_rows"].copy_(torch.arange(rows + 1, dtype=torch.int32))
+            else:
+                device["row_seg"].fill_(-1)
+            self.rows = H.Rows(positions=self.positions, row_seg=device["row_seg"], cu_rows=device["cu_rows"], page_table=self.page_table,
+                               slots=device["slots"], decode=self.decode)
+            self.synced_owner_state = None
+            self.repeat_key: tuple | None = None
+            self.repeat_tokens: list[int] = []
+            self.repeat_left = 0
+            self.repeat_version = -1
+            self.program: list[Callable[[], None]] = []
+            self.launches_per_step = 0
+            self.cuda_graph = None
+            self.feedback_graph = None
+            self.h2d_done = torch.cuda.Event()
+            self.steps_run = 0
+            self.logits: torch.Tensor | None = None
+            self._lower()
+
+        # -- metadata ----------------------------------------------------------------------
+        def sync_sessions(self, sessions: list[Any]) -> None:
+            before = self.synced_owner_state
+            super().sync_sessions(sessions)
+            if before is None or [(s[0], s[3]) for s in before] != [(s[0], s[3]) for s in self.synced_owner_state]:
+                slots = self._host["slots"]
+                slots.numpy()[:] = [s.kv_cache.state_slot or 0 for s in sessions]
+                self._device_slots.copy_(slots, non_blocking=True)
+
+        def sync_portions(self, portions: list[tuple[Any, int, list[int]]], wanted_rows: list[int]) -> None:
+            """Rows of this step: `portions` = (cache, first position, tokens) per sequence, pages reserved; `wanted_rows`
+            are the rows whose logits the head computes. What is beyond them is padding."""
+            self.h2d_done.synchronize()          # the pinned staging buffers must not change under a pending copy
+            host = {k: v.numpy() for k, v in self._host.items()}
+            ids, table = self.host_ids.numpy(), self.host_table.numpy()
+            host["lens"][:] = 0
+            host["row_seg"][:] = -1
+            ids[:] = 0
+            row = 0
+            for seg, (cache, start, tokens) in enumerate(portions):
+                n = len(tokens)
+                ids[row:row + n] = tokens
+                host["lens"][row:row + n] = np.arange(start, start + n)
+                host["row_seg"][row:row + n] = seg
+                host["cu_rows"][seg] = row
+                host["slots"][seg] = cache.state_slot or 0
+                table[seg] = cache.page_table_row(self.width)
+                row += n
+            host["cu_rows"][len(portions):] = row
+            host["logit_index"][:] = 0
+            host["logit_index"][:len(wanted_rows)] = wanted_rows
+            self.ids.copy_(self.host_ids, non_blocking=True)
+            self._meta.copy_(self._host_meta, non_blocking=True)
+            self.h2d_done.record()
+
+        # -- lowering ----------------------------------------------------------------------
+        def _scratch(self, role: str, cols: int, dtype: torch.dtype | None = None, rows: int | None = None) -> torch.Tensor:
+            """A [rows, cols] buffer from the engine's storage for `role`: plans run one after the other on one stream, and
+            within a step a role is rewritten layer by layer."""
+            dtype = self.engine.dtype if dtype is None else dtype
+            rows = self.batch if rows is None else rows
+            flat = self.engine.scratch(role, rows * cols * torch.empty((), dtype=dtype).element_size())
+            return flat.view(dtype)[:rows * cols].view(rows, cols)
+
+        def _dyt(self, names: list[str]) -> H.DynamicTanh:
+            w = self.engine.weights
+            return H.DynamicTanh(w.get_f32(names[0]), w.get_f32(names[1]), float(w.get_f32(names[2]).item()))
+
+        def _next_after(self, idx: int) -> tuple[H.Next | None, str | None]:
+            """What the kernel finishing the residual at node `idx` can leave for the node behind it."""
+            nxt = self._nodes[idx + 1]
+            width = int(self.engine.config.hidden_size)
+            if nxt.op == "dynamic_tanh" and nxt.attrs.get("rows") != "logits" and nxt.inputs[0] == self._nodes[idx].outputs[0]:
+                out = self._scratch("normed", width)
+                return H.Next(out, self._dyt(nxt.inputs[1:4])), nxt.outputs[0]
+            if nxt.op == "token_side_gate" and nxt.inputs[0] == self._nodes[idx].outputs[0]:
+                return H.Next(self._scratch("copied", width)), None
+            return None, None
+
+        def _finish_residual(self, idx: int, emit: Callable[[H.Next | None], None]) -> None:
+            """Emit the kernel that updates the residual at node `idx` and record its outputs."""
+            nx, normed = self._next_after(idx)
+            emit(nx)
+            node = self._nodes[idx]
+            self._env[node.outputs[0]] = self._residual
+            if normed is not None:
+                self._env[normed] = nx.out
+                self._skip.add(idx + 1)
+            elif nx is not None:
+                self._env["copy:" + node.outputs[0]] = nx.out
+
+        def _lower(self) -> None:
+            eng = self.engine
+            self._nodes = list(eng.graph.nodes)
+            self._env: dict[str, Any] = {}
+            self._skip: set[int] = set()
+            self._count_keys: list[tuple[str, int]] = []
+            self._count_totals = None
+            self._residual = self._scratch("residual", int(eng.config.hidden_size), torch.float32)
+            self._emit(lambda: ops.advance_positions(self.positions, self.seq_lens), "b200.advance_positions")
+            for idx, node in enumerate(self._nodes):
+                if idx in self._skip:
+                    continue
+                lower = getattr(self, "_lower_" + node.op, None)
+                if lower is None:
+                    raise NotImplementedError(f"ragged plans do not implement op {node.op}")
+                lower(idx, node)
+            logits = self._env[eng.graph.outputs[0]]
+            self.logits = logits
+            self.feedback_tail = lambda: ops.argmax_rows(logits, self.ids)
+
+        def _dense(self, x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, **kwargs: Any) -> None:
+            """Plain product into `out` (float32 for logits): tensor cores where they take it, else CUDA cores."""
+            if H.dense_supported(int(w.shape[1]), w.stride(0), x.stride(0), dtype=x.dtype):
+                epilogue = H.DENSE_F32 if out.dtype == torch.float32 else H.DENSE_PLAIN
+                self._emit(lambda: H.dense_gemm(x, w, out, epilogue=epilogue), "b200.dense_gemm")
+            else:
+                self._emit(lambda: H.dense_simple(x, w, out), "b200.dense_simple")
+
+        def _lower_scaled_token_embedding(self, idx: int, node: Any) -> None:
+            table = self.engine.weights.get_checked(node.inputs[1])
+            scale, x = float(node.attrs["scale"]), self._residual
+            self._finish_residual(idx, lambda nx: self._emit(lambda: H.scaled_embedding(table, self.ids, x, scale, nx), "b200.scaled_embedding"))
+
+        def _lower_dynamic_tanh(self, idx: int, node: Any) -> None:
+            norm = self._dyt(node.inputs[1:4])
+            width = int(self.engine.config.hidden_size)
+            if node.attrs.get("rows") == "logits":
+                out = self._scratch("final", width, rows=self.logit_rows)
+                self._emit(lambda: H.dyt_rows(self._residual, norm, out, self.logit_index), "b200.dyt_rows")
+            else:
+                out = self._scratch("normed", width)
+                self._emit(lambda: H.dyt_rows(self._residual, norm, out), "b200.dyt_rows")
+            self._env[node.outputs[0]] = out
+
+        def _lower_concat_matmul(self, idx: int, node: Any) -> None:
+            eng, x = self.engine, self._env[node.inputs[0]]
+            names = tuple(node.inputs[1:])
+            sizes = [int(eng.graph.weights[n].shape[0]) for n in names]
+            w = eng.concat_weight(names)
+            total = int(w.shape[0])
+            out = self._scratch("projected", (total + 7) // 8 * 8)
+            act = sum(sizes[: int(node.attrs.get("activated", 0))])
+            if H.dense_supported(int(w.shape[1]), w.stride(0), x.stride(0), dtype=x.dtype):
+                epilogue = H.DENSE_SILU if act else H.DENSE_PLAIN
+                self._emit(lambda: H.dense_gemm(x, w, out, epilogue=epilogue, act_cols=act), "b200.dense_gemm" + (".silu" if act else ""))
+            else:
+                self._emit(lambda: H.dense_simple(x, w, out), "b200.dense_simple")
+                if act:
+                    self._emit(lambda: H.silu_cols(out, act), "b200.silu_cols")
+            col = 0
+            for name, n in zip(node.outputs, sizes):
+                self._env[name] = out[:, col:col + n]
+                col += n
+
+        def _lower_latent_attention(self, idx: int, node: Any) -> None:
+            eng, at = self.engine, node.attrs
+            q, gate = self._env[node.inputs[0]], self._env[node.inputs[1]]
+            uk, uv = eng.weights.get_checked(node.inputs[2]), eng.weights.get_checked(node.inputs[3])
+            sink = eng.weights.get_f32(node.inputs[4])
+            down = self._env[node.inputs[5]] if len(node.inputs) > 5 else None
+            down_norm = eng.weights.get_f32(node.inputs[6]) if len(node.inputs) > 6 else None
+            heads, dim, rot, vdim, rank = (int(at[k]) for k in ("heads", "dim", "rot_dim", "vdim", "kv_rank"))
+            pool = eng.allocator.pool_for_layer(int(at["cache_layer"]))["latent"]
+            table = eng.rotate_half_table(int(at["rot_dims"]), float(at["rot_base"]))
+            args = H.latent_args(self.rows, pool, heads=heads, dim=dim, rot_dim=rot, vdim=vdim, kv_rank=rank, window=int(at["window"]),
+                                 scale=float(at["scale"]))
+            out = self._scratch("mixed", heads * vdim)
+            fast = (H.latent_attention_supported(rank, rot, eng.page_size, eng.dtype) and dim % 8 == 0
+                    and H.dense_supported(dim, dim, q.stride(0), dtype=q.dtype, batch=heads, x_batch_cols=dim + rot)
+                    and H.dense_supported(rank, rank, heads * rank, dtype=q.dtype, batch=heads, x_batch_cols=rank))
+            if fast:
+                q_lat = self._scratch("latent_q", heads * (rank + rot))
+                q_rot, head_stride = q_lat[:, rank:], rank + rot
+            else:
+                q_rot, head_stride = q[:, dim:], dim + rot           # turned in place
+            self._emit(lambda: H.latent_prepare(args, q, q_rot, q_rot_head_stride=head_stride, table=table, rot_dims=int(at["rot_dims"]),
+                                                down=down, norm_weight=down_norm, eps=float(at["eps"])), "b200.latent_prepare")
+            if not fast:
+                self._emit(lambda: H.latent_attention_simple(args, q, uk, uv, sink, gate, out), "b200.latent_attention_simple")
+                self._env[node.outputs[0]] = out
+                return
+            # key up-projection absorbed into the queries, attention over latents, value up-projection with the output gate
+            uk_t = eng.absorbed_weight(node.inputs[2], heads, dim, rank)
+            o_lat = self._scratch("latent_o", heads * rank)
+            splits = H.latent_attention_splits(self.batch, heads, int(at["window"]), self.width, eng.page_size) if self.decode else 1
+            ws_bytes = H.latent_attention_workspace_bytes(self.batch, heads, rank, splits)
+            ws = eng.scratch("latent_ws", ws_bytes) if ws_bytes else None
+            self._emit(lambda: H.dense_gemm(q, uk_t, q_lat, batch=heads, x_batch_cols=dim + rot, y_batch_cols=rank + rot), "b200.dense_gemm.heads")
+            self._emit(lambda: H.latent_attention(args, q_lat, sink, o_lat, splits=splits, workspace=ws), "b200.latent_attention",
+                       launches=2 if splits > 1 else 1)
+            self._emit(lambda: H.dense_gemm(o_lat, uv, out, epilogue=H.DENSE_GATED, batch=heads, x_batch_cols=rank, gate=gate),
+                       "b200.dense_gemm.heads_gated")
+            self._env[node.outputs[0]] = out
+
+        def _lower_linear_recurrence(self, idx: int, node: Any) -> None:
+            eng, at = self.engine, node.attrs
+            q, k, v = (self._env[n] for n in node.inputs)
+            heads, dim, vdim = int(at["heads"]), int(at["dim"]), int(at["vdim"])
+            state = eng.allocator.state_for_layer(int(at["layer"]))
+            out = self._scratch("recurrence", heads * vdim)
+            args = H.recurrence_args(self.rows, q, k, v, eng.decay_powers(tuple(at["decay"])), state, out, heads=heads, dim=dim, vdim=vdim)
+            if self.decode and vdim % 4 == 0 and vdim <= 1024:
+                self._emit(lambda: H.recurrence_step(args), "b200.recurrence_step")
+            elif H.recurrence_chunked_supported(dim, vdim, eng.dtype) and q.stride(0) % 8 == 0:
+                need = H.recurrence_workspace_bytes(self.batch, self.segments, heads, dim, vdim)
+                ws = eng.scratch("recurrence_ws", need) if need else None
+                self._emit(lambda: H.recurrence_chunked(args, ws), "b200.recurrence_chunked", launches=3 if need else 1)
+            else:
+                self._emit(lambda: H.recurrence_simple(args), "b200.recurrence_simple")
+            self._env[node.outputs[0]] = out
+
+        def _lower_gated_rms_norm(self, idx: int, node: Any) -> None:
+            o, gate = self._env[node.inputs[0]], self._env[node.inputs[1]]
+            w, eps = self.engine.weights.get_f32(node.inputs[2]), float(node.attrs["eps"])
+            out = self._scratch("mixed", int(o.shape[1]))
+            self._emit(lambda: H.gated_rms(o, gate, w, eps, out), "b200.gated_rms")
+            self._env[node.outputs[0]] = out
+
+        def _lower_matmul(self, idx: int, node: Any) -> None:
+            eng, x = self.engine, self._env[node.inputs[0]]
+            w = eng.weights.get_checked(node.inputs[1])
+            nxt = self._nodes[idx + 1] if idx + 1 < len(self._nodes) else None
+            if (nxt is not None and nxt.op == "residual_dynamic_tanh" and nxt.inputs[1] == node.outputs[0]
+                    and H.dense_supported(int(w.shape[1]), w.stride(0), x.stride(0), dtype=x.dtype)):
+                norm, res = self._dyt(nxt.inputs[2:5]), self._residual
+                self._finish_residual(idx + 1, lambda nx: self._emit(
+                    lambda: H.dense_gemm(x, w, epilogue=H.DENSE_RESIDUAL, residual=res, norm=norm, nx=nx), "b200.dense_gemm.residual_dyt"))
+                self._skip.add(idx + 1)
+                return
+            if nxt is None:
+                out = self._scratch("logits", int(w.shape[0]), torch.float32, rows=self.logit_rows)
+            else:
+                out = self._scratch("sublayer", int(w.shape[0]))
+            self._dense(x, w, out)
+            self._env[node.outputs[0]] = out
+
+        def _lower_residual_dynamic_tanh(self, idx: int, node: Any) -> None:
+            y, norm, res = self._env[node.inputs[1]], self._dyt(node.inputs[2:5]), self._residual
+            self._finish_residual(idx, lambda nx: self._emit(lambda: H.residual_dyt(res, y, norm, nx), "b200.residual_dyt"))
+
+        def _lower_fused_geglu(self, idx: int, node: Any) -> None:
+            eng, x = self.engine, self._env[node.inputs[0]]
+            w = eng.paired_weight(tuple(node.inputs[1:3]))
+            ff = int(w.shape[0]) // 2
+            out = self._scratch("gated", ff)
+            if H.dense_supported(int(w.shape[1]), w.stride(0), x.stride(0), dtype=x.dtype):
+                self._emit(lambda: H.dense_gemm(x, w, out, epilogue=H.DENSE_GEGLU), "b200.dense_gemm.geglu")
+            else:
+                both = self._scratch("gate_up", 2 * ff)
+                self._emit(lambda: H.dense_simple(x, w, both), "b200.dense_simple")
+                self._emit(lambda: H.geglu_pairs(both, out), "b200.geglu_pairs")
+            self._env[node.outputs[0]] = out
+
+        def _lower_token_side_gate(self, idx: int, node: Any) -> None:
+            eng = self.engine
+            x = self._env["copy:" + node.inputs[0]]
+            w, table = eng.weights.get_checked(node.inputs[1]), eng.weights.get_checked(node.inputs[2])
+            dim, col = int(w.shape[0]), int(node.attrs["column"])
+            out = self._scratch("side", dim)
+            if H.dense_supported(int(w.shape[1]), w.stride(0), x.stride(0), dtype=x.dtype):
+                self._emit(lambda: H.dense_gemm(x, w, out, epilogue=H.DENSE_GELU_EMBED, ids=self.ids, table=table, table_col=col),
+                           "b200.dense_gemm.gelu_embed")
+            else:
+                g = self._scratch("side_gate", dim)
+                self._emit(lambda: H.dense_simple(x, w, g), "b200.dense_simple")
+                self._emit(lambda: H.gelu_embed(g, self.ids, table, col, out), "b200.gelu_embed")
+            self._env[node.outputs[0]] = out
+
+        def _lower_residual_rms_norm(self, idx: int, node: Any) -> None:
+            y, res = self._env[node.inputs[1]], self._residual
+            w, eps = self.engine.weights.get_f32(node.inputs[2]), float(node.attrs["eps"])
+            self._finish_residual(idx, lambda nx: self._emit(lambda: H.residual_rms(res, y, w, eps, nx), "b200.residual_rms"))
+
+    return RaggedPlan

@@ -31,10 +31,11 @@ from typing import Any, Callable, Iterable
 import numpy as np
 import torch
 
-from . import ops
+from . import hybrid_ops, ops
 from .artifact import CompileArtifact
 from .kv_cache import B200KVPageAllocator, B200PagedKVCache, KVPoolExhausted
 from .quantization import B200PackedWeight, concat_rows, quant_bits, to_tiled
+from .ragged import bucket, make_plan_class, rotate_half_table
 from .tensor_parallel import PeerCollectives, TensorParallel, shard_columns, shard_rows
 from .weights import B200WeightStore, TensorSource
 
@@ -87,6 +88,8 @@ class B200PrefixCache:
         self.hits = self.misses = self.evictions = 0
 
     def put(self, token_ids, cache: B200PagedKVCache) -> None:
+        if self.allocator.has_state:      # pages do not hold a recurrent state: such prefixes are not reusable
+            return
         page = cache.page_size
         key = tuple(int(t) for t in token_ids)[: (min(len(token_ids), cache.tokens) // page) * page]
         if not key:
@@ -145,12 +148,20 @@ class _Engine:
         self.allocator = kv_allocator or B200KVPageAllocator(page_size=self.page_size)
         if self.allocator.page_size != self.page_size:
             raise ValueError("kv_allocator page_size differs from the artifact's decode page size")
-        self.tp.check_model(heads=int(self.config.num_attention_heads), kv_heads=int(self.config.num_key_value_heads),
-                            intermediate=int(self.config.intermediate_size), vocab=int(self.config.vocab_size))
-        # under tensor parallelism a rank's pool holds only its own KV heads
-        self.allocator.configure(torch=torch, device=device, dtype=dtype, num_layers=int(self.config.num_layers),
-                                 kv_heads=int(self.config.num_key_value_heads) // self.tp.world,
-                                 head_dim=int(self.config.head_dim), kv_dtype=kv_dtype)
+        self.ragged = bool(getattr(self.config, "ragged", False))
+        self.plan_class: type = RaggedPlan if self.ragged else _DecodePlan
+        if self.ragged:
+            if self.tp.enabled or kv_dtype != "same" or dtype == torch.float16:
+                raise ValueError(f"{self.config.architecture} runs on one GPU in bfloat16 or float32 with caches of that type")
+            pools, states = self.config.cache_layout(self.page_size, dtype)
+            self.allocator.configure_layout(torch=torch, device=device, pools=pools, states=states)
+        else:
+            self.tp.check_model(heads=int(self.config.num_attention_heads), kv_heads=int(self.config.num_key_value_heads),
+                                intermediate=int(self.config.intermediate_size), vocab=int(self.config.vocab_size))
+            # under tensor parallelism a rank's pool holds only its own KV heads
+            self.allocator.configure(torch=torch, device=device, dtype=dtype, num_layers=int(self.config.num_layers),
+                                     kv_heads=int(self.config.num_key_value_heads) // self.tp.world,
+                                     head_dim=int(self.config.head_dim), kv_dtype=kv_dtype)
         self.max_seq_len = int(max_seq_len or self.config.max_position_embeddings)
         # Tensor-parallel collectives: this package's own kernels over peer memory (graph-capturable), or the
         # process group's library collectives launched eagerly (CB200_TP_COLLECTIVES=nccl; never captured).
@@ -160,10 +171,13 @@ class _Engine:
         self.tile_weights = True
         self.validated_batch: tuple[int, ...] | None = None      # identity of the last decode batch that passed the checks
         self.validated_sessions: list[Any] = []
-        self.prefill_chunk = 64        # prompt tokens per pass of the chunked prefill (0: one token per step)
+        # prompt tokens per pass of the chunked prefill (0: one token per step)
+        self.prefill_chunk = 2048 if self.ragged else 64
         self._rope_tables: dict[tuple[int, float], torch.Tensor] = {}
         self.attention_splits = int(attention_splits)
-        self.max_plans = max(1, int(max_plans))
+        self.max_plans = max(1, int(max_plans)) * (4 if self.ragged else 1)     # (ragged plans share their buffers)
+        self._scratch: dict[str, torch.Tensor] = {}
+        self._derived: dict[tuple, torch.Tensor] = {}
         self.plans: OrderedDict[tuple, "_DecodePlan"] = OrderedDict()
         self.plans_lowered = 0          # decode graphs lowered to launch lists so far
         self.graph_captures = 0         # CUDA graphs captured so far
@@ -236,17 +250,55 @@ class _Engine:
             self._rope_tables[key] = ops.rope_table(self.max_seq_len, head_dim, theta, self.device)
         return self._rope_tables[key]
 
-    def prefill_plan(self, rows: int, needed_pages: int) -> "_DecodePlan":
-        """The plan that pushes `rows` prompt tokens through the decode graph at once: row i is one (sequence,
-        position) pair, reads that sequence's page table and attends to position+1 tokens."""
-        key = ("prefill", rows)
+    # -- what ragged plans share ---------------------------------------------------------
+    def scratch(self, role: str, size: int) -> torch.Tensor:
+        """Device bytes for `role`, shared by every plan and grown on demand (a plan keeps the storage it was lowered with)."""
+        have = self._scratch.get(role)
+        if have is None or have.numel() < size:
+            self._scratch[role] = have = torch.zeros((max(1, size),), device=self.device, dtype=torch.uint8)
+        return have
+
+    def _derive(self, key: tuple, make: Callable[[], torch.Tensor], release: Iterable[str] = ()) -> torch.Tensor:
+        if key not in self._derived:
+            self._derived[key] = make()
+            for name in release:
+                self.weights.release(name)
+        return self._derived[key]
+
+    def concat_weight(self, names: tuple[str, ...]) -> torch.Tensor:
+        """Several weights of one input, row after row."""
+        return self._derive(("concat",) + names, lambda: torch.cat([self.weights.get_checked(n) for n in names]).contiguous(), names)
+
+    def paired_weight(self, names: tuple[str, ...]) -> torch.Tensor:
+        """gate and up rows alternating, the order the gated epilogue wants."""
+        return self._derive(("paired",) + names, lambda: torch.stack([self.weights.get_checked(n) for n in names], dim=1)
+                            .reshape(-1, self.weights.get_checked(names[0]).shape[1]).contiguous(), names)
+
+    def absorbed_weight(self, name: str, heads: int, dim: int, rank: int) -> torch.Tensor:
+        """A key up-projection [heads*dim, rank] turned per head: [heads*rank, dim], applied to queries."""
+        return self._derive(("absorbed", name), lambda: self.weights.get_checked(name).view(heads, dim, rank).transpose(1, 2)
+                            .reshape(heads * rank, dim).contiguous())
+
+    def rotate_half_table(self, dims: int, base: float) -> torch.Tensor:
+        return self._derive(("rotate_half", dims, base),
+                            lambda: torch.from_numpy(rotate_half_table(self.max_seq_len, dims, base)).to(self.device))
+
+    def decay_powers(self, decay: tuple[float, ...]) -> torch.Tensor:
+        return self._derive(("decay",) + decay, lambda: hybrid_ops.decay_powers(decay, self.device))
+
+    def portion_plan(self, rows: int, segments: int, logit_rows: int) -> "_DecodePlan":
+        """The ragged plan for up to `rows` rows of `segments` sequences with `logit_rows` wanted logits."""
+        return self._plan(("portions", bucket(rows), bucket(segments), bucket(max(1, logit_rows))), 0,
+                          lambda width: self.plan_class(self, bucket(rows), width, segments=bucket(segments),
+                                                        logit_rows=bucket(max(1, logit_rows))))
+
+    def _plan(self, key: tuple, needed_pages: int, make: Callable[[int], "_DecodePlan"]) -> "_DecodePlan":
         plan = self.plans.get(key)
         if plan is not None and (plan.pool_generation != self.allocator.generation or plan.width < needed_pages):
             self.plans.pop(key)
             plan = None
         if plan is None:
-            width = max(needed_pages, (self.max_seq_len + self.page_size - 1) // self.page_size)
-            plan = _DecodePlan(self, rows, width)
+            plan = make(max(needed_pages, (self.max_seq_len + self.page_size - 1) // self.page_size))
             self.plans_lowered += 1
             self.plans[key] = plan
             while len(self.plans) > self.max_plans:
@@ -255,27 +307,18 @@ class _Engine:
             self.plans.move_to_end(key)
         return plan
 
+    def prefill_plan(self, rows: int, needed_pages: int) -> "_DecodePlan":
+        """The plan that pushes `rows` prompt tokens through the decode graph at once: row i is one (sequence,
+        position) pair, reads that sequence's page table and attends to position+1 tokens."""
+        return self._plan(("prefill", rows), needed_pages, lambda width: _DecodePlan(self, rows, width))
+
     def plan_for(self, sessions: list["B200DecodeRuntime"]) -> "_DecodePlan":
         """The plan for a decode batch of this size. Plans are keyed by batch size, not by who is in the batch:
         a session is bound to a row for one step only, and `sync_sessions` rewrites the rows whose occupant,
         length or page list changed. Admitting or retiring a request therefore costs a few small copies, not
         a new lowering and a new CUDA-graph capture."""
-        key = ("decode", len(sessions))
-        plan = self.plans.get(key)
         needed_pages = max((s.kv_cache.tokens + 1 + self.page_size - 1) // self.page_size for s in sessions)
-        if plan is not None and (plan.pool_generation != self.allocator.generation or plan.width < needed_pages):
-            self.plans.pop(key)
-            plan = None
-        if plan is None:
-            width = max(needed_pages, (self.max_seq_len + self.page_size - 1) // self.page_size)
-            plan = _DecodePlan(self, len(sessions), width)
-            self.plans_lowered += 1
-            self.plans[key] = plan
-            while len(self.plans) > self.max_plans:
-                self.plans.popitem(last=False)
-        else:
-            self.plans.move_to_end(key)
-        return plan
+        return self._plan(("decode", len(sessions)), needed_pages, lambda width: self.plan_class(self, len(sessions), width))
 
 
 class _DecodePlan:
@@ -725,6 +768,9 @@ class _DecodePlan:
         return out
 
 
+RaggedPlan = make_plan_class(_DecodePlan)
+
+
 class B200DecodeRuntime:
     """Execute compiled CacheIR decode graphs on a B200 (see module docstring)."""
 
@@ -762,7 +808,10 @@ class B200DecodeRuntime:
                 dev = torch.device("cuda", torch.cuda.current_device())
             selected = _dtype_from_name(dtype)
             if selected is None:
-                selected = torch.float16 if str(artifact.config.dtype).lower() in {"float16", "fp16", "bfloat16", "bf16"} else torch.float32
+                if getattr(artifact.config, "ragged", False):
+                    selected = torch.bfloat16
+                else:
+                    selected = torch.float16 if str(artifact.config.dtype).lower() in {"float16", "fp16", "bfloat16", "bf16"} else torch.float32
             with torch.cuda.device(dev):
                 _engine = _Engine(artifact, device=dev, dtype=selected, weights=weights, tensor_source=tensor_source,
                                   kv_allocator=kv_allocator, max_seq_len=max_seq_len, use_cuda_graph=use_cuda_graph,
@@ -884,11 +933,7 @@ class B200DecodeRuntime:
         eng.plans.move_to_end(("decode", n))
         return plan
 
-    def _prepare_batch(self, sessions, token_ids) -> _DecodePlan:
-        if not sessions:
-            raise ValueError("run_decode_batch requires at least one session")
-        if len(sessions) != len(token_ids):
-            raise ValueError("sessions and token_ids must have the same length")
+    def _check_sessions(self, sessions) -> None:
         batch_key = tuple(map(id, sessions))
         if batch_key != self._engine.validated_batch:      # the same sessions as last step were checked then
             for session in sessions:
@@ -900,6 +945,13 @@ class B200DecodeRuntime:
                 raise ValueError("a session may appear only once in a decode batch")
             self._engine.validated_batch = batch_key
             self._engine.validated_sessions = list(sessions)      # keeps the ids above from being recycled
+
+    def _prepare_batch(self, sessions, token_ids) -> _DecodePlan:
+        if not sessions:
+            raise ValueError("run_decode_batch requires at least one session")
+        if len(sessions) != len(token_ids):
+            raise ValueError("sessions and token_ids must have the same length")
+        self._check_sessions(sessions)
         with torch.cuda.device(self.device):
             for session in sessions:
                 session.kv_cache.extend(1)      # opens a page when the new token starts one
@@ -956,6 +1008,8 @@ class B200DecodeRuntime:
         if ids.shape[1] == 0:
             raise ValueError("run needs at least one token")
         tokens = [int(t) for t in ids[0]]
+        if self._engine.ragged and mode == "prefill":
+            return self.run_step_batch([self], [tokens], [list(range(len(tokens)))]).unsqueeze(0)
         chunk = self._engine.prefill_chunk
         if mode == "prefill" and chunk > 1 and len(tokens) > chunk // 4:
             self._enforce_memory_limit()
@@ -974,6 +1028,88 @@ class B200DecodeRuntime:
         finally:
             self.clone_outputs = keep
         return torch.cat(steps, dim=1) if len(steps) > 1 else steps[0]
+
+    # -- mixed steps -----------------------------------------------------------------------
+    def run_step_batch(self, sessions: list["B200DecodeRuntime"], token_batches: list[list[int]],
+                       wanted: list[list[int]] | None = None) -> torch.Tensor:
+        """One step of several sequences, each with its own number of next tokens: portions of prompts beside single
+        decoded tokens, as one batch. `wanted[i]` lists the places among session i's tokens whose logits are returned
+        (default: the last one). Returns [sum of wanted, vocab], session by session. Nothing is reserved or run unless
+        the pages (and state slots) of the whole step are available."""
+        eng = self._engine
+        if wanted is None:
+            wanted = [[len(t) - 1] for t in token_batches]
+        if not sessions or not (len(sessions) == len(token_batches) == len(wanted)):
+            raise ValueError("run_step_batch needs a token batch and a list of wanted places for every session")
+        if any(len(t) == 0 for t in token_batches):
+            raise ValueError("run_step_batch requires non-empty token batches")
+        if any(not 0 <= int(p) < len(t) for t, places in zip(token_batches, wanted) for p in places):
+            raise ValueError("a wanted place lies outside its session's tokens")
+        vocab = int(eng.config.vocab_size)
+        if any(not 0 <= int(t) < vocab for tokens in token_batches for t in tokens):
+            raise ValueError(f"token ids must be in [0, {vocab})")
+        self._check_sessions(sessions)
+        self._enforce_memory_limit()
+        self._check_room(sessions, [len(t) for t in token_batches])
+        if all(len(t) == 1 for t in token_batches):
+            logits = self.run_decode_batch(sessions, [int(t[0]) for t in token_batches])[:, 0]
+            rows = [i for i, places in enumerate(wanted) for _ in places]
+            return logits if rows == list(range(len(sessions))) else logits[rows]
+        starts = [s.kv_cache.tokens for s in sessions]
+        for session, tokens in zip(sessions, token_batches):
+            session.kv_cache.extend(len(tokens))
+        results = []
+        with torch.cuda.device(self.device):
+            passes = cut_passes(token_batches, eng.prefill_chunk or 64)
+            for part in passes:                                   # (session, first token, last token + 1)
+                want = [(i, int(p)) for i, lo, hi in part for p in wanted[i] if lo <= int(p) < hi]
+                logits = self._run_rows(sessions, token_batches, starts, part, want)
+                if want:
+                    results.append((want, logits if len(passes) == 1 and not self.clone_outputs else logits.clone()))
+        eng.count("cacheir.b200_step_batch", len(passes))
+        if not results:
+            return torch.empty((0, vocab), device=self.device, dtype=torch.float32 if eng.ragged else self.dtype)
+        found = {place: (r, j) for r, (want, _) in enumerate(results) for j, place in enumerate(want)}
+        order = [found[(i, int(p))] for i, places in enumerate(wanted) for p in places]
+        if order == [(0, j) for j in range(len(order))] and len(results) == 1:
+            return results[0][1]
+        return torch.stack([results[r][1][j] for r, j in order])
+
+    def _run_rows(self, sessions, token_batches, starts, part, want) -> torch.Tensor:
+        """One pass over the rows of `part`; returns the logits of `want`, in its order (valid until the next pass)."""
+        eng = self._engine
+        row0, row = {}, 0
+        for i, lo, hi in part:
+            row0[i] = row - lo
+            row += hi - lo
+        rows = [row0[i] + p for i, p in want]
+        if eng.ragged:
+            plan = eng.portion_plan(row, len(part), len(rows))
+            plan.sync_portions([(sessions[i].kv_cache, starts[i] + lo, [int(t) for t in token_batches[i][lo:hi]]) for i, lo, hi in part], rows)
+            plan.run_program()
+            return plan.logits[: len(rows)]
+        needed = max(len(s.kv_cache.pages) for s in sessions)
+        plan = eng.prefill_plan(eng.prefill_chunk or 64, needed)
+        plan.sync_prefill_rows([(sessions[i].kv_cache, starts[i] + p, int(token_batches[i][p])) for i, lo, hi in part for p in range(lo, hi)])
+        plan.run_program()
+        return plan.logits[rows]
+
+    def _check_room(self, sessions, lengths: list[int]) -> None:
+        """Raise before anything is reserved when a step cannot get its pages, state slots or positions."""
+        alloc, limit = self._engine.allocator, self._engine.max_seq_len
+        for session, n in zip(sessions, lengths):
+            if session.kv_cache.tokens + n > limit:
+                raise ValueError(f"sequence of {session.kv_cache.tokens + n} tokens exceeds max_seq_len={limit}; "
+                                 "construct the runtime with a larger max_seq_len")
+        free = alloc.free_slots()
+        need = sum(s.kv_cache.pages_needed(n) for s, n in zip(sessions, lengths))
+        if free is not None and need > free:
+            raise KVPoolExhausted(f"the step needs {need} new pages, the pool has {free}")
+        if alloc.has_state:
+            free = alloc.free_states()
+            need = sum(s.kv_cache.state_slot is None for s in sessions)
+            if free is not None and need > free:
+                raise KVPoolExhausted(f"the step needs {need} new state slots, {free} are free")
 
     def _prefill_chunked(self, tokens: list[int], chunk: int) -> torch.Tensor:
         """Prefill that fills the page pool directly, `chunk` prompt tokens per pass through the decode
@@ -1039,7 +1175,14 @@ class B200DecodeRuntime:
         for session in sessions:
             session.kv_cache.clear()
         vocab = int(self._engine.config.vocab_size)
-        out = torch.zeros((len(sessions), max(lens), vocab), device=self.device, dtype=self.dtype)
+        out = torch.zeros((len(sessions), max(lens), vocab), device=self.device,
+                          dtype=torch.float32 if self._engine.ragged else self.dtype)
+        if self._engine.ragged:
+            logits = self.run_step_batch(sessions, token_id_batches, [list(range(n)) for n in lens])
+            for i, part in enumerate(logits.split(lens)):
+                out[i, : lens[i]] = part
+            self._engine.count("cacheir.b200_prefill_batch_graph")
+            return out
         chunk = self._engine.prefill_chunk
         if chunk > 1 and sum(lens) > chunk // 4:
             # Packed prefill: the prompt tokens of all sequences are the rows of 64-row passes through the decode
@@ -1125,10 +1268,28 @@ class B200DecodeRuntime:
         and clears the word."""
         from . import _lib
         with torch.cuda.device(self.device):
-            status = int(_lib.load().cacheir_b200_device_status(1))
+            status = hybrid_ops.device_status() if self._engine.ragged else int(_lib.load().cacheir_b200_device_status(1))
         if status != 0:
             raise RuntimeError(f"cacheir_b200 device status {status:#x}: a bounded wait on the GPU gave up "
                                f"(kernel class {status >> 8}, wait {status & 0xFF}); the last results are undefined")
+
+
+def cut_passes(token_batches: list[list[int]], rows: int) -> list[list[tuple[int, int, int]]]:
+    """Cut a step into passes of at most `rows` rows: lists of (sequence, first token, last token + 1). A sequence's
+    tokens stay in order across passes."""
+    passes: list[list[tuple[int, int, int]]] = [[]]
+    room = rows
+    for i, tokens in enumerate(token_batches):
+        lo = 0
+        while lo < len(tokens):
+            if room == 0:
+                passes.append([])
+                room = rows
+            hi = min(len(tokens), lo + room)
+            passes[-1].append((i, lo, hi))
+            room -= hi - lo
+            lo = hi
+    return passes
 
 
 def create_runtime(artifact: Any, *, backend: str = "auto", **kwargs) -> B200DecodeRuntime:

@@ -8,6 +8,8 @@ form. The pack itself runs on the device (`quantization.pack_weight_device`).
 """
 from __future__ import annotations
 
+import json
+import struct
 from pathlib import Path
 from typing import Any, Callable, Mapping
 
@@ -17,8 +19,45 @@ import torch
 from .quantization import B200PackedWeight, dequantize_device, pack_weight_device
 
 
+_SAFETENSORS_DTYPES = {"F64": torch.float64, "F32": torch.float32, "F16": torch.float16, "BF16": torch.bfloat16,
+                       "I64": torch.int64, "I32": torch.int32, "I16": torch.int16, "I8": torch.int8, "U8": torch.uint8,
+                       "BOOL": torch.bool}
+
+
+class SafetensorsFile:
+    """A .safetensors file: an 8-byte little-endian length, that many bytes of JSON (name -> dtype, shape,
+    data_offsets), then the data. Tensors are CPU views of a private memory map."""
+
+    def __init__(self, path: str | Path):
+        self.path = Path(path)
+        with open(self.path, "rb") as f:
+            head = f.read(8)
+            if len(head) != 8:
+                raise ValueError(f"{self.path}: not a safetensors file")
+            size = struct.unpack("<Q", head)[0]
+            if size > self.path.stat().st_size - 8:
+                raise ValueError(f"{self.path}: the header is longer than the file")
+            self.entries: dict[str, dict] = json.loads(f.read(size))
+        self.entries.pop("__metadata__", None)
+        self._data = np.memmap(self.path, dtype=np.uint8, mode="c", offset=8 + size) if self.entries else np.empty(0, np.uint8)
+
+    def __contains__(self, key: str) -> bool:
+        return key in self.entries
+
+    def tensor(self, key: str) -> torch.Tensor:
+        entry = self.entries[key]
+        begin, end = entry["data_offsets"]
+        dtype = _SAFETENSORS_DTYPES[entry["dtype"]]
+        shape = tuple(int(n) for n in entry["shape"])
+        count = int(np.prod(shape, dtype=np.int64))
+        if end - begin != count * torch.empty((), dtype=dtype).element_size() or end > self._data.size:
+            raise ValueError(f"{self.path}: tensor {key!r} does not fit its data")
+        raw = torch.from_numpy(np.array(self._data[begin:end]))     # (a copy: views of the map need not be aligned)
+        return raw.view(dtype).reshape(shape) if count else torch.empty(shape, dtype=dtype)
+
+
 class TensorSource:
-    """Where raw tensors come from: an .npz file/directory, a mapping key -> array,
+    """Where raw tensors come from: an .npz or .safetensors file, a directory with one, a mapping key -> array,
     or a callable key -> tensor (synthetic weights generated on the device)."""
 
     def __init__(self, source: str | Path | Mapping[str, Any] | Callable[[str, tuple[int, ...]], torch.Tensor]):
@@ -26,6 +65,7 @@ class TensorSource:
         self._mapping: Mapping[str, Any] | None = None
         self._callable = None
         self._path: Path | None = None
+        self._safetensors: SafetensorsFile | None = None
         if callable(source):
             self._callable = source
         elif isinstance(source, Mapping):
@@ -40,6 +80,11 @@ class TensorSource:
             return self._mapping[key]
         path = self._path
         assert path is not None
+        archive = path if path.suffix == ".safetensors" else path / "model.safetensors"
+        if self._safetensors is None and archive.is_file() and not ((file or "").endswith(".npz") and (path / file).exists()):
+            self._safetensors = SafetensorsFile(archive)
+        if self._safetensors is not None:
+            return self._safetensors.tensor(key)
         if path.is_file() and path.suffix == ".npz":
             npz_path = path
         elif path.is_dir():
@@ -47,7 +92,7 @@ class TensorSource:
         else:
             raise FileNotFoundError(f"could not load weight {key!r} from {path}")
         if npz_path.suffix != ".npz" or not npz_path.exists():
-            raise FileNotFoundError(f"cacheir_b200 loads .npz weights; {npz_path} not found")
+            raise FileNotFoundError(f"cacheir_b200 loads .npz or .safetensors weights; {npz_path} not found")
         if self._npz is None:
             with np.load(npz_path) as data:
                 self._npz = {k: data[k] for k in data.files}
@@ -63,6 +108,7 @@ class B200WeightStore:
         self.device = device
         self.dtype = dtype
         self._cache: dict[str, torch.Tensor] = {}
+        self._f32: dict[str, torch.Tensor] = {}
         self._qcache: dict[str, B200PackedWeight] = {}
 
     def _raw_fp32(self, value_name: str) -> torch.Tensor:
@@ -83,6 +129,25 @@ class B200WeightStore:
                     raise ValueError(f"Unsupported quantization mode {self.quant!r}")
                 tensor = dequantize_device(packed, self.dtype)
             self._cache[value_name] = tensor.to(self.dtype).contiguous()
+        return self._cache[value_name]
+
+    def get_f32(self, value_name: str) -> torch.Tensor:
+        """A parameter that stays in float32 whatever the runtime dtype is (norm weights, sinks, scalars)."""
+        if value_name not in self._f32:
+            self._f32[value_name] = self._checked(value_name).contiguous()
+        return self._f32[value_name]
+
+    def _checked(self, value_name: str) -> torch.Tensor:
+        tensor = self._raw_fp32(value_name)
+        want = tuple(self.specs[value_name].shape)
+        if tuple(tensor.shape) != want:
+            raise ValueError(f"weight {value_name!r} has shape {tuple(tensor.shape)}, the configuration needs {want}")
+        return tensor
+
+    def get_checked(self, value_name: str) -> torch.Tensor:
+        """`get` of a weight whose shape the model's configuration fixes."""
+        if value_name not in self._cache:
+            self._cache[value_name] = self._checked(value_name).to(self.dtype).contiguous()
         return self._cache[value_name]
 
     def get_quantized(self, value_name: str) -> B200PackedWeight:
@@ -108,4 +173,5 @@ class B200WeightStore:
     def release(self, value_name: str) -> None:
         """Forget the cached copies of a weight (its owner keeps a fused form)."""
         self._cache.pop(value_name, None)
+        self._f32.pop(value_name, None)
         self._qcache.pop(value_name, None)
