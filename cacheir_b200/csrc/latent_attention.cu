@@ -155,6 +155,11 @@ struct FastParams {
   int row_bytes;               // padded shared-memory row
 };
 
+constexpr int kProbPitch = 144;          // bytes per row of the probability tile when it has memory of its own
+// With 64 rotated dimensions and more, the scores' last use of a key tile frees 128 bytes in each of its 64 rows: the
+// probabilities go there and the largest latents fit with 64 query rows.
+__host__ __device__ constexpr bool prob_in_keys(int rot_dim) { return rot_dim >= 64; }
+
 template <int MROWS, int RANKMAX>
 __global__ void __launch_bounds__(kThreads, 1)
 latent_attention_kernel(const FastParams p) {
@@ -169,8 +174,10 @@ latent_attention_kernel(const FastParams p) {
   const int rb = p.row_bytes;
   uint8_t* s_kv = smem;                                  // [2][64][rb]
   uint8_t* s_q = s_kv + 2 * kPage * rb;                  // [MROWS][rb]
-  __nv_bfloat16* s_p = reinterpret_cast<__nv_bfloat16*>(s_q + MROWS * rb);   // [MROWS][72]
-  float* s_red = reinterpret_cast<float*>(s_p + MROWS * 72);                 // [MROWS][NW]
+  const bool shared_p = prob_in_keys(a.rot_dim);
+  const int pp = shared_p ? rb : kProbPitch;
+  uint8_t* s_own_p = s_q + MROWS * rb;                   // [MROWS][kProbPitch], absent when shared_p
+  float* s_red = reinterpret_cast<float*>(s_own_p + (shared_p ? 0 : MROWS * kProbPitch));   // [MROWS][NW]
   uint64_t* bars = reinterpret_cast<uint64_t*>(s_red + MROWS * NW);          // [2]
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -256,6 +263,7 @@ latent_attention_kernel(const FastParams p) {
     if (warp == 0 && pg + 1 < pg_end) load_page(pg + 1, stage ^ 1);
     ok = ptx::mbar_wait(smem_addr(&bars[stage]), (it >> 1) & 1, &g_latent_status, (7 << 8) | 1) && ok;
     const uint32_t kv = smem_addr(s_kv + stage * kPage * rb);
+    uint8_t* s_p = shared_p ? s_kv + stage * kPage * rb + a.kv_rank * 2 : s_own_p;
     // scores: 16 rows x (8 NT) keys
     float s[NT][4];
 #pragma unroll
@@ -325,9 +333,9 @@ latent_attention_kernel(const FastParams p) {
         s[t][e] = exp2f(s[t][e] - m_run[e >> 1]);       // masked: exp2(-inf) = 0
         l_run[e >> 1] += s[t][e];
       }
-      __nv_bfloat16* dst = s_p + (mw * 16 + (lane >> 2)) * 72 + key0 + t * 8 + (lane & 3) * 2;
+      uint8_t* dst = s_p + (mw * 16 + (lane >> 2)) * pp + (key0 + t * 8 + (lane & 3) * 2) * 2;
       *reinterpret_cast<uint32_t*>(dst) = pack_bf16(s[t][0], s[t][1]);
-      *reinterpret_cast<uint32_t*>(dst + 8 * 72) = pack_bf16(s[t][2], s[t][3]);
+      *reinterpret_cast<uint32_t*>(dst + 8 * pp) = pack_bf16(s[t][2], s[t][3]);
     }
     __syncthreads();
     // output columns
@@ -338,7 +346,7 @@ latent_attention_kernel(const FastParams p) {
         acc[i][j][0] *= alpha[0]; acc[i][j][1] *= alpha[0];
         acc[i][j][2] *= alpha[1]; acc[i][j][3] *= alpha[1];
       }
-    const uint32_t pa = smem_addr(s_p) + ((mw * 16 + (lane & 15)) * 72 + (lane >> 4) * 8) * 2;
+    const uint32_t pa = smem_addr(s_p) + (mw * 16 + (lane & 15)) * pp + (lane >> 4) * 16;
     const uint32_t va = kv + ((lane & 7) + ((lane >> 3) & 1) * 8) * rb + (lane >> 4) * 16;
 #pragma unroll
     for (int k = 0; k < kPage / 16; ++k) {
@@ -354,6 +362,7 @@ latent_attention_kernel(const FastParams p) {
         }
       }
     }
+    if (shared_p) asm volatile("fence.proxy.async.shared::cta;" ::: "memory");   // s_p lies where the next page lands
     __syncthreads();        // the stage, s_p and s_red are free again
   }
 
@@ -425,15 +434,15 @@ latent_combine_kernel(const float* __restrict__ part_o, const float* __restrict_
 }
 
 int padded_row_bytes(int width) { return (width + 15) / 16 * 32 + 16; }
-size_t fast_smem(int mrows, int width) {
-  const int rb = padded_row_bytes(width);
-  return 128 + static_cast<size_t>(2 * kPage + mrows) * rb + static_cast<size_t>(mrows) * 72 * 2 + static_cast<size_t>(mrows) * 8 * 4 + 64;
+size_t fast_smem(int mrows, int kv_rank, int rot_dim) {
+  const int rb = padded_row_bytes(kv_rank + rot_dim);
+  return 128 + static_cast<size_t>(2 * kPage + mrows) * rb + (prob_in_keys(rot_dim) ? 0 : static_cast<size_t>(mrows) * kProbPitch) + static_cast<size_t>(mrows) * 8 * 4 + 64;
 }
 int head_groups(int heads, bool decode) { const int cap = decode ? 32 : 64; return (heads + cap - 1) / cap; }
 
 template <int MROWS, int RANKMAX>
 int launch_fast(const FastParams& p, dim3 grid, cudaStream_t st) {
-  const size_t smem = fast_smem(MROWS, p.a.kv_rank + p.a.rot_dim);
+  const size_t smem = fast_smem(MROWS, p.a.kv_rank, p.a.rot_dim);
   auto kern = latent_attention_kernel<MROWS, RANKMAX>;
   cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
   if (e != cudaSuccess) return static_cast<int>(e);
@@ -506,7 +515,7 @@ extern "C" int cacheir_b200_latent_attention_simple(const cacheir_b200_latent_ar
 
 extern "C" int cacheir_b200_latent_attention_supported(int kv_rank, int rot_dim, int page_size, int dtype) {
   return dtype == CACHEIR_B200_BF16 && page_size == kPage && kv_rank >= 16 && kv_rank % 16 == 0 && kv_rank <= 512 && rot_dim % 8 == 0 &&
-         rot_dim <= 128 && fast_smem(64, kv_rank + rot_dim) <= 227 * 1024 ? 1 : 0;
+         rot_dim <= 128 && fast_smem(64, kv_rank, rot_dim) <= 227 * 1024 ? 1 : 0;
 }
 
 extern "C" int cacheir_b200_latent_attention_splits(int rows, int heads, int window, int max_pages, int page_size) {

@@ -1224,8 +1224,12 @@ class B200DecodeRuntime:
     def generate(self, prompt: str, *, max_new_tokens: int = 16, use_prefix_cache: bool = False,
                  remember_prefix: bool = True) -> Iterable[str]:
         token_ids = self.tokenizer.encode(prompt)
-        logits, _ = self.prefill_tokens(token_ids, use_prefix_cache=use_prefix_cache,
-                                        remember_prefix=remember_prefix and use_prefix_cache)
+        if self._engine.ragged:            # only the last position's logits are needed
+            self.kv_cache.clear()
+            logits = self.run_step_batch([self], [token_ids]).unsqueeze(0)
+        else:
+            logits, _ = self.prefill_tokens(token_ids, use_prefix_cache=use_prefix_cache,
+                                            remember_prefix=remember_prefix and use_prefix_cache)
         vocab = int(self._engine.config.vocab_size)
         for _ in range(max_new_tokens):
             next_id = int(torch.argmax(logits[0, -1]).item()) % vocab
