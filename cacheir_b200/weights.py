@@ -117,7 +117,8 @@ class B200WeightStore:
         raw = self.source.load(spec.key, shape, getattr(spec, "file", None))
         if isinstance(raw, torch.Tensor):
             return raw.to(device=self.device, dtype=torch.float32)
-        return torch.from_numpy(np.ascontiguousarray(np.asarray(raw, dtype=np.float32))).to(self.device)
+        raw = np.array(raw, dtype=np.float32, order="C")        # (a scalar stays 0-dimensional)
+        return torch.from_numpy(raw).to(self.device)
 
     def get(self, value_name: str) -> torch.Tensor:
         if value_name not in self._cache:

@@ -61,7 +61,7 @@ def random_weights(cfg, seed=0):
         elif name in ("embed", "side.embed"):
             a = rng.normal(0, 0.5, shape)
         else:
-            gain = 2.5 if name.endswith(("mix.q", "mix.uk", "mix.dkv")) else 1.2      # sharp scores: single keys matter
+            gain = 1.7 if name.endswith(("mix.q", "mix.uk", "mix.dkv")) else 1.2      # sharp scores: single keys matter
             a = rng.normal(0, gain / np.sqrt(shape[1]), shape)
         out[name] = torch.from_numpy(np.asarray(a, np.float32)).to(torch.bfloat16).float().numpy()
     return out
