@@ -859,6 +859,11 @@ def main() -> None:
     parser.add_argument("--separate-attention-prepass", action="store_true",
                         help="diagnostic: run the o projection's activation pre-pass as its own launch instead of inside the attention kernel")
     parser.add_argument("--no-tp-leg", action="store_true", help="with --gpus N > 1: skip the tensor-parallel leg attached to the line")
+    parser.add_argument("--family", choices=["gutorax"], help="throughput and per-kernel rooflines of this model family beside the "
+                        "Llama-shaped one at equal size (bench_hybrid.py); prints one JSON line per size")
+    parser.add_argument("--family-sizes", default="4096,2048")
+    parser.add_argument("--prompt", type=int, default=2048, help="--family: prompt tokens of the prefill measurement")
+    parser.add_argument("--ctx", type=int, default=2048, help="--family: cached tokens per sequence when decoding")
     parser.add_argument("--micro", choices=["qgemv", "attention", "layer"],
                         help="time one kernel alone, or the kernels of one decoder layer of the 8B-shaped step (profiling aid)")
     parser.add_argument("--m", type=int, default=32)
@@ -881,6 +886,20 @@ def main() -> None:
     claim_stdout()
     if args.micro:
         run_micro(args)
+        return
+    if args.family:
+        import torch
+
+        import bench_hybrid
+        peaks_path = ROOT / "MEASURED_PEAKS.json"
+        peaks = json.loads(peaks_path.read_text()) if peaks_path.exists() else {"hbm_gbs": 6650.0, "bf16_tflops": 1590.0}
+        torch.cuda.set_device(0)
+        batch = 32 if args.batch == parser.get_default("batch") else args.batch
+        for size in args.family_sizes.split(","):
+            clocks = ClockSampler(0)
+            clocks.start()
+            line = bench_hybrid.run(size, batch, args.ctx, args.prompt, min(args.steps, 32), peaks)
+            emit(dict(line, clocks=clocks.stop(), peaks="measured" if peaks_path.exists() else "fallback"))
         return
     cfg = dict(WORKLOADS[args.workload])
     if args.kv == "int8":

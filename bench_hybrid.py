@@ -1,0 +1,238 @@
+"""`bench.py --family gutorax`: prefill and decode throughput of the Gutorax family beside the Llama-shaped family at
+equal width, feed-forward, heads and layer count (random weights), and every kernel's distance from its roofline.
+
+Throughput: decode is `decode_greedy_batch` (CUDA-graph replay, argmax fed back on the device) over `batch` sequences
+with `ctx` cached tokens; prefill is one prompt through the runtime's own entry point, with the last position's logits
+wanted where the runtime lets a caller say so. Kernel times: all launches of one kind in a step (every layer's, so that
+weights and caches come from HBM) as one CUDA graph, timed with events; the roofline is the larger of algorithmic bytes
+over the measured copy bandwidth and FLOPs over the measured bf16 rate, summed over the same launches.
+"""
+from __future__ import annotations
+
+from collections import defaultdict
+
+SIZES = {
+    # width, ff, heads, kv_heads (Llama), head dim, latent rank, rotated dims, window, layers, vocab
+    "4096": dict(width=4096, ff=14336, heads=32, kv_heads=8, dim=128, rank=512, rot=64, window=4096, layers=8, vocab=32768, side=256),
+    "2048": dict(width=2048, ff=5632, heads=16, kv_heads=8, dim=128, rank=256, rot=64, window=1024, layers=12, vocab=32768, side=128),
+}
+
+
+def gutorax_config(s: dict) -> dict:
+    """Layers in groups of four: latent attention, recurrence, latent attention on the first one's cache, recurrence."""
+    layers = []
+    for i in range(s["layers"]):
+        if i % 2:
+            t, m = "lightning", {"heads": s["heads"], "dim": s["dim"], "vdim": s["dim"], "decay": [1 - 2.0 ** -(2 + h * 8 / s["heads"]) for h in range(s["heads"])]}
+        else:
+            t, m = "latent_attention", {"heads": s["heads"], "dim": s["dim"], "rot_dim": s["rot"], "vdim": s["dim"], "kv_rank": s["rank"],
+                                        "scale": (s["dim"] + s["rot"]) ** -0.5, "mask": {"size": s["window"]},
+                                        "rot": {"base": 500000.0, "dims": s["rot"]}}
+            if i % 4 == 2:
+                m["kv_from"] = i - 2
+        layers.append({"type": t, "mixer": m, "mlp": {"kind": "dense", "ff": s["ff"]}})
+    return {"architecture": "Gutorax", "width": s["width"], "vocab": s["vocab"], "embedding": {"scale": s["width"] ** 0.5},
+            "norm": {"eps": 1e-5}, "token_side": {"dim": s["side"]}, "layers": layers}
+
+
+def synthetic(device):
+    import zlib
+
+    import torch
+    gen = torch.Generator(device=device)
+
+    def make(key: str, shape: tuple[int, ...]):
+        if len(shape) <= 1:
+            return torch.full(shape, 0.6 if key.endswith("alpha") else 1.0, device=device)
+        gen.manual_seed(zlib.crc32(key.encode()))
+        return torch.randn(shape, device=device, generator=gen) * 0.02
+    return make
+
+
+def build(family: str, s: dict, *, batch: int, positions: int):
+    import torch
+
+    from cacheir_b200 import (B200DecodeRuntime, B200KVPageAllocator, GutoraxConfig, ModelConfig, build_decoder_artifact,
+                              build_gutorax_artifact)
+    dev = torch.device("cuda", torch.cuda.current_device())
+    if family == "gutorax":
+        art, page = build_gutorax_artifact(GutoraxConfig.from_dict(gutorax_config(s))), 64
+        dtype = "bfloat16"
+    else:
+        art = build_decoder_artifact(ModelConfig(
+            architecture="LlamaForCausalLM", hidden_size=s["width"], intermediate_size=s["ff"], num_layers=s["layers"],
+            num_attention_heads=s["heads"], num_key_value_heads=s["kv_heads"], vocab_size=s["vocab"], max_position_embeddings=positions,
+            rope_theta=500000.0, dtype="float16"), quant="int8", modes=("decode",))
+        page, dtype = 16, "float16"
+    alloc = B200KVPageAllocator(page_size=page, initial_slots=(batch + 1) * ((positions + page - 1) // page), initial_states=batch + 1)
+    return B200DecodeRuntime(art, dtype=dtype, tensor_source=synthetic(dev), kv_allocator=alloc, max_seq_len=positions, clone_outputs=False)
+
+
+def fill(rt, batch: int, ctx: int):
+    """`batch` sessions with `ctx` cached tokens of synthetic content."""
+    sessions = [rt.fork() for _ in range(batch)]
+    for s in sessions:
+        s.kv_cache.extend(ctx)
+    for pool in rt.kv_allocator._pools.values():
+        for t in pool.values():
+            t.normal_()
+    for state in rt.kv_allocator._states.values():
+        state.normal_()
+    return sessions
+
+
+def timed(fn, iters: int) -> float:
+    """Milliseconds per call on the device."""
+    import torch
+    for _ in range(3):
+        fn()
+    start, stop = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+    torch.cuda.synchronize()
+    start.record()
+    for _ in range(iters):
+        fn()
+    stop.record()
+    torch.cuda.synchronize()
+    return start.elapsed_time(stop) / iters
+
+
+def kind_times(plan, iters: int = 5) -> dict[str, tuple[int, float]]:
+    """kind -> (launch groups per step, microseconds per step)."""
+    import torch
+    groups: dict[str, list] = defaultdict(list)
+    for fn, (key, _) in zip(plan.program, plan._count_keys):
+        if key != "b200.advance_positions":
+            groups[key].append(fn)
+    out = {}
+    for key, fns in groups.items():
+        graph = torch.cuda.CUDAGraph()
+        for fn in fns:
+            fn()
+        torch.cuda.synchronize()
+        with torch.cuda.graph(graph):
+            for _ in range(2):
+                for fn in fns:
+                    fn()
+        out[key] = (len(fns), timed(graph.replay, iters) * 1e3 / 2)
+    return out
+
+
+def gutorax_work(s: dict, rows: int, logit_rows: int, keys_per_row: float, cached_rows: float, decode: bool) -> dict[str, list[tuple[float, float]]]:
+    """kind -> (bytes, FLOPs) of every launch. `keys_per_row`: cache rows a token attends to on average; `cached_rows`:
+    distinct cache rows of the step."""
+    w, ff, h, d, rank, rot, side = s["width"], s["ff"], s["heads"], s["dim"], s["rank"], s["rot"], s["side"]
+    work: dict[str, list[tuple[float, float]]] = defaultdict(list)
+
+    def gemm(kind, n, k, n_out, t=rows, extra=0.0):
+        work["b200.dense_gemm" + kind].append((2.0 * (n * k + t * k + t * n_out) + extra, 2.0 * t * n * k))
+
+    for i in range(s["layers"]):
+        if i % 2:
+            gemm(".silu", 4 * h * d, w, 4 * h * d)
+            state = rows * h * d * d * 4.0 * 2 if decode else h * d * d * 4.0 * 2
+            io = rows * h * d * 4 * 2.0
+            work["b200.recurrence_step" if decode else "b200.recurrence_chunked"].append((state + io, rows * h * 4.0 * d * d))
+            work["b200.gated_rms"].append((rows * h * d * 3 * 2.0, 0.0))
+        else:
+            own = i % 4 == 0
+            n = h * (d + rot) + (rank + rot if own else 0) + h * d
+            gemm("", n, w, n)
+            work["b200.latent_prepare"].append((rows * (h * rot * 2 + (2 * (rank + rot) if own else 0)) * 2.0, 0.0))
+            work["b200.dense_gemm.heads"].append((2.0 * (h * rank * d + rows * h * (d + rank)), 2.0 * rows * h * rank * d))
+            work["b200.latent_attention"].append((2.0 * (cached_rows * (rank + rot) + rows * h * (2 * rank + rot)),
+                                                  2.0 * rows * h * keys_per_row * (2 * rank + rot)))
+            work["b200.dense_gemm.heads_gated"].append((2.0 * (h * rank * d + rows * h * (rank + 2 * d)), 2.0 * rows * h * rank * d))
+        gemm(".residual_dyt", w, h * d, 0, extra=rows * w * (8 + 2))
+        gemm(".geglu", 2 * ff, w, ff)
+        gemm(".residual_dyt", w, ff, 0, extra=rows * w * (8 + 2))
+        gemm(".gelu_embed", side, w, 2 * side)
+        gemm("", w, side, w)
+        work["b200.residual_rms"].append((rows * w * (2 + 8 + 2.0), 0.0))
+    work["b200.scaled_embedding"].append((rows * w * (2 + 4 + 2.0), 0.0))
+    work["b200.dyt_rows"].append((logit_rows * w * 6.0, 0.0))
+    gemm("", s["vocab"], w, 2 * s["vocab"], t=logit_rows)
+    return work
+
+
+def llama_work(s: dict, rows: int, keys_per_row: float, cached_rows: float) -> dict[str, list[tuple[float, float]]]:
+    w, ff, d = s["width"], s["ff"], s["width"] // s["heads"]
+    kv = s["kv_heads"] * d
+    work: dict[str, list[tuple[float, float]]] = defaultdict(list)
+
+    def gemm(key, n, k, n_out):
+        work[key].append((n * k + 8.0 * n + 2.0 * rows * (k + n_out), 2.0 * rows * n * k))
+
+    for _ in range(s["layers"]):
+        gemm("b200.qkv_rope_append", w + 2 * kv, w, w + 2 * kv)
+        work["b200.paged_attention_decode_batch.persistent_shared"].append(
+            (2.0 * (cached_rows * 2 * kv + 2 * rows * w), 4.0 * rows * w * keys_per_row))
+        gemm("b200.qgemv.int8.residual", w, w, 2 * w)
+        gemm("b200.qgemv.int8.swiglu", 2 * ff, w, ff)
+        gemm("b200.qgemv.int8.residual", w, ff, 2 * w)
+        work["b200.rms_norm_quantize"] += [(rows * w * 4.0, 0.0)] * 2
+    work["b200.rms_norm_quantize"].append((rows * w * 4.0, 0.0))
+    gemm("b200.qgemv.int8", s["vocab"], w, s["vocab"])
+    return work
+
+
+def against_roofline(times: dict[str, tuple[int, float]], work: dict, hbm_gbs: float, tflops: float) -> list[dict]:
+    out = []
+    for key, (n, us) in sorted(times.items(), key=lambda kv: -kv[1][1]):
+        ideal = sum(max(b / hbm_gbs / 1e3, f / tflops / 1e6) for b, f in work.get(key, []))
+        memory = sum(b / hbm_gbs / 1e3 for b, _ in work.get(key, []))
+        out.append({"kernel": key.replace("b200.", ""), "launches": n, "us": round(us / n, 2), "us_per_step": round(us, 1),
+                    "bound": "hbm" if memory >= ideal * 0.999 else "tensor", "frac_of_roofline": round(ideal / us, 3) if ideal else None})
+    return out
+
+
+def run(size: str, batch: int, ctx: int, prompt: int, steps: int, peaks: dict) -> dict:
+    import torch
+
+    s = SIZES[size]
+    hbm, tf = peaks["hbm_gbs"], peaks["bf16_tflops"]
+    line: dict = {"size": size, **s, "batch": batch, "ctx": ctx, "prompt": prompt}
+    for family in ("gutorax", "llama-shaped int8"):
+        rt = build(family, s, batch=batch, positions=max(ctx, prompt) + 8 * steps + 64)
+        sessions = fill(rt, batch, ctx)
+        first = [1] * batch
+        torch.cuda.synchronize()
+        rt.decode_greedy_batch(sessions, first, 3)
+        start, stop = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        start.record()
+        rt.decode_greedy_batch(sessions, first, steps)
+        stop.record()
+        torch.cuda.synchronize()
+        ms = start.elapsed_time(stop) / steps
+        seen = ctx + steps // 2
+        plan = rt._engine.plans[("decode", batch)]
+        if family == "gutorax":
+            keys = min(seen, s["window"])
+            decode_kernels = against_roofline(kind_times(plan), gutorax_work(s, batch, batch, keys, batch * keys, True), hbm, tf)
+        else:
+            decode_kernels = against_roofline(kind_times(plan), llama_work(s, batch, seen, batch * seen), hbm, tf)
+        for x in sessions:
+            x.kv_cache.clear()
+        session = rt.fork()
+        ids = [int(t) for t in torch.randint(0, s["vocab"], (prompt,))]
+
+        def prefill():
+            session.kv_cache.clear()
+            if family == "gutorax":
+                session.run_step_batch([session], [ids])
+            else:
+                session.run([ids], mode="prefill")
+        prefill_ms = timed(prefill, 5)
+        if family == "gutorax":
+            plan = rt._engine.portion_plan(prompt, 1, 1)
+            avg = sum(min(i + 1, s["window"]) for i in range(prompt)) / prompt
+            prefill_kernels = against_roofline(kind_times(plan), gutorax_work(s, prompt, 1, avg, prompt, False), hbm, tf)
+        else:      # the last pass of the prompt: 64 rows that attend to all of it
+            plan = rt._engine.prefill_plan(64, 1)
+            prefill_kernels = against_roofline(kind_times(plan), llama_work(s, 64, prompt, prompt), hbm, tf)
+        rt.check_device_status()
+        line[family] = {"decode_ms_per_step": round(ms, 3), "decode_tokens_per_s": round(batch / ms * 1e3, 1),
+                        "prefill_ms": round(prefill_ms, 3), "prefill_tokens_per_s": round(prompt / prefill_ms * 1e3, 1),
+                        "decode_kernels": decode_kernels, "prefill_kernels": prefill_kernels}
+        del rt, sessions, session, plan
+        torch.cuda.empty_cache()
+    return line

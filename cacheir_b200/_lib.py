@@ -158,8 +158,7 @@ HYBRID_SIGNATURES: dict[str, tuple[object, list[object]]] = {
         c_int, [c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_void_p]),
     "cacheir_b200_latent_attention_supported": (c_int, [c_int] * 4),
     "cacheir_b200_latent_attention_splits": (c_int, [c_int] * 5),
-    "cacheir_b200_latent_attention_workspace_bytes": (c_size_t, [c_int] * 4),
-    "cacheir_b200_latent_attention": (c_int, [c_void_p] * 4 + [c_int, c_void_p, c_size_t, c_void_p]),
+    "cacheir_b200_latent_attention": (c_int, [c_void_p] * 4 + [c_int, c_void_p]),
     "cacheir_b200_recurrence_simple": (c_int, [c_void_p, c_void_p]),
     "cacheir_b200_recurrence_step": (c_int, [c_void_p, c_void_p]),
     "cacheir_b200_recurrence_chunked_supported": (c_int, [c_int] * 3),

@@ -191,6 +191,24 @@ dense_gemm_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_const
             static_cast<__nv_bfloat16*>(p.next_out)[static_cast<long long>(t) * p.N + n] = __float2bfloat16_rn(s);
         }
       } else {
+        // what the epilogue multiplies with is loaded for all tokens before anything is stored
+        float f[G];
+        if constexpr (EPI == CACHEIR_B200_DENSE_GATED) {
+#pragma unroll
+          for (int j = 0; j < G; ++j) {
+            const int t = t0 + c0 + j;
+            f[j] = (n_ok && t < p.T) ? __bfloat162float(static_cast<const __nv_bfloat16*>(p.gate)[static_cast<long long>(t) * p.gate_stride + ycol]) : 0.f;
+          }
+        } else if constexpr (EPI == CACHEIR_B200_DENSE_GELU_EMBED) {
+          int64_t id[G];
+#pragma unroll
+          for (int j = 0; j < G; ++j) id[j] = p.ids[min(t0 + c0 + j, p.T - 1)];
+#pragma unroll
+          for (int j = 0; j < G; ++j) {
+            id[j] = min(max(id[j], static_cast<int64_t>(0)), static_cast<int64_t>(p.vocab - 1));
+            f[j] = n_ok ? __bfloat162float(static_cast<const __nv_bfloat16*>(p.table)[id[j] * p.table_stride + p.table_col + n]) : 0.f;
+          }
+        }
 #pragma unroll
         for (int j = 0; j < G; ++j) {
           const int t = t0 + c0 + j;
@@ -202,11 +220,9 @@ dense_gemm_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_const
           } else if constexpr (EPI == CACHEIR_B200_DENSE_SILU) {
             if (n < p.act_cols) y = silu_exact(y);
           } else if constexpr (EPI == CACHEIR_B200_DENSE_GATED) {
-            const float g = __bfloat162float(static_cast<const __nv_bfloat16*>(p.gate)[static_cast<long long>(t) * p.gate_stride + ycol]);
-            y *= sigmoid_exact(g);
+            y *= sigmoid_exact(f[j]);
           } else if constexpr (EPI == CACHEIR_B200_DENSE_GELU_EMBED) {
-            const int64_t id = min(max(p.ids[t], static_cast<int64_t>(0)), static_cast<int64_t>(p.vocab - 1));
-            y = gelu_tanh(y) * __bfloat162float(static_cast<const __nv_bfloat16*>(p.table)[id * p.table_stride + p.table_col + n]);
+            y = gelu_tanh(y) * f[j];
           }
           static_cast<__nv_bfloat16*>(p.y)[static_cast<long long>(t) * p.y_stride + ycol] = __float2bfloat16_rn(y);
         }

@@ -254,20 +254,14 @@ def latent_attention_splits(rows: int, heads: int, window: int, max_pages: int, 
     return int(_lib.load_hybrid().cacheir_b200_latent_attention_splits(rows, heads, window, max_pages, page_size))
 
 
-def latent_attention_workspace_bytes(rows: int, heads: int, kv_rank: int, splits: int) -> int:
-    return int(_lib.load_hybrid().cacheir_b200_latent_attention_workspace_bytes(rows, heads, kv_rank, splits))
-
-
-def latent_attention(a: LatentArgs, q: torch.Tensor, sink: torch.Tensor, out: torch.Tensor, *, splits: int = 1,
-                     workspace: torch.Tensor | None = None) -> torch.Tensor:
+def latent_attention(a: LatentArgs, q: torch.Tensor, sink: torch.Tensor, out: torch.Tensor, *, splits: int = 1) -> torch.Tensor:
     """q [T, heads*(kv_rank + rot_dim)] in latent space, out [T, heads*kv_rank], both dense bf16."""
-    _require_cuda(q, sink, out, workspace)
+    _require_cuda(q, sink, out)
     _f32(sink)
     if not q.is_contiguous() or not out.is_contiguous():
         raise ValueError("latent_attention expects contiguous q and out")
     check(_lib.load_hybrid().cacheir_b200_latent_attention(
-        ctypes.byref(a), q.data_ptr(), sink.data_ptr(), out.data_ptr(), int(splits), _ptr(workspace),
-        0 if workspace is None else workspace.numel() * workspace.element_size(), _stream()), "latent_attention")
+        ctypes.byref(a), q.data_ptr(), sink.data_ptr(), out.data_ptr(), int(splits), _stream()), "latent_attention")
     return out
 
 

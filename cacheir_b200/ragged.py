@@ -252,11 +252,8 @@ def make_plan_class(base: type) -> type:
             uk_t = eng.absorbed_weight(node.inputs[2], heads, dim, rank)
             o_lat = self._scratch("latent_o", heads * rank)
             splits = H.latent_attention_splits(self.batch, heads, int(at["window"]), self.width, eng.page_size) if self.decode else 1
-            ws_bytes = H.latent_attention_workspace_bytes(self.batch, heads, rank, splits)
-            ws = eng.scratch("latent_ws", ws_bytes) if ws_bytes else None
             self._emit(lambda: H.dense_gemm(q, uk_t, q_lat, batch=heads, x_batch_cols=dim + rot, y_batch_cols=rank + rot), "b200.dense_gemm.heads")
-            self._emit(lambda: H.latent_attention(args, q_lat, sink, o_lat, splits=splits, workspace=ws), "b200.latent_attention",
-                       launches=2 if splits > 1 else 1)
+            self._emit(lambda: H.latent_attention(args, q_lat, sink, o_lat, splits=splits), "b200.latent_attention")
             self._emit(lambda: H.dense_gemm(o_lat, uv, out, epilogue=H.DENSE_GATED, batch=heads, x_batch_cols=rank, gate=gate),
                        "b200.dense_gemm.heads_gated")
             self._env[node.outputs[0]] = out

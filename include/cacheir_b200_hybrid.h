@@ -119,12 +119,11 @@ int cacheir_b200_latent_attention_simple(const cacheir_b200_latent_args* a, cons
                                          const void* uv, const float* sink, const void* gate, long long gate_stride, void* out,
                                          void* stream);
 /* Tensor-core form in latent space (bf16): q [rows, heads, kv_rank + rot_dim] (keys' up-projection already absorbed),
- * out [rows, heads, kv_rank]. `splits` > 1 (decode only) needs workspace; 0 = choose. */
+ * out [rows, heads, kv_rank]. `splits` (decode only, at most 8): CTAs that share a sequence's window; 0 = choose. */
 int cacheir_b200_latent_attention_supported(int kv_rank, int rot_dim, int page_size, int dtype);
 int cacheir_b200_latent_attention_splits(int rows, int heads, int window, int max_pages, int page_size);
-size_t cacheir_b200_latent_attention_workspace_bytes(int rows, int heads, int kv_rank, int splits);
 int cacheir_b200_latent_attention(const cacheir_b200_latent_args* a, const void* q, const float* sink, void* out, int splits,
-                                  void* workspace, size_t workspace_bytes, void* stream);
+                                  void* stream);
 
 /* ---- linear recurrence S <- decay S + k v^T, o = S^T q, one float32 state [heads, dim, vdim] per slot ------------- */
 typedef struct {
