@@ -116,6 +116,7 @@ dense_gemm_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_const
   bool ok = true;
   if (warp == 0) {
     if (lane == 0) {
+      int issued = 0;
       for (int i = 0; i < total; ++i) {
         const int s = i % kStages;
         if (i >= kStages && !mbar_wait(smem_u32(&empty[s]), ((i / kStages) & 1) ^ 1, &g_dense_status, (6 << 8) | 1)) break;
@@ -124,7 +125,11 @@ dense_gemm_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_const
         const int k = (kb_begin + i) * kBlockK;
         tma_load_2d(smem_u32(s_w + s * kWBytes), &tmap_w, bar, k, z * p.w_batch_rows + n0);
         tma_load_2d(smem_u32(s_x + s * MT * kBlockK * 2), &tmap_x, bar, z * p.x_batch_cols + k, t0);
+        issued = i + 1;
       }
+      if (issued < total)          // a wait gave up: nothing may still be on its way when the block ends
+        for (int i = issued > kStages ? issued - kStages : 0; i < issued; ++i)
+          mbar_wait(smem_u32(&full[i % kStages]), (i / kStages) & 1, &g_dense_status, (6 << 8) | 4);
     }
     __syncwarp();
   } else if (warp == 1) {

@@ -3,9 +3,9 @@
 // prepare   RMS-norms the latent, turns the rotated parts (rotate-half pairs) and appends one cache row per token.
 // simple    any extents, float32 arithmetic: one CTA per (token, head) absorbs the key up-projection into the query,
 //           attends over the window in latent space, projects the result up and gates it.
-// fast      bf16 tensor cores, flash style, in latent space: all heads share the cached row, so the 16 or 32 rows of a
-//           CTA's tile are (token, head) pairs of neighbouring tokens of one sequence. Half pages of 32 cache rows land
-//           in a ring as TMA boxes of 64 columns (128-byte swizzle: conflict-free ldmatrix). Softmax in float32
+// fast      bf16, 5th-generation tensor cores, in latent space: all heads share the cached row, so the 32 or 64 rows of a
+//           CTA's tile are (token, head) pairs of neighbouring tokens of one sequence. Pages of 64 cache rows land in a
+//           ring as TMA boxes of 64 columns and serve as keys and, read the other way, as values. Softmax in float32
 //           with the sink as the initial maximum and denominator. A decode batch too small for the SMs splits the
 //           window over the CTAs of a cluster, which combine their parts through distributed shared memory.
 #include "hybrid_common.cuh"
@@ -143,26 +143,28 @@ latent_simple_kernel(const cacheir_b200_latent_args a, const T* __restrict__ q, 
 }
 
 // ---- tensor-core form ----------------------------------------------------------------------------------------------
-// 16 warps. Scores: MW bands of 16 rows x KG key groups x 4 quarters of the inner dimension; a warp's part of Q stays in
-// registers for the whole kernel. The quarters meet in shared memory, where warp w finishes rows w MW .. w MW + MW - 1
-// (scale, mask, running maximum and sum, probabilities as bf16). Output: MW bands x 16/MW groups of latent columns.
-constexpr int kThreads = 512;
-constexpr int kHalf = kPage / 2;         // the ring moves half pages, so that it prefetches while a page is in use
-constexpr int kScorePitch = 72;          // floats: conflict-free for the accumulator layout
-constexpr int kProbPitch = 144;          // bytes
+// Per 64-key page:   S [rows, keys] = Q K^T          A = the query tile (M 64), B = the page (N 64)
+//                    O^T [latent, rows] += V^T P^T   A = the same page read MN-major (M 128 latent columns), B = P
+// so the page is used twice as it lies in shared memory and the probabilities go back as the K-major operand that a row's
+// threads write. O^T stays in tensor memory. Its columns are rescaled only when a row's maximum has grown by more than
+// 2^8 since its reference was chosen (a stale reference costs nothing: numerator and denominator share it).
+//   warps 0..3  softmax, rescaling, output (lane quarter = warp)     warp 4  MMA issue, tensor memory     warp 5  copies
+constexpr int kThreads = 192;
 constexpr int kMaxSplits = 8;            // CTAs of a cluster
-constexpr int kMaxStages = 8;
-constexpr int kBoxBytes = kHalf * 128;   // 32 rows x 64 columns
+constexpr int kMaxStages = 6;            // pages in the ring
+constexpr int kBoxBytes = kPage * 128;   // 64 rows x 64 columns
+constexpr float kStale = 8.f;
 
 struct FastParams {
   cacheir_b200_latent_args a;
-  const __nv_bfloat16* q;      // [rows, heads, kv_rank + rot_dim]
   const float* sink;
   __nv_bfloat16* out;          // [rows, heads, kv_rank]
   int heads_per_cta, tokens_per_tile, splits;
   int boxes;                   // 64-column boxes of a cache row
-  int stages;                  // half pages in the ring
-  int ring_bytes;              // ring, at least the combine's float tile
+  int blocks;                  // 128-column blocks of the latent
+  int stages;
+  int ahead;                   // the next page's scores are issued before this page's output (three pages in the ring)
+  int tmem_cols;
 };
 
 __device__ __forceinline__ float ld_peer_f32(uint32_t local_addr, uint32_t rank) {
@@ -176,27 +178,83 @@ __device__ __forceinline__ void cluster_sync_all() {
   asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory");
   asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory");
 }
+__device__ __forceinline__ void mma_f16_ss(uint32_t tmem_d, uint64_t a_desc, uint64_t b_desc, uint32_t idesc, uint32_t accumulate) {
+  asm volatile(
+      "{\n\t.reg .pred p;\n\t"
+      "setp.ne.b32 p, %4, 0;\n\t"
+      "tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, p;\n\t}"
+      ::"r"(tmem_d), "l"(a_desc), "l"(b_desc), "r"(idesc), "r"(accumulate) : "memory");
+}
+// MN-major operand as 128-byte swizzled rows: 64 columns a box, `box` bytes between boxes, 8-row groups 1024 bytes apart
+__device__ __forceinline__ uint64_t smem_desc_mn_sw128(uint32_t addr, uint32_t box) {
+  return static_cast<uint64_t>((addr >> 4) & 0x3FFF) | static_cast<uint64_t>((box >> 4) & 0x3FFF) << 16 |
+         static_cast<uint64_t>(1024 >> 4) << 32 | static_cast<uint64_t>(1) << 46 | static_cast<uint64_t>(2) << 61;
+}
+// 16 lanes x 64 columns in the warp-MMA accumulator order: r[4 j + e] = row lane / 4 + 8 (e / 2), column 8 j + 2 (lane % 4) + e % 2
+__device__ __forceinline__ void tmem_ld_rows16(uint32_t taddr, float (&v)[32]) {
+  uint32_t r[32];
+  asm volatile(
+      "tcgen05.ld.sync.aligned.16x256b.x8.b32 {%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,%16,%17,%18,%19,%20,%21,%22,%23,%24,"
+      "%25,%26,%27,%28,%29,%30,%31}, [%32];"
+      : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]), "=r"(r[4]), "=r"(r[5]), "=r"(r[6]), "=r"(r[7]), "=r"(r[8]), "=r"(r[9]),
+        "=r"(r[10]), "=r"(r[11]), "=r"(r[12]), "=r"(r[13]), "=r"(r[14]), "=r"(r[15]), "=r"(r[16]), "=r"(r[17]), "=r"(r[18]),
+        "=r"(r[19]), "=r"(r[20]), "=r"(r[21]), "=r"(r[22]), "=r"(r[23]), "=r"(r[24]), "=r"(r[25]), "=r"(r[26]), "=r"(r[27]),
+        "=r"(r[28]), "=r"(r[29]), "=r"(r[30]), "=r"(r[31])
+      : "r"(taddr) : "memory");
+  ptx::tc_wait_ld();
+#pragma unroll
+  for (int i = 0; i < 32; ++i) v[i] = __uint_as_float(r[i]);
+}
+__device__ __forceinline__ void tmem_ld_x16(uint32_t taddr, float (&v)[16]) {
+  uint32_t r[16];
+  asm volatile(
+      "tcgen05.ld.sync.aligned.32x32b.x16.b32 {%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15}, [%16];"
+      : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]), "=r"(r[4]), "=r"(r[5]), "=r"(r[6]), "=r"(r[7]), "=r"(r[8]), "=r"(r[9]),
+        "=r"(r[10]), "=r"(r[11]), "=r"(r[12]), "=r"(r[13]), "=r"(r[14]), "=r"(r[15])
+      : "r"(taddr) : "memory");
+  ptx::tc_wait_ld();
+#pragma unroll
+  for (int i = 0; i < 16; ++i) v[i] = __uint_as_float(r[i]);
+}
+__device__ __forceinline__ void tmem_st_x16(uint32_t taddr, const float (&v)[16]) {
+  asm volatile(
+      "tcgen05.st.sync.aligned.32x32b.x16.b32 [%0], {%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,%16};"
+      ::"r"(taddr), "f"(v[0]), "f"(v[1]), "f"(v[2]), "f"(v[3]), "f"(v[4]), "f"(v[5]), "f"(v[6]), "f"(v[7]), "f"(v[8]), "f"(v[9]), "f"(v[10]),
+      "f"(v[11]), "f"(v[12]), "f"(v[13]), "f"(v[14]), "f"(v[15]) : "memory");
+}
+// true in all 128 softmax threads if `p` holds in one of them
+__device__ __forceinline__ bool any_of_128(bool p) {
+  uint32_t out;
+  asm volatile(
+      "{\n\t.reg .pred a, b;\n\t"
+      "setp.ne.u32 a, %1, 0;\n\t"
+      "barrier.cta.red.or.pred b, 1, 128, a;\n\t"
+      "selp.u32 %0, 1, 0, b;\n\t}"
+      : "=r"(out) : "r"(static_cast<uint32_t>(p)) : "memory");
+  return out != 0;
+}
+__device__ __forceinline__ void sync_128() { asm volatile("barrier.cta.sync 1, 128;" ::: "memory"); }
 
-// RANKMAX: latent columns the accumulators have room for; KSQ: 16-wide inner steps of a quarter
-template <int MW, int RANKMAX, int KSQ>
+template <int NR>
 __global__ void __launch_bounds__(kThreads, 1)
-latent_attention_kernel(const __grid_constant__ CUtensorMap tmap, const FastParams p) {
-  constexpr int MROWS = MW * 16;
-  constexpr int KG = 4 / MW;               // key groups of a page
-  constexpr int NT = 8 / KG;               // 8-key score tiles per warp
-  constexpr int CW = 16 / MW;              // column groups
-  constexpr int PW = (RANKMAX / 16 + CW - 1) / CW;
+latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_kv, const __grid_constant__ CUtensorMap tmap_q, const FastParams p) {
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~static_cast<uintptr_t>(1023));
   const cacheir_b200_latent_args& a = p.a;
+  const int page_bytes = p.boxes * kBoxBytes;
   const int width = a.kv_rank + a.rot_dim;
-  uint8_t* s_kv = smem;                                                      // [stages][boxes][32 rows][128 bytes], swizzled
-  const int half_bytes = p.boxes * kBoxBytes;
-  float* s_score = reinterpret_cast<float*>(smem + p.ring_bytes);            // [4][MROWS][kScorePitch]
-  uint8_t* s_p = reinterpret_cast<uint8_t*>(s_score + 4 * MROWS * kScorePitch);   // [MROWS][kProbPitch]
-  float* s_alpha = reinterpret_cast<float*>(s_p + MROWS * kProbPitch);       // [MROWS]
-  float* s_ml = s_alpha + MROWS;                                             // [MROWS][2]
-  uint64_t* bars = reinterpret_cast<uint64_t*>(s_ml + 2 * MROWS);            // [stages]
+  uint8_t* s_kv = smem;                                         // [stages][boxes][64 rows][128 bytes], swizzled
+  uint8_t* s_q = s_kv + p.stages * page_bytes;                  // [boxes][NR rows][128 bytes], swizzled
+  uint8_t* s_p = s_q + p.boxes * NR * 128;                      // [1 + ahead][NR rows][128 bytes], swizzled
+  float* s_alpha = reinterpret_cast<float*>(s_p + (1 + p.ahead) * NR * 128);   // [NR]
+  float* s_ml = s_alpha + NR;                                   // [NR][2]
+  uint64_t* full = reinterpret_cast<uint64_t*>(s_ml + 2 * NR);  // [stages] a page has landed
+  uint64_t* empty = full + kMaxStages;                          // [stages] its output MMAs have retired
+  uint64_t* bar_q = empty + kMaxStages;
+  uint64_t* bar_s = bar_q + 1;                                  // [2] scores in tensor memory
+  uint64_t* bar_p = bar_s + 2;                                  // [2] probabilities in shared memory
+  uint64_t* bar_o = bar_p + 2;                                  // the output MMAs of one more page have retired
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bar_o + 1);
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int head0 = blockIdx.y * p.heads_per_cta;
@@ -214,296 +272,336 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap, const FastPara
   }
   const int pos0 = a.positions[row0];
   const int pos_last = pos0 + ntok - 1;
-  const int used = ntok * nheads;          // tile row = token * nheads + head
+  const int used = ntok * nheads;          // tile row = token * nheads + head: neighbouring rows of q
   // pages of this tile's keys, cut evenly over the splits
   const int key_lo = max(0, pos0 - a.window + 1);
   const int page_lo = key_lo / kPage, pages = pos_last / kPage - page_lo + 1;
   const int pg_begin = page_lo + pages * split / p.splits;
   const int npages = page_lo + pages * (split + 1) / p.splits - pg_begin;
 
-  auto page_slot = [&](int pg) {
-    const int slot = pg < a.max_pages ? a.page_table[static_cast<size_t>(seg) * a.max_pages + pg] : 0;
-    return min(max(slot, 0), a.num_slots - 1);
-  };
-  // One box of a half page. Rows that nobody attends to come along (their probabilities are zero), columns beyond the
-  // cache row read as zero.
-  auto load_box = [&](int stage, int slot, int half, int box) {
-    const uint32_t bar = smem_addr(&bars[stage]);
-    if (box == 0) ptx::mbar_expect_tx(bar, half_bytes);
-    ptx::tma_load_2d(smem_addr(s_kv + stage * half_bytes + box * kBoxBytes), &tmap, bar, box * 64, slot * kPage + half * kHalf);
-  };
   if (threadIdx.x == 0) {
-    for (int s = 0; s < p.stages; ++s) ptx::mbar_init(smem_addr(&bars[s]), 1);
+    for (int s = 0; s < p.stages; ++s) { ptx::mbar_init(smem_addr(&full[s]), 1); ptx::mbar_init(smem_addr(&empty[s]), 1); }
+    ptx::mbar_init(smem_addr(bar_q), 1);
+    for (int s = 0; s < 2; ++s) { ptx::mbar_init(smem_addr(&bar_s[s]), 1); ptx::mbar_init(smem_addr(&bar_p[s]), 128); }
+    ptx::mbar_init(smem_addr(bar_o), 1);
     ptx::mbar_fence_init();
   }
+  if (warp == 4) ptx::tc_alloc(smem_addr(tmem_slot), p.tmem_cols);
+  ptx::tc_fence_before();
   __syncthreads();
-  // boxes are dealt over the warps: this warp's lane 0 requests boxes warp, warp + 16 of the 2 * boxes of a page pair
-  const int pre = min(p.stages, 2 * npages);
-  if (lane == 0)
-    for (int b = warp; b < pre * p.boxes; b += 16) {
-      const int j = b / p.boxes;
-      load_box(j, page_slot(pg_begin + (j >> 1)), j & 1, b - j * p.boxes);
-    }
-  const int hi_box = warp >= p.boxes ? 1 : 0;      // which of the two halves box `warp` belongs to, box warp + 16 the second
-  // half page j = 2 it - 2 + stages (+1) goes where half page 2 it - 2 (+1) was
-  int next_slot[2];
-#pragma unroll
-  for (int u = 0; u < 2; ++u) next_slot[u] = page_slot(pg_begin + ((p.stages + (u ? 1 : hi_box)) >> 1));
+  ptx::tc_fence_after();
+  const uint32_t tmem = *tmem_slot;
+  const uint32_t tmem_s = tmem + p.blocks * NR;       // scores: two buffers of 64 columns behind the output blocks
+  bool ok = true;
 
-  // roles in the score phase
-  const int kq = warp & 3, band = (warp >> 2) % MW, kg = (warp >> 2) / MW;
-  const int ksteps = (width + 15) / 16;
-  const int k_begin = ksteps * kq / 4, k_count = ksteps * (kq + 1) / 4 - k_begin;
-  uint32_t qf[KSQ][4];
-#pragma unroll
-  for (int k = 0; k < KSQ; ++k)
-#pragma unroll
-    for (int e = 0; e < 4; ++e) {
-      const int r = band * 16 + (lane >> 2) + (e & 1) * 8, c = (k_begin + k) * 16 + (lane & 3) * 2 + (e >> 1) * 8;
-      qf[k][e] = (k < k_count && r < used && c < width)
-                     ? *reinterpret_cast<const uint32_t*>(p.q + (static_cast<size_t>(row0 + r / nheads) * a.heads + head0 + r % nheads) * width + c)
-                     : 0u;
+  if (warp == 5) {
+    // ---------------- copies ----------------
+    if (lane == 0 && npages > 0) {
+      ptx::mbar_expect_tx(smem_addr(bar_q), p.boxes * NR * 128);
+      for (int b = 0; b < p.boxes; ++b)
+        ptx::tma_load_2d(smem_addr(s_q + b * NR * 128), &tmap_q, smem_addr(bar_q), b * 64, row0 * a.heads + head0);
+      int stage = 0, phase = 1;
+      for (int it = 0; it < npages; ++it) {
+        const int pg = pg_begin + it;
+        int slot = pg < a.max_pages ? a.page_table[static_cast<size_t>(seg) * a.max_pages + pg] : 0;
+        slot = min(max(slot, 0), a.num_slots - 1);
+        if (it >= p.stages) ok = ok && ptx::mbar_wait(smem_addr(&empty[stage]), phase, &g_latent_status, (7 << 8) | 1);
+        if (!ok) break;
+        const uint32_t bar = smem_addr(&full[stage]);
+        ptx::mbar_expect_tx(bar, page_bytes);
+        for (int b = 0; b < p.boxes; ++b)
+          ptx::tma_load_2d(smem_addr(s_kv + stage * page_bytes + b * kBoxBytes), &tmap_kv, bar, b * 64, slot * kPage);
+        if (++stage == p.stages) { stage = 0; phase ^= 1; }
+      }
+      // nothing may still be on its way when the block ends, also after a wait that gave up
+      ptx::mbar_wait(smem_addr(bar_q), 0, &g_latent_status, (7 << 8) | 8);
+      if (!ok)
+        for (int s = 0; s < p.stages; ++s) ptx::mbar_wait(smem_addr(&full[s]), s < stage ? phase ^ 1 : phase, &g_latent_status, (7 << 8) | 9);
     }
-  // roles in the softmax phase: rows warp * MW + i
-  float m_run[MW], l_run[MW];
-  int row_pos[MW];
+    __syncwarp();
+  } else if (warp == 4) {
+    // ---------------- MMA issue ----------------
+    if (lane == 0 && npages > 0) {
+      const uint32_t id_s = (1u << 4) | (1u << 7) | (1u << 10) | (static_cast<uint32_t>(kPage >> 3) << 17) | (static_cast<uint32_t>(64 >> 4) << 24);
+      const uint32_t id_o = (1u << 4) | (1u << 7) | (1u << 10) | (1u << 15) | (static_cast<uint32_t>(NR >> 3) << 17) |
+                            (static_cast<uint32_t>(128 >> 4) << 24);
+      const uint64_t dq = ptx::smem_desc_sw128(smem_addr(s_q)), dk = ptx::smem_desc_sw128(smem_addr(s_kv)), dp = ptx::smem_desc_sw128(smem_addr(s_p));
+      const uint64_t dv = smem_desc_mn_sw128(smem_addr(s_kv), kBoxBytes);
+      const int ksteps = (width + 15) / 16;
+      int s_stage = 0, s_phase = 0;          // next page to score
+      auto scores = [&](int it) {
+        ok = ok && ptx::mbar_wait(smem_addr(&full[s_stage]), s_phase, &g_latent_status, (7 << 8) | 2);
+        ptx::tc_fence_after();
+        const uint64_t k0 = dk + static_cast<uint64_t>(s_stage * page_bytes >> 4);
+        const uint32_t d = tmem_s + (it & 1) * kPage;
+        int k = 0;
+        for (int b = 0; b < p.boxes; ++b) {
+          const uint64_t aq = dq + static_cast<uint64_t>(b * (NR * 128 >> 4)), bk = k0 + static_cast<uint64_t>(b * (kBoxBytes >> 4));
 #pragma unroll
-  for (int i = 0; i < MW; ++i) {
-    const int r = warp * MW + i;
-    const bool real = r < used;
-    row_pos[i] = real ? pos0 + r / nheads : -1;
-    m_run[i] = (real && split == 0) ? p.sink[head0 + r % nheads] * kLog2e : -1e30f;
-    l_run[i] = (real && split == 0 && lane == 0) ? 1.f : 0.f;
-  }
-  const float qscale = a.scale * kLog2e;
-  // roles in the output phase
-  const int oband = warp % MW, cw = warp / MW;
-  const int pairs = a.kv_rank / 16, pair0 = cw * PW;
-  float acc[PW][2][4];
+          for (int j = 0; j < 4; ++j, ++k)
+            if (k < ksteps) mma_f16_ss(d, aq + 2 * j, bk + 2 * j, id_s, k > 0 ? 1u : 0u);
+        }
+        ptx::tc_commit(smem_addr(&bar_s[it & 1]));
+        if (++s_stage == p.stages) { s_stage = 0; s_phase ^= 1; }
+      };
+      ok = ptx::mbar_wait(smem_addr(bar_q), 0, &g_latent_status, (7 << 8) | 3);
+      scores(0);
+      int o_stage = 0;
+      for (int it = 0; it < npages && ok; ++it) {
+        if (p.ahead && it + 1 < npages) scores(it + 1);
+        ok = ok && ptx::mbar_wait(smem_addr(&bar_p[it & 1]), (it >> 1) & 1, &g_latent_status, (7 << 8) | 4);
+        ptx::tc_fence_after();
+        const uint64_t v0 = dv + static_cast<uint64_t>(o_stage * page_bytes >> 4);
+        const uint64_t pb = dp + static_cast<uint64_t>((p.ahead ? it & 1 : 0) * (NR * 128 >> 4));
+        for (int m = 0; m < p.blocks; ++m) {
+          const uint64_t av = v0 + static_cast<uint64_t>(m * (2 * kBoxBytes >> 4));
 #pragma unroll
-  for (int i = 0; i < PW; ++i)
+          for (int j = 0; j < 4; ++j)        // 16 keys
+            mma_f16_ss(tmem + m * NR, av + j * (2048 >> 4), pb + 2 * j, id_o, (it > 0 || j > 0) ? 1u : 0u);
+        }
+        ptx::tc_commit(smem_addr(&empty[o_stage]));
+        ptx::tc_commit(smem_addr(bar_o));
+        if (++o_stage == p.stages) o_stage = 0;
+        if (!p.ahead && it + 1 < npages) scores(it + 1);
+      }
+    }
+    __syncwarp();
+  } else {
+    // ---------------- softmax: rows r0 = 16 warp + lane / 4 and r0 + 8, columns 8 j + 2 (lane % 4) + {0, 1} ----------------
+    const bool band = warp * 16 < NR;        // (a 32-row tile keeps two of the four warps for the rescaling only)
+    float m_ref[2], l_run[2];
+    int row_pos[2];
 #pragma unroll
-    for (int j = 0; j < 2; ++j)
+    for (int e = 0; e < 2; ++e) {
+      const int r = warp * 16 + (lane >> 2) + 8 * e;
+      const bool real = band && r < used;
+      row_pos[e] = real ? pos0 + r / nheads : -1;
+      m_ref[e] = (real && split == 0) ? p.sink[head0 + r % nheads] * kLog2e : -1e30f;
+      l_run[e] = (real && split == 0 && (lane & 3) == 0) ? 1.f : 0.f;
+    }
+    const float qscale = a.scale * kLog2e;
+    const uint32_t lane_addr = static_cast<uint32_t>(warp * 32) << 16;
+    int stage = 0;
+    for (int it = 0; it < npages; ++it) {
+      const int buf = p.ahead ? it & 1 : 0;
+      ok = ok && ptx::mbar_wait(smem_addr(&bar_s[it & 1]), (it >> 1) & 1, &g_latent_status, (7 << 8) | 5);
+      __syncwarp();
+      ptx::tc_fence_after();
+      float s[32], alpha[2] = {1.f, 1.f};
+      bool grown = false;
+      if (band) {
+        tmem_ld_rows16(tmem_s + (it & 1) * kPage + lane_addr, s);
+        const int base = (pg_begin + it) * kPage;
+        float mx[2] = {-1e30f, -1e30f};
+        if (base + kPage - 1 <= pos0 && base > pos_last - a.window) {      // the whole page is seen by every row
 #pragma unroll
-      for (int e = 0; e < 4; ++e) acc[i][j][e] = 0.f;
-
-  int free0 = 0, free1 = 0;                // stages of the previous page
-  int st0 = 0, parity0 = 0;                // stage and phase of the current page's first half
-  for (int it = 0; it < npages; ++it) {
-    const bool wrap1 = st0 + 1 == p.stages;
-    const int st1 = wrap1 ? 0 : st0 + 1, parity1 = parity0 ^ (wrap1 ? 1 : 0);
-    ptx::mbar_wait(smem_addr(&bars[st0]), parity0, &g_latent_status, (7 << 8) | 1);
-    ptx::mbar_wait(smem_addr(&bars[st1]), parity1, &g_latent_status, (7 << 8) | 2);
-    const uint32_t kv0 = smem_addr(s_kv) + st0 * half_bytes, kv1 = smem_addr(s_kv) + st1 * half_bytes;
-    {
-      float s[NT][4];
+          for (int i = 0; i < 32; ++i) {
+            s[i] *= qscale;
+            mx[(i >> 1) & 1] = fmaxf(mx[(i >> 1) & 1], s[i]);
+          }
+        } else {
 #pragma unroll
-      for (int t = 0; t < NT; ++t)
+          for (int i = 0; i < 32; ++i) {
+            const int key = base + (i >> 2) * 8 + (lane & 3) * 2 + (i & 1), rp = row_pos[(i >> 1) & 1];
+            s[i] = (key <= rp && key > rp - a.window) ? s[i] * qscale : -INFINITY;
+            mx[(i >> 1) & 1] = fmaxf(mx[(i >> 1) & 1], s[i]);
+          }
+        }
 #pragma unroll
-        for (int e = 0; e < 4; ++e) s[t][e] = 0.f;
-      const int key0 = kg * NT * 8;        // a group lies inside one half
-      const uint32_t ka = (key0 < kHalf ? kv0 : kv1) + ((key0 % kHalf) + (lane & 7) + ((lane >> 4) << 3)) * 128;
-#pragma unroll
-      for (int k = 0; k < KSQ; ++k) {
-        if (k < k_count) {                  // (the same for all warps up to one step)
-          const int chunk = 2 * (k_begin + k) + ((lane >> 3) & 1);        // 16-byte pieces of the row
-          const uint32_t kc = ka + (chunk >> 3) * kBoxBytes + (((chunk ^ lane) & 7) << 4);
-#pragma unroll
-          for (int t = 0; t < NT; t += 2) {
-            uint32_t bf[4];
-            ldsm_x4(kc + t * 8 * 128, bf);
-            mma_bf16(s[t], qf[k], bf[0], bf[1]);
-            mma_bf16(s[t + 1], qf[k], bf[2], bf[3]);
+        for (int e = 0; e < 2; ++e) {
+          mx[e] = fmaxf(mx[e], __shfl_xor_sync(0xffffffffu, mx[e], 1));
+          mx[e] = fmaxf(mx[e], __shfl_xor_sync(0xffffffffu, mx[e], 2));
+          if (row_pos[e] >= 0 && (it == 0 ? mx[e] > m_ref[e] : mx[e] > m_ref[e] + kStale)) {
+            alpha[e] = exp2f(m_ref[e] - mx[e]);
+            m_ref[e] = mx[e];
+            grown = it > 0;
           }
         }
       }
-      float* dst = s_score + (kq * MROWS + band * 16 + (lane >> 2)) * kScorePitch + key0 + (lane & 3) * 2;
-#pragma unroll
-      for (int t = 0; t < NT; ++t) {
-        *reinterpret_cast<float2*>(dst + t * 8) = make_float2(s[t][0], s[t][1]);
-        *reinterpret_cast<float2*>(dst + 8 * kScorePitch + t * 8) = make_float2(s[t][2], s[t][3]);
+      const int tail = pos_last + 1 - (pg_begin + it) * kPage;
+      if (tail < kPage) {                    // rows behind the last token may hold anything: zero, so that 0 * row stays 0
+        for (int i = threadIdx.x; i < (kPage - tail) * p.boxes * 8; i += 128) {
+          const int r = tail + i / (p.boxes * 8), c = i % (p.boxes * 8);
+          *reinterpret_cast<uint4*>(s_kv + stage * page_bytes + (c >> 3) * kBoxBytes + r * 128 + (c & 7) * 16) = make_uint4(0u, 0u, 0u, 0u);
+        }
+        asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
       }
-    }
-    __syncthreads();                       // scores complete; everyone has left the previous page
-    if (it > 0) {                          // the previous page's halves are free: every warp requests a box or two
-      const int j0 = 2 * it - 2 + p.stages;
-      if (lane == 0) {
+      if (++stage == p.stages) stage = 0;
+      if (any_of_128(grown)) {               // rare: bring O^T to the new references
+        if (band && (lane & 3) == 0) {
 #pragma unroll
-        for (int u = 0; u < 2; ++u) {
-          const int b = warp + 16 * u, h = u ? 1 : hi_box;
-          if (b < 2 * p.boxes && j0 + h < 2 * npages) load_box(h ? free1 : free0, next_slot[u], (j0 + h) & 1, b - h * p.boxes);
+          for (int e = 0; e < 2; ++e) s_alpha[warp * 16 + (lane >> 2) + 8 * e] = alpha[e];
+        }
+        ok = ok && ptx::mbar_wait(smem_addr(bar_o), (it - 1) & 1, &g_latent_status, (7 << 8) | 6);     // the page before is in
+        ptx::tc_fence_after();
+        sync_128();
+        for (int c = 0; c < p.blocks * NR; c += 16) {
+          float o[16];
+          tmem_ld_x16(tmem + lane_addr + c, o);
+#pragma unroll
+          for (int j = 0; j < 16; ++j) o[j] *= s_alpha[(c + j) % NR];
+          tmem_st_x16(tmem + lane_addr + c, o);
+        }
+        asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory");
+        sync_128();                          // s_alpha may be written again
+      }
+      if (band) {
+#pragma unroll
+        for (int e = 0; e < 2; ++e) l_run[e] *= alpha[e];
+        uint8_t* dst = s_p + (buf * NR + warp * 16 + (lane >> 2)) * 128 + (lane & 3) * 4;
+        const int swz = lane >> 2;           // row % 8 of both rows
+#pragma unroll
+        for (int j = 0; j < 8; ++j) {
+#pragma unroll
+          for (int e = 0; e < 4; ++e) {
+            s[4 * j + e] = (e < 2 ? row_pos[0] : row_pos[1]) >= 0 ? exp2f(s[4 * j + e] - m_ref[e >> 1]) : 0.f;
+            l_run[e >> 1] += s[4 * j + e];
+          }
+          *reinterpret_cast<uint32_t*>(dst + ((j ^ swz) << 4)) = pack_bf16(s[4 * j], s[4 * j + 1]);
+          *reinterpret_cast<uint32_t*>(dst + 8 * 128 + ((j ^ swz) << 4)) = pack_bf16(s[4 * j + 2], s[4 * j + 3]);
+        }
+        asm volatile("fence.proxy.async.shared::cta;" ::: "memory");       // the tensor core reads what was just written
+      }
+      ptx::tc_fence_before();
+      ptx::mbar_arrive(smem_addr(&bar_p[it & 1]));
+    }
+    // row sums and references
+    if (band) {
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        l_run[e] += __shfl_xor_sync(0xffffffffu, l_run[e], 1);
+        l_run[e] += __shfl_xor_sync(0xffffffffu, l_run[e], 2);
+        if ((lane & 3) == 0) {
+          s_ml[(warp * 16 + (lane >> 2) + 8 * e) * 2] = m_ref[e];
+          s_ml[(warp * 16 + (lane >> 2) + 8 * e) * 2 + 1] = p.splits == 1 ? 1.f / l_run[e] : l_run[e];
         }
       }
-#pragma unroll
-      for (int u = 0; u < 2; ++u) next_slot[u] = page_slot(pg_begin + ((j0 + 2 + (u ? 1 : hi_box)) >> 1));
     }
-    free0 = st0;
-    free1 = st1;
-    st0 = st1 + 1 == p.stages ? 0 : st1 + 1;
-    parity0 = parity1 ^ (st0 == 0 ? 1 : 0);
-    const int key = (pg_begin + it) * kPage + lane * 2;
-    float2 v[MW];
-    float mx[MW], alpha[MW];
+    if (npages > 0) ok = ok && ptx::mbar_wait(smem_addr(bar_o), (npages - 1) & 1, &g_latent_status, (7 << 8) | 7);
+    __syncwarp();
+    ptx::tc_fence_after();
+    sync_128();                              // s_ml is complete, every page has been read
+    // O^T: lane = latent column of the block, tensor-memory column = tile row
+    float* s_o = reinterpret_cast<float*>(smem);
+    const int opitch = a.kv_rank + 8;
+    for (int m = 0; m < p.blocks; ++m) {
+      const int col = m * 128 + warp * 32 + lane;
+      for (int c = 0; c < NR; c += 16) {
+        if (c >= used) break;
+        float o[16];
+        if (npages > 0) {
+          tmem_ld_x16(tmem + lane_addr + m * NR + c, o);
+        } else {
 #pragma unroll
-    for (int i = 0; i < MW; ++i) v[i] = *reinterpret_cast<const float2*>(s_score + (warp * MW + i) * kScorePitch + lane * 2);
-#pragma unroll
-    for (int part = 1; part < 4; ++part)
-#pragma unroll
-      for (int i = 0; i < MW; ++i) {
-        const float2 x = *reinterpret_cast<const float2*>(s_score + (part * MROWS + warp * MW + i) * kScorePitch + lane * 2);
-        v[i].x += x.x; v[i].y += x.y;
-      }
-#pragma unroll
-    for (int i = 0; i < MW; ++i) {
-      v[i].x = (key <= row_pos[i] && key > row_pos[i] - a.window) ? v[i].x * qscale : -INFINITY;
-      v[i].y = (key + 1 <= row_pos[i] && key + 1 > row_pos[i] - a.window) ? v[i].y * qscale : -INFINITY;
-      mx[i] = fmaxf(v[i].x, v[i].y);
-    }
-#pragma unroll
-    for (int off = 16; off > 0; off >>= 1)
-#pragma unroll
-      for (int i = 0; i < MW; ++i) mx[i] = fmaxf(mx[i], __shfl_xor_sync(0xffffffffu, mx[i], off));
-#pragma unroll
-    for (int i = 0; i < MW; ++i) {
-      const int r = warp * MW + i;
-      mx[i] = fmaxf(mx[i], m_run[i]);
-      alpha[i] = exp2f(m_run[i] - mx[i]);
-      v[i].x = exp2f(v[i].x - mx[i]);
-      v[i].y = exp2f(v[i].y - mx[i]);
-      m_run[i] = mx[i];
-      *reinterpret_cast<uint32_t*>(s_p + r * kProbPitch + lane * 4) = pack_bf16(v[i].x, v[i].y);
-      if (lane == 0) s_alpha[r] = alpha[i];
-      l_run[i] = fmaf(l_run[i], alpha[i], v[i].x + v[i].y);
-    }
-    __syncthreads();                       // probabilities complete
-    const float f0 = s_alpha[oband * 16 + (lane >> 2)], f1 = s_alpha[oband * 16 + (lane >> 2) + 8];
-    if (__any_sync(0xffffffffu, f0 != 1.f || f1 != 1.f)) {
-#pragma unroll
-      for (int i = 0; i < PW; ++i)
-#pragma unroll
-        for (int j = 0; j < 2; ++j) {
-          acc[i][j][0] *= f0; acc[i][j][1] *= f0;
-          acc[i][j][2] *= f1; acc[i][j][3] *= f1;
+          for (int j = 0; j < 16; ++j) o[j] = 0.f;
         }
-    }
-    const uint32_t pa = smem_addr(s_p) + (oband * 16 + (lane & 15)) * kProbPitch + (lane >> 4) * 16;
-    const uint32_t voff = ((lane & 7) + ((lane >> 3) & 1) * 8) * 128;
+        if (col >= a.kv_rank) {
+        } else if (p.splits == 1) {
+          __nv_bfloat16* dst = p.out + (static_cast<size_t>(row0) * a.heads + head0 + c) * a.kv_rank + col;
 #pragma unroll
-    for (int k = 0; k < kPage / 16; ++k) {
-      uint32_t af[4], bf[PW][4];
-      ldsm_x4(pa + k * 32, af);
-      const uint32_t va = (k < 2 ? kv0 : kv1) + (k & 1) * 16 * 128 + voff;
+          for (int j = 0; j < 16; ++j)
+            if (c + j < used) dst[static_cast<size_t>(j) * a.kv_rank] = __float2bfloat16_rn(o[j] * s_ml[(c + j) * 2 + 1]);
+        } else {
 #pragma unroll
-      for (int i = 0; i < PW; ++i) {
-        const int chunk = 2 * min(pair0 + i, pairs - 1) + (lane >> 4);      // (columns beyond the latent are not stored)
-        ldsm_x4_t(va + (chunk >> 3) * kBoxBytes + (((chunk ^ lane) & 7) << 4), bf[i]);
-      }
-#pragma unroll
-      for (int i = 0; i < PW; ++i) {
-        mma_bf16(acc[i][0], af, bf[i][0], bf[i][1]);
-        mma_bf16(acc[i][1], af, bf[i][2], bf[i][3]);
+          for (int j = 0; j < 16; ++j) s_o[(c + j) * opitch + col] = o[j];
+        }
+        __syncwarp();
       }
     }
   }
-
-  // row sums and maxima
+  if (p.splits > 1) {
+    // the cluster's CTAs share one tile: rows dealt out, parts added in rank order
+    __syncwarp();
+    cluster_sync_all();
+    float* s_o = reinterpret_cast<float*>(smem);
+    const int opitch = a.kv_rank + 8;
+    for (int r = split; r < used; r += p.splits) {
+      float m[kMaxSplits], top = -1e30f, l = 0.f;
 #pragma unroll
-  for (int i = 0; i < MW; ++i) {
-    const float l = warp_sum(l_run[i]);
-    if (lane == 0) {
-      s_ml[(warp * MW + i) * 2] = m_run[i];
-      s_ml[(warp * MW + i) * 2 + 1] = l;
+      for (int s = 0; s < kMaxSplits; ++s) {
+        m[s] = s < p.splits ? ld_peer_f32(smem_addr(s_ml + r * 2), s) : -1e30f;
+        top = fmaxf(top, m[s]);
+      }
+#pragma unroll
+      for (int s = 0; s < kMaxSplits; ++s) {
+        m[s] = exp2f(m[s] - top);
+        if (s < p.splits) l = fmaf(ld_peer_f32(smem_addr(s_ml + r * 2 + 1), s), m[s], l);
+      }
+      const float inv = 1.f / l;
+      __nv_bfloat16* dst = p.out + (static_cast<size_t>(row0) * a.heads + head0 + r) * a.kv_rank;
+      for (int c = threadIdx.x; c < a.kv_rank; c += kThreads) {
+        float v = 0.f;
+#pragma unroll
+        for (int s = 0; s < kMaxSplits; ++s)
+          if (s < p.splits) v = fmaf(ld_peer_f32(smem_addr(s_o + r * opitch + c), s), m[s], v);
+        dst[c] = __float2bfloat16_rn(v * inv);
+      }
     }
+    cluster_sync_all();                    // nobody leaves while its part is being read
   }
-  __syncthreads();                         // (also: the ring is free)
-  if (p.splits == 1) {
-#pragma unroll
-    for (int e = 0; e < 2; ++e) {
-      const int r = oband * 16 + (lane >> 2) + e * 8;
-      if (r >= used) continue;
-      const float inv = 1.f / s_ml[r * 2 + 1];
-      __nv_bfloat16* dst = p.out + (static_cast<size_t>(row0 + r / nheads) * a.heads + head0 + r % nheads) * a.kv_rank + (lane & 3) * 2;
-#pragma unroll
-      for (int i = 0; i < PW; ++i)
-        if (pair0 + i < pairs)
-#pragma unroll
-          for (int j = 0; j < 2; ++j)
-            *reinterpret_cast<uint32_t*>(dst + (pair0 + i) * 16 + j * 8) = pack_bf16(acc[i][j][e * 2] * inv, acc[i][j][e * 2 + 1] * inv);
-    }
-    return;
+  ptx::tc_fence_before();
+  __syncthreads();
+  if (warp == 4) {
+    ptx::tc_fence_after();
+    ptx::tc_dealloc(tmem, p.tmem_cols);
   }
-  // the cluster's CTAs share one tile: partial outputs in shared memory, rows dealt out, parts added in rank order
-  const int opitch = a.kv_rank + 8;
-  float* s_o = reinterpret_cast<float*>(smem);
-#pragma unroll
-  for (int e = 0; e < 2; ++e) {
-    float* dst = s_o + (oband * 16 + (lane >> 2) + e * 8) * opitch + (lane & 3) * 2;
-#pragma unroll
-    for (int i = 0; i < PW; ++i)
-      if (pair0 + i < pairs)
-#pragma unroll
-        for (int j = 0; j < 2; ++j)
-          *reinterpret_cast<float2*>(dst + (pair0 + i) * 16 + j * 8) = make_float2(acc[i][j][e * 2], acc[i][j][e * 2 + 1]);
-  }
-  cluster_sync_all();
-  for (int r = split; r < used; r += p.splits) {
-    float m[kMaxSplits], top = -1e30f, l = 0.f;
-#pragma unroll
-    for (int s = 0; s < kMaxSplits; ++s) {
-      m[s] = s < p.splits ? ld_peer_f32(smem_addr(s_ml + r * 2), s) : -1e30f;
-      top = fmaxf(top, m[s]);
-    }
-#pragma unroll
-    for (int s = 0; s < kMaxSplits; ++s) {
-      m[s] = exp2f(m[s] - top);
-      if (s < p.splits) l = fmaf(ld_peer_f32(smem_addr(s_ml + r * 2 + 1), s), m[s], l);
-    }
-    const float inv = 1.f / l;
-    __nv_bfloat16* dst = p.out + (static_cast<size_t>(row0 + r / nheads) * a.heads + head0 + r % nheads) * a.kv_rank;
-    for (int c = threadIdx.x; c < a.kv_rank; c += kThreads) {
-      float v = 0.f;
-#pragma unroll
-      for (int s = 0; s < kMaxSplits; ++s)
-        if (s < p.splits) v = fmaf(ld_peer_f32(smem_addr(s_o + r * opitch + c), s), m[s], v);
-      dst[c] = __float2bfloat16_rn(v * inv);
-    }
-  }
-  cluster_sync_all();                      // nobody leaves while its part is being read
 }
 
-int row_boxes(int width) { return (width + 63) / 64; }
-// shared memory beside the ring
-size_t fast_fixed_smem(int mrows) { return 1024 + static_cast<size_t>(mrows) * (4 * kScorePitch * 4 + kProbPitch + 12) + 16 + kMaxStages * 8; }
 constexpr size_t kSmemLimit = 227 * 1024;
-int fast_stages(int mrows, int width) {
-  const int s = static_cast<int>((kSmemLimit - fast_fixed_smem(mrows)) / (static_cast<size_t>(row_boxes(width)) * kBoxBytes));
-  return s > kMaxStages ? kMaxStages : s;
+int row_boxes(int width) { return (width + 63) / 64; }
+// Shared memory beside the ring, and the ring's pages: `ahead` when three fit.
+size_t fast_fixed_smem(int nr, int boxes, int ahead) {
+  return 1024 + static_cast<size_t>(boxes + 1 + ahead) * nr * 128 + nr * 12 + (2 * kMaxStages + 6) * 8 + 16;
 }
-int head_groups(int heads) { return (heads + 31) / 32; }
+struct Ring { int stages, ahead; };
+Ring fast_ring(int nr, int width) {
+  const int boxes = row_boxes(width);
+  const size_t page = static_cast<size_t>(boxes) * kBoxBytes;
+  for (int ahead = 1; ahead >= 0; --ahead) {
+    const size_t fixed = fast_fixed_smem(nr, boxes, ahead);
+    int s = fixed > kSmemLimit ? 0 : static_cast<int>((kSmemLimit - fixed) / page);
+    if (s > kMaxStages) s = kMaxStages;
+    if (s >= (ahead ? 3 : 2)) return {s, ahead};
+  }
+  return {0, 0};
+}
+int tile_rows(int width) { return fast_ring(64, width).stages > 0 ? 64 : 32; }
+int head_groups(int heads, int rows) { return (heads + rows - 1) / rows; }
 
-bool encode_pool(CUtensorMap* map, const void* base, uint64_t width, uint64_t rows) {
+bool encode_rows(CUtensorMap* map, const void* base, uint64_t width, uint64_t rows, uint32_t box_rows) {
   ptx::EncodeTiledFn fn = ptx::tensor_map_encoder();
   if (!fn) return false;
   const cuuint64_t dims[2] = {width, rows};
   const cuuint64_t strides[1] = {width * 2};
-  const cuuint32_t box[2] = {64, kHalf};
+  const cuuint32_t box[2] = {64, box_rows};
   const cuuint32_t elem_strides[2] = {1, 1};
   return fn(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(base), dims, strides, box, elem_strides,
             CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
             CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
 }
 
-template <int MW, int RANKMAX, int KSQ>
-int launch_fast(FastParams p, dim3 grid, cudaStream_t st) {
+template <int NR>
+int launch_fast(FastParams p, const void* q, dim3 grid, cudaStream_t st) {
   const int width = p.a.kv_rank + p.a.rot_dim;
-  p.stages = fast_stages(MW * 16, width);
-  const size_t ring = static_cast<size_t>(p.stages) * p.boxes * kBoxBytes, combine = static_cast<size_t>(MW) * 16 * (p.a.kv_rank + 8) * 4;
-  p.ring_bytes = static_cast<int>(((p.splits > 1 && combine > ring ? combine : ring) + 15) / 16 * 16);
-  const size_t smem = p.ring_bytes + fast_fixed_smem(MW * 16);
-  if (p.stages < 4 || smem > kSmemLimit) return CACHEIR_B200_EUNSUPPORTED;
-  CUtensorMap tmap;
-  if (!encode_pool(&tmap, p.a.pool, width, static_cast<uint64_t>(p.a.num_slots) * kPage)) return CACHEIR_B200_EUNSUPPORTED;
-  auto kern = latent_attention_kernel<MW, RANKMAX, KSQ>;
+  const Ring ring = fast_ring(NR, width);
+  if (ring.stages == 0) return CACHEIR_B200_EUNSUPPORTED;
+  p.boxes = row_boxes(width);
+  p.blocks = (p.a.kv_rank + 127) / 128;
+  p.stages = ring.stages;
+  p.ahead = ring.ahead;
+  const int cols = p.blocks * NR + 2 * kPage;
+  p.tmem_cols = cols <= 256 ? 256 : 512;
+  size_t smem = fast_fixed_smem(NR, p.boxes, p.ahead) + static_cast<size_t>(p.stages) * p.boxes * kBoxBytes;
+  if (p.splits > 1 && static_cast<size_t>(NR) * (p.a.kv_rank + 8) * 4 > static_cast<size_t>(p.stages) * p.boxes * kBoxBytes)
+    return CACHEIR_B200_EUNSUPPORTED;        // (the combine's tile lies over the ring)
+  // No more CTAs on an SM than its tensor memory serves: one that waited for an allocation could hold up its cluster.
+  const size_t least = kSmemLimit / (512 / p.tmem_cols + 1) + 1024;
+  if (smem < least) smem = least;
+  CUtensorMap tkv, tq;
+  if (!encode_rows(&tkv, p.a.pool, width, static_cast<uint64_t>(p.a.num_slots) * kPage, kPage) ||
+      !encode_rows(&tq, q, width, static_cast<uint64_t>(p.a.rows) * p.a.heads, NR))
+    return CACHEIR_B200_EUNSUPPORTED;
+  auto kern = latent_attention_kernel<NR>;
   cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
   if (e != cudaSuccess) return static_cast<int>(e);
   cudaLaunchConfig_t cfg{};
@@ -518,18 +616,9 @@ int launch_fast(FastParams p, dim3 grid, cudaStream_t st) {
   attr[0].val.clusterDim.z = p.splits;
   cfg.attrs = attr;
   cfg.numAttrs = p.splits > 1 ? 1 : 0;
-  e = cudaLaunchKernelEx(&cfg, kern, tmap, p);
+  e = cudaLaunchKernelEx(&cfg, kern, tkv, tq, p);
   if (e != cudaSuccess) return static_cast<int>(e);
   return launch_status();
-}
-
-template <int MW>
-int launch_fast_size(const FastParams& p, dim3 grid, cudaStream_t st) {
-  const int width = p.a.kv_rank + p.a.rot_dim;
-  if (p.a.kv_rank <= 128 && width <= 192) return launch_fast<MW, 128, 3>(p, grid, st);
-  if (p.a.kv_rank <= 256 && width <= 320) return launch_fast<MW, 256, 5>(p, grid, st);
-  if (width <= 576) return launch_fast<MW, 512, 9>(p, grid, st);
-  return launch_fast<MW, 512, 10>(p, grid, st);
 }
 
 bool latent_args_ok(
@@ -600,13 +689,13 @@ extern "C" int cacheir_b200_latent_attention_simple(const cacheir_b200_latent_ar
 }
 
 extern "C" int cacheir_b200_latent_attention_supported(int kv_rank, int rot_dim, int page_size, int dtype) {
-  return dtype == CACHEIR_B200_BF16 && page_size == kPage && kv_rank >= 16 && kv_rank % 16 == 0 && kv_rank <= 512 && rot_dim >= 0 &&
-         rot_dim % 8 == 0 && kv_rank + rot_dim <= 640 && fast_stages(32, kv_rank + rot_dim) >= 4 ? 1 : 0;
+  return dtype == CACHEIR_B200_BF16 && page_size == kPage && kv_rank >= 8 && kv_rank % 8 == 0 && kv_rank <= 512 && rot_dim >= 0 &&
+         rot_dim % 8 == 0 && fast_ring(32, kv_rank + rot_dim).stages > 0 ? 1 : 0;
 }
 
 extern "C" int cacheir_b200_latent_attention_splits(int rows, int heads, int window, int max_pages, int page_size) {
   if (rows <= 0 || heads <= 0 || page_size <= 0) return 1;
-  const int units = rows * head_groups(heads);
+  const int units = rows * head_groups(heads, 64);
   int pages = (window + page_size - 2) / page_size + 1;
   if (pages > max_pages) pages = max_pages;
   int s = kNumSMs / units;
@@ -628,16 +717,15 @@ extern "C" int cacheir_b200_latent_attention(const cacheir_b200_latent_args* arg
   if (splits > kMaxSplits) return CACHEIR_B200_ELIMIT;
   FastParams p{};
   p.a = a;
-  p.q = static_cast<const __nv_bfloat16*>(q);
   p.sink = sink;
   p.out = static_cast<__nv_bfloat16*>(out);
   p.splits = splits;
-  p.boxes = row_boxes(a.kv_rank + a.rot_dim);
-  const int groups = head_groups(a.heads);
+  int rows = tile_rows(a.kv_rank + a.rot_dim);
+  const int groups = head_groups(a.heads, rows);
   p.heads_per_cta = (a.heads + groups - 1) / groups;
-  const bool narrow = decode && p.heads_per_cta <= 16;
-  p.tokens_per_tile = decode ? 1 : 32 / p.heads_per_cta;
+  if (decode && p.heads_per_cta <= 32) rows = 32;
+  p.tokens_per_tile = decode ? 1 : rows / p.heads_per_cta;
   const int items = decode ? a.rows : ragged_items(a.rows, a.segments, p.tokens_per_tile);
   const dim3 grid(items, groups, splits);
-  return narrow ? launch_fast_size<1>(p, grid, as_stream(stream)) : launch_fast_size<2>(p, grid, as_stream(stream));
+  return rows == 64 ? launch_fast<64>(p, q, grid, as_stream(stream)) : launch_fast<32>(p, q, grid, as_stream(stream));
 }
