@@ -148,8 +148,10 @@ latent_simple_kernel(const cacheir_b200_latent_args a, const T* __restrict__ q, 
 // so the page is used twice as it lies in shared memory and the probabilities go back as the K-major operand that a row's
 // threads write. O^T stays in tensor memory. Its columns are rescaled only when a row's maximum has grown by more than
 // 2^8 since its reference was chosen (a stale reference costs nothing: numerator and denominator share it).
-//   warps 0..3  softmax, rescaling, output (lane quarter = warp)     warp 4  MMA issue, tensor memory     warp 5  copies
-constexpr int kThreads = 192;
+//   warps 0..7  softmax (lane quarter = warp % 4, key half = warp / 4), rescaling, output
+//   warp 8      MMA issue, tensor memory           warp 9  copies
+constexpr int kThreads = 320;
+constexpr int kSoftThreads = 256;
 constexpr int kMaxSplits = 8;            // CTAs of a cluster
 constexpr int kMaxStages = 6;            // pages in the ring
 constexpr int kBoxBytes = kPage * 128;   // 64 rows x 64 columns
@@ -171,39 +173,50 @@ __device__ __forceinline__ float ld_peer_f32(uint32_t local_addr, uint32_t rank)
   uint32_t remote;
   float v;
   asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(remote) : "r"(local_addr), "r"(rank));
-  asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(v) : "r"(remote) : "memory");
+  asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(v) : "r"(remote));
+  return v;
+}
+__device__ __forceinline__ float4 ld_peer_f32x4(uint32_t local_addr, uint32_t rank) {
+  uint32_t remote;
+  float4 v;
+  asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(remote) : "r"(local_addr), "r"(rank));
+  asm volatile("ld.shared::cluster.v4.f32 {%0, %1, %2, %3}, [%4];" : "=f"(v.x), "=f"(v.y), "=f"(v.z), "=f"(v.w) : "r"(remote));
   return v;
 }
 __device__ __forceinline__ void cluster_sync_all() {
   asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory");
   asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory");
 }
-__device__ __forceinline__ void mma_f16_ss(uint32_t tmem_d, uint64_t a_desc, uint64_t b_desc, uint32_t idesc, uint32_t accumulate) {
+// Executed by a whole warp so that the operands stay in uniform registers; `lead` picks the issuing lane.
+__device__ __forceinline__ void mma_f16_ss(uint32_t lead, uint32_t tmem_d, uint64_t a_desc, uint64_t b_desc, uint32_t idesc, uint32_t accumulate) {
   asm volatile(
-      "{\n\t.reg .pred p;\n\t"
+      "{\n\t.reg .pred p, q;\n\t"
       "setp.ne.b32 p, %4, 0;\n\t"
-      "tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, p;\n\t}"
-      ::"r"(tmem_d), "l"(a_desc), "l"(b_desc), "r"(idesc), "r"(accumulate) : "memory");
+      "setp.ne.b32 q, %5, 0;\n\t"
+      "@q tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, p;\n\t}"
+      ::"r"(tmem_d), "l"(a_desc), "l"(b_desc), "r"(idesc), "r"(accumulate), "r"(lead) : "memory");
+}
+__device__ __forceinline__ float ex2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
 }
 // MN-major operand as 128-byte swizzled rows: 64 columns a box, `box` bytes between boxes, 8-row groups 1024 bytes apart
 __device__ __forceinline__ uint64_t smem_desc_mn_sw128(uint32_t addr, uint32_t box) {
   return static_cast<uint64_t>((addr >> 4) & 0x3FFF) | static_cast<uint64_t>((box >> 4) & 0x3FFF) << 16 |
          static_cast<uint64_t>(1024 >> 4) << 32 | static_cast<uint64_t>(1) << 46 | static_cast<uint64_t>(2) << 61;
 }
-// 16 lanes x 64 columns in the warp-MMA accumulator order: r[4 j + e] = row lane / 4 + 8 (e / 2), column 8 j + 2 (lane % 4) + e % 2
-__device__ __forceinline__ void tmem_ld_rows16(uint32_t taddr, float (&v)[32]) {
-  uint32_t r[32];
+// 16 lanes x 32 columns in the warp-MMA accumulator order: v[4 j + e] = row lane / 4 + 8 (e / 2), column 8 j + 2 (lane % 4) + e % 2
+__device__ __forceinline__ void tmem_ld_rows16(uint32_t taddr, float (&v)[16]) {
+  uint32_t r[16];
   asm volatile(
-      "tcgen05.ld.sync.aligned.16x256b.x8.b32 {%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,%16,%17,%18,%19,%20,%21,%22,%23,%24,"
-      "%25,%26,%27,%28,%29,%30,%31}, [%32];"
+      "tcgen05.ld.sync.aligned.16x256b.x4.b32 {%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15}, [%16];"
       : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]), "=r"(r[4]), "=r"(r[5]), "=r"(r[6]), "=r"(r[7]), "=r"(r[8]), "=r"(r[9]),
-        "=r"(r[10]), "=r"(r[11]), "=r"(r[12]), "=r"(r[13]), "=r"(r[14]), "=r"(r[15]), "=r"(r[16]), "=r"(r[17]), "=r"(r[18]),
-        "=r"(r[19]), "=r"(r[20]), "=r"(r[21]), "=r"(r[22]), "=r"(r[23]), "=r"(r[24]), "=r"(r[25]), "=r"(r[26]), "=r"(r[27]),
-        "=r"(r[28]), "=r"(r[29]), "=r"(r[30]), "=r"(r[31])
+        "=r"(r[10]), "=r"(r[11]), "=r"(r[12]), "=r"(r[13]), "=r"(r[14]), "=r"(r[15])
       : "r"(taddr) : "memory");
   ptx::tc_wait_ld();
 #pragma unroll
-  for (int i = 0; i < 32; ++i) v[i] = __uint_as_float(r[i]);
+  for (int i = 0; i < 16; ++i) v[i] = __uint_as_float(r[i]);
 }
 __device__ __forceinline__ void tmem_ld_x16(uint32_t taddr, float (&v)[16]) {
   uint32_t r[16];
@@ -222,18 +235,18 @@ __device__ __forceinline__ void tmem_st_x16(uint32_t taddr, const float (&v)[16]
       ::"r"(taddr), "f"(v[0]), "f"(v[1]), "f"(v[2]), "f"(v[3]), "f"(v[4]), "f"(v[5]), "f"(v[6]), "f"(v[7]), "f"(v[8]), "f"(v[9]), "f"(v[10]),
       "f"(v[11]), "f"(v[12]), "f"(v[13]), "f"(v[14]), "f"(v[15]) : "memory");
 }
-// true in all 128 softmax threads if `p` holds in one of them
-__device__ __forceinline__ bool any_of_128(bool p) {
+// true in all softmax threads if `p` holds in one of them
+__device__ __forceinline__ bool any_softmax(bool p) {
   uint32_t out;
   asm volatile(
       "{\n\t.reg .pred a, b;\n\t"
       "setp.ne.u32 a, %1, 0;\n\t"
-      "barrier.cta.red.or.pred b, 1, 128, a;\n\t"
+      "barrier.cta.red.or.pred b, 1, %2, a;\n\t"
       "selp.u32 %0, 1, 0, b;\n\t}"
-      : "=r"(out) : "r"(static_cast<uint32_t>(p)) : "memory");
+      : "=r"(out) : "r"(static_cast<uint32_t>(p)), "n"(kSoftThreads) : "memory");
   return out != 0;
 }
-__device__ __forceinline__ void sync_128() { asm volatile("barrier.cta.sync 1, 128;" ::: "memory"); }
+__device__ __forceinline__ void sync_softmax() { asm volatile("barrier.cta.sync 1, %0;" ::"n"(kSoftThreads) : "memory"); }
 
 template <int NR>
 __global__ void __launch_bounds__(kThreads, 1)
@@ -247,14 +260,17 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_kv, const __gri
   uint8_t* s_q = s_kv + p.stages * page_bytes;                  // [boxes][NR rows][128 bytes], swizzled
   uint8_t* s_p = s_q + p.boxes * NR * 128;                      // [1 + ahead][NR rows][128 bytes], swizzled
   float* s_alpha = reinterpret_cast<float*>(s_p + (1 + p.ahead) * NR * 128);   // [NR]
-  float* s_ml = s_alpha + NR;                                   // [NR][2]
+  float* s_max = s_alpha + NR;                                  // [2 key halves][NR]
+  float* s_ml = s_max + 2 * NR;                                 // [NR] references, [NR] denominators
+  float* s_w = reinterpret_cast<float*>(s_p);                   // [NR][kMaxSplits] weights of the combine (over s_p)
   uint64_t* full = reinterpret_cast<uint64_t*>(s_ml + 2 * NR);  // [stages] a page has landed
   uint64_t* empty = full + kMaxStages;                          // [stages] its output MMAs have retired
   uint64_t* bar_q = empty + kMaxStages;
   uint64_t* bar_s = bar_q + 1;                                  // [2] scores in tensor memory
   uint64_t* bar_p = bar_s + 2;                                  // [2] probabilities in shared memory
   uint64_t* bar_o = bar_p + 2;                                  // the output MMAs of one more page have retired
-  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bar_o + 1);
+  uint64_t* bar_done = bar_o + 1;                               // all output MMAs have retired
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bar_done + 1);
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int head0 = blockIdx.y * p.heads_per_cta;
@@ -282,11 +298,12 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_kv, const __gri
   if (threadIdx.x == 0) {
     for (int s = 0; s < p.stages; ++s) { ptx::mbar_init(smem_addr(&full[s]), 1); ptx::mbar_init(smem_addr(&empty[s]), 1); }
     ptx::mbar_init(smem_addr(bar_q), 1);
-    for (int s = 0; s < 2; ++s) { ptx::mbar_init(smem_addr(&bar_s[s]), 1); ptx::mbar_init(smem_addr(&bar_p[s]), 128); }
+    for (int s = 0; s < 2; ++s) { ptx::mbar_init(smem_addr(&bar_s[s]), 1); ptx::mbar_init(smem_addr(&bar_p[s]), kSoftThreads); }
     ptx::mbar_init(smem_addr(bar_o), 1);
+    ptx::mbar_init(smem_addr(bar_done), 1);
     ptx::mbar_fence_init();
   }
-  if (warp == 4) ptx::tc_alloc(smem_addr(tmem_slot), p.tmem_cols);
+  if (warp == 8) ptx::tc_alloc(smem_addr(tmem_slot), p.tmem_cols);
   ptx::tc_fence_before();
   __syncthreads();
   ptx::tc_fence_after();
@@ -294,12 +311,9 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_kv, const __gri
   const uint32_t tmem_s = tmem + p.blocks * NR;       // scores: two buffers of 64 columns behind the output blocks
   bool ok = true;
 
-  if (warp == 5) {
+  if (warp == 9) {
     // ---------------- copies ----------------
     if (lane == 0 && npages > 0) {
-      ptx::mbar_expect_tx(smem_addr(bar_q), p.boxes * NR * 128);
-      for (int b = 0; b < p.boxes; ++b)
-        ptx::tma_load_2d(smem_addr(s_q + b * NR * 128), &tmap_q, smem_addr(bar_q), b * 64, row0 * a.heads + head0);
       int stage = 0, phase = 1;
       for (int it = 0; it < npages; ++it) {
         const int pg = pg_begin + it;
@@ -312,6 +326,11 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_kv, const __gri
         for (int b = 0; b < p.boxes; ++b)
           ptx::tma_load_2d(smem_addr(s_kv + stage * page_bytes + b * kBoxBytes), &tmap_kv, bar, b * 64, slot * kPage);
         if (++stage == p.stages) { stage = 0; phase ^= 1; }
+        if (it == 0) {
+          ptx::mbar_expect_tx(smem_addr(bar_q), p.boxes * NR * 128);
+          for (int b = 0; b < p.boxes; ++b)
+            ptx::tma_load_2d(smem_addr(s_q + b * NR * 128), &tmap_q, smem_addr(bar_q), b * 64, row0 * a.heads + head0);
+        }
       }
       // nothing may still be on its way when the block ends, also after a wait that gave up
       ptx::mbar_wait(smem_addr(bar_q), 0, &g_latent_status, (7 << 8) | 8);
@@ -319,123 +338,142 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_kv, const __gri
         for (int s = 0; s < p.stages; ++s) ptx::mbar_wait(smem_addr(&full[s]), s < stage ? phase ^ 1 : phase, &g_latent_status, (7 << 8) | 9);
     }
     __syncwarp();
-  } else if (warp == 4) {
+  } else if (warp == 8) {
     // ---------------- MMA issue ----------------
-    if (lane == 0 && npages > 0) {
+    if (npages > 0) {
+      const uint32_t lead = lane == 0 ? 1u : 0u;
       const uint32_t id_s = (1u << 4) | (1u << 7) | (1u << 10) | (static_cast<uint32_t>(kPage >> 3) << 17) | (static_cast<uint32_t>(64 >> 4) << 24);
       const uint32_t id_o = (1u << 4) | (1u << 7) | (1u << 10) | (1u << 15) | (static_cast<uint32_t>(NR >> 3) << 17) |
                             (static_cast<uint32_t>(128 >> 4) << 24);
       const uint64_t dq = ptx::smem_desc_sw128(smem_addr(s_q)), dk = ptx::smem_desc_sw128(smem_addr(s_kv)), dp = ptx::smem_desc_sw128(smem_addr(s_p));
       const uint64_t dv = smem_desc_mn_sw128(smem_addr(s_kv), kBoxBytes);
-      const int ksteps = (width + 15) / 16;
       int s_stage = 0, s_phase = 0;          // next page to score
       auto scores = [&](int it) {
         ok = ok && ptx::mbar_wait(smem_addr(&full[s_stage]), s_phase, &g_latent_status, (7 << 8) | 2);
+        __syncwarp();
         ptx::tc_fence_after();
-        const uint64_t k0 = dk + static_cast<uint64_t>(s_stage * page_bytes >> 4);
+        uint64_t aq = dq, bk = dk + static_cast<uint64_t>(s_stage * page_bytes >> 4);
         const uint32_t d = tmem_s + (it & 1) * kPage;
-        int k = 0;
-        for (int b = 0; b < p.boxes; ++b) {
-          const uint64_t aq = dq + static_cast<uint64_t>(b * (NR * 128 >> 4)), bk = k0 + static_cast<uint64_t>(b * (kBoxBytes >> 4));
+        for (int b = 0; b < p.boxes; ++b) {  // (columns beyond the row are zero in both operands)
 #pragma unroll
-          for (int j = 0; j < 4; ++j, ++k)
-            if (k < ksteps) mma_f16_ss(d, aq + 2 * j, bk + 2 * j, id_s, k > 0 ? 1u : 0u);
+          for (int j = 0; j < 4; ++j) mma_f16_ss(lead, d, aq + 2 * j, bk + 2 * j, id_s, (b | j) > 0 ? 1u : 0u);
+          aq += NR * 128 >> 4;
+          bk += kBoxBytes >> 4;
         }
-        ptx::tc_commit(smem_addr(&bar_s[it & 1]));
+        if (lead) ptx::tc_commit(smem_addr(&bar_s[it & 1]));
+        __syncwarp();
         if (++s_stage == p.stages) { s_stage = 0; s_phase ^= 1; }
       };
       ok = ptx::mbar_wait(smem_addr(bar_q), 0, &g_latent_status, (7 << 8) | 3);
       scores(0);
       int o_stage = 0;
-      for (int it = 0; it < npages && ok; ++it) {
+      for (int it = 0; it < npages; ++it) {
         if (p.ahead && it + 1 < npages) scores(it + 1);
         ok = ok && ptx::mbar_wait(smem_addr(&bar_p[it & 1]), (it >> 1) & 1, &g_latent_status, (7 << 8) | 4);
+        __syncwarp();
         ptx::tc_fence_after();
-        const uint64_t v0 = dv + static_cast<uint64_t>(o_stage * page_bytes >> 4);
+        uint64_t av = dv + static_cast<uint64_t>(o_stage * page_bytes >> 4);
         const uint64_t pb = dp + static_cast<uint64_t>((p.ahead ? it & 1 : 0) * (NR * 128 >> 4));
         for (int m = 0; m < p.blocks; ++m) {
-          const uint64_t av = v0 + static_cast<uint64_t>(m * (2 * kBoxBytes >> 4));
 #pragma unroll
           for (int j = 0; j < 4; ++j)        // 16 keys
-            mma_f16_ss(tmem + m * NR, av + j * (2048 >> 4), pb + 2 * j, id_o, (it > 0 || j > 0) ? 1u : 0u);
+            mma_f16_ss(lead, tmem + m * NR, av + j * (2048 >> 4), pb + 2 * j, id_o, (it | j) > 0 ? 1u : 0u);
+          av += 2 * kBoxBytes >> 4;
         }
-        ptx::tc_commit(smem_addr(&empty[o_stage]));
-        ptx::tc_commit(smem_addr(bar_o));
+        if (lead) {
+          ptx::tc_commit(smem_addr(&empty[o_stage]));
+          ptx::tc_commit(smem_addr(bar_o));
+        }
+        __syncwarp();
         if (++o_stage == p.stages) o_stage = 0;
         if (!p.ahead && it + 1 < npages) scores(it + 1);
       }
+      if (lead) ptx::tc_commit(smem_addr(bar_done));
     }
     __syncwarp();
   } else {
-    // ---------------- softmax: rows r0 = 16 warp + lane / 4 and r0 + 8, columns 8 j + 2 (lane % 4) + {0, 1} ----------------
-    const bool band = warp * 16 < NR;        // (a 32-row tile keeps two of the four warps for the rescaling only)
+    // ------- softmax: rows r0 = 16 (warp % 4) + lane / 4 and r0 + 8, keys 32 (warp / 4) + 8 j + 2 (lane % 4) + {0, 1} -------
+    const int quarter = warp & 3, half = warp >> 2;
+    const bool band = quarter * 16 < NR;     // (with a 32-row tile half of the warps only rescale and store)
+    const int r0 = quarter * 16 + (lane >> 2);
     float m_ref[2], l_run[2];
     int row_pos[2];
 #pragma unroll
     for (int e = 0; e < 2; ++e) {
-      const int r = warp * 16 + (lane >> 2) + 8 * e;
+      const int r = r0 + 8 * e;
       const bool real = band && r < used;
       row_pos[e] = real ? pos0 + r / nheads : -1;
       m_ref[e] = (real && split == 0) ? p.sink[head0 + r % nheads] * kLog2e : -1e30f;
-      l_run[e] = (real && split == 0 && (lane & 3) == 0) ? 1.f : 0.f;
+      l_run[e] = (real && split == 0 && half == 0 && (lane & 3) == 0) ? 1.f : 0.f;
     }
     const float qscale = a.scale * kLog2e;
-    const uint32_t lane_addr = static_cast<uint32_t>(warp * 32) << 16;
+    const uint32_t lane_addr = static_cast<uint32_t>(quarter * 32) << 16;
     int stage = 0;
     for (int it = 0; it < npages; ++it) {
       const int buf = p.ahead ? it & 1 : 0;
       ok = ok && ptx::mbar_wait(smem_addr(&bar_s[it & 1]), (it >> 1) & 1, &g_latent_status, (7 << 8) | 5);
       __syncwarp();
       ptx::tc_fence_after();
-      float s[32], alpha[2] = {1.f, 1.f};
-      bool grown = false;
+      float s[16], alpha[2] = {1.f, 1.f};
+      const int base = (pg_begin + it) * kPage;
       if (band) {
-        tmem_ld_rows16(tmem_s + (it & 1) * kPage + lane_addr, s);
-        const int base = (pg_begin + it) * kPage;
+        tmem_ld_rows16(tmem_s + (it & 1) * kPage + half * 32 + lane_addr, s);
         float mx[2] = {-1e30f, -1e30f};
         if (base + kPage - 1 <= pos0 && base > pos_last - a.window) {      // the whole page is seen by every row
 #pragma unroll
-          for (int i = 0; i < 32; ++i) {
+          for (int i = 0; i < 16; ++i) {
             s[i] *= qscale;
             mx[(i >> 1) & 1] = fmaxf(mx[(i >> 1) & 1], s[i]);
           }
         } else {
 #pragma unroll
-          for (int i = 0; i < 32; ++i) {
-            const int key = base + (i >> 2) * 8 + (lane & 3) * 2 + (i & 1), rp = row_pos[(i >> 1) & 1];
+          for (int i = 0; i < 16; ++i) {
+            const int key = base + half * 32 + (i >> 2) * 8 + (lane & 3) * 2 + (i & 1), rp = row_pos[(i >> 1) & 1];
             s[i] = (key <= rp && key > rp - a.window) ? s[i] * qscale : -INFINITY;
             mx[(i >> 1) & 1] = fmaxf(mx[(i >> 1) & 1], s[i]);
           }
         }
 #pragma unroll
-        for (int e = 0; e < 2; ++e) {
-          mx[e] = fmaxf(mx[e], __shfl_xor_sync(0xffffffffu, mx[e], 1));
-          mx[e] = fmaxf(mx[e], __shfl_xor_sync(0xffffffffu, mx[e], 2));
-          if (row_pos[e] >= 0 && (it == 0 ? mx[e] > m_ref[e] : mx[e] > m_ref[e] + kStale)) {
-            alpha[e] = exp2f(m_ref[e] - mx[e]);
-            m_ref[e] = mx[e];
-            grown = it > 0;
-          }
+        for (int off = 1; off < 4; off <<= 1)
+#pragma unroll
+          for (int e = 0; e < 2; ++e) mx[e] = fmaxf(mx[e], __shfl_xor_sync(0xffffffffu, mx[e], off));
+        if ((lane & 3) == 0) {
+          s_max[half * NR + r0] = mx[0];
+          s_max[half * NR + r0 + 8] = mx[1];
         }
       }
-      const int tail = pos_last + 1 - (pg_begin + it) * kPage;
+      const int tail = pos_last + 1 - base;
       if (tail < kPage) {                    // rows behind the last token may hold anything: zero, so that 0 * row stays 0
-        for (int i = threadIdx.x; i < (kPage - tail) * p.boxes * 8; i += 128) {
+        for (int i = threadIdx.x; i < (kPage - tail) * p.boxes * 8; i += kSoftThreads) {
           const int r = tail + i / (p.boxes * 8), c = i % (p.boxes * 8);
           *reinterpret_cast<uint4*>(s_kv + stage * page_bytes + (c >> 3) * kBoxBytes + r * 128 + (c & 7) * 16) = make_uint4(0u, 0u, 0u, 0u);
         }
         asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
       }
       if (++stage == p.stages) stage = 0;
-      if (any_of_128(grown)) {               // rare: bring O^T to the new references
-        if (band && (lane & 3) == 0) {
+      sync_softmax();
+      bool grown = false;
+      if (band) {
 #pragma unroll
-          for (int e = 0; e < 2; ++e) s_alpha[warp * 16 + (lane >> 2) + 8 * e] = alpha[e];
+        for (int e = 0; e < 2; ++e) {
+          const float mx = fmaxf(s_max[r0 + 8 * e], s_max[NR + r0 + 8 * e]);
+          if (row_pos[e] >= 0 && mx > m_ref[e] + (it == 0 ? 0.f : kStale)) {
+            alpha[e] = ex2(m_ref[e] - mx);
+            m_ref[e] = mx;
+            grown = it > 0;
+          }
         }
-        ok = ok && ptx::mbar_wait(smem_addr(bar_o), (it - 1) & 1, &g_latent_status, (7 << 8) | 6);     // the page before is in
+      }
+      if (any_softmax(grown)) {              // rare: bring O^T to the new references
+        if (band && half == 0 && (lane & 3) == 0) {
+          s_alpha[r0] = alpha[0];
+          s_alpha[r0 + 8] = alpha[1];
+        }
+        ok = ok && ptx::mbar_wait(smem_addr(bar_o), (it - 1) & 1, &g_latent_status, (7 << 8) | 6);     // the page before is in (the one before that is: this page's scores follow it)
+        __syncwarp();
         ptx::tc_fence_after();
-        sync_128();
-        for (int c = 0; c < p.blocks * NR; c += 16) {
+        sync_softmax();
+        for (int c = half * 16; c < p.blocks * NR; c += 32) {
           float o[16];
           tmem_ld_x16(tmem + lane_addr + c, o);
 #pragma unroll
@@ -443,69 +481,87 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_kv, const __gri
           tmem_st_x16(tmem + lane_addr + c, o);
         }
         asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory");
-        sync_128();                          // s_alpha may be written again
+        sync_softmax();                      // s_alpha may be written again
       }
       if (band) {
 #pragma unroll
         for (int e = 0; e < 2; ++e) l_run[e] *= alpha[e];
-        uint8_t* dst = s_p + (buf * NR + warp * 16 + (lane >> 2)) * 128 + (lane & 3) * 4;
-        const int swz = lane >> 2;           // row % 8 of both rows
+        uint8_t* dst = s_p + (buf * NR + r0) * 128 + (lane & 3) * 4;
 #pragma unroll
-        for (int j = 0; j < 8; ++j) {
+        for (int j = 0; j < 4; ++j) {
 #pragma unroll
           for (int e = 0; e < 4; ++e) {
-            s[4 * j + e] = (e < 2 ? row_pos[0] : row_pos[1]) >= 0 ? exp2f(s[4 * j + e] - m_ref[e >> 1]) : 0.f;
+            s[4 * j + e] = row_pos[e >> 1] >= 0 ? ex2(s[4 * j + e] - m_ref[e >> 1]) : 0.f;
             l_run[e >> 1] += s[4 * j + e];
           }
-          *reinterpret_cast<uint32_t*>(dst + ((j ^ swz) << 4)) = pack_bf16(s[4 * j], s[4 * j + 1]);
-          *reinterpret_cast<uint32_t*>(dst + 8 * 128 + ((j ^ swz) << 4)) = pack_bf16(s[4 * j + 2], s[4 * j + 3]);
+          const int chunk = ((half * 4 + j) ^ (lane >> 2)) << 4;           // (both rows are lane / 4 modulo 8)
+          *reinterpret_cast<uint32_t*>(dst + chunk) = pack_bf16(s[4 * j], s[4 * j + 1]);
+          *reinterpret_cast<uint32_t*>(dst + 8 * 128 + chunk) = pack_bf16(s[4 * j + 2], s[4 * j + 3]);
         }
         asm volatile("fence.proxy.async.shared::cta;" ::: "memory");       // the tensor core reads what was just written
       }
       ptx::tc_fence_before();
       ptx::mbar_arrive(smem_addr(&bar_p[it & 1]));
     }
-    // row sums and references
-    if (band) {
+    // references and denominators (s_max: the two key halves' sums)
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      l_run[e] += __shfl_xor_sync(0xffffffffu, l_run[e], 1);
+      l_run[e] += __shfl_xor_sync(0xffffffffu, l_run[e], 2);
+    }
+    sync_softmax();
+    if (band && (lane & 3) == 0) {
 #pragma unroll
       for (int e = 0; e < 2; ++e) {
-        l_run[e] += __shfl_xor_sync(0xffffffffu, l_run[e], 1);
-        l_run[e] += __shfl_xor_sync(0xffffffffu, l_run[e], 2);
-        if ((lane & 3) == 0) {
-          s_ml[(warp * 16 + (lane >> 2) + 8 * e) * 2] = m_ref[e];
-          s_ml[(warp * 16 + (lane >> 2) + 8 * e) * 2 + 1] = p.splits == 1 ? 1.f / l_run[e] : l_run[e];
-        }
+        if (half == 0) s_ml[r0 + 8 * e] = m_ref[e];
+        s_max[half * NR + r0 + 8 * e] = l_run[e];
       }
     }
-    if (npages > 0) ok = ok && ptx::mbar_wait(smem_addr(bar_o), (npages - 1) & 1, &g_latent_status, (7 << 8) | 7);
+    // (not by bar_o: with scores issued ahead the page before the last may still be in the works, and its phase would alias)
+    if (npages > 0) ok = ok && ptx::mbar_wait(smem_addr(bar_done), 0, &g_latent_status, (7 << 8) | 7);
     __syncwarp();
     ptx::tc_fence_after();
-    sync_128();                              // s_ml is complete, every page has been read
-    // O^T: lane = latent column of the block, tensor-memory column = tile row
+    sync_softmax();                          // every page has been read: the ring is free
+    if (threadIdx.x < NR) {
+      const float l = s_max[threadIdx.x] + s_max[NR + threadIdx.x];
+      s_ml[NR + threadIdx.x] = l;
+      s_alpha[threadIdx.x] = 1.f / l;
+    }
+    sync_softmax();
+    // O^T (lane = latent column of the block, tensor-memory column = tile row) turns in shared memory: as finished bf16
+    // rows, or as float parts of a split tile
+    __nv_bfloat16* s_out = reinterpret_cast<__nv_bfloat16*>(smem);
     float* s_o = reinterpret_cast<float*>(smem);
-    const int opitch = a.kv_rank + 8;
-    for (int m = 0; m < p.blocks; ++m) {
-      const int col = m * 128 + warp * 32 + lane;
-      for (int c = 0; c < NR; c += 16) {
-        if (c >= used) break;
-        float o[16];
-        if (npages > 0) {
-          tmem_ld_x16(tmem + lane_addr + m * NR + c, o);
-        } else {
+    const int bpitch = a.kv_rank + 8, opitch = a.kv_rank + 4;
+    for (int u = half; u < p.blocks * (NR / 16); u += 2) {
+      const int m = u / (NR / 16), c = (u % (NR / 16)) * 16;
+      if (c >= used) continue;
+      const int col = m * 128 + quarter * 32 + lane;
+      float o[16];
+      if (npages > 0) {
+        tmem_ld_x16(tmem + lane_addr + m * NR + c, o);
+      } else {
 #pragma unroll
-          for (int j = 0; j < 16; ++j) o[j] = 0.f;
-        }
-        if (col >= a.kv_rank) {
-        } else if (p.splits == 1) {
-          __nv_bfloat16* dst = p.out + (static_cast<size_t>(row0) * a.heads + head0 + c) * a.kv_rank + col;
+        for (int j = 0; j < 16; ++j) o[j] = 0.f;
+      }
+      if (col < a.kv_rank) {
+        if (p.splits == 1) {
 #pragma unroll
-          for (int j = 0; j < 16; ++j)
-            if (c + j < used) dst[static_cast<size_t>(j) * a.kv_rank] = __float2bfloat16_rn(o[j] * s_ml[(c + j) * 2 + 1]);
+          for (int j = 0; j < 16; ++j) s_out[(c + j) * bpitch + col] = __float2bfloat16_rn(o[j] * s_alpha[c + j]);
         } else {
 #pragma unroll
           for (int j = 0; j < 16; ++j) s_o[(c + j) * opitch + col] = o[j];
         }
-        __syncwarp();
+      }
+      __syncwarp();
+    }
+    if (p.splits == 1) {
+      sync_softmax();
+      const int pieces = a.kv_rank / 8;
+      __nv_bfloat16* dst = p.out + (static_cast<size_t>(row0) * a.heads + head0) * a.kv_rank;      // neighbouring rows
+      for (int i = threadIdx.x; i < used * pieces; i += kSoftThreads) {
+        const int r = i / pieces, c = i % pieces;
+        *reinterpret_cast<uint4*>(dst + static_cast<size_t>(i) * 8) = *reinterpret_cast<const uint4*>(s_out + r * bpitch + c * 8);
       }
     }
   }
@@ -513,35 +569,51 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_kv, const __gri
     // the cluster's CTAs share one tile: rows dealt out, parts added in rank order
     __syncwarp();
     cluster_sync_all();
-    float* s_o = reinterpret_cast<float*>(smem);
-    const int opitch = a.kv_rank + 8;
-    for (int r = split; r < used; r += p.splits) {
-      float m[kMaxSplits], top = -1e30f, l = 0.f;
+    const float* s_o = reinterpret_cast<const float*>(smem);
+    const int opitch = a.kv_rank + 4, mine = (used - split + p.splits - 1) / p.splits;       // rows split, split + splits, ...
+    if (static_cast<int>(threadIdx.x) < mine) {
+      const int r = split + threadIdx.x * p.splits;
+      float m[kMaxSplits], l[kMaxSplits], top = -1e30f, sum = 0.f;
 #pragma unroll
       for (int s = 0; s < kMaxSplits; ++s) {
-        m[s] = s < p.splits ? ld_peer_f32(smem_addr(s_ml + r * 2), s) : -1e30f;
-        top = fmaxf(top, m[s]);
+        m[s] = s < p.splits ? ld_peer_f32(smem_addr(s_ml + r), s) : -1e30f;
+        l[s] = s < p.splits ? ld_peer_f32(smem_addr(s_ml + NR + r), s) : 0.f;
       }
+#pragma unroll
+      for (int s = 0; s < kMaxSplits; ++s) top = fmaxf(top, m[s]);
 #pragma unroll
       for (int s = 0; s < kMaxSplits; ++s) {
-        m[s] = exp2f(m[s] - top);
-        if (s < p.splits) l = fmaf(ld_peer_f32(smem_addr(s_ml + r * 2 + 1), s), m[s], l);
+        m[s] = ex2(m[s] - top);
+        sum = fmaf(l[s], m[s], sum);
       }
-      const float inv = 1.f / l;
-      __nv_bfloat16* dst = p.out + (static_cast<size_t>(row0) * a.heads + head0 + r) * a.kv_rank;
-      for (int c = threadIdx.x; c < a.kv_rank; c += kThreads) {
-        float v = 0.f;
 #pragma unroll
-        for (int s = 0; s < kMaxSplits; ++s)
-          if (s < p.splits) v = fmaf(ld_peer_f32(smem_addr(s_o + r * opitch + c), s), m[s], v);
-        dst[c] = __float2bfloat16_rn(v * inv);
-      }
+      for (int s = 0; s < kMaxSplits; ++s) s_w[threadIdx.x * kMaxSplits + s] = m[s] / sum;
+    }
+    __syncthreads();
+    const int pieces = a.kv_rank / 4;
+    for (int i = threadIdx.x; i < mine * pieces; i += kThreads) {
+      const int k = i / pieces, c = (i % pieces) * 4, r = split + k * p.splits;
+      float4 part[kMaxSplits];
+#pragma unroll
+      for (int s = 0; s < kMaxSplits; ++s)
+        if (s < p.splits) part[s] = ld_peer_f32x4(smem_addr(s_o + r * opitch + c), s);
+      float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+      for (int s = 0; s < kMaxSplits; ++s)
+        if (s < p.splits) {
+          const float w = s_w[k * kMaxSplits + s];
+          v.x = fmaf(part[s].x, w, v.x); v.y = fmaf(part[s].y, w, v.y); v.z = fmaf(part[s].z, w, v.z); v.w = fmaf(part[s].w, w, v.w);
+        }
+      uint2 raw;
+      raw.x = pack_bf16(v.x, v.y);
+      raw.y = pack_bf16(v.z, v.w);
+      *reinterpret_cast<uint2*>(p.out + (static_cast<size_t>(row0) * a.heads + head0 + r) * a.kv_rank + c) = raw;
     }
     cluster_sync_all();                    // nobody leaves while its part is being read
   }
   ptx::tc_fence_before();
   __syncthreads();
-  if (warp == 4) {
+  if (warp == 8) {
     ptx::tc_fence_after();
     ptx::tc_dealloc(tmem, p.tmem_cols);
   }
@@ -551,7 +623,7 @@ constexpr size_t kSmemLimit = 227 * 1024;
 int row_boxes(int width) { return (width + 63) / 64; }
 // Shared memory beside the ring, and the ring's pages: `ahead` when three fit.
 size_t fast_fixed_smem(int nr, int boxes, int ahead) {
-  return 1024 + static_cast<size_t>(boxes + 1 + ahead) * nr * 128 + nr * 12 + (2 * kMaxStages + 6) * 8 + 16;
+  return 1024 + static_cast<size_t>(boxes + 1 + ahead) * nr * 128 + nr * 5 * 4 + (2 * kMaxStages + 8) * 8 + 16;
 }
 struct Ring { int stages, ahead; };
 Ring fast_ring(int nr, int width) {
@@ -592,7 +664,7 @@ int launch_fast(FastParams p, const void* q, dim3 grid, cudaStream_t st) {
   const int cols = p.blocks * NR + 2 * kPage;
   p.tmem_cols = cols <= 256 ? 256 : 512;
   size_t smem = fast_fixed_smem(NR, p.boxes, p.ahead) + static_cast<size_t>(p.stages) * p.boxes * kBoxBytes;
-  if (p.splits > 1 && static_cast<size_t>(NR) * (p.a.kv_rank + 8) * 4 > static_cast<size_t>(p.stages) * p.boxes * kBoxBytes)
+  if (p.splits > 1 && static_cast<size_t>(NR) * (p.a.kv_rank + 4) * 4 > static_cast<size_t>(p.stages) * p.boxes * kBoxBytes)
     return CACHEIR_B200_EUNSUPPORTED;        // (the combine's tile lies over the ring)
   // No more CTAs on an SM than its tensor memory serves: one that waited for an allocation could hold up its cluster.
   const size_t least = kSmemLimit / (512 / p.tmem_cols + 1) + 1024;
