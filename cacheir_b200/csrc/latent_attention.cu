@@ -176,13 +176,6 @@ __device__ __forceinline__ float ld_peer_f32(uint32_t local_addr, uint32_t rank)
   asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(v) : "r"(remote));
   return v;
 }
-__device__ __forceinline__ float4 ld_peer_f32x4(uint32_t local_addr, uint32_t rank) {
-  uint32_t remote;
-  float4 v;
-  asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(remote) : "r"(local_addr), "r"(rank));
-  asm volatile("ld.shared::cluster.v4.f32 {%0, %1, %2, %3}, [%4];" : "=f"(v.x), "=f"(v.y), "=f"(v.z), "=f"(v.w) : "r"(remote));
-  return v;
-}
 __device__ __forceinline__ void cluster_sync_all() {
   asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory");
   asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory");
@@ -262,7 +255,7 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_kv, const __gri
   float* s_alpha = reinterpret_cast<float*>(s_p + (1 + p.ahead) * NR * 128);   // [NR]
   float* s_max = s_alpha + NR;                                  // [2 key halves][NR]
   float* s_ml = s_max + 2 * NR;                                 // [NR] references, [NR] denominators
-  float* s_w = reinterpret_cast<float*>(s_p);                   // [NR][kMaxSplits] weights of the combine (over s_p)
+  float* s_w = reinterpret_cast<float*>(s_p);                   // [rows][kMaxSplits][2]: what the combine weighs with (over s_p)
   uint64_t* full = reinterpret_cast<uint64_t*>(s_ml + 2 * NR);  // [stages] a page has landed
   uint64_t* empty = full + kMaxStages;                          // [stages] its output MMAs have retired
   uint64_t* bar_q = empty + kMaxStages;
@@ -295,14 +288,34 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_kv, const __gri
   const int pg_begin = page_lo + pages * split / p.splits;
   const int npages = page_lo + pages * (split + 1) / p.splits - pg_begin;
 
-  if (threadIdx.x == 0) {
+  // The copy warp sets the barriers up and requests the first pages before the block meets.
+  int stage = 0, phase = 1;                // its place in the ring
+  auto load_page = [&](int it) {
+    const int pg = pg_begin + it;
+    int slot = pg < a.max_pages ? a.page_table[static_cast<size_t>(seg) * a.max_pages + pg] : 0;
+    slot = min(max(slot, 0), a.num_slots - 1);
+    const uint32_t bar = smem_addr(&full[stage]);
+    ptx::mbar_expect_tx(bar, page_bytes);
+    for (int b = 0; b < p.boxes; ++b)
+      ptx::tma_load_2d(smem_addr(s_kv + stage * page_bytes + b * kBoxBytes), &tmap_kv, bar, b * 64, slot * kPage);
+    if (++stage == p.stages) { stage = 0; phase ^= 1; }
+  };
+  const int first = min(npages, p.stages);
+  if (warp == 9 && lane == 0) {
     for (int s = 0; s < p.stages; ++s) { ptx::mbar_init(smem_addr(&full[s]), 1); ptx::mbar_init(smem_addr(&empty[s]), 1); }
     ptx::mbar_init(smem_addr(bar_q), 1);
     for (int s = 0; s < 2; ++s) { ptx::mbar_init(smem_addr(&bar_s[s]), 1); ptx::mbar_init(smem_addr(&bar_p[s]), kSoftThreads); }
     ptx::mbar_init(smem_addr(bar_o), 1);
     ptx::mbar_init(smem_addr(bar_done), 1);
     ptx::mbar_fence_init();
+    if (npages > 0) {
+      ptx::mbar_expect_tx(smem_addr(bar_q), p.boxes * NR * 128);
+      for (int b = 0; b < p.boxes; ++b)
+        ptx::tma_load_2d(smem_addr(s_q + b * NR * 128), &tmap_q, smem_addr(bar_q), b * 64, row0 * a.heads + head0);
+      for (int it = 0; it < first; ++it) load_page(it);
+    }
   }
+  __syncwarp();
   if (warp == 8) ptx::tc_alloc(smem_addr(tmem_slot), p.tmem_cols);
   ptx::tc_fence_before();
   __syncthreads();
@@ -314,23 +327,10 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_kv, const __gri
   if (warp == 9) {
     // ---------------- copies ----------------
     if (lane == 0 && npages > 0) {
-      int stage = 0, phase = 1;
-      for (int it = 0; it < npages; ++it) {
-        const int pg = pg_begin + it;
-        int slot = pg < a.max_pages ? a.page_table[static_cast<size_t>(seg) * a.max_pages + pg] : 0;
-        slot = min(max(slot, 0), a.num_slots - 1);
-        if (it >= p.stages) ok = ok && ptx::mbar_wait(smem_addr(&empty[stage]), phase, &g_latent_status, (7 << 8) | 1);
+      for (int it = first; it < npages; ++it) {
+        ok = ok && ptx::mbar_wait(smem_addr(&empty[stage]), phase, &g_latent_status, (7 << 8) | 1);
         if (!ok) break;
-        const uint32_t bar = smem_addr(&full[stage]);
-        ptx::mbar_expect_tx(bar, page_bytes);
-        for (int b = 0; b < p.boxes; ++b)
-          ptx::tma_load_2d(smem_addr(s_kv + stage * page_bytes + b * kBoxBytes), &tmap_kv, bar, b * 64, slot * kPage);
-        if (++stage == p.stages) { stage = 0; phase ^= 1; }
-        if (it == 0) {
-          ptx::mbar_expect_tx(smem_addr(bar_q), p.boxes * NR * 128);
-          for (int b = 0; b < p.boxes; ++b)
-            ptx::tma_load_2d(smem_addr(s_q + b * NR * 128), &tmap_q, smem_addr(bar_q), b * 64, row0 * a.heads + head0);
-        }
+        load_page(it);
       }
       // nothing may still be on its way when the block ends, also after a wait that gave up
       ptx::mbar_wait(smem_addr(bar_q), 0, &g_latent_status, (7 << 8) | 8);
@@ -354,6 +354,7 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_kv, const __gri
         ptx::tc_fence_after();
         uint64_t aq = dq, bk = dk + static_cast<uint64_t>(s_stage * page_bytes >> 4);
         const uint32_t d = tmem_s + (it & 1) * kPage;
+#pragma unroll 1
         for (int b = 0; b < p.boxes; ++b) {  // (columns beyond the row are zero in both operands)
 #pragma unroll
           for (int j = 0; j < 4; ++j) mma_f16_ss(lead, d, aq + 2 * j, bk + 2 * j, id_s, (b | j) > 0 ? 1u : 0u);
@@ -364,20 +365,23 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_kv, const __gri
         __syncwarp();
         if (++s_stage == p.stages) { s_stage = 0; s_phase ^= 1; }
       };
-      ok = ptx::mbar_wait(smem_addr(bar_q), 0, &g_latent_status, (7 << 8) | 3);
-      scores(0);
       int o_stage = 0;
-      for (int it = 0; it < npages; ++it) {
-        if (p.ahead && it + 1 < npages) scores(it + 1);
+      ok = ptx::mbar_wait(smem_addr(bar_q), 0, &g_latent_status, (7 << 8) | 3);
+#pragma unroll 1
+      for (int step = 0; step < npages + p.ahead; ++step) {      // (one copy of the code: it is fetched cold)
+        if (step < npages) scores(step);
+        const int it = step - p.ahead;
+        if (it < 0) continue;
         ok = ok && ptx::mbar_wait(smem_addr(&bar_p[it & 1]), (it >> 1) & 1, &g_latent_status, (7 << 8) | 4);
         __syncwarp();
         ptx::tc_fence_after();
         uint64_t av = dv + static_cast<uint64_t>(o_stage * page_bytes >> 4);
         const uint64_t pb = dp + static_cast<uint64_t>((p.ahead ? it & 1 : 0) * (NR * 128 >> 4));
+#pragma unroll 1
         for (int m = 0; m < p.blocks; ++m) {
 #pragma unroll
           for (int j = 0; j < 4; ++j)        // 16 keys
-            mma_f16_ss(lead, tmem + m * NR, av + j * (2048 >> 4), pb + 2 * j, id_o, (it | j) > 0 ? 1u : 0u);
+            mma_f16_ss(lead, tmem + m * NR, av + j * (2048 >> 4), pb + 2 * j, id_o, it > 0 || j > 0 ? 1u : 0u);
           av += 2 * kBoxBytes >> 4;
         }
         if (lead) {
@@ -386,7 +390,6 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_kv, const __gri
         }
         __syncwarp();
         if (++o_stage == p.stages) o_stage = 0;
-        if (!p.ahead && it + 1 < npages) scores(it + 1);
       }
       if (lead) ptx::tc_commit(smem_addr(bar_done));
     }
@@ -408,7 +411,6 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_kv, const __gri
     }
     const float qscale = a.scale * kLog2e;
     const uint32_t lane_addr = static_cast<uint32_t>(quarter * 32) << 16;
-    int stage = 0;
     for (int it = 0; it < npages; ++it) {
       const int buf = p.ahead ? it & 1 : 0;
       ok = ok && ptx::mbar_wait(smem_addr(&bar_s[it & 1]), (it >> 1) & 1, &g_latent_status, (7 << 8) | 5);
@@ -566,49 +568,54 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_kv, const __gri
     }
   }
   if (p.splits > 1) {
-    // the cluster's CTAs share one tile: rows dealt out, parts added in rank order
+    // The cluster's CTAs share one tile. CTA d finishes rows d * share ..; every CTA sends it those rows of its part with one
+    // bulk copy, so that the sums read local memory. Parts are added in rank order.
+    const int opitch = a.kv_rank + 4, share = (used + p.splits - 1) / p.splits;
+    const int mine = min(max(used - split * share, 0), share);
+    float* s_o = reinterpret_cast<float*>(smem);
+    float* s_in = s_o + NR * opitch;                            // [splits][share][opitch]
+    const uint32_t bar_in = smem_addr(bar_q);                   // its second phase
+    asm volatile("fence.proxy.async.shared::cta;" ::: "memory");   // this CTA's part, before the copy engine reads it
+    if (threadIdx.x == 0) ptx::mbar_expect_tx(bar_in, p.splits * mine * opitch * 4);
     __syncwarp();
-    cluster_sync_all();
-    const float* s_o = reinterpret_cast<const float*>(smem);
-    const int opitch = a.kv_rank + 4, mine = (used - split + p.splits - 1) / p.splits;       // rows split, split + splits, ...
-    if (static_cast<int>(threadIdx.x) < mine) {
-      const int r = split + threadIdx.x * p.splits;
-      float m[kMaxSplits], l[kMaxSplits], top = -1e30f, sum = 0.f;
-#pragma unroll
-      for (int s = 0; s < kMaxSplits; ++s) {
-        m[s] = s < p.splits ? ld_peer_f32(smem_addr(s_ml + r), s) : -1e30f;
-        l[s] = s < p.splits ? ld_peer_f32(smem_addr(s_ml + NR + r), s) : 0.f;
-      }
-#pragma unroll
-      for (int s = 0; s < kMaxSplits; ++s) top = fmaxf(top, m[s]);
-#pragma unroll
-      for (int s = 0; s < kMaxSplits; ++s) {
-        m[s] = ex2(m[s] - top);
-        sum = fmaf(l[s], m[s], sum);
-      }
-#pragma unroll
-      for (int s = 0; s < kMaxSplits; ++s) s_w[threadIdx.x * kMaxSplits + s] = m[s] / sum;
+    cluster_sync_all();                    // every ring is drained, every barrier is armed
+    if (threadIdx.x < p.splits) {
+      const int d = (split + threadIdx.x) % p.splits, rows = min(max(used - d * share, 0), share);
+      if (rows > 0)
+        ptx::bulk_copy_to_rank(smem_addr(s_in + split * share * opitch), smem_addr(s_o + d * share * opitch), rows * opitch * 4, bar_in, d);
+    }
+    // references and denominators of my rows in every part
+    for (int i = threadIdx.x; i < mine * p.splits; i += kThreads) {
+      const int k = i / p.splits, src = i - k * p.splits;
+      s_w[(k * kMaxSplits + src) * 2] = ld_peer_f32(smem_addr(s_ml + split * share + k), src);
+      s_w[(k * kMaxSplits + src) * 2 + 1] = ld_peer_f32(smem_addr(s_ml + NR + split * share + k), src);
     }
     __syncthreads();
-    const int pieces = a.kv_rank / 4;
+    // (phase 0 is over when this CTA loaded its queries, else it is the current one)
+    ok = ptx::mbar_wait(bar_in, npages > 0 ? 1 : 0, &g_latent_status, (7 << 8) | 10) && ok;
+    const int pieces = a.kv_rank / 8;
+#pragma unroll 1
     for (int i = threadIdx.x; i < mine * pieces; i += kThreads) {
-      const int k = i / pieces, c = (i % pieces) * 4, r = split + k * p.splits;
-      float4 part[kMaxSplits];
+      const int k = i / pieces, c = (i - k * pieces) * 8;
+      const float* ml = s_w + k * kMaxSplits * 2;
+      float top = ml[0], sum = 0.f, v[8] = {};
+#pragma unroll 1
+      for (int part = 1; part < p.splits; ++part) top = fmaxf(top, ml[2 * part]);
+#pragma unroll 1
+      for (int part = 0; part < p.splits; ++part) {
+        const float w = ex2(ml[2 * part] - top);
+        sum = fmaf(ml[2 * part + 1], w, sum);
+        const float4* src = reinterpret_cast<const float4*>(s_in + (part * share + k) * opitch + c);
+        const float4 x = src[0], y = src[1];
+        v[0] = fmaf(x.x, w, v[0]); v[1] = fmaf(x.y, w, v[1]); v[2] = fmaf(x.z, w, v[2]); v[3] = fmaf(x.w, w, v[3]);
+        v[4] = fmaf(y.x, w, v[4]); v[5] = fmaf(y.y, w, v[5]); v[6] = fmaf(y.z, w, v[6]); v[7] = fmaf(y.w, w, v[7]);
+      }
+      const float inv = 1.f / sum;
 #pragma unroll
-      for (int s = 0; s < kMaxSplits; ++s)
-        if (s < p.splits) part[s] = ld_peer_f32x4(smem_addr(s_o + r * opitch + c), s);
-      float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-#pragma unroll
-      for (int s = 0; s < kMaxSplits; ++s)
-        if (s < p.splits) {
-          const float w = s_w[k * kMaxSplits + s];
-          v.x = fmaf(part[s].x, w, v.x); v.y = fmaf(part[s].y, w, v.y); v.z = fmaf(part[s].z, w, v.z); v.w = fmaf(part[s].w, w, v.w);
-        }
-      uint2 raw;
-      raw.x = pack_bf16(v.x, v.y);
-      raw.y = pack_bf16(v.z, v.w);
-      *reinterpret_cast<uint2*>(p.out + (static_cast<size_t>(row0) * a.heads + head0 + r) * a.kv_rank + c) = raw;
+      for (int e = 0; e < 8; ++e) v[e] *= inv;
+      VecIO<__nv_bfloat16, 8>::st(p.out + (static_cast<size_t>(row0) * a.heads + head0 + split * share + k) * a.kv_rank + c, v);
     }
+    __syncwarp();
     cluster_sync_all();                    // nobody leaves while its part is being read
   }
   ptx::tc_fence_before();
@@ -664,8 +671,10 @@ int launch_fast(FastParams p, const void* q, dim3 grid, cudaStream_t st) {
   const int cols = p.blocks * NR + 2 * kPage;
   p.tmem_cols = cols <= 256 ? 256 : 512;
   size_t smem = fast_fixed_smem(NR, p.boxes, p.ahead) + static_cast<size_t>(p.stages) * p.boxes * kBoxBytes;
-  if (p.splits > 1 && static_cast<size_t>(NR) * (p.a.kv_rank + 4) * 4 > static_cast<size_t>(p.stages) * p.boxes * kBoxBytes)
-    return CACHEIR_B200_EUNSUPPORTED;        // (the combine's tile lies over the ring)
+  // the combine's tile and what the peers send lie over ring, queries and probabilities
+  const size_t combine = static_cast<size_t>(NR + (NR + p.splits - 1) / p.splits * p.splits) * (p.a.kv_rank + 4) * 4;
+  if (p.splits > 1 && combine > static_cast<size_t>(p.stages) * p.boxes * kBoxBytes + static_cast<size_t>(p.boxes) * NR * 128)
+    return CACHEIR_B200_EUNSUPPORTED;
   // No more CTAs on an SM than its tensor memory serves: one that waited for an allocation could hold up its cluster.
   const size_t least = kSmemLimit / (512 / p.tmem_cols + 1) + 1024;
   if (smem < least) smem = least;
@@ -792,7 +801,7 @@ extern "C" int cacheir_b200_latent_attention(const cacheir_b200_latent_args* arg
   p.sink = sink;
   p.out = static_cast<__nv_bfloat16*>(out);
   p.splits = splits;
-  int rows = tile_rows(a.kv_rank + a.rot_dim);
+  int rows = splits > 1 ? 32 : tile_rows(a.kv_rank + a.rot_dim);      // (a split 64-row tile would not fit its combine)
   const int groups = head_groups(a.heads, rows);
   p.heads_per_cta = (a.heads + groups - 1) / groups;
   if (decode && p.heads_per_cta <= 32) rows = 32;
