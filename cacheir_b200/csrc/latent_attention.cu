@@ -165,7 +165,8 @@ struct FastParams {
   int boxes;                   // 64-column boxes of a cache row
   int blocks;                  // 128-column blocks of the latent
   int stages;
-  int ahead;                   // the next page's scores are issued before this page's output (three pages in the ring)
+  int ahead;                   // three pages in the ring: the next page's scores are issued before this page's output
+  int p_in_page;               // probabilities overwrite the page's box of rotated key parts, which the scores are done with
   int tmem_cols;
 };
 
@@ -180,14 +181,18 @@ __device__ __forceinline__ void cluster_sync_all() {
   asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory");
   asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory");
 }
-// Executed by a whole warp so that the operands stay in uniform registers; `lead` picks the issuing lane.
-__device__ __forceinline__ void mma_f16_ss(uint32_t lead, uint32_t tmem_d, uint64_t a_desc, uint64_t b_desc, uint32_t idesc, uint32_t accumulate) {
+// Executed by a whole warp so that the operands stay in uniform registers; `lead` picks the issuing lane. Descriptors come as
+// their two words: only the address word changes.
+__device__ __forceinline__ void mma_f16_ss(uint32_t lead, uint32_t tmem_d, uint32_t a_lo, uint32_t a_hi, uint32_t b_lo, uint32_t b_hi,
+                                           uint32_t idesc, uint32_t accumulate) {
   asm volatile(
-      "{\n\t.reg .pred p, q;\n\t"
-      "setp.ne.b32 p, %4, 0;\n\t"
-      "setp.ne.b32 q, %5, 0;\n\t"
-      "@q tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, p;\n\t}"
-      ::"r"(tmem_d), "l"(a_desc), "l"(b_desc), "r"(idesc), "r"(accumulate), "r"(lead) : "memory");
+      "{\n\t.reg .pred p, q;\n\t.reg .b64 a, b;\n\t"
+      "mov.b64 a, {%1, %2};\n\t"
+      "mov.b64 b, {%3, %4};\n\t"
+      "setp.ne.b32 p, %6, 0;\n\t"
+      "setp.ne.b32 q, %7, 0;\n\t"
+      "@q tcgen05.mma.cta_group::1.kind::f16 [%0], a, b, %5, p;\n\t}"
+      ::"r"(tmem_d), "r"(a_lo), "r"(a_hi), "r"(b_lo), "r"(b_hi), "r"(idesc), "r"(accumulate), "r"(lead) : "memory");
 }
 __device__ __forceinline__ float ex2(float x) {
   float y;
@@ -251,11 +256,11 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_kv, const __gri
   const int width = a.kv_rank + a.rot_dim;
   uint8_t* s_kv = smem;                                         // [stages][boxes][64 rows][128 bytes], swizzled
   uint8_t* s_q = s_kv + p.stages * page_bytes;                  // [boxes][NR rows][128 bytes], swizzled
-  uint8_t* s_p = s_q + p.boxes * NR * 128;                      // [1 + ahead][NR rows][128 bytes], swizzled
-  float* s_alpha = reinterpret_cast<float*>(s_p + (1 + p.ahead) * NR * 128);   // [NR]
-  float* s_max = s_alpha + NR;                                  // [2 key halves][NR]
-  float* s_ml = s_max + 2 * NR;                                 // [NR] references, [NR] denominators
-  float* s_w = reinterpret_cast<float*>(s_p);                   // [rows][kMaxSplits][2]: what the combine weighs with (over s_p)
+  uint8_t* s_p = s_q + p.boxes * NR * 128;                      // [2][NR rows][128 bytes], swizzled; absent with p_in_page
+  float* s_alpha = reinterpret_cast<float*>(s_p + (p.p_in_page ? 0 : 2 * NR * 128));   // [NR]
+  float* s_max = s_alpha + NR;                                  // [2 pages][2 key halves][NR]
+  float* s_ml = s_max + 4 * NR;                                 // [NR] references, [NR] denominators
+  float* s_w = reinterpret_cast<float*>(s_q);                   // [rows][kMaxSplits][2]: what the combine weighs with (over the queries)
   uint64_t* full = reinterpret_cast<uint64_t*>(s_ml + 2 * NR);  // [stages] a page has landed
   uint64_t* empty = full + kMaxStages;                          // [stages] its output MMAs have retired
   uint64_t* bar_q = empty + kMaxStages;
@@ -345,43 +350,49 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_kv, const __gri
       const uint32_t id_s = (1u << 4) | (1u << 7) | (1u << 10) | (static_cast<uint32_t>(kPage >> 3) << 17) | (static_cast<uint32_t>(64 >> 4) << 24);
       const uint32_t id_o = (1u << 4) | (1u << 7) | (1u << 10) | (1u << 15) | (static_cast<uint32_t>(NR >> 3) << 17) |
                             (static_cast<uint32_t>(128 >> 4) << 24);
-      const uint64_t dq = ptx::smem_desc_sw128(smem_addr(s_q)), dk = ptx::smem_desc_sw128(smem_addr(s_kv)), dp = ptx::smem_desc_sw128(smem_addr(s_p));
+      const uint64_t dq = ptx::smem_desc_sw128(smem_addr(s_q)), dk = ptx::smem_desc_sw128(smem_addr(s_kv));
+      const uint64_t dp = ptx::smem_desc_sw128(smem_addr(p.p_in_page ? s_kv + 2 * p.blocks * kBoxBytes : s_p));
       const uint64_t dv = smem_desc_mn_sw128(smem_addr(s_kv), kBoxBytes);
-      int s_stage = 0, s_phase = 0;          // next page to score
-      auto scores = [&](int it) {
-        ok = ok && ptx::mbar_wait(smem_addr(&full[s_stage]), s_phase, &g_latent_status, (7 << 8) | 2);
-        __syncwarp();
-        ptx::tc_fence_after();
-        uint64_t aq = dq, bk = dk + static_cast<uint64_t>(s_stage * page_bytes >> 4);
-        const uint32_t d = tmem_s + (it & 1) * kPage;
-#pragma unroll 1
-        for (int b = 0; b < p.boxes; ++b) {  // (columns beyond the row are zero in both operands)
-#pragma unroll
-          for (int j = 0; j < 4; ++j) mma_f16_ss(lead, d, aq + 2 * j, bk + 2 * j, id_s, (b | j) > 0 ? 1u : 0u);
-          aq += NR * 128 >> 4;
-          bk += kBoxBytes >> 4;
-        }
-        if (lead) ptx::tc_commit(smem_addr(&bar_s[it & 1]));
-        __syncwarp();
-        if (++s_stage == p.stages) { s_stage = 0; s_phase ^= 1; }
-      };
-      int o_stage = 0;
+      const uint32_t k_hi = static_cast<uint32_t>(dk >> 32), v_hi = static_cast<uint32_t>(dv >> 32);     // (dq, dk, dp share theirs)
+      const uint32_t stage_step = static_cast<uint32_t>(page_bytes >> 4);
+      int s_stage = 0, s_phase = 0, o_stage = 0;
+      int next_s = 0, next_o = 0;            // next page to score, next page to add to the output
+      bool fill = true;
       ok = ptx::mbar_wait(smem_addr(bar_q), 0, &g_latent_status, (7 << 8) | 3);
+      // Two pages are scored before the first one's output, so that softmax runs beside MMAs. With a ring of two pages they go
+      // pair by pair: the second page's output overlaps the next pair's loads.
 #pragma unroll 1
-      for (int step = 0; step < npages + p.ahead; ++step) {      // (one copy of the code: it is fetched cold)
-        if (step < npages) scores(step);
-        const int it = step - p.ahead;
-        if (it < 0) continue;
-        ok = ok && ptx::mbar_wait(smem_addr(&bar_p[it & 1]), (it >> 1) & 1, &g_latent_status, (7 << 8) | 4);
+      while (next_o < npages) {
+        if (next_s < npages && (p.ahead ? next_s - next_o < 2 : fill)) {
+          ok = ok && ptx::mbar_wait(smem_addr(&full[s_stage]), s_phase, &g_latent_status, (7 << 8) | 2);
+          __syncwarp();
+          ptx::tc_fence_after();
+          uint32_t aq = static_cast<uint32_t>(dq), bk = static_cast<uint32_t>(dk) + s_stage * stage_step;
+          const uint32_t d = tmem_s + (next_s & 1) * kPage;
+#pragma unroll 1
+          for (int b = 0; b < p.boxes; ++b) {  // (columns beyond the row are zero in both operands)
+#pragma unroll
+            for (int j = 0; j < 4; ++j) mma_f16_ss(lead, d, aq + 2 * j, k_hi, bk + 2 * j, k_hi, id_s, (b | j) > 0 ? 1u : 0u);
+            aq += NR * 128 >> 4;
+            bk += kBoxBytes >> 4;
+          }
+          if (lead) ptx::tc_commit(smem_addr(&bar_s[next_s & 1]));
+          __syncwarp();
+          if (++s_stage == p.stages) { s_stage = 0; s_phase ^= 1; }
+          ++next_s;
+          fill = next_s - next_o < 2;
+          continue;
+        }
+        ok = ok && ptx::mbar_wait(smem_addr(&bar_p[next_o & 1]), (next_o >> 1) & 1, &g_latent_status, (7 << 8) | 4);
         __syncwarp();
         ptx::tc_fence_after();
-        uint64_t av = dv + static_cast<uint64_t>(o_stage * page_bytes >> 4);
-        const uint64_t pb = dp + static_cast<uint64_t>((p.ahead ? it & 1 : 0) * (NR * 128 >> 4));
+        uint32_t av = static_cast<uint32_t>(dv) + o_stage * stage_step;
+        const uint32_t pb = static_cast<uint32_t>(dp) + (p.p_in_page ? o_stage * stage_step : (next_o & 1) * (NR * 128 >> 4));
 #pragma unroll 1
         for (int m = 0; m < p.blocks; ++m) {
 #pragma unroll
           for (int j = 0; j < 4; ++j)        // 16 keys
-            mma_f16_ss(lead, tmem + m * NR, av + j * (2048 >> 4), pb + 2 * j, id_o, it > 0 || j > 0 ? 1u : 0u);
+            mma_f16_ss(lead, tmem + m * NR, av + j * (2048 >> 4), v_hi, pb + 2 * j, k_hi, id_o, next_o > 0 || j > 0 ? 1u : 0u);
           av += 2 * kBoxBytes >> 4;
         }
         if (lead) {
@@ -390,6 +401,8 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_kv, const __gri
         }
         __syncwarp();
         if (++o_stage == p.stages) o_stage = 0;
+        ++next_o;
+        fill = next_o == next_s;
       }
       if (lead) ptx::tc_commit(smem_addr(bar_done));
     }
@@ -412,11 +425,12 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_kv, const __gri
     const float qscale = a.scale * kLog2e;
     const uint32_t lane_addr = static_cast<uint32_t>(quarter * 32) << 16;
     for (int it = 0; it < npages; ++it) {
-      const int buf = p.ahead ? it & 1 : 0;
+      uint8_t* p_tile = p.p_in_page ? s_kv + stage * page_bytes + 2 * p.blocks * kBoxBytes : s_p + (it & 1) * NR * 128;
       ok = ok && ptx::mbar_wait(smem_addr(&bar_s[it & 1]), (it >> 1) & 1, &g_latent_status, (7 << 8) | 5);
       __syncwarp();
       ptx::tc_fence_after();
       float s[16], alpha[2] = {1.f, 1.f};
+      bool grown = false;
       const int base = (pg_begin + it) * kPage;
       if (band) {
         tmem_ld_rows16(tmem_s + (it & 1) * kPage + half * 32 + lane_addr, s);
@@ -440,9 +454,11 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_kv, const __gri
 #pragma unroll
           for (int e = 0; e < 2; ++e) mx[e] = fmaxf(mx[e], __shfl_xor_sync(0xffffffffu, mx[e], off));
         if ((lane & 3) == 0) {
-          s_max[half * NR + r0] = mx[0];
-          s_max[half * NR + r0 + 8] = mx[1];
+          s_max[((it & 1) * 2 + half) * NR + r0] = mx[0];
+          s_max[((it & 1) * 2 + half) * NR + r0 + 8] = mx[1];
         }
+        // (this half's keys decide for the row as soon as they exceed the bound)
+        grown = it > 0 && ((row_pos[0] >= 0 && mx[0] > m_ref[0] + kStale) || (row_pos[1] >= 0 && mx[1] > m_ref[1] + kStale));
       }
       const int tail = pos_last + 1 - base;
       if (tail < kPage) {                    // rows behind the last token may hold anything: zero, so that 0 * row stays 0
@@ -453,20 +469,18 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_kv, const __gri
         asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
       }
       if (++stage == p.stages) stage = 0;
-      sync_softmax();
-      bool grown = false;
+      const bool rescale = any_softmax(grown);       // (also publishes s_max)
       if (band) {
 #pragma unroll
         for (int e = 0; e < 2; ++e) {
-          const float mx = fmaxf(s_max[r0 + 8 * e], s_max[NR + r0 + 8 * e]);
+          const float mx = fmaxf(s_max[(it & 1) * 2 * NR + r0 + 8 * e], s_max[((it & 1) * 2 + 1) * NR + r0 + 8 * e]);
           if (row_pos[e] >= 0 && mx > m_ref[e] + (it == 0 ? 0.f : kStale)) {
             alpha[e] = ex2(m_ref[e] - mx);
             m_ref[e] = mx;
-            grown = it > 0;
           }
         }
       }
-      if (any_softmax(grown)) {              // rare: bring O^T to the new references
+      if (rescale) {                         // rare: bring O^T to the new references
         if (band && half == 0 && (lane & 3) == 0) {
           s_alpha[r0] = alpha[0];
           s_alpha[r0 + 8] = alpha[1];
@@ -488,7 +502,7 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_kv, const __gri
       if (band) {
 #pragma unroll
         for (int e = 0; e < 2; ++e) l_run[e] *= alpha[e];
-        uint8_t* dst = s_p + (buf * NR + r0) * 128 + (lane & 3) * 4;
+        uint8_t* dst = p_tile + r0 * 128 + (lane & 3) * 4;
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
 #pragma unroll
@@ -628,23 +642,22 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_kv, const __gri
 
 constexpr size_t kSmemLimit = 227 * 1024;
 int row_boxes(int width) { return (width + 63) / 64; }
-// Shared memory beside the ring, and the ring's pages: `ahead` when three fit.
-size_t fast_fixed_smem(int nr, int boxes, int ahead) {
-  return 1024 + static_cast<size_t>(boxes + 1 + ahead) * nr * 128 + nr * 5 * 4 + (2 * kMaxStages + 8) * 8 + 16;
+// Shared memory beside the ring, and the pages that fit (at least two).
+size_t fast_fixed_smem(int nr, int boxes, int p_in_page) {
+  // (the score MMAs read 64 query rows: behind a 32-row tile's last box lies memory of this block)
+  const size_t behind = p_in_page && nr == 32 ? 4096 : 0;
+  return 1024 + behind + static_cast<size_t>(boxes + (p_in_page ? 0 : 2)) * nr * 128 + nr * 7 * 4 + (2 * kMaxStages + 8) * 8 + 16;
 }
-struct Ring { int stages, ahead; };
-Ring fast_ring(int nr, int width) {
+int latent_blocks(int kv_rank) { return (kv_rank + 127) / 128; }
+int prob_in_page(int kv_rank, int width) { return row_boxes(width) > 2 * latent_blocks(kv_rank) ? 1 : 0; }
+int fast_stages(int nr, int kv_rank, int width) {
   const int boxes = row_boxes(width);
-  const size_t page = static_cast<size_t>(boxes) * kBoxBytes;
-  for (int ahead = 1; ahead >= 0; --ahead) {
-    const size_t fixed = fast_fixed_smem(nr, boxes, ahead);
-    int s = fixed > kSmemLimit ? 0 : static_cast<int>((kSmemLimit - fixed) / page);
-    if (s > kMaxStages) s = kMaxStages;
-    if (s >= (ahead ? 3 : 2)) return {s, ahead};
-  }
-  return {0, 0};
+  const size_t page = static_cast<size_t>(boxes) * kBoxBytes, fixed = fast_fixed_smem(nr, boxes, prob_in_page(kv_rank, width));
+  int s = fixed > kSmemLimit ? 0 : static_cast<int>((kSmemLimit - fixed) / page);
+  if (s > kMaxStages) s = kMaxStages;
+  return s >= 2 ? s : 0;
 }
-int tile_rows(int width) { return fast_ring(64, width).stages > 0 ? 64 : 32; }
+int tile_rows(int kv_rank, int width) { return fast_stages(64, kv_rank, width) > 0 ? 64 : 32; }
 int head_groups(int heads, int rows) { return (heads + rows - 1) / rows; }
 
 bool encode_rows(CUtensorMap* map, const void* base, uint64_t width, uint64_t rows, uint32_t box_rows) {
@@ -662,19 +675,18 @@ bool encode_rows(CUtensorMap* map, const void* base, uint64_t width, uint64_t ro
 template <int NR>
 int launch_fast(FastParams p, const void* q, dim3 grid, cudaStream_t st) {
   const int width = p.a.kv_rank + p.a.rot_dim;
-  const Ring ring = fast_ring(NR, width);
-  if (ring.stages == 0) return CACHEIR_B200_EUNSUPPORTED;
+  p.stages = fast_stages(NR, p.a.kv_rank, width);
+  if (p.stages == 0) return CACHEIR_B200_EUNSUPPORTED;
   p.boxes = row_boxes(width);
-  p.blocks = (p.a.kv_rank + 127) / 128;
-  p.stages = ring.stages;
-  p.ahead = ring.ahead;
+  p.blocks = latent_blocks(p.a.kv_rank);
+  p.ahead = p.stages >= 3 ? 1 : 0;
+  p.p_in_page = prob_in_page(p.a.kv_rank, width);
   const int cols = p.blocks * NR + 2 * kPage;
   p.tmem_cols = cols <= 256 ? 256 : 512;
-  size_t smem = fast_fixed_smem(NR, p.boxes, p.ahead) + static_cast<size_t>(p.stages) * p.boxes * kBoxBytes;
-  // the combine's tile and what the peers send lie over ring, queries and probabilities
+  size_t smem = fast_fixed_smem(NR, p.boxes, p.p_in_page) + static_cast<size_t>(p.stages) * p.boxes * kBoxBytes;
+  // the combine's tile and what the peers send lie over the ring
   const size_t combine = static_cast<size_t>(NR + (NR + p.splits - 1) / p.splits * p.splits) * (p.a.kv_rank + 4) * 4;
-  if (p.splits > 1 && combine > static_cast<size_t>(p.stages) * p.boxes * kBoxBytes + static_cast<size_t>(p.boxes) * NR * 128)
-    return CACHEIR_B200_EUNSUPPORTED;
+  if (p.splits > 1 && combine > static_cast<size_t>(p.stages) * p.boxes * kBoxBytes) return CACHEIR_B200_EUNSUPPORTED;
   // No more CTAs on an SM than its tensor memory serves: one that waited for an allocation could hold up its cluster.
   const size_t least = kSmemLimit / (512 / p.tmem_cols + 1) + 1024;
   if (smem < least) smem = least;
@@ -771,7 +783,7 @@ extern "C" int cacheir_b200_latent_attention_simple(const cacheir_b200_latent_ar
 
 extern "C" int cacheir_b200_latent_attention_supported(int kv_rank, int rot_dim, int page_size, int dtype) {
   return dtype == CACHEIR_B200_BF16 && page_size == kPage && kv_rank >= 8 && kv_rank % 8 == 0 && kv_rank <= 512 && rot_dim >= 0 &&
-         rot_dim % 8 == 0 && fast_ring(32, kv_rank + rot_dim).stages > 0 ? 1 : 0;
+         rot_dim % 8 == 0 && fast_stages(32, kv_rank, kv_rank + rot_dim) > 0 ? 1 : 0;
 }
 
 extern "C" int cacheir_b200_latent_attention_splits(int rows, int heads, int window, int max_pages, int page_size) {
@@ -801,7 +813,7 @@ extern "C" int cacheir_b200_latent_attention(const cacheir_b200_latent_args* arg
   p.sink = sink;
   p.out = static_cast<__nv_bfloat16*>(out);
   p.splits = splits;
-  int rows = splits > 1 ? 32 : tile_rows(a.kv_rank + a.rot_dim);      // (a split 64-row tile would not fit its combine)
+  int rows = splits > 1 ? 32 : tile_rows(a.kv_rank, a.kv_rank + a.rot_dim);      // (a split 64-row tile would not fit its combine)
   const int groups = head_groups(a.heads, rows);
   p.heads_per_cta = (a.heads + groups - 1) / groups;
   if (decode && p.heads_per_cta <= 32) rows = 32;
