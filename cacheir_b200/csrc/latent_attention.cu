@@ -295,14 +295,24 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_kv, const __gri
 
   // The copy warp sets the barriers up and requests the first pages before the block meets.
   int stage = 0, phase = 1;                // its place in the ring
-  auto load_page = [&](int it) {
+  auto page_row = [&](int it) {            // the page's first row in the pool
     const int pg = pg_begin + it;
-    int slot = pg < a.max_pages ? a.page_table[static_cast<size_t>(seg) * a.max_pages + pg] : 0;
-    slot = min(max(slot, 0), a.num_slots - 1);
+    const int slot = pg < a.max_pages ? a.page_table[static_cast<size_t>(seg) * a.max_pages + pg] : 0;
+    return min(max(slot, 0), a.num_slots - 1) * kPage;
+  };
+  auto prefetch_page = [&](int it) {       // into L2, before the ring has room
+    if (it >= npages || !a.decode) return;       // (a prompt's tiles find their pages there)
+    const int row = page_row(it);
+    for (int b = 0; b < p.boxes; ++b)
+      asm volatile("cp.async.bulk.prefetch.tensor.2d.L2.global [%0, {%1, %2}];"
+                   ::"l"(reinterpret_cast<uint64_t>(&tmap_kv)), "r"(b * 64), "r"(row) : "memory");
+  };
+  auto load_page = [&](int it) {
+    const int row = page_row(it);
     const uint32_t bar = smem_addr(&full[stage]);
     ptx::mbar_expect_tx(bar, page_bytes);
     for (int b = 0; b < p.boxes; ++b)
-      ptx::tma_load_2d(smem_addr(s_kv + stage * page_bytes + b * kBoxBytes), &tmap_kv, bar, b * 64, slot * kPage);
+      ptx::tma_load_2d(smem_addr(s_kv + stage * page_bytes + b * kBoxBytes), &tmap_kv, bar, b * 64, row);
     if (++stage == p.stages) { stage = 0; phase ^= 1; }
   };
   const int first = min(npages, p.stages);
@@ -318,6 +328,7 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_kv, const __gri
       for (int b = 0; b < p.boxes; ++b)
         ptx::tma_load_2d(smem_addr(s_q + b * NR * 128), &tmap_q, smem_addr(bar_q), b * 64, row0 * a.heads + head0);
       for (int it = 0; it < first; ++it) load_page(it);
+      for (int it = first; it < first + 2; ++it) prefetch_page(it);
     }
   }
   __syncwarp();
@@ -336,6 +347,7 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_kv, const __gri
         ok = ok && ptx::mbar_wait(smem_addr(&empty[stage]), phase, &g_latent_status, (7 << 8) | 1);
         if (!ok) break;
         load_page(it);
+        prefetch_page(it + 2);
       }
       // nothing may still be on its way when the block ends, also after a wait that gave up
       ptx::mbar_wait(smem_addr(bar_q), 0, &g_latent_status, (7 << 8) | 8);
