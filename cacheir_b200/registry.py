@@ -52,6 +52,22 @@ KERNEL_FOR_OP: dict[str, tuple[str, tuple[str, ...]]] = {
     "add": ("triton.vector_add", ("cacheir_b200_add", "cacheir_b200_qgemv")),
 }
 
+# graph ops of the hybrid families -> C entry points of libcacheir_b200_hybrid.so (tensor-core forms first)
+HYBRID_KERNELS_FOR_OP: dict[str, tuple[str, ...]] = {
+    "scaled_token_embedding": ("cacheir_b200_scaled_embedding",),
+    "dynamic_tanh": ("cacheir_b200_dyt_rows",),
+    "concat_matmul": ("cacheir_b200_dense_gemm", "cacheir_b200_dense_simple", "cacheir_b200_silu_cols"),
+    "matmul": ("cacheir_b200_dense_gemm", "cacheir_b200_dense_simple"),
+    "latent_attention": ("cacheir_b200_latent_prepare", "cacheir_b200_dense_gemm", "cacheir_b200_latent_attention",
+                         "cacheir_b200_latent_attention_simple"),
+    "linear_recurrence": ("cacheir_b200_recurrence_step", "cacheir_b200_recurrence_chunked", "cacheir_b200_recurrence_simple"),
+    "gated_rms_norm": ("cacheir_b200_gated_rms",),
+    "residual_dynamic_tanh": ("cacheir_b200_dense_gemm", "cacheir_b200_residual_dyt"),
+    "fused_geglu": ("cacheir_b200_dense_gemm", "cacheir_b200_dense_simple", "cacheir_b200_geglu_pairs"),
+    "token_side_gate": ("cacheir_b200_dense_gemm", "cacheir_b200_dense_simple", "cacheir_b200_gelu_embed"),
+    "residual_rms_norm": ("cacheir_b200_residual_rms",),
+}
+
 B200_BACKEND = Backend(
     name="cuda-b200",
     devices=("sm100a",),
@@ -72,6 +88,9 @@ B200_BACKEND = Backend(
         "kv_page_append",
         "quant_pack_rows",
         "cuda_graph_decode_replay",
+        "dense_gemm_bf16",
+        "latent_attention",
+        "linear_recurrence",
     ),
     notes="Hand-written sm_100a kernels behind a C ABI (libcacheir_b200.so): split-K paged decode attention over a "
           "shared page pool, packed int4/int8 dequant-GEMV, fused glue ops; decode step replayed as a CUDA graph.",

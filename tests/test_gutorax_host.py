@@ -89,6 +89,15 @@ def test_graph_follows_the_configuration():
     assert "token_side_gate" not in [n.op for n in build_gutorax_graph(GutoraxConfig.from_dict(CONFIGS["no_side"])).nodes]
 
 
+def test_every_graph_op_has_kernels_in_the_registry():
+    from cacheir_b200 import _lib, registry
+    from cacheir_b200.gutorax import GutoraxConfig, build_gutorax_graph
+
+    used = {n.op for cfg in CONFIGS.values() for n in build_gutorax_graph(GutoraxConfig.from_dict(cfg)).nodes}
+    assert used == set(registry.HYBRID_KERNELS_FOR_OP)
+    assert {k for names in registry.HYBRID_KERNELS_FOR_OP.values() for k in names} <= set(_lib.HYBRID_SIGNATURES)
+
+
 @pytest.mark.parametrize("change", [
     lambda c: c["layers"][1]["mixer"]["decay"].append(0.5),
     lambda c: c["layers"][2]["mixer"].update(kv_from=1),
