@@ -253,7 +253,6 @@ latent_attention_kernel(const __grid_constant__ CUtensorMap tmap_kv, const __gri
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~static_cast<uintptr_t>(1023));
   const cacheir_b200_latent_args& a = p.a;
   const int page_bytes = p.boxes * kBoxBytes;
-  const int width = a.kv_rank + a.rot_dim;
   uint8_t* s_kv = smem;                                         // [stages][boxes][64 rows][128 bytes], swizzled
   uint8_t* s_q = s_kv + p.stages * page_bytes;                  // [boxes][NR rows][128 bytes], swizzled
   uint8_t* s_p = s_q + p.boxes * NR * 128;                      // [2][NR rows][128 bytes], swizzled; absent with p_in_page
