@@ -28,7 +28,7 @@ def main(argv: list[str] | None = None) -> int:
     from . import build, models
     from .scheduler import BatchedDecodeLauncher
     artifact = models.load_model(args.model, quant=args.quant)
-    build.build(groups=(models.family_for({"architecture": artifact.config.architecture}).kernel_group,))
+    build.build(groups=models.family_for({"architecture": artifact.config.architecture}).kernel_groups)
     from .runtime import B200DecodeRuntime
     runtime = B200DecodeRuntime(artifact, dtype=args.dtype, max_seq_len=args.max_seq_len)
     prompts = [runtime.tokenizer.encode(text) for text in args.prompt] + [[int(t) for t in ids.split(",")] for ids in args.tokens]

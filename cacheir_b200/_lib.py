@@ -1,5 +1,5 @@
-"""ctypes binding of libcacheir_b200.so (the C ABI declared in include/cacheir_b200.h)
-and libcacheir_b200_hybrid.so (include/cacheir_b200_hybrid.h).
+"""ctypes binding of libcacheir_b200.so (the C ABI declared in include/cacheir_b200.h) and of the libraries of the
+ragged families: libcacheir_b200_ragged.so, _hybrid.so and _experts.so (headers of the same names).
 
 There is no fallback: if the shared library is missing the import of any
 compute entry point raises, telling the user to build it.
@@ -11,7 +11,7 @@ from ctypes import c_char_p, c_float, c_int, c_longlong, c_size_t, c_void_p
 from pathlib import Path
 
 LIB_PATH = Path(__file__).resolve().parent / "lib" / "libcacheir_b200.so"
-HYBRID_LIB_PATH = LIB_PATH.with_name("libcacheir_b200_hybrid.so")
+GROUP_PATHS = {name: LIB_PATH.with_name(f"libcacheir_b200_{name}.so") for name in ("ragged", "hybrid", "experts")}
 
 # name -> (restype, argtypes); mirrors include/cacheir_b200.h one to one
 SIGNATURES: dict[str, tuple[object, list[object]]] = {
@@ -105,7 +105,6 @@ SIGNATURES: dict[str, tuple[object, list[object]]] = {
 }
 
 
-
 class DenseArgs(ctypes.Structure):
     """cacheir_b200_dense_args"""
 
@@ -116,7 +115,8 @@ class DenseArgs(ctypes.Structure):
                 ("act_cols", c_int), ("next_mode", c_int), ("vocab", c_int), ("table_col", c_int),
                 ("gate", c_void_p), ("gate_stride", c_longlong), ("residual", c_void_p), ("norm_w", c_void_p), ("norm_b", c_void_p),
                 ("next_w", c_void_p), ("next_b", c_void_p), ("next_out", c_void_p), ("norm_alpha", c_float), ("next_alpha", c_float),
-                ("ids", c_void_p), ("table", c_void_p), ("table_stride", c_longlong)]
+                ("ids", c_void_p), ("table", c_void_p), ("table_stride", c_longlong),
+                ("bias", c_void_p), ("limit", c_float), ("tail_cols", c_int), ("tail", c_void_p), ("tail_stride", c_longlong)]
 
 
 class LatentArgs(ctypes.Structure):
@@ -137,90 +137,119 @@ class RecurrenceArgs(ctypes.Structure):
                 ("dtype", c_int)]
 
 
+class TiedArgs(ctypes.Structure):
+    """cacheir_b200_tied_args"""
+
+    _fields_ = [("positions", c_void_p), ("row_seg", c_void_p), ("cu_rows", c_void_p), ("page_table", c_void_p),
+                ("rows", c_int), ("segments", c_int), ("max_pages", c_int), ("page_size", c_int), ("num_slots", c_int),
+                ("heads", c_int), ("kv_heads", c_int), ("dim", c_int), ("rot_dims", c_int), ("window", c_int), ("keep_first", c_int),
+                ("scale", c_float), ("cap", c_float), ("pool", c_void_p), ("inv_rms", c_void_p), ("sink", c_void_p),
+                ("dtype", c_int), ("decode", c_int)]
+
+
 _NEXT = [c_int, c_void_p, c_void_p, c_float, c_void_p]      # next_mode next_w next_b next_alpha next_out
-# mirrors include/cacheir_b200_hybrid.h one to one
-HYBRID_SIGNATURES: dict[str, tuple[object, list[object]]] = {
-    "cacheir_b200_dense_supported": (c_int, [c_int, c_longlong, c_longlong, c_int, c_int]),
-    "cacheir_b200_dense_gemm": (c_int, [c_void_p, c_void_p]),
-    "cacheir_b200_dense_simple": (c_int, [c_void_p] * 3 + [c_int] * 7 + [c_longlong] * 3 + [c_int, c_int, c_void_p]),
-    "cacheir_b200_scaled_embedding": (c_int, [c_void_p] * 3 + [c_int, c_int, c_int, c_float] + _NEXT + [c_int, c_void_p]),
-    "cacheir_b200_dyt_rows": (c_int, [c_void_p] * 4 + [c_float, c_void_p, c_int, c_int, c_int, c_void_p]),
-    "cacheir_b200_residual_dyt": (c_int, [c_void_p] * 4 + [c_float, c_int, c_int] + _NEXT + [c_int, c_void_p]),
-    "cacheir_b200_residual_rms": (c_int, [c_void_p] * 3 + [c_float, c_int, c_int] + _NEXT + [c_int, c_void_p]),
-    "cacheir_b200_gated_rms": (c_int, [c_void_p, c_void_p, c_longlong, c_void_p, c_float, c_void_p, c_int, c_int, c_int, c_void_p]),
-    "cacheir_b200_geglu_pairs": (c_int, [c_void_p, c_void_p, c_int, c_int, c_int, c_void_p]),
-    "cacheir_b200_gelu_embed": (c_int, [c_void_p] * 3 + [c_longlong, c_int, c_void_p, c_int, c_int, c_int, c_int, c_void_p]),
-    "cacheir_b200_silu_cols": (c_int, [c_void_p, c_int, c_longlong, c_int, c_int, c_void_p]),
-    "cacheir_b200_latent_prepare": (
-        c_int, [c_void_p, c_void_p, c_longlong, c_void_p, c_float, c_void_p, c_longlong, c_void_p, c_longlong, c_int, c_void_p,
-                c_int, c_int, c_void_p]),
-    "cacheir_b200_latent_attention_simple": (
-        c_int, [c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_void_p]),
-    "cacheir_b200_latent_attention_supported": (c_int, [c_int] * 4),
-    "cacheir_b200_latent_attention_splits": (c_int, [c_int] * 5),
-    "cacheir_b200_latent_attention": (c_int, [c_void_p] * 4 + [c_int, c_void_p]),
-    "cacheir_b200_recurrence_simple": (c_int, [c_void_p, c_void_p]),
-    "cacheir_b200_recurrence_step": (c_int, [c_void_p, c_void_p]),
-    "cacheir_b200_recurrence_chunked_supported": (c_int, [c_int] * 3),
-    "cacheir_b200_recurrence_workspace_bytes": (c_size_t, [c_int] * 5),
-    "cacheir_b200_recurrence_chunked": (c_int, [c_void_p, c_void_p, c_size_t, c_void_p]),
-    "cacheir_b200_hybrid_device_status": (c_int, [c_int]),
+# group -> signatures; each mirrors include/cacheir_b200_<group>.h one to one
+GROUP_SIGNATURES: dict[str, dict[str, tuple[object, list[object]]]] = {
+    "ragged": {
+        "cacheir_b200_dense_supported": (c_int, [c_int, c_longlong, c_longlong, c_int, c_int]),
+        "cacheir_b200_dense_gemm": (c_int, [c_void_p, c_void_p]),
+        "cacheir_b200_dense_simple": (c_int, [c_void_p] * 3 + [c_int] * 7 + [c_longlong] * 3 + [c_void_p, c_int, c_int, c_void_p]),
+        "cacheir_b200_scaled_embedding": (c_int, [c_void_p] * 3 + [c_int, c_int, c_int, c_float] + _NEXT + [c_int, c_void_p]),
+        "cacheir_b200_dyt_rows": (c_int, [c_void_p] * 4 + [c_float, c_void_p, c_int, c_int, c_int, c_void_p]),
+        "cacheir_b200_rms_rows": (c_int, [c_void_p] * 3 + [c_float, c_void_p, c_int, c_int, c_int, c_void_p]),
+        "cacheir_b200_residual_dyt": (c_int, [c_void_p] * 4 + [c_float, c_int, c_int] + _NEXT + [c_int, c_void_p]),
+        "cacheir_b200_residual_rms": (c_int, [c_void_p] * 3 + [c_float, c_int, c_int] + _NEXT + [c_int, c_void_p]),
+        "cacheir_b200_gated_rms": (c_int, [c_void_p, c_void_p, c_longlong, c_void_p, c_float, c_void_p, c_int, c_int, c_int, c_void_p]),
+        "cacheir_b200_glu_pairs": (c_int, [c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_int, c_void_p]),
+        "cacheir_b200_gelu_embed": (c_int, [c_void_p] * 3 + [c_longlong, c_int, c_void_p, c_int, c_int, c_int, c_int, c_void_p]),
+        "cacheir_b200_silu_cols": (c_int, [c_void_p, c_int, c_longlong, c_int, c_int, c_void_p]),
+        "cacheir_b200_ragged_device_status": (c_int, [c_int]),
+    },
+    "hybrid": {
+        "cacheir_b200_latent_prepare": (
+            c_int, [c_void_p, c_void_p, c_longlong, c_void_p, c_float, c_void_p, c_longlong, c_void_p, c_longlong, c_int, c_void_p,
+                    c_int, c_int, c_void_p]),
+        "cacheir_b200_latent_attention_simple": (
+            c_int, [c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_void_p]),
+        "cacheir_b200_latent_attention_supported": (c_int, [c_int] * 4),
+        "cacheir_b200_latent_attention_splits": (c_int, [c_int] * 5),
+        "cacheir_b200_latent_attention": (c_int, [c_void_p] * 4 + [c_int, c_void_p]),
+        "cacheir_b200_recurrence_simple": (c_int, [c_void_p, c_void_p]),
+        "cacheir_b200_recurrence_step": (c_int, [c_void_p, c_void_p]),
+        "cacheir_b200_recurrence_chunked_supported": (c_int, [c_int] * 3),
+        "cacheir_b200_recurrence_workspace_bytes": (c_size_t, [c_int] * 5),
+        "cacheir_b200_recurrence_chunked": (c_int, [c_void_p, c_void_p, c_size_t, c_void_p]),
+        "cacheir_b200_hybrid_device_status": (c_int, [c_int]),
+    },
+    "experts": {
+        "cacheir_b200_tied_prepare": (
+            c_int, [c_void_p, c_void_p, c_longlong, c_void_p, c_longlong, c_float, c_void_p, c_int, c_void_p, c_void_p]),
+        "cacheir_b200_tied_attention_simple": (c_int, [c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_void_p]),
+        "cacheir_b200_tied_step_supported": (c_int, [c_int] * 6),
+        "cacheir_b200_tied_step_splits": (c_int, [c_int] * 7),
+        "cacheir_b200_tied_attention_step": (c_int, [c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_int, c_void_p]),
+        "cacheir_b200_route": (c_int, [c_void_p, c_longlong, c_void_p, c_int, c_int, c_int, c_float] + [c_void_p] * 7),
+        "cacheir_b200_grouped_gemm": (c_int, [c_void_p, c_void_p, c_void_p, c_int, c_void_p]),
+        "cacheir_b200_grouped_simple": (c_int, [c_void_p] * 5 + [c_int] * 4 + [c_longlong] * 3 + [c_int, c_void_p]),
+        "cacheir_b200_combine_residual_rms": (
+            c_int, [c_void_p] * 4 + [c_int, c_void_p, c_void_p, c_float, c_int, c_int, c_int, c_void_p, c_int, c_void_p]),
+        "cacheir_b200_experts_device_status": (c_int, [c_int]),
+    },
 }
-# entry points of glue.cu and misc.cu, which both libraries carry
+# entry points of glue.cu and misc.cu, which the core and the ragged library carry
 SHARED_NAMES = ("cacheir_b200_version", "cacheir_b200_error_string", "cacheir_b200_argmax_rows", "cacheir_b200_advance_positions")
 
 _LIB: ctypes.CDLL | None = None
-_HYBRID_LIB: ctypes.CDLL | None = None
+_GROUPS: dict[str, ctypes.CDLL] = {}
 
 
 class CacheIRB200Error(RuntimeError):
     """A C-ABI call returned a non-zero status."""
 
 
-def load() -> ctypes.CDLL:
-    """Load the library once and attach the prototypes. Raises if it is not built."""
-    global _LIB
-    if _LIB is not None:
-        return _LIB
-    if not LIB_PATH.exists():
-        raise CacheIRB200Error(
-            f"{LIB_PATH} is missing: build the CUDA library first (python -m cacheir_b200.build). "
-            "cacheir_b200 has no CPU or PyTorch fallback.")
-    lib = ctypes.CDLL(str(LIB_PATH))
-    for name, (restype, argtypes) in SIGNATURES.items():
+def _open(path: Path, table: dict[str, tuple[object, list[object]]], how: str) -> ctypes.CDLL:
+    if not path.exists():
+        raise CacheIRB200Error(f"{path} is missing: build the CUDA library first (python -m cacheir_b200.build{how}). "
+                               "cacheir_b200 has no CPU or PyTorch fallback.")
+    lib = ctypes.CDLL(str(path))
+    for name, (restype, argtypes) in table.items():
         fn = getattr(lib, name)  # AttributeError here means header and library disagree
         fn.restype = restype
         fn.argtypes = argtypes
-    _LIB = lib
     return lib
 
 
-def load_hybrid() -> ctypes.CDLL:
-    """The library of the hybrid families, loaded once. Raises if it is not built."""
-    global _HYBRID_LIB
-    if _HYBRID_LIB is not None:
-        return _HYBRID_LIB
-    if not HYBRID_LIB_PATH.exists():
-        raise CacheIRB200Error(
-            f"{HYBRID_LIB_PATH} is missing: build it first (python -m cacheir_b200.build --group hybrid). "
-            "cacheir_b200 has no CPU or PyTorch fallback.")
-    lib = ctypes.CDLL(str(HYBRID_LIB_PATH))
-    table = dict(HYBRID_SIGNATURES, **{name: SIGNATURES[name] for name in SHARED_NAMES})
-    for name, (restype, argtypes) in table.items():
-        fn = getattr(lib, name)
-        fn.restype = restype
-        fn.argtypes = argtypes
-    _HYBRID_LIB = lib
-    return lib
+def load() -> ctypes.CDLL:
+    """Load the core library once and attach the prototypes. Raises if it is not built."""
+    global _LIB
+    if _LIB is None:
+        _LIB = _open(LIB_PATH, SIGNATURES, "")
+    return _LIB
+
+
+def load_group(name: str) -> ctypes.CDLL:
+    """A library of the ragged families, loaded once. Raises if it is not built."""
+    if name not in _GROUPS:
+        table = dict(GROUP_SIGNATURES[name])
+        if name == "ragged":
+            table.update({shared: SIGNATURES[shared] for shared in SHARED_NAMES})
+        _GROUPS[name] = _open(GROUP_PATHS[name], table, f" --group {name}")
+    return _GROUPS[name]
 
 
 def load_shared() -> ctypes.CDLL:
     """A library that has the entry points of SHARED_NAMES: the one in use, else whichever is built."""
     if _LIB is not None:
         return _LIB
-    if _HYBRID_LIB is not None or (HYBRID_LIB_PATH.exists() and not LIB_PATH.exists()):
-        return load_hybrid()
+    if "ragged" in _GROUPS or (GROUP_PATHS["ragged"].exists() and not LIB_PATH.exists()):
+        return load_group("ragged")
     return load()
+
+
+def group_device_status(reset: bool = True) -> int:
+    """First bounded wait that gave up in any loaded library of the ragged families (0: none)."""
+    found = [int(getattr(lib, f"cacheir_b200_{name}_device_status")(int(reset))) for name, lib in _GROUPS.items()]
+    return next((status for status in found if status != 0), 0)
 
 
 def check(code: int, what: str) -> None:

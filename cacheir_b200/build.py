@@ -1,14 +1,15 @@
 """Build the CUDA libraries in-tree with nvcc for sm_100a.
 
-Usage: python -m cacheir_b200.build [--force] [--verbose] [--group core|hybrid]
+Usage: python -m cacheir_b200.build [--force] [--verbose] [--group NAME]
 
-Two plain C-ABI shared objects (no torch, no pybind), each a group of the .cu
-files under csrc/ compiled with -gencode arch=compute_100a,code=sm_100a and
-linked with the static CUDA runtime: `core` (libcacheir_b200.so, Llama-shaped
-models) and `hybrid` (libcacheir_b200_hybrid.so, latent attention + linear
-recurrences). A model family names the group it needs, so a fresh checkout
-compiles only that. Objects are rebuilt only when their source or a header is
-newer.
+Plain C-ABI shared objects (no torch, no pybind), each a group of the .cu files
+under csrc/ compiled with -gencode arch=compute_100a,code=sm_100a and linked
+with the static CUDA runtime: `core` (libcacheir_b200.so, Llama-shaped models),
+`ragged` (dense products and row operators of the families with ragged steps),
+`hybrid` (latent attention, linear recurrences) and `experts` (tied attention,
+mixtures of experts). A model family names the groups it needs, so a fresh
+checkout compiles only those. Objects are rebuilt only when their source or a
+header is newer.
 """
 from __future__ import annotations
 
@@ -25,10 +26,14 @@ CSRC = PKG_DIR / "csrc"
 INCLUDE = PKG_DIR.parent / "include"
 BUILD_DIR = PKG_DIR / "build"
 LIB_DIR = PKG_DIR / "lib"
-LIB_PATHS = {"core": LIB_DIR / "libcacheir_b200.so", "hybrid": LIB_DIR / "libcacheir_b200_hybrid.so"}
+SHARED = ("glue", "misc")            # in the core and the ragged library: argmax, position bookkeeping, error text
+GROUP_FILES = {
+    "ragged": ("dense_gemm", "hybrid_glue") + SHARED,
+    "hybrid": ("latent_attention", "linear_recurrence"),
+    "experts": ("tied_attention", "grouped_gemm", "expert_routing"),
+}
+LIB_PATHS = {"core": LIB_DIR / "libcacheir_b200.so", **{name: LIB_DIR / f"libcacheir_b200_{name}.so" for name in GROUP_FILES}}
 LIB_PATH = LIB_PATHS["core"]
-HYBRID_ONLY = ("dense_gemm", "hybrid_glue", "latent_attention", "linear_recurrence")
-SHARED = ("glue", "misc")            # in both libraries: argmax, position bookkeeping, error text
 
 NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a",
@@ -53,12 +58,13 @@ def _stale(target: Path, deps: list[Path]) -> bool:
 
 
 def group_sources(group: str) -> list[Path]:
-    if group == "hybrid":
-        return sorted(CSRC / f"{name}.cu" for name in HYBRID_ONLY + SHARED)
-    return sorted(src for src in CSRC.glob("*.cu") if src.stem not in HYBRID_ONLY)
+    if group in GROUP_FILES:
+        return sorted(CSRC / f"{name}.cu" for name in GROUP_FILES[group])
+    others = {name for names in GROUP_FILES.values() for name in names} - set(SHARED)
+    return sorted(src for src in CSRC.glob("*.cu") if src.stem not in others)
 
 
-def build(force: bool = False, verbose: bool = False, groups: tuple[str, ...] = ("core", "hybrid")) -> Path:
+def build(force: bool = False, verbose: bool = False, groups: tuple[str, ...] = tuple(LIB_PATHS)) -> Path:
     """Bring the libraries of `groups` up to date; returns the path of the first one."""
     nvcc = find_nvcc()
     BUILD_DIR.mkdir(parents=True, exist_ok=True)
@@ -101,5 +107,5 @@ if __name__ == "__main__":
     parser.add_argument("--verbose", action="store_true", help="print ptxas register/smem usage")
     parser.add_argument("--group", choices=sorted(LIB_PATHS), help="build one library only")
     args = parser.parse_args()
-    for name in (args.group,) if args.group else ("core", "hybrid"):
+    for name in (args.group,) if args.group else tuple(LIB_PATHS):
         print(build(force=args.force, verbose=args.verbose, groups=(name,)))

@@ -1,7 +1,7 @@
 // Shared by the kernels of the hybrid decoder families (latent attention, linear recurrences, Dynamic Tanh layers).
 #pragma once
 
-#include "cacheir_b200_hybrid.h"
+#include "cacheir_b200_ragged.h"
 #include "common.cuh"
 
 namespace cb200 {
@@ -12,6 +12,11 @@ __device__ __forceinline__ float silu_exact(float z) { return z / (1.f + expf(-z
 __device__ __forceinline__ float gelu_tanh(float z) {
   constexpr float kRoot2OverPi = 0.7978845608028654f;
   return 0.5f * z * (1.f + tanhf(kRoot2OverPi * fmaf(0.044715f * z * z, z, z)));
+}
+
+__device__ __forceinline__ float clamped_glu(float gate, float up, float limit) {
+  const float g = fminf(gate, limit), u = fminf(fmaxf(up, -limit), limit);
+  return g * sigmoid_exact(1.702f * g) * (u + 1.f);
 }
 
 __device__ __forceinline__ uint32_t smem_addr(const void* p) { return static_cast<uint32_t>(__cvta_generic_to_shared(p)); }
@@ -54,4 +59,52 @@ __device__ __forceinline__ void split_bf16(float v, float* hi, float* lo) {
   *lo = v - *hi;
 }
 
+// VEC neighbouring elements per access
+template <typename T, int VEC>
+__device__ __forceinline__ void load_vec(const T* p, float (&v)[VEC]) {
+  if constexpr (VEC == 4 && sizeof(T) == 2) {
+    const uint2 raw = *reinterpret_cast<const uint2*>(p);
+    v[0] = __uint_as_float(raw.x << 16); v[1] = __uint_as_float(raw.x & 0xffff0000u);
+    v[2] = __uint_as_float(raw.y << 16); v[3] = __uint_as_float(raw.y & 0xffff0000u);
+  } else if constexpr (VEC == 4) {
+    const float4 f = *reinterpret_cast<const float4*>(p);
+    v[0] = f.x; v[1] = f.y; v[2] = f.z; v[3] = f.w;
+  } else {
+    v[0] = Elem<T>::ld(p);
+  }
+}
+template <typename T, int VEC>
+__device__ __forceinline__ void store_vec(T* p, const float (&v)[VEC]) {
+  if constexpr (VEC == 4 && sizeof(T) == 2) {
+    uint2 raw;
+    raw.x = pack_bf16(v[0], v[1]);
+    raw.y = pack_bf16(v[2], v[3]);
+    *reinterpret_cast<uint2*>(p) = raw;
+  } else if constexpr (VEC == 4) {
+    *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+  } else {
+    Elem<T>::st(p, v[0]);
+  }
+}
+
+// reads a kernel's status word (a __device__ int), clearing it on request; synchronises
+template <typename Symbol>
+int device_status_word(Symbol& word, bool reset) {
+  int status = 0;
+  if (cudaMemcpyFromSymbol(&status, word, sizeof(int)) != cudaSuccess) return -1;
+  if (reset && status != 0) {
+    const int zero = 0;
+    cudaMemcpyToSymbol(word, &zero, sizeof(int));
+  }
+  return status;
+}
+
 }  // namespace cb200
+
+// runs a statement with T = the activation type
+#define CB200_HYBRID_DTYPE(dtype, ...)                                                  \
+  switch (dtype) {                                                                      \
+    case CACHEIR_B200_F32: { using T = float; __VA_ARGS__; break; }                     \
+    case CACHEIR_B200_BF16: { using T = __nv_bfloat16; __VA_ARGS__; break; }            \
+    default: return CACHEIR_B200_EUNSUPPORTED;                                          \
+  }

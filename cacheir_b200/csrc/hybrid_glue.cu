@@ -43,6 +43,31 @@ dyt_rows_kernel(const float* __restrict__ x, const int32_t* __restrict__ row_ind
     Elem<T>::st(out + row * width + c, fmaf(tanhf(alpha * x[src * width + c]), w[c], b[c]));
 }
 
+template <typename T, int VEC>
+__global__ void __launch_bounds__(512)
+rms_rows_kernel(const float* __restrict__ x, const int32_t* __restrict__ row_index, const float* __restrict__ w, float eps,
+                T* __restrict__ out, int width) {
+  __shared__ float scratch[32];
+  const size_t row = blockIdx.x;
+  const float* xr = x + (row_index ? static_cast<size_t>(max(row_index[row], 0)) : row) * width;
+  float ss = 0.f;
+  for (int c = threadIdx.x * VEC; c < width; c += 512 * VEC) {
+    float v[VEC];
+    load_vec<float, VEC>(xr + c, v);
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) ss = fmaf(v[i], v[i], ss);
+  }
+  const float inv = 1.f / sqrtf(block_sum_all(ss, scratch) / static_cast<float>(width) + eps);
+  for (int c = threadIdx.x * VEC; c < width; c += 512 * VEC) {
+    float v[VEC], wv[VEC];
+    load_vec<float, VEC>(xr + c, v);
+    load_vec<float, VEC>(w + c, wv);
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) v[i] = v[i] * inv * wv[i];
+    store_vec<T, VEC>(out + row * width + c, v);
+  }
+}
+
 template <typename T>
 __global__ void __launch_bounds__(256)
 residual_dyt_kernel(float* __restrict__ x, const T* __restrict__ y, const float* __restrict__ w, const float* __restrict__ b,
@@ -53,34 +78,6 @@ residual_dyt_kernel(float* __restrict__ x, const T* __restrict__ y, const float*
     const float s = x[i] + fmaf(tanhf(alpha * Elem<T>::ld(y + i)), w[c], b[c]);
     x[i] = s;
     leave_next<T>(nx, i, c, s);
-  }
-}
-
-// VEC neighbouring elements per access, PT accesses per thread kept in registers between the two passes
-template <typename T, int VEC>
-__device__ __forceinline__ void load_vec(const T* p, float (&v)[VEC]) {
-  if constexpr (VEC == 4 && sizeof(T) == 2) {
-    const uint2 raw = *reinterpret_cast<const uint2*>(p);
-    v[0] = __uint_as_float(raw.x << 16); v[1] = __uint_as_float(raw.x & 0xffff0000u);
-    v[2] = __uint_as_float(raw.y << 16); v[3] = __uint_as_float(raw.y & 0xffff0000u);
-  } else if constexpr (VEC == 4) {
-    const float4 f = *reinterpret_cast<const float4*>(p);
-    v[0] = f.x; v[1] = f.y; v[2] = f.z; v[3] = f.w;
-  } else {
-    v[0] = Elem<T>::ld(p);
-  }
-}
-template <typename T, int VEC>
-__device__ __forceinline__ void store_vec(T* p, const float (&v)[VEC]) {
-  if constexpr (VEC == 4 && sizeof(T) == 2) {
-    uint2 raw;
-    raw.x = pack_bf16(v[0], v[1]);
-    raw.y = pack_bf16(v[2], v[3]);
-    *reinterpret_cast<uint2*>(p) = raw;
-  } else if constexpr (VEC == 4) {
-    *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
-  } else {
-    Elem<T>::st(p, v[0]);
   }
 }
 
@@ -149,11 +146,13 @@ gated_rms_kernel(const T* __restrict__ o, const T* __restrict__ gate, long long 
 
 template <typename T>
 __global__ void __launch_bounds__(256)
-geglu_pairs_kernel(const T* __restrict__ y, T* __restrict__ out, int ff) {
+glu_pairs_kernel(const T* __restrict__ y, T* __restrict__ out, int ff, int epilogue, float limit) {
   const size_t row = blockIdx.x;
   for (int c = blockIdx.y * 256 + threadIdx.x; c < ff; c += gridDim.y * 256) {
     const T* p = y + row * 2 * ff + 2 * c;
-    Elem<T>::st(out + row * ff + c, gelu_tanh(Elem<T>::ld(p)) * Elem<T>::ld(p + 1));
+    const float a = Elem<T>::ld(p), u = Elem<T>::ld(p + 1);
+    Elem<T>::st(out + row * ff + c, epilogue == CACHEIR_B200_DENSE_GEGLU ? gelu_tanh(a) * u
+                                    : epilogue == CACHEIR_B200_DENSE_SWIGLU ? silu_exact(a) * u : clamped_glu(a, u, limit));
   }
 }
 
@@ -179,7 +178,7 @@ constexpr int kTile = 64, kTileK = 16;
 template <typename T, typename TY>
 __global__ void __launch_bounds__(256)
 dense_simple_kernel(const T* __restrict__ x, const T* __restrict__ w, TY* __restrict__ y, int rows, int N, int K, int w_batch_rows,
-                    int x_batch_cols, int y_batch_cols, long long ws, long long xs, long long ys) {
+                    int x_batch_cols, int y_batch_cols, long long ws, long long xs, long long ys, const float* __restrict__ bias) {
   __shared__ float sx[kTileK][kTile + 4], sw[kTileK][kTile + 4];
   const int z = blockIdx.z;
   x += static_cast<long long>(z) * x_batch_cols;
@@ -212,7 +211,7 @@ dense_simple_kernel(const T* __restrict__ x, const T* __restrict__ w, TY* __rest
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const int t = t0 + ty * 4 + i, n = n0 + tx * 4 + j;
-      if (t < rows && n < N) Elem<TY>::st(y + t * ys + n, acc[i][j]);
+      if (t < rows && n < N) Elem<TY>::st(y + t * ys + n, acc[i][j] + (bias ? bias[n] : 0.f));
     }
 }
 
@@ -233,13 +232,6 @@ bool next_ok(int mode, const float* w, const float* b, const void* out) {
 
 using namespace cb200;
 
-#define CB200_HYBRID_DTYPE(dtype, ...)                                                  \
-  switch (dtype) {                                                                      \
-    case CACHEIR_B200_F32: { using T = float; __VA_ARGS__; break; }                     \
-    case CACHEIR_B200_BF16: { using T = __nv_bfloat16; __VA_ARGS__; break; }            \
-    default: return CACHEIR_B200_EUNSUPPORTED;                                          \
-  }
-
 extern "C" int cacheir_b200_scaled_embedding(const void* table, const int64_t* ids, float* residual, int rows, int width, int vocab,
                                              float scale, int next_mode, const float* next_w, const float* next_b, float next_alpha,
                                              void* next_out, int dtype, void* stream) {
@@ -257,6 +249,18 @@ extern "C" int cacheir_b200_dyt_rows(const float* residual, const int32_t* row_i
   if (!residual || !w || !b || !out) return CACHEIR_B200_EINVAL;
   CB200_HYBRID_DTYPE(dtype, (dyt_rows_kernel<T><<<row_grid(rows, width), 256, 0, as_stream(stream)>>>(
                                 residual, row_index, w, b, alpha, static_cast<T*>(out), width)));
+  return launch_status();
+}
+
+extern "C" int cacheir_b200_rms_rows(const float* residual, const int32_t* row_index, const float* w, float eps, void* out, int rows,
+                                     int width, int dtype, void* stream) {
+  if (rows <= 0 || width <= 0) return 0;
+  if (!residual || !w || !out) return CACHEIR_B200_EINVAL;
+  const bool vec = width % 4 == 0 && aligned_to(residual, 16) && aligned_to(w, 16) && aligned_to(out, 16);
+  CB200_HYBRID_DTYPE(dtype, {
+    if (vec) rms_rows_kernel<T, 4><<<rows, 512, 0, as_stream(stream)>>>(residual, row_index, w, eps, static_cast<T*>(out), width);
+    else rms_rows_kernel<T, 1><<<rows, 512, 0, as_stream(stream)>>>(residual, row_index, w, eps, static_cast<T*>(out), width);
+  });
   return launch_status();
 }
 
@@ -301,11 +305,12 @@ extern "C" int cacheir_b200_gated_rms(const void* o, const void* gate, long long
   return launch_status();
 }
 
-extern "C" int cacheir_b200_geglu_pairs(const void* y, void* out, int rows, int ff, int dtype, void* stream) {
+extern "C" int cacheir_b200_glu_pairs(const void* y, void* out, int rows, int ff, int epilogue, float limit, int dtype, void* stream) {
   if (rows <= 0 || ff <= 0) return 0;
-  if (!y || !out) return CACHEIR_B200_EINVAL;
-  CB200_HYBRID_DTYPE(dtype, (geglu_pairs_kernel<T><<<row_grid(rows, ff), 256, 0, as_stream(stream)>>>(
-                                static_cast<const T*>(y), static_cast<T*>(out), ff)));
+  if (!y || !out || (epilogue != CACHEIR_B200_DENSE_GEGLU && epilogue != CACHEIR_B200_DENSE_SWIGLU && epilogue != CACHEIR_B200_DENSE_CLAMPED_GLU))
+    return CACHEIR_B200_EINVAL;
+  CB200_HYBRID_DTYPE(dtype, (glu_pairs_kernel<T><<<row_grid(rows, ff), 256, 0, as_stream(stream)>>>(
+                                static_cast<const T*>(y), static_cast<T*>(out), ff, epilogue, limit)));
   return launch_status();
 }
 
@@ -328,30 +333,19 @@ extern "C" int cacheir_b200_silu_cols(void* y, int rows, long long stride, int c
 
 extern "C" int cacheir_b200_dense_simple(const void* x, const void* w, void* y, int rows, int N, int K, int batch, int w_batch_rows,
                                          int x_batch_cols, int y_batch_cols, long long w_stride, long long x_stride,
-                                         long long y_stride, int dtype, int y_dtype, void* stream) {
+                                         long long y_stride, const float* bias, int dtype, int y_dtype, void* stream) {
   if (rows <= 0 || N <= 0) return 0;
-  if (K <= 0 || !x || !w || !y || batch < 1) return CACHEIR_B200_EINVAL;
+  if (K <= 0 || !x || !w || !y || batch < 1 || (batch > 1 && bias)) return CACHEIR_B200_EINVAL;
   const dim3 grid((N + kTile - 1) / kTile, (rows + kTile - 1) / kTile, batch);
   if (grid.y > 65535 || grid.z > 65535) return CACHEIR_B200_ELIMIT;
   cudaStream_t st = as_stream(stream);
 #define CB200_SIMPLE(T, TY)                                                                                              \
   dense_simple_kernel<T, TY><<<grid, 256, 0, st>>>(static_cast<const T*>(x), static_cast<const T*>(w), static_cast<TY*>(y), rows, N, \
-                                                   K, w_batch_rows, x_batch_cols, y_batch_cols, w_stride, x_stride, y_stride)
+                                                   K, w_batch_rows, x_batch_cols, y_batch_cols, w_stride, x_stride, y_stride, bias)
   if (dtype == CACHEIR_B200_F32 && y_dtype == CACHEIR_B200_F32) CB200_SIMPLE(float, float);
   else if (dtype == CACHEIR_B200_BF16 && y_dtype == CACHEIR_B200_F32) CB200_SIMPLE(__nv_bfloat16, float);
   else if (dtype == CACHEIR_B200_BF16 && y_dtype == CACHEIR_B200_BF16) CB200_SIMPLE(__nv_bfloat16, __nv_bfloat16);
   else return CACHEIR_B200_EUNSUPPORTED;
 #undef CB200_SIMPLE
   return launch_status();
-}
-
-namespace cb200 {
-int dense_gemm_device_status(bool reset);
-int latent_attention_device_status(bool reset);
-}
-
-extern "C" int cacheir_b200_hybrid_device_status(int reset) {
-  const int gemm = dense_gemm_device_status(reset != 0);
-  const int attn = latent_attention_device_status(reset != 0);
-  return gemm != 0 ? gemm : attn;
 }

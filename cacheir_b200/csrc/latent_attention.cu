@@ -8,6 +8,7 @@
 //           ring as TMA boxes of 64 columns and serve as keys and, read the other way, as values. Softmax in float32
 //           with the sink as the initial maximum and denominator. A decode batch too small for the SMs splits the
 //           window over the CTAs of a cluster, which combine their parts through distributed shared memory.
+#include "cacheir_b200_hybrid.h"
 #include "hybrid_common.cuh"
 #include "ragged.cuh"
 #include "tc_ptx.cuh"
@@ -725,23 +726,12 @@ int launch_fast(FastParams p, const void* q, dim3 grid, cudaStream_t st) {
   return launch_status();
 }
 
-bool latent_args_ok(
-const cacheir_b200_latent_args& a) {
+bool latent_args_ok(const cacheir_b200_latent_args& a) {
   return a.positions && a.row_seg && a.page_table && a.pool && a.segments > 0 && a.max_pages > 0 && a.page_size > 0 && a.num_slots > 0 &&
          a.heads > 0 && a.dim > 0 && a.rot_dim >= 0 && a.vdim > 0 && a.kv_rank > 0 && a.window > 0 && a.heads <= 65535;
 }
 
 }  // namespace
-
-int latent_attention_device_status(bool reset) {
-  int status = 0;
-  if (cudaMemcpyFromSymbol(&status, g_latent_status, sizeof(int)) != cudaSuccess) return -1;
-  if (reset && status != 0) {
-    const int zero = 0;
-    cudaMemcpyToSymbol(g_latent_status, &zero, sizeof(int));
-  }
-  return status;
-}
 
 }  // namespace cb200
 
@@ -833,3 +823,5 @@ extern "C" int cacheir_b200_latent_attention(const cacheir_b200_latent_args* arg
   const dim3 grid(items, groups, splits);
   return rows == 64 ? launch_fast<64>(p, q, grid, as_stream(stream)) : launch_fast<32>(p, q, grid, as_stream(stream));
 }
+
+extern "C" int cacheir_b200_hybrid_device_status(int reset) { return device_status_word(g_latent_status, reset != 0); }

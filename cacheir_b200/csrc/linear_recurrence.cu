@@ -8,6 +8,7 @@
 //          decayed scores, the decayed values) goes in as a sum of two bf16 numbers. Sequences are cut into 256-token
 //          pieces that run in parallel: a first pass finds every piece's own contribution, a scan turns these into the
 //          pieces' initial states, and the main pass starts from them.
+#include "cacheir_b200_hybrid.h"
 #include "hybrid_common.cuh"
 #include "ragged.cuh"
 

@@ -1,0 +1,155 @@
+"""Torch-tensor wrappers over include/cacheir_b200_experts.h: tied attention and mixtures of experts. Same rules as
+`hybrid_ops`."""
+from __future__ import annotations
+
+import ctypes
+from dataclasses import dataclass
+
+import torch
+
+from . import _lib
+from ._lib import DenseArgs, TiedArgs, check
+from .hybrid_ops import DENSE_CLAMPED_GLU, DENSE_PLAIN, DENSE_SWIGLU, NEXT_COPY, NEXT_NONE, Next, Rows, _f32
+from .ops import _ptr, _require_cuda, _stream, dtype_code
+
+
+# ---- tied attention --------------------------------------------------------------------------------------------------
+def query_width(dim: int, rot_dims: int) -> int:
+    """Columns of a prepared query: a cached row without the whole 64-column boxes that would meet zeros."""
+    return dim + rot_dims - rot_dims // 64 * 64
+
+
+def tied_args(rows: Rows, pool: torch.Tensor, inv_rms: torch.Tensor, *, heads: int, kv_heads: int, dim: int, rot_dims: int, window: int,
+              keep_first: int, scale: float, softcap: float | None, sink: torch.Tensor | None) -> TiedArgs:
+    """pool [slots, kv_heads, page, dim + rot_dims], inv_rms [slots, kv_heads, page] float32."""
+    _require_cuda(pool, inv_rms, sink)
+    if pool.dim() != 4 or int(pool.shape[1]) != kv_heads or int(pool.shape[3]) != dim + rot_dims or not pool.is_contiguous():
+        raise ValueError("the pool must be a contiguous [slots, kv_heads, page, dim + rot_dims] tensor")
+    _f32(inv_rms, *([] if sink is None else [sink]))
+    if inv_rms.shape != pool.shape[:3] or (sink is not None and sink.numel() != heads):
+        raise ValueError("inv_rms has one entry per cached row, sink one per head")
+    a = TiedArgs()
+    a.positions, a.row_seg, a.cu_rows = rows.positions.data_ptr(), rows.row_seg.data_ptr(), rows.cu_rows.data_ptr()
+    a.page_table, a.rows, a.segments = rows.page_table.data_ptr(), rows.rows, rows.segments
+    a.max_pages, a.page_size, a.num_slots = int(rows.page_table.shape[1]), int(pool.shape[2]), int(pool.shape[0])
+    a.heads, a.kv_heads, a.dim, a.rot_dims, a.window, a.keep_first = heads, kv_heads, dim, rot_dims, window, keep_first
+    a.scale, a.cap = float(scale), 0.0 if softcap is None else float(softcap)
+    a.pool, a.inv_rms, a.sink = pool.data_ptr(), inv_rms.data_ptr(), _ptr(sink)
+    a.dtype, a.decode = dtype_code(pool.dtype), int(rows.decode)
+    return a
+
+
+def tied_prepare(a: TiedArgs, q: torch.Tensor, k: torch.Tensor, q_out: torch.Tensor, *, eps: float, table: torch.Tensor | None) -> None:
+    """Cache rows of `k` [T, kv_heads*dim]; prepared queries of `q` [T, heads*dim] in `q_out`."""
+    _require_cuda(q, k, q_out, table)
+    if q.stride(1) != 1 or k.stride(1) != 1 or not q_out.is_contiguous() or int(q_out.shape[1]) != a.heads * query_width(a.dim, a.rot_dims):
+        raise ValueError("tied_prepare expects dense rows and a contiguous [T, heads * query_width] output")
+    check(_lib.load_group("experts").cacheir_b200_tied_prepare(
+        ctypes.byref(a), q.data_ptr(), q.stride(0), k.data_ptr(), k.stride(0), float(eps), _ptr(table),
+        (1 << 30) if table is None else int(table.shape[0]), q_out.data_ptr(), _stream()), "tied_prepare")
+
+
+def _attend(a: TiedArgs, q: torch.Tensor, gate: torch.Tensor | None, out: torch.Tensor) -> tuple:
+    _require_cuda(q, gate, out)
+    if not q.is_contiguous() or not out.is_contiguous() or int(out.shape[1]) != a.heads * a.dim:
+        raise ValueError("tied attention expects contiguous q and [T, heads*dim] out")
+    if gate is not None and (gate.stride(1) != 1 or int(gate.shape[1]) != a.heads * a.dim):
+        raise ValueError("the gate has one column per output column")
+    return (ctypes.byref(a), q.data_ptr(), _ptr(gate), 0 if gate is None else gate.stride(0), out.data_ptr())
+
+
+def tied_attention_simple(a: TiedArgs, q: torch.Tensor, gate: torch.Tensor | None, out: torch.Tensor) -> torch.Tensor:
+    check(_lib.load_group("experts").cacheir_b200_tied_attention_simple(*_attend(a, q, gate, out), _stream()), "tied_attention_simple")
+    return out
+
+
+def tied_step_supported(heads: int, kv_heads: int, dim: int, rot_dims: int, page_size: int, dtype: torch.dtype) -> bool:
+    return bool(_lib.load_group("experts").cacheir_b200_tied_step_supported(heads, kv_heads, dim, rot_dims, page_size, dtype_code(dtype)))
+
+
+def tied_step_splits(rows: int, heads: int, kv_heads: int, window: int, keep_first: int, max_pages: int, page_size: int) -> int:
+    return int(_lib.load_group("experts").cacheir_b200_tied_step_splits(rows, heads, kv_heads, window, keep_first, max_pages, page_size))
+
+
+def tied_attention_step(a: TiedArgs, q: torch.Tensor, gate: torch.Tensor | None, out: torch.Tensor, *, splits: int = 0) -> torch.Tensor:
+    check(_lib.load_group("experts").cacheir_b200_tied_attention_step(*_attend(a, q, gate, out), int(splits), _stream()), "tied_attention_step")
+    return out
+
+
+# ---- mixtures of experts -----------------------------------------------------------------------------------------------
+@dataclass
+class Routing:
+    """Which rows go where: places in expert order (see the header)."""
+
+    experts: int
+    top: int
+    counters: torch.Tensor       # [experts + 1] zeros
+    cu: torch.Tensor             # [experts + 1]
+    token_of: torch.Tensor       # [rows * top]
+    place_of: torch.Tensor       # [rows, top]
+    chosen: torch.Tensor         # [rows, top]
+    weight: torch.Tensor         # [rows, top] float32
+
+    @property
+    def places(self) -> int:
+        return int(self.token_of.numel())
+
+
+def route(logits: torch.Tensor, row_seg: torch.Tensor, routing: Routing, scale: float) -> None:
+    _require_cuda(logits, row_seg, routing.counters)
+    rows = int(logits.shape[0])
+    if logits.dtype != torch.float32 or logits.stride(1) != 1 or tuple(routing.place_of.shape) != (rows, routing.top):
+        raise ValueError("route takes float32 logits with dense rows and a routing of their row count")
+    check(_lib.load_group("experts").cacheir_b200_route(
+        logits.data_ptr(), logits.stride(0), row_seg.data_ptr(), rows, routing.experts, routing.top, float(scale), routing.counters.data_ptr(),
+        routing.cu.data_ptr(), routing.token_of.data_ptr(), routing.place_of.data_ptr(), routing.weight.data_ptr(),
+        routing.chosen.data_ptr(), _stream()), "route")
+
+
+def grouped_supported(k: int, x_stride: int, dtype: torch.dtype) -> bool:
+    return dtype == torch.bfloat16 and k % 8 == 0 and x_stride % 8 == 0
+
+
+def grouped_gemm(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, routing: Routing, *, gather: bool, epilogue: int = DENSE_PLAIN,
+                 limit: float = 0.0) -> torch.Tensor:
+    """out[place] = f(x[row] W_e^T), w [experts*N, K]; row = the place's token when `gather`, else the place."""
+    _require_cuda(x, w, out)
+    n = int(w.shape[0]) // routing.experts
+    cols = n // 2 if epilogue in (DENSE_SWIGLU, DENSE_CLAMPED_GLU) else n
+    if x.dtype != torch.bfloat16 or w.dtype != torch.bfloat16 or x.stride(1) != 1 or w.stride(1) != 1 or out.dtype != torch.bfloat16:
+        raise ValueError("grouped_gemm takes bf16 operands with dense rows")
+    if int(out.shape[0]) != routing.places or int(out.shape[1]) < cols or out.stride(1) != 1 or (not gather and int(x.shape[0]) < routing.places):
+        raise ValueError("out must have a row per place")
+    a = DenseArgs()
+    a.x, a.w, a.y, a.T, a.N, a.K, a.batch, a.w_batch_rows = x.data_ptr(), w.data_ptr(), out.data_ptr(), routing.places, n, int(w.shape[1]), routing.experts, n
+    a.epilogue, a.w_stride, a.x_stride, a.y_stride, a.limit = epilogue, w.stride(0), x.stride(0), out.stride(0), float(limit)
+    check(_lib.load_group("experts").cacheir_b200_grouped_gemm(
+        ctypes.byref(a), routing.cu.data_ptr(), routing.token_of.data_ptr() if gather else None, int(x.shape[0]), _stream()), "grouped_gemm")
+    return out
+
+
+def grouped_simple(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, routing: Routing, *, gather: bool) -> torch.Tensor:
+    """The plain grouped product in float32 arithmetic, any extents."""
+    _require_cuda(x, w, out)
+    n = int(w.shape[0]) // routing.experts
+    if x.dtype != w.dtype or out.dtype != x.dtype or x.stride(1) != 1 or w.stride(1) != 1 or out.stride(1) != 1 or int(out.shape[0]) != routing.places:
+        raise ValueError("grouped_simple takes operands of one type with dense rows and an out row per place")
+    check(_lib.load_group("experts").cacheir_b200_grouped_simple(
+        x.data_ptr(), w.data_ptr(), out.data_ptr(), routing.cu.data_ptr(), routing.token_of.data_ptr() if gather else None, routing.places,
+        routing.experts, n, int(w.shape[1]), w.stride(0), x.stride(0), out.stride(0), dtype_code(x.dtype), _stream()), "grouped_simple")
+    return out
+
+
+def combine_residual_rms(residual: torch.Tensor, y: torch.Tensor, routing: Routing, shared: torch.Tensor | None, weight: torch.Tensor,
+                         eps: float, nx: Next | None = None) -> None:
+    """residual += rms_norm(sum of the chosen experts' rows by weight + shared) * weight"""
+    _require_cuda(residual, y, shared, weight)
+    _f32(residual, weight)
+    if not y.is_contiguous() or y.shape[1] != residual.shape[1] or (shared is not None and (shared.shape != residual.shape or not shared.is_contiguous())):
+        raise ValueError("y and shared have the residual's width and dense rows")
+    if nx is not None and (nx.norm is not None or nx.out.shape != residual.shape or not nx.out.is_contiguous()):
+        raise ValueError("the combine leaves a copy of the residual or nothing")
+    check(_lib.load_group("experts").cacheir_b200_combine_residual_rms(
+        residual.data_ptr(), y.data_ptr(), routing.place_of.data_ptr(), routing.weight.data_ptr(), routing.top, _ptr(shared), weight.data_ptr(),
+        float(eps), int(residual.shape[0]), int(residual.shape[1]), NEXT_NONE if nx is None else NEXT_COPY,
+        None if nx is None else nx.out.data_ptr(), dtype_code(y.dtype), _stream()), "combine_residual_rms")

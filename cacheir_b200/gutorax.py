@@ -43,7 +43,7 @@ class LayerConfig:
     ff: int | None           # dense feed-forward width, None: no feed-forward
 
 
-def _positive(value: Any, what: str) -> int:
+def positive_int(value: Any, what: str) -> int:
     n = int(value)
     if n <= 0 or n != value:
         raise ValueError(f"{what} must be a positive integer, got {value!r}")
@@ -53,18 +53,18 @@ def _positive(value: Any, what: str) -> int:
 def _mixer(kind: str, m: dict[str, Any], index: int) -> LatentMixer | LightningMixer:
     where = f"layer {index} mixer"
     if kind == "lightning":
-        heads = _positive(m["heads"], f"{where} heads")
+        heads = positive_int(m["heads"], f"{where} heads")
         decay = tuple(float(v) for v in m["decay"])
         if len(decay) != heads:
             raise ValueError(f"{where}: {len(decay)} decays for {heads} heads")
-        return LightningMixer(heads, _positive(m["dim"], f"{where} dim"), _positive(m["vdim"], f"{where} vdim"), decay)
+        return LightningMixer(heads, positive_int(m["dim"], f"{where} dim"), positive_int(m["vdim"], f"{where} vdim"), decay)
     if kind == "latent_attention":
         rot = m["rot"]
         mixer = LatentMixer(
-            heads=_positive(m["heads"], f"{where} heads"), dim=_positive(m["dim"], f"{where} dim"),
-            rot_dim=_positive(m["rot_dim"], f"{where} rot_dim"), vdim=_positive(m["vdim"], f"{where} vdim"),
-            kv_rank=_positive(m["kv_rank"], f"{where} kv_rank"), scale=float(m["scale"]),
-            window=_positive(m["mask"]["size"], f"{where} mask.size"), rot_dims=_positive(rot["dims"], f"{where} rot.dims"),
+            heads=positive_int(m["heads"], f"{where} heads"), dim=positive_int(m["dim"], f"{where} dim"),
+            rot_dim=positive_int(m["rot_dim"], f"{where} rot_dim"), vdim=positive_int(m["vdim"], f"{where} vdim"),
+            kv_rank=positive_int(m["kv_rank"], f"{where} kv_rank"), scale=float(m["scale"]),
+            window=positive_int(m["mask"]["size"], f"{where} mask.size"), rot_dims=positive_int(rot["dims"], f"{where} rot.dims"),
             rot_base=float(rot["base"]), kv_from=None if m.get("kv_from") is None else int(m["kv_from"]))
         if mixer.rot_dims % 2 or mixer.rot_dims > mixer.rot_dim:
             raise ValueError(f"{where}: rot.dims must be even and at most rot_dim")
@@ -86,7 +86,6 @@ class GutoraxConfig:
     layers: list[LayerConfig] = field(default_factory=list)
     max_position_embeddings: int = 8192
     dtype: str = "bfloat16"
-    kernel_group = "hybrid"
     ragged = True                 # steps carry portions of any length (see ragged.RaggedPlan)
 
     @classmethod
@@ -105,11 +104,11 @@ class GutoraxConfig:
                 same = ("kv_rank", "rot_dim", "rot_dims", "rot_base")
                 if any(getattr(owner, k) != getattr(mixer, k) for k in same):
                     raise ValueError(f"layer {i}: latent size and rotation differ from those of layer {j}, whose cache it reads")
-            layers.append(LayerConfig(mixer, None if mlp is None else _positive(mlp["ff"], f"layer {i} mlp.ff")))
+            layers.append(LayerConfig(mixer, None if mlp is None else positive_int(mlp["ff"], f"layer {i} mlp.ff")))
         side = data.get("token_side")
-        return cls(raw=dict(data), hidden_size=_positive(data["width"], "width"), vocab_size=_positive(data["vocab"], "vocab"),
+        return cls(raw=dict(data), hidden_size=positive_int(data["width"], "width"), vocab_size=positive_int(data["vocab"], "vocab"),
                    embedding_scale=float((data.get("embedding") or {}).get("scale", 1.0)), norm_eps=float(data["norm"]["eps"]),
-                   side_dim=None if side is None else _positive(side["dim"], "token_side.dim"), layers=layers,
+                   side_dim=None if side is None else positive_int(side["dim"], "token_side.dim"), layers=layers,
                    max_position_embeddings=int(data.get("max_position_embeddings", 8192)))
 
     def to_dict(self) -> dict[str, Any]:

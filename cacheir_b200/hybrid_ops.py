@@ -1,4 +1,4 @@
-"""Torch-tensor wrappers over the C ABI of the hybrid families (include/cacheir_b200_hybrid.h).
+"""Torch-tensor wrappers over the C ABI of the ragged families (include/cacheir_b200_ragged.h, cacheir_b200_hybrid.h).
 
 Same rules as `ops`: validate, pass device pointers on the current stream, raise on a non-zero status. The residual
 stream and every norm parameter are float32; activations are float32 or bfloat16.
@@ -15,7 +15,9 @@ from ._lib import DenseArgs, LatentArgs, RecurrenceArgs, check
 from .ops import _ptr, _require_cuda, _stream, dtype_code
 
 NEXT_NONE, NEXT_COPY, NEXT_DYT = 0, 1, 2
-DENSE_PLAIN, DENSE_F32, DENSE_SILU, DENSE_GEGLU, DENSE_GATED, DENSE_RESIDUAL, DENSE_GELU_EMBED = range(7)
+(DENSE_PLAIN, DENSE_F32, DENSE_SILU, DENSE_GEGLU, DENSE_GATED, DENSE_RESIDUAL, DENSE_GELU_EMBED, DENSE_SWIGLU,
+ DENSE_CLAMPED_GLU) = range(9)
+GLU_EPILOGUES = {"gelu_tanh": DENSE_GEGLU, "silu": DENSE_SWIGLU, "clamped": DENSE_CLAMPED_GLU}
 RECURRENCE_POWERS = 65
 
 
@@ -76,15 +78,17 @@ def _f32(*tensors: torch.Tensor) -> None:
 
 def dense_supported(k: int, w_stride: int, x_stride: int, *, dtype: torch.dtype, batch: int = 1, x_batch_cols: int = 0) -> bool:
     """Can the tensor-core GEMM take this product?"""
-    return dtype == torch.bfloat16 and bool(_lib.load_hybrid().cacheir_b200_dense_supported(k, w_stride, x_stride, batch, x_batch_cols))
+    return dtype == torch.bfloat16 and bool(_lib.load_group("ragged").cacheir_b200_dense_supported(k, w_stride, x_stride, batch, x_batch_cols))
 
 
 def dense_gemm(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor | None = None, *, epilogue: int = DENSE_PLAIN,
                batch: int = 1, x_batch_cols: int = 0, y_batch_cols: int | None = None, act_cols: int = 0, gate: torch.Tensor | None = None,
                residual: torch.Tensor | None = None, norm: DynamicTanh | None = None, nx: Next | None = None,
-               ids: torch.Tensor | None = None, table: torch.Tensor | None = None, table_col: int = 0) -> None:
-    """Tensor-core Y = f(X W^T). x [T, >=K] and w [N, K] bf16 with dense rows. `batch` > 1: w [batch*N, K], entry z reads
-    x columns from z*x_batch_cols and writes output columns from z*y_batch_cols (default z*N)."""
+               ids: torch.Tensor | None = None, table: torch.Tensor | None = None, table_col: int = 0,
+               bias: torch.Tensor | None = None, limit: float = 0.0, tail: torch.Tensor | None = None) -> None:
+    """Tensor-core Y = f(X W^T + bias). x [T, >=K] and w [N, K] bf16 with dense rows. `batch` > 1: w [batch*N, K], entry z
+    reads x columns from z*x_batch_cols and writes output columns from z*y_batch_cols (default z*N). `tail` (paired
+    epilogues): the last columns of the product go there as float32."""
     _require_cuda(x, w, out, gate, residual, ids, table)
     if x.dtype != torch.bfloat16 or w.dtype != torch.bfloat16 or x.stride(1) != 1 or w.stride(1) != 1:
         raise ValueError("dense_gemm takes bf16 x and w with dense rows")
@@ -102,11 +106,22 @@ def dense_gemm(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor | None = None
         if nx is not None and (tuple(nx.out.shape) != (a.T, a.N) or nx.out.dtype != torch.bfloat16 or not nx.out.is_contiguous()):
             raise ValueError("the next operator's input must be a contiguous bf16 [T, N] tensor")
     else:
-        cols = a.y_batch_cols * (batch - 1) + a.N if epilogue != DENSE_GEGLU else a.N // 2
+        paired = epilogue in GLU_EPILOGUES.values()
+        if tail is not None:
+            if not paired or tail.dtype != torch.float32 or tail.stride(1) != 1 or int(tail.shape[0]) != a.T:
+                raise ValueError("tail is a float32 [T, columns] tensor of a paired epilogue")
+            a.tail, a.tail_cols, a.tail_stride = tail.data_ptr(), int(tail.shape[1]), tail.stride(0)
+        cols = (a.N - a.tail_cols) // 2 if paired else a.y_batch_cols * (batch - 1) + a.N
         want = torch.float32 if epilogue == DENSE_F32 else torch.bfloat16
         if out is None or out.dtype != want or int(out.shape[0]) != a.T or int(out.shape[1]) < cols or out.stride(1) != 1:
             raise ValueError("out must be [T, N] of the epilogue's type with dense rows")
         a.y, a.y_stride, a.act_cols = out.data_ptr(), out.stride(0), act_cols
+    a.limit = float(limit)
+    if bias is not None:
+        _f32(bias)
+        if batch != 1 or bias.numel() != a.N:
+            raise ValueError("bias has one entry per output column")
+        a.bias = bias.data_ptr()
     if epilogue == DENSE_GATED:
         if gate is None or gate.dtype != torch.bfloat16 or gate.stride(1) != 1 or int(gate.shape[1]) < a.N * batch:
             raise ValueError("the gated epilogue needs a bf16 gate per output column")
@@ -115,18 +130,19 @@ def dense_gemm(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor | None = None
         if ids is None or table is None or ids.dtype != torch.int64 or int(table.shape[1]) < table_col + a.N:
             raise ValueError("the embedding epilogue needs int64 ids and a table with a part for every output column")
         a.ids, a.table, a.table_stride, a.table_col, a.vocab = ids.data_ptr(), table.data_ptr(), table.stride(0), table_col, int(table.shape[0])
-    check(_lib.load_hybrid().cacheir_b200_dense_gemm(ctypes.byref(a), _stream()), "dense_gemm")
+    check(_lib.load_group("ragged").cacheir_b200_dense_gemm(ctypes.byref(a), _stream()), "dense_gemm")
 
 
-def dense_simple(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, *, batch: int = 1, x_batch_cols: int = 0) -> torch.Tensor:
+def dense_simple(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, *, batch: int = 1, x_batch_cols: int = 0,
+                 bias: torch.Tensor | None = None) -> torch.Tensor:
     """The plain product in float32 arithmetic on the CUDA cores, any extents (see dense_gemm for `batch`)."""
-    _require_cuda(x, w, out)
+    _require_cuda(x, w, out, bias)
     n, k = int(w.shape[0]) // batch, int(w.shape[1])
     if x.dtype != w.dtype or x.stride(1) != 1 or w.stride(1) != 1 or out.stride(1) != 1 or int(out.shape[1]) < n * batch:
         raise ValueError("dense_simple takes x, w of one type with dense rows and out [T, N]")
-    check(_lib.load_hybrid().cacheir_b200_dense_simple(
+    check(_lib.load_group("ragged").cacheir_b200_dense_simple(
         x.data_ptr(), w.data_ptr(), out.data_ptr(), int(x.shape[0]), n, k, batch, n, x_batch_cols, n, w.stride(0), x.stride(0),
-        out.stride(0), dtype_code(x.dtype), dtype_code(out.dtype), _stream()), "dense_simple")
+        out.stride(0), _ptr(bias), dtype_code(x.dtype), dtype_code(out.dtype), _stream()), "dense_simple")
     return out
 
 
@@ -135,7 +151,7 @@ def scaled_embedding(table: torch.Tensor, ids: torch.Tensor, residual: torch.Ten
     _f32(residual)
     if ids.dtype != torch.int64 or not table.is_contiguous() or residual.shape[1] != table.shape[1]:
         raise ValueError("scaled_embedding expects int64 ids and a contiguous [vocab, width] table")
-    check(_lib.load_hybrid().cacheir_b200_scaled_embedding(
+    check(_lib.load_group("ragged").cacheir_b200_scaled_embedding(
         table.data_ptr(), ids.data_ptr(), residual.data_ptr(), int(residual.shape[0]), int(table.shape[1]), int(table.shape[0]),
         float(scale), *_next(nx), dtype_code(table.dtype), _stream()), "scaled_embedding")
 
@@ -144,9 +160,19 @@ def dyt_rows(residual: torch.Tensor, norm: DynamicTanh, out: torch.Tensor, row_i
     """out[j] = dynamic tanh of residual row row_index[j] (row j without an index)."""
     _require_cuda(residual, out, row_index)
     _f32(residual, norm.weight, norm.bias)
-    check(_lib.load_hybrid().cacheir_b200_dyt_rows(
+    check(_lib.load_group("ragged").cacheir_b200_dyt_rows(
         residual.data_ptr(), _ptr(row_index), norm.weight.data_ptr(), norm.bias.data_ptr(), float(norm.alpha), out.data_ptr(),
         int(out.shape[0]), int(out.shape[1]), dtype_code(out.dtype), _stream()), "dyt_rows")
+    return out
+
+
+def rms_rows(residual: torch.Tensor, weight: torch.Tensor, eps: float, out: torch.Tensor, row_index: torch.Tensor | None = None) -> torch.Tensor:
+    """out[j] = rms_norm(residual row row_index[j]) * weight (row j without an index)."""
+    _require_cuda(residual, weight, out, row_index)
+    _f32(residual, weight)
+    check(_lib.load_group("ragged").cacheir_b200_rms_rows(
+        residual.data_ptr(), _ptr(row_index), weight.data_ptr(), float(eps), out.data_ptr(), int(out.shape[0]), int(out.shape[1]),
+        dtype_code(out.dtype), _stream()), "rms_rows")
     return out
 
 
@@ -155,7 +181,7 @@ def residual_dyt(residual: torch.Tensor, y: torch.Tensor, norm: DynamicTanh, nx:
     _f32(residual, norm.weight, norm.bias)
     if y.shape != residual.shape or not y.is_contiguous():
         raise ValueError("y must be a contiguous tensor of the residual's shape")
-    check(_lib.load_hybrid().cacheir_b200_residual_dyt(
+    check(_lib.load_group("ragged").cacheir_b200_residual_dyt(
         residual.data_ptr(), y.data_ptr(), norm.weight.data_ptr(), norm.bias.data_ptr(), float(norm.alpha), int(y.shape[0]),
         int(y.shape[1]), *_next(nx), dtype_code(y.dtype), _stream()), "residual_dyt")
 
@@ -166,7 +192,7 @@ def residual_rms(residual: torch.Tensor, y: torch.Tensor, weight: torch.Tensor, 
     _f32(residual, weight)
     if y.shape != residual.shape or not y.is_contiguous():
         raise ValueError("y must be a contiguous tensor of the residual's shape")
-    check(_lib.load_hybrid().cacheir_b200_residual_rms(
+    check(_lib.load_group("ragged").cacheir_b200_residual_rms(
         residual.data_ptr(), y.data_ptr(), weight.data_ptr(), float(eps), int(y.shape[0]), int(y.shape[1]), *_next(nx),
         dtype_code(y.dtype), _stream()), "residual_rms")
 
@@ -177,19 +203,19 @@ def gated_rms(o: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, eps: fl
     _f32(weight)
     if not o.is_contiguous() or not out.is_contiguous() or gate.stride(1) != 1 or gate.shape != o.shape or out.shape != o.shape:
         raise ValueError("gated_rms expects contiguous o and out and a gate of their shape")
-    check(_lib.load_hybrid().cacheir_b200_gated_rms(
+    check(_lib.load_group("ragged").cacheir_b200_gated_rms(
         o.data_ptr(), gate.data_ptr(), gate.stride(0), weight.data_ptr(), float(eps), out.data_ptr(), int(o.shape[0]), int(o.shape[1]),
         dtype_code(o.dtype), _stream()), "gated_rms")
     return out
 
 
-def geglu_pairs(y: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
-    """y [T, 2*ff] with columns alternating gate, up."""
+def glu_pairs(y: torch.Tensor, out: torch.Tensor, epilogue: int = DENSE_GEGLU, limit: float = 0.0) -> torch.Tensor:
+    """y [T, 2*ff] with columns alternating gate, up; out as the paired epilogue leaves it."""
     _require_cuda(y, out)
     if not y.is_contiguous() or not out.is_contiguous() or y.shape[1] != 2 * out.shape[1]:
-        raise ValueError("geglu_pairs expects contiguous [T, 2*ff] and [T, ff]")
-    check(_lib.load_hybrid().cacheir_b200_geglu_pairs(y.data_ptr(), out.data_ptr(), int(out.shape[0]), int(out.shape[1]),
-                                                      dtype_code(y.dtype), _stream()), "geglu_pairs")
+        raise ValueError("glu_pairs expects contiguous [T, 2*ff] and [T, ff]")
+    check(_lib.load_group("ragged").cacheir_b200_glu_pairs(y.data_ptr(), out.data_ptr(), int(out.shape[0]), int(out.shape[1]), int(epilogue),
+                                                           float(limit), dtype_code(y.dtype), _stream()), "glu_pairs")
     return out
 
 
@@ -197,7 +223,7 @@ def gelu_embed(g: torch.Tensor, ids: torch.Tensor, table: torch.Tensor, table_co
     _require_cuda(g, ids, table, out)
     if not g.is_contiguous() or not out.is_contiguous() or table.stride(1) != 1 or int(table.shape[1]) < table_col + int(g.shape[1]):
         raise ValueError("gelu_embed expects contiguous g and out and a table with a part for every column")
-    check(_lib.load_hybrid().cacheir_b200_gelu_embed(
+    check(_lib.load_group("ragged").cacheir_b200_gelu_embed(
         g.data_ptr(), ids.data_ptr(), table.data_ptr(), table.stride(0), int(table_col), out.data_ptr(), int(g.shape[0]),
         int(g.shape[1]), int(table.shape[0]), dtype_code(g.dtype), _stream()), "gelu_embed")
     return out
@@ -205,7 +231,7 @@ def gelu_embed(g: torch.Tensor, ids: torch.Tensor, table: torch.Tensor, table_co
 
 def silu_cols(y: torch.Tensor, cols: int) -> torch.Tensor:
     _require_cuda(y)
-    check(_lib.load_hybrid().cacheir_b200_silu_cols(y.data_ptr(), int(y.shape[0]), y.stride(0), int(cols), dtype_code(y.dtype), _stream()),
+    check(_lib.load_group("ragged").cacheir_b200_silu_cols(y.data_ptr(), int(y.shape[0]), y.stride(0), int(cols), dtype_code(y.dtype), _stream()),
           "silu_cols")
     return y
 
@@ -230,7 +256,7 @@ def latent_prepare(a: LatentArgs, q: torch.Tensor, q_rot: torch.Tensor, *, q_rot
     """Append one cache row per token (unless `down` is None) and turn the queries' rotated part into `q_rot`, a tensor
     whose first element is row 0, head 0's first rotated entry."""
     _require_cuda(q, q_rot, table, down, norm_weight)
-    check(_lib.load_hybrid().cacheir_b200_latent_prepare(
+    check(_lib.load_group("hybrid").cacheir_b200_latent_prepare(
         ctypes.byref(a), _ptr(down), 0 if down is None else down.stride(0), _ptr(norm_weight), float(eps), q.data_ptr(), q.stride(0),
         q_rot.data_ptr(), q_rot.stride(0), int(q_rot_head_stride), table.data_ptr(), int(table.shape[0]), int(rot_dims), _stream()),
         "latent_prepare")
@@ -240,18 +266,18 @@ def latent_attention_simple(a: LatentArgs, q: torch.Tensor, uk: torch.Tensor, uv
                             out: torch.Tensor) -> torch.Tensor:
     _require_cuda(q, uk, uv, sink, gate, out)
     _f32(sink)
-    check(_lib.load_hybrid().cacheir_b200_latent_attention_simple(
+    check(_lib.load_group("hybrid").cacheir_b200_latent_attention_simple(
         ctypes.byref(a), q.data_ptr(), q.stride(0), uk.data_ptr(), uv.data_ptr(), sink.data_ptr(), gate.data_ptr(), gate.stride(0),
         out.data_ptr(), _stream()), "latent_attention_simple")
     return out
 
 
 def latent_attention_supported(kv_rank: int, rot_dim: int, page_size: int, dtype: torch.dtype) -> bool:
-    return bool(_lib.load_hybrid().cacheir_b200_latent_attention_supported(kv_rank, rot_dim, page_size, dtype_code(dtype)))
+    return bool(_lib.load_group("hybrid").cacheir_b200_latent_attention_supported(kv_rank, rot_dim, page_size, dtype_code(dtype)))
 
 
 def latent_attention_splits(rows: int, heads: int, window: int, max_pages: int, page_size: int) -> int:
-    return int(_lib.load_hybrid().cacheir_b200_latent_attention_splits(rows, heads, window, max_pages, page_size))
+    return int(_lib.load_group("hybrid").cacheir_b200_latent_attention_splits(rows, heads, window, max_pages, page_size))
 
 
 def latent_attention(a: LatentArgs, q: torch.Tensor, sink: torch.Tensor, out: torch.Tensor, *, splits: int = 1) -> torch.Tensor:
@@ -260,7 +286,7 @@ def latent_attention(a: LatentArgs, q: torch.Tensor, sink: torch.Tensor, out: to
     _f32(sink)
     if not q.is_contiguous() or not out.is_contiguous():
         raise ValueError("latent_attention expects contiguous q and out")
-    check(_lib.load_hybrid().cacheir_b200_latent_attention(
+    check(_lib.load_group("hybrid").cacheir_b200_latent_attention(
         ctypes.byref(a), q.data_ptr(), sink.data_ptr(), out.data_ptr(), int(splits), _stream()), "latent_attention")
     return out
 
@@ -291,26 +317,26 @@ def recurrence_args(rows: Rows, q: torch.Tensor, k: torch.Tensor, v: torch.Tenso
 
 
 def recurrence_simple(a: RecurrenceArgs) -> None:
-    check(_lib.load_hybrid().cacheir_b200_recurrence_simple(ctypes.byref(a), _stream()), "recurrence_simple")
+    check(_lib.load_group("hybrid").cacheir_b200_recurrence_simple(ctypes.byref(a), _stream()), "recurrence_simple")
 
 
 def recurrence_step(a: RecurrenceArgs) -> None:
-    check(_lib.load_hybrid().cacheir_b200_recurrence_step(ctypes.byref(a), _stream()), "recurrence_step")
+    check(_lib.load_group("hybrid").cacheir_b200_recurrence_step(ctypes.byref(a), _stream()), "recurrence_step")
 
 
 def recurrence_chunked_supported(dim: int, vdim: int, dtype: torch.dtype) -> bool:
-    return bool(_lib.load_hybrid().cacheir_b200_recurrence_chunked_supported(dim, vdim, dtype_code(dtype)))
+    return bool(_lib.load_group("hybrid").cacheir_b200_recurrence_chunked_supported(dim, vdim, dtype_code(dtype)))
 
 
 def recurrence_workspace_bytes(rows: int, segments: int, heads: int, dim: int, vdim: int) -> int:
-    return int(_lib.load_hybrid().cacheir_b200_recurrence_workspace_bytes(rows, segments, heads, dim, vdim))
+    return int(_lib.load_group("hybrid").cacheir_b200_recurrence_workspace_bytes(rows, segments, heads, dim, vdim))
 
 
 def recurrence_chunked(a: RecurrenceArgs, workspace: torch.Tensor | None) -> None:
-    check(_lib.load_hybrid().cacheir_b200_recurrence_chunked(
+    check(_lib.load_group("hybrid").cacheir_b200_recurrence_chunked(
         ctypes.byref(a), _ptr(workspace), 0 if workspace is None else workspace.numel() * workspace.element_size(), _stream()),
         "recurrence_chunked")
 
 
 def device_status(reset: bool = True) -> int:
-    return int(_lib.load_hybrid().cacheir_b200_hybrid_device_status(int(reset)))
+    return _lib.group_device_status(reset)

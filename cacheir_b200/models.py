@@ -6,7 +6,7 @@ from dataclasses import dataclass
 from pathlib import Path
 from typing import Any, Callable
 
-from . import gutorax
+from . import gutorax, topunex
 from .artifact import CompileArtifact, ModelConfig, build_decoder_artifact
 
 
@@ -15,7 +15,7 @@ class ModelFamily:
     name: str
     config_from_dict: Callable[[dict[str, Any]], Any]
     build_artifact: Callable[..., CompileArtifact]
-    kernel_group: str = "core"          # library group the family needs (cacheir_b200.build)
+    kernel_groups: tuple[str, ...] = ("core",)          # libraries the family needs (cacheir_b200.build)
 
 
 _FAMILIES: dict[str, ModelFamily] = {}
@@ -48,4 +48,5 @@ def load_model(path: str | Path, *, quant: str | None = None) -> CompileArtifact
     return family.build_artifact(family.config_from_dict(data), model_path=str(folder), quant=quant)
 
 
-register_family(gutorax.ARCHITECTURE, ModelFamily("gutorax", gutorax.GutoraxConfig.from_dict, gutorax.build_gutorax_artifact, "hybrid"))
+register_family(gutorax.ARCHITECTURE, ModelFamily("gutorax", gutorax.GutoraxConfig.from_dict, gutorax.build_gutorax_artifact, ("ragged", "hybrid")))
+register_family(topunex.ARCHITECTURE, ModelFamily("topunex", topunex.TopunexConfig.from_dict, topunex.build_topunex_artifact, ("ragged", "experts")))

@@ -1,7 +1,7 @@
 """Ragged steps: portions of prompts beside single decoded tokens as one pass through a lowered graph.
 
 `RaggedPlan` is the plan class of families whose layers need to know which rows belong to one sequence (linear
-recurrences, windowed attention over tiles of neighbouring tokens). It keeps `_DecodePlan`'s contract (static buffers,
+recurrences, windowed attention over tiles of neighbouring tokens) or which rows are real (mixtures of experts). It keeps `_DecodePlan`'s contract (static buffers,
 a flat launch list, CUDA-graph replay from the second step) and adds the segment arrays. A decode plan has one row per
 sequence and advances on the device; a portion plan has room for `rows` rows of `segments` sequences and takes its
 metadata in one copy per step. Residual stream float32; in bfloat16 runs each sublayer boundary (norm, residual add,
@@ -14,6 +14,7 @@ from typing import Any, Callable
 import numpy as np
 import torch
 
+from . import expert_ops as X
 from . import hybrid_ops as H
 from . import ops
 
@@ -28,9 +29,27 @@ def bucket(n: int) -> int:
     return (n + 1023) // 1024 * 1024
 
 
-def rotate_half_table(positions: int, dims: int, base: float) -> np.ndarray:
-    """float32 [positions, dims/2, 2] (cos, sin) of p * base^(-2i/dims), evaluated in double precision."""
+# ops that take the residual stream itself, as a copy in the activation type
+READS_RESIDUAL = {"token_side_gate", "concat_matmul", "fused_glu", "expert_router"}
+
+
+def rotary_frequencies(dims: int, base: float, scaling: tuple[float, float, float, float] | None = None) -> np.ndarray:
+    """base^(-2i/dims) in double precision. `scaling` = (factor, low, high, original): wavelengths above original/low are
+    stretched by factor, those below original/high kept, and the blend between is linear in original/wavelength."""
     freq = float(base) ** (-2.0 * np.arange(dims // 2, dtype=np.float64) / dims)
+    if scaling is None:
+        return freq
+    factor, low, high, original = scaling
+    turns = original * freq / (2.0 * np.pi)              # original / wavelength
+    with np.errstate(divide="ignore", invalid="ignore"):
+        keep = (turns - low) / (high - low)
+    blended = (1.0 - keep) * freq / factor + keep * freq
+    return np.where(turns > high, freq, np.where(turns < low, freq / factor, blended))
+
+
+def rotate_half_table(positions: int, dims: int, base: float, scaling: tuple[float, float, float, float] | None = None) -> np.ndarray:
+    """float32 [positions, dims/2, 2] (cos, sin) of position times frequency, evaluated in double precision."""
+    freq = rotary_frequencies(dims, base, scaling)
     angle = np.arange(positions, dtype=np.float64)[:, None] * freq[None, :]
     return np.stack([np.cos(angle), np.sin(angle)], axis=-1).astype(np.float32)
 
@@ -141,7 +160,7 @@ def make_plan_class(base: type) -> type:
             if nxt.op == "dynamic_tanh" and nxt.attrs.get("rows") != "logits" and nxt.inputs[0] == self._nodes[idx].outputs[0]:
                 out = self._scratch("normed", width)
                 return H.Next(out, self._dyt(nxt.inputs[1:4])), nxt.outputs[0]
-            if nxt.op == "token_side_gate" and nxt.inputs[0] == self._nodes[idx].outputs[0]:
+            if nxt.op in READS_RESIDUAL and nxt.inputs[0] == self._nodes[idx].outputs[0]:
                 return H.Next(self._scratch("copied", width)), None
             return None, None
 
@@ -177,13 +196,17 @@ def make_plan_class(base: type) -> type:
             self.logits = logits
             self.feedback_tail = lambda: ops.argmax_rows(logits, self.ids)
 
-        def _dense(self, x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, **kwargs: Any) -> None:
+        def _dense(self, x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, bias: torch.Tensor | None = None) -> None:
             """Plain product into `out` (float32 for logits): tensor cores where they take it, else CUDA cores."""
             if H.dense_supported(int(w.shape[1]), w.stride(0), x.stride(0), dtype=x.dtype):
                 epilogue = H.DENSE_F32 if out.dtype == torch.float32 else H.DENSE_PLAIN
-                self._emit(lambda: H.dense_gemm(x, w, out, epilogue=epilogue), "b200.dense_gemm")
+                self._emit(lambda: H.dense_gemm(x, w, out, epilogue=epilogue, bias=bias), "b200.dense_gemm")
             else:
-                self._emit(lambda: H.dense_simple(x, w, out), "b200.dense_simple")
+                self._emit(lambda: H.dense_simple(x, w, out, bias=bias), "b200.dense_simple")
+
+        def _input(self, name: str) -> torch.Tensor:
+            """A product's input: an activation, or the residual's copy."""
+            return self._env.get("copy:" + name, self._env[name])
 
         def _lower_scaled_token_embedding(self, idx: int, node: Any) -> None:
             table = self.engine.weights.get_checked(node.inputs[1])
@@ -202,8 +225,9 @@ def make_plan_class(base: type) -> type:
             self._env[node.outputs[0]] = out
 
         def _lower_concat_matmul(self, idx: int, node: Any) -> None:
-            eng, x = self.engine, self._env[node.inputs[0]]
+            eng, x = self.engine, self._input(node.inputs[0])
             names = tuple(node.inputs[1:])
+            bias = eng.concat_bias(tuple(node.attrs["bias"]), names) if node.attrs.get("bias") else None
             sizes = [int(eng.graph.weights[n].shape[0]) for n in names]
             w = eng.concat_weight(names)
             total = int(w.shape[0])
@@ -211,9 +235,10 @@ def make_plan_class(base: type) -> type:
             act = sum(sizes[: int(node.attrs.get("activated", 0))])
             if H.dense_supported(int(w.shape[1]), w.stride(0), x.stride(0), dtype=x.dtype):
                 epilogue = H.DENSE_SILU if act else H.DENSE_PLAIN
-                self._emit(lambda: H.dense_gemm(x, w, out, epilogue=epilogue, act_cols=act), "b200.dense_gemm" + (".silu" if act else ""))
+                self._emit(lambda: H.dense_gemm(x, w, out, epilogue=epilogue, act_cols=act, bias=bias),
+                           "b200.dense_gemm" + (".silu" if act else ""))
             else:
-                self._emit(lambda: H.dense_simple(x, w, out), "b200.dense_simple")
+                self._emit(lambda: H.dense_simple(x, w, out, bias=bias), "b200.dense_simple")
                 if act:
                     self._emit(lambda: H.silu_cols(out, act), "b200.silu_cols")
             col = 0
@@ -296,8 +321,9 @@ def make_plan_class(base: type) -> type:
             if nxt is None:
                 out = self._scratch("logits", int(w.shape[0]), torch.float32, rows=self.logit_rows)
             else:
-                out = self._scratch("sublayer", int(w.shape[0]))
-            self._dense(x, w, out)
+                out = self._scratch("sublayer", int(w.shape[0]))      # (a shared expert's lives until the combine)
+            bias = node.attrs.get("bias")
+            self._dense(x, w, out, None if bias is None else eng.weights.get_f32(bias))
             self._env[node.outputs[0]] = out
 
         def _lower_residual_dynamic_tanh(self, idx: int, node: Any) -> None:
@@ -305,17 +331,29 @@ def make_plan_class(base: type) -> type:
             self._finish_residual(idx, lambda nx: self._emit(lambda: H.residual_dyt(res, y, norm, nx), "b200.residual_dyt"))
 
         def _lower_fused_geglu(self, idx: int, node: Any) -> None:
-            eng, x = self.engine, self._env[node.inputs[0]]
-            w = eng.paired_weight(tuple(node.inputs[1:3]))
-            ff = int(w.shape[0]) // 2
-            out = self._scratch("gated", ff)
+            self._env[node.outputs[0]] = self._glu(self._env[node.inputs[0]], node, "gelu_tanh")
+
+        def _lower_fused_glu(self, idx: int, node: Any) -> None:
+            self._env[node.outputs[0]] = self._glu(self._input(node.inputs[0]), node, node.attrs["activation"])
+
+        def _glu(self, x: torch.Tensor, node: Any, activation: str, tail_weight: str | None = None,
+                 tail: torch.Tensor | None = None) -> torch.Tensor:
+            """activation(gate, up) of one product; `tail_weight`'s rows behind the pairs leave plain float32 columns."""
+            eng = self.engine
+            names = tuple(node.inputs[1:3])
+            w = eng.paired_weight(names, tail_weight)
+            ff = int(eng.graph.weights[names[0]].shape[0])
+            bias = eng.paired_bias(tuple(node.attrs["bias"])) if node.attrs.get("bias") else None
+            kind, limit = H.GLU_EPILOGUES[activation], float(node.attrs.get("limit", 0.0))
+            out = self._scratch("gated", (ff + 7) // 8 * 8)[:, :ff]
             if H.dense_supported(int(w.shape[1]), w.stride(0), x.stride(0), dtype=x.dtype):
-                self._emit(lambda: H.dense_gemm(x, w, out, epilogue=H.DENSE_GEGLU), "b200.dense_gemm.geglu")
+                label = {"gelu_tanh": ".geglu", "silu": ".swiglu", "clamped": ".clamped_glu"}[activation]
+                self._emit(lambda: H.dense_gemm(x, w, out, epilogue=kind, bias=bias, limit=limit, tail=tail), "b200.dense_gemm" + label)
             else:
-                both = self._scratch("gate_up", 2 * ff)
-                self._emit(lambda: H.dense_simple(x, w, both), "b200.dense_simple")
-                self._emit(lambda: H.geglu_pairs(both, out), "b200.geglu_pairs")
-            self._env[node.outputs[0]] = out
+                both, out = self._scratch("gate_up", 2 * ff), self._scratch("gated", ff)
+                self._emit(lambda: H.dense_simple(x, w, both, bias=bias), "b200.dense_simple")
+                self._emit(lambda: H.glu_pairs(both, out, kind, limit), "b200.glu_pairs")
+            return out
 
         def _lower_token_side_gate(self, idx: int, node: Any) -> None:
             eng = self.engine
@@ -336,5 +374,81 @@ def make_plan_class(base: type) -> type:
             y, res = self._env[node.inputs[1]], self._residual
             w, eps = self.engine.weights.get_f32(node.inputs[2]), float(node.attrs["eps"])
             self._finish_residual(idx, lambda nx: self._emit(lambda: H.residual_rms(res, y, w, eps, nx), "b200.residual_rms"))
+
+        def _lower_rms_norm(self, idx: int, node: Any) -> None:
+            w, eps = self.engine.weights.get_f32(node.inputs[1]), float(node.attrs["eps"])
+            logits = node.attrs.get("rows") == "logits"
+            out = self._scratch("final" if logits else "normed", int(w.numel()), rows=self.logit_rows if logits else None)
+            index = self.logit_index if logits else None
+            self._emit(lambda: H.rms_rows(self._residual, w, eps, out, index), "b200.rms_rows")
+            self._env[node.outputs[0]] = out
+
+        def _lower_tied_attention(self, idx: int, node: Any) -> None:
+            eng, at = self.engine, node.attrs
+            q, k, gate = (self._env[n] for n in node.inputs[:3])
+            heads, kv_heads, dim, rot = (int(at[n]) for n in ("heads", "kv_heads", "dim", "rot_dims"))
+            pool = eng.allocator.pool_for_layer(int(at["layer"]))
+            scaling = at.get("rot_scaling")
+            table = eng.rotate_half_table(rot, float(at["rot_base"]), None if scaling is None else tuple(map(float, scaling))) if rot else None
+            args = X.tied_args(self.rows, pool["rows"], pool["inv_rms"], heads=heads, kv_heads=kv_heads, dim=dim, rot_dims=rot,
+                               window=int(at["window"]), keep_first=int(at["keep_first"]), scale=float(at["scale"]), softcap=at.get("softcap"),
+                               sink=eng.weights.get_f32(node.inputs[3]))
+            prepared = self._scratch("prepared_q", heads * X.query_width(dim, rot))
+            out = self._scratch("mixed", heads * dim)
+            self._emit(lambda: X.tied_prepare(args, q, k, prepared, eps=float(at["eps"]), table=table), "b200.tied_prepare")
+            if self.decode and X.tied_step_supported(heads, kv_heads, dim, rot, eng.page_size, eng.dtype):
+                splits = X.tied_step_splits(self.batch, heads, kv_heads, int(at["window"]), int(at["keep_first"]), self.width, eng.page_size)
+                self._emit(lambda: X.tied_attention_step(args, prepared, gate, out, splits=splits), "b200.tied_attention_step")
+            else:
+                self._emit(lambda: X.tied_attention_simple(args, prepared, gate, out), "b200.tied_attention_simple")
+            self._env[node.outputs[0]] = out
+
+        def _lower_expert_router(self, idx: int, node: Any) -> None:
+            eng, x = self.engine, self._input(node.inputs[0])
+            spec = eng.graph.weights[node.inputs[1]]
+            experts, width, top, scale = int(spec.shape[0]), int(spec.shape[1]), int(node.attrs["top"]), float(node.attrs["scale"])
+            logits = self._scratch("router_logits", experts, torch.float32)
+            nxt = self._nodes[idx + 1]
+            if (nxt.op == "fused_glu" and nxt.inputs[0] == node.inputs[0] and not nxt.attrs.get("bias")
+                    and H.dense_supported(width, width, x.stride(0), dtype=x.dtype)):
+                # a shared expert reads the same rows: the router's columns ride behind its gate and up
+                self._env[nxt.outputs[0]] = self._glu(x, nxt, nxt.attrs["activation"], node.inputs[1], logits)
+                self._skip.add(idx + 1)
+            else:
+                self._dense(x, eng.weights.get_checked(node.inputs[1]), logits)
+            i32 = torch.int32
+            routing = X.Routing(experts, top, counters=self._scratch("route_counters", experts + 1, i32, rows=1).view(-1),
+                                cu=self._scratch("route_cu", experts + 1, i32, rows=1).view(-1), token_of=self._scratch("route_token", top, i32).view(-1),
+                                place_of=self._scratch("route_place", top, i32), chosen=self._scratch("route_chosen", top, i32),
+                                weight=self._scratch("route_weight", top, torch.float32))
+            self._emit(lambda: X.route(logits, self.rows.row_seg, routing, scale), "b200.route")
+            self._env[node.outputs[0]] = routing
+
+        def _lower_expert_mixture(self, idx: int, node: Any) -> None:
+            eng, x, routing = self.engine, self._input(node.inputs[0]), self._env[node.inputs[1]]
+            n = int(node.attrs["experts"])
+            gates, ups, downs = (tuple(node.inputs[2 + i * n:2 + (i + 1) * n]) for i in range(3))
+            w_in, w_out = eng.expert_pairs(gates, ups), eng.concat_weight(downs)
+            ff, width = int(w_in.shape[0]) // (2 * n), int(w_out.shape[0]) // n
+            kind, limit = H.GLU_EPILOGUES[node.attrs["activation"]], float(node.attrs["limit"])
+            places = routing.places
+            out = self._scratch("expert_out", width, rows=places)
+            if X.grouped_supported(int(w_in.shape[1]), x.stride(0), eng.dtype) and X.grouped_supported(ff, ff, eng.dtype):
+                hidden = self._scratch("expert_hidden", ff, rows=places)
+                self._emit(lambda: X.grouped_gemm(x, w_in, hidden, routing, gather=True, epilogue=kind, limit=limit), "b200.grouped_gemm.clamped_glu")
+                self._emit(lambda: X.grouped_gemm(hidden, w_out, out, routing, gather=False), "b200.grouped_gemm")
+            else:
+                both, hidden = self._scratch("expert_gate_up", 2 * ff, rows=places), self._scratch("expert_hidden", ff, rows=places)
+                self._emit(lambda: X.grouped_simple(x, w_in, both, routing, gather=True), "b200.grouped_simple")
+                self._emit(lambda: H.glu_pairs(both, hidden, kind, limit), "b200.glu_pairs")
+                self._emit(lambda: X.grouped_simple(hidden, w_out, out, routing, gather=False), "b200.grouped_simple")
+            self._env[node.outputs[0]] = out
+
+        def _lower_combine_residual_rms_norm(self, idx: int, node: Any) -> None:
+            y, routing, res = self._env[node.inputs[1]], self._env[node.inputs[2]], self._residual
+            w, eps = self.engine.weights.get_f32(node.inputs[3]), float(node.attrs["eps"])
+            shared = self._env[node.inputs[4]] if len(node.inputs) > 4 else None
+            self._finish_residual(idx, lambda nx: self._emit(lambda: X.combine_residual_rms(res, y, routing, shared, w, eps, nx),
+                                                             "b200.combine_residual_rms"))
 
     return RaggedPlan

@@ -52,7 +52,7 @@ KERNEL_FOR_OP: dict[str, tuple[str, tuple[str, ...]]] = {
     "add": ("triton.vector_add", ("cacheir_b200_add", "cacheir_b200_qgemv")),
 }
 
-# graph ops of the hybrid families -> C entry points of libcacheir_b200_hybrid.so (tensor-core forms first)
+# graph ops of the ragged families -> C entry points of their libraries (tensor-core forms first)
 HYBRID_KERNELS_FOR_OP: dict[str, tuple[str, ...]] = {
     "scaled_token_embedding": ("cacheir_b200_scaled_embedding",),
     "dynamic_tanh": ("cacheir_b200_dyt_rows",),
@@ -63,9 +63,15 @@ HYBRID_KERNELS_FOR_OP: dict[str, tuple[str, ...]] = {
     "linear_recurrence": ("cacheir_b200_recurrence_step", "cacheir_b200_recurrence_chunked", "cacheir_b200_recurrence_simple"),
     "gated_rms_norm": ("cacheir_b200_gated_rms",),
     "residual_dynamic_tanh": ("cacheir_b200_dense_gemm", "cacheir_b200_residual_dyt"),
-    "fused_geglu": ("cacheir_b200_dense_gemm", "cacheir_b200_dense_simple", "cacheir_b200_geglu_pairs"),
+    "fused_geglu": ("cacheir_b200_dense_gemm", "cacheir_b200_dense_simple", "cacheir_b200_glu_pairs"),
     "token_side_gate": ("cacheir_b200_dense_gemm", "cacheir_b200_dense_simple", "cacheir_b200_gelu_embed"),
     "residual_rms_norm": ("cacheir_b200_residual_rms",),
+    "fused_glu": ("cacheir_b200_dense_gemm", "cacheir_b200_dense_simple", "cacheir_b200_glu_pairs"),
+    "rms_norm": ("cacheir_b200_rms_rows",),
+    "tied_attention": ("cacheir_b200_tied_prepare", "cacheir_b200_tied_attention_step", "cacheir_b200_tied_attention_simple"),
+    "expert_router": ("cacheir_b200_dense_gemm", "cacheir_b200_dense_simple", "cacheir_b200_route"),
+    "expert_mixture": ("cacheir_b200_grouped_gemm", "cacheir_b200_grouped_simple", "cacheir_b200_glu_pairs"),
+    "combine_residual_rms_norm": ("cacheir_b200_combine_residual_rms",),
 }
 
 B200_BACKEND = Backend(
@@ -91,6 +97,9 @@ B200_BACKEND = Backend(
         "dense_gemm_bf16",
         "latent_attention",
         "linear_recurrence",
+        "tied_attention",
+        "grouped_gemm_bf16",
+        "expert_routing",
     ),
     notes="Hand-written sm_100a kernels behind a C ABI (libcacheir_b200.so): split-K paged decode attention over a "
           "shared page pool, packed int4/int8 dequant-GEMV, fused glue ops; decode step replayed as a CUDA graph.",

@@ -269,19 +269,42 @@ class _Engine:
         """Several weights of one input, row after row."""
         return self._derive(("concat",) + names, lambda: torch.cat([self.weights.get_checked(n) for n in names]).contiguous(), names)
 
-    def paired_weight(self, names: tuple[str, ...]) -> torch.Tensor:
-        """gate and up rows alternating, the order the gated epilogue wants."""
-        return self._derive(("paired",) + names, lambda: torch.stack([self.weights.get_checked(n) for n in names], dim=1)
-                            .reshape(-1, self.weights.get_checked(names[0]).shape[1]).contiguous(), names)
+    def concat_bias(self, biases: tuple[str | None, ...], names: tuple[str, ...]) -> torch.Tensor:
+        """float32 biases of `concat_weight(names)`, zeros where a weight has none."""
+        return self._derive(("concat_bias",) + biases + names, lambda: torch.cat([
+            torch.zeros(int(self.graph.weights[n].shape[0]), device=self.device) if b is None else self.weights.get_f32(b)
+            for b, n in zip(biases, names)]).contiguous(), [b for b in biases if b is not None])
+
+    def paired_weight(self, names: tuple[str, ...], tail: str | None = None) -> torch.Tensor:
+        """gate and up rows alternating, the order the gated epilogues want; `tail`'s rows behind them."""
+        def make() -> torch.Tensor:
+            pairs = torch.stack([self.weights.get_checked(n) for n in names], dim=1).flatten(0, 1)
+            return (pairs if tail is None else torch.cat([pairs, self.weights.get_checked(tail)])).contiguous()
+        return self._derive(("paired", tail) + names, make, names + (() if tail is None else (tail,)))
+
+    def paired_bias(self, names: tuple[str, ...]) -> torch.Tensor:
+        return self._derive(("paired_bias",) + names, lambda: torch.stack([self.weights.get_f32(n) for n in names], dim=1).flatten().contiguous(), names)
+
+    def expert_pairs(self, gates: tuple[str, ...], ups: tuple[str, ...]) -> torch.Tensor:
+        """[experts * 2 ff, width]: expert after expert, gate and up rows alternating."""
+        def make() -> torch.Tensor:
+            ff, width = (int(n) for n in self.graph.weights[gates[0]].shape)
+            out = torch.empty((len(gates), ff, 2, width), device=self.device, dtype=self.dtype)
+            for e, pair in enumerate(zip(gates, ups)):
+                for i, name in enumerate(pair):
+                    out[e, :, i] = self.weights.get_checked(name)
+                    self.weights.release(name)
+            return out.view(-1, width)
+        return self._derive(("expert_pairs",) + gates + ups, make)
 
     def absorbed_weight(self, name: str, heads: int, dim: int, rank: int) -> torch.Tensor:
         """A key up-projection [heads*dim, rank] turned per head: [heads*rank, dim], applied to queries."""
         return self._derive(("absorbed", name), lambda: self.weights.get_checked(name).view(heads, dim, rank).transpose(1, 2)
                             .reshape(heads * rank, dim).contiguous())
 
-    def rotate_half_table(self, dims: int, base: float) -> torch.Tensor:
-        return self._derive(("rotate_half", dims, base),
-                            lambda: torch.from_numpy(rotate_half_table(self.max_seq_len, dims, base)).to(self.device))
+    def rotate_half_table(self, dims: int, base: float, scaling: tuple[float, ...] | None = None) -> torch.Tensor:
+        return self._derive(("rotate_half", dims, base, scaling),
+                            lambda: torch.from_numpy(rotate_half_table(self.max_seq_len, dims, base, scaling)).to(self.device))
 
     def decay_powers(self, decay: tuple[float, ...]) -> torch.Tensor:
         return self._derive(("decay",) + decay, lambda: hybrid_ops.decay_powers(decay, self.device))

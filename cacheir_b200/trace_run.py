@@ -70,7 +70,7 @@ def main(argv: list[str] | None = None) -> int:
     from . import build, models
     folder = Path(args.model)
     config = json.loads((folder / "config.json").read_text(encoding="utf-8"))
-    build.build(groups=(models.family_for(config).kernel_group,))
+    build.build(groups=models.family_for(config).kernel_groups)
 
     from .kv_cache import B200KVPageAllocator
     from .runtime import B200DecodeRuntime

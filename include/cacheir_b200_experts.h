@@ -1,0 +1,82 @@
+/*
+ * cacheir_b200_experts.h -- C ABI of libcacheir_b200_experts.so: attention whose values are its keys, and mixtures of
+ * experts (Topunex). Rows of a step as in cacheir_b200_ragged.h.
+ */
+#ifndef CACHEIR_B200_EXPERTS_H_
+#define CACHEIR_B200_EXPERTS_H_
+
+#include "cacheir_b200_ragged.h"
+
+#ifdef __cplusplus
+extern "C" {
+#endif
+
+/* ---- tied attention: grouped-query attention with v = k as projected -------------------------------------------------
+ * Queries and keys are rotated (rotate-half pairs on the first rot_dims entries of a head) and divided by their root mean
+ * square. A cached row of a key/value head is (k as projected | its first rot_dims entries rotated), so that it serves as
+ * value and, with its reciprocal root mean square kept beside it, as key:
+ *   q . key = (q[rot_dims:] . k[rot_dims:] + q[:rot_dims] . rotated) * inv_rms
+ * score = cap * tanh(q . key * scale / cap) (cap <= 0: no cap). A row at position i sees j <= i with i - j < window or
+ * j < keep_first. exp(sink[head]) joins the denominator (sink NULL: nothing does). */
+typedef struct {
+  /* rows */
+  const int32_t* positions;
+  const int32_t* row_seg;
+  const int32_t* cu_rows;
+  const int32_t* page_table;
+  int rows, segments, max_pages, page_size, num_slots;
+  /* sizes */
+  int heads, kv_heads, dim, rot_dims, window, keep_first;
+  float scale, cap;
+  /* cache: rows [num_slots, kv_heads, page_size, dim + rot_dims] of `dtype`, inv_rms [num_slots, kv_heads, page_size] */
+  void* pool;
+  float* inv_rms;
+  const float* sink;
+  int dtype;
+  int decode;               /* every segment has exactly one row (row i belongs to segment i) */
+} cacheir_b200_tied_args;
+
+/* q [rows, q_stride] heads*dim columns, k [rows, k_stride] kv_heads*dim columns, both as projected: the cache rows go to
+ * the pool, queries to q_out [rows, heads, dim + rot_dims - lead] as what a cached row is multiplied with: rot_dims zeros,
+ * unrotated entries, rotated entries, without the first lead = rot_dims / 64 * 64 zeros. rope_table: float2 (cos, sin)
+ * [rope_positions, rot_dims / 2]. */
+int cacheir_b200_tied_prepare(const cacheir_b200_tied_args* a, const void* q, long long q_stride, const void* k, long long k_stride,
+                              float eps, const float* rope_table, int rope_positions, void* q_out, void* stream);
+/* out [rows, heads*dim] = attention * sigmoid(gate), gate [rows, gate_stride] before its sigmoid (NULL: no gate).
+ * simple: any extents, float32 arithmetic. prompt: tiles of neighbouring tokens on the tensor cores. step: one row per
+ * segment, `splits` CTAs (at most 8, 0 = choose) share a sequence. */
+int cacheir_b200_tied_attention_simple(const cacheir_b200_tied_args* a, const void* q, const void* gate, long long gate_stride, void* out,
+                                       void* stream);
+int cacheir_b200_tied_step_supported(int heads, int kv_heads, int dim, int rot_dims, int page_size, int dtype);
+int cacheir_b200_tied_step_splits(int rows, int heads, int kv_heads, int window, int keep_first, int max_pages, int page_size);
+int cacheir_b200_tied_attention_step(const cacheir_b200_tied_args* a, const void* q, const void* gate, long long gate_stride, void* out,
+                                     int splits, void* stream);
+
+/* ---- mixtures of experts ----------------------------------------------------------------------------------------------
+ * route: per row of logits [rows, stride] the `top` experts with the largest values (lower index first among equals),
+ * weight = sigmoid(logit) * scale. The rows x top choices get places 0.. in expert order:
+ *   cu [experts + 1] first place of every expert; token_of [rows*top] row of a place; place_of, weight [rows, top].
+ *   chosen [rows, top] the experts
+ * Rows with row_seg < 0 choose nothing (place_of = -1). `counters`: experts + 1 zeroed ints, left zeroed. */
+int cacheir_b200_route(const float* logits, long long stride, const int32_t* row_seg, int rows, int experts, int top, float scale,
+                       int32_t* counters, int32_t* cu, int32_t* token_of, int32_t* place_of, float* weight, int32_t* chosen, void* stream);
+/* Y[place] = f(X[row] W_e^T) for the places of every expert e, whose W rows start at e*w_batch_rows; row = token_of[place],
+ * or the place itself when token_of is NULL. a->T places at most, a->batch experts, a->x has x_rows rows. Epilogues:
+ * BF16, SWIGLU, CLAMPED_GLU. Strides must be multiples of 8 elements. */
+int cacheir_b200_grouped_gemm(const cacheir_b200_dense_args* a, const int32_t* cu, const int32_t* token_of, int x_rows, void* stream);
+/* The same product without its epilogue in float32 arithmetic, any extents. */
+int cacheir_b200_grouped_simple(const void* x, const void* w, void* y, const int32_t* cu, const int32_t* token_of, int places, int experts,
+                                int N, int K, long long w_stride, long long x_stride, long long y_stride, int dtype, void* stream);
+/* m = sum_k weight[t, k] * y[place_of[t, k]] + shared[t] (shared may be NULL); residual += m / sqrt(mean(m^2) + eps) * w,
+ * then next_mode (NONE or COPY) */
+int cacheir_b200_combine_residual_rms(float* residual, const void* y, const int32_t* place_of, const float* weight, int top,
+                                      const void* shared, const float* w, float eps, int rows, int width, int next_mode, void* next_out,
+                                      int dtype, void* stream);
+
+/* First bounded wait of this library's kernels that gave up since the last reset (0: none). Synchronises. */
+int cacheir_b200_experts_device_status(int reset);
+
+#ifdef __cplusplus
+}
+#endif
+#endif

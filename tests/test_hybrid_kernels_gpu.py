@@ -189,7 +189,7 @@ def test_row_operators(rows, width, dtype):
     got = H.gated_rms(y, gate[:, 3:3 + width], w, 1e-5, torch.empty_like(y))
     _close(got, G.rms(yn, 1e-5) * wn * G.sigmoid(gn[:, 3:3 + width]), tol)
     pair, pn = _rand(rng, rows, 2 * width, dtype=td)
-    _close(H.geglu_pairs(pair, torch.empty_like(y)), G.gelu_tanh(pn[:, 0::2]) * pn[:, 1::2], tol)
+    _close(H.glu_pairs(pair, torch.empty_like(y)), G.gelu_tanh(pn[:, 0::2]) * pn[:, 1::2], tol)
     side, sn = _rand(rng, 13, width + 7, dtype=td)
     _close(H.gelu_embed(y, ids, side, 5, torch.empty_like(y)), G.gelu_tanh(yn) * sn[ids.cpu().numpy(), 5:5 + width], tol)
     z = y.clone()
