@@ -185,6 +185,8 @@ GROUP_SIGNATURES: dict[str, dict[str, tuple[object, list[object]]]] = {
         "cacheir_b200_tied_prepare": (
             c_int, [c_void_p, c_void_p, c_longlong, c_void_p, c_longlong, c_float, c_void_p, c_int, c_void_p, c_void_p]),
         "cacheir_b200_tied_attention_simple": (c_int, [c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_void_p]),
+        "cacheir_b200_tied_prompt_supported": (c_int, [c_int] * 6),
+        "cacheir_b200_tied_attention_prompt": (c_int, [c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_void_p]),
         "cacheir_b200_tied_step_supported": (c_int, [c_int] * 6),
         "cacheir_b200_tied_step_splits": (c_int, [c_int] * 7),
         "cacheir_b200_tied_attention_step": (c_int, [c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_int, c_void_p]),

@@ -30,7 +30,7 @@ SHARED = ("glue", "misc")            # in the core and the ragged library: argma
 GROUP_FILES = {
     "ragged": ("dense_gemm", "hybrid_glue") + SHARED,
     "hybrid": ("latent_attention", "linear_recurrence"),
-    "experts": ("tied_attention", "grouped_gemm", "expert_routing"),
+    "experts": ("tied_attention", "tied_prompt", "grouped_gemm", "expert_routing"),
 }
 LIB_PATHS = {"core": LIB_DIR / "libcacheir_b200.so", **{name: LIB_DIR / f"libcacheir_b200_{name}.so" for name in GROUP_FILES}}
 LIB_PATH = LIB_PATHS["core"]

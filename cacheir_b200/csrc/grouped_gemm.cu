@@ -72,6 +72,7 @@ grouped_simple_kernel(const T* __restrict__ x, const T* __restrict__ w, T* __res
 }  // namespace
 
 int tied_attention_status(bool reset);
+int tied_prompt_status(bool reset);
 
 }  // namespace cb200
 
@@ -111,6 +112,6 @@ extern "C" int cacheir_b200_grouped_simple(const void* x, const void* w, void* y
 }
 
 extern "C" int cacheir_b200_experts_device_status(int reset) {
-  const int gemm = device_status_word(g_dense_status, reset != 0), attn = tied_attention_status(reset != 0);
-  return gemm != 0 ? gemm : attn;
+  const int gemm = device_status_word(g_dense_status, reset != 0), step = tied_attention_status(reset != 0), prompt = tied_prompt_status(reset != 0);
+  return gemm != 0 ? gemm : step != 0 ? step : prompt;
 }

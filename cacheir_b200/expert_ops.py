@@ -63,6 +63,15 @@ def tied_attention_simple(a: TiedArgs, q: torch.Tensor, gate: torch.Tensor | Non
     return out
 
 
+def tied_prompt_supported(heads: int, kv_heads: int, dim: int, rot_dims: int, page_size: int, dtype: torch.dtype) -> bool:
+    return bool(_lib.load_group("experts").cacheir_b200_tied_prompt_supported(heads, kv_heads, dim, rot_dims, page_size, dtype_code(dtype)))
+
+
+def tied_attention_prompt(a: TiedArgs, q: torch.Tensor, gate: torch.Tensor | None, out: torch.Tensor) -> torch.Tensor:
+    check(_lib.load_group("experts").cacheir_b200_tied_attention_prompt(*_attend(a, q, gate, out), _stream()), "tied_attention_prompt")
+    return out
+
+
 def tied_step_supported(heads: int, kv_heads: int, dim: int, rot_dims: int, page_size: int, dtype: torch.dtype) -> bool:
     return bool(_lib.load_group("experts").cacheir_b200_tied_step_supported(heads, kv_heads, dim, rot_dims, page_size, dtype_code(dtype)))
 

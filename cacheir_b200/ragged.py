@@ -399,6 +399,8 @@ def make_plan_class(base: type) -> type:
             if self.decode and X.tied_step_supported(heads, kv_heads, dim, rot, eng.page_size, eng.dtype):
                 splits = X.tied_step_splits(self.batch, heads, kv_heads, int(at["window"]), int(at["keep_first"]), self.width, eng.page_size)
                 self._emit(lambda: X.tied_attention_step(args, prepared, gate, out, splits=splits), "b200.tied_attention_step")
+            elif X.tied_prompt_supported(heads, kv_heads, dim, rot, eng.page_size, eng.dtype) and gate.stride(0) % 8 == 0:
+                self._emit(lambda: X.tied_attention_prompt(args, prepared, gate, out), "b200.tied_attention_prompt")
             else:
                 self._emit(lambda: X.tied_attention_simple(args, prepared, gate, out), "b200.tied_attention_simple")
             self._env[node.outputs[0]] = out

@@ -68,7 +68,8 @@ HYBRID_KERNELS_FOR_OP: dict[str, tuple[str, ...]] = {
     "residual_rms_norm": ("cacheir_b200_residual_rms",),
     "fused_glu": ("cacheir_b200_dense_gemm", "cacheir_b200_dense_simple", "cacheir_b200_glu_pairs"),
     "rms_norm": ("cacheir_b200_rms_rows",),
-    "tied_attention": ("cacheir_b200_tied_prepare", "cacheir_b200_tied_attention_step", "cacheir_b200_tied_attention_simple"),
+    "tied_attention": ("cacheir_b200_tied_prepare", "cacheir_b200_tied_attention_step", "cacheir_b200_tied_attention_prompt",
+                       "cacheir_b200_tied_attention_simple"),
     "expert_router": ("cacheir_b200_dense_gemm", "cacheir_b200_dense_simple", "cacheir_b200_route"),
     "expert_mixture": ("cacheir_b200_grouped_gemm", "cacheir_b200_grouped_simple", "cacheir_b200_glu_pairs"),
     "combine_residual_rms_norm": ("cacheir_b200_combine_residual_rms",),

@@ -47,6 +47,9 @@ int cacheir_b200_tied_prepare(const cacheir_b200_tied_args* a, const void* q, lo
  * segment, `splits` CTAs (at most 8, 0 = choose) share a sequence. */
 int cacheir_b200_tied_attention_simple(const cacheir_b200_tied_args* a, const void* q, const void* gate, long long gate_stride, void* out,
                                        void* stream);
+int cacheir_b200_tied_prompt_supported(int heads, int kv_heads, int dim, int rot_dims, int page_size, int dtype);
+int cacheir_b200_tied_attention_prompt(const cacheir_b200_tied_args* a, const void* q, const void* gate, long long gate_stride, void* out,
+                                       void* stream);
 int cacheir_b200_tied_step_supported(int heads, int kv_heads, int dim, int rot_dims, int page_size, int dtype);
 int cacheir_b200_tied_step_splits(int rows, int heads, int kv_heads, int window, int keep_first, int max_pages, int page_size);
 int cacheir_b200_tied_attention_step(const cacheir_b200_tied_args* a, const void* q, const void* gate, long long gate_stride, void* out,
