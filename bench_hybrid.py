@@ -1,5 +1,5 @@
-"""`bench.py --family gutorax`: prefill and decode throughput of the Gutorax family beside the Llama-shaped family at
-equal width, feed-forward, heads and layer count (random weights), and every kernel's distance from its roofline.
+"""`bench.py --family gutorax|topunex`: prefill and decode throughput of a ragged family beside the other ones at equal
+width, (active) feed-forward, heads and layer count (random weights), and every kernel's distance from its roofline.
 
 Throughput: decode is `decode_greedy_batch` (CUDA-graph replay, argmax fed back on the device) over `batch` sequences
 with `ctx` cached tokens; prefill is one prompt through the runtime's own entry point, with the last position's logits
@@ -12,9 +12,12 @@ from __future__ import annotations
 from collections import defaultdict
 
 SIZES = {
-    # width, ff, heads, kv_heads (Llama), head dim, latent rank, rotated dims, window, layers, vocab
-    "4096": dict(width=4096, ff=14336, heads=32, kv_heads=8, dim=128, rank=512, rot=64, window=4096, layers=8, vocab=32768, side=256),
-    "2048": dict(width=2048, ff=5632, heads=16, kv_heads=8, dim=128, rank=256, rot=64, window=1024, layers=12, vocab=32768, side=128),
+    # width, ff, heads, kv_heads, head dim, latent rank, rotated dims, window, layers, vocab; mixtures (every second Topunex
+    # layer): top experts and the shared one add up to ff
+    "4096": dict(width=4096, ff=14336, heads=32, kv_heads=8, dim=128, rank=512, rot=64, window=4096, layers=8, vocab=32768, side=256,
+                 experts=32, top=4, expert_ff=1792, shared_ff=7168, keep=4),
+    "2048": dict(width=2048, ff=5632, heads=16, kv_heads=8, dim=128, rank=256, rot=64, window=1024, layers=12, vocab=32768, side=128,
+                 experts=32, top=4, expert_ff=704, shared_ff=2816, keep=4),
 }
 
 
@@ -35,6 +38,17 @@ def gutorax_config(s: dict) -> dict:
             "norm": {"eps": 1e-5}, "token_side": {"dim": s["side"]}, "layers": layers}
 
 
+def topunex_config(s: dict) -> dict:
+    """Dense layers and mixtures of experts in turn."""
+    mixer = {"heads": s["heads"], "kv_heads": s["kv_heads"], "dim": s["dim"], "vdim": s["dim"], "scale": s["dim"] ** -0.5, "softcap": 30.0,
+             "mask": {"size": s["window"], "keep_first": s["keep"]},
+             "rot": {"base": 500000.0, "dims": s["rot"], "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}}
+    moe = {"kind": "moe", "expert": {"ff": s["expert_ff"], "limit": 7.0}, "shared": {"ff": s["shared_ff"], "limit": 7.0},
+           "router": {"experts": s["experts"], "top": s["top"], "scale": 2.0}}
+    return {"architecture": "Topunex", "width": s["width"], "vocab": s["vocab"], "norm": {"eps": 1e-6},
+            "layers": [{"type": "attention", "mixer": mixer, "mlp": moe if i % 2 else {"kind": "dense", "ff": s["ff"]}} for i in range(s["layers"])]}
+
+
 def synthetic(device):
     import zlib
 
@@ -53,11 +67,13 @@ def build(family: str, s: dict, *, batch: int, positions: int):
     import torch
 
     from cacheir_b200 import (B200DecodeRuntime, B200KVPageAllocator, GutoraxConfig, ModelConfig, build_decoder_artifact,
-                              build_gutorax_artifact)
+                              TopunexConfig, build_gutorax_artifact, build_topunex_artifact)
     dev = torch.device("cuda", torch.cuda.current_device())
     if family == "gutorax":
         art, page = build_gutorax_artifact(GutoraxConfig.from_dict(gutorax_config(s))), 64
         dtype = "bfloat16"
+    elif family == "topunex":
+        art, page, dtype = build_topunex_artifact(TopunexConfig.from_dict(topunex_config(s))), 64, "bfloat16"
     else:
         art = build_decoder_artifact(ModelConfig(
             architecture="LlamaForCausalLM", hidden_size=s["width"], intermediate_size=s["ff"], num_layers=s["layers"],
@@ -74,8 +90,8 @@ def fill(rt, batch: int, ctx: int):
     for s in sessions:
         s.kv_cache.extend(ctx)
     for pool in rt.kv_allocator._pools.values():
-        for t in pool.values():
-            t.normal_()
+        for name, t in pool.items():
+            t.fill_(1.0) if name == "inv_rms" else t.normal_()
     for state in rt.kv_allocator._states.values():
         state.normal_()
     return sessions
@@ -146,11 +162,46 @@ def gutorax_work(s: dict, rows: int, logit_rows: int, keys_per_row: float, cache
         gemm(".geglu", 2 * ff, w, ff)
         gemm(".residual_dyt", w, ff, 0, extra=rows * w * (8 + 2))
         gemm(".gelu_embed", side, w, 2 * side)
-        gemm("", w, side, w)
+        gemm(".side", w, side, w)
         work["b200.residual_rms"].append((rows * w * (2 + 8 + 2.0), 0.0))
     work["b200.scaled_embedding"].append((rows * w * (2 + 4 + 2.0), 0.0))
     work["b200.dyt_rows"].append((logit_rows * w * 6.0, 0.0))
-    gemm("", s["vocab"], w, 2 * s["vocab"], t=logit_rows)
+    gemm(".lm_head", s["vocab"], w, 2 * s["vocab"], t=logit_rows)
+    return work
+
+
+def topunex_work(s: dict, rows: int, logit_rows: int, keys_per_row: float, cached_rows: float, decode: bool) -> dict[str, list[tuple[float, float]]]:
+    w, ff, h, g, d, rot = s["width"], s["ff"], s["heads"], s["kv_heads"], s["dim"], s["rot"]
+    work: dict[str, list[tuple[float, float]]] = defaultdict(list)
+
+    def gemm(kind, n, k, n_out, t=rows, weights=1.0):
+        work["b200." + kind].append((2.0 * (weights * n * k + t * k + t * n_out), 2.0 * t * n * k))
+
+    qw = d + rot - rot // 64 * 64
+    touched = s["experts"] * (1.0 - (1.0 - s["top"] / s["experts"]) ** rows)
+    for i in range(s["layers"]):
+        n = (2 * h + g) * d
+        gemm("dense_gemm", n, w, n)
+        work["b200.tied_prepare"].append((2.0 * rows * (h * (d + qw) + g * (2 * d + rot)), 0.0))
+        work["b200.tied_attention_step" if decode else "b200.tied_attention_prompt"].append(
+            (cached_rows * g * (2.0 * (d + rot) + 4) + 2.0 * rows * h * (qw + 2 * d), 4.0 * rows * h * keys_per_row * d))
+        gemm("dense_gemm.o", w, h * d, w)
+        work["b200.residual_rms"].append((rows * w * (2 + 8 + 2.0), 0.0))
+        if i % 2:
+            places = rows * s["top"]
+            gemm("dense_gemm.clamped_glu", 2 * s["shared_ff"] + s["experts"], w, s["shared_ff"])
+            gemm("dense_gemm.down", w, s["shared_ff"], w)
+            work["b200.route"].append((rows * (s["experts"] * 4.0 + s["top"] * 16), 0.0))
+            gemm("grouped_gemm.clamped_glu", 2 * s["expert_ff"], w, s["expert_ff"], t=places, weights=touched)
+            gemm("grouped_gemm", w, s["expert_ff"], w, t=places, weights=touched)
+            work["b200.combine_residual_rms"].append((rows * w * (2 * s["top"] + 2 + 8 + 2.0), 0.0))
+        else:
+            gemm("dense_gemm.swiglu", 2 * ff, w, ff)
+            gemm("dense_gemm.down", w, ff, w)
+            work["b200.residual_rms"].append((rows * w * (2 + 8 + 2.0), 0.0))
+    work["b200.scaled_embedding"].append((rows * w * (2 + 4 + 2.0), 0.0))
+    work["b200.rms_rows"].append((logit_rows * w * 6.0, 0.0))
+    gemm("dense_gemm.lm_head", s["vocab"], w, 2 * s["vocab"], t=logit_rows)
     return work
 
 
@@ -185,13 +236,16 @@ def against_roofline(times: dict[str, tuple[int, float]], work: dict, hbm_gbs: f
     return out
 
 
-def run(size: str, batch: int, ctx: int, prompt: int, steps: int, peaks: dict) -> dict:
+RAGGED_WORK = {"gutorax": gutorax_work, "topunex": topunex_work}
+
+
+def run(size: str, batch: int, ctx: int, prompt: int, steps: int, peaks: dict, families: tuple[str, ...] = ("gutorax",)) -> dict:
     import torch
 
     s = SIZES[size]
     hbm, tf = peaks["hbm_gbs"], peaks["bf16_tflops"]
     line: dict = {"size": size, **s, "batch": batch, "ctx": ctx, "prompt": prompt}
-    for family in ("gutorax", "llama-shaped int8"):
+    for family in families + ("llama-shaped int8",):
         rt = build(family, s, batch=batch, positions=max(ctx, prompt) + 8 * steps + 64)
         sessions = fill(rt, batch, ctx)
         first = [1] * batch
@@ -205,9 +259,9 @@ def run(size: str, batch: int, ctx: int, prompt: int, steps: int, peaks: dict) -
         ms = start.elapsed_time(stop) / steps
         seen = ctx + steps // 2
         plan = rt._engine.plans[("decode", batch)]
-        if family == "gutorax":
+        if family in RAGGED_WORK:
             keys = min(seen, s["window"])
-            decode_kernels = against_roofline(kind_times(plan), gutorax_work(s, batch, batch, keys, batch * keys, True), hbm, tf)
+            decode_kernels = against_roofline(kind_times(plan), RAGGED_WORK[family](s, batch, batch, keys, batch * keys, True), hbm, tf)
         else:
             decode_kernels = against_roofline(kind_times(plan), llama_work(s, batch, seen, batch * seen), hbm, tf)
         for x in sessions:
@@ -217,15 +271,15 @@ def run(size: str, batch: int, ctx: int, prompt: int, steps: int, peaks: dict) -
 
         def prefill():
             session.kv_cache.clear()
-            if family == "gutorax":
+            if family in RAGGED_WORK:
                 session.run_step_batch([session], [ids])
             else:
                 session.run([ids], mode="prefill")
         prefill_ms = timed(prefill, 5)
-        if family == "gutorax":
+        if family in RAGGED_WORK:
             plan = rt._engine.portion_plan(prompt, 1, 1)
             avg = sum(min(i + 1, s["window"]) for i in range(prompt)) / prompt
-            prefill_kernels = against_roofline(kind_times(plan), gutorax_work(s, prompt, 1, avg, prompt, False), hbm, tf)
+            prefill_kernels = against_roofline(kind_times(plan), RAGGED_WORK[family](s, prompt, 1, avg, prompt, False), hbm, tf)
         else:      # the last pass of the prompt: 64 rows that attend to all of it
             plan = rt._engine.prefill_plan(64, 1)
             prefill_kernels = against_roofline(kind_times(plan), llama_work(s, 64, prompt, prompt), hbm, tf)

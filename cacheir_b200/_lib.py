@@ -190,8 +190,9 @@ GROUP_SIGNATURES: dict[str, dict[str, tuple[object, list[object]]]] = {
         "cacheir_b200_tied_step_supported": (c_int, [c_int] * 6),
         "cacheir_b200_tied_step_splits": (c_int, [c_int] * 7),
         "cacheir_b200_tied_attention_step": (c_int, [c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_int, c_void_p]),
-        "cacheir_b200_route": (c_int, [c_void_p, c_longlong, c_void_p, c_int, c_int, c_int, c_float] + [c_void_p] * 7),
-        "cacheir_b200_grouped_gemm": (c_int, [c_void_p, c_void_p, c_void_p, c_int, c_void_p]),
+        "cacheir_b200_route": (c_int, [c_void_p, c_longlong, c_void_p, c_int, c_int, c_int, c_float] + [c_void_p] * 8 + [c_int, c_void_p]),
+        "cacheir_b200_grouped_all_rows": (c_int, []),
+        "cacheir_b200_grouped_gemm": (c_int, [c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p]),
         "cacheir_b200_grouped_simple": (c_int, [c_void_p] * 5 + [c_int] * 4 + [c_longlong] * 3 + [c_int, c_void_p]),
         "cacheir_b200_combine_residual_rms": (
             c_int, [c_void_p] * 4 + [c_int, c_void_p, c_void_p, c_float, c_int, c_int, c_int, c_void_p, c_int, c_void_p]),

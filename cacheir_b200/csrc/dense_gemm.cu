@@ -21,11 +21,11 @@ template <int EPI>
 int launch_mt(const cacheir_b200_dense_args& p, cudaStream_t stream) {
   const Shape s = choose_shape(p.T, p.N, p.K, p.batch);
   switch (s.mt) {
-    case 16: return launch<EPI, 16, false>(p, s.split, stream, {}, p.T);
-    case 32: return launch<EPI, 32, false>(p, s.split, stream, {}, p.T);
-    case 64: return launch<EPI, 64, false>(p, s.split, stream, {}, p.T);
-    case 128: return launch<EPI, 128, false>(p, s.split, stream, {}, p.T);
-    default: return launch<EPI, 256, false>(p, s.split, stream, {}, p.T);
+    case 16: return launch<EPI, 16, false>(p, s.split, stream, {});
+    case 32: return launch<EPI, 32, false>(p, s.split, stream, {});
+    case 64: return launch<EPI, 64, false>(p, s.split, stream, {});
+    case 128: return launch<EPI, 128, false>(p, s.split, stream, {});
+    default: return launch<EPI, 256, false>(p, s.split, stream, {});
   }
 }
 

@@ -17,7 +17,9 @@
 // (32-bit) -> the next norm's output as the next GEMM's bf16 operand.
 // `batch` > 1 runs one GEMM per head: head z takes W rows z*w_batch_rows.. and X columns z*x_batch_cols...
 // GROUPED runs one GEMM per expert over the places [cu[e], cu[e+1]) of a routed step: a token tile belongs to one expert
-// (found from cu on the device), takes W rows e*w_batch_rows.. and X rows token_of[place], four gathered per copy.
+// (found from cu on the device) and takes W rows e*w_batch_rows... X rows are places; or, with place_of, the step's rows
+// themselves: an expert multiplies all of them (at most a tile, and the weights are what takes the time) and keeps those
+// that chose it.
 #pragma once
 
 #include "hybrid_common.cuh"
@@ -33,7 +35,7 @@ constexpr int kTileN = 128;
 constexpr int kBlockK = 64;               // elements of k per stage: one 128-byte swizzle span
 constexpr int kWBytes = kTileN * kBlockK * 2;
 constexpr int kThreads = 320;
-constexpr int kTailBytes = 256;
+constexpr int kTailBytes = 512;                    // barriers; from byte 128 on the places of up to 64 rows
 
 __device__ int g_dense_status = 0;
 
@@ -76,14 +78,9 @@ __device__ __forceinline__ void cluster_sync_all() {
 
 struct Groups {
   const int32_t* cu;         // [batch + 1]
-  const int32_t* token_of;   // X row of a place; NULL: the place itself
+  const int32_t* place_of;   // [x_rows, top]: X rows are the step's rows; NULL: they are places
+  int top, x_rows;
 };
-
-__device__ __forceinline__ void tma_gather4(uint32_t dst, const CUtensorMap* map, uint32_t bar, int x, int r0, int r1, int r2, int r3) {
-  asm volatile(
-      "cp.async.bulk.tensor.2d.shared::cluster.global.tile::gather4.mbarrier::complete_tx::bytes [%0], [%1, {%3, %4, %5, %6, %7}], [%2];"
-      ::"r"(dst), "l"(reinterpret_cast<uint64_t>(map)), "r"(bar), "r"(x), "r"(r0), "r"(r1), "r"(r2), "r"(r3) : "memory");
-}
 
 // gate and up of one unit -> its activation
 template <int EPI>
@@ -117,9 +114,10 @@ dense_gemm_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_const
   const int krank = static_cast<int>(blockIdx.y);      // the cluster spans the whole y extent
   int t0 = blockIdx.x * MT, t_end = p.T, z = blockIdx.z / n_tiles;
   if constexpr (GROUPED) {
-    const RaggedItem it = find_item(groups.cu, p.batch, MT, blockIdx.x);
+    const RaggedItem it = find_item(groups.cu, p.batch, groups.place_of ? 1 << 30 : MT, blockIdx.x);
     if (it.seg < 0) return;                // (the whole cluster)
     z = it.seg; t0 = it.row0; t_end = it.row0 + it.count;
+    if (groups.place_of) { t0 = 0; t_end = groups.x_rows; }
   }
   const int n0 = (blockIdx.z % n_tiles) * kTileN;
   const int kblocks_all = (p.K + kBlockK - 1) / kBlockK;
@@ -146,40 +144,22 @@ dense_gemm_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_const
 
   bool ok = true;
   if (warp == 0) {
-    bool gathers = false;
-    if constexpr (GROUPED) gathers = groups.token_of != nullptr;
-    int rows[MT > 128 ? 8 : 4] = {};       // gathered: this lane's X rows (a place behind the tile repeats the last one)
-    if (gathers) {
-#pragma unroll
-      for (int i = 0; i < (MT > 128 ? 8 : 4); ++i)
-        rows[i] = groups.token_of[min(t0 + (i >> 2) * 128 + lane * 4 + (i & 3), t_end - 1)];
-    }
-    int issued = 0;
-    for (int i = 0; i < total; ++i) {
-      const int s = i % kStages;
-      bool free = true;
-      if (lane == 0 && i >= kStages) free = mbar_wait(smem_u32(&empty[s]), ((i / kStages) & 1) ^ 1, &g_dense_status, (6 << 8) | 1);
-      if (!__shfl_sync(0xffffffffu, free ? 1 : 0, 0)) break;
-      const uint32_t bar = smem_u32(&full[s]);
-      const int k = (kb_begin + i) * kBlockK;
-      if (lane == 0) {
+    if (lane == 0) {
+      int issued = 0;
+      for (int i = 0; i < total; ++i) {
+        const int s = i % kStages;
+        if (i >= kStages && !mbar_wait(smem_u32(&empty[s]), ((i / kStages) & 1) ^ 1, &g_dense_status, (6 << 8) | 1)) break;
+        const uint32_t bar = smem_u32(&full[s]);
         mbar_expect_tx(bar, stage_bytes(MT));
+        const int k = (kb_begin + i) * kBlockK;
         tma_load_2d(smem_u32(s_w + s * kWBytes), &tmap_w, bar, k, z * p.w_batch_rows + n0);
-        if (!gathers) tma_load_2d(smem_u32(s_x + s * MT * kBlockK * 2), &tmap_x, bar, GROUPED ? k : z * p.x_batch_cols + k, t0);
+        tma_load_2d(smem_u32(s_x + s * MT * kBlockK * 2), &tmap_x, bar, GROUPED ? k : z * p.x_batch_cols + k, t0);
+        issued = i + 1;
       }
-      if (gathers) {
-        __syncwarp();
-#pragma unroll
-        for (int i4 = 0; i4 < (MT > 128 ? 2 : 1); ++i4)
-          if (lane * 4 < MT)
-            tma_gather4(smem_u32(s_x + s * MT * kBlockK * 2 + (i4 * 128 + lane * 4) * 128), &tmap_x, bar, k, rows[4 * i4], rows[4 * i4 + 1],
-                        rows[4 * i4 + 2], rows[4 * i4 + 3]);
-      }
-      issued = i + 1;
+      if (issued < total)          // a wait gave up: nothing may still be on its way when the block ends
+        for (int i = issued > kStages ? issued - kStages : 0; i < issued; ++i)
+          mbar_wait(smem_u32(&full[i % kStages]), (i / kStages) & 1, &g_dense_status, (6 << 8) | 4);
     }
-    if (lane == 0 && issued < total)       // a wait gave up: nothing may still be on its way when the block ends
-      for (int i = issued > kStages ? issued - kStages : 0; i < issued; ++i)
-        mbar_wait(smem_u32(&full[i % kStages]), (i / kStages) & 1, &g_dense_status, (6 << 8) | 4);
     __syncwarp();
   } else if (warp == 1) {
     if (lane == 0) {
@@ -209,6 +189,29 @@ dense_gemm_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_const
       w1 = p.norm_w[n]; b1 = p.norm_b[n];
       if (p.next_mode == CACHEIR_B200_NEXT_DYT) { w2 = p.next_w[n]; b2 = p.next_b[n]; }
     }
+    const int* s_place = reinterpret_cast<const int*>(smem + kStages * stage_bytes(MT) + 128);
+    if constexpr (GROUPED && MT <= 64) {
+      if (groups.place_of) {               // where each row's result goes, if this expert has one
+        const int t = threadIdx.x - 64, lo = groups.cu[z], hi = groups.cu[z + 1];
+        if (t < MT) {
+          int place = -1;
+          if (t < t_end)
+            for (int k = 0; k < groups.top; ++k) {
+              const int at = groups.place_of[t * groups.top + k];
+              if (at >= lo && at < hi) place = at;
+            }
+          const_cast<int*>(s_place)[t] = place;
+        }
+        asm volatile("barrier.cta.sync 2, 256;" ::: "memory");
+      }
+    }
+    auto row_of = [&](int t) {             // output row, -1: none
+      if (t >= t_end) return -1;
+      if constexpr (GROUPED && MT <= 64) {
+        if (groups.place_of) return s_place[t];
+      }
+      return t;
+    };
     ok = mbar_wait(smem_u32(acc_full), 0, &g_dense_status, (6 << 8) | 3);
     tc_fence_after();
     const long long ycol = GROUPED ? n : static_cast<long long>(z) * p.y_batch_cols + n;
@@ -224,9 +227,9 @@ dense_gemm_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_const
         for (int j = 0; j < G; j += 2) {
           const float got = __shfl_xor_sync(0xffffffffu, odd ? v[j] : v[j + 1], 1);
           const float y = odd ? paired<EPI>(got, v[j + 1], p.limit) : paired<EPI>(v[j], got, p.limit);
-          const int t = t0 + c0 + j + (odd ? 1 : 0);
-          if (n_ok && !tail && t < t_end)
-            static_cast<__nv_bfloat16*>(p.y)[static_cast<long long>(t) * p.y_stride + (n >> 1)] = __float2bfloat16_rn(y);
+          const int row = row_of(t0 + c0 + j + (odd ? 1 : 0));
+          if (n_ok && !tail && row >= 0)
+            static_cast<__nv_bfloat16*>(p.y)[static_cast<long long>(row) * p.y_stride + (n >> 1)] = __float2bfloat16_rn(y);
           if (n_ok && tail) {
             float* dst = p.tail + static_cast<long long>(t0 + c0 + j) * p.tail_stride + (n - (p.N - p.tail_cols));
             if (t0 + c0 + j < t_end) dst[0] = v[j];
@@ -273,8 +276,8 @@ dense_gemm_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_const
         }
 #pragma unroll
         for (int j = 0; j < G; ++j) {
-          const int t = t0 + c0 + j;
-          if (!(n_ok && t < t_end)) continue;
+          const int t = row_of(t0 + c0 + j);
+          if (!n_ok || t < 0) continue;
           float y = v[j];
           if constexpr (EPI == CACHEIR_B200_DENSE_F32) {
             static_cast<float*>(p.y)[static_cast<long long>(t) * p.y_stride + ycol] = y;
@@ -348,7 +351,7 @@ bool encode_bf16_rows(CUtensorMap* map, const void* base, uint64_t inner, uint64
 }
 
 template <int EPI, int MT, bool GROUPED>
-int launch(const cacheir_b200_dense_args& p, int split, cudaStream_t stream, const Groups& groups, int x_rows) {
+int launch(const cacheir_b200_dense_args& p, int split, cudaStream_t stream, const Groups& groups) {
   constexpr size_t kSmem = 1024 + static_cast<size_t>(num_stages(MT)) * stage_bytes(MT) + kTailBytes;
   static_assert(kSmem * ctas_per_sm(MT) <= 227 * 1024, "ring must fit");
   static_assert(static_cast<size_t>(MT) * kTileN * 4 <= static_cast<size_t>(num_stages(MT)) * stage_bytes(MT), "partials must fit the ring");
@@ -356,14 +359,14 @@ int launch(const cacheir_b200_dense_args& p, int split, cudaStream_t stream, con
   const uint64_t w_rows = p.batch > 1 ? static_cast<uint64_t>(p.w_batch_rows) * (p.batch - 1) + p.N : p.N;
   const uint64_t x_cols = GROUPED ? p.K : static_cast<uint64_t>(p.x_batch_cols) * (p.batch - 1) + p.K;
   if (!encode_bf16_rows(&tw, p.w, p.K, w_rows, p.w_stride, kTileN) ||
-      !encode_bf16_rows(&tx, p.x, x_cols, x_rows, p.x_stride, groups.token_of ? 1 : MT))
+      !encode_bf16_rows(&tx, p.x, x_cols, GROUPED ? groups.x_rows : p.T, p.x_stride, MT))
     return CACHEIR_B200_EUNSUPPORTED;
   auto kern = dense_gemm_kernel<EPI, MT, GROUPED>;
   cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(kSmem));
   if (e != cudaSuccess) return static_cast<int>(e);
   const int n_tiles = (p.N + kTileN - 1) / kTileN;
   cudaLaunchConfig_t cfg{};
-  cfg.gridDim = GROUPED ? dim3(ragged_items(p.T, p.batch, MT), split, n_tiles) : dim3((p.T + MT - 1) / MT, split, n_tiles * p.batch);
+  cfg.gridDim = GROUPED ? dim3((groups.place_of ? 0 : p.T / MT) + (p.T < p.batch ? p.T : p.batch), split, n_tiles) : dim3((p.T + MT - 1) / MT, split, n_tiles * p.batch);
   cfg.blockDim = dim3(kThreads, 1, 1);
   cfg.dynamicSmemBytes = kSmem;
   cfg.stream = stream;

@@ -7,8 +7,58 @@ namespace cb200 {
 namespace {
 
 constexpr int kRouteThreads = 256;      // a warp per token
+constexpr int kHeld = 4;                // logits a lane keeps in registers
+
+// The warp's token: its choices in order, each with its rank among the tokens of that expert (in no particular order).
+template <bool HELD>
+__device__ __forceinline__ void choose(const float* z, bool real, int row, int experts, int top, float scale, int32_t* counters,
+                                       int32_t* place_of, float* weight, int32_t* chosen) {
+  const int lane = threadIdx.x & 31;
+  float held[kHeld];
+  if (HELD) {
+#pragma unroll
+    for (int i = 0; i < kHeld; ++i) held[i] = lane + 32 * i < experts ? z[lane + 32 * i] : 0.f;
+  }
+  float bound = INFINITY;               // the last choice: what follows it in (value descending, index ascending) order is next
+  int after = -1, mine = -1;
+  float mine_z = 0.f;
+  for (int k = 0; k < top; ++k) {
+    float best = -INFINITY;
+    int at = experts;
+    auto look = [&](int e, float v) {
+      if ((v < bound || (v == bound && e > after)) && (v > best || at == experts)) { best = v; at = e; }
+    };
+    if (HELD) {
+#pragma unroll
+      for (int i = 0; i < kHeld; ++i)
+        if (lane + 32 * i < experts) look(lane + 32 * i, held[i]);
+    } else {
+      for (int e = lane; e < experts; e += 32) look(e, z[e]);
+    }
+#pragma unroll
+    for (int off = 16; off > 0; off >>= 1) {
+      const float v = __shfl_xor_sync(0xffffffffu, best, off);
+      const int e = __shfl_xor_sync(0xffffffffu, at, off);
+      if (e < experts && (at == experts || v > best || (v == best && e < at))) { best = v; at = e; }
+    }
+    bound = best;
+    after = at;
+    if (lane == k % 32) { mine = at; mine_z = best; }
+    if (k % 32 == 31 || k == top - 1) { // the lanes record what they hold: one round of atomics for up to 32 choices
+      const int j = k / 32 * 32 + lane;
+      if (j <= k) {
+        const bool take = real && mine < experts;      // (a row of NaNs chooses nothing)
+        chosen[row * top + j] = take ? mine : -1;
+        weight[row * top + j] = take ? sigmoid_exact(mine_z) * scale : 0.f;
+        place_of[row * top + j] = take ? atomicAdd(&counters[mine], 1) : -1;
+      }
+    }
+  }
+}
 
 // Every block chooses for its tokens and counts; the block that finishes last turns counts into places (nobody waits).
+// PLACE false: choices and ranks only.
+template <bool HELD, bool PLACE>
 __global__ void __launch_bounds__(kRouteThreads)
 route_kernel(const float* __restrict__ logits, long long stride, const int32_t* __restrict__ row_seg, int rows, int experts, int top,
              float scale, int32_t* counters, int32_t* __restrict__ cu, int32_t* __restrict__ token_of, int32_t* place_of,
@@ -18,34 +68,9 @@ route_kernel(const float* __restrict__ logits, long long stride, const int32_t* 
   __shared__ bool s_last;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int row = blockIdx.x * (kRouteThreads / 32) + warp;
-  if (row < rows) {
-    const float* z = logits + static_cast<long long>(row) * stride;
-    const bool real = row_seg[row] >= 0;
-    float bound = INFINITY;             // the last choice: what follows it in (value descending, index ascending) order is next
-    int after = -1;
-    for (int k = 0; k < top; ++k) {
-      float best = -INFINITY;
-      int at = experts;
-      for (int e = lane; e < experts; e += 32) {
-        const float v = z[e];
-        if ((v < bound || (v == bound && e > after)) && (v > best || at == experts)) { best = v; at = e; }
-      }
-#pragma unroll
-      for (int off = 16; off > 0; off >>= 1) {
-        const float v = __shfl_xor_sync(0xffffffffu, best, off);
-        const int e = __shfl_xor_sync(0xffffffffu, at, off);
-        if (e < experts && (at == experts || v > best || (v == best && e < at))) { best = v; at = e; }
-      }
-      bound = best;
-      after = at;
-      if (lane == 0) {
-        const bool take = real && at < experts;      // (a row of NaNs chooses nothing)
-        chosen[row * top + k] = take ? at : -1;
-        weight[row * top + k] = take ? sigmoid_exact(best) * scale : 0.f;
-        place_of[row * top + k] = take ? atomicAdd(&counters[at], 1) : -1;      // its rank within the expert, for now
-      }
-    }
-  }
+  if (row < rows)
+    choose<HELD>(logits + static_cast<long long>(row) * stride, row_seg[row] >= 0, row, experts, top, scale, counters, place_of, weight, chosen);
+  if (!PLACE) return;
   __threadfence();
   __syncthreads();
   if (threadIdx.x == 0) s_last = atomicAdd(&counters[experts], 1) == static_cast<int>(gridDim.x) - 1;
@@ -82,11 +107,57 @@ route_kernel(const float* __restrict__ logits, long long stride, const int32_t* 
     counters[experts] = 0;
   }
   for (int i = threadIdx.x; i < rows * top; i += kRouteThreads) {
-    const int e = __ldcg(&chosen[i]);
+    const int e = __ldcg(&chosen[i]), rank = __ldcg(&place_of[i]);
     if (e < 0) continue;
-    const int place = s_first[e] + __ldcg(&place_of[i]);
+    const int place = s_first[e] + rank;
     place_of[i] = place;
     token_of[place] = i / top;
+  }
+}
+
+// Places from ranks, and every row's copy at each of its places: a block per row, each adding up the counts it needs.
+__global__ void __launch_bounds__(kRouteThreads)
+place_kernel(int rows, int experts, int top, int32_t* counters, int32_t* __restrict__ cu, int32_t* __restrict__ token_of,
+             int32_t* __restrict__ place_of, const int32_t* __restrict__ chosen, const uint4* __restrict__ x, uint4* __restrict__ placed,
+             int pieces) {
+  extern __shared__ int s_count[];      // [experts], then [top] places
+  __shared__ bool s_last;
+  int* s_place = s_count + experts;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, row = blockIdx.x;
+  for (int e = threadIdx.x; e < experts; e += kRouteThreads) s_count[e] = __ldcg(&counters[e]);
+  __syncthreads();
+  if (threadIdx.x == 0) s_last = atomicAdd(&counters[experts], 1) == static_cast<int>(gridDim.x) - 1;
+  for (int k = warp; k < top; k += kRouteThreads / 32) {
+    const int e = chosen[row * top + k];
+    int before = 0;
+    for (int i = lane; i < e; i += 32) before += s_count[i];
+#pragma unroll
+    for (int off = 16; off > 0; off >>= 1) before += __shfl_xor_sync(0xffffffffu, before, off);
+    if (lane == 0) {
+      const int place = e < 0 ? -1 : before + place_of[row * top + k];
+      s_place[k] = place;
+      if (e >= 0) {
+        place_of[row * top + k] = place;
+        token_of[place] = row;
+      }
+    }
+  }
+  __syncthreads();
+  for (int c = threadIdx.x; c < pieces; c += kRouteThreads) {
+    const uint4 v = x[static_cast<size_t>(row) * pieces + c];
+    for (int k = 0; k < top; ++k)
+      if (s_place[k] >= 0) placed[static_cast<size_t>(s_place[k]) * pieces + c] = v;
+  }
+  if (s_last) {                         // every block has read the counts
+    if (threadIdx.x == 0) {
+      int at = 0;
+      for (int e = 0; e < experts; ++e) {
+        cu[e] = at;
+        at += s_count[e];
+      }
+      cu[experts] = at;
+    }
+    for (int e = threadIdx.x; e <= experts; e += kRouteThreads) counters[e] = 0;
   }
 }
 
@@ -144,15 +215,29 @@ using namespace cb200;
 
 extern "C" int cacheir_b200_route(const float* logits, long long stride, const int32_t* row_seg, int rows, int experts, int top, float scale,
                                   int32_t* counters, int32_t* cu, int32_t* token_of, int32_t* place_of, float* weight, int32_t* chosen,
-                                  void* stream) {
+                                  const void* x, void* placed, int row_bytes, void* stream) {
   if (rows <= 0) return 0;
   if (!logits || !row_seg || experts < 1 || top < 1 || top > experts || stride < experts || !counters || !cu || !token_of || !place_of ||
-      !weight || !chosen)
+      !weight || !chosen || (placed && (!x || row_bytes <= 0)))
     return CACHEIR_B200_EINVAL;
-  const size_t smem = static_cast<size_t>(experts + 1) * 4;
+  if (placed && (row_bytes % 16 != 0 || !aligned_to(x, 16) || !aligned_to(placed, 16))) return CACHEIR_B200_EALIGN;
+  const size_t smem = static_cast<size_t>(experts + top + 1) * 4;
   if (smem > 40 * 1024) return CACHEIR_B200_ELIMIT;
-  route_kernel<<<(rows + 7) / 8, kRouteThreads, smem, as_stream(stream)>>>(logits, stride, row_seg, rows, experts, top, scale, counters, cu,
-                                                                          token_of, place_of, weight, chosen);
+  const int blocks = (rows + 7) / 8;
+  cudaStream_t st = as_stream(stream);
+#define CB200_ROUTE(HELD, PLACE)                                                                                                    \
+  route_kernel<HELD, PLACE><<<blocks, kRouteThreads, PLACE ? smem : 0, st>>>(logits, stride, row_seg, rows, experts, top, scale, counters, \
+                                                                             cu, token_of, place_of, weight, chosen)
+  if (!placed) {
+    if (experts <= 32 * kHeld) CB200_ROUTE(true, true);
+    else CB200_ROUTE(false, true);
+    return launch_status();
+  }
+  if (experts <= 32 * kHeld) CB200_ROUTE(true, false);
+  else CB200_ROUTE(false, false);
+#undef CB200_ROUTE
+  place_kernel<<<rows, kRouteThreads, smem, st>>>(rows, experts, top, counters, cu, token_of, place_of, chosen, static_cast<const uint4*>(x),
+                                                  static_cast<uint4*>(placed), row_bytes / 16);
   return launch_status();
 }
 

@@ -5,15 +5,18 @@
 namespace cb200 {
 namespace {
 
-// Tile width from the mean number of places per expert: a wider tile reads an expert's weights once, a narrower one wastes
-// less of the tensor core.
-int choose_tile(int places, int experts) {
+constexpr int kAllRows = 64;      // a step of at most this many rows is multiplied as a whole by every expert in use
+
+// Tile width from the mean number of places per expert: a wider tile reads an expert's weights fewer times, a narrower one
+// leaves less of its last tile unused.
+int choose_tile(int places, int experts, const Groups& g) {
+  if (g.place_of) return g.x_rows <= 16 ? 16 : g.x_rows <= 32 ? 32 : 64;
   const int mean = (places + experts - 1) / experts;
-  return mean <= 8 ? 16 : mean <= 16 ? 32 : mean <= 32 ? 64 : mean <= 160 ? 128 : 256;
+  return mean <= 8 ? 16 : mean <= 16 ? 32 : mean <= 48 ? 64 : mean <= 1024 ? 128 : 256;
 }
 
-int choose_split(int places, int experts, int N, int K, int mt) {
-  const int items = places / mt + (places < experts ? places : experts);
+int choose_split(int places, int experts, int N, int K, int mt, const Groups& g) {
+  const int items = (g.place_of ? 0 : places / mt) + (places < experts ? places : experts);
   const int tiles = (N + kTileN - 1) / kTileN * items;
   const int kblocks = (K + kBlockK - 1) / kBlockK;
   int split = 1;
@@ -22,15 +25,15 @@ int choose_split(int places, int experts, int N, int K, int mt) {
 }
 
 template <int EPI>
-int launch_grouped(const cacheir_b200_dense_args& p, const Groups& g, int x_rows, cudaStream_t st) {
-  const int mt = choose_tile(p.T, p.batch);
-  const int split = choose_split(p.T, p.batch, p.N, p.K, mt);
+int launch_grouped(const cacheir_b200_dense_args& p, const Groups& g, cudaStream_t st) {
+  const int mt = choose_tile(p.T, p.batch, g);
+  const int split = choose_split(p.T, p.batch, p.N, p.K, mt, g);
   switch (mt) {
-    case 16: return launch<EPI, 16, true>(p, split, st, g, x_rows);
-    case 32: return launch<EPI, 32, true>(p, split, st, g, x_rows);
-    case 64: return launch<EPI, 64, true>(p, split, st, g, x_rows);
-    case 128: return launch<EPI, 128, true>(p, split, st, g, x_rows);
-    default: return launch<EPI, 256, true>(p, split, st, g, x_rows);
+    case 16: return launch<EPI, 16, true>(p, split, st, g);
+    case 32: return launch<EPI, 32, true>(p, split, st, g);
+    case 64: return launch<EPI, 64, true>(p, split, st, g);
+    case 128: return launch<EPI, 128, true>(p, split, st, g);
+    default: return launch<EPI, 256, true>(p, split, st, g);
   }
 }
 
@@ -78,22 +81,25 @@ int tied_prompt_status(bool reset);
 
 using namespace cb200;
 
-extern "C" int cacheir_b200_grouped_gemm(const cacheir_b200_dense_args* args, const int32_t* cu, const int32_t* token_of, int x_rows,
+extern "C" int cacheir_b200_grouped_all_rows(void) { return kAllRows; }
+
+extern "C" int cacheir_b200_grouped_gemm(const cacheir_b200_dense_args* args, const int32_t* cu, const int32_t* place_of, int top, int x_rows,
                                          void* stream) {
   if (!args) return CACHEIR_B200_EINVAL;
   const cacheir_b200_dense_args& p = *args;
   if (p.T <= 0 || p.N <= 0) return 0;
-  if (p.batch < 1 || p.K <= 0 || !p.x || !p.w || !p.y || !cu || x_rows <= 0 || p.bias || p.tail_cols != 0 || p.w_batch_rows < p.N)
+  if (p.batch < 1 || p.K <= 0 || !p.x || !p.w || !p.y || !cu || x_rows <= 0 || p.bias || p.tail_cols != 0 || p.w_batch_rows < p.N ||
+      (place_of && top < 1))
     return CACHEIR_B200_EINVAL;
+  if (place_of && x_rows > kAllRows) return CACHEIR_B200_ELIMIT;
   if (p.w_stride % 8 != 0 || p.x_stride % 8 != 0 || !aligned_to(p.x, 16) || !aligned_to(p.w, 16)) return CACHEIR_B200_EALIGN;
   if (p.w_stride < p.K || p.x_stride < p.K) return CACHEIR_B200_EINVAL;
-  const Groups g{cu, token_of};
+  const Groups g{cu, place_of, top, x_rows};
   cudaStream_t st = as_stream(stream);
   switch (p.epilogue) {
-    case CACHEIR_B200_DENSE_BF16: return launch_grouped<CACHEIR_B200_DENSE_BF16>(p, g, x_rows, st);
-    case CACHEIR_B200_DENSE_SWIGLU: return p.N % 2 ? CACHEIR_B200_EINVAL : launch_grouped<CACHEIR_B200_DENSE_SWIGLU>(p, g, x_rows, st);
-    case CACHEIR_B200_DENSE_CLAMPED_GLU:
-      return p.N % 2 ? CACHEIR_B200_EINVAL : launch_grouped<CACHEIR_B200_DENSE_CLAMPED_GLU>(p, g, x_rows, st);
+    case CACHEIR_B200_DENSE_BF16: return launch_grouped<CACHEIR_B200_DENSE_BF16>(p, g, st);
+    case CACHEIR_B200_DENSE_SWIGLU: return p.N % 2 ? CACHEIR_B200_EINVAL : launch_grouped<CACHEIR_B200_DENSE_SWIGLU>(p, g, st);
+    case CACHEIR_B200_DENSE_CLAMPED_GLU: return p.N % 2 ? CACHEIR_B200_EINVAL : launch_grouped<CACHEIR_B200_DENSE_CLAMPED_GLU>(p, g, st);
     default: return CACHEIR_B200_EINVAL;
   }
 }

@@ -6,9 +6,10 @@
 
 namespace cb200 {
 
-// These families bound their logits against 32-bit arithmetic, so activations use the accurate expf / tanhf.
-__device__ __forceinline__ float sigmoid_exact(float z) { return 1.f / (1.f + expf(-z)); }
-__device__ __forceinline__ float silu_exact(float z) { return z / (1.f + expf(-z)); }
+// These families bound their logits against 32-bit arithmetic, so activations use the accurate expf / tanhf. The quotient
+// (2 ulp) has no slow path to branch to, so that a thread's many elements overlap; past the exponential's range it is 0.
+__device__ __forceinline__ float sigmoid_exact(float z) { return __fdividef(1.f, 1.f + expf(-z)); }
+__device__ __forceinline__ float silu_exact(float z) { return z * sigmoid_exact(z); }
 __device__ __forceinline__ float gelu_tanh(float z) {
   constexpr float kRoot2OverPi = 0.7978845608028654f;
   return 0.5f * z * (1.f + tanhf(kRoot2OverPi * fmaf(0.044715f * z * z, z, z)));

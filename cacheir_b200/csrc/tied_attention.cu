@@ -166,11 +166,10 @@ __device__ __forceinline__ void cluster_sync_all() {
   asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory");
 }
 
-// DB: 64-column boxes of the values
-template <int DB>
+// DB: 64-column boxes of the values; kSteps: 32-column pieces of a row that queries meet
+template <int DB, int kSteps>
 __global__ void __launch_bounds__(kStepThreads, DB <= 2 ? 2 : 1)
 tied_step_kernel(const __grid_constant__ CUtensorMap tmap, const StepParams p) {
-  constexpr int kSteps = 2 * DB + 1;             // 32-column pieces of a row that queries meet, at most
   constexpr int kTiles = DB * 8;                 // 8-column tiles of the output
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~static_cast<uintptr_t>(1023));
@@ -230,7 +229,7 @@ tied_step_kernel(const __grid_constant__ CUtensorMap tmap, const StepParams p) {
   } else {
     // ---------------- four warps, 16 keys of every page each ----------------
     const int width = a.dim + a.rot_dims, lead = tied_lead(a.rot_dims), qw = width - lead;
-    const int k_first = a.rot_dims / 32, k_steps = (width + 31) / 32 - k_first;
+    const int k_first = a.rot_dims / 32, last_piece = p.boxes * 2 - 1;      // (a piece behind the row meets zero queries: any data will do)
     uint32_t qa[kSteps][2][4];
     const __nv_bfloat16* qb = p.q + (static_cast<size_t>(seg) * a.heads + head0) * qw - lead;
 #pragma unroll
@@ -259,21 +258,29 @@ tied_step_kernel(const __grid_constant__ CUtensorMap tmap, const StepParams p) {
         __syncwarp();
       }
       const uint32_t rows = smem_addr(page) + warp * 16 * 128;
-      float sc[2][4];
+      // scores: both 8-key tiles side by side, even and odd pieces in sums of their own (shorter dependent chains)
+      float sc[2][4], sd[2][4];
 #pragma unroll
-      for (int nt = 0; nt < 2; ++nt) {
-        sc[nt][0] = sc[nt][1] = sc[nt][2] = sc[nt][3] = 0.f;
-        const uint32_t token = nt * 8 + lrow;
+      for (int nt = 0; nt < 2; ++nt)
 #pragma unroll
-        for (int k = 0; k < kSteps; ++k) {
-          if (k >= k_steps) break;
-          const uint32_t c = 4 * (k_first + k) + lmat;       // 16-byte piece of the row
-          uint32_t kb[4];
-          ldsm_x4(rows + (c >> 3) * kTiedBox + token * 128 + (((c & 7) ^ lrow) << 4), kb);
-          mma_bf16(sc[nt], qa[k][0], kb[0], kb[1]);
-          mma_bf16(sc[nt], qa[k][1], kb[2], kb[3]);
+        for (int e = 0; e < 4; ++e) sc[nt][e] = sd[nt][e] = 0.f;
+#pragma unroll
+      for (int k = 0; k < kSteps; ++k) {
+        const uint32_t c = 4 * min(k_first + k, last_piece) + lmat;        // 16-byte piece of the row
+        const uint32_t at = rows + (c >> 3) * kTiedBox + lrow * 128 + (((c & 7) ^ lrow) << 4);
+        uint32_t kb[2][4];
+        ldsm_x4(at, kb[0]);
+        ldsm_x4(at + 8 * 128, kb[1]);
+#pragma unroll
+        for (int nt = 0; nt < 2; ++nt) {
+          mma_bf16(sc[nt], qa[k][0], kb[nt][0], kb[nt][1]);
+          mma_bf16(sd[nt], qa[k][1], kb[nt][2], kb[nt][3]);
         }
       }
+#pragma unroll
+      for (int nt = 0; nt < 2; ++nt)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) sc[nt][e] += sd[nt][e];
       float pmax[2] = {-INFINITY, -INFINITY};
 #pragma unroll
       for (int nt = 0; nt < 2; ++nt) {
@@ -310,8 +317,7 @@ tied_step_kernel(const __grid_constant__ CUtensorMap tmap, const StepParams p) {
       }
 #pragma unroll
       for (int j = 0; j < kTiles / 2; ++j) {
-        if (j * 16 >= a.dim) break;
-        const uint32_t token = (lmat & 1) * 8 + lrow, c = 2 * j + (lmat >> 1);
+        const uint32_t token = (lmat & 1) * 8 + lrow, c = 2 * j + (lmat >> 1);       // (columns behind dim are computed and not kept)
         uint32_t vb[4];
         ldsm_x4_t(rows + (c >> 3) * kTiedBox + token * 128 + (((c & 7) ^ lrow) << 4), vb);
         mma_bf16(o[2 * j], pa, vb[0], vb[1]);
@@ -419,13 +425,13 @@ int step_stages(int dim, int rot) {
   return 0;
 }
 
-template <int DB>
+template <int DB, int kSteps>
 int launch_step(const StepParams& p, int segments, cudaStream_t st) {
   const cacheir_b200_tied_args& a = p.a;
   CUtensorMap map;
   if (!tied_encode(&map, a.pool, a.dim + a.rot_dims, static_cast<uint64_t>(a.num_slots) * a.kv_heads * kTiedPage)) return CACHEIR_B200_EUNSUPPORTED;
   const size_t smem = step_fixed(p.stages) + static_cast<size_t>(p.stages) * p.boxes * kTiedBox;
-  auto kern = tied_step_kernel<DB>;
+  auto kern = tied_step_kernel<DB, kSteps>;
   cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
   if (e != cudaSuccess) return static_cast<int>(e);
   cudaLaunchConfig_t cfg{};
@@ -526,10 +532,12 @@ extern "C" int cacheir_b200_tied_attention_step(const cacheir_b200_tied_args* ar
   p.splits = splits;
   p.boxes = step_boxes(a.dim, a.rot_dims);
   p.stages = step_stages(a.dim, a.rot_dims);
+  cudaStream_t st = as_stream(stream);
+  const bool odd = (a.dim + a.rot_dims + 31) / 32 - a.rot_dims / 32 > (a.dim + 63) / 64 * 2;
   switch ((a.dim + 63) / 64) {
-    case 1: return launch_step<1>(p, a.rows, as_stream(stream));
-    case 2: return launch_step<2>(p, a.rows, as_stream(stream));
-    case 3: return launch_step<3>(p, a.rows, as_stream(stream));
-    default: return launch_step<4>(p, a.rows, as_stream(stream));
+    case 1: return odd ? launch_step<1, 3>(p, a.rows, st) : launch_step<1, 2>(p, a.rows, st);
+    case 2: return odd ? launch_step<2, 5>(p, a.rows, st) : launch_step<2, 4>(p, a.rows, st);
+    case 3: return odd ? launch_step<3, 7>(p, a.rows, st) : launch_step<3, 6>(p, a.rows, st);
+    default: return odd ? launch_step<4, 9>(p, a.rows, st) : launch_step<4, 8>(p, a.rows, st);
   }
 }

@@ -10,7 +10,7 @@
 // Queries and keys have unit root mean square, so |score| <= bound is known before any key is read. While exp(-2 bound) is
 // far from underflow the softmax refers to the bound itself (FIXED): no running maximum, no rescaling. Otherwise a row's
 // reference follows its maximum, and O is rescaled when that has grown by more than 2^8. The bound also makes the capped
-// score a polynomial on a known interval: an odd one of eight terms, interpolated at Chebyshev nodes (POLY).
+// score a polynomial on a known interval: an odd one of five or eight terms, interpolated at Chebyshev nodes (TERMS).
 #include "ragged.cuh"
 #include "tied_attention.cuh"
 
@@ -22,7 +22,7 @@ __device__ int g_prompt_status = 0;
 constexpr int kThreads = 320;
 constexpr int kMaxStages = 6;
 constexpr int kTile = 128;
-constexpr int kTerms = 8;
+constexpr int kTerms = 8;                   // of the polynomial, at most
 constexpr float kStale = 8.f;
 
 struct PromptParams {
@@ -32,7 +32,7 @@ struct PromptParams {
   __nv_bfloat16* out;
   TiedScore score;
   float bound;                 // of |score| * log2 e
-  float pre;                   // POLY: raw product -> [-1, 1]
+  float pre;                   // with a polynomial: raw product -> [-1, 1]
   float coef[kTerms];          // score * log2 e = y (coef[0] + coef[1] y^2 + ...)
   int subs, heads_per_cta, tokens_per_tile;
   int boxes, lead_boxes, stages, k_first, k_end;     // 16-column pieces of a query row that the scores take
@@ -90,27 +90,31 @@ __device__ __forceinline__ void tmem_st_x16(uint32_t taddr, const float (&v)[16]
       "f"(v[11]), "f"(v[12]), "f"(v[13]), "f"(v[14]), "f"(v[15]) : "memory");
 }
 // pairs of float32 in one instruction
-__device__ __forceinline__ float2 mul2(float2 a, float2 b) {
-  float2 d;
-  asm("{\n\t.reg .b64 a, b, d;\n\tmov.b64 a, {%2, %3};\n\tmov.b64 b, {%4, %5};\n\tmul.rn.f32x2 d, a, b;\n\tmov.b64 {%0, %1}, d;\n\t}"
-      : "=f"(d.x), "=f"(d.y) : "f"(a.x), "f"(a.y), "f"(b.x), "f"(b.y));
+using f32x2 = unsigned long long;
+__device__ __forceinline__ f32x2 pair(float lo, float hi) {
+  f32x2 d;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(d) : "f"(lo), "f"(hi));
   return d;
 }
-__device__ __forceinline__ float2 add2(float2 a, float2 b) {
-  float2 d;
-  asm("{\n\t.reg .b64 a, b, d;\n\tmov.b64 a, {%2, %3};\n\tmov.b64 b, {%4, %5};\n\tadd.rn.f32x2 d, a, b;\n\tmov.b64 {%0, %1}, d;\n\t}"
-      : "=f"(d.x), "=f"(d.y) : "f"(a.x), "f"(a.y), "f"(b.x), "f"(b.y));
+__device__ __forceinline__ void unpair(f32x2 a, float& lo, float& hi) { asm("mov.b64 {%0, %1}, %2;" : "=f"(lo), "=f"(hi) : "l"(a)); }
+__device__ __forceinline__ f32x2 mul2(f32x2 a, f32x2 b) {
+  f32x2 d;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
   return d;
 }
-__device__ __forceinline__ float2 fma2(float2 a, float2 b, float2 c) {
-  float2 d;
-  asm("{\n\t.reg .b64 a, b, c, d;\n\tmov.b64 a, {%2, %3};\n\tmov.b64 b, {%4, %5};\n\tmov.b64 c, {%6, %7};\n\t"
-      "fma.rn.f32x2 d, a, b, c;\n\tmov.b64 {%0, %1}, d;\n\t}"
-      : "=f"(d.x), "=f"(d.y) : "f"(a.x), "f"(a.y), "f"(b.x), "f"(b.y), "f"(c.x), "f"(c.y));
+__device__ __forceinline__ f32x2 add2(f32x2 a, f32x2 b) {
+  f32x2 d;
+  asm("add.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+  return d;
+}
+__device__ __forceinline__ f32x2 fma2(f32x2 a, f32x2 b, f32x2 c) {
+  f32x2 d;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
   return d;
 }
 
-template <int TILES, bool FIXED, bool POLY>
+// TERMS: of the polynomial, 0: the formula
+template <int TILES, bool FIXED, int TERMS>
 __global__ void __launch_bounds__(kThreads, 1)
 tied_prompt_kernel(const __grid_constant__ CUtensorMap tmap_kv, const __grid_constant__ CUtensorMap tmap_q, const PromptParams p) {
   extern __shared__ uint8_t smem_raw[];
@@ -249,7 +253,11 @@ tied_prompt_kernel(const __grid_constant__ CUtensorMap tmap_kv, const __grid_con
     const int tile_pos = pos0 + t * p.tokens_per_tile, rp = real ? tile_pos + tok : -1;
     const float sink = (a.sink && real) ? a.sink[head0 + h] * kLog2e : -1e30f;
     float m_ref = FIXED ? fmaxf(p.bound, sink) : sink;
-    float2 l2 = make_float2(a.sink && real ? tied_ex2(sink - m_ref) : 0.f, 0.f);
+    f32x2 l2 = pair(a.sink && real ? tied_ex2(sink - m_ref) : 0.f, 0.f);
+    f32x2 coef[TERMS > 0 ? TERMS : 1];
+#pragma unroll
+    for (int k = 0; k < TERMS; ++k) coef[k] = pair(p.coef[k], p.coef[k]);
+    const f32x2 pre = pair(p.pre, p.pre), minus_ref = pair(-m_ref, -m_ref);
     const uint32_t lanes = static_cast<uint32_t>((warp & 3) * 32) << 16;
     uint8_t* p_row = s_p + t * kTile * 128 + r * 128;
     for (int it = 0; it < n; ++it) {
@@ -266,28 +274,42 @@ tied_prompt_kernel(const __grid_constant__ CUtensorMap tmap_kv, const __grid_con
       for (int i = 0; i < kTiedPage; ++i) asm volatile("" : "+f"(v[i]));      // (the values exist from here on)
       ptx::tc_fence_before();
       ptx::mbar_arrive(smem_addr(&bar_free[t]));
-      // scores * log2 e; FIXED: minus the reference
+      // scores * log2 e; FIXED: minus the reference. Eight pairs side by side, so that their chains overlap.
       const float4* inv4 = reinterpret_cast<const float4*>(s_inv + s * kTiedPage);
 #pragma unroll
-      for (int i = 0; i < kTiedPage; i += 4) {
-        const float4 f = inv4[i / 4];
+      for (int i0 = 0; i0 < kTiedPage; i0 += 16) {
+        f32x2 u[8], c[8];
 #pragma unroll
-        for (int e = 0; e < 4; e += 2) {
-          float2 u = mul2(make_float2(v[i + e], v[i + e + 1]), e == 0 ? make_float2(f.x, f.y) : make_float2(f.z, f.w));
-          if constexpr (POLY) {
-            u = mul2(u, make_float2(p.pre, p.pre));
-            const float2 w = mul2(u, u);
-            float2 c = make_float2(p.coef[kTerms - 1], p.coef[kTerms - 1]);
-#pragma unroll
-            for (int k = kTerms - 2; k >= 0; --k) c = fma2(c, w, make_float2(p.coef[k], p.coef[k]));
-            u = FIXED ? fma2(c, u, make_float2(-m_ref, -m_ref)) : mul2(c, u);
-          } else {
-            u = make_float2(p.score(u.x), p.score(u.y));
-            if (FIXED) u = add2(u, make_float2(-m_ref, -m_ref));
-          }
-          v[i + e] = u.x;
-          v[i + e + 1] = u.y;
+        for (int j = 0; j < 8; j += 2) {
+          const float4 f = inv4[(i0 + 2 * j) / 4];
+          u[j] = mul2(pair(v[i0 + 2 * j], v[i0 + 2 * j + 1]), pair(f.x, f.y));
+          u[j + 1] = mul2(pair(v[i0 + 2 * j + 2], v[i0 + 2 * j + 3]), pair(f.z, f.w));
         }
+        if constexpr (TERMS > 0) {
+          f32x2 w[8];
+#pragma unroll
+          for (int j = 0; j < 8; ++j) u[j] = mul2(u[j], pre);
+#pragma unroll
+          for (int j = 0; j < 8; ++j) w[j] = mul2(u[j], u[j]);
+#pragma unroll
+          for (int j = 0; j < 8; ++j) c[j] = fma2(coef[TERMS - 1], w[j], coef[TERMS - 2]);
+#pragma unroll
+          for (int k = TERMS - 3; k >= 0; --k)
+#pragma unroll
+            for (int j = 0; j < 8; ++j) c[j] = fma2(c[j], w[j], coef[k]);
+#pragma unroll
+          for (int j = 0; j < 8; ++j) c[j] = FIXED ? fma2(c[j], u[j], minus_ref) : mul2(c[j], u[j]);
+        } else {
+#pragma unroll
+          for (int j = 0; j < 8; ++j) {
+            float x, y;
+            unpair(u[j], x, y);
+            c[j] = pair(p.score(x), p.score(y));
+            if (FIXED) c[j] = add2(c[j], minus_ref);
+          }
+        }
+#pragma unroll
+        for (int j = 0; j < 8; ++j) unpair(c[j], v[i0 + 2 * j], v[i0 + 2 * j + 1]);
       }
       // (rows without a token may hold anything: a row of P reaches its own row of O only, which is not stored)
       if (!(base + kTiedPage - 1 <= tile_pos && (base > tile_pos + count - 1 - a.window || base + kTiedPage <= a.keep_first))) {
@@ -307,15 +329,14 @@ tied_prompt_kernel(const __grid_constant__ CUtensorMap tmap_kv, const __grid_con
         }
 #pragma unroll
         for (int i = 0; i < kTiedPage; ++i) v[i] -= m_ref;
-        l2.x *= alpha;
-        l2.y *= alpha;
+        l2 = mul2(l2, pair(alpha, alpha));
       }
       uint32_t packed[kTiedPage / 2];
 #pragma unroll
       for (int i = 0; i < kTiedPage; i += 2) {
-        const float2 e = make_float2(tied_ex2(v[i]), tied_ex2(v[i + 1]));
-        l2 = add2(l2, e);
-        packed[i / 2] = pack_bf16(e.x, e.y);
+        const float x = tied_ex2(v[i]), y = tied_ex2(v[i + 1]);
+        l2 = add2(l2, pair(x, y));
+        packed[i / 2] = pack_bf16(x, y);
       }
       if (it > 0) ok = ok && ptx::mbar_wait(smem_addr(&bar_o[t]), (it - 1) & 1, &g_prompt_status, (9 << 8) | 10);
       if constexpr (!FIXED) {
@@ -344,28 +365,34 @@ tied_prompt_kernel(const __grid_constant__ CUtensorMap tmap_kv, const __grid_con
       ptx::tc_fence_before();
       ptx::mbar_arrive(smem_addr(&bar_p[t]));
     }
-    ok = ok && ptx::mbar_wait(smem_addr(&bar_o[t]), (n - 1) & 1, &g_prompt_status, (9 << 8) | 11);
-    __syncwarp();
-    ptx::tc_fence_after();
-    const float inv = 1.f / (l2.x + l2.y);
     const size_t row = first + tok, col0 = static_cast<size_t>(head0 + h) * a.dim;
-    for (int c = 0; c < p.n_cols; c += 16) {
-      float o[16];
-      tmem_ld_x16(tmem + t * p.n_cols + c + lanes, o);
-      if (!real) continue;
+    float l, l_odd;
+    unpair(l2, l, l_odd);
+    const float inv = 1.f / (l + l_odd);
+    for (int c0 = 0; c0 < p.n_cols; c0 += 128) {
+      uint4 g[16];                           // the gates travel while the last MMAs run
 #pragma unroll
-      for (int j = 0; j < 16; j += 8) {
-        if (c + j >= a.dim) break;
-        float y[8];
+      for (int i = 0; i < 16; ++i)
+        g[i] = p.gate && real && c0 + 8 * i < a.dim ? *reinterpret_cast<const uint4*>(p.gate + row * p.gate_stride + col0 + c0 + 8 * i) : make_uint4(0u, 0u, 0u, 0u);
+      if (c0 == 0) ok = ok && ptx::mbar_wait(smem_addr(&bar_o[t]), (n - 1) & 1, &g_prompt_status, (9 << 8) | 11);
+      __syncwarp();
+      ptx::tc_fence_after();
 #pragma unroll
-        for (int e = 0; e < 8; ++e) y[e] = o[j + e] * inv;
-        if (p.gate) {
-          float g[8];
-          VecIO<__nv_bfloat16, 8>::ld(p.gate + row * p.gate_stride + col0 + c + j, g);
+      for (int c = 0; c < 128; c += 16) {
+        if (c0 + c >= p.n_cols) break;
+        float o[16];
+        tmem_ld_x16(tmem + t * p.n_cols + c0 + c + lanes, o);
 #pragma unroll
-          for (int e = 0; e < 8; ++e) y[e] *= sigmoid_exact(g[e]);
+        for (int j = 0; j < 16; j += 8) {
+          const uint32_t bits[4] = {g[(c + j) / 8].x, g[(c + j) / 8].y, g[(c + j) / 8].z, g[(c + j) / 8].w};
+          float y[8];
+#pragma unroll
+          for (int e = 0; e < 8; ++e) {
+            const float gate = __uint_as_float(e & 1 ? bits[e / 2] & 0xffff0000u : bits[e / 2] << 16);
+            y[e] = o[j + e] * inv * (p.gate ? sigmoid_exact(gate) : 1.f);
+          }
+          if (real && c0 + c + j < a.dim) VecIO<__nv_bfloat16, 8>::st(p.out + row * a.heads * a.dim + col0 + c0 + c + j, y);
         }
-        VecIO<__nv_bfloat16, 8>::st(p.out + row * a.heads * a.dim + col0 + c + j, y);
       }
     }
     __syncwarp();
@@ -392,29 +419,30 @@ int prompt_stages(int dim, int rot) {
 }
 
 // Odd polynomial for cap2 * tanh(reach * y) on [-1, 1]: y times the interpolant, at the Chebyshev nodes of [0, 1], of the
-// even quotient as a function of y^2. Double precision; returns false where eight terms are not enough (the quotient's
-// poles lie at y^2 = -(pi / 2 reach)^2).
-bool fit_tanh(double cap2, double reach, float (&coef)[kTerms]) {
-  if (!(reach > 0.0) || reach > 1.25) return false;
+// even quotient as a function of y^2. Double precision. Returns the number of terms: the quotient's poles lie at
+// y^2 = -(pi / 2 reach)^2, which puts the error near 2^-21 of cap2 or below; 0 where eight are not enough.
+int fit_tanh(double cap2, double reach, float (&coef)[kTerms]) {
+  if (!(reach > 0.0) || reach > 1.25) return 0;
+  const int terms = reach <= 0.7 ? 5 : 8;
   const double pi = 3.14159265358979323846;
   double node[kTerms], table[kTerms];
-  for (int i = 0; i < kTerms; ++i) {
-    node[i] = 0.5 + 0.5 * cos((2 * i + 1) * pi / (2 * kTerms));
+  for (int i = 0; i < terms; ++i) {
+    node[i] = 0.5 + 0.5 * cos((2 * i + 1) * pi / (2 * terms));
     const double y = sqrt(node[i]);
     table[i] = cap2 * tanh(reach * y) / y;
   }
-  for (int k = 1; k < kTerms; ++k)                      // divided differences
-    for (int i = kTerms - 1; i >= k; --i) table[i] = (table[i] - table[i - 1]) / (node[i] - node[i - k]);
+  for (int k = 1; k < terms; ++k)                       // divided differences
+    for (int i = terms - 1; i >= k; --i) table[i] = (table[i] - table[i - 1]) / (node[i] - node[i - k]);
   double c[kTerms] = {};
-  for (int k = kTerms - 1; k >= 0; --k) {               // Newton form -> powers
-    for (int i = kTerms - 1; i > 0; --i) c[i] = c[i - 1] - node[k] * c[i];
+  for (int k = terms - 1; k >= 0; --k) {                // Newton form -> powers
+    for (int i = terms - 1; i > 0; --i) c[i] = c[i - 1] - node[k] * c[i];
     c[0] = table[k] - node[k] * c[0];
   }
-  for (int i = 0; i < kTerms; ++i) coef[i] = static_cast<float>(c[i]);
-  return true;
+  for (int i = 0; i < terms; ++i) coef[i] = static_cast<float>(c[i]);
+  return terms;
 }
 
-template <int TILES, bool FIXED, bool POLY>
+template <int TILES, bool FIXED, int TERMS>
 int launch_prompt(const PromptParams& p, const void* q, int items, cudaStream_t st) {
   const cacheir_b200_tied_args& a = p.a;
   size_t smem = prompt_fixed(a.dim, a.rot_dims) + static_cast<size_t>(p.stages) * p.boxes * kTiedBox;
@@ -431,7 +459,7 @@ int launch_prompt(const PromptParams& p, const void* q, int items, cudaStream_t 
   if (fn(&tq, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(q), dims, strides, box, elem_strides, CU_TENSOR_MAP_INTERLEAVE_NONE,
          CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) != CUDA_SUCCESS)
     return CACHEIR_B200_EUNSUPPORTED;
-  auto kern = tied_prompt_kernel<TILES, FIXED, POLY>;
+  auto kern = tied_prompt_kernel<TILES, FIXED, TERMS>;
   cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
   if (e != cudaSuccess) return static_cast<int>(e);
   kern<<<dim3(a.kv_heads * p.subs, items), kThreads, smem, st>>>(tkv, tq, p);
@@ -439,10 +467,11 @@ int launch_prompt(const PromptParams& p, const void* q, int items, cudaStream_t 
 }
 
 template <int TILES>
-int launch_tiles(const PromptParams& p, bool fixed, bool poly, const void* q, int items, cudaStream_t st) {
-  if (fixed && poly) return launch_prompt<TILES, true, true>(p, q, items, st);
-  if (fixed) return launch_prompt<TILES, true, false>(p, q, items, st);
-  return launch_prompt<TILES, false, false>(p, q, items, st);
+int launch_tiles(const PromptParams& p, bool fixed, int terms, const void* q, int items, cudaStream_t st) {
+  if (fixed && terms == 5) return launch_prompt<TILES, true, 5>(p, q, items, st);
+  if (fixed && terms == 8) return launch_prompt<TILES, true, 8>(p, q, items, st);
+  if (fixed) return launch_prompt<TILES, true, 0>(p, q, items, st);
+  return launch_prompt<TILES, false, 0>(p, q, items, st);
 }
 
 }  // namespace
@@ -479,10 +508,10 @@ extern "C" int cacheir_b200_tied_attention_prompt(const cacheir_b200_tied_args* 
   const double bound = a.cap > 0.f ? a.cap * tanh(reach / a.cap) : reach;
   p.bound = static_cast<float>(bound * kLog2e);
   const bool fixed = 2.0 * bound * kLog2e <= 100.0;
-  bool poly = false;
+  int terms = 0;
   if (a.cap > 0.f) {
     p.pre = static_cast<float>((a.scale < 0.f ? -1.0 : 1.0) / most);
-    poly = fit_tanh(static_cast<double>(a.cap) * kLog2e, reach / a.cap, p.coef);
+    terms = fit_tanh(static_cast<double>(a.cap) * kLog2e, reach / a.cap, p.coef);
   }
   const int group = a.heads / a.kv_heads, tiles = prompt_tiles(a.dim);
   p.subs = (group + kTile - 1) / kTile;
@@ -498,5 +527,5 @@ extern "C" int cacheir_b200_tied_attention_prompt(const cacheir_b200_tied_args* 
   p.tmem_cols = cols <= 128 ? 128 : cols <= 256 ? 256 : 512;
   const int items = ragged_items(a.rows, a.segments, tiles * p.tokens_per_tile);
   if (items > 65535) return CACHEIR_B200_ELIMIT;
-  return tiles == 2 ? launch_tiles<2>(p, fixed, poly, q, items, as_stream(stream)) : launch_tiles<1>(p, fixed, poly, q, items, as_stream(stream));
+  return tiles == 2 ? launch_tiles<2>(p, fixed, terms, q, items, as_stream(stream)) : launch_tiles<1>(p, fixed, terms, q, items, as_stream(stream));
 }

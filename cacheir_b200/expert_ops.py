@@ -104,36 +104,47 @@ class Routing:
         return int(self.token_of.numel())
 
 
-def route(logits: torch.Tensor, row_seg: torch.Tensor, routing: Routing, scale: float) -> None:
+def route(logits: torch.Tensor, row_seg: torch.Tensor, routing: Routing, scale: float, x: torch.Tensor | None = None,
+          placed: torch.Tensor | None = None) -> None:
+    """Choices and places; with `placed` [rows * top, width] also a copy of every row of `x` at its places."""
     _require_cuda(logits, row_seg, routing.counters)
     rows = int(logits.shape[0])
     if logits.dtype != torch.float32 or logits.stride(1) != 1 or tuple(routing.place_of.shape) != (rows, routing.top):
         raise ValueError("route takes float32 logits with dense rows and a routing of their row count")
+    if placed is not None and (x is None or not x.is_contiguous() or not placed.is_contiguous() or x.dtype != placed.dtype
+                               or int(x.shape[0]) != rows or tuple(placed.shape) != (routing.places, int(x.shape[1]))):
+        raise ValueError("placed has a row per place, x one per logits row, both dense")
     check(_lib.load_group("experts").cacheir_b200_route(
         logits.data_ptr(), logits.stride(0), row_seg.data_ptr(), rows, routing.experts, routing.top, float(scale), routing.counters.data_ptr(),
         routing.cu.data_ptr(), routing.token_of.data_ptr(), routing.place_of.data_ptr(), routing.weight.data_ptr(),
-        routing.chosen.data_ptr(), _stream()), "route")
+        routing.chosen.data_ptr(), None if placed is None else x.data_ptr(), _ptr(placed),
+        0 if placed is None else int(x.shape[1]) * x.element_size(), _stream()), "route")
 
 
 def grouped_supported(k: int, x_stride: int, dtype: torch.dtype) -> bool:
     return dtype == torch.bfloat16 and k % 8 == 0 and x_stride % 8 == 0
 
 
-def grouped_gemm(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, routing: Routing, *, gather: bool, epilogue: int = DENSE_PLAIN,
+def grouped_all_rows() -> int:
+    """Rows of a step up to which an expert multiplies all of them and keeps those that chose it."""
+    return int(_lib.load_group("experts").cacheir_b200_grouped_all_rows())
+
+
+def grouped_gemm(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, routing: Routing, *, by_row: bool, epilogue: int = DENSE_PLAIN,
                  limit: float = 0.0) -> torch.Tensor:
-    """out[place] = f(x[row] W_e^T), w [experts*N, K]; row = the place's token when `gather`, else the place."""
+    """out[place] = f(x[.] W_e^T), w [experts*N, K]; x has a row per token (`by_row`, see grouped_all_rows) or per place."""
     _require_cuda(x, w, out)
     n = int(w.shape[0]) // routing.experts
     cols = n // 2 if epilogue in (DENSE_SWIGLU, DENSE_CLAMPED_GLU) else n
     if x.dtype != torch.bfloat16 or w.dtype != torch.bfloat16 or x.stride(1) != 1 or w.stride(1) != 1 or out.dtype != torch.bfloat16:
         raise ValueError("grouped_gemm takes bf16 operands with dense rows")
-    if int(out.shape[0]) != routing.places or int(out.shape[1]) < cols or out.stride(1) != 1 or (not gather and int(x.shape[0]) < routing.places):
-        raise ValueError("out must have a row per place")
+    if int(out.shape[0]) != routing.places or int(out.shape[1]) < cols or out.stride(1) != 1 or int(x.shape[0]) != (routing.places // routing.top if by_row else routing.places):
+        raise ValueError("out must have a row per place, x one per place or token")
     a = DenseArgs()
     a.x, a.w, a.y, a.T, a.N, a.K, a.batch, a.w_batch_rows = x.data_ptr(), w.data_ptr(), out.data_ptr(), routing.places, n, int(w.shape[1]), routing.experts, n
     a.epilogue, a.w_stride, a.x_stride, a.y_stride, a.limit = epilogue, w.stride(0), x.stride(0), out.stride(0), float(limit)
     check(_lib.load_group("experts").cacheir_b200_grouped_gemm(
-        ctypes.byref(a), routing.cu.data_ptr(), routing.token_of.data_ptr() if gather else None, int(x.shape[0]), _stream()), "grouped_gemm")
+        ctypes.byref(a), routing.cu.data_ptr(), routing.place_of.data_ptr() if by_row else None, routing.top, int(x.shape[0]), _stream()), "grouped_gemm")
     return out
 
 

@@ -196,11 +196,11 @@ def make_plan_class(base: type) -> type:
             self.logits = logits
             self.feedback_tail = lambda: ops.argmax_rows(logits, self.ids)
 
-        def _dense(self, x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, bias: torch.Tensor | None = None) -> None:
+        def _dense(self, x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, bias: torch.Tensor | None = None, label: str = "") -> None:
             """Plain product into `out` (float32 for logits): tensor cores where they take it, else CUDA cores."""
             if H.dense_supported(int(w.shape[1]), w.stride(0), x.stride(0), dtype=x.dtype):
                 epilogue = H.DENSE_F32 if out.dtype == torch.float32 else H.DENSE_PLAIN
-                self._emit(lambda: H.dense_gemm(x, w, out, epilogue=epilogue, bias=bias), "b200.dense_gemm")
+                self._emit(lambda: H.dense_gemm(x, w, out, epilogue=epilogue, bias=bias), "b200.dense_gemm" + label)
             else:
                 self._emit(lambda: H.dense_simple(x, w, out, bias=bias), "b200.dense_simple")
 
@@ -323,7 +323,7 @@ def make_plan_class(base: type) -> type:
             else:
                 out = self._scratch("sublayer", int(w.shape[0]))      # (a shared expert's lives until the combine)
             bias = node.attrs.get("bias")
-            self._dense(x, w, out, None if bias is None else eng.weights.get_f32(bias))
+            self._dense(x, w, out, None if bias is None else eng.weights.get_f32(bias), "." + str(node.attrs["projection"]))
             self._env[node.outputs[0]] = out
 
         def _lower_residual_dynamic_tanh(self, idx: int, node: Any) -> None:
@@ -423,11 +423,15 @@ def make_plan_class(base: type) -> type:
                                 cu=self._scratch("route_cu", experts + 1, i32, rows=1).view(-1), token_of=self._scratch("route_token", top, i32).view(-1),
                                 place_of=self._scratch("route_place", top, i32), chosen=self._scratch("route_chosen", top, i32),
                                 weight=self._scratch("route_weight", top, torch.float32))
-            self._emit(lambda: X.route(logits, self.rows.row_seg, routing, scale), "b200.route")
-            self._env[node.outputs[0]] = routing
+            placed = None
+            if self.batch > X.grouped_all_rows() and X.grouped_supported(width, x.stride(0), eng.dtype):
+                placed = self._scratch("placed", width, rows=routing.places)       # the experts' products read rows in expert order
+            self._emit(lambda: X.route(logits, self.rows.row_seg, routing, scale, x, placed), "b200.route", launches=1 if placed is None else 2)
+            self._env[node.outputs[0]] = (routing, placed)
 
         def _lower_expert_mixture(self, idx: int, node: Any) -> None:
-            eng, x, routing = self.engine, self._input(node.inputs[0]), self._env[node.inputs[1]]
+            eng, x = self.engine, self._input(node.inputs[0])
+            routing, placed = self._env[node.inputs[1]]
             n = int(node.attrs["experts"])
             gates, ups, downs = (tuple(node.inputs[2 + i * n:2 + (i + 1) * n]) for i in range(3))
             w_in, w_out = eng.expert_pairs(gates, ups), eng.concat_weight(downs)
@@ -437,8 +441,10 @@ def make_plan_class(base: type) -> type:
             out = self._scratch("expert_out", width, rows=places)
             if X.grouped_supported(int(w_in.shape[1]), x.stride(0), eng.dtype) and X.grouped_supported(ff, ff, eng.dtype):
                 hidden = self._scratch("expert_hidden", ff, rows=places)
-                self._emit(lambda: X.grouped_gemm(x, w_in, hidden, routing, gather=True, epilogue=kind, limit=limit), "b200.grouped_gemm.clamped_glu")
-                self._emit(lambda: X.grouped_gemm(hidden, w_out, out, routing, gather=False), "b200.grouped_gemm")
+                source = x if placed is None else placed
+                self._emit(lambda: X.grouped_gemm(source, w_in, hidden, routing, by_row=placed is None, epilogue=kind, limit=limit),
+                           "b200.grouped_gemm.clamped_glu")
+                self._emit(lambda: X.grouped_gemm(hidden, w_out, out, routing, by_row=False), "b200.grouped_gemm")
             else:
                 both, hidden = self._scratch("expert_gate_up", 2 * ff, rows=places), self._scratch("expert_hidden", ff, rows=places)
                 self._emit(lambda: X.grouped_simple(x, w_in, both, routing, gather=True), "b200.grouped_simple")
@@ -447,7 +453,7 @@ def make_plan_class(base: type) -> type:
             self._env[node.outputs[0]] = out
 
         def _lower_combine_residual_rms_norm(self, idx: int, node: Any) -> None:
-            y, routing, res = self._env[node.inputs[1]], self._env[node.inputs[2]], self._residual
+            y, (routing, _), res = self._env[node.inputs[1]], self._env[node.inputs[2]], self._residual
             w, eps = self.engine.weights.get_f32(node.inputs[3]), float(node.attrs["eps"])
             shared = self._env[node.inputs[4]] if len(node.inputs) > 4 else None
             self._finish_residual(idx, lambda nx: self._emit(lambda: X.combine_residual_rms(res, y, routing, shared, w, eps, nx),

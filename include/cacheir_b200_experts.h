@@ -58,16 +58,18 @@ int cacheir_b200_tied_attention_step(const cacheir_b200_tied_args* a, const void
 /* ---- mixtures of experts ----------------------------------------------------------------------------------------------
  * route: per row of logits [rows, stride] the `top` experts with the largest values (lower index first among equals),
  * weight = sigmoid(logit) * scale. The rows x top choices get places 0.. in expert order:
- *   cu [experts + 1] first place of every expert; token_of [rows*top] row of a place; place_of, weight [rows, top].
- *   chosen [rows, top] the experts
- * Rows with row_seg < 0 choose nothing (place_of = -1). `counters`: experts + 1 zeroed ints, left zeroed. */
+ *   cu [experts + 1] first place of every expert; token_of [rows*top] row of a place; place_of, weight, chosen [rows, top]
+ * Rows with row_seg < 0 choose nothing (place_of = -1). `counters`: experts + 1 zeroed ints, left zeroed. With `placed`
+ * [rows*top, row_bytes] every row of x [rows, row_bytes] is also copied to its places (multiples of 16 bytes). */
 int cacheir_b200_route(const float* logits, long long stride, const int32_t* row_seg, int rows, int experts, int top, float scale,
-                       int32_t* counters, int32_t* cu, int32_t* token_of, int32_t* place_of, float* weight, int32_t* chosen, void* stream);
-/* Y[place] = f(X[row] W_e^T) for the places of every expert e, whose W rows start at e*w_batch_rows; row = token_of[place],
- * or the place itself when token_of is NULL. a->T places at most, a->batch experts, a->x has x_rows rows. Epilogues:
- * BF16, SWIGLU, CLAMPED_GLU. Strides must be multiples of 8 elements. */
-int cacheir_b200_grouped_gemm(const cacheir_b200_dense_args* a, const int32_t* cu, const int32_t* token_of, int x_rows, void* stream);
-/* The same product without its epilogue in float32 arithmetic, any extents. */
+                       int32_t* counters, int32_t* cu, int32_t* token_of, int32_t* place_of, float* weight, int32_t* chosen,
+                       const void* x, void* placed, int row_bytes, void* stream);
+/* Y[place] = f(X[.] W_e^T) for the places of every expert e, whose W rows start at e*w_batch_rows. X rows are places; with
+ * place_of [x_rows, top] they are the step's rows (at most cacheir_b200_grouped_all_rows() of them). a->T places at most,
+ * a->batch experts. Epilogues: BF16, SWIGLU, CLAMPED_GLU. Strides must be multiples of 8 elements. */
+int cacheir_b200_grouped_all_rows(void);
+int cacheir_b200_grouped_gemm(const cacheir_b200_dense_args* a, const int32_t* cu, const int32_t* place_of, int top, int x_rows, void* stream);
+/* The same product without its epilogue in float32 arithmetic, any extents; X rows are places, or token_of[place]. */
 int cacheir_b200_grouped_simple(const void* x, const void* w, void* y, const int32_t* cu, const int32_t* token_of, int places, int experts,
                                 int N, int K, long long w_stride, long long x_stride, long long y_stride, int dtype, void* stream);
 /* m = sum_k weight[t, k] * y[place_of[t, k]] + shared[t] (shared may be NULL); residual += m / sqrt(mean(m^2) + eps) * w,

@@ -89,7 +89,7 @@ def _routing(rows, experts, top, counters=None):
                      torch.empty((rows, top), device="cuda"))
 
 
-def _route(rng, rows, experts, top, padding=0, scale=2.5):
+def _route(rng, rows, experts, top, padding=0, scale=2.5, x=None, placed=None):
     from cacheir_b200 import expert_ops as X
 
     z, zn = _rand(rng, rows, experts + 3, dtype=torch.float32)
@@ -97,14 +97,17 @@ def _route(rng, rows, experts, top, padding=0, scale=2.5):
     if padding:
         seg[rows - padding:] = -1
     routing = _routing(rows, experts, top)
-    X.route(z[:, :experts], seg, routing, scale)
+    X.route(z[:, :experts], seg, routing, scale, x, placed)
     return routing, zn[:, :experts]
 
 
+@pytest.mark.parametrize("copies", [False, True])
 @pytest.mark.parametrize("rows,experts,top,padding", [(1, 1, 1, 0), (3, 5, 2, 1), (9, 300, 9, 0), (700, 16, 4, 100), (33, 8, 8, 2), (16, 64, 1, 16)])
-def test_route(rows, experts, top, padding):
+def test_route(rows, experts, top, padding, copies):
     rng = np.random.default_rng(rows)
-    routing, z = _route(rng, rows, experts, top, padding)
+    x, xn = _rand(rng, rows, 72)
+    placed = torch.full((rows * top, 72), 9.0, device="cuda", dtype=torch.bfloat16) if copies else None
+    routing, z = _route(rng, rows, experts, top, padding, x=x, placed=placed)
     real = rows - padding
     chosen, weight = O.route(z[:real], top, 2.5)
     assert np.array_equal(routing.chosen.cpu().numpy()[:real], chosen)
@@ -117,6 +120,9 @@ def test_route(rows, experts, top, padding):
             e = chosen[t, k]
             assert cu[e] <= place[t, k] < cu[e + 1] and token[place[t, k]] == t
     assert int(routing.counters.abs().max()) == 0
+    if copies:
+        got = placed.double().cpu().numpy()
+        assert np.array_equal(got[:real * top], xn[token[:real * top]]) and (got[real * top:] == 9.0).all()
 
 
 def test_equal_logits_go_to_the_lower_index():
@@ -129,33 +135,34 @@ def test_equal_logits_go_to_the_lower_index():
 
 
 @pytest.mark.parametrize("rows,experts,top,n,k", [(1, 4, 2, 16, 8), (5, 3, 2, 136, 72), (40, 7, 3, 64, 264), (300, 5, 2, 256, 128), (600, 9, 4, 40, 64),
-                                                  (900, 2, 2, 24, 512), (64, 40, 8, 520, 96)])
+                                                  (900, 2, 2, 24, 512), (64, 40, 8, 520, 96), (17, 6, 6, 128, 1024), (65, 3, 1, 200, 136), (2300, 2, 2, 72, 64)])
 def test_grouped_products(rows, experts, top, n, k):
     from cacheir_b200 import expert_ops as X
     from cacheir_b200 import hybrid_ops as H
 
     rng = np.random.default_rng(rows + n)
-    routing, _ = _route(rng, rows, experts, top, padding=rows // 5)
+    x, xn = _rand(rng, rows, k)
+    placed = torch.zeros((rows * top, k), device="cuda", dtype=torch.bfloat16)
+    routing, _ = _route(rng, rows, experts, top, padding=rows // 5, x=x, placed=placed)
     cu, token = routing.cu.cpu().numpy(), routing.token_of.cpu().numpy()
     used = cu[-1]
-    x, xn = _rand(rng, rows, k)
     w, wn = _rand(rng, experts * n, k, scale=1.5 * k ** -0.5)
     expert = np.searchsorted(cu, np.arange(used), side="right") - 1
 
     def product(values):
         return np.stack([wn[e * n:(e + 1) * n] @ v for e, v in zip(expert, values)])
     y = product(xn[token[:used]])
-    out = torch.full((routing.places, n), 3.0, device="cuda", dtype=torch.bfloat16)
-    X.grouped_gemm(x, w, out, routing, gather=True)
-    _close(out[:used], y, 5e-3)
-    assert float((out[used:] - 3).abs().max() if used < routing.places else 0) == 0.0
-    half = torch.empty((routing.places, n // 2), device="cuda", dtype=torch.bfloat16)
-    X.grouped_gemm(x, w, half, routing, gather=True, epilogue=H.DENSE_CLAMPED_GLU, limit=0.8)
-    g, u = np.minimum(y[:, 0::2], 0.8), np.clip(y[:, 1::2], -0.8, 0.8)
-    _close(half[:used], g * O.sigmoid(1.702 * g) * (u + 1), 6e-3)
-    placed, pn = _rand(rng, routing.places, k)
-    X.grouped_gemm(placed, w, out, routing, gather=False)
-    _close(out[:used], product(pn[:used]), 5e-3)
+    for source, by_row in [(placed, False)] + ([(x, True)] if rows <= X.grouped_all_rows() else []):
+        out = torch.full((routing.places, n), 3.0, device="cuda", dtype=torch.bfloat16)
+        X.grouped_gemm(source, w, out, routing, by_row=by_row)
+        _close(out[:used], y, 5e-3)
+        assert float((out[used:] - 3).abs().max() if used < routing.places else 0) == 0.0
+        half = torch.empty((routing.places, n // 2), device="cuda", dtype=torch.bfloat16)
+        X.grouped_gemm(source, w, half, routing, by_row=by_row, epilogue=H.DENSE_CLAMPED_GLU, limit=0.8)
+        g, u = np.minimum(y[:, 0::2], 0.8), np.clip(y[:, 1::2], -0.8, 0.8)
+        _close(half[:used], g * O.sigmoid(1.702 * g) * (u + 1), 6e-3)
+        X.grouped_gemm(source, w, half, routing, by_row=by_row, epilogue=H.DENSE_SWIGLU)
+        _close(half[:used], y[:, 0::2] * O.sigmoid(y[:, 0::2]) * y[:, 1::2], 6e-3)
     f32 = torch.empty((routing.places, n), device="cuda")
     X.grouped_simple(x.float(), w.float(), f32, routing, gather=True)
     _close(f32[:used], y, 3e-6)
@@ -361,6 +368,6 @@ def test_what_the_kernels_refuse():
     routing = _routing(2, 4, 2)
     with pytest.raises(CacheIRB200Error):
         X.grouped_gemm(torch.zeros((2, 12), device="cuda", dtype=torch.bfloat16), torch.zeros((32, 12), device="cuda", dtype=torch.bfloat16),
-                       torch.zeros((4, 8), device="cuda", dtype=torch.bfloat16), routing, gather=True)
+                       torch.zeros((4, 8), device="cuda", dtype=torch.bfloat16), routing, by_row=True)
     with pytest.raises(ValueError):
         X.route(torch.zeros((3, 4), device="cuda"), torch.zeros(3, device="cuda", dtype=torch.int32), routing, 1.0)
