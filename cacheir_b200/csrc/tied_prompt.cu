@@ -5,7 +5,7 @@
 //   S [rows, keys] = Q K^T     A = queries (M 128), B = the page's key columns (N 64), K-major
 //   O [rows, dim] += P V       A = probabilities (M 128), B = the page's value columns read MN-major
 // A softmax thread owns a row (a tensor-memory lane), so row sums need no exchange.
-//   warps 0..3, 4..7  softmax of tile 0, tile 1      warp 8  MMA issue, tensor memory      warp 9  copies
+//   warp 0  copies      warp 1  MMA issue, tensor memory      warps 2..5, 6..9  softmax of tile 0, tile 1 (lane quarter = warp % 4)
 //
 // Queries and keys have unit root mean square, so |score| <= bound is known before any key is read. While exp(-2 bound) is
 // far from underflow the softmax refers to the bound itself (FIXED): no running maximum, no rescaling. Otherwise a row's
@@ -35,7 +35,7 @@ struct PromptParams {
   float pre;                   // with a polynomial: raw product -> [-1, 1]
   float coef[kTerms];          // score * log2 e = y (coef[0] + coef[1] y^2 + ...)
   int subs, heads_per_cta, tokens_per_tile;
-  int boxes, lead_boxes, stages, k_first, k_end;     // 16-column pieces of a query row that the scores take
+  int boxes, lead_boxes, stages;
   int n_cols;                  // output columns of the MMA
   int tmem_cols;
 };
@@ -60,17 +60,6 @@ __device__ __forceinline__ void tma_load_3d(uint32_t dst, const CUtensorMap* map
   asm volatile(
       "cp.async.bulk.tensor.3d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%3, %4, %5}], [%2];"
       ::"r"(dst), "l"(reinterpret_cast<uint64_t>(map)), "r"(bar), "r"(x), "r"(y), "r"(z) : "memory");
-}
-__device__ __forceinline__ void tmem_ld_x32(uint32_t taddr, float* v) {      // without the wait
-  uint32_t* r = reinterpret_cast<uint32_t*>(v);
-  asm volatile(
-      "tcgen05.ld.sync.aligned.32x32b.x32.b32 {%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,%16,%17,%18,%19,%20,%21,%22,%23,%24,%25,"
-      "%26,%27,%28,%29,%30,%31}, [%32];"
-      : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]), "=r"(r[4]), "=r"(r[5]), "=r"(r[6]), "=r"(r[7]), "=r"(r[8]), "=r"(r[9]),
-        "=r"(r[10]), "=r"(r[11]), "=r"(r[12]), "=r"(r[13]), "=r"(r[14]), "=r"(r[15]), "=r"(r[16]), "=r"(r[17]), "=r"(r[18]), "=r"(r[19]),
-        "=r"(r[20]), "=r"(r[21]), "=r"(r[22]), "=r"(r[23]), "=r"(r[24]), "=r"(r[25]), "=r"(r[26]), "=r"(r[27]), "=r"(r[28]), "=r"(r[29]),
-        "=r"(r[30]), "=r"(r[31])
-      : "r"(taddr) : "memory");
 }
 __device__ __forceinline__ void tmem_ld_x16(uint32_t taddr, float (&v)[16]) {
   uint32_t r[16];
@@ -113,6 +102,9 @@ __device__ __forceinline__ f32x2 fma2(f32x2 a, f32x2 b, f32x2 c) {
   return d;
 }
 
+// Out of line: most waits find their barrier complete, and the loop's code would crowd theirs.
+__device__ __noinline__ bool wait_long(uint32_t bar, uint32_t parity, int code) { return ptx::mbar_wait(bar, parity, &g_prompt_status, code); }
+
 // TERMS: of the polynomial, 0: the formula
 template <int TILES, bool FIXED, int TERMS>
 __global__ void __launch_bounds__(kThreads, 1)
@@ -123,16 +115,17 @@ tied_prompt_kernel(const __grid_constant__ CUtensorMap tmap_kv, const __grid_con
   const int page_bytes = p.boxes * kTiedBox, q_boxes = p.boxes - p.lead_boxes, q_bytes = q_boxes * kTile * 128;
   uint8_t* s_kv = smem;                                         // [stages][boxes][64 rows][128 bytes], swizzled
   uint8_t* s_q = s_kv + p.stages * page_bytes;                  // [tiles][q_boxes][128 rows][128 bytes], swizzled
-  uint8_t* s_p = s_q + TILES * q_bytes;                         // [tiles][128 rows][128 bytes], swizzled
-  float* s_inv = reinterpret_cast<float*>(s_p + TILES * kTile * 128);      // [stages][64]
+  uint8_t* s_p = s_q + TILES * q_bytes;                         // [page & 1][tiles][128 rows][128 bytes], swizzled
+  float* s_inv = reinterpret_cast<float*>(s_p + 2 * TILES * kTile * 128);      // [stages][64]
   uint64_t* full = reinterpret_cast<uint64_t*>(s_inv + p.stages * kTiedPage);
   uint64_t* empty = full + kMaxStages;
   uint64_t* bar_q = empty + kMaxStages;
-  uint64_t* bar_s = bar_q + 1;             // [2] scores in tensor memory
-  uint64_t* bar_free = bar_s + 2;          // [2] scores have been read
-  uint64_t* bar_p = bar_free + 2;          // [2] probabilities in shared memory
-  uint64_t* bar_o = bar_p + 2;             // [2] the page's output MMAs have retired
-  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bar_o + 2);
+  // [page & 1][tile]: with one barrier per parity nobody can be two phases behind (a page's successor of the same parity
+  // needs this page's probabilities from every thread)
+  uint64_t* bar_s = bar_q + 1;             // scores in tensor memory
+  uint64_t* bar_p = bar_s + 4;             // probabilities in shared memory
+  uint64_t* bar_o = bar_p + 4;             // the page's output MMAs have retired
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bar_o + 4);
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int kvh = blockIdx.x / p.subs, sub = blockIdx.x % p.subs, group = a.heads / a.kv_heads;
@@ -146,26 +139,28 @@ tied_prompt_kernel(const __grid_constant__ CUtensorMap tmap_kv, const __grid_con
   const TiedPages pages(a, pos0, pos0 + item.count - 1);
   const int n = pages.total;
 
-  if (warp == 9 && lane == 0) {
+  if (warp == 0 && lane == 0) {
     for (int s = 0; s < p.stages; ++s) { ptx::mbar_init(smem_addr(&full[s]), 1); ptx::mbar_init(smem_addr(&empty[s]), 1); }
     ptx::mbar_init(smem_addr(bar_q), 1);
-    for (int t = 0; t < 2; ++t) {
+    for (int t = 0; t < 4; ++t) {
       ptx::mbar_init(smem_addr(&bar_s[t]), 1);
-      ptx::mbar_init(smem_addr(&bar_free[t]), kTile);
-      ptx::mbar_init(smem_addr(&bar_p[t]), kTile);
+      ptx::mbar_init(smem_addr(&bar_p[t]), 4);            // a warp each
       ptx::mbar_init(smem_addr(&bar_o[t]), 1);
     }
     ptx::mbar_fence_init();
   }
-  if (warp == 8) ptx::tc_alloc(smem_addr(tmem_slot), p.tmem_cols);
+  if (warp == 1) ptx::tc_alloc(smem_addr(tmem_slot), p.tmem_cols);
   ptx::tc_fence_before();
   __syncthreads();
   ptx::tc_fence_after();
   const uint32_t tmem = *tmem_slot;                             // output of tile t at column t * n_cols, scores behind
-  const uint32_t tmem_s = tmem + TILES * p.n_cols;
+  const uint32_t tmem_s = tmem + TILES * p.n_cols;              // [page & 1][tile][64]
   bool ok = true;
+  auto wait = [&](uint32_t bar, uint32_t parity, int code) {
+    if (!ptx::mbar_try_wait(bar, parity)) ok = ok && wait_long(bar, parity, code);
+  };
 
-  if (warp == 9) {
+  if (warp == 0) {
     // ---------------- copies ----------------
     int slots = 0, issued = 0;
     if (lane == 0) {
@@ -199,7 +194,7 @@ tied_prompt_kernel(const __grid_constant__ CUtensorMap tmap_kv, const __grid_con
           ptx::mbar_wait(smem_addr(&full[it % p.stages]), (it / p.stages) & 1, &g_prompt_status, (9 << 8) | 3);
     }
     __syncwarp();
-  } else if (warp == 8) {
+  } else if (warp == 1) {
     // ---------------- MMA issue ----------------
     const uint32_t lead = lane == 0 ? 1u : 0u;
     const uint32_t id_s = (1u << 4) | (1u << 7) | (1u << 10) | (static_cast<uint32_t>(kTiedPage >> 3) << 17) | (static_cast<uint32_t>(kTile >> 4) << 24);
@@ -208,45 +203,50 @@ tied_prompt_kernel(const __grid_constant__ CUtensorMap tmap_kv, const __grid_con
     const uint64_t dq = ptx::smem_desc_sw128(smem_addr(s_q)), dk = ptx::smem_desc_sw128(smem_addr(s_kv + p.lead_boxes * kTiedBox));
     const uint64_t dp = ptx::smem_desc_sw128(smem_addr(s_p)), dv = smem_desc_mn_sw128(smem_addr(s_kv), kTiedBox);
     const uint32_t k_hi = static_cast<uint32_t>(dk >> 32), v_hi = static_cast<uint32_t>(dv >> 32);      // (dq, dk, dp share theirs)
-    ok = ptx::mbar_wait(smem_addr(bar_q), 0, &g_prompt_status, (9 << 8) | 4);
+    wait(smem_addr(bar_q), 0, (9 << 8) | 4);
     auto output = [&](int it) {
       const int s = it % p.stages;
       for (int t = 0; t < tiles; ++t) {
-        ok = ok && ptx::mbar_wait(smem_addr(&bar_p[t]), it & 1, &g_prompt_status, (9 << 8) | 5);
+        wait(smem_addr(&bar_p[(it & 1) * 2 + t]), (it >> 1) & 1, (9 << 8) | 5);
         __syncwarp();
         ptx::tc_fence_after();
-        const uint32_t pa = static_cast<uint32_t>(dp) + t * (kTile * 128 >> 4), vb = static_cast<uint32_t>(dv) + s * (page_bytes >> 4);
+        const uint32_t pa = static_cast<uint32_t>(dp) + ((it & 1) * TILES + t) * (kTile * 128 >> 4), vb = static_cast<uint32_t>(dv) + s * (page_bytes >> 4);
 #pragma unroll
         for (int j = 0; j < 4; ++j)          // 16 keys
           mma_f16_ss(lead, tmem + t * p.n_cols, pa + 2 * j, k_hi, vb + j * (2048 >> 4), v_hi, id_o, it > 0 || j > 0 ? 1u : 0u);
-        if (lead) ptx::tc_commit(smem_addr(&bar_o[t]));
+        if (lead) ptx::tc_commit(smem_addr(&bar_o[(it & 1) * 2 + t]));
         __syncwarp();
       }
       if (lead) ptx::tc_commit(smem_addr(&empty[s]));
       __syncwarp();
     };
 #pragma unroll 1
-    for (int it = 0; it < n; ++it) {
+    for (int it = 0; it < n; ++it) {       // (a score buffer is free: the probabilities of two pages before have been waited for)
       const int s = it % p.stages;
-      ok = ok && ptx::mbar_wait(smem_addr(&full[s]), (it / p.stages) & 1, &g_prompt_status, (9 << 8) | 6);
+      wait(smem_addr(&full[s]), (it / p.stages) & 1, (9 << 8) | 6);
+      __syncwarp();
+      ptx::tc_fence_after();
 #pragma unroll 1
       for (int t = 0; t < tiles; ++t) {
-        if (it > 0) ok = ok && ptx::mbar_wait(smem_addr(&bar_free[t]), (it - 1) & 1, &g_prompt_status, (9 << 8) | 7);
-        __syncwarp();
-        ptx::tc_fence_after();
-        const uint32_t qa = static_cast<uint32_t>(dq) + t * (q_bytes >> 4), kb = static_cast<uint32_t>(dk) + s * (page_bytes >> 4);
-        for (int k = p.k_first; k < p.k_end; ++k)      // (columns beyond the row are zero in both operands)
-          mma_f16_ss(lead, tmem_s + t * kTiedPage, qa + (k >> 2) * (kTile * 128 >> 4) + (k & 3) * 2, k_hi,
-                     kb + (k >> 2) * (kTiedBox >> 4) + (k & 3) * 2, k_hi, id_s, k > p.k_first ? 1u : 0u);
-        if (lead) ptx::tc_commit(smem_addr(&bar_s[t]));
+        const uint32_t d = tmem_s + ((it & 1) * TILES + t) * kTiedPage;
+        uint32_t qa = static_cast<uint32_t>(dq) + t * (q_bytes >> 4), kb = static_cast<uint32_t>(dk) + s * (page_bytes >> 4);
+#pragma unroll 1
+        for (int b = 0; b < q_boxes; ++b) {
+#pragma unroll
+          for (int j = 0; j < 4; ++j)      // (columns beyond the row are zero in both operands)
+            mma_f16_ss(lead, d, qa + 2 * j, k_hi, kb + 2 * j, k_hi, id_s, (b | j) > 0 ? 1u : 0u);
+          qa += kTile * 128 >> 4;
+          kb += kTiedBox >> 4;
+        }
+        if (lead) ptx::tc_commit(smem_addr(&bar_s[(it & 1) * 2 + t]));
         __syncwarp();
       }
       if (it > 0) output(it - 1);
     }
     output(n - 1);
-  } else if (warp < 4 * tiles) {
+  } else if (warp < 2 + 4 * tiles) {
     // ---------------- softmax: thread = row ----------------
-    const int t = warp >> 2, r = (warp & 3) * 32 + lane;
+    const int t = (warp - 2) >> 2, r = (warp & 3) * 32 + lane;
     const int tok = r / p.heads_per_cta, h = r % p.heads_per_cta;
     const int first = item.row0 + t * p.tokens_per_tile, count = min(p.tokens_per_tile, item.count - t * p.tokens_per_tile);
     const bool real = tok < count && h < nheads;
@@ -259,31 +259,29 @@ tied_prompt_kernel(const __grid_constant__ CUtensorMap tmap_kv, const __grid_con
     for (int k = 0; k < TERMS; ++k) coef[k] = pair(p.coef[k], p.coef[k]);
     const f32x2 pre = pair(p.pre, p.pre), minus_ref = pair(-m_ref, -m_ref);
     const uint32_t lanes = static_cast<uint32_t>((warp & 3) * 32) << 16;
-    uint8_t* p_row = s_p + t * kTile * 128 + r * 128;
+    const int hi_row = rp, lo_row = rp - a.window;
     for (int it = 0; it < n; ++it) {
       const int s = it % p.stages, base = pages.page(it) * kTiedPage;
-      ok = ok && ptx::mbar_wait(smem_addr(&full[s]), (it / p.stages) & 1, &g_prompt_status, (9 << 8) | 8);
-      ok = ok && ptx::mbar_wait(smem_addr(&bar_s[t]), it & 1, &g_prompt_status, (9 << 8) | 9);
+      const uint32_t scores = tmem_s + ((it & 1) * TILES + t) * kTiedPage + lanes;
+      uint8_t* p_row = s_p + ((it & 1) * TILES + t) * kTile * 128 + r * 128;
+      const float4* inv4 = reinterpret_cast<const float4*>(s_inv + s * kTiedPage);
+      // (rows without a token may hold anything: a row of P reaches its own row of O only, which is not stored)
+      const bool whole = base + kTiedPage - 1 <= tile_pos && (base > tile_pos + count - 1 - a.window || base + kTiedPage <= a.keep_first);
+      if (it > 1) wait(smem_addr(&bar_o[(it & 1) * 2 + t]), ((it >> 1) & 1) ^ 1, (9 << 8) | 10);      // the P buffer is free
+      wait(smem_addr(&full[s]), (it / p.stages) & 1, (9 << 8) | 8);
+      wait(smem_addr(&bar_s[(it & 1) * 2 + t]), (it >> 1) & 1, (9 << 8) | 9);
       __syncwarp();
       ptx::tc_fence_after();
-      float v[kTiedPage];
-      tmem_ld_x32(tmem_s + t * kTiedPage + lanes, v);
-      tmem_ld_x32(tmem_s + t * kTiedPage + 32 + lanes, v + 32);
-      ptx::tc_wait_ld();
-#pragma unroll
-      for (int i = 0; i < kTiedPage; ++i) asm volatile("" : "+f"(v[i]));      // (the values exist from here on)
-      ptx::tc_fence_before();
-      ptx::mbar_arrive(smem_addr(&bar_free[t]));
-      // scores * log2 e; FIXED: minus the reference. Eight pairs side by side, so that their chains overlap.
-      const float4* inv4 = reinterpret_cast<const float4*>(s_inv + s * kTiedPage);
-#pragma unroll
-      for (int i0 = 0; i0 < kTiedPage; i0 += 16) {
-        f32x2 u[8], c[8];
+      // 16 scores * log2 e (FIXED: minus the reference) as pairs side by side, so that their chains overlap
+      auto score16 = [&](int i0, f32x2 (&c)[8]) {
+        float v[16];
+        tmem_ld_x16(scores + i0, v);
+        f32x2 u[8];
 #pragma unroll
         for (int j = 0; j < 8; j += 2) {
-          const float4 f = inv4[(i0 + 2 * j) / 4];
-          u[j] = mul2(pair(v[i0 + 2 * j], v[i0 + 2 * j + 1]), pair(f.x, f.y));
-          u[j + 1] = mul2(pair(v[i0 + 2 * j + 2], v[i0 + 2 * j + 3]), pair(f.z, f.w));
+          const float4 f = inv4[i0 / 4 + j / 2];
+          u[j] = mul2(pair(v[2 * j], v[2 * j + 1]), pair(f.x, f.y));
+          u[j + 1] = mul2(pair(v[2 * j + 2], v[2 * j + 3]), pair(f.z, f.w));
         }
         if constexpr (TERMS > 0) {
           f32x2 w[8];
@@ -308,40 +306,41 @@ tied_prompt_kernel(const __grid_constant__ CUtensorMap tmap_kv, const __grid_con
             if (FIXED) c[j] = add2(c[j], minus_ref);
           }
         }
+        if (!whole) {
+          const int hi = hi_row - base - i0, lo = lo_row - base - i0, kept = a.keep_first - base - i0;
 #pragma unroll
-        for (int j = 0; j < 8; ++j) unpair(c[j], v[i0 + 2 * j], v[i0 + 2 * j + 1]);
-      }
-      // (rows without a token may hold anything: a row of P reaches its own row of O only, which is not stored)
-      if (!(base + kTiedPage - 1 <= tile_pos && (base > tile_pos + count - 1 - a.window || base + kTiedPage <= a.keep_first))) {
-        const int hi = rp - base, lo = rp - a.window - base, kept = a.keep_first - base;
-#pragma unroll
-        for (int i = 0; i < kTiedPage; ++i)
-          if (!(i <= hi && (i > lo || i < kept))) v[i] = -INFINITY;
-      }
-      float alpha = 1.f;
+          for (int j = 0; j < 8; ++j) {
+            float x, y;
+            unpair(c[j], x, y);
+            if (!(2 * j <= hi && (2 * j > lo || 2 * j < kept))) x = -INFINITY;
+            if (!(2 * j + 1 <= hi && (2 * j + 1 > lo || 2 * j + 1 < kept))) y = -INFINITY;
+            c[j] = pair(x, y);
+          }
+        }
+      };
       if constexpr (!FIXED) {
-        float mx = v[0];
+        float mx = -INFINITY, alpha = 1.f;
+#pragma unroll 1
+        for (int i0 = 0; i0 < kTiedPage; i0 += 16) {
+          f32x2 c[8];
+          score16(i0, c);
 #pragma unroll
-        for (int i = 1; i < kTiedPage; ++i) mx = fmaxf(mx, v[i]);
+          for (int j = 0; j < 8; ++j) {
+            float x, y;
+            unpair(c[j], x, y);
+            mx = fmaxf(mx, fmaxf(x, y));
+          }
+        }
         if (mx > m_ref + (it == 0 ? 0.f : kStale)) {
           alpha = tied_ex2(m_ref - mx);
           m_ref = mx;
         }
-#pragma unroll
-        for (int i = 0; i < kTiedPage; ++i) v[i] -= m_ref;
         l2 = mul2(l2, pair(alpha, alpha));
-      }
-      uint32_t packed[kTiedPage / 2];
-#pragma unroll
-      for (int i = 0; i < kTiedPage; i += 2) {
-        const float x = tied_ex2(v[i]), y = tied_ex2(v[i + 1]);
-        l2 = add2(l2, pair(x, y));
-        packed[i / 2] = pack_bf16(x, y);
-      }
-      if (it > 0) ok = ok && ptx::mbar_wait(smem_addr(&bar_o[t]), (it - 1) & 1, &g_prompt_status, (9 << 8) | 10);
-      if constexpr (!FIXED) {
         if (__any_sync(0xffffffffu, it > 0 && alpha != 1.f)) {        // rare: this warp's rows of O to the new references
+          wait(smem_addr(&bar_o[((it - 1) & 1) * 2 + t]), ((it - 1) >> 1) & 1, (9 << 8) | 12);
+          __syncwarp();
           ptx::tc_fence_after();
+#pragma unroll 1
           for (int c = 0; c < p.n_cols; c += 16) {
             float o[16];
             tmem_ld_x16(tmem + t * p.n_cols + c + lanes, o);
@@ -353,17 +352,33 @@ tied_prompt_kernel(const __grid_constant__ CUtensorMap tmap_kv, const __grid_con
         }
       }
 #pragma unroll
-      for (int c = 0; c < 8; ++c)
-        *reinterpret_cast<uint4*>(p_row + ((c ^ (r & 7)) << 4)) = make_uint4(packed[4 * c], packed[4 * c + 1], packed[4 * c + 2], packed[4 * c + 3]);
+      for (int i0 = 0; i0 < kTiedPage; i0 += 16) {
+        f32x2 c[8];
+        score16(i0, c);
+        uint32_t packed[8];
+#pragma unroll
+        for (int j = 0; j < 8; ++j) {
+          float x, y;
+          unpair(c[j], x, y);
+          if (!FIXED) { x -= m_ref; y -= m_ref; }
+          x = tied_ex2(x);
+          y = tied_ex2(y);
+          l2 = add2(l2, pair(x, y));
+          packed[j] = pack_bf16(x, y);
+        }
+        *reinterpret_cast<uint4*>(p_row + (((i0 / 8) ^ (r & 7)) << 4)) = make_uint4(packed[0], packed[1], packed[2], packed[3]);
+        *reinterpret_cast<uint4*>(p_row + (((i0 / 8 + 1) ^ (r & 7)) << 4)) = make_uint4(packed[4], packed[5], packed[6], packed[7]);
+      }
       const int tail = pos0 + item.count - base;
       if (tail < kTiedPage && t == 0)        // rows behind the last token may hold anything: zero, so that 0 * row stays 0
-        for (int i = threadIdx.x; i < (kTiedPage - tail) * p.boxes * 8; i += kTile) {
+        for (int i = threadIdx.x - 64; i < (kTiedPage - tail) * p.boxes * 8; i += kTile) {
           const int row = tail + i / (p.boxes * 8), c = i % (p.boxes * 8);
           *reinterpret_cast<uint4*>(s_kv + s * page_bytes + (c >> 3) * kTiedBox + row * 128 + (c & 7) * 16) = make_uint4(0u, 0u, 0u, 0u);
         }
       asm volatile("fence.proxy.async.shared::cta;" ::: "memory");       // the tensor core reads what was just written
       ptx::tc_fence_before();
-      ptx::mbar_arrive(smem_addr(&bar_p[t]));
+      __syncwarp();
+      if (lane == 0) ptx::mbar_arrive(smem_addr(&bar_p[(it & 1) * 2 + t]));
     }
     const size_t row = first + tok, col0 = static_cast<size_t>(head0 + h) * a.dim;
     float l, l_odd;
@@ -374,7 +389,7 @@ tied_prompt_kernel(const __grid_constant__ CUtensorMap tmap_kv, const __grid_con
 #pragma unroll
       for (int i = 0; i < 16; ++i)
         g[i] = p.gate && real && c0 + 8 * i < a.dim ? *reinterpret_cast<const uint4*>(p.gate + row * p.gate_stride + col0 + c0 + 8 * i) : make_uint4(0u, 0u, 0u, 0u);
-      if (c0 == 0) ok = ok && ptx::mbar_wait(smem_addr(&bar_o[t]), (n - 1) & 1, &g_prompt_status, (9 << 8) | 11);
+      if (c0 == 0) wait(smem_addr(&bar_o[((n - 1) & 1) * 2 + t]), ((n - 1) >> 1) & 1, (9 << 8) | 11);
       __syncwarp();
       ptx::tc_fence_after();
 #pragma unroll
@@ -399,7 +414,7 @@ tied_prompt_kernel(const __grid_constant__ CUtensorMap tmap_kv, const __grid_con
   }
   ptx::tc_fence_before();
   __syncthreads();
-  if (warp == 8) {
+  if (warp == 1) {
     ptx::tc_fence_after();
     ptx::tc_dealloc(tmem, p.tmem_cols);
   }
@@ -410,7 +425,7 @@ int prompt_tiles(int dim) { return dim <= 128 ? 2 : 1; }
 int row_boxes(int dim, int rot) { return (dim + rot + 63) / 64; }
 size_t prompt_fixed(int dim, int rot) {
   const int tiles = prompt_tiles(dim);
-  return 1024 + static_cast<size_t>(tiles) * (row_boxes(dim, rot) - rot / 64 + 1) * kTile * 128 + kMaxStages * kTiedPage * 4 + (2 * kMaxStages + 9) * 8 + 16;
+  return 1024 + static_cast<size_t>(tiles) * (row_boxes(dim, rot) - rot / 64 + 2) * kTile * 128 + kMaxStages * kTiedPage * 4 + (2 * kMaxStages + 13) * 8 + 16;
 }
 int prompt_stages(int dim, int rot) {
   const size_t fixed = prompt_fixed(dim, rot), page = static_cast<size_t>(row_boxes(dim, rot)) * kTiedBox;
@@ -520,10 +535,8 @@ extern "C" int cacheir_b200_tied_attention_prompt(const cacheir_b200_tied_args* 
   p.boxes = row_boxes(a.dim, a.rot_dims);
   p.lead_boxes = a.rot_dims / 64;
   p.stages = prompt_stages(a.dim, a.rot_dims);
-  p.k_first = (a.rot_dims - tied_lead(a.rot_dims)) / 16;
-  p.k_end = (a.dim + a.rot_dims - tied_lead(a.rot_dims) + 15) / 16;
   p.n_cols = (a.dim + 15) / 16 * 16;
-  const int cols = tiles * (p.n_cols + kTiedPage);
+  const int cols = tiles * (p.n_cols + 2 * kTiedPage);
   p.tmem_cols = cols <= 128 ? 128 : cols <= 256 ? 256 : 512;
   const int items = ragged_items(a.rows, a.segments, tiles * p.tokens_per_tile);
   if (items > 65535) return CACHEIR_B200_ELIMIT;
