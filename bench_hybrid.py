@@ -56,6 +56,8 @@ def synthetic(device):
     gen = torch.Generator(device=device)
 
     def make(key: str, shape: tuple[int, ...]):
+        if len(shape) == 1 and key.endswith((".q.b", ".k.b", ".o.b", ".gate.b", ".up.b", ".down.b")):
+            return torch.zeros(shape, device=device)      # (a constant added to every token would send them all to the same experts)
         if len(shape) <= 1:
             return torch.full(shape, 0.6 if key.endswith("alpha") else 1.0, device=device)
         gen.manual_seed(zlib.crc32(key.encode()))
@@ -170,7 +172,8 @@ def gutorax_work(s: dict, rows: int, logit_rows: int, keys_per_row: float, cache
     return work
 
 
-def topunex_work(s: dict, rows: int, logit_rows: int, keys_per_row: float, cached_rows: float, decode: bool) -> dict[str, list[tuple[float, float]]]:
+def topunex_work(s: dict, rows: int, logit_rows: int, keys_per_row: float, cached_rows: float, decode: bool, touched: int) -> dict[str, list[tuple[float, float]]]:
+    """`touched`: experts with at least one token."""
     w, ff, h, g, d, rot = s["width"], s["ff"], s["heads"], s["kv_heads"], s["dim"], s["rot"]
     work: dict[str, list[tuple[float, float]]] = defaultdict(list)
 
@@ -178,7 +181,6 @@ def topunex_work(s: dict, rows: int, logit_rows: int, keys_per_row: float, cache
         work["b200." + kind].append((2.0 * (weights * n * k + t * k + t * n_out), 2.0 * t * n * k))
 
     qw = d + rot - rot // 64 * 64
-    touched = s["experts"] * (1.0 - (1.0 - s["top"] / s["experts"]) ** rows)
     for i in range(s["layers"]):
         n = (2 * h + g) * d
         gemm("dense_gemm", n, w, n)
@@ -236,7 +238,16 @@ def against_roofline(times: dict[str, tuple[int, float]], work: dict, hbm_gbs: f
     return out
 
 
-RAGGED_WORK = {"gutorax": gutorax_work, "topunex": topunex_work}
+RAGGED = ("gutorax", "topunex")
+
+
+def ragged_kernels(family: str, rt, plan, s: dict, rows: int, logit_rows: int, keys: float, cached: float, decode: bool, hbm: float, tf: float) -> list[dict]:
+    import torch
+    times = kind_times(plan)
+    if family == "gutorax":
+        return against_roofline(times, gutorax_work(s, rows, logit_rows, keys, cached, decode), hbm, tf)
+    cu = rt._engine.scratch("route_cu", 0).view(torch.int32)[: s["experts"] + 1]      # what the timed products ran on
+    return against_roofline(times, topunex_work(s, rows, logit_rows, keys, cached, decode, int((cu.diff() > 0).sum())), hbm, tf)
 
 
 def run(size: str, batch: int, ctx: int, prompt: int, steps: int, peaks: dict, families: tuple[str, ...] = ("gutorax",)) -> dict:
@@ -248,7 +259,7 @@ def run(size: str, batch: int, ctx: int, prompt: int, steps: int, peaks: dict, f
     for family in families + ("llama-shaped int8",):
         rt = build(family, s, batch=batch, positions=max(ctx, prompt) + 8 * steps + 64)
         sessions = fill(rt, batch, ctx)
-        first = [1] * batch
+        first = [(7919 * i + 1) % s["vocab"] for i in range(batch)]
         torch.cuda.synchronize()
         rt.decode_greedy_batch(sessions, first, 3)
         start, stop = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
@@ -259,9 +270,9 @@ def run(size: str, batch: int, ctx: int, prompt: int, steps: int, peaks: dict, f
         ms = start.elapsed_time(stop) / steps
         seen = ctx + steps // 2
         plan = rt._engine.plans[("decode", batch)]
-        if family in RAGGED_WORK:
+        if family in RAGGED:
             keys = min(seen, s["window"])
-            decode_kernels = against_roofline(kind_times(plan), RAGGED_WORK[family](s, batch, batch, keys, batch * keys, True), hbm, tf)
+            decode_kernels = ragged_kernels(family, rt, plan, s, batch, batch, keys, batch * keys, True, hbm, tf)
         else:
             decode_kernels = against_roofline(kind_times(plan), llama_work(s, batch, seen, batch * seen), hbm, tf)
         for x in sessions:
@@ -271,15 +282,15 @@ def run(size: str, batch: int, ctx: int, prompt: int, steps: int, peaks: dict, f
 
         def prefill():
             session.kv_cache.clear()
-            if family in RAGGED_WORK:
+            if family in RAGGED:
                 session.run_step_batch([session], [ids])
             else:
                 session.run([ids], mode="prefill")
         prefill_ms = timed(prefill, 5)
-        if family in RAGGED_WORK:
+        if family in RAGGED:
             plan = rt._engine.portion_plan(prompt, 1, 1)
             avg = sum(min(i + 1, s["window"]) for i in range(prompt)) / prompt
-            prefill_kernels = against_roofline(kind_times(plan), RAGGED_WORK[family](s, prompt, 1, avg, prompt, False), hbm, tf)
+            prefill_kernels = ragged_kernels(family, rt, plan, s, prompt, 1, avg, prompt, False, hbm, tf)
         else:      # the last pass of the prompt: 64 rows that attend to all of it
             plan = rt._engine.prefill_plan(64, 1)
             prefill_kernels = against_roofline(kind_times(plan), llama_work(s, 64, prompt, prompt), hbm, tf)
