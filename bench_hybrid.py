@@ -1,4 +1,4 @@
-"""`bench.py --family gutorax|topunex`: prefill and decode throughput of a ragged family beside the other ones at equal
+"""`bench.py --family gutorax|topunex|rekodra`: prefill and decode throughput of a ragged family beside the other ones at equal
 width, (active) feed-forward, heads and layer count (random weights), and every kernel's distance from its roofline.
 
 Throughput: decode is `decode_greedy_batch` (CUDA-graph replay, argmax fed back on the device) over `batch` sequences
@@ -13,7 +13,7 @@ from collections import defaultdict
 
 SIZES = {
     # width, ff, heads, kv_heads, head dim, latent rank, rotated dims, window, layers, vocab; mixtures (every second Topunex
-    # layer): top experts and the shared one add up to ff
+    # layer, every Rekodra layer): top experts and the shared one add up to ff
     "4096": dict(width=4096, ff=14336, heads=32, kv_heads=8, dim=128, rank=512, rot=64, window=4096, layers=8, vocab=32768, side=256,
                  experts=32, top=4, expert_ff=1792, shared_ff=7168, keep=4),
     "2048": dict(width=2048, ff=5632, heads=16, kv_heads=8, dim=128, rank=256, rot=64, window=1024, layers=12, vocab=32768, side=128,
@@ -49,6 +49,21 @@ def topunex_config(s: dict) -> dict:
             "layers": [{"type": "attention", "mixer": mixer, "mlp": moe if i % 2 else {"kind": "dense", "ff": s["ff"]}} for i in range(s["layers"])]}
 
 
+def rekodra_config(s: dict) -> dict:
+    """Attention over all tokens, and window attention beside matrix memory with half of the heads each, in turn. An eighth of the
+    router's outputs are identity experts."""
+    half = s["heads"] // 2
+    full = {"heads": s["heads"], "kv_heads": s["kv_heads"], "dim": s["dim"], "vdim": s["dim"], "scale": s["dim"] ** -0.5,
+            "rot": {"base": 500000.0, "dims": s["rot"]}}
+    both = {"left": {"heads": half, "kv_heads": s["kv_heads"], "dim": s["dim"], "vdim": s["dim"], "scale": s["dim"] ** -0.5, "mask": {"size": s["window"]}},
+            "right": {"heads": half, "dim": s["dim"], "vdim": s["dim"], "gate_cap": 15.0}}
+    moe = {"kind": "moe", "expert": {"ff": s["expert_ff"]}, "shared": {"ff": s["shared_ff"]},
+           "router": {"experts": s["experts"] * 7 // 8, "identity": s["experts"] // 8, "top": s["top"], "groups": {"count": 4, "keep": 2}}}
+    return {"architecture": "Rekodra", "width": s["width"], "vocab": s["vocab"], "norm": {"eps": 1e-6}, "embedding": {"scale": 1.0}, "logit_scale": 1.0,
+            "layers": [{"type": "parallel", "mixer": both, "mlp": moe} if i % 2 else {"type": "attention", "mixer": full, "mlp": moe}
+                       for i in range(s["layers"])]}
+
+
 def synthetic(device):
     import zlib
 
@@ -58,6 +73,10 @@ def synthetic(device):
     def make(key: str, shape: tuple[int, ...]):
         if len(shape) == 1 and key.endswith((".q.b", ".k.b", ".o.b", ".gate.b", ".up.b", ".down.b")):
             return torch.zeros(shape, device=device)      # (a constant added to every token would send them all to the same experts)
+        if key.endswith(("mix.right.i.b", "mlp.correction")):
+            return torch.zeros(shape, device=device)
+        if key.endswith("mix.right.f.b"):
+            return torch.full(shape, 4.0, device=device)
         if len(shape) <= 1:
             return torch.full(shape, 0.6 if key.endswith("alpha") else 1.0, device=device)
         gen.manual_seed(zlib.crc32(key.encode()))
@@ -69,13 +88,15 @@ def build(family: str, s: dict, *, batch: int, positions: int):
     import torch
 
     from cacheir_b200 import (B200DecodeRuntime, B200KVPageAllocator, GutoraxConfig, ModelConfig, build_decoder_artifact,
-                              TopunexConfig, build_gutorax_artifact, build_topunex_artifact)
+                              RekodraConfig, TopunexConfig, build_gutorax_artifact, build_rekodra_artifact, build_topunex_artifact)
     dev = torch.device("cuda", torch.cuda.current_device())
     if family == "gutorax":
         art, page = build_gutorax_artifact(GutoraxConfig.from_dict(gutorax_config(s))), 64
         dtype = "bfloat16"
     elif family == "topunex":
         art, page, dtype = build_topunex_artifact(TopunexConfig.from_dict(topunex_config(s))), 64, "bfloat16"
+    elif family == "rekodra":
+        art, page, dtype = build_rekodra_artifact(RekodraConfig.from_dict(rekodra_config(s))), 64, "bfloat16"
     else:
         art = build_decoder_artifact(ModelConfig(
             architecture="LlamaForCausalLM", hidden_size=s["width"], intermediate_size=s["ff"], num_layers=s["layers"],
@@ -95,7 +116,7 @@ def fill(rt, batch: int, ctx: int):
         for name, t in pool.items():
             t.fill_(1.0) if name == "inv_rms" else t.normal_()
     for state in rt.kv_allocator._states.values():
-        state.normal_()
+        state.normal_()            # (a matrix memory's maxima and normalisers too: any values do)
     return sessions
 
 
@@ -207,6 +228,56 @@ def topunex_work(s: dict, rows: int, logit_rows: int, keys_per_row: float, cache
     return work
 
 
+def rekodra_work(s: dict, rows: int, logit_rows: int, span: int, decode: bool, touched: int, places: int) -> dict[str, list[tuple[float, float]]]:
+    """`span`: tokens a decoded row has seen, or the prompt's; `touched`: experts with at least one token, `places`: their rows."""
+    w, h, g, d, rot = s["width"], s["heads"], s["kv_heads"], s["dim"], s["rot"]
+    half, scored = h // 2, s["experts"]
+    work: dict[str, list[tuple[float, float]]] = defaultdict(list)
+
+    def gemm(kind, n, k, n_out, t=rows, weights=1.0):
+        work["b200." + kind].append((2.0 * (weights * n * k + t * k + t * n_out), 2.0 * t * n * k))
+
+    def attention(heads, width, qw, window):
+        keys = min(span, window) if decode else sum(min(i + 1, window) for i in range(span)) / span
+        cached = rows * keys if decode else span
+        work["b200.tied_prepare"].append((2.0 * rows * (heads * (d + qw) + g * (2 * width - rot if width < 2 * d else 2 * width)), 0.0))
+        work["b200.tied_attention_step" if decode else "b200.tied_attention_prompt"].append(
+            (cached * g * (2.0 * width + 4) + 2.0 * rows * heads * (qw + d), 2.0 * rows * heads * keys * (qw + d)))
+
+    for i in range(s["layers"]):
+        if i % 2:
+            n = (half + 2 * g) * d + 4 * half * d + 2 * half
+            gemm("dense_gemm", n, w, n)
+            attention(half, 2 * d, d, s["window"])
+            gemm("dense_gemm.o", w, half * d, w)
+            io = rows * half * d * 2.0
+            state = half * d * (d + 1) * 8.0
+            if decode:
+                work["b200.memory_step"].append((rows * state + 5 * io, rows * half * 4.0 * d * d))
+            else:
+                work["b200.memory_gates"].append((rows * half * 20.0, 0.0))
+                work["b200.recurrence_chunked"].append((state + 4 * io, rows * half * 4.0 * d * d))
+                work["b200.memory_norm"].append((3 * io, 0.0))
+            gemm("dense_gemm.o", w, half * d, w)
+            work["b200.residual_rms_pair"].append((rows * w * (4 + 8 + 2.0), 0.0))
+        else:
+            n = (h + g) * d
+            gemm("dense_gemm", n, w, n)
+            attention(h, d + rot, d + rot - rot // 64 * 64, 1 << 30)
+            gemm("dense_gemm.o", w, h * d, w)
+            work["b200.residual_add"].append((rows * w * (2 + 8 + 2.0), 0.0))
+        gemm("dense_gemm.swiglu", 2 * s["shared_ff"] + scored + 1, w, s["shared_ff"])
+        gemm("dense_gemm.down", w, s["shared_ff"], w)
+        work["b200.route"].append((rows * (scored * 4.0 + s["top"] * 16) + (0 if decode else 2.0 * w * (rows + places)), 0.0))
+        gemm("grouped_gemm.swiglu", 2 * s["expert_ff"], w, s["expert_ff"], t=places, weights=touched)
+        gemm("grouped_gemm", w, s["expert_ff"], w, t=places, weights=touched)
+        work["b200.combine_residual"].append((2.0 * places * w + rows * w * (2 + 2 + 8 + 2.0), 0.0))
+    work["b200.scaled_embedding"].append((rows * w * (2 + 4 + 2.0), 0.0))
+    work["b200.rms_rows"].append((logit_rows * w * 6.0, 0.0))
+    gemm("dense_gemm.lm_head", s["vocab"], w, 2 * s["vocab"], t=logit_rows)
+    return work
+
+
 def llama_work(s: dict, rows: int, keys_per_row: float, cached_rows: float) -> dict[str, list[tuple[float, float]]]:
     w, ff, d = s["width"], s["ff"], s["width"] // s["heads"]
     kv = s["kv_heads"] * d
@@ -238,14 +309,18 @@ def against_roofline(times: dict[str, tuple[int, float]], work: dict, hbm_gbs: f
     return out
 
 
-RAGGED = ("gutorax", "topunex")
+RAGGED = ("gutorax", "topunex", "rekodra")
 
 
-def ragged_kernels(family: str, rt, plan, s: dict, rows: int, logit_rows: int, keys: float, cached: float, decode: bool, hbm: float, tf: float) -> list[dict]:
+def ragged_kernels(family: str, rt, plan, s: dict, rows: int, logit_rows: int, keys: float, cached: float, span: int, decode: bool, hbm: float,
+                   tf: float) -> list[dict]:
     import torch
     times = kind_times(plan)
     if family == "gutorax":
         return against_roofline(times, gutorax_work(s, rows, logit_rows, keys, cached, decode), hbm, tf)
+    if family == "rekodra":
+        cu = rt._engine.scratch("route_cu", 0).view(torch.int32)[: s["experts"] * 7 // 8 + 1]
+        return against_roofline(times, rekodra_work(s, rows, logit_rows, span, decode, int((cu.diff() > 0).sum()), int(cu[-1])), hbm, tf)
     cu = rt._engine.scratch("route_cu", 0).view(torch.int32)[: s["experts"] + 1]      # what the timed products ran on
     return against_roofline(times, topunex_work(s, rows, logit_rows, keys, cached, decode, int((cu.diff() > 0).sum())), hbm, tf)
 
@@ -272,7 +347,7 @@ def run(size: str, batch: int, ctx: int, prompt: int, steps: int, peaks: dict, f
         plan = rt._engine.plans[("decode", batch)]
         if family in RAGGED:
             keys = min(seen, s["window"])
-            decode_kernels = ragged_kernels(family, rt, plan, s, batch, batch, keys, batch * keys, True, hbm, tf)
+            decode_kernels = ragged_kernels(family, rt, plan, s, batch, batch, keys, batch * keys, seen, True, hbm, tf)
         else:
             decode_kernels = against_roofline(kind_times(plan), llama_work(s, batch, seen, batch * seen), hbm, tf)
         for x in sessions:
@@ -290,7 +365,7 @@ def run(size: str, batch: int, ctx: int, prompt: int, steps: int, peaks: dict, f
         if family in RAGGED:
             plan = rt._engine.portion_plan(prompt, 1, 1)
             avg = sum(min(i + 1, s["window"]) for i in range(prompt)) / prompt
-            prefill_kernels = ragged_kernels(family, rt, plan, s, prompt, 1, avg, prompt, False, hbm, tf)
+            prefill_kernels = ragged_kernels(family, rt, plan, s, prompt, 1, avg, prompt, prompt, False, hbm, tf)
         else:      # the last pass of the prompt: 64 rows that attend to all of it
             plan = rt._engine.prefill_plan(64, 1)
             prefill_kernels = against_roofline(kind_times(plan), llama_work(s, 64, prompt, prompt), hbm, tf)

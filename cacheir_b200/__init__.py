@@ -13,13 +13,15 @@ from .gutorax import GutoraxConfig, build_gutorax_artifact
 from .kv_cache import B200KVPageAllocator, B200PagedKVCache, KVPage
 from .models import load_model
 from .registry import B200_BACKEND, Backend, BackendRegistry, default_registry
+from .rekodra import RekodraConfig, build_rekodra_artifact
 from .topunex import TopunexConfig, build_topunex_artifact
 
 __all__ = [
     "B200DecodeRuntime", "create_runtime", "b200_runtime_available",
     "B200KVPageAllocator", "B200PagedKVCache", "KVPage",
     "CompileArtifact", "Graph", "ModelConfig", "Node", "build_decoder_artifact", "build_decoder_graph",
-    "GutoraxConfig", "build_gutorax_artifact", "TopunexConfig", "build_topunex_artifact", "load_model",
+    "GutoraxConfig", "build_gutorax_artifact", "TopunexConfig", "build_topunex_artifact", "RekodraConfig",
+    "build_rekodra_artifact", "load_model",
     "B200_BACKEND", "Backend", "BackendRegistry", "default_registry",
 ]
 

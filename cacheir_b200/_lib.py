@@ -11,7 +11,7 @@ from ctypes import c_char_p, c_float, c_int, c_longlong, c_size_t, c_void_p
 from pathlib import Path
 
 LIB_PATH = Path(__file__).resolve().parent / "lib" / "libcacheir_b200.so"
-GROUP_PATHS = {name: LIB_PATH.with_name(f"libcacheir_b200_{name}.so") for name in ("ragged", "hybrid", "experts")}
+GROUP_PATHS = {name: LIB_PATH.with_name(f"libcacheir_b200_{name}.so") for name in ("ragged", "hybrid", "recurrence", "experts")}
 
 # name -> (restype, argtypes); mirrors include/cacheir_b200.h one to one
 SIGNATURES: dict[str, tuple[object, list[object]]] = {
@@ -134,7 +134,8 @@ class RecurrenceArgs(ctypes.Structure):
     _fields_ = [("positions", c_void_p), ("cu_rows", c_void_p), ("slots", c_void_p), ("rows", c_int), ("segments", c_int),
                 ("heads", c_int), ("dim", c_int), ("vdim", c_int), ("q", c_void_p), ("k", c_void_p), ("v", c_void_p),
                 ("stride", c_longlong), ("decay_pow", c_void_p), ("state", c_void_p), ("num_slots", c_int), ("out", c_void_p),
-                ("dtype", c_int)]
+                ("dtype", c_int), ("slot_stride", c_longlong), ("log_decay", c_void_p), ("log_take", c_void_p),
+                ("normaliser", c_void_p), ("q_scale", c_float)]
 
 
 class TiedArgs(ctypes.Structure):
@@ -142,9 +143,15 @@ class TiedArgs(ctypes.Structure):
 
     _fields_ = [("positions", c_void_p), ("row_seg", c_void_p), ("cu_rows", c_void_p), ("page_table", c_void_p),
                 ("rows", c_int), ("segments", c_int), ("max_pages", c_int), ("page_size", c_int), ("num_slots", c_int),
-                ("heads", c_int), ("kv_heads", c_int), ("dim", c_int), ("rot_dims", c_int), ("window", c_int), ("keep_first", c_int),
-                ("scale", c_float), ("cap", c_float), ("pool", c_void_p), ("inv_rms", c_void_p), ("sink", c_void_p),
+                ("heads", c_int), ("kv_heads", c_int), ("dim", c_int), ("width", c_int), ("key_from", c_int), ("window", c_int),
+                ("keep_first", c_int), ("scale", c_float), ("cap", c_float), ("reach", c_float), ("pool", c_void_p), ("inv_rms", c_void_p), ("sink", c_void_p),
                 ("dtype", c_int), ("decode", c_int)]
+
+
+class RouteRule(ctypes.Structure):
+    """cacheir_b200_route_rule"""
+
+    _fields_ = [("softmax", c_int), ("identity", c_int), ("groups", c_int), ("keep", c_int), ("correction", c_void_p), ("scale", c_float)]
 
 
 _NEXT = [c_int, c_void_p, c_void_p, c_float, c_void_p]      # next_mode next_w next_b next_alpha next_out
@@ -154,10 +161,12 @@ GROUP_SIGNATURES: dict[str, dict[str, tuple[object, list[object]]]] = {
         "cacheir_b200_dense_supported": (c_int, [c_int, c_longlong, c_longlong, c_int, c_int]),
         "cacheir_b200_dense_gemm": (c_int, [c_void_p, c_void_p]),
         "cacheir_b200_dense_simple": (c_int, [c_void_p] * 3 + [c_int] * 7 + [c_longlong] * 3 + [c_void_p, c_int, c_int, c_void_p]),
-        "cacheir_b200_scaled_embedding": (c_int, [c_void_p] * 3 + [c_int, c_int, c_int, c_float] + _NEXT + [c_int, c_void_p]),
+        "cacheir_b200_scaled_embedding": (c_int, [c_void_p] * 3 + [c_int, c_int, c_int, c_float, c_int] + _NEXT + [c_int, c_void_p]),
         "cacheir_b200_dyt_rows": (c_int, [c_void_p] * 4 + [c_float, c_void_p, c_int, c_int, c_int, c_void_p]),
         "cacheir_b200_rms_rows": (c_int, [c_void_p] * 3 + [c_float, c_void_p, c_int, c_int, c_int, c_void_p]),
         "cacheir_b200_residual_dyt": (c_int, [c_void_p] * 4 + [c_float, c_int, c_int] + _NEXT + [c_int, c_void_p]),
+        "cacheir_b200_residual_add": (c_int, [c_void_p] * 2 + [c_int, c_int] + _NEXT + [c_int, c_void_p]),
+        "cacheir_b200_residual_rms_pair": (c_int, [c_void_p] * 5 + [c_float, c_float, c_int, c_int] + _NEXT + [c_int, c_void_p]),
         "cacheir_b200_residual_rms": (c_int, [c_void_p] * 3 + [c_float, c_int, c_int] + _NEXT + [c_int, c_void_p]),
         "cacheir_b200_gated_rms": (c_int, [c_void_p, c_void_p, c_longlong, c_void_p, c_float, c_void_p, c_int, c_int, c_int, c_void_p]),
         "cacheir_b200_glu_pairs": (c_int, [c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_int, c_void_p]),
@@ -174,28 +183,38 @@ GROUP_SIGNATURES: dict[str, dict[str, tuple[object, list[object]]]] = {
         "cacheir_b200_latent_attention_supported": (c_int, [c_int] * 4),
         "cacheir_b200_latent_attention_splits": (c_int, [c_int] * 5),
         "cacheir_b200_latent_attention": (c_int, [c_void_p] * 4 + [c_int, c_void_p]),
+        "cacheir_b200_hybrid_device_status": (c_int, [c_int]),
+    },
+    "recurrence": {
         "cacheir_b200_recurrence_simple": (c_int, [c_void_p, c_void_p]),
         "cacheir_b200_recurrence_step": (c_int, [c_void_p, c_void_p]),
         "cacheir_b200_recurrence_chunked_supported": (c_int, [c_int] * 3),
         "cacheir_b200_recurrence_workspace_bytes": (c_size_t, [c_int] * 5),
         "cacheir_b200_recurrence_chunked": (c_int, [c_void_p, c_void_p, c_size_t, c_void_p]),
-        "cacheir_b200_hybrid_device_status": (c_int, [c_int]),
+        "cacheir_b200_memory_gates": (c_int, [c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_float] + [c_void_p] * 4),
+        "cacheir_b200_memory_norm": (c_int, [c_void_p] * 4 + [c_longlong, c_void_p, c_float, c_void_p, c_int, c_int, c_int, c_int, c_void_p]),
+        "cacheir_b200_memory_step": (
+            c_int, [c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_float, c_void_p, c_longlong, c_void_p, c_float, c_void_p]),
+        "cacheir_b200_recurrence_device_status": (c_int, [c_int]),
     },
     "experts": {
         "cacheir_b200_tied_prepare": (
-            c_int, [c_void_p, c_void_p, c_longlong, c_void_p, c_longlong, c_float, c_void_p, c_int, c_void_p, c_void_p]),
+            c_int, [c_void_p, c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_longlong, c_int, c_int, c_void_p, c_void_p, c_float,
+                    c_void_p, c_int, c_void_p, c_void_p]),
         "cacheir_b200_tied_attention_simple": (c_int, [c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_void_p]),
-        "cacheir_b200_tied_prompt_supported": (c_int, [c_int] * 6),
+        "cacheir_b200_tied_prompt_supported": (c_int, [c_int] * 7),
         "cacheir_b200_tied_attention_prompt": (c_int, [c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_void_p]),
-        "cacheir_b200_tied_step_supported": (c_int, [c_int] * 6),
+        "cacheir_b200_tied_step_supported": (c_int, [c_int] * 7),
         "cacheir_b200_tied_step_splits": (c_int, [c_int] * 7),
         "cacheir_b200_tied_attention_step": (c_int, [c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_int, c_void_p]),
-        "cacheir_b200_route": (c_int, [c_void_p, c_longlong, c_void_p, c_int, c_int, c_int, c_float] + [c_void_p] * 8 + [c_int, c_void_p]),
+        "cacheir_b200_route": (c_int, [c_void_p, c_longlong, c_void_p, c_int, c_int, c_int] + [c_void_p] * 9 + [c_int, c_void_p]),
         "cacheir_b200_grouped_all_rows": (c_int, []),
         "cacheir_b200_grouped_gemm": (c_int, [c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p]),
         "cacheir_b200_grouped_simple": (c_int, [c_void_p] * 5 + [c_int] * 4 + [c_longlong] * 3 + [c_int, c_void_p]),
         "cacheir_b200_combine_residual_rms": (
             c_int, [c_void_p] * 4 + [c_int, c_void_p, c_void_p, c_float, c_int, c_int, c_int, c_void_p, c_int, c_void_p]),
+        "cacheir_b200_combine_residual": (
+            c_int, [c_void_p] * 4 + [c_int, c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_int] + _NEXT + [c_int, c_void_p]),
         "cacheir_b200_experts_device_status": (c_int, [c_int]),
     },
 }

@@ -6,8 +6,8 @@ Plain C-ABI shared objects (no torch, no pybind), each a group of the .cu files
 under csrc/ compiled with -gencode arch=compute_100a,code=sm_100a and linked
 with the static CUDA runtime: `core` (libcacheir_b200.so, Llama-shaped models),
 `ragged` (dense products and row operators of the families with ragged steps),
-`hybrid` (latent attention, linear recurrences) and `experts` (tied attention,
-mixtures of experts). A model family names the groups it needs, so a fresh
+`hybrid` (latent attention), `recurrence` (linear recurrences, matrix memory) and
+`experts` (tied attention, mixtures of experts). A model family names the groups it needs, so a fresh
 checkout compiles only those. Objects are rebuilt only when their source or a
 header is newer.
 """
@@ -29,7 +29,8 @@ LIB_DIR = PKG_DIR / "lib"
 SHARED = ("glue", "misc")            # in the core and the ragged library: argmax, position bookkeeping, error text
 GROUP_FILES = {
     "ragged": ("dense_gemm", "hybrid_glue") + SHARED,
-    "hybrid": ("latent_attention", "linear_recurrence"),
+    "hybrid": ("latent_attention",),
+    "recurrence": ("linear_recurrence",),
     "experts": ("tied_attention", "tied_prompt", "grouped_gemm", "expert_routing"),
 }
 LIB_PATHS = {"core": LIB_DIR / "libcacheir_b200.so", **{name: LIB_DIR / f"libcacheir_b200_{name}.so" for name in GROUP_FILES}}

@@ -50,15 +50,16 @@ extern "C" int cacheir_b200_dense_gemm(const cacheir_b200_dense_args* args, void
   if (p.w_stride < p.K || p.x_stride < static_cast<long long>(p.x_batch_cols) * (p.batch - 1) + p.K) return CACHEIR_B200_EINVAL;
   if (p.batch > 1 && (p.w_batch_rows < p.N || p.bias)) return CACHEIR_B200_EINVAL;
   if ((static_cast<long long>(p.N) + kTileN - 1) / kTileN * p.batch > 65535) return CACHEIR_B200_ELIMIT;
+  const bool tail_ok = p.tail_cols >= 0 && p.tail_cols <= p.N && (p.tail_cols == 0 || (p.tail && p.batch == 1));
   cudaStream_t st = as_stream(stream);
   switch (p.epilogue) {
-    case CACHEIR_B200_DENSE_BF16: return p.y ? launch_mt<CACHEIR_B200_DENSE_BF16>(p, st) : CACHEIR_B200_EINVAL;
+    case CACHEIR_B200_DENSE_BF16: return p.y && tail_ok ? launch_mt<CACHEIR_B200_DENSE_BF16>(p, st) : CACHEIR_B200_EINVAL;
     case CACHEIR_B200_DENSE_F32: return p.y ? launch_mt<CACHEIR_B200_DENSE_F32>(p, st) : CACHEIR_B200_EINVAL;
-    case CACHEIR_B200_DENSE_SILU: return p.y ? launch_mt<CACHEIR_B200_DENSE_SILU>(p, st) : CACHEIR_B200_EINVAL;
+    case CACHEIR_B200_DENSE_SILU: return p.y && tail_ok ? launch_mt<CACHEIR_B200_DENSE_SILU>(p, st) : CACHEIR_B200_EINVAL;
     case CACHEIR_B200_DENSE_GEGLU:
     case CACHEIR_B200_DENSE_SWIGLU:
     case CACHEIR_B200_DENSE_CLAMPED_GLU:
-      if (!p.y || p.tail_cols < 0 || p.tail_cols > p.N || (p.N - p.tail_cols) % 2 != 0 || (p.tail_cols > 0 && !p.tail) || p.batch != 1)
+      if (!p.y || !tail_ok || (p.N - p.tail_cols) % 2 != 0 || p.batch != 1)
         return CACHEIR_B200_EINVAL;
       if (p.epilogue == CACHEIR_B200_DENSE_GEGLU) return launch_mt<CACHEIR_B200_DENSE_GEGLU>(p, st);
       if (p.epilogue == CACHEIR_B200_DENSE_SWIGLU) return launch_mt<CACHEIR_B200_DENSE_SWIGLU>(p, st);

@@ -279,6 +279,12 @@ dense_gemm_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_const
           const int t = row_of(t0 + c0 + j);
           if (!n_ok || t < 0) continue;
           float y = v[j];
+          if constexpr (!GROUPED && (EPI == CACHEIR_B200_DENSE_BF16 || EPI == CACHEIR_B200_DENSE_SILU)) {
+            if (n >= p.N - p.tail_cols) {        // plain float32 columns behind the others
+              p.tail[static_cast<long long>(t) * p.tail_stride + (n - (p.N - p.tail_cols))] = y;
+              continue;
+            }
+          }
           if constexpr (EPI == CACHEIR_B200_DENSE_F32) {
             static_cast<float*>(p.y)[static_cast<long long>(t) * p.y_stride + ycol] = y;
             continue;

@@ -1,7 +1,7 @@
 // Row operators of the hybrid families that are not a GEMM epilogue: embedding into the 32-bit residual stream, Dynamic
 // Tanh, the RMS-normed residual add, the gated RMS norm behind a recurrence, and the stand-alone forms of the dense
 // kernel's epilogues (used in 32-bit runs and for extents the tensor-core kernel does not take).
-#include "hybrid_common.cuh"
+#include "residual_rows.cuh"
 
 namespace cb200 {
 namespace {
@@ -115,6 +115,63 @@ residual_rms_kernel(float* __restrict__ x, const T* __restrict__ y, const float*
     }
     if (nx.mode != CACHEIR_B200_NEXT_NONE) store_vec<T, VEC>(static_cast<T*>(nx.out) + row * width + c, s);
   }
+}
+
+// residual = table[ids] * scale, or that much more
+template <typename T, int VEC, bool ADD>
+__global__ void __launch_bounds__(kRowThreads)
+embedding_rows_kernel(const T* __restrict__ table, const int64_t* __restrict__ ids, float* x, int width, int vocab, float scale, RowNext nx) {
+  __shared__ float scratch[32];
+  const size_t row = blockIdx.x;
+  const T* src = table + min(max(ids[row], static_cast<int64_t>(0)), static_cast<int64_t>(vocab - 1)) * width;
+  finish_row<T, VEC>(x + row * width, row, width, nx, scratch, [&](int c, float (&s)[VEC]) {
+    float v[VEC];
+    load_vec<T, VEC>(src + c, v);
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) s[i] = ADD ? s[i] + v[i] * scale : v[i] * scale;
+  });
+}
+
+template <typename T, int VEC>
+__global__ void __launch_bounds__(kRowThreads)
+residual_add_kernel(float* x, const T* __restrict__ y, int width, RowNext nx) {
+  __shared__ float scratch[32];
+  const size_t row = blockIdx.x;
+  finish_row<T, VEC>(x + row * width, row, width, nx, scratch, [&](int c, float (&s)[VEC]) {
+    float v[VEC];
+    load_vec<T, VEC>(y + row * width + c, v);
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) s[i] += v[i];
+  });
+}
+
+template <typename T, int VEC>
+__global__ void __launch_bounds__(kRowThreads)
+residual_rms_pair_kernel(float* x, const T* __restrict__ y1, const float* __restrict__ w1, const T* __restrict__ y2,
+                         const float* __restrict__ w2, float factor, float eps, int width, RowNext nx) {
+  __shared__ float scratch[32];
+  const size_t row = blockIdx.x;
+  y1 += row * width;
+  y2 += row * width;
+  float ss1 = 0.f, ss2 = 0.f;
+  for (int c = threadIdx.x * VEC; c < width; c += kRowThreads * VEC) {
+    float a[VEC], b[VEC];
+    load_vec<T, VEC>(y1 + c, a);
+    load_vec<T, VEC>(y2 + c, b);
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) { ss1 = fmaf(a[i], a[i], ss1); ss2 = fmaf(b[i], b[i], ss2); }
+  }
+  const float f1 = factor / sqrtf(block_sum_all(ss1, scratch) / static_cast<float>(width) + eps);
+  const float f2 = factor / sqrtf(block_sum_all(ss2, scratch) / static_cast<float>(width) + eps);
+  finish_row<T, VEC>(x + row * width, row, width, nx, scratch, [&](int c, float (&s)[VEC]) {
+    float a[VEC], b[VEC], u[VEC], v[VEC];
+    load_vec<T, VEC>(y1 + c, a);
+    load_vec<T, VEC>(y2 + c, b);
+    load_vec<float, VEC>(w1 + c, u);
+    load_vec<float, VEC>(w2 + c, v);
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) s[i] += a[i] * f1 * u[i] + b[i] * f2 * v[i];
+  });
 }
 
 template <typename T, int VEC>
@@ -233,10 +290,26 @@ bool next_ok(int mode, const float* w, const float* b, const void* out) {
 using namespace cb200;
 
 extern "C" int cacheir_b200_scaled_embedding(const void* table, const int64_t* ids, float* residual, int rows, int width, int vocab,
-                                             float scale, int next_mode, const float* next_w, const float* next_b, float next_alpha,
+                                             float scale, int accumulate, int next_mode, const float* next_w, const float* next_b, float next_alpha,
                                              void* next_out, int dtype, void* stream) {
   if (rows <= 0 || width <= 0) return 0;
-  if (!table || !ids || !residual || vocab <= 0 || !next_ok(next_mode, next_w, next_b, next_out)) return CACHEIR_B200_EINVAL;
+  if (!table || !ids || !residual || vocab <= 0) return CACHEIR_B200_EINVAL;
+  if (accumulate || next_mode == CACHEIR_B200_NEXT_RMS) {
+    if (!row_next_ok(next_mode, next_w, next_out)) return CACHEIR_B200_EINVAL;
+    const RowNext rn{next_mode, next_w, next_alpha, next_out};
+    const bool vec = width % 4 == 0 && aligned_to(table, 16) && aligned_to(residual, 16) && row_next_aligned(next_mode, next_w, next_out);
+#define CB200_ROWS(VEC, ADD)                                                                  \
+  embedding_rows_kernel<T, VEC, ADD><<<rows, kRowThreads, 0, as_stream(stream)>>>(static_cast<const T*>(table), ids, residual, width, vocab, scale, rn)
+    CB200_HYBRID_DTYPE(dtype, {
+      if (vec && accumulate) CB200_ROWS(4, true);
+      else if (vec) CB200_ROWS(4, false);
+      else if (accumulate) CB200_ROWS(1, true);
+      else CB200_ROWS(1, false);
+    });
+#undef CB200_ROWS
+    return launch_status();
+  }
+  if (!next_ok(next_mode, next_w, next_b, next_out)) return CACHEIR_B200_EINVAL;
   const NextArgs nx{next_mode, next_w, next_b, next_alpha, next_out};
   CB200_HYBRID_DTYPE(dtype, (scaled_embedding_kernel<T><<<row_grid(rows, width), 256, 0, as_stream(stream)>>>(
                                 static_cast<const T*>(table), ids, residual, width, vocab, scale, nx)));
@@ -272,6 +345,38 @@ extern "C" int cacheir_b200_residual_dyt(float* residual, const void* y, const f
   const NextArgs nx{next_mode, next_w, next_b, next_alpha, next_out};
   CB200_HYBRID_DTYPE(dtype, (residual_dyt_kernel<T><<<row_grid(rows, width), 256, 0, as_stream(stream)>>>(
                                 residual, static_cast<const T*>(y), w, b, alpha, width, nx)));
+  return launch_status();
+}
+
+extern "C" int cacheir_b200_residual_add(float* residual, const void* y, int rows, int width, int next_mode, const float* next_w,
+                                         const float* next_b, float next_alpha, void* next_out, int dtype, void* stream) {
+  if (rows <= 0 || width <= 0) return 0;
+  if (!residual || !y || next_b || !row_next_ok(next_mode, next_w, next_out)) return CACHEIR_B200_EINVAL;
+  const RowNext nx{next_mode, next_w, next_alpha, next_out};
+  const bool vec = width % 4 == 0 && aligned_to(residual, 16) && aligned_to(y, 16) && row_next_aligned(next_mode, next_w, next_out);
+  CB200_HYBRID_DTYPE(dtype, {
+    if (vec) residual_add_kernel<T, 4><<<rows, kRowThreads, 0, as_stream(stream)>>>(residual, static_cast<const T*>(y), width, nx);
+    else residual_add_kernel<T, 1><<<rows, kRowThreads, 0, as_stream(stream)>>>(residual, static_cast<const T*>(y), width, nx);
+  });
+  return launch_status();
+}
+
+extern "C" int cacheir_b200_residual_rms_pair(float* residual, const void* y1, const float* w1, const void* y2, const float* w2, float factor,
+                                              float eps, int rows, int width, int next_mode, const float* next_w, const float* next_b,
+                                              float next_alpha, void* next_out, int dtype, void* stream) {
+  if (rows <= 0 || width <= 0) return 0;
+  if (!residual || !y1 || !w1 || !y2 || !w2 || next_b || !row_next_ok(next_mode, next_w, next_out)) return CACHEIR_B200_EINVAL;
+  const RowNext nx{next_mode, next_w, next_alpha, next_out};
+  const bool vec = width % 4 == 0 && aligned_to(residual, 16) && aligned_to(y1, 16) && aligned_to(y2, 16) && aligned_to(w1, 16) &&
+                   aligned_to(w2, 16) && row_next_aligned(next_mode, next_w, next_out);
+#define CB200_PAIR(VEC)                                                                                                                  \
+  residual_rms_pair_kernel<T, VEC><<<rows, kRowThreads, 0, as_stream(stream)>>>(residual, static_cast<const T*>(y1), w1, static_cast<const T*>(y2), \
+                                                                               w2, factor, eps, width, nx)
+  CB200_HYBRID_DTYPE(dtype, {
+    if (vec) CB200_PAIR(4);
+    else CB200_PAIR(1);
+  });
+#undef CB200_PAIR
   return launch_status();
 }
 

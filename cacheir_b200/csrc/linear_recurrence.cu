@@ -1,4 +1,6 @@
-// Linear recurrence S <- decay S + k v^T, o = S^T q per head, float32 state carried per sequence slot, sm_100a.
+// Linear recurrence S <- decay S + take k v^T, o = S^T q per head, float32 state carried per sequence slot, sm_100a.
+// decay is a constant per head and take one; or (GATED) both belong to the token and the head, given as logarithms, and a
+// vector n <- decay n + take k runs along, of which q . n is kept for whoever normalises o.
 //
 // simple   any extents and types: one CTA per (sequence, head, 32 value columns) walks the tokens, state in shared memory
 // step     decode: one CTA per (sequence, head) streams the state once (16-byte accesses), HBM bound
@@ -7,8 +9,11 @@
 //          The state stays in float32 registers; whatever is float32 by nature and has to enter an MMA (the state, the
 //          decayed scores, the decayed values) goes in as a sum of two bf16 numbers. Sequences are cut into 256-token
 //          pieces that run in parallel: a first pass finds every piece's own contribution, a scan turns these into the
-//          pieces' initial states, and the main pass starts from them.
-#include "cacheir_b200_hybrid.h"
+//          pieces' initial states, and the main pass starts from them. GATED: with c the running sum of log decays in a
+//          chunk, decay^(i-j) becomes exp(c_i - c_j + log take_j), and so on; n rides with the first value columns.
+// gates    matrix memory: log decay and log take from gate logits, relative to a running maximum (a scan over the tokens)
+// memory   matrix memory, decode: gates, state, normaliser, the head's norm and the output gate in one pass over the state
+#include "cacheir_b200_recurrence.h"
 #include "hybrid_common.cuh"
 #include "ragged.cuh"
 
@@ -23,19 +28,30 @@ constexpr int kPitchV = kCols + 8; // bf16 elements per shared-memory row (16 by
 
 using Args = cacheir_b200_recurrence_args;
 
-__device__ __forceinline__ float* slot_state(const Args& a, int seg, int h) {
+// A slot: [heads][dim][vdim] state; with gates also [heads][dim] normaliser and [heads] running maxima behind it.
+__device__ __forceinline__ float* slot_base(const Args& a, int seg) {
   const int slot = min(max(a.slots[seg], 0), a.num_slots - 1);
-  return a.state + (static_cast<size_t>(slot) * a.heads + h) * a.dim * a.vdim;
+  return a.state + static_cast<size_t>(slot) * a.slot_stride;
+}
+__device__ __forceinline__ float* slot_state(const Args& a, int seg, int h) {
+  return slot_base(a, seg) + static_cast<size_t>(h) * a.dim * a.vdim;
+}
+__device__ __forceinline__ float* slot_normaliser(const Args& a, int seg, int h) {
+  return slot_base(a, seg) + static_cast<size_t>(a.heads) * a.dim * a.vdim + static_cast<size_t>(h) * a.dim;
+}
+__device__ __forceinline__ float* slot_maximum(const Args& a, int seg, int h) {
+  return slot_base(a, seg) + static_cast<size_t>(a.heads) * a.dim * (a.vdim + 1) + h;
 }
 
-template <typename T>
+template <typename T, bool GATED>
 __global__ void __launch_bounds__(256)
 recurrence_simple_kernel(const Args a) {
   extern __shared__ float sm[];
   float* s_state = sm;                       // [dim][32]
   float* s_k = s_state + a.dim * 32;         // [dim]
   float* s_q = s_k + a.dim;                  // [dim]
-  float* s_red = s_q + a.dim;                // [8][32]
+  float* s_n = s_q + a.dim;                  // [dim]
+  float* s_red = s_n + a.dim;                // [8][32]
   const int seg = blockIdx.x, h = blockIdx.y;
   const int row0 = a.cu_rows[seg], row1 = a.cu_rows[seg + 1];
   if (row0 >= row1) return;
@@ -46,13 +62,20 @@ recurrence_simple_kernel(const Args a) {
   const bool fresh = a.positions[row0] == 0;
   for (int d = group; d < a.dim; d += 8)
     s_state[d * 32 + lane] = (fresh || !col_ok) ? 0.f : state[static_cast<size_t>(d) * a.vdim + col];
-  const float decay = a.decay_pow[h * kPowers + 1];
+  const bool first = GATED && blockIdx.z == 0;        // this block also has the normaliser
+  if (first)
+    for (int d = threadIdx.x; d < a.dim; d += 256) s_n[d] = fresh ? 0.f : slot_normaliser(a, seg, h)[d];
+  float decay = GATED ? 0.f : a.decay_pow[h * kPowers + 1], take = 1.f;
   for (int row = row0; row < row1; ++row) {
     __syncthreads();
+    if (GATED) {
+      decay = expf(a.log_decay[static_cast<size_t>(row) * a.heads + h]);
+      take = expf(a.log_take[static_cast<size_t>(row) * a.heads + h]);
+    }
     const size_t off = static_cast<size_t>(row) * a.stride;
     for (int d = threadIdx.x; d < a.dim; d += 256) {
-      s_k[d] = Elem<T>::ld(static_cast<const T*>(a.k) + off + static_cast<size_t>(h) * a.dim + d);
-      s_q[d] = Elem<T>::ld(static_cast<const T*>(a.q) + off + static_cast<size_t>(h) * a.dim + d);
+      s_k[d] = Elem<T>::ld(static_cast<const T*>(a.k) + off + static_cast<size_t>(h) * a.dim + d) * take;
+      s_q[d] = Elem<T>::ld(static_cast<const T*>(a.q) + off + static_cast<size_t>(h) * a.dim + d) * (GATED ? a.q_scale : 1.f);
     }
     const float v = col_ok ? Elem<T>::ld(static_cast<const T*>(a.v) + off + static_cast<size_t>(h) * a.vdim + col) : 0.f;
     __syncthreads();
@@ -70,7 +93,19 @@ recurrence_simple_kernel(const Args a) {
       for (int g = 0; g < 8; ++g) t += s_red[g * 32 + lane];
       Elem<T>::st(static_cast<T*>(a.out) + (static_cast<size_t>(row) * a.heads + h) * a.vdim + col, t);
     }
+    if (first) {
+      float nq = 0.f;
+      for (int d = threadIdx.x; d < a.dim; d += 256) {
+        const float n = fmaf(s_n[d], decay, s_k[d]);
+        s_n[d] = n;
+        nq = fmaf(n, s_q[d], nq);
+      }
+      nq = block_sum_all(nq, s_red + 256);
+      if (threadIdx.x == 0) a.normaliser[static_cast<size_t>(row) * a.heads + h] = nq;
+    }
   }
+  if (first)
+    for (int d = threadIdx.x; d < a.dim; d += 256) slot_normaliser(a, seg, h)[d] = s_n[d];
   if (col_ok)
     for (int d = group; d < a.dim; d += 8) state[static_cast<size_t>(d) * a.vdim + col] = s_state[d * 32 + lane];
 }
@@ -132,10 +167,22 @@ recurrence_step_kernel(const Args a) {
 }
 
 // ---- chunked form ----------------------------------------------------------------------------------------------------
+// Between the passes: every piece's state [pieces][heads][dim][vdim]; with gates also its normaliser [pieces][heads][dim] and
+// the sum of its log decays [pieces][heads].
+struct PieceSpace {
+  float* state;
+  float* normaliser;
+  float* log_decay;
+};
+PieceSpace piece_space(const Args& a, float* ws, int items) {
+  float* n = ws + static_cast<size_t>(items) * a.heads * a.dim * a.vdim;
+  return {ws, n, n + static_cast<size_t>(items) * a.heads * a.dim};
+}
+
 // MT = 16-row state tiles per warp (dim <= 64 MT)
-template <int MT, bool LOCAL>
+template <int MT, bool LOCAL, bool GATED>
 __global__ void __launch_bounds__(128)
-recurrence_chunk_kernel(const Args a, float* __restrict__ ws) {
+recurrence_chunk_kernel(const Args a, const PieceSpace ws) {
   extern __shared__ __align__(16) uint8_t raw[];
   const int dim = a.dim;
   const int pitch = dim + 8;
@@ -145,6 +192,7 @@ recurrence_chunk_kernel(const Args a, float* __restrict__ ws) {
   __nv_bfloat16* s_dv = s_v + kChunk * kPitchV;                      // [2][64][72] decayed values, hi | lo
   __nv_bfloat16* s_s = s_dv + 2 * kChunk * kPitchV;                  // [2][dim][72] state, hi | lo
   __shared__ float s_pow[kPowers];
+  __shared__ float s_cum[kChunk], s_take[kChunk], s_left[kChunk], s_n[128];      // log decays summed, log take, weight in the chunk's last state
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int h = blockIdx.y, v0 = blockIdx.z * kCols;
 
@@ -152,14 +200,20 @@ recurrence_chunk_kernel(const Args a, float* __restrict__ ws) {
   if (it.seg < 0) return;
   const bool alone = it.last && static_cast<int>(blockIdx.x) == it.first;     // the segment is a single piece
   if (LOCAL && it.last) return;                                               // nobody needs its contribution
-  for (int i = threadIdx.x; i < kPowers; i += 128) s_pow[i] = a.decay_pow[h * kPowers + i];
+  if (!GATED)
+    for (int i = threadIdx.x; i < kPowers; i += 128) s_pow[i] = a.decay_pow[h * kPowers + i];
 
   float st[MT][8][4];          // state rows (warp + 4 t)*16 .. +15, columns v0 .. v0+63
   float* state = slot_state(a, it.seg, h);
-  float* piece = ws + (static_cast<size_t>(blockIdx.x) * a.heads + h) * dim * a.vdim;
+  float* piece = ws.state + (static_cast<size_t>(blockIdx.x) * a.heads + h) * dim * a.vdim;
+  float* piece_n = ws.normaliser + (static_cast<size_t>(blockIdx.x) * a.heads + h) * dim;
   const float* init = alone ? state : piece;
   const bool zero = LOCAL || (alone && a.positions[it.row0] == 0);
   const int cols = min(kCols, a.vdim - v0);
+  const bool first = GATED && blockIdx.z == 0;        // this block also has the normaliser
+  float sum = 0.f;                                    // of the piece's log decays
+  if (first && static_cast<int>(threadIdx.x) < dim)
+    s_n[threadIdx.x] = zero ? 0.f : (alone ? slot_normaliser(a, it.seg, h) : piece_n)[threadIdx.x];
 #pragma unroll
   for (int t = 0; t < MT; ++t)
 #pragma unroll
@@ -178,6 +232,33 @@ recurrence_chunk_kernel(const Args a, float* __restrict__ ws) {
   for (int r0 = 0; r0 < it.count; r0 += kChunk) {
     const int n = min(kChunk, it.count - r0);
     const size_t base = static_cast<size_t>(it.row0 + r0);
+    if (GATED) {
+      if (warp == 0) {
+        float c[2], take[2], last = 0.f;
+#pragma unroll
+        for (int u = 0; u < 2; ++u) {
+          const int r = u * 32 + lane;
+          const size_t at = (base + r) * a.heads + h;
+          c[u] = r < n ? a.log_decay[at] : 0.f;
+          take[u] = r < n ? a.log_take[at] : 0.f;
+#pragma unroll
+          for (int off = 1; off < 32; off <<= 1) {
+            const float up = __shfl_up_sync(0xffffffffu, c[u], off);
+            if (lane >= off) c[u] += up;
+          }
+          c[u] += last;
+          last = __shfl_sync(0xffffffffu, c[u], 31);
+        }
+#pragma unroll
+        for (int u = 0; u < 2; ++u) {
+          const int r = u * 32 + lane;
+          s_cum[r] = c[u];
+          s_take[r] = take[u];
+          s_left[r] = r < n ? __expf(last - c[u] + take[u]) : 0.f;
+        }
+      }
+      __syncthreads();
+    }
     for (int i = threadIdx.x; i < kChunk * kc; i += 128) {
       const int r = i / kc, c = i % kc;
       uint4 q = make_uint4(0u, 0u, 0u, 0u), k = q;
@@ -195,7 +276,7 @@ recurrence_chunk_kernel(const Args a, float* __restrict__ ws) {
       if (r < n && c * 8 < cols)
         v = *reinterpret_cast<const uint4*>(static_cast<const __nv_bfloat16*>(a.v) + (base + r) * a.stride + static_cast<size_t>(h) * a.vdim + v0 + c * 8);
       if (!LOCAL) *reinterpret_cast<uint4*>(s_v + r * kPitchV + c * 8) = v;
-      const float f = s_pow[max(n - 1 - r, 0)];
+      const float f = GATED ? s_left[r] : s_pow[max(n - 1 - r, 0)];
       const uint32_t* w = reinterpret_cast<const uint32_t*>(&v);
       uint4 hi, lo;
       uint32_t* hw = reinterpret_cast<uint32_t*>(&hi);
@@ -267,7 +348,16 @@ recurrence_chunk_kernel(const Args a, float* __restrict__ ws) {
           }
       }
       const int i0 = warp * 16 + (lane >> 2);
-      const float f0 = s_pow[i0 + 1], f1 = s_pow[i0 + 9];
+      const float f0 = GATED ? __expf(s_cum[i0]) * a.q_scale : s_pow[i0 + 1], f1 = GATED ? __expf(s_cum[i0 + 8]) * a.q_scale : s_pow[i0 + 9];
+      float nq[2] = {0.f, 0.f};
+      if (first) {                                    // q . (n before the chunk): a quarter of the entries per lane of the row
+        for (int d = lane & 3; d < dim; d += 4) {
+          nq[0] = fmaf(__bfloat162float(s_q[i0 * pitch + d]), s_n[d], nq[0]);
+          nq[1] = fmaf(__bfloat162float(s_q[(i0 + 8) * pitch + d]), s_n[d], nq[1]);
+        }
+        nq[0] *= f0;
+        nq[1] *= f1;
+      }
 #pragma unroll
       for (int nn = 0; nn < 8; ++nn) {
         o[nn][0] *= f0; o[nn][1] *= f0; o[nn][2] *= f1; o[nn][3] *= f1;
@@ -282,7 +372,9 @@ recurrence_chunk_kernel(const Args a, float* __restrict__ ws) {
 #pragma unroll
           for (int e = 0; e < 4; ++e) {
             const int i = i0 + (e >> 1) * 8, j = kk * 16 + u * 8 + (lane & 3) * 2 + (e & 1);
-            d[u][e] = j <= i ? sc[2 * kk + u][e] * s_pow[i - j] : 0.f;
+            if (GATED) d[u][e] = j <= i ? sc[2 * kk + u][e] * (__expf(s_cum[i] - s_cum[j] + s_take[j]) * a.q_scale) : 0.f;
+            else d[u][e] = j <= i ? sc[2 * kk + u][e] * s_pow[i - j] : 0.f;
+            if (GATED) nq[e >> 1] += d[u][e];
           }
         uint32_t hi[4], lo[4];
 #pragma unroll
@@ -309,6 +401,11 @@ recurrence_chunk_kernel(const Args a, float* __restrict__ ws) {
 #pragma unroll
       for (int e = 0; e < 2; ++e) {
         const int i = i0 + e * 8;
+        if (first) {
+          nq[e] += __shfl_xor_sync(0xffffffffu, nq[e], 1);
+          nq[e] += __shfl_xor_sync(0xffffffffu, nq[e], 2);
+          if ((lane & 3) == 0 && i < n) a.normaliser[(base + i) * a.heads + h] = nq[e];
+        }
         if (i < n) {
           __nv_bfloat16* dst = out + ((base + i) * a.heads + h) * a.vdim + v0;
 #pragma unroll
@@ -321,7 +418,8 @@ recurrence_chunk_kernel(const Args a, float* __restrict__ ws) {
     }
 
     // S' = decay^n S + K^T (decayed V)
-    const float fn = s_pow[n];
+    const float fn = GATED ? __expf(s_cum[n - 1]) : s_pow[n];
+    if (GATED) sum += s_cum[n - 1];
     const uint32_t kt = smem_addr(s_k) + (((lane & 7) + ((lane >> 4) & 1) * 8) * pitch + ((lane >> 3) & 1) * 8) * 2;
     const uint32_t dv = smem_addr(s_dv) + (((lane & 7) + ((lane >> 3) & 1) * 8) * kPitchV + (lane >> 4) * 8) * 2;
 #pragma unroll
@@ -347,11 +445,22 @@ recurrence_chunk_kernel(const Args a, float* __restrict__ ws) {
           }
       }
     }
+    if (first) {
+      __syncthreads();                                // everyone has met the old n
+      const int d = threadIdx.x;
+      if (d < dim) {
+        float x = s_n[d] * fn;
+        for (int r = 0; r < n; ++r) x = fmaf(s_left[r], __bfloat162float(s_k[r * pitch + d]), x);
+        s_n[d] = x;
+      }
+    }
     __syncthreads();
   }
 
   float* dst = LOCAL ? piece : state;
   if (LOCAL || it.last) {
+    if (first && static_cast<int>(threadIdx.x) < dim) (LOCAL ? piece_n : slot_normaliser(a, it.seg, h))[threadIdx.x] = s_n[threadIdx.x];
+    if (LOCAL && first && threadIdx.x == 0) ws.log_decay[static_cast<size_t>(blockIdx.x) * a.heads + h] = sum;
 #pragma unroll
     for (int t = 0; t < MT; ++t)
 #pragma unroll
@@ -366,8 +475,9 @@ recurrence_chunk_kernel(const Args a, float* __restrict__ ws) {
 }
 
 // Contributions of a segment's pieces -> their initial states (in place).
+template <bool GATED>
 __global__ void __launch_bounds__(256)
-recurrence_scan_kernel(const Args a, float* __restrict__ ws) {
+recurrence_scan_kernel(const Args a, const PieceSpace ws) {
   const int seg = blockIdx.x, h = blockIdx.y;
   int first = 0;
   for (int s = 0; s < seg; ++s) first += (a.cu_rows[s + 1] - a.cu_rows[s] + kPiece - 1) / kPiece;
@@ -375,23 +485,205 @@ recurrence_scan_kernel(const Args a, float* __restrict__ ws) {
   const int pieces = (rows + kPiece - 1) / kPiece;
   if (pieces < 2) return;
   const size_t plane = static_cast<size_t>(a.dim) * a.vdim;
-  const float p64 = a.decay_pow[h * kPowers + 64];
-  const float f = (p64 * p64) * (p64 * p64);
+  float f = 1.f;
+  if (!GATED) {
+    const float p64 = a.decay_pow[h * kPowers + 64];
+    f = (p64 * p64) * (p64 * p64);
+  }
   const bool fresh = a.positions[a.cu_rows[seg]] == 0;
-  const float* state = slot_state(a, seg, h);
-  for (size_t e = static_cast<size_t>(blockIdx.z) * 256 + threadIdx.x; e < plane; e += static_cast<size_t>(gridDim.z) * 256) {
-    float run = fresh ? 0.f : state[e];
-    for (int i = 0; i < pieces; ++i) {
-      float* w = ws + (static_cast<size_t>(first + i) * a.heads + h) * plane + e;
+  auto scan = [&](float* w, size_t stride, float run) {          // w: the first piece's entry
+    for (int i = 0; i < pieces; ++i, w += stride) {
       const float own = i + 1 < pieces ? *w : 0.f;
       *w = run;
+      if (GATED && i + 1 < pieces) f = expf(ws.log_decay[static_cast<size_t>(first + i) * a.heads + h]);
       run = fmaf(run, f, own);
     }
+  };
+  const float* state = slot_state(a, seg, h);
+  for (size_t e = static_cast<size_t>(blockIdx.z) * 256 + threadIdx.x; e < plane; e += static_cast<size_t>(gridDim.z) * 256)
+    scan(ws.state + (static_cast<size_t>(first) * a.heads + h) * plane + e, a.heads * plane, fresh ? 0.f : state[e]);
+  if (GATED && blockIdx.z == 0)
+    for (int d = threadIdx.x; d < a.dim; d += 256)
+      scan(ws.normaliser + (static_cast<size_t>(first) * a.heads + h) * a.dim + d, static_cast<size_t>(a.heads) * a.dim,
+           fresh ? 0.f : slot_normaliser(a, seg, h)[d]);
+}
+
+// ---- matrix memory ---------------------------------------------------------------------------------------------------
+struct Gates {
+  const float* logits;          // [rows, stride]: input gates of all heads, then forget gates
+  long long stride;
+  const float* in_bias;
+  const float* forget_bias;
+  float cap;
+};
+
+__device__ __forceinline__ float log_sigmoid(float z) { return fminf(z, 0.f) - log1pf(expf(-fabsf(z))); }
+__device__ __forceinline__ void log_gates(const Gates& g, int row, int heads, int h, float* in, float* forget) {
+  const float* z = g.logits + static_cast<long long>(row) * g.stride;
+  *in = g.cap * tanhf((z[h] + g.in_bias[h]) / g.cap);
+  *forget = log_sigmoid(g.cap * tanhf((z[heads + h] + g.forget_bias[h]) / g.cap));
+}
+
+// One block per (sequence, head), 256 tokens at a time. m_t = max(m_(t-1) + f_t, i_t) is a scan of pairs
+// (sum of f, maximum): (F1, M1) before (F2, M2) gives (F1 + F2, max(M1 + F2, M2)).
+__global__ void __launch_bounds__(256)
+memory_gates_kernel(const Args a, const Gates g, float* __restrict__ log_decay, float* __restrict__ log_take, float* __restrict__ maximum) {
+  __shared__ float s_f[8], s_m[8], s_top[257];
+  const int seg = blockIdx.x, h = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int row0 = a.cu_rows[seg], row1 = a.cu_rows[seg + 1];
+  if (row0 >= row1) return;
+  float* slot = slot_maximum(a, seg, h);
+  float before = a.positions[row0] == 0 ? 0.f : *slot;
+  for (int base = row0; base < row1; base += 256) {
+    const int row = base + threadIdx.x;
+    float in = -INFINITY, forget = 0.f;
+    if (row < row1) log_gates(g, row, a.heads, h, &in, &forget);
+    float f = forget, m = in;
+#pragma unroll
+    for (int off = 1; off < 32; off <<= 1) {
+      const float fu = __shfl_up_sync(0xffffffffu, f, off), mu = __shfl_up_sync(0xffffffffu, m, off);
+      if (lane >= off) { m = fmaxf(mu + f, m); f += fu; }
+    }
+    if (lane == 31) { s_f[warp] = f; s_m[warp] = m; }
+    __syncthreads();
+    float top = before;                     // the maximum ahead of this warp's tokens
+    for (int w = 0; w < warp; ++w) top = fmaxf(top + s_f[w], s_m[w]);
+    top = fmaxf(top + f, m);
+    s_top[threadIdx.x + 1] = top;
+    if (threadIdx.x == 0) s_top[0] = before;
+    __syncthreads();
+    if (row < row1) {
+      const size_t at = static_cast<size_t>(row) * a.heads + h;
+      log_decay[at] = forget + s_top[threadIdx.x] - top;
+      log_take[at] = in - top;
+      maximum[at] = top;
+    }
+    before = s_top[min(row1 - base, 256)];
+    __syncthreads();
+  }
+  if (threadIdx.x == 0) *slot = before;
+}
+
+// What a head's sums become: o over max(|q . n|, exp(-m)) + 1e-6.
+__device__ __forceinline__ float over_normaliser(float nq, float m) { return 1.f / (fmaxf(fabsf(nq), expf(-m)) + 1e-6f); }
+
+// out = o / rms(o) * weight * sigmoid(gate), a warp per (row, head); o is first divided by its normaliser
+template <typename T, int VEC>
+__global__ void __launch_bounds__(256)
+memory_norm_kernel(const T* __restrict__ o, const float* __restrict__ normaliser, const float* __restrict__ maximum, const T* __restrict__ gate,
+                   long long gate_stride, const float* __restrict__ w, float eps, T* __restrict__ out, int units, int heads, int vdim) {
+  const int unit = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (unit >= units) return;
+  const int row = unit / heads, h = unit % heads;
+  const float by = over_normaliser(normaliser[unit], maximum[unit]);
+  const T* src = o + static_cast<size_t>(unit) * vdim;
+  float ss = 0.f;
+  for (int c = lane * VEC; c < vdim; c += 32 * VEC) {
+    float x[VEC];
+    load_vec<T, VEC>(src + c, x);
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) ss = fmaf(x[i] * by, x[i] * by, ss);
+  }
+  const float inv = by / sqrtf(warp_sum(ss) / static_cast<float>(vdim) + eps);
+  for (int c = lane * VEC; c < vdim; c += 32 * VEC) {
+    float x[VEC], gt[VEC], wv[VEC];
+    load_vec<T, VEC>(src + c, x);
+    load_vec<T, VEC>(gate + static_cast<size_t>(row) * gate_stride + static_cast<size_t>(h) * vdim + c, gt);
+    load_vec<float, VEC>(w + static_cast<size_t>(h) * vdim + c, wv);
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) x[i] = x[i] * inv * wv[i] * sigmoid_exact(gt[i]);
+    store_vec<T, VEC>(out + static_cast<size_t>(unit) * vdim + c, x);
+  }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(256)
+memory_step_kernel(const Args a, const Gates g, const T* __restrict__ gate, long long gate_stride, const float* __restrict__ w, float eps) {
+  __shared__ float4 s_red[256];
+  __shared__ float scratch[32];
+  extern __shared__ float s_kq[];           // [2][dim]
+  const int seg = blockIdx.x, h = blockIdx.y;
+  const int row = a.cu_rows[seg];
+  const int groups_per_row = a.vdim / 4;                 // float4 columns
+  const int lanes_rows = 256 / groups_per_row;           // state rows per pass
+  const int cg = threadIdx.x % groups_per_row, rg = threadIdx.x / groups_per_row;
+  const bool active = rg < lanes_rows;
+  const size_t off = static_cast<size_t>(row) * a.stride;
+  const bool fresh = a.positions[row] == 0;
+  float4* state = reinterpret_cast<float4*>(slot_state(a, seg, h));
+  constexpr int U = 8;                                   // loads in flight per thread
+  float4 s[U];
+  auto fetch = [&](int d0) {
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      const int d = d0 + u * lanes_rows;
+      s[u] = (d < a.dim && !fresh) ? state[static_cast<size_t>(d) * groups_per_row + cg] : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+  };
+  if (active) fetch(rg);                                 // (the state travels while the gates are worked out)
+  float in, forget;
+  log_gates(g, row, a.heads, h, &in, &forget);
+  float* slot_m = slot_maximum(a, seg, h);
+  const float before = fresh ? 0.f : *slot_m;
+  const float top = fmaxf(forget + before, in);
+  const float decay = fresh ? 0.f : expf(forget + before - top), take = expf(in - top);
+  float* slot_n = slot_normaliser(a, seg, h);
+  float nq = 0.f;
+  for (int d = threadIdx.x; d < a.dim; d += 256) {
+    const float k = Elem<T>::ld(static_cast<const T*>(a.k) + off + static_cast<size_t>(h) * a.dim + d) * take;
+    const float q = Elem<T>::ld(static_cast<const T*>(a.q) + off + static_cast<size_t>(h) * a.dim + d) * a.q_scale;
+    s_kq[d] = k;
+    s_kq[a.dim + d] = q;
+    const float n = fmaf(fresh ? 0.f : slot_n[d], decay, k);
+    slot_n[d] = n;
+    nq = fmaf(n, q, nq);
+  }
+  float v[4];
+#pragma unroll
+  for (int i = 0; i < 4; ++i)
+    v[i] = active ? Elem<T>::ld(static_cast<const T*>(a.v) + off + static_cast<size_t>(h) * a.vdim + cg * 4 + i) : 0.f;
+  nq = block_sum_all(nq, scratch);                       // (its barriers also publish s_kq, and everyone has read the maximum)
+  if (threadIdx.x == 0) *slot_m = top;
+  float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
+  for (int d0 = rg; active && d0 < a.dim; d0 += U * lanes_rows) {
+    if (d0 != rg) fetch(d0);
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      const int d = d0 + u * lanes_rows;
+      if (d >= a.dim) break;
+      const float k = s_kq[d], q = s_kq[a.dim + d];
+      s[u].x = fmaf(s[u].x, decay, k * v[0]); s[u].y = fmaf(s[u].y, decay, k * v[1]);
+      s[u].z = fmaf(s[u].z, decay, k * v[2]); s[u].w = fmaf(s[u].w, decay, k * v[3]);
+      state[static_cast<size_t>(d) * groups_per_row + cg] = s[u];
+      o.x = fmaf(s[u].x, q, o.x); o.y = fmaf(s[u].y, q, o.y); o.z = fmaf(s[u].z, q, o.z); o.w = fmaf(s[u].w, q, o.w);
+    }
+  }
+  s_red[threadIdx.x] = o;
+  __syncthreads();
+  float ss = 0.f;
+  if (rg == 0) {
+    for (int r = 1; r < lanes_rows; ++r) {
+      const float4 t = s_red[r * groups_per_row + cg];
+      o.x += t.x; o.y += t.y; o.z += t.z; o.w += t.w;
+    }
+    const float by = over_normaliser(nq, top);
+    o.x *= by; o.y *= by; o.z *= by; o.w *= by;
+    ss = o.x * o.x + o.y * o.y + o.z * o.z + o.w * o.w;
+  }
+  const float inv = 1.f / sqrtf(block_sum_all(ss, scratch) / static_cast<float>(a.vdim) + eps);
+  if (rg == 0) {
+    const size_t col = static_cast<size_t>(h) * a.vdim + cg * 4;
+    const T* gt = gate + static_cast<size_t>(row) * gate_stride + col;
+    T* dst = static_cast<T*>(a.out) + static_cast<size_t>(row) * a.heads * a.vdim + col;
+    const float x[4] = {o.x, o.y, o.z, o.w};
+#pragma unroll
+    for (int i = 0; i < 4; ++i) Elem<T>::st(dst + i, x[i] * inv * w[col + i] * sigmoid_exact(Elem<T>::ld(gt + i)));
   }
 }
 
 bool recurrence_args_ok(const Args& a) {
-  return a.positions && a.cu_rows && a.slots && a.q && a.k && a.v && a.decay_pow && a.state && a.out && a.segments > 0 && a.heads > 0 &&
+  return a.positions && a.cu_rows && a.slots && a.q && a.k && a.v && a.state && a.out &&
+         a.slot_stride >= static_cast<long long>(a.heads) * a.dim * a.vdim + (a.decay_pow ? 0 : static_cast<long long>(a.heads) * (a.dim + 1)) && a.segments > 0 && a.heads > 0 &&
          a.heads <= 65535 && a.dim > 0 && a.vdim > 0 && a.num_slots > 0;
 }
 
@@ -399,15 +691,41 @@ size_t chunk_smem(int dim) {
   return (static_cast<size_t>(2) * kChunk * (dim + 8) + static_cast<size_t>(3) * kChunk * kPitchV + static_cast<size_t>(2) * dim * kPitchV) * 2;
 }
 
-template <int MT, bool LOCAL>
-int launch_chunk(const Args& a, float* ws, cudaStream_t st) {
-  auto kern = recurrence_chunk_kernel<MT, LOCAL>;
+template <int MT, bool LOCAL, bool GATED>
+int launch_chunk(const Args& a, const PieceSpace& ws, cudaStream_t st) {
+  auto kern = recurrence_chunk_kernel<MT, LOCAL, GATED>;
   const size_t smem = chunk_smem(a.dim);
   cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
   if (e != cudaSuccess) return static_cast<int>(e);
   kern<<<dim3(ragged_items(a.rows, a.segments, kPiece), a.heads, (a.vdim + kCols - 1) / kCols), 128, smem, st>>>(a, ws);
   return launch_status();
 }
+
+template <bool GATED>
+int launch_passes(const Args& a, float* workspace, bool pieces, cudaStream_t st) {
+  const PieceSpace ws = piece_space(a, workspace, ragged_items(a.rows, a.segments, kPiece));
+  if (pieces) {
+    const int rc = a.dim <= 64 ? launch_chunk<1, true, GATED>(a, ws, st) : launch_chunk<2, true, GATED>(a, ws, st);
+    if (rc != 0) return rc;
+    const int z = (a.dim * a.vdim + 1023) / 1024;
+    recurrence_scan_kernel<GATED><<<dim3(a.segments, a.heads, z), 256, 0, st>>>(a, ws);
+  }
+  return a.dim <= 64 ? launch_chunk<1, false, GATED>(a, ws, st) : launch_chunk<2, false, GATED>(a, ws, st);
+}
+
+template <typename T, bool GATED>
+int launch_simple(const Args& a, cudaStream_t st) {
+  const size_t smem = (static_cast<size_t>(a.dim) * 35 + 256 + 32) * 4;
+  if (smem > 200 * 1024) return CACHEIR_B200_ELIMIT;
+  const dim3 grid(a.segments, a.heads, (a.vdim + 31) / 32);
+  cudaError_t e = cudaFuncSetAttribute(recurrence_simple_kernel<T, GATED>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
+  if (e != cudaSuccess) return static_cast<int>(e);
+  recurrence_simple_kernel<T, GATED><<<grid, 256, smem, st>>>(a);
+  return launch_status();
+}
+
+bool decay_ok(const Args& a) { return a.decay_pow || (a.log_decay && a.log_take && a.normaliser); }
+bool gates_ok(const Gates& g, int heads) { return g.logits && g.in_bias && g.forget_bias && g.cap > 0.f && g.stride >= 2ll * heads; }
 
 }  // namespace
 }  // namespace cb200
@@ -418,28 +736,17 @@ extern "C" int cacheir_b200_recurrence_simple(const cacheir_b200_recurrence_args
   if (!a) return CACHEIR_B200_EINVAL;
   if (a->rows <= 0) return 0;
   if (!recurrence_args_ok(*a)) return CACHEIR_B200_EINVAL;
-  const size_t smem = (static_cast<size_t>(a->dim) * 34 + 256) * 4;
-  if (smem > 200 * 1024) return CACHEIR_B200_ELIMIT;
-  const dim3 grid(a->segments, a->heads, (a->vdim + 31) / 32);
-  cudaStream_t st = as_stream(stream);
-  if (a->dtype == CACHEIR_B200_F32) {
-    cudaFuncSetAttribute(recurrence_simple_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
-    recurrence_simple_kernel<float><<<grid, 256, smem, st>>>(*a);
-  } else if (a->dtype == CACHEIR_B200_BF16) {
-    cudaFuncSetAttribute(recurrence_simple_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
-    recurrence_simple_kernel<__nv_bfloat16><<<grid, 256, smem, st>>>(*a);
-  } else {
-    return CACHEIR_B200_EUNSUPPORTED;
-  }
-  return launch_status();
+  if (!decay_ok(*a)) return CACHEIR_B200_EINVAL;
+  CB200_HYBRID_DTYPE(a->dtype, return a->decay_pow ? launch_simple<T, false>(*a, as_stream(stream)) : launch_simple<T, true>(*a, as_stream(stream)));
+  return CACHEIR_B200_EUNSUPPORTED;
 }
 
 extern "C" int cacheir_b200_recurrence_step(const cacheir_b200_recurrence_args* a, void* stream) {
   if (!a) return CACHEIR_B200_EINVAL;
   if (a->rows <= 0) return 0;
-  if (!recurrence_args_ok(*a) || a->rows != a->segments) return CACHEIR_B200_EINVAL;
+  if (!recurrence_args_ok(*a) || !a->decay_pow || a->rows != a->segments) return CACHEIR_B200_EINVAL;
   if (a->vdim % 4 != 0 || a->vdim > 1024 || a->dim > 4096) return CACHEIR_B200_EUNSUPPORTED;
-  if (!aligned_to(a->state, 16)) return CACHEIR_B200_EALIGN;
+  if (!aligned_to(a->state, 16) || a->slot_stride % 4 != 0) return CACHEIR_B200_EALIGN;
   const dim3 grid(a->segments, a->heads);
   const size_t smem = static_cast<size_t>(a->dim) * 8;
   if (a->dtype == CACHEIR_B200_F32) recurrence_step_kernel<float><<<grid, 256, smem, as_stream(stream)>>>(*a);
@@ -454,26 +761,64 @@ extern "C" int cacheir_b200_recurrence_chunked_supported(int dim, int vdim, int 
 
 extern "C" size_t cacheir_b200_recurrence_workspace_bytes(int rows, int segments, int heads, int dim, int vdim) {
   if (rows <= kPiece) return 0;
-  return static_cast<size_t>(ragged_items(rows, segments, kPiece)) * heads * dim * vdim * 4;
+  return static_cast<size_t>(ragged_items(rows, segments, kPiece)) * heads * (static_cast<size_t>(dim) * (vdim + 1) + 1) * 4;
 }
 
 extern "C" int cacheir_b200_recurrence_chunked(const cacheir_b200_recurrence_args* a, void* workspace, size_t workspace_bytes, void* stream) {
   if (!a) return CACHEIR_B200_EINVAL;
   if (a->rows <= 0) return 0;
-  if (!recurrence_args_ok(*a)) return CACHEIR_B200_EINVAL;
+  if (!recurrence_args_ok(*a) || !decay_ok(*a)) return CACHEIR_B200_EINVAL;
   if (!cacheir_b200_recurrence_chunked_supported(a->dim, a->vdim, a->dtype)) return CACHEIR_B200_EUNSUPPORTED;
   if (!aligned_to(a->q, 16) || !aligned_to(a->k, 16) || !aligned_to(a->v, 16) || !aligned_to(a->out, 16) || a->stride % 8 != 0 ||
-      !aligned_to(a->state, 16))
+      !aligned_to(a->state, 16) || a->slot_stride % 4 != 0)
     return CACHEIR_B200_EALIGN;
   const size_t need = cacheir_b200_recurrence_workspace_bytes(a->rows, a->segments, a->heads, a->dim, a->vdim);
   if (need > 0 && (!workspace || workspace_bytes < need)) return CACHEIR_B200_EWORKSPACE;
-  cudaStream_t st = as_stream(stream);
   float* ws = static_cast<float*>(workspace);
-  if (need > 0) {
-    const int rc = a->dim <= 64 ? launch_chunk<1, true>(*a, ws, st) : launch_chunk<2, true>(*a, ws, st);
-    if (rc != 0) return rc;
-    const int z = (a->dim * a->vdim + 1023) / 1024;
-    recurrence_scan_kernel<<<dim3(a->segments, a->heads, z), 256, 0, st>>>(*a, ws);
-  }
-  return a->dim <= 64 ? launch_chunk<1, false>(*a, ws, st) : launch_chunk<2, false>(*a, ws, st);
+  return a->decay_pow ? launch_passes<false>(*a, ws, need > 0, as_stream(stream)) : launch_passes<true>(*a, ws, need > 0, as_stream(stream));
 }
+
+extern "C" int cacheir_b200_memory_gates(const cacheir_b200_recurrence_args* a, const float* logits, long long stride, const float* in_bias,
+                                         const float* forget_bias, float cap, float* log_decay, float* log_take, float* maximum, void* stream) {
+  if (!a) return CACHEIR_B200_EINVAL;
+  if (a->rows <= 0) return 0;
+  const Gates g{logits, stride, in_bias, forget_bias, cap};
+  if (!recurrence_args_ok(*a) || a->decay_pow || !gates_ok(g, a->heads) || !log_decay || !log_take || !maximum) return CACHEIR_B200_EINVAL;
+  memory_gates_kernel<<<dim3(a->segments, a->heads), 256, 0, as_stream(stream)>>>(*a, g, log_decay, log_take, maximum);
+  return launch_status();
+}
+
+extern "C" int cacheir_b200_memory_norm(const void* o, const float* normaliser, const float* maximum, const void* gate, long long gate_stride,
+                                        const float* w, float eps, void* out, int rows, int heads, int vdim, int dtype, void* stream) {
+  if (rows <= 0) return 0;
+  if (!o || !normaliser || !maximum || !gate || !w || !out || heads <= 0 || vdim <= 0) return CACHEIR_B200_EINVAL;
+  const int quad = 4 * (dtype == CACHEIR_B200_F32 ? 4 : 2), units = rows * heads;
+  const bool vec = vdim % 4 == 0 && gate_stride % 4 == 0 && aligned_to(o, quad) && aligned_to(gate, quad) && aligned_to(w, 16) && aligned_to(out, quad);
+  const int grid = (units + 7) / 8;
+#define CB200_NORM(VEC)                                                                                                              \
+  memory_norm_kernel<T, VEC><<<grid, 256, 0, as_stream(stream)>>>(static_cast<const T*>(o), normaliser, maximum, static_cast<const T*>(gate), \
+                                                                 gate_stride, w, eps, static_cast<T*>(out), units, heads, vdim)
+  CB200_HYBRID_DTYPE(dtype, {
+    if (vec) CB200_NORM(4);
+    else CB200_NORM(1);
+  });
+#undef CB200_NORM
+  return launch_status();
+}
+
+extern "C" int cacheir_b200_memory_step(const cacheir_b200_recurrence_args* a, const float* logits, long long stride, const float* in_bias,
+                                        const float* forget_bias, float cap, const void* gate, long long gate_stride, const float* w, float eps,
+                                        void* stream) {
+  if (!a) return CACHEIR_B200_EINVAL;
+  if (a->rows <= 0) return 0;
+  const Gates g{logits, stride, in_bias, forget_bias, cap};
+  if (!recurrence_args_ok(*a) || a->decay_pow || !gates_ok(g, a->heads) || !gate || !w || a->rows != a->segments) return CACHEIR_B200_EINVAL;
+  if (a->vdim % 4 != 0 || a->vdim > 1024 || a->dim > 4096) return CACHEIR_B200_EUNSUPPORTED;
+  if (!aligned_to(a->state, 16) || a->slot_stride % 4 != 0) return CACHEIR_B200_EALIGN;
+  const dim3 grid(a->segments, a->heads);
+  const size_t smem = static_cast<size_t>(a->dim) * 8;
+  CB200_HYBRID_DTYPE(a->dtype, (memory_step_kernel<T><<<grid, 256, smem, as_stream(stream)>>>(*a, g, static_cast<const T*>(gate), gate_stride, w, eps)));
+  return launch_status();
+}
+
+extern "C" int cacheir_b200_recurrence_device_status(int) { return 0; }

@@ -1,9 +1,9 @@
-// Tied attention (values are the projected keys) over a paged cache, sm_100a: preparation, the plain form, and decoding.
+// Tied attention (a cached row is key and value) over a paged cache, sm_100a: preparation, the plain form, and decoding.
 //
-// prepare   one warp per head: root mean square, rotation; queries go to a buffer, keys to their cache row.
+// prepare   one warp per head: root mean square, weights, rotation; queries go to a buffer, keys (and values) to their row.
 // simple    any extents, float32 arithmetic: one CTA per (row, head).
 // step      one CTA per (sequence, key/value head, split). Pages of 64 cached rows land in a ring as TMA boxes of 64 columns;
-//           a row is read once and serves as key (columns from rot_dims on, times its reciprocal root mean square) and as
+//           a row is read once and serves as key (columns from key_from on, times its reciprocal root mean square) and as
 //           value (the first dim columns). Four warps take 16 rows of a page each with warp MMAs, the heads of the group
 //           being the 16-row operand; they meet once per CTA, and splits meet in distributed shared memory.
 #include "tied_attention.cuh"
@@ -13,66 +13,128 @@ namespace {
 
 __device__ int g_tied_status = 0;
 
-template <typename T, int VEC>
-__global__ void __launch_bounds__(256)
-tied_prepare_kernel(const cacheir_b200_tied_args a, const T* __restrict__ q, long long q_stride, const T* __restrict__ k, long long k_stride,
-                    float eps, const float2* __restrict__ table, int table_positions, T* __restrict__ q_out) {
-  const int row = blockIdx.x, lane = threadIdx.x & 31;
-  const int unit = blockIdx.y * 8 + (threadIdx.x >> 5);      // query heads, then key heads
-  const int seg = a.row_seg[row], pos = a.positions[row];
-  if (seg < 0 || unit >= a.heads + a.kv_heads || pos < 0 || pos >= table_positions || pos / a.page_size >= a.max_pages) return;
-  const bool key = unit >= a.heads;
-  const int head = key ? unit - a.heads : unit;
-  const T* src = key ? k + static_cast<size_t>(row) * k_stride + static_cast<size_t>(head) * a.dim
-                     : q + static_cast<size_t>(row) * q_stride + static_cast<size_t>(head) * a.dim;
-  const int half = a.rot_dims / 2, lead = tied_lead(a.rot_dims);
-  T *plain, *turned;            // where entry c goes as it is, and rotated entry c
-  float* inv_out = nullptr;
-  if (key) {
-    const int slot = a.page_table[static_cast<size_t>(seg) * a.max_pages + pos / a.page_size];
-    if (slot < 0 || slot >= a.num_slots) return;
-    const size_t at = (static_cast<size_t>(slot) * a.kv_heads + head) * a.page_size + pos % a.page_size;
-    plain = static_cast<T*>(a.pool) + at * (a.dim + a.rot_dims);
-    turned = plain + a.dim;
-    inv_out = a.inv_rms + at;
-  } else {
-    plain = q_out + (static_cast<size_t>(row) * a.heads + head) * (a.dim + a.rot_dims - lead) - lead;
-    turned = plain + a.dim;
+struct PrepareParams {
+  cacheir_b200_tied_args a;
+  long long q_stride, k_stride, v_stride;
+  const float* q_weight;        // per column of a head, or (whole) of the projection; NULL: ones
+  const float* k_weight;
+  const float2* table;
+  int table_positions, rot_dims, head_dim;
+  float eps;
+};
+
+// Entry c of a head: where it stands in a row, as rotated (c < rot_dims) or as projected.
+__device__ __forceinline__ int key_column(const PrepareParams& p, bool tied, int c) {
+  return tied ? (c < p.rot_dims ? p.a.dim + c : c) : p.a.dim + c;
+}
+
+// A warp per head. WHOLE: one block has all heads of a row and its root mean squares run over them; otherwise blocks share a row.
+template <typename T, int VEC, bool WHOLE>
+__global__ void __launch_bounds__(WHOLE ? 512 : 256)
+tied_prepare_kernel(const PrepareParams p, const T* __restrict__ q, const T* __restrict__ k, const T* __restrict__ v, T* __restrict__ q_out) {
+  constexpr int kWarpsHere = (WHOLE ? 512 : 256) / 32;
+  __shared__ float s_part[2][kWarpsHere];
+  const cacheir_b200_tied_args& a = p.a;
+  const int row = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const int seg = a.row_seg[row], pos = a.positions[row], units = a.heads + a.kv_heads;      // query heads, then key heads
+  if (seg < 0 || pos < 0 || pos >= p.table_positions || pos / a.page_size >= a.max_pages) return;
+  const bool tied = v == nullptr;
+  const int d = p.head_dim, half = p.rot_dims / 2, lead = tied_lead(a.key_from), group = a.heads / a.kv_heads;
+  auto source = [&](int unit) {
+    return unit < a.heads ? q + static_cast<size_t>(row) * p.q_stride + static_cast<size_t>(unit) * d
+                          : k + static_cast<size_t>(row) * p.k_stride + static_cast<size_t>(unit - a.heads) * d;
+  };
+  auto squares = [&](const T* src) {
+    float ss = 0.f;
+    for (int c = lane * VEC; c < d; c += 32 * VEC) {
+      float x[VEC];
+      load_vec<T, VEC>(src + c, x);
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) ss = fmaf(x[i], x[i], ss);
+    }
+    return ss;
+  };
+  float inv_q = 0.f, inv_k = 0.f;
+  if (WHOLE) {
+    float part[2] = {0.f, 0.f};
+    for (int u = warp; u < units; u += kWarpsHere) part[u >= a.heads] += squares(source(u));
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+      part[i] = warp_sum(part[i]);
+      if (lane == 0) s_part[i][warp] = part[i];
+    }
+    __syncthreads();
+    float total[2] = {0.f, 0.f};
+    for (int w = 0; w < kWarpsHere; ++w) { total[0] += s_part[0][w]; total[1] += s_part[1][w]; }
+    inv_q = 1.f / sqrtf(total[0] / static_cast<float>(a.heads * d) + p.eps);
+    inv_k = 1.f / sqrtf(total[1] / static_cast<float>(a.kv_heads * d) + p.eps);
   }
-  float ss = 0.f;
-  for (int c = lane * VEC; c < a.dim; c += 32 * VEC) {
-    float v[VEC];
-    load_vec<T, VEC>(src + c, v);
-#pragma unroll
-    for (int i = 0; i < VEC; ++i) ss = fmaf(v[i], v[i], ss);
-  }
-  const float inv = 1.f / sqrtf(warp_sum(ss) / static_cast<float>(a.dim) + eps);
-  const float by = key ? 1.f : inv;        // keys keep their length: the values are the same rows
-  const float2* cs = table + static_cast<size_t>(pos) * half;
-  for (int c = lane * VEC; c < a.dim; c += 32 * VEC) {
-    float v[VEC];
-    load_vec<T, VEC>(src + c, v);
-    if (c < a.rot_dims) {
-      const bool low = c < half;
-      float other[VEC], r[VEC];
-      load_vec<T, VEC>(src + (low ? c + half : c - half), other);
-#pragma unroll
-      for (int i = 0; i < VEC; ++i) {
-        const float2 t = cs[(low ? c : c - half) + i];
-        r[i] = (low ? v[i] * t.x - other[i] * t.y : v[i] * t.x + other[i] * t.y) * by;
-      }
-      store_vec<T, VEC>(turned + c, r);
-      if (!key) {
-#pragma unroll
-        for (int i = 0; i < VEC; ++i) v[i] = 0.f;
+  const int step = WHOLE ? kWarpsHere : units;
+  for (int unit = (WHOLE ? 0 : blockIdx.y * kWarpsHere) + warp; unit < units; unit += step) {
+    const bool key = unit >= a.heads;
+    const int head = key ? unit - a.heads : unit, kv_head = key ? head : head / group;
+    const T* src = source(unit);
+    const float inv = WHOLE ? (key ? inv_k : inv_q) : 1.f / sqrtf(warp_sum(squares(src)) / static_cast<float>(d) + p.eps);
+    // weights of this unit's own norm, and of the key that a query meets
+    const float* own = key ? p.k_weight : p.q_weight;
+    const float* met = p.k_weight;
+    if (WHOLE && own) own += static_cast<size_t>(head) * d;
+    if (WHOLE && met) met += static_cast<size_t>(kv_head) * d;
+    T* dst;
+    if (key) {
+      const int slot = a.page_table[static_cast<size_t>(seg) * a.max_pages + pos / a.page_size];
+      if (slot < 0 || slot >= a.num_slots) continue;
+      const size_t at = (static_cast<size_t>(slot) * a.kv_heads + head) * a.page_size + pos % a.page_size;
+      dst = static_cast<T*>(a.pool) + at * a.width;
+      if (lane == 0) a.inv_rms[at] = inv;
+      if (!tied) {
+        const T* vs = v + static_cast<size_t>(row) * p.v_stride + static_cast<size_t>(head) * a.dim;
+        for (int c = lane * VEC; c < a.dim; c += 32 * VEC) {
+          float x[VEC];
+          load_vec<T, VEC>(vs + c, x);
+          store_vec<T, VEC>(dst + c, x);
+        }
       }
     } else {
-#pragma unroll
-      for (int i = 0; i < VEC; ++i) v[i] *= by;
+      dst = q_out + (static_cast<size_t>(row) * a.heads + head) * (a.width - lead) - lead;
+      const float zero[VEC] = {};
+      for (int c = lead + lane * VEC; c < a.key_from; c += 32 * VEC) store_vec<T, VEC>(dst + c, zero);
     }
-    if (key || c >= lead) store_vec<T, VEC>(plain + c, v);
+    const float by = key ? 1.f : inv;        // keys keep their length: their factor lies beside the row
+    const float2* cs = p.table + static_cast<size_t>(pos) * half;
+    auto weigh = [&](const float* w, int c, float (&x)[VEC]) {
+      if (!w) return;
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) x[i] *= w[c + i];
+    };
+    for (int c = lane * VEC; c < d; c += 32 * VEC) {
+      float x[VEC];
+      load_vec<T, VEC>(src + c, x);
+      if (c < p.rot_dims) {
+        if (key && tied) store_vec<T, VEC>(dst + c, x);          // the value
+        const bool low = c < half;
+        const int oc = low ? c + half : c - half;
+        float other[VEC], r[VEC];
+        load_vec<T, VEC>(src + oc, other);
+        weigh(own, c, x);
+        weigh(own, oc, other);
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) {
+          const float2 t = cs[(low ? c : oc) + i];
+          r[i] = (low ? x[i] * t.x - other[i] * t.y : x[i] * t.x + other[i] * t.y) * by;
+        }
+        store_vec<T, VEC>(dst + key_column(p, tied, c), r);
+      } else {
+        if (!key) {                          // a key's unrotated entries stay as projected: their weights join the query's
+          weigh(own, c, x);
+          weigh(met, c, x);
+#pragma unroll
+          for (int i = 0; i < VEC; ++i) x[i] *= by;
+        }
+        store_vec<T, VEC>(dst + key_column(p, tied, c), x);
+      }
+    }
   }
-  if (key && lane == 0) *inv_out = inv;
 }
 
 // ---- plain form ------------------------------------------------------------------------------------------------------
@@ -82,7 +144,7 @@ tied_simple_kernel(const cacheir_b200_tied_args a, const T* __restrict__ q, cons
                    T* __restrict__ out) {
   extern __shared__ float sm[];
   __shared__ float scratch[32];
-  const int lead = tied_lead(a.rot_dims), width = a.dim + a.rot_dims, qw = width - lead;
+  const int lead = tied_lead(a.key_from), width = a.width, qw = width - lead;
   float* sq = sm;                     // [qw]
   float* so = sq + qw;                // [dim]
   float* sp = so + a.dim;             // [128]
@@ -228,8 +290,8 @@ tied_step_kernel(const __grid_constant__ CUtensorMap tmap, const StepParams p) {
         ptx::mbar_wait(smem_addr(&full[it % p.stages]), (it / p.stages) & 1, &g_tied_status, (8 << 8) | 2);
   } else {
     // ---------------- four warps, 16 keys of every page each ----------------
-    const int width = a.dim + a.rot_dims, lead = tied_lead(a.rot_dims), qw = width - lead;
-    const int k_first = a.rot_dims / 32, last_piece = p.boxes * 2 - 1;      // (a piece behind the row meets zero queries: any data will do)
+    const int width = a.width, lead = tied_lead(a.key_from), qw = width - lead;
+    const int k_first = a.key_from / 32, last_piece = p.boxes * 2 - 1;      // (a piece behind the row meets zero queries: any data will do)
     uint32_t qa[kSteps][2][4];
     const __nv_bfloat16* qb = p.q + (static_cast<size_t>(seg) * a.heads + head0) * qw - lead;
 #pragma unroll
@@ -410,11 +472,11 @@ tied_step_kernel(const __grid_constant__ CUtensorMap tmap, const StepParams p) {
   cluster_sync_all();                      // nobody leaves while its part is being read
 }
 
-int step_boxes(int dim, int rot) { return (dim + rot + 63) / 64; }
+int step_boxes(int width) { return (width + 63) / 64; }
 size_t step_fixed(int stages) { return 1024 + static_cast<size_t>(stages) * kTiedPage * 4 + 2 * kMaxStages * 8; }
 // Two CTAs per SM where at least two pages of each fit.
-int step_stages(int dim, int rot) {
-  const size_t page = static_cast<size_t>(step_boxes(dim, rot)) * kTiedBox;
+int step_stages(int dim, int width) {
+  const size_t page = static_cast<size_t>(step_boxes(width)) * kTiedBox;
   for (size_t limit : {size_t(113) * 1024, size_t(227) * 1024}) {
     if (limit < 200 * 1024 && dim > 128) continue;
     int s = static_cast<int>((limit - step_fixed(kMaxStages)) / page);
@@ -429,7 +491,7 @@ template <int DB, int kSteps>
 int launch_step(const StepParams& p, int segments, cudaStream_t st) {
   const cacheir_b200_tied_args& a = p.a;
   CUtensorMap map;
-  if (!tied_encode(&map, a.pool, a.dim + a.rot_dims, static_cast<uint64_t>(a.num_slots) * a.kv_heads * kTiedPage)) return CACHEIR_B200_EUNSUPPORTED;
+  if (!tied_encode(&map, a.pool, a.width, static_cast<uint64_t>(a.num_slots) * a.kv_heads * kTiedPage)) return CACHEIR_B200_EUNSUPPORTED;
   const size_t smem = step_fixed(p.stages) + static_cast<size_t>(p.stages) * p.boxes * kTiedBox;
   auto kern = tied_step_kernel<DB, kSteps>;
   cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
@@ -451,6 +513,10 @@ int launch_step(const StepParams& p, int segments, cudaStream_t st) {
   return launch_status();
 }
 
+// 32-column pieces of a row that a query meets
+constexpr int kMaxPieces = 9;
+int step_pieces(int width, int key_from) { return (width + 31) / 32 - key_from / 32; }
+
 int head_groups(int group) { return (group + 15) / 16; }
 
 }  // namespace
@@ -462,21 +528,33 @@ int tied_attention_status(bool reset) { return device_status_word(g_tied_status,
 using namespace cb200;
 
 extern "C" int cacheir_b200_tied_prepare(const cacheir_b200_tied_args* args, const void* q, long long q_stride, const void* k,
-                                         long long k_stride, float eps, const float* rope_table, int rope_positions, void* q_out, void* stream) {
+                                         long long k_stride, const void* v, long long v_stride, int rot_dims, int whole,
+                                         const float* q_weight, const float* k_weight, float eps, const float* rope_table,
+                                         int rope_positions, void* q_out, void* stream) {
   if (!args) return CACHEIR_B200_EINVAL;
-  if (args->rows <= 0) return 0;
-  if (!tied_args_ok(*args) || !q || !k || !q_out || (args->rot_dims > 0 && !rope_table) || rope_positions <= 0) return CACHEIR_B200_EINVAL;
-  const float2* table = reinterpret_cast<const float2*>(rope_table);
-  const dim3 grid(args->rows, (args->heads + args->kv_heads + 7) / 8);
+  const cacheir_b200_tied_args& a = *args;
+  if (a.rows <= 0) return 0;
+  if (!tied_args_ok(a) || !q || !k || !q_out || (rot_dims > 0 && !rope_table) || rope_positions <= 0) return CACHEIR_B200_EINVAL;
+  const int d = v ? a.width - a.dim : a.dim;
+  if (d <= 0 || rot_dims < 0 || rot_dims > d || rot_dims % 2 != 0 || a.key_from != (v ? a.dim : rot_dims) || (!v && a.width != a.dim + rot_dims))
+    return CACHEIR_B200_EINVAL;
+  const PrepareParams p{a, q_stride, k_stride, v_stride, q_weight, k_weight, reinterpret_cast<const float2*>(rope_table),
+                        rope_positions, rot_dims, d, eps};
+  const dim3 grid(a.rows, whole ? 1 : (a.heads + a.kv_heads + 7) / 8);
   if (grid.y > 65535) return CACHEIR_B200_ELIMIT;
-  const bool vec = args->dim % 4 == 0 && args->rot_dims % 8 == 0 && q_stride % 4 == 0 && k_stride % 4 == 0 && aligned_to(q, 16) &&
-                   aligned_to(k, 8 * (args->dtype == CACHEIR_B200_F32 ? 2 : 1)) && aligned_to(args->pool, 16) && aligned_to(q_out, 16);
-  CB200_HYBRID_DTYPE(args->dtype, {
-    if (vec) tied_prepare_kernel<T, 4><<<grid, 256, 0, as_stream(stream)>>>(*args, static_cast<const T*>(q), q_stride, static_cast<const T*>(k),
-                                                                           k_stride, eps, table, rope_positions, static_cast<T*>(q_out));
-    else tied_prepare_kernel<T, 1><<<grid, 256, 0, as_stream(stream)>>>(*args, static_cast<const T*>(q), q_stride, static_cast<const T*>(k),
-                                                                       k_stride, eps, table, rope_positions, static_cast<T*>(q_out));
+  const int quad = 4 * (a.dtype == CACHEIR_B200_F32 ? 4 : 2);      // bytes of four elements
+  const bool vec = d % 4 == 0 && a.dim % 4 == 0 && rot_dims % 8 == 0 && q_stride % 4 == 0 && k_stride % 4 == 0 && aligned_to(q, quad) &&
+                   aligned_to(k, quad) && (!v || (v_stride % 4 == 0 && aligned_to(v, quad))) && aligned_to(a.pool, quad) && aligned_to(q_out, quad);
+#define CB200_PREPARE(VEC, WHOLE)                                                                                              \
+  tied_prepare_kernel<T, VEC, WHOLE><<<grid, WHOLE ? 512 : 256, 0, as_stream(stream)>>>(                                        \
+      p, static_cast<const T*>(q), static_cast<const T*>(k), static_cast<const T*>(v), static_cast<T*>(q_out))
+  CB200_HYBRID_DTYPE(a.dtype, {
+    if (vec && whole) CB200_PREPARE(4, true);
+    else if (vec) CB200_PREPARE(4, false);
+    else if (whole) CB200_PREPARE(1, true);
+    else CB200_PREPARE(1, false);
   });
+#undef CB200_PREPARE
   return launch_status();
 }
 
@@ -485,7 +563,7 @@ extern "C" int cacheir_b200_tied_attention_simple(const cacheir_b200_tied_args* 
   if (!args) return CACHEIR_B200_EINVAL;
   if (args->rows <= 0) return 0;
   if (!tied_args_ok(*args) || !q || !out) return CACHEIR_B200_EINVAL;
-  const size_t smem = static_cast<size_t>(2 * args->dim + args->rot_dims - tied_lead(args->rot_dims) + 128) * 4;
+  const size_t smem = static_cast<size_t>(args->dim + args->width - tied_lead(args->key_from) + 128) * 4;
   if (smem > 48 * 1024) return CACHEIR_B200_ELIMIT;
   const dim3 grid(args->rows, args->heads);
   CB200_HYBRID_DTYPE(args->dtype, (tied_simple_kernel<T><<<grid, 128, smem, as_stream(stream)>>>(
@@ -493,9 +571,10 @@ extern "C" int cacheir_b200_tied_attention_simple(const cacheir_b200_tied_args* 
   return launch_status();
 }
 
-extern "C" int cacheir_b200_tied_step_supported(int heads, int kv_heads, int dim, int rot_dims, int page_size, int dtype) {
+extern "C" int cacheir_b200_tied_step_supported(int heads, int kv_heads, int dim, int width, int key_from, int page_size, int dtype) {
   return dtype == CACHEIR_B200_BF16 && page_size == kTiedPage && kv_heads > 0 && heads % kv_heads == 0 && dim >= 8 && dim % 8 == 0 &&
-         dim <= 256 && rot_dims >= 0 && rot_dims % 8 == 0 && rot_dims <= dim && step_stages(dim, rot_dims) > 0 &&
+         dim <= 256 && width >= dim && width % 8 == 0 && key_from >= 0 && key_from % 8 == 0 && key_from < width &&
+         step_pieces(width, key_from) <= kMaxPieces && step_stages(dim, width) > 0 &&
          static_cast<long long>(kv_heads) * head_groups(heads / kv_heads) <= 65535 ? 1 : 0;
 }
 
@@ -515,7 +594,7 @@ extern "C" int cacheir_b200_tied_attention_step(const cacheir_b200_tied_args* ar
   const cacheir_b200_tied_args& a = *args;
   if (a.rows <= 0) return 0;
   if (!tied_args_ok(a) || !q || !out || !a.decode || a.rows != a.segments) return CACHEIR_B200_EINVAL;
-  if (!cacheir_b200_tied_step_supported(a.heads, a.kv_heads, a.dim, a.rot_dims, a.page_size, a.dtype)) return CACHEIR_B200_EUNSUPPORTED;
+  if (!cacheir_b200_tied_step_supported(a.heads, a.kv_heads, a.dim, a.width, a.key_from, a.page_size, a.dtype)) return CACHEIR_B200_EUNSUPPORTED;
   if (!aligned_to(q, 16) || !aligned_to(a.pool, 16) || !aligned_to(a.inv_rms, 16)) return CACHEIR_B200_EALIGN;
   if (splits <= 0) splits = cacheir_b200_tied_step_splits(a.rows, a.heads, a.kv_heads, a.window, a.keep_first, a.max_pages, a.page_size);
   if (splits > kMaxSplits || a.rows > 65535) return CACHEIR_B200_ELIMIT;
@@ -530,14 +609,18 @@ extern "C" int cacheir_b200_tied_attention_step(const cacheir_b200_tied_args* ar
   p.subs = head_groups(group);
   p.heads_per_cta = (group + p.subs - 1) / p.subs;
   p.splits = splits;
-  p.boxes = step_boxes(a.dim, a.rot_dims);
-  p.stages = step_stages(a.dim, a.rot_dims);
+  p.boxes = step_boxes(a.width);
+  p.stages = step_stages(a.dim, a.width);
   cudaStream_t st = as_stream(stream);
-  const bool odd = (a.dim + a.rot_dims + 31) / 32 - a.rot_dims / 32 > (a.dim + 63) / 64 * 2;
+  const int pieces = step_pieces(a.width, a.key_from);
   switch ((a.dim + 63) / 64) {
-    case 1: return odd ? launch_step<1, 3>(p, a.rows, st) : launch_step<1, 2>(p, a.rows, st);
-    case 2: return odd ? launch_step<2, 5>(p, a.rows, st) : launch_step<2, 4>(p, a.rows, st);
-    case 3: return odd ? launch_step<3, 7>(p, a.rows, st) : launch_step<3, 6>(p, a.rows, st);
-    default: return odd ? launch_step<4, 9>(p, a.rows, st) : launch_step<4, 8>(p, a.rows, st);
+    case 1: return pieces <= 2 ? launch_step<1, 2>(p, a.rows, st) : pieces == 3 ? launch_step<1, 3>(p, a.rows, st)
+                 : pieces <= 5 ? launch_step<1, 5>(p, a.rows, st) : launch_step<1, kMaxPieces>(p, a.rows, st);
+    case 2: return pieces <= 2 ? launch_step<2, 2>(p, a.rows, st) : pieces <= 4 ? launch_step<2, 4>(p, a.rows, st)
+                 : pieces == 5 ? launch_step<2, 5>(p, a.rows, st) : launch_step<2, kMaxPieces>(p, a.rows, st);
+    case 3: return pieces <= 3 ? launch_step<3, 3>(p, a.rows, st) : pieces <= 6 ? launch_step<3, 6>(p, a.rows, st)
+                 : pieces == 7 ? launch_step<3, 7>(p, a.rows, st) : launch_step<3, kMaxPieces>(p, a.rows, st);
+    default: return pieces <= 4 ? launch_step<4, 4>(p, a.rows, st) : pieces <= 8 ? launch_step<4, 8>(p, a.rows, st)
+                 : launch_step<4, kMaxPieces>(p, a.rows, st);
   }
 }

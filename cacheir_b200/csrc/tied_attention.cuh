@@ -12,7 +12,7 @@ constexpr int kTiedBox = kTiedPage * 128;        // 64 rows x 64 columns, 128-by
 constexpr float kLog2e = 1.4426950408889634f;
 
 // Columns of a cached row that prepared queries leave out: whole 64-column boxes of which they would be zero.
-__host__ __device__ inline int tied_lead(int rot_dims) { return rot_dims / 64 * 64; }
+__host__ __device__ inline int tied_lead(int key_from) { return key_from / 64 * 64; }
 
 __device__ __forceinline__ float tied_ex2(float x) {
   float y;
@@ -64,8 +64,8 @@ inline bool tied_encode(CUtensorMap* map, const void* base, uint64_t width, uint
 
 inline bool tied_args_ok(const cacheir_b200_tied_args& a) {
   return a.positions && a.row_seg && a.page_table && a.pool && a.inv_rms && a.segments > 0 && a.max_pages > 0 && a.page_size > 0 &&
-         a.num_slots > 0 && a.heads > 0 && a.kv_heads > 0 && a.heads % a.kv_heads == 0 && a.dim > 0 && a.rot_dims >= 0 && a.rot_dims <= a.dim &&
-         a.rot_dims % 2 == 0 && a.window > 0 && a.keep_first >= 0 && a.heads <= 65535;
+         a.num_slots > 0 && a.heads > 0 && a.kv_heads > 0 && a.heads % a.kv_heads == 0 && a.dim > 0 && a.dim <= a.width && a.key_from >= 0 &&
+         a.key_from < a.width && a.window > 0 && a.keep_first >= 0 && a.heads <= 65535;
 }
 
 }  // namespace cb200

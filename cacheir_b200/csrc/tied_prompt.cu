@@ -7,7 +7,7 @@
 // A softmax thread owns a row (a tensor-memory lane), so row sums need no exchange.
 //   warp 0  copies      warp 1  MMA issue, tensor memory      warps 2..5, 6..9  softmax of tile 0, tile 1 (lane quarter = warp % 4)
 //
-// Queries and keys have unit root mean square, so |score| <= bound is known before any key is read. While exp(-2 bound) is
+// Where queries and keys have a known length (`reach`), |score| <= bound is known before any key is read. While exp(-2 bound) is
 // far from underflow the softmax refers to the bound itself (FIXED): no running maximum, no rescaling. Otherwise a row's
 // reference follows its maximum, and O is rescaled when that has grown by more than 2^8. The bound also makes the capped
 // score a polynomial on a known interval: an odd one of five or eight terms, interpolated at Chebyshev nodes (TERMS).
@@ -422,13 +422,13 @@ tied_prompt_kernel(const __grid_constant__ CUtensorMap tmap_kv, const __grid_con
 
 constexpr size_t kSmemLimit = 227 * 1024;
 int prompt_tiles(int dim) { return dim <= 128 ? 2 : 1; }
-int row_boxes(int dim, int rot) { return (dim + rot + 63) / 64; }
-size_t prompt_fixed(int dim, int rot) {
+int row_boxes(int width) { return (width + 63) / 64; }
+size_t prompt_fixed(int dim, int width, int key_from) {
   const int tiles = prompt_tiles(dim);
-  return 1024 + static_cast<size_t>(tiles) * (row_boxes(dim, rot) - rot / 64 + 2) * kTile * 128 + kMaxStages * kTiedPage * 4 + (2 * kMaxStages + 13) * 8 + 16;
+  return 1024 + static_cast<size_t>(tiles) * (row_boxes(width) - key_from / 64 + 2) * kTile * 128 + kMaxStages * kTiedPage * 4 + (2 * kMaxStages + 13) * 8 + 16;
 }
-int prompt_stages(int dim, int rot) {
-  const size_t fixed = prompt_fixed(dim, rot), page = static_cast<size_t>(row_boxes(dim, rot)) * kTiedBox;
+int prompt_stages(int dim, int width, int key_from) {
+  const size_t fixed = prompt_fixed(dim, width, key_from), page = static_cast<size_t>(row_boxes(width)) * kTiedBox;
   const int s = fixed > kSmemLimit ? 0 : static_cast<int>((kSmemLimit - fixed) / page);
   return s > kMaxStages ? kMaxStages : (s >= 2 ? s : 0);
 }
@@ -460,13 +460,13 @@ int fit_tanh(double cap2, double reach, float (&coef)[kTerms]) {
 template <int TILES, bool FIXED, int TERMS>
 int launch_prompt(const PromptParams& p, const void* q, int items, cudaStream_t st) {
   const cacheir_b200_tied_args& a = p.a;
-  size_t smem = prompt_fixed(a.dim, a.rot_dims) + static_cast<size_t>(p.stages) * p.boxes * kTiedBox;
+  size_t smem = prompt_fixed(a.dim, a.width, a.key_from) + static_cast<size_t>(p.stages) * p.boxes * kTiedBox;
   const size_t least = kSmemLimit / 2 + 1024;           // one CTA per SM: one that waited for tensor memory would be late
   if (smem < least) smem = least;
   CUtensorMap tkv, tq;
-  if (!tied_encode(&tkv, a.pool, a.dim + a.rot_dims, static_cast<uint64_t>(a.num_slots) * a.kv_heads * kTiedPage)) return CACHEIR_B200_EUNSUPPORTED;
+  if (!tied_encode(&tkv, a.pool, a.width, static_cast<uint64_t>(a.num_slots) * a.kv_heads * kTiedPage)) return CACHEIR_B200_EUNSUPPORTED;
   ptx::EncodeTiledFn fn = ptx::tensor_map_encoder();
-  const cuuint64_t qw = a.dim + a.rot_dims - tied_lead(a.rot_dims);
+  const cuuint64_t qw = a.width - tied_lead(a.key_from);
   const cuuint64_t dims[3] = {qw, static_cast<cuuint64_t>(a.heads), static_cast<cuuint64_t>(a.rows)};
   const cuuint64_t strides[2] = {qw * 2, qw * 2 * a.heads};
   const cuuint32_t box[3] = {64, static_cast<cuuint32_t>(p.heads_per_cta), static_cast<cuuint32_t>(p.tokens_per_tile)};
@@ -497,9 +497,10 @@ int tied_prompt_status(bool reset) { return device_status_word(g_prompt_status, 
 
 using namespace cb200;
 
-extern "C" int cacheir_b200_tied_prompt_supported(int heads, int kv_heads, int dim, int rot_dims, int page_size, int dtype) {
+extern "C" int cacheir_b200_tied_prompt_supported(int heads, int kv_heads, int dim, int width, int key_from, int page_size, int dtype) {
   return dtype == CACHEIR_B200_BF16 && page_size == kTiedPage && kv_heads > 0 && heads % kv_heads == 0 && dim >= 8 && dim % 8 == 0 &&
-         dim <= 256 && rot_dims >= 0 && rot_dims % 8 == 0 && rot_dims <= dim && prompt_stages(dim, rot_dims) > 0 ? 1 : 0;
+         dim <= 256 && width >= dim && width % 8 == 0 && key_from >= 0 && key_from % 8 == 0 && key_from < width &&
+         prompt_stages(dim, width, key_from) > 0 ? 1 : 0;
 }
 
 extern "C" int cacheir_b200_tied_attention_prompt(const cacheir_b200_tied_args* args, const void* q, const void* gate, long long gate_stride,
@@ -508,7 +509,7 @@ extern "C" int cacheir_b200_tied_attention_prompt(const cacheir_b200_tied_args* 
   const cacheir_b200_tied_args& a = *args;
   if (a.rows <= 0) return 0;
   if (!tied_args_ok(a) || !q || !out || !a.cu_rows) return CACHEIR_B200_EINVAL;
-  if (!cacheir_b200_tied_prompt_supported(a.heads, a.kv_heads, a.dim, a.rot_dims, a.page_size, a.dtype)) return CACHEIR_B200_EUNSUPPORTED;
+  if (!cacheir_b200_tied_prompt_supported(a.heads, a.kv_heads, a.dim, a.width, a.key_from, a.page_size, a.dtype)) return CACHEIR_B200_EUNSUPPORTED;
   if (!aligned_to(q, 16) || !aligned_to(a.pool, 16) || !aligned_to(a.inv_rms, 16) || !aligned_to(out, 16) ||
       (gate && (!aligned_to(gate, 16) || gate_stride % 8 != 0)))
     return CACHEIR_B200_EALIGN;
@@ -518,13 +519,13 @@ extern "C" int cacheir_b200_tied_attention_prompt(const cacheir_b200_tied_args* 
   p.gate_stride = gate_stride;
   p.out = static_cast<__nv_bfloat16*>(out);
   p.score = tied_score(a.scale, a.cap);
-  // unit root mean squares, and a little room for the operands' rounding
-  const double most = a.dim * 1.02, reach = most * fabs(static_cast<double>(a.scale));
+  // a little room for the operands' rounding
+  const double most = a.reach * 1.02, reach = most * fabs(static_cast<double>(a.scale));
   const double bound = a.cap > 0.f ? a.cap * tanh(reach / a.cap) : reach;
   p.bound = static_cast<float>(bound * kLog2e);
-  const bool fixed = 2.0 * bound * kLog2e <= 100.0;
+  const bool fixed = a.reach > 0.f && 2.0 * bound * kLog2e <= 100.0;
   int terms = 0;
-  if (a.cap > 0.f) {
+  if (a.cap > 0.f && fixed) {
     p.pre = static_cast<float>((a.scale < 0.f ? -1.0 : 1.0) / most);
     terms = fit_tanh(static_cast<double>(a.cap) * kLog2e, reach / a.cap, p.coef);
   }
@@ -532,9 +533,9 @@ extern "C" int cacheir_b200_tied_attention_prompt(const cacheir_b200_tied_args* 
   p.subs = (group + kTile - 1) / kTile;
   p.heads_per_cta = (group + p.subs - 1) / p.subs;
   p.tokens_per_tile = kTile / p.heads_per_cta;
-  p.boxes = row_boxes(a.dim, a.rot_dims);
-  p.lead_boxes = a.rot_dims / 64;
-  p.stages = prompt_stages(a.dim, a.rot_dims);
+  p.boxes = row_boxes(a.width);
+  p.lead_boxes = a.key_from / 64;
+  p.stages = prompt_stages(a.dim, a.width, a.key_from);
   p.n_cols = (a.dim + 15) / 16 * 16;
   const int cols = tiles * (p.n_cols + 2 * kTiedPage);
   p.tmem_cols = cols <= 128 ? 128 : cols <= 256 ? 256 : 512;

@@ -1,4 +1,5 @@
-"""Torch-tensor wrappers over the C ABI of the ragged families (include/cacheir_b200_ragged.h, cacheir_b200_hybrid.h).
+"""Torch-tensor wrappers over the C ABI of the ragged families (include/cacheir_b200_ragged.h, cacheir_b200_hybrid.h,
+cacheir_b200_recurrence.h).
 
 Same rules as `ops`: validate, pass device pointers on the current stream, raise on a non-zero status. The residual
 stream and every norm parameter are float32; activations are float32 or bfloat16.
@@ -14,7 +15,7 @@ from . import _lib
 from ._lib import DenseArgs, LatentArgs, RecurrenceArgs, check
 from .ops import _ptr, _require_cuda, _stream, dtype_code
 
-NEXT_NONE, NEXT_COPY, NEXT_DYT = 0, 1, 2
+NEXT_NONE, NEXT_COPY, NEXT_DYT, NEXT_RMS = range(4)
 (DENSE_PLAIN, DENSE_F32, DENSE_SILU, DENSE_GEGLU, DENSE_GATED, DENSE_RESIDUAL, DENSE_GELU_EMBED, DENSE_SWIGLU,
  DENSE_CLAMPED_GLU) = range(9)
 GLU_EPILOGUES = {"gelu_tanh": DENSE_GEGLU, "silu": DENSE_SWIGLU, "clamped": DENSE_CLAMPED_GLU}
@@ -31,15 +32,19 @@ class DynamicTanh:
 
 
 @dataclass
+class RmsNorm:
+    """x / sqrt(mean(x^2) + eps) * weight; weight float32 on the device."""
+
+    weight: torch.Tensor
+    eps: float
+
+
+@dataclass
 class Next:
-    """What a kernel that finishes the residual leaves in `out`: the residual itself or its Dynamic Tanh."""
+    """What a kernel that finishes the residual leaves in `out`: the residual itself, its Dynamic Tanh, or its RMS norm."""
 
     out: torch.Tensor
-    norm: DynamicTanh | None = None
-
-    @property
-    def mode(self) -> int:
-        return NEXT_COPY if self.norm is None else NEXT_DYT
+    norm: DynamicTanh | RmsNorm | None = None
 
 
 @dataclass
@@ -67,6 +72,9 @@ def _next(nx: Next | None) -> tuple:
         return (NEXT_NONE, None, None, 0.0, None)
     if nx.norm is None:
         return (NEXT_COPY, None, None, 0.0, nx.out.data_ptr())
+    if isinstance(nx.norm, RmsNorm):
+        _f32(nx.norm.weight)
+        return (NEXT_RMS, nx.norm.weight.data_ptr(), None, float(nx.norm.eps), nx.out.data_ptr())
     return (NEXT_DYT, nx.norm.weight.data_ptr(), nx.norm.bias.data_ptr(), float(nx.norm.alpha), nx.out.data_ptr())
 
 
@@ -87,8 +95,8 @@ def dense_gemm(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor | None = None
                ids: torch.Tensor | None = None, table: torch.Tensor | None = None, table_col: int = 0,
                bias: torch.Tensor | None = None, limit: float = 0.0, tail: torch.Tensor | None = None) -> None:
     """Tensor-core Y = f(X W^T + bias). x [T, >=K] and w [N, K] bf16 with dense rows. `batch` > 1: w [batch*N, K], entry z
-    reads x columns from z*x_batch_cols and writes output columns from z*y_batch_cols (default z*N). `tail` (paired
-    epilogues): the last columns of the product go there as float32."""
+    reads x columns from z*x_batch_cols and writes output columns from z*y_batch_cols (default z*N). `tail` (plain, SiLU and
+    paired epilogues): the last columns of the product go there as float32."""
     _require_cuda(x, w, out, gate, residual, ids, table)
     if x.dtype != torch.bfloat16 or w.dtype != torch.bfloat16 or x.stride(1) != 1 or w.stride(1) != 1:
         raise ValueError("dense_gemm takes bf16 x and w with dense rows")
@@ -108,10 +116,10 @@ def dense_gemm(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor | None = None
     else:
         paired = epilogue in GLU_EPILOGUES.values()
         if tail is not None:
-            if not paired or tail.dtype != torch.float32 or tail.stride(1) != 1 or int(tail.shape[0]) != a.T:
-                raise ValueError("tail is a float32 [T, columns] tensor of a paired epilogue")
+            if not (paired or epilogue in (DENSE_PLAIN, DENSE_SILU)) or tail.dtype != torch.float32 or tail.stride(1) != 1 or int(tail.shape[0]) != a.T:
+                raise ValueError("tail is a float32 [T, columns] tensor of a plain, SiLU or paired epilogue")
             a.tail, a.tail_cols, a.tail_stride = tail.data_ptr(), int(tail.shape[1]), tail.stride(0)
-        cols = (a.N - a.tail_cols) // 2 if paired else a.y_batch_cols * (batch - 1) + a.N
+        cols = (a.N - a.tail_cols) // 2 if paired else a.y_batch_cols * (batch - 1) + a.N - a.tail_cols
         want = torch.float32 if epilogue == DENSE_F32 else torch.bfloat16
         if out is None or out.dtype != want or int(out.shape[0]) != a.T or int(out.shape[1]) < cols or out.stride(1) != 1:
             raise ValueError("out must be [T, N] of the epilogue's type with dense rows")
@@ -146,14 +154,16 @@ def dense_simple(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, *, batch: 
     return out
 
 
-def scaled_embedding(table: torch.Tensor, ids: torch.Tensor, residual: torch.Tensor, scale: float, nx: Next | None = None) -> None:
+def scaled_embedding(table: torch.Tensor, ids: torch.Tensor, residual: torch.Tensor, scale: float, nx: Next | None = None, *,
+                     accumulate: bool = False) -> None:
+    """residual = table[ids] * scale, or (`accumulate`) that much more."""
     _require_cuda(table, ids, residual)
     _f32(residual)
     if ids.dtype != torch.int64 or not table.is_contiguous() or residual.shape[1] != table.shape[1]:
         raise ValueError("scaled_embedding expects int64 ids and a contiguous [vocab, width] table")
     check(_lib.load_group("ragged").cacheir_b200_scaled_embedding(
         table.data_ptr(), ids.data_ptr(), residual.data_ptr(), int(residual.shape[0]), int(table.shape[1]), int(table.shape[0]),
-        float(scale), *_next(nx), dtype_code(table.dtype), _stream()), "scaled_embedding")
+        float(scale), int(accumulate), *_next(nx), dtype_code(table.dtype), _stream()), "scaled_embedding")
 
 
 def dyt_rows(residual: torch.Tensor, norm: DynamicTanh, out: torch.Tensor, row_index: torch.Tensor | None = None) -> torch.Tensor:
@@ -184,6 +194,28 @@ def residual_dyt(residual: torch.Tensor, y: torch.Tensor, norm: DynamicTanh, nx:
     check(_lib.load_group("ragged").cacheir_b200_residual_dyt(
         residual.data_ptr(), y.data_ptr(), norm.weight.data_ptr(), norm.bias.data_ptr(), float(norm.alpha), int(y.shape[0]),
         int(y.shape[1]), *_next(nx), dtype_code(y.dtype), _stream()), "residual_dyt")
+
+
+def residual_add(residual: torch.Tensor, y: torch.Tensor, nx: Next | None = None) -> None:
+    """residual += y"""
+    _require_cuda(residual, y)
+    _f32(residual)
+    if y.shape != residual.shape or not y.is_contiguous():
+        raise ValueError("y must be a contiguous tensor of the residual's shape")
+    check(_lib.load_group("ragged").cacheir_b200_residual_add(
+        residual.data_ptr(), y.data_ptr(), int(y.shape[0]), int(y.shape[1]), *_next(nx), dtype_code(y.dtype), _stream()), "residual_add")
+
+
+def residual_rms_pair(residual: torch.Tensor, y1: torch.Tensor, w1: torch.Tensor, y2: torch.Tensor, w2: torch.Tensor, factor: float, eps: float,
+                      nx: Next | None = None) -> None:
+    """residual += factor * (rms_norm(y1) * w1 + rms_norm(y2) * w2)"""
+    _require_cuda(residual, y1, y2, w1, w2)
+    _f32(residual, w1, w2)
+    if any(y.shape != residual.shape or not y.is_contiguous() or y.dtype != y1.dtype for y in (y1, y2)):
+        raise ValueError("y1 and y2 must be contiguous tensors of the residual's shape and one type")
+    check(_lib.load_group("ragged").cacheir_b200_residual_rms_pair(
+        residual.data_ptr(), y1.data_ptr(), w1.data_ptr(), y2.data_ptr(), w2.data_ptr(), float(factor), float(eps), int(y1.shape[0]),
+        int(y1.shape[1]), *_next(nx), dtype_code(y1.dtype), _stream()), "residual_rms_pair")
 
 
 def residual_rms(residual: torch.Tensor, y: torch.Tensor, weight: torch.Tensor, eps: float, nx: Next | None = None) -> None:
@@ -299,43 +331,108 @@ def decay_powers(decay, device: torch.device | str) -> torch.Tensor:
     return torch.pow(d[:, None], e[None, :]).to(torch.float32).contiguous().to(device)
 
 
-def recurrence_args(rows: Rows, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, powers: torch.Tensor, state: torch.Tensor,
-                    out: torch.Tensor, *, heads: int, dim: int, vdim: int) -> RecurrenceArgs:
-    """q, k [T, heads*dim] and v [T, heads*vdim] with one common row stride; state [slots, heads, dim, vdim] float32."""
+def recurrence_args(rows: Rows, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, powers: torch.Tensor | None, state: torch.Tensor,
+                    out: torch.Tensor, *, heads: int, dim: int, vdim: int, gated: tuple[torch.Tensor, torch.Tensor, torch.Tensor] | None = None,
+                    q_scale: float = 1.0) -> RecurrenceArgs:
+    """q, k [T, heads*dim] and v [T, heads*vdim] with one common row stride. Constant decays: state [slots, heads, dim, vdim]
+    float32. Without `powers` the recurrence is gated: state [slots, memory_state_size(...)], and `gated` = (log_decay,
+    log_take, normaliser), [T, heads] float32 each (not needed by memory_step)."""
     _require_cuda(q, k, v, powers, state, out)
-    _f32(powers, state)
+    _f32(state, *([] if powers is None else [powers]), *(gated or ()))
     if not (q.stride(0) == k.stride(0) == v.stride(0)) or q.stride(1) != 1 or k.stride(1) != 1 or v.stride(1) != 1:
         raise ValueError("q, k and v must share one row stride and have dense rows")
-    if tuple(state.shape[1:]) != (heads, dim, vdim) or tuple(powers.shape) != (heads, RECURRENCE_POWERS) or not out.is_contiguous():
+    if not out.is_contiguous() or (powers is not None and (tuple(state.shape[1:]) != (heads, dim, vdim) or tuple(powers.shape) != (heads, RECURRENCE_POWERS))):
         raise ValueError("state must be [slots, heads, dim, vdim], powers [heads, 65] and out contiguous")
+    if powers is None and tuple(state.shape[1:]) != (memory_state_size(heads, dim, vdim),):
+        raise ValueError("a gated recurrence's state must be [slots, memory_state_size]")
+    if gated is not None and any(tuple(t.shape) != (rows.rows, heads) for t in gated):
+        raise ValueError("log_decay, log_take and normaliser are [rows, heads]")
     a = RecurrenceArgs()
     a.positions, a.cu_rows, a.slots = rows.positions.data_ptr(), rows.cu_rows.data_ptr(), rows.slots.data_ptr()
     a.rows, a.segments, a.heads, a.dim, a.vdim = rows.rows, rows.segments, heads, dim, vdim
     a.q, a.k, a.v, a.stride = q.data_ptr(), k.data_ptr(), v.data_ptr(), q.stride(0)
-    a.decay_pow, a.state, a.num_slots, a.out, a.dtype = powers.data_ptr(), state.data_ptr(), int(state.shape[0]), out.data_ptr(), dtype_code(q.dtype)
+    a.decay_pow, a.state, a.num_slots, a.out, a.dtype = _ptr(powers), state.data_ptr(), int(state.shape[0]), out.data_ptr(), dtype_code(q.dtype)
+    a.slot_stride, a.q_scale = state.stride(0), float(q_scale)
+    if gated is not None:
+        a.log_decay, a.log_take, a.normaliser = (t.data_ptr() for t in gated)
     return a
 
 
 def recurrence_simple(a: RecurrenceArgs) -> None:
-    check(_lib.load_group("hybrid").cacheir_b200_recurrence_simple(ctypes.byref(a), _stream()), "recurrence_simple")
+    check(_lib.load_group("recurrence").cacheir_b200_recurrence_simple(ctypes.byref(a), _stream()), "recurrence_simple")
 
 
 def recurrence_step(a: RecurrenceArgs) -> None:
-    check(_lib.load_group("hybrid").cacheir_b200_recurrence_step(ctypes.byref(a), _stream()), "recurrence_step")
+    check(_lib.load_group("recurrence").cacheir_b200_recurrence_step(ctypes.byref(a), _stream()), "recurrence_step")
 
 
 def recurrence_chunked_supported(dim: int, vdim: int, dtype: torch.dtype) -> bool:
-    return bool(_lib.load_group("hybrid").cacheir_b200_recurrence_chunked_supported(dim, vdim, dtype_code(dtype)))
+    return bool(_lib.load_group("recurrence").cacheir_b200_recurrence_chunked_supported(dim, vdim, dtype_code(dtype)))
 
 
 def recurrence_workspace_bytes(rows: int, segments: int, heads: int, dim: int, vdim: int) -> int:
-    return int(_lib.load_group("hybrid").cacheir_b200_recurrence_workspace_bytes(rows, segments, heads, dim, vdim))
+    return int(_lib.load_group("recurrence").cacheir_b200_recurrence_workspace_bytes(rows, segments, heads, dim, vdim))
 
 
 def recurrence_chunked(a: RecurrenceArgs, workspace: torch.Tensor | None) -> None:
-    check(_lib.load_group("hybrid").cacheir_b200_recurrence_chunked(
+    check(_lib.load_group("recurrence").cacheir_b200_recurrence_chunked(
         ctypes.byref(a), _ptr(workspace), 0 if workspace is None else workspace.numel() * workspace.element_size(), _stream()),
         "recurrence_chunked")
+
+
+# ---- matrix memory -------------------------------------------------------------------------------------------------------
+def memory_state_size(heads: int, dim: int, vdim: int) -> int:
+    """float32 entries of one sequence's state: matrices, normalisers, running maxima; whole 16-byte pieces."""
+    return (heads * (dim * vdim + dim + 1) + 3) // 4 * 4
+
+
+@dataclass
+class MemoryGates:
+    """Gate logits [T, 2*heads] float32 (input gates, then forget gates), their biases [heads] and the cap."""
+
+    logits: torch.Tensor
+    in_bias: torch.Tensor
+    forget_bias: torch.Tensor
+    cap: float
+
+    def args(self) -> tuple:
+        _require_cuda(self.logits, self.in_bias, self.forget_bias)
+        _f32(self.in_bias, self.forget_bias)
+        if self.logits.dtype != torch.float32 or self.logits.stride(1) != 1 or int(self.logits.shape[1]) != 2 * self.in_bias.numel():
+            raise ValueError("gate logits are float32 [T, 2*heads] with dense rows")
+        return (self.logits.data_ptr(), self.logits.stride(0), self.in_bias.data_ptr(), self.forget_bias.data_ptr(), float(self.cap))
+
+
+def memory_gates(a: RecurrenceArgs, gates: MemoryGates, log_decay: torch.Tensor, log_take: torch.Tensor, maximum: torch.Tensor) -> None:
+    _require_cuda(log_decay, log_take, maximum)
+    check(_lib.load_group("recurrence").cacheir_b200_memory_gates(
+        ctypes.byref(a), *gates.args(), log_decay.data_ptr(), log_take.data_ptr(), maximum.data_ptr(), _stream()), "memory_gates")
+
+
+def _memory_gate(gate: torch.Tensor, weight: torch.Tensor, columns: int) -> None:
+    _require_cuda(gate, weight)
+    _f32(weight)
+    if gate.stride(1) != 1 or int(gate.shape[1]) != columns or weight.numel() != columns:
+        raise ValueError("the output gate and the norm weight have one column per output column")
+
+
+def memory_norm(o: torch.Tensor, normaliser: torch.Tensor, maximum: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, eps: float,
+                out: torch.Tensor, *, heads: int, vdim: int) -> torch.Tensor:
+    _require_cuda(o, normaliser, maximum, out)
+    _f32(normaliser, maximum)
+    _memory_gate(gate, weight, heads * vdim)
+    if not o.is_contiguous() or not out.is_contiguous() or o.shape != out.shape or int(o.shape[1]) != heads * vdim:
+        raise ValueError("memory_norm expects contiguous [T, heads*vdim] o and out")
+    check(_lib.load_group("recurrence").cacheir_b200_memory_norm(
+        o.data_ptr(), normaliser.data_ptr(), maximum.data_ptr(), gate.data_ptr(), gate.stride(0), weight.data_ptr(), float(eps), out.data_ptr(),
+        int(o.shape[0]), heads, vdim, dtype_code(o.dtype), _stream()), "memory_norm")
+    return out
+
+
+def memory_step(a: RecurrenceArgs, gates: MemoryGates, gate: torch.Tensor, weight: torch.Tensor, eps: float) -> None:
+    _memory_gate(gate, weight, a.heads * a.vdim)
+    check(_lib.load_group("recurrence").cacheir_b200_memory_step(
+        ctypes.byref(a), *gates.args(), gate.data_ptr(), gate.stride(0), weight.data_ptr(), float(eps), _stream()), "memory_step")
 
 
 def device_status(reset: bool = True) -> int:

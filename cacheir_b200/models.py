@@ -6,7 +6,7 @@ from dataclasses import dataclass
 from pathlib import Path
 from typing import Any, Callable
 
-from . import gutorax, topunex
+from . import gutorax, rekodra, topunex
 from .artifact import CompileArtifact, ModelConfig, build_decoder_artifact
 
 
@@ -48,5 +48,7 @@ def load_model(path: str | Path, *, quant: str | None = None) -> CompileArtifact
     return family.build_artifact(family.config_from_dict(data), model_path=str(folder), quant=quant)
 
 
-register_family(gutorax.ARCHITECTURE, ModelFamily("gutorax", gutorax.GutoraxConfig.from_dict, gutorax.build_gutorax_artifact, ("ragged", "hybrid")))
+register_family(gutorax.ARCHITECTURE, ModelFamily("gutorax", gutorax.GutoraxConfig.from_dict, gutorax.build_gutorax_artifact, ("ragged", "hybrid", "recurrence")))
 register_family(topunex.ARCHITECTURE, ModelFamily("topunex", topunex.TopunexConfig.from_dict, topunex.build_topunex_artifact, ("ragged", "experts")))
+register_family(rekodra.ARCHITECTURE, ModelFamily("rekodra", rekodra.RekodraConfig.from_dict, rekodra.build_rekodra_artifact,
+                                                  ("ragged", "recurrence", "experts")))

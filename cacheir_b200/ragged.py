@@ -29,6 +29,7 @@ def bucket(n: int) -> int:
     return (n + 1023) // 1024 * 1024
 
 
+GLU_LABELS = {"gelu_tanh": ".geglu", "silu": ".swiglu", "clamped": ".clamped_glu"}
 # ops that take the residual stream itself, as a copy in the activation type
 READS_RESIDUAL = {"token_side_gate", "concat_matmul", "fused_glu", "expert_router"}
 
@@ -160,6 +161,9 @@ def make_plan_class(base: type) -> type:
             if nxt.op == "dynamic_tanh" and nxt.attrs.get("rows") != "logits" and nxt.inputs[0] == self._nodes[idx].outputs[0]:
                 out = self._scratch("normed", width)
                 return H.Next(out, self._dyt(nxt.inputs[1:4])), nxt.outputs[0]
+            if nxt.op == "rms_norm" and nxt.attrs.get("rows") != "logits" and nxt.inputs[0] == self._nodes[idx].outputs[0]:
+                norm = H.RmsNorm(self.engine.weights.get_f32(nxt.inputs[1]), float(nxt.attrs["eps"]))
+                return H.Next(self._scratch("normed", width), norm), nxt.outputs[0]
             if nxt.op in READS_RESIDUAL and nxt.inputs[0] == self._nodes[idx].outputs[0]:
                 return H.Next(self._scratch("copied", width)), None
             return None, None
@@ -213,6 +217,13 @@ def make_plan_class(base: type) -> type:
             scale, x = float(node.attrs["scale"]), self._residual
             self._finish_residual(idx, lambda nx: self._emit(lambda: H.scaled_embedding(table, self.ids, x, scale, nx), "b200.scaled_embedding"))
 
+        def _lower_add_token_embedding(self, idx: int, node: Any) -> None:
+            """The embedding output once more, from the table."""
+            table = self.engine.weights.get_checked(node.inputs[2])
+            scale, x = float(node.attrs["scale"]), self._residual
+            self._finish_residual(idx, lambda nx: self._emit(lambda: H.scaled_embedding(table, self.ids, x, scale, nx, accumulate=True),
+                                                             "b200.add_embedding"))
+
         def _lower_dynamic_tanh(self, idx: int, node: Any) -> None:
             norm = self._dyt(node.inputs[1:4])
             width = int(self.engine.config.hidden_size)
@@ -230,18 +241,27 @@ def make_plan_class(base: type) -> type:
             bias = eng.concat_bias(tuple(node.attrs["bias"]), names) if node.attrs.get("bias") else None
             sizes = [int(eng.graph.weights[n].shape[0]) for n in names]
             w = eng.concat_weight(names)
-            total = int(w.shape[0])
+            floats = sum(sizes[len(sizes) - int(node.attrs.get("float_tail", 0)):])     # columns of the last weights: float32, one output
+            total = int(w.shape[0]) - floats
             out = self._scratch("projected", (total + 7) // 8 * 8)
+            tail = self._scratch("projected_float", floats, torch.float32) if floats else None
             act = sum(sizes[: int(node.attrs.get("activated", 0))])
             if H.dense_supported(int(w.shape[1]), w.stride(0), x.stride(0), dtype=x.dtype):
                 epilogue = H.DENSE_SILU if act else H.DENSE_PLAIN
-                self._emit(lambda: H.dense_gemm(x, w, out, epilogue=epilogue, act_cols=act, bias=bias),
+                self._emit(lambda: H.dense_gemm(x, w, out, epilogue=epilogue, act_cols=act, bias=bias, tail=tail),
                            "b200.dense_gemm" + (".silu" if act else ""))
             else:
-                self._emit(lambda: H.dense_simple(x, w, out, bias=bias), "b200.dense_simple")
+                main, main_bias = w[:total], None if bias is None else bias[:total]
+                self._emit(lambda: H.dense_simple(x, main, out, bias=main_bias), "b200.dense_simple")
+                if tail is not None:
+                    rest, rest_bias = w[total:], None if bias is None else bias[total:]
+                    self._emit(lambda: H.dense_simple(x, rest, tail, bias=rest_bias), "b200.dense_simple")
                 if act:
                     self._emit(lambda: H.silu_cols(out, act), "b200.silu_cols")
             col = 0
+            if tail is not None:
+                self._env[node.outputs[-1]] = tail
+                sizes = sizes[:len(sizes) - int(node.attrs["float_tail"])]
             for name, n in zip(node.outputs, sizes):
                 self._env[name] = out[:, col:col + n]
                 col += n
@@ -300,6 +320,34 @@ def make_plan_class(base: type) -> type:
                 self._emit(lambda: H.recurrence_simple(args), "b200.recurrence_simple")
             self._env[node.outputs[0]] = out
 
+        def _lower_matrix_memory(self, idx: int, node: Any) -> None:
+            eng, at = self.engine, node.attrs
+            q, k, v, logits, gate = (self._env[n] for n in node.inputs[:5])
+            in_bias, forget_bias, norm = (eng.weights.get_f32(n) for n in node.inputs[5:8])
+            heads, dim, vdim, eps = int(at["heads"]), int(at["dim"]), int(at["vdim"]), float(at["eps"])
+            state = eng.allocator.state_for_layer(int(at["layer"]))
+            gates = H.MemoryGates(logits, in_bias, forget_bias, float(at["gate_cap"]))
+            mixed, scale = self._scratch("memory_mixed", heads * vdim), float(dim) ** -0.5
+            self._env[node.outputs[0]] = mixed
+            if self.decode and vdim % 4 == 0 and vdim <= 1024 and dim <= 4096:
+                args = H.recurrence_args(self.rows, q, k, v, None, state, mixed, heads=heads, dim=dim, vdim=vdim, q_scale=scale)
+                self._emit(lambda: H.memory_step(args, gates, gate, norm, eps), "b200.memory_step")
+                return
+            log_decay, log_take, maximum, normaliser = (self._scratch("memory_" + role, heads, torch.float32)
+                                                        for role in ("decay", "take", "maximum", "normaliser"))
+            out = self._scratch("recurrence", heads * vdim)
+            args = H.recurrence_args(self.rows, q, k, v, None, state, out, heads=heads, dim=dim, vdim=vdim, gated=(log_decay, log_take, normaliser),
+                                     q_scale=scale)
+            self._emit(lambda: H.memory_gates(args, gates, log_decay, log_take, maximum), "b200.memory_gates")
+            aligned = q.stride(0) % 8 == 0 and not any(t.data_ptr() % 16 for t in (q, k, v))
+            if H.recurrence_chunked_supported(dim, vdim, eng.dtype) and aligned:
+                need = H.recurrence_workspace_bytes(self.batch, self.segments, heads, dim, vdim)
+                ws = eng.scratch("recurrence_ws", need) if need else None
+                self._emit(lambda: H.recurrence_chunked(args, ws), "b200.recurrence_chunked", launches=3 if need else 1)
+            else:
+                self._emit(lambda: H.recurrence_simple(args), "b200.recurrence_simple")
+            self._emit(lambda: H.memory_norm(out, normaliser, maximum, gate, norm, eps, mixed, heads=heads, vdim=vdim), "b200.memory_norm")
+
         def _lower_gated_rms_norm(self, idx: int, node: Any) -> None:
             o, gate = self._env[node.inputs[0]], self._env[node.inputs[1]]
             w, eps = self.engine.weights.get_f32(node.inputs[2]), float(node.attrs["eps"])
@@ -321,7 +369,7 @@ def make_plan_class(base: type) -> type:
             if nxt is None:
                 out = self._scratch("logits", int(w.shape[0]), torch.float32, rows=self.logit_rows)
             else:
-                out = self._scratch("sublayer", int(w.shape[0]))      # (a shared expert's lives until the combine)
+                out = self._scratch(str(node.attrs.get("role", "sublayer")), int(w.shape[0]))      # (a shared expert's lives until the combine)
             bias = node.attrs.get("bias")
             self._dense(x, w, out, None if bias is None else eng.weights.get_f32(bias), "." + str(node.attrs["projection"]))
             self._env[node.outputs[0]] = out
@@ -336,18 +384,18 @@ def make_plan_class(base: type) -> type:
         def _lower_fused_glu(self, idx: int, node: Any) -> None:
             self._env[node.outputs[0]] = self._glu(self._input(node.inputs[0]), node, node.attrs["activation"])
 
-        def _glu(self, x: torch.Tensor, node: Any, activation: str, tail_weight: str | None = None,
+        def _glu(self, x: torch.Tensor, node: Any, activation: str, tail_weights: tuple[str, ...] = (),
                  tail: torch.Tensor | None = None) -> torch.Tensor:
-            """activation(gate, up) of one product; `tail_weight`'s rows behind the pairs leave plain float32 columns."""
+            """activation(gate, up) of one product; rows of `tail_weights` behind the pairs leave plain float32 columns."""
             eng = self.engine
             names = tuple(node.inputs[1:3])
-            w = eng.paired_weight(names, tail_weight)
+            w = eng.paired_weight(names, tail_weights)
             ff = int(eng.graph.weights[names[0]].shape[0])
             bias = eng.paired_bias(tuple(node.attrs["bias"])) if node.attrs.get("bias") else None
             kind, limit = H.GLU_EPILOGUES[activation], float(node.attrs.get("limit", 0.0))
             out = self._scratch("gated", (ff + 7) // 8 * 8)[:, :ff]
             if H.dense_supported(int(w.shape[1]), w.stride(0), x.stride(0), dtype=x.dtype):
-                label = {"gelu_tanh": ".geglu", "silu": ".swiglu", "clamped": ".clamped_glu"}[activation]
+                label = GLU_LABELS[activation]
                 self._emit(lambda: H.dense_gemm(x, w, out, epilogue=kind, bias=bias, limit=limit, tail=tail), "b200.dense_gemm" + label)
             else:
                 both, out = self._scratch("gate_up", 2 * ff), self._scratch("gated", ff)
@@ -375,8 +423,19 @@ def make_plan_class(base: type) -> type:
             w, eps = self.engine.weights.get_f32(node.inputs[2]), float(node.attrs["eps"])
             self._finish_residual(idx, lambda nx: self._emit(lambda: H.residual_rms(res, y, w, eps, nx), "b200.residual_rms"))
 
+        def _lower_residual_add(self, idx: int, node: Any) -> None:
+            y, res = self._env[node.inputs[1]], self._residual
+            self._finish_residual(idx, lambda nx: self._emit(lambda: H.residual_add(res, y, nx), "b200.residual_add"))
+
+        def _lower_residual_rms_pair(self, idx: int, node: Any) -> None:
+            y1, y2, res = self._env[node.inputs[1]], self._env[node.inputs[3]], self._residual
+            w1, w2 = (self.engine.weights.get_f32(node.inputs[i]) for i in (2, 4))
+            factor, eps = float(node.attrs["factor"]), float(node.attrs["eps"])
+            self._finish_residual(idx, lambda nx: self._emit(lambda: H.residual_rms_pair(res, y1, w1, y2, w2, factor, eps, nx),
+                                                             "b200.residual_rms_pair"))
+
         def _lower_rms_norm(self, idx: int, node: Any) -> None:
-            w, eps = self.engine.weights.get_f32(node.inputs[1]), float(node.attrs["eps"])
+            w, eps = self.engine.scaled_weight(node.inputs[1], float(node.attrs.get("scale", 1.0))), float(node.attrs["eps"])
             logits = node.attrs.get("rows") == "logits"
             out = self._scratch("final" if logits else "normed", int(w.numel()), rows=self.logit_rows if logits else None)
             index = self.logit_index if logits else None
@@ -384,40 +443,57 @@ def make_plan_class(base: type) -> type:
             self._env[node.outputs[0]] = out
 
         def _lower_tied_attention(self, idx: int, node: Any) -> None:
+            """Inputs: q, k, then by name or "" output gate, sink, values of their own, weights of the query and key norm."""
             eng, at = self.engine, node.attrs
-            q, k, gate = (self._env[n] for n in node.inputs[:3])
+            names = list(node.inputs) + [""] * (7 - len(node.inputs))
+            q, k, gate, v = (self._env[n] if n else None for n in (names[0], names[1], names[2], names[4]))
+            sink, q_weight, k_weight = (eng.weights.get_f32(n) if n else None for n in (names[3], names[5], names[6]))
             heads, kv_heads, dim, rot = (int(at[n]) for n in ("heads", "kv_heads", "dim", "rot_dims"))
+            key_dim = None if v is None else int(at["key_dim"])
+            whole = bool(at.get("whole_norm", False))
             pool = eng.allocator.pool_for_layer(int(at["layer"]))
             scaling = at.get("rot_scaling")
             table = eng.rotate_half_table(rot, float(at["rot_base"]), None if scaling is None else tuple(map(float, scaling))) if rot else None
+            reach = float(dim if key_dim is None else key_dim)              # of unit root mean squares
+            reach *= ((heads * kv_heads) ** 0.5 if whole else 1.0) * eng.largest_weight(names[5]) * eng.largest_weight(names[6])
             args = X.tied_args(self.rows, pool["rows"], pool["inv_rms"], heads=heads, kv_heads=kv_heads, dim=dim, rot_dims=rot,
                                window=int(at["window"]), keep_first=int(at["keep_first"]), scale=float(at["scale"]), softcap=at.get("softcap"),
-                               sink=eng.weights.get_f32(node.inputs[3]))
-            prepared = self._scratch("prepared_q", heads * X.query_width(dim, rot))
+                               sink=sink, key_dim=key_dim, reach=reach)
+            prepared = self._scratch("prepared_q", heads * X.query_width(dim, rot, key_dim))
             out = self._scratch("mixed", heads * dim)
-            self._emit(lambda: X.tied_prepare(args, q, k, prepared, eps=float(at["eps"]), table=table), "b200.tied_prepare")
-            if self.decode and X.tied_step_supported(heads, kv_heads, dim, rot, eng.page_size, eng.dtype):
+            self._emit(lambda: X.tied_prepare(args, q, k, prepared, eps=float(at["eps"]), table=table, v=v, q_weight=q_weight, k_weight=k_weight,
+                                              whole=whole), "b200.tied_prepare")
+            if self.decode and X.tied_step_supported(heads, kv_heads, dim, rot, eng.page_size, eng.dtype, key_dim):
                 splits = X.tied_step_splits(self.batch, heads, kv_heads, int(at["window"]), int(at["keep_first"]), self.width, eng.page_size)
                 self._emit(lambda: X.tied_attention_step(args, prepared, gate, out, splits=splits), "b200.tied_attention_step")
-            elif X.tied_prompt_supported(heads, kv_heads, dim, rot, eng.page_size, eng.dtype) and gate.stride(0) % 8 == 0:
+            elif (X.tied_prompt_supported(heads, kv_heads, dim, rot, eng.page_size, eng.dtype, key_dim)
+                  and (gate is None or gate.stride(0) % 8 == 0)):
                 self._emit(lambda: X.tied_attention_prompt(args, prepared, gate, out), "b200.tied_attention_prompt")
             else:
                 self._emit(lambda: X.tied_attention_simple(args, prepared, gate, out), "b200.tied_attention_simple")
             self._env[node.outputs[0]] = out
 
         def _lower_expert_router(self, idx: int, node: Any) -> None:
-            eng, x = self.engine, self._input(node.inputs[0])
-            spec = eng.graph.weights[node.inputs[1]]
-            experts, width, top, scale = int(spec.shape[0]), int(spec.shape[1]), int(node.attrs["top"]), float(node.attrs["scale"])
-            logits = self._scratch("router_logits", experts, torch.float32)
+            """Inputs: x, router, then by name or "" correction and the shared expert's gate (one row)."""
+            eng, x, at = self.engine, self._input(node.inputs[0]), node.attrs
+            names = list(node.inputs) + [""] * (4 - len(node.inputs))
+            spec = eng.graph.weights[names[1]]
+            scored, width, top, scale = int(spec.shape[0]), int(spec.shape[1]), int(at["top"]), float(at["scale"])
+            identity = int(at.get("identity", 0))
+            experts = scored - identity
+            rule = None
+            if at.get("scores") == "softmax":
+                rule = X.SoftmaxRule(eng.weights.get_f32(names[2]) if names[2] else None, int(at["groups"]), int(at["keep"]), identity)
+            rows_of = (names[1],) + ((names[3],) if names[3] else ())
+            logits = self._scratch("router_logits", scored + len(rows_of) - 1, torch.float32)
             nxt = self._nodes[idx + 1]
             if (nxt.op == "fused_glu" and nxt.inputs[0] == node.inputs[0] and not nxt.attrs.get("bias")
                     and H.dense_supported(width, width, x.stride(0), dtype=x.dtype)):
                 # a shared expert reads the same rows: the router's columns ride behind its gate and up
-                self._env[nxt.outputs[0]] = self._glu(x, nxt, nxt.attrs["activation"], node.inputs[1], logits)
+                self._env[nxt.outputs[0]] = self._glu(x, nxt, nxt.attrs["activation"], rows_of, logits)
                 self._skip.add(idx + 1)
             else:
-                self._dense(x, eng.weights.get_checked(node.inputs[1]), logits)
+                self._dense(x, eng.concat_weight(rows_of), logits)
             i32 = torch.int32
             routing = X.Routing(experts, top, counters=self._scratch("route_counters", experts + 1, i32, rows=1).view(-1),
                                 cu=self._scratch("route_cu", experts + 1, i32, rows=1).view(-1), token_of=self._scratch("route_token", top, i32).view(-1),
@@ -426,8 +502,10 @@ def make_plan_class(base: type) -> type:
             placed = None
             if self.batch > X.grouped_all_rows() and X.grouped_supported(width, x.stride(0), eng.dtype):
                 placed = self._scratch("placed", width, rows=routing.places)       # the experts' products read rows in expert order
-            self._emit(lambda: X.route(logits, self.rows.row_seg, routing, scale, x, placed), "b200.route", launches=1 if placed is None else 2)
+            self._emit(lambda: X.route(logits, self.rows.row_seg, routing, scale, x, placed, rule), "b200.route", launches=1 if placed is None else 2)
             self._env[node.outputs[0]] = (routing, placed)
+            if names[3]:
+                self._env[node.outputs[1]] = logits[:, scored]
 
         def _lower_expert_mixture(self, idx: int, node: Any) -> None:
             eng, x = self.engine, self._input(node.inputs[0])
@@ -436,14 +514,15 @@ def make_plan_class(base: type) -> type:
             gates, ups, downs = (tuple(node.inputs[2 + i * n:2 + (i + 1) * n]) for i in range(3))
             w_in, w_out = eng.expert_pairs(gates, ups), eng.concat_weight(downs)
             ff, width = int(w_in.shape[0]) // (2 * n), int(w_out.shape[0]) // n
-            kind, limit = H.GLU_EPILOGUES[node.attrs["activation"]], float(node.attrs["limit"])
+            activation = node.attrs["activation"]
+            kind, limit = H.GLU_EPILOGUES[activation], float(node.attrs.get("limit", 0.0))
             places = routing.places
             out = self._scratch("expert_out", width, rows=places)
             if X.grouped_supported(int(w_in.shape[1]), x.stride(0), eng.dtype) and X.grouped_supported(ff, ff, eng.dtype):
                 hidden = self._scratch("expert_hidden", ff, rows=places)
                 source = x if placed is None else placed
                 self._emit(lambda: X.grouped_gemm(source, w_in, hidden, routing, by_row=placed is None, epilogue=kind, limit=limit),
-                           "b200.grouped_gemm.clamped_glu")
+                           "b200.grouped_gemm" + GLU_LABELS[activation])
                 self._emit(lambda: X.grouped_gemm(hidden, w_out, out, routing, by_row=False), "b200.grouped_gemm")
             else:
                 both, hidden = self._scratch("expert_gate_up", 2 * ff, rows=places), self._scratch("expert_hidden", ff, rows=places)
@@ -458,5 +537,12 @@ def make_plan_class(base: type) -> type:
             shared = self._env[node.inputs[4]] if len(node.inputs) > 4 else None
             self._finish_residual(idx, lambda nx: self._emit(lambda: X.combine_residual_rms(res, y, routing, shared, w, eps, nx),
                                                              "b200.combine_residual_rms"))
+
+        def _lower_combine_residual(self, idx: int, node: Any) -> None:
+            """Inputs: residual, experts' rows, routing, the experts' input, then the shared expert's output and its gate."""
+            y, (routing, _), x, res = self._env[node.inputs[1]], self._env[node.inputs[2]], self._input(node.inputs[3]), self._residual
+            shared, gate = (self._env[node.inputs[i]] if len(node.inputs) > i else None for i in (4, 5))
+            self._finish_residual(idx, lambda nx: self._emit(lambda: X.combine_residual(res, y, routing, x, shared, gate, nx),
+                                                             "b200.combine_residual"))
 
     return RaggedPlan

@@ -73,6 +73,12 @@ HYBRID_KERNELS_FOR_OP: dict[str, tuple[str, ...]] = {
     "expert_router": ("cacheir_b200_dense_gemm", "cacheir_b200_dense_simple", "cacheir_b200_route"),
     "expert_mixture": ("cacheir_b200_grouped_gemm", "cacheir_b200_grouped_simple", "cacheir_b200_glu_pairs"),
     "combine_residual_rms_norm": ("cacheir_b200_combine_residual_rms",),
+    "add_token_embedding": ("cacheir_b200_scaled_embedding",),
+    "matrix_memory": ("cacheir_b200_memory_step", "cacheir_b200_memory_gates", "cacheir_b200_recurrence_chunked", "cacheir_b200_recurrence_simple",
+                      "cacheir_b200_memory_norm"),
+    "residual_add": ("cacheir_b200_residual_add",),
+    "residual_rms_pair": ("cacheir_b200_residual_rms_pair",),
+    "combine_residual": ("cacheir_b200_combine_residual",),
 }
 
 B200_BACKEND = Backend(
@@ -99,6 +105,7 @@ B200_BACKEND = Backend(
         "latent_attention",
         "linear_recurrence",
         "tied_attention",
+        "matrix_memory",
         "grouped_gemm_bf16",
         "expert_routing",
     ),

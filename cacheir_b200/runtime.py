@@ -178,6 +178,7 @@ class _Engine:
         self.max_plans = max(1, int(max_plans)) * (4 if self.ragged else 1)     # (ragged plans share their buffers)
         self._scratch: dict[str, torch.Tensor] = {}
         self._derived: dict[tuple, torch.Tensor] = {}
+        self._largest: dict[str, float] = {}
         self.plans: OrderedDict[tuple, "_DecodePlan"] = OrderedDict()
         self.plans_lowered = 0          # decode graphs lowered to launch lists so far
         self.graph_captures = 0         # CUDA graphs captured so far
@@ -275,12 +276,24 @@ class _Engine:
             torch.zeros(int(self.graph.weights[n].shape[0]), device=self.device) if b is None else self.weights.get_f32(b)
             for b, n in zip(biases, names)]).contiguous(), [b for b in biases if b is not None])
 
-    def paired_weight(self, names: tuple[str, ...], tail: str | None = None) -> torch.Tensor:
-        """gate and up rows alternating, the order the gated epilogues want; `tail`'s rows behind them."""
+    def paired_weight(self, names: tuple[str, ...], tail: tuple[str, ...] = ()) -> torch.Tensor:
+        """gate and up rows alternating, the order the gated epilogues want; the rows of `tail` behind them."""
         def make() -> torch.Tensor:
             pairs = torch.stack([self.weights.get_checked(n) for n in names], dim=1).flatten(0, 1)
-            return (pairs if tail is None else torch.cat([pairs, self.weights.get_checked(tail)])).contiguous()
-        return self._derive(("paired", tail) + names, make, names + (() if tail is None else (tail,)))
+            return torch.cat([pairs] + [self.weights.get_checked(n) for n in tail]).contiguous()
+        return self._derive(("paired", tail) + names, make, names + tail)
+
+    def scaled_weight(self, name: str, scale: float) -> torch.Tensor:
+        """A float32 parameter times a constant."""
+        if scale == 1.0:
+            return self.weights.get_f32(name)
+        return self._derive(("scaled", name, scale), lambda: self.weights.get_f32(name) * scale, (name,))
+
+    def largest_weight(self, name: str) -> float:
+        """Largest magnitude in a float32 parameter; 1 for the absent one."""
+        if name and name not in self._largest:
+            self._largest[name] = float(self.weights.get_f32(name).abs().max().item())
+        return self._largest[name] if name else 1.0
 
     def paired_bias(self, names: tuple[str, ...]) -> torch.Tensor:
         return self._derive(("paired_bias",) + names, lambda: torch.stack([self.weights.get_f32(n) for n in names], dim=1).flatten().contiguous(), names)

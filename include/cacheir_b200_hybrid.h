@@ -1,6 +1,6 @@
 /*
- * cacheir_b200_hybrid.h -- C ABI of libcacheir_b200_hybrid.so: latent attention and linear recurrences (Gutorax). Rows of
- * a step as in cacheir_b200_ragged.h.
+ * cacheir_b200_hybrid.h -- C ABI of libcacheir_b200_hybrid.so: latent attention (Gutorax). Rows of a step as in
+ * cacheir_b200_ragged.h.
  */
 #ifndef CACHEIR_B200_HYBRID_H_
 #define CACHEIR_B200_HYBRID_H_
@@ -46,34 +46,6 @@ int cacheir_b200_latent_attention_supported(int kv_rank, int rot_dim, int page_s
 int cacheir_b200_latent_attention_splits(int rows, int heads, int window, int max_pages, int page_size);
 int cacheir_b200_latent_attention(const cacheir_b200_latent_args* a, const void* q, const float* sink, void* out, int splits,
                                   void* stream);
-
-/* ---- linear recurrence S <- decay S + k v^T, o = S^T q, one float32 state [heads, dim, vdim] per slot ------------- */
-typedef struct {
-  const int32_t* positions;
-  const int32_t* cu_rows;
-  const int32_t* slots;
-  int rows, segments;
-  int heads, dim, vdim;
-  const void* q;            /* [rows, stride], heads*dim columns, activation already applied */
-  const void* k;
-  const void* v;            /* heads*vdim columns */
-  long long stride;         /* common row stride of q, k, v */
-  const float* decay_pow;   /* [heads, 65]: decay^0 .. decay^64 */
-  float* state;             /* [num_slots, heads, dim, vdim] */
-  int num_slots;
-  void* out;                /* [rows, heads*vdim] */
-  int dtype;
-} cacheir_b200_recurrence_args;
-
-/* Token by token, any extents. A sequence whose first row has position 0 starts from a zero state. */
-int cacheir_b200_recurrence_simple(const cacheir_b200_recurrence_args* a, void* stream);
-/* One row per segment, streaming the state once (vdim % 4 == 0, otherwise EUNSUPPORTED). */
-int cacheir_b200_recurrence_step(const cacheir_b200_recurrence_args* a, void* stream);
-/* Chunked tensor-core form (bf16 q, k, v; dim % 16 == 0, dim <= 128, vdim % 8 == 0). Sequences longer than 256 rows use the
- * workspace for the states between their 256-row parts. */
-int cacheir_b200_recurrence_chunked_supported(int dim, int vdim, int dtype);
-size_t cacheir_b200_recurrence_workspace_bytes(int rows, int segments, int heads, int dim, int vdim);
-int cacheir_b200_recurrence_chunked(const cacheir_b200_recurrence_args* a, void* workspace, size_t workspace_bytes, void* stream);
 
 /* First bounded wait of this library's kernels that gave up since the last reset (0: none). Synchronises. */
 int cacheir_b200_hybrid_device_status(int reset);

@@ -24,6 +24,7 @@ extern "C" {
 #define CACHEIR_B200_NEXT_NONE 0
 #define CACHEIR_B200_NEXT_COPY 1   /* the residual itself, rounded to the activation type */
 #define CACHEIR_B200_NEXT_DYT 2    /* tanh(alpha * residual) * w + b                      */
+#define CACHEIR_B200_NEXT_RMS 3    /* residual / sqrt(mean(residual^2) + alpha) * w       */
 
 /* Epilogues of cacheir_b200_dense_gemm */
 #define CACHEIR_B200_DENSE_BF16 0        /* y                                                        */
@@ -58,7 +59,7 @@ typedef struct {
   long long table_stride;
   const float* bias;        /* [N] added to y before the epilogue, or NULL (batch 1) */
   float limit;
-  int tail_cols;            /* the paired epilogues: the last tail_cols columns of y go to `tail` as float32 instead */
+  int tail_cols;            /* BF16, SILU and the paired epilogues: the last tail_cols columns of y go to `tail` as float32 instead */
   float* tail;              /* [T, tail_stride] */
   long long tail_stride;
 } cacheir_b200_dense_args;
@@ -72,9 +73,9 @@ int cacheir_b200_dense_simple(const void* x, const void* w, void* y, int T, int 
                               int x_batch_cols, int y_batch_cols, long long w_stride, long long x_stride, long long y_stride,
                               const float* bias, int dtype, int y_dtype, void* stream);
 
-/* residual = table[ids] * scale, then next_mode. `table` and `next_out` are of `dtype`. */
+/* residual = table[ids] * scale (`accumulate`: +=), then next_mode. `table` and `next_out` are of `dtype`. */
 int cacheir_b200_scaled_embedding(const void* table, const int64_t* ids, float* residual, int rows, int width, int vocab,
-                                  float scale, int next_mode, const float* next_w, const float* next_b, float next_alpha,
+                                  float scale, int accumulate, int next_mode, const float* next_w, const float* next_b, float next_alpha,
                                   void* next_out, int dtype, void* stream);
 /* out[j] = dyt(residual[row_index ? row_index[j] : j]) */
 int cacheir_b200_dyt_rows(const float* residual, const int32_t* row_index, const float* w, const float* b, float alpha, void* out,
@@ -82,6 +83,13 @@ int cacheir_b200_dyt_rows(const float* residual, const int32_t* row_index, const
 /* out[j] = x / sqrt(mean(x^2) + eps) * w, x = residual[row_index ? row_index[j] : j] */
 int cacheir_b200_rms_rows(const float* residual, const int32_t* row_index, const float* w, float eps, void* out, int rows, int width,
                           int dtype, void* stream);
+/* residual += y, then next_mode (NONE, COPY or RMS) */
+int cacheir_b200_residual_add(float* residual, const void* y, int rows, int width, int next_mode, const float* next_w, const float* next_b,
+                              float next_alpha, void* next_out, int dtype, void* stream);
+/* residual += factor * (rms(y1) * w1 + rms(y2) * w2) with rms(y) = y / sqrt(mean(y^2) + eps), then next_mode (NONE, COPY or RMS) */
+int cacheir_b200_residual_rms_pair(float* residual, const void* y1, const float* w1, const void* y2, const float* w2, float factor, float eps,
+                                   int rows, int width, int next_mode, const float* next_w, const float* next_b, float next_alpha,
+                                   void* next_out, int dtype, void* stream);
 /* residual += dyt(y), then next_mode */
 int cacheir_b200_residual_dyt(float* residual, const void* y, const float* w, const float* b, float alpha, int rows, int width,
                               int next_mode, const float* next_w, const float* next_b, float next_alpha, void* next_out,

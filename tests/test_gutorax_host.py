@@ -18,7 +18,7 @@ from oracle import gutorax as G
 ROOT = Path(__file__).resolve().parents[1]
 
 
-@pytest.mark.parametrize("group", ["ragged", "hybrid", "experts"])
+@pytest.mark.parametrize("group", ["ragged", "hybrid", "recurrence", "experts"])
 def test_libraries_export_every_declared_symbol(group):
     from cacheir_b200 import _lib, build
 
@@ -34,23 +34,24 @@ def test_libraries_export_every_declared_symbol(group):
 def test_what_the_tensor_core_kernels_take():
     from cacheir_b200 import _lib, build
 
-    build.build(groups=("ragged", "hybrid"))
-    ragged, hybrid = _lib.load_group("ragged"), _lib.load_group("hybrid")
+    build.build(groups=("ragged", "hybrid", "recurrence"))
+    ragged, hybrid, recurrence = (_lib.load_group(g) for g in ("ragged", "hybrid", "recurrence"))
     assert ragged.cacheir_b200_dense_supported(24, 24, 24, 1, 0) == 1
     assert ragged.cacheir_b200_dense_supported(20, 20, 24, 1, 0) == 0
     assert hybrid.cacheir_b200_latent_attention_supported(512, 64, 64, 2) == 1
     assert hybrid.cacheir_b200_latent_attention_supported(512, 64, 64, 0) == 0
-    assert hybrid.cacheir_b200_recurrence_workspace_bytes(256, 3, 4, 16, 8) == 0
-    assert hybrid.cacheir_b200_recurrence_workspace_bytes(512, 3, 4, 16, 8) == 5 * 4 * 16 * 8 * 4
+    assert recurrence.cacheir_b200_recurrence_workspace_bytes(256, 3, 4, 16, 8) == 0
+    assert recurrence.cacheir_b200_recurrence_workspace_bytes(512, 3, 4, 16, 8) == 5 * 4 * (16 * (8 + 1) + 1) * 4
 
 
 def test_a_family_s_libraries_hold_only_what_it_needs():
     from cacheir_b200 import build, models
 
     files = {name: {src.stem for g in models.family_for({"architecture": name}).kernel_groups for src in build.group_sources(g)}
-             for name in ("Gutorax", "Topunex", "LlamaForCausalLM")}
+             for name in ("Gutorax", "Topunex", "Rekodra", "LlamaForCausalLM")}
     assert {"latent_attention", "linear_recurrence", "dense_gemm"} <= files["Gutorax"] and "tied_attention" not in files["Gutorax"]
     assert {"tied_attention", "grouped_gemm", "dense_gemm"} <= files["Topunex"] and not {"latent_attention", "qgemm_i8"} & files["Topunex"]
+    assert {"tied_attention", "linear_recurrence", "grouped_gemm"} <= files["Rekodra"] and not {"latent_attention", "qgemm_i8"} & files["Rekodra"]
     assert "paged_attention_mma" in files["LlamaForCausalLM"] and "dense_gemm" not in files["LlamaForCausalLM"]
     assert {src.stem for g in build.LIB_PATHS for src in build.group_sources(g)} == {src.stem for src in build.CSRC.glob("*.cu")}
 
@@ -59,13 +60,13 @@ def test_argument_structs_have_the_compiler_s_layout(tmp_path):
     from cacheir_b200 import _lib
 
     names = {"cacheir_b200_dense_args": _lib.DenseArgs, "cacheir_b200_latent_args": _lib.LatentArgs,
-             "cacheir_b200_recurrence_args": _lib.RecurrenceArgs, "cacheir_b200_tied_args": _lib.TiedArgs}
+             "cacheir_b200_recurrence_args": _lib.RecurrenceArgs, "cacheir_b200_tied_args": _lib.TiedArgs, "cacheir_b200_route_rule": _lib.RouteRule}
     lines = []
     for c_name, cls in names.items():
         lines.append(f'printf("%zu ", sizeof({c_name}));')
         lines += [f'printf("%zu ", offsetof({c_name}, {f[0]}));' for f in cls._fields_]
     src = tmp_path / "layout.c"
-    src.write_text('#include <stdio.h>\n#include <stddef.h>\n#include "cacheir_b200_hybrid.h"\n#include "cacheir_b200_experts.h"\nint main(void){'
+    src.write_text('#include <stdio.h>\n#include <stddef.h>\n#include "cacheir_b200_hybrid.h"\n#include "cacheir_b200_recurrence.h"\n#include "cacheir_b200_experts.h"\nint main(void){'
                    + "".join(lines) + "return 0;}")
     subprocess.run(["gcc", "-I", str(ROOT / "include"), str(src), "-o", str(tmp_path / "layout")], check=True)
     got = [int(v) for v in subprocess.run([str(tmp_path / "layout")], capture_output=True, text=True, check=True).stdout.split()]

@@ -50,11 +50,14 @@ def test_graph_follows_the_configuration():
 def test_every_graph_op_has_kernels_in_the_registry():
     from cacheir_b200 import _lib, registry
     from cacheir_b200.gutorax import GutoraxConfig, build_gutorax_graph
+    from cacheir_b200.rekodra import RekodraConfig, build_rekodra_graph
     from cacheir_b200.topunex import build_topunex_graph
     from gutorax_models import CONFIGS as OTHERS
+    from rekodra_models import CONFIGS as THIRD
 
     used = {n.op for name in CONFIGS for n in build_topunex_graph(_config(name)).nodes}
     used |= {n.op for cfg in OTHERS.values() for n in build_gutorax_graph(GutoraxConfig.from_dict(cfg)).nodes}
+    used |= {n.op for cfg in THIRD.values() for n in build_rekodra_graph(RekodraConfig.from_dict(cfg)).nodes}
     assert used == set(registry.HYBRID_KERNELS_FOR_OP)
     exported = {name for table in _lib.GROUP_SIGNATURES.values() for name in table}
     assert {k for names in registry.HYBRID_KERNELS_FOR_OP.values() for k in names} <= exported
@@ -128,7 +131,7 @@ def test_derived_weights_interleave_and_stack():
     eng = _Engine.__new__(_Engine)
     eng.graph, eng.device, eng.dtype, eng._derived = build_topunex_graph(_config("fast")), torch.device("cpu"), torch.float32, {}
     eng.weights = B200WeightStore(TensorSource(w), eng.graph.weights, None, device=eng.device, dtype=eng.dtype)
-    pairs = eng.paired_weight(("l1.mlp.shared.gate", "l1.mlp.shared.up"), "l1.mlp.router").numpy()
+    pairs = eng.paired_weight(("l1.mlp.shared.gate", "l1.mlp.shared.up"), ("l1.mlp.router",)).numpy()
     assert np.array_equal(pairs[0:80:2], w["l1.mlp.shared.gate"]) and np.array_equal(pairs[1:80:2], w["l1.mlp.shared.up"])
     assert np.array_equal(pairs[80:], w["l1.mlp.router"])
     experts = eng.expert_pairs(tuple(f"l1.mlp.e{e}.gate" for e in range(7)), tuple(f"l1.mlp.e{e}.up" for e in range(7))).numpy()
