@@ -145,33 +145,97 @@ residual_add_kernel(float* x, const T* __restrict__ y, int width, RowNext nx) {
   });
 }
 
-template <typename T, int VEC>
-__global__ void __launch_bounds__(kRowThreads)
+// HELD: a thread's columns (PIECES vectors at most) stay in registers from the first read to the last write, and what a later
+// step needs is requested before the sums.
+constexpr int kPairThreads = 256, kPairPieces = 4;
+template <typename T, int VEC, bool HELD>
+__global__ void __launch_bounds__(kPairThreads)
 residual_rms_pair_kernel(float* x, const T* __restrict__ y1, const float* __restrict__ w1, const T* __restrict__ y2,
                          const float* __restrict__ w2, float factor, float eps, int width, RowNext nx) {
   __shared__ float scratch[32];
+  __shared__ float2 s_pair[kPairThreads / 32];
   const size_t row = blockIdx.x;
   y1 += row * width;
   y2 += row * width;
-  float ss1 = 0.f, ss2 = 0.f;
-  for (int c = threadIdx.x * VEC; c < width; c += kRowThreads * VEC) {
-    float a[VEC], b[VEC];
-    load_vec<T, VEC>(y1 + c, a);
-    load_vec<T, VEC>(y2 + c, b);
+  float* xr = x + row * width;
+  auto factors = [&](float ss1, float ss2) {           // both root mean squares in one meeting
+    ss1 = warp_sum(ss1);
+    ss2 = warp_sum(ss2);
+    if ((threadIdx.x & 31) == 0) s_pair[threadIdx.x >> 5] = make_float2(ss1, ss2);
+    __syncthreads();
+    float2 t = make_float2(0.f, 0.f);
 #pragma unroll
-    for (int i = 0; i < VEC; ++i) { ss1 = fmaf(a[i], a[i], ss1); ss2 = fmaf(b[i], b[i], ss2); }
+    for (int w = 0; w < kPairThreads / 32; ++w) { t.x += s_pair[w].x; t.y += s_pair[w].y; }
+    return make_float2(factor / sqrtf(t.x / static_cast<float>(width) + eps), factor / sqrtf(t.y / static_cast<float>(width) + eps));
+  };
+  if constexpr (HELD) {
+    float a[kPairPieces][VEC], b[kPairPieces][VEC], s[kPairPieces][VEC], ss1 = 0.f, ss2 = 0.f;
+#pragma unroll
+    for (int k = 0; k < kPairPieces; ++k) {
+      const int c = (k * kPairThreads + static_cast<int>(threadIdx.x)) * VEC;
+      if (c < width) {
+        load_vec<T, VEC>(y1 + c, a[k]);
+        load_vec<T, VEC>(y2 + c, b[k]);
+        load_vec<float, VEC>(xr + c, s[k]);
+      }
+    }
+#pragma unroll
+    for (int k = 0; k < kPairPieces; ++k)
+      if ((k * kPairThreads + static_cast<int>(threadIdx.x)) * VEC < width)
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) { ss1 = fmaf(a[k][i], a[k][i], ss1); ss2 = fmaf(b[k][i], b[k][i], ss2); }
+    const float2 f = factors(ss1, ss2);
+    float ss = 0.f;
+    T* out = static_cast<T*>(nx.out) + row * width;
+#pragma unroll
+    for (int k = 0; k < kPairPieces; ++k) {
+      const int c = (k * kPairThreads + static_cast<int>(threadIdx.x)) * VEC;
+      if (c < width) {
+        float u[VEC], v[VEC];
+        load_vec<float, VEC>(w1 + c, u);
+        load_vec<float, VEC>(w2 + c, v);
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) {
+          s[k][i] += a[k][i] * f.x * u[i] + b[k][i] * f.y * v[i];
+          ss = fmaf(s[k][i], s[k][i], ss);
+        }
+        store_vec<float, VEC>(xr + c, s[k]);
+        if (nx.mode == CACHEIR_B200_NEXT_COPY) store_vec<T, VEC>(out + c, s[k]);
+      }
+    }
+    if (nx.mode != CACHEIR_B200_NEXT_RMS) return;
+    const float inv = 1.f / sqrtf(block_sum_all(ss, scratch) / static_cast<float>(width) + nx.eps);
+#pragma unroll
+    for (int k = 0; k < kPairPieces; ++k) {
+      const int c = (k * kPairThreads + static_cast<int>(threadIdx.x)) * VEC;
+      if (c < width) {
+        float w[VEC];
+        load_vec<float, VEC>(nx.w + c, w);
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) w[i] = s[k][i] * inv * w[i];
+        store_vec<T, VEC>(out + c, w);
+      }
+    }
+  } else {
+    float ss1 = 0.f, ss2 = 0.f;
+    for (int c = threadIdx.x * VEC; c < width; c += kPairThreads * VEC) {
+      float a[VEC], b[VEC];
+      load_vec<T, VEC>(y1 + c, a);
+      load_vec<T, VEC>(y2 + c, b);
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) { ss1 = fmaf(a[i], a[i], ss1); ss2 = fmaf(b[i], b[i], ss2); }
+    }
+    const float2 f = factors(ss1, ss2);
+    finish_row<T, VEC>(xr, row, width, nx, scratch, [&](int c, float (&s)[VEC]) {
+      float a[VEC], b[VEC], u[VEC], v[VEC];
+      load_vec<T, VEC>(y1 + c, a);
+      load_vec<T, VEC>(y2 + c, b);
+      load_vec<float, VEC>(w1 + c, u);
+      load_vec<float, VEC>(w2 + c, v);
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) s[i] += a[i] * f.x * u[i] + b[i] * f.y * v[i];
+    });
   }
-  const float f1 = factor / sqrtf(block_sum_all(ss1, scratch) / static_cast<float>(width) + eps);
-  const float f2 = factor / sqrtf(block_sum_all(ss2, scratch) / static_cast<float>(width) + eps);
-  finish_row<T, VEC>(x + row * width, row, width, nx, scratch, [&](int c, float (&s)[VEC]) {
-    float a[VEC], b[VEC], u[VEC], v[VEC];
-    load_vec<T, VEC>(y1 + c, a);
-    load_vec<T, VEC>(y2 + c, b);
-    load_vec<float, VEC>(w1 + c, u);
-    load_vec<float, VEC>(w2 + c, v);
-#pragma unroll
-    for (int i = 0; i < VEC; ++i) s[i] += a[i] * f1 * u[i] + b[i] * f2 * v[i];
-  });
 }
 
 template <typename T, int VEC>
@@ -369,12 +433,13 @@ extern "C" int cacheir_b200_residual_rms_pair(float* residual, const void* y1, c
   const RowNext nx{next_mode, next_w, next_alpha, next_out};
   const bool vec = width % 4 == 0 && aligned_to(residual, 16) && aligned_to(y1, 16) && aligned_to(y2, 16) && aligned_to(w1, 16) &&
                    aligned_to(w2, 16) && row_next_aligned(next_mode, next_w, next_out);
-#define CB200_PAIR(VEC)                                                                                                                  \
-  residual_rms_pair_kernel<T, VEC><<<rows, kRowThreads, 0, as_stream(stream)>>>(residual, static_cast<const T*>(y1), w1, static_cast<const T*>(y2), \
-                                                                               w2, factor, eps, width, nx)
+#define CB200_PAIR(VEC, HELD)                                                                                                        \
+  residual_rms_pair_kernel<T, VEC, HELD><<<rows, kPairThreads, 0, as_stream(stream)>>>(residual, static_cast<const T*>(y1), w1,        \
+                                                                                      static_cast<const T*>(y2), w2, factor, eps, width, nx)
   CB200_HYBRID_DTYPE(dtype, {
-    if (vec) CB200_PAIR(4);
-    else CB200_PAIR(1);
+    if (vec && width <= 4 * kPairThreads * kPairPieces) CB200_PAIR(4, true);
+    else if (vec) CB200_PAIR(4, false);
+    else CB200_PAIR(1, false);
   });
 #undef CB200_PAIR
   return launch_status();

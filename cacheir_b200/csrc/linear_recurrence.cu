@@ -7,8 +7,8 @@
 // chunked  prompts, bf16 operands on the tensor cores, 64 tokens at a time. With D_ij = decay^(i-j) for j <= i:
 //            O = diag(decay^(i+1)) Q S + ((Q K^T) o D) V        S' = decay^n S + K^T diag(decay^(n-1-j)) V
 //          The state stays in float32 registers; whatever is float32 by nature and has to enter an MMA (the state, the
-//          decayed scores, the decayed values) goes in as a sum of two bf16 numbers. Sequences are cut into 256-token
-//          pieces that run in parallel: a first pass finds every piece's own contribution, a scan turns these into the
+//          decayed scores, the decayed values) goes in as a sum of two bf16 numbers. Sequences are cut into pieces of
+//          64 to 256 tokens that run in parallel: a first pass finds every piece's own contribution, a scan turns these into the
 //          pieces' initial states, and the main pass starts from them. GATED: with c the running sum of log decays in a
 //          chunk, decay^(i-j) becomes exp(c_i - c_j + log take_j), and so on; n rides with the first value columns.
 // gates    matrix memory: log decay and log take from gate logits, relative to a running maximum (a scan over the tokens)
@@ -22,7 +22,7 @@ namespace {
 
 constexpr int kPowers = 65;
 constexpr int kChunk = 64;
-constexpr int kPiece = 256;
+constexpr int kPiece = 256;        // tokens of a piece at most, and of a step that is not cut
 constexpr int kCols = 64;          // value columns per CTA of the chunked form
 constexpr int kPitchV = kCols + 8; // bf16 elements per shared-memory row (16 bytes over a multiple of 128: conflict-free)
 
@@ -182,7 +182,7 @@ PieceSpace piece_space(const Args& a, float* ws, int items) {
 // MT = 16-row state tiles per warp (dim <= 64 MT)
 template <int MT, bool LOCAL, bool GATED>
 __global__ void __launch_bounds__(128)
-recurrence_chunk_kernel(const Args a, const PieceSpace ws) {
+recurrence_chunk_kernel(const Args a, const PieceSpace ws, int piece_rows) {
   extern __shared__ __align__(16) uint8_t raw[];
   const int dim = a.dim;
   const int pitch = dim + 8;
@@ -192,11 +192,12 @@ recurrence_chunk_kernel(const Args a, const PieceSpace ws) {
   __nv_bfloat16* s_dv = s_v + kChunk * kPitchV;                      // [2][64][72] decayed values, hi | lo
   __nv_bfloat16* s_s = s_dv + 2 * kChunk * kPitchV;                  // [2][dim][72] state, hi | lo
   __shared__ float s_pow[kPowers];
-  __shared__ float s_cum[kChunk], s_take[kChunk], s_left[kChunk], s_n[128];      // log decays summed, log take, weight in the chunk's last state
+  __shared__ float s_cum[kChunk], s_take[kChunk], s_left[kChunk];      // log decays summed, log take, weight in the chunk's last state
+  __shared__ float s_n[2][128];                       // the normaliser before and after a chunk
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int h = blockIdx.y, v0 = blockIdx.z * kCols;
 
-  const RaggedItem it = find_item(a.cu_rows, a.segments, kPiece, blockIdx.x);
+  const RaggedItem it = find_item(a.cu_rows, a.segments, piece_rows, blockIdx.x);
   if (it.seg < 0) return;
   const bool alone = it.last && static_cast<int>(blockIdx.x) == it.first;     // the segment is a single piece
   if (LOCAL && it.last) return;                                               // nobody needs its contribution
@@ -213,7 +214,7 @@ recurrence_chunk_kernel(const Args a, const PieceSpace ws) {
   const bool first = GATED && blockIdx.z == 0;        // this block also has the normaliser
   float sum = 0.f;                                    // of the piece's log decays
   if (first && static_cast<int>(threadIdx.x) < dim)
-    s_n[threadIdx.x] = zero ? 0.f : (alone ? slot_normaliser(a, it.seg, h) : piece_n)[threadIdx.x];
+    s_n[0][threadIdx.x] = zero ? 0.f : (alone ? slot_normaliser(a, it.seg, h) : piece_n)[threadIdx.x];
 #pragma unroll
   for (int t = 0; t < MT; ++t)
 #pragma unroll
@@ -229,6 +230,18 @@ recurrence_chunk_kernel(const Args a, const PieceSpace ws) {
   __syncthreads();
 
   const int kc = dim / 8;      // 16-byte pieces per q / k row
+  int now = 0;                 // which of s_n is the current one
+  float ahead[4] = {};         // warp 0: the next chunk's log decays and log takes, two rows per lane
+  auto fetch_gates = [&](int r0) {
+#pragma unroll
+    for (int u = 0; u < 2; ++u) {
+      const int r = r0 + u * 32 + lane;
+      const size_t at = (static_cast<size_t>(it.row0) + r) * a.heads + h;
+      ahead[u] = r < it.count ? a.log_decay[at] : 0.f;
+      ahead[2 + u] = r < it.count ? a.log_take[at] : 0.f;
+    }
+  };
+  if (GATED && warp == 0) fetch_gates(0);
   for (int r0 = 0; r0 < it.count; r0 += kChunk) {
     const int n = min(kChunk, it.count - r0);
     const size_t base = static_cast<size_t>(it.row0 + r0);
@@ -237,10 +250,8 @@ recurrence_chunk_kernel(const Args a, const PieceSpace ws) {
         float c[2], take[2], last = 0.f;
 #pragma unroll
         for (int u = 0; u < 2; ++u) {
-          const int r = u * 32 + lane;
-          const size_t at = (base + r) * a.heads + h;
-          c[u] = r < n ? a.log_decay[at] : 0.f;
-          take[u] = r < n ? a.log_take[at] : 0.f;
+          c[u] = ahead[u];
+          take[u] = ahead[2 + u];
 #pragma unroll
           for (int off = 1; off < 32; off <<= 1) {
             const float up = __shfl_up_sync(0xffffffffu, c[u], off);
@@ -256,6 +267,7 @@ recurrence_chunk_kernel(const Args a, const PieceSpace ws) {
           s_take[r] = take[u];
           s_left[r] = r < n ? __expf(last - c[u] + take[u]) : 0.f;
         }
+        if (r0 + kChunk < it.count) fetch_gates(r0 + kChunk);
       }
       __syncthreads();
     }
@@ -352,8 +364,8 @@ recurrence_chunk_kernel(const Args a, const PieceSpace ws) {
       float nq[2] = {0.f, 0.f};
       if (first) {                                    // q . (n before the chunk): a quarter of the entries per lane of the row
         for (int d = lane & 3; d < dim; d += 4) {
-          nq[0] = fmaf(__bfloat162float(s_q[i0 * pitch + d]), s_n[d], nq[0]);
-          nq[1] = fmaf(__bfloat162float(s_q[(i0 + 8) * pitch + d]), s_n[d], nq[1]);
+          nq[0] = fmaf(__bfloat162float(s_q[i0 * pitch + d]), s_n[now][d], nq[0]);
+          nq[1] = fmaf(__bfloat162float(s_q[(i0 + 8) * pitch + d]), s_n[now][d], nq[1]);
         }
         nq[0] *= f0;
         nq[1] *= f1;
@@ -446,20 +458,23 @@ recurrence_chunk_kernel(const Args a, const PieceSpace ws) {
       }
     }
     if (first) {
-      __syncthreads();                                // everyone has met the old n
       const int d = threadIdx.x;
-      if (d < dim) {
-        float x = s_n[d] * fn;
-        for (int r = 0; r < n; ++r) x = fmaf(s_left[r], __bfloat162float(s_k[r * pitch + d]), x);
-        s_n[d] = x;
+      if (d < dim) {                                  // (rows behind the last are zero)
+        float x[4] = {s_n[now][d] * fn, 0.f, 0.f, 0.f};
+#pragma unroll 4
+        for (int r = 0; r < kChunk; r += 4)
+#pragma unroll
+          for (int u = 0; u < 4; ++u) x[u] = fmaf(s_left[r + u], __bfloat162float(s_k[(r + u) * pitch + d]), x[u]);
+        s_n[now ^ 1][d] = (x[0] + x[1]) + (x[2] + x[3]);
       }
     }
+    now ^= 1;
     __syncthreads();
   }
 
   float* dst = LOCAL ? piece : state;
   if (LOCAL || it.last) {
-    if (first && static_cast<int>(threadIdx.x) < dim) (LOCAL ? piece_n : slot_normaliser(a, it.seg, h))[threadIdx.x] = s_n[threadIdx.x];
+    if (first && static_cast<int>(threadIdx.x) < dim) (LOCAL ? piece_n : slot_normaliser(a, it.seg, h))[threadIdx.x] = s_n[now][threadIdx.x];
     if (LOCAL && first && threadIdx.x == 0) ws.log_decay[static_cast<size_t>(blockIdx.x) * a.heads + h] = sum;
 #pragma unroll
     for (int t = 0; t < MT; ++t)
@@ -474,38 +489,61 @@ recurrence_chunk_kernel(const Args a, const PieceSpace ws) {
   }
 }
 
-// Contributions of a segment's pieces -> their initial states (in place).
+// Contributions of a segment's pieces -> their initial states (in place). A thread has four neighbouring entries; several
+// pieces' are requested before the first is used.
 template <bool GATED>
 __global__ void __launch_bounds__(256)
-recurrence_scan_kernel(const Args a, const PieceSpace ws) {
+recurrence_scan_kernel(const Args a, const PieceSpace ws, int piece_rows) {
+  constexpr int kAhead = 8;
+  __shared__ float s_f[256];
   const int seg = blockIdx.x, h = blockIdx.y;
   int first = 0;
-  for (int s = 0; s < seg; ++s) first += (a.cu_rows[s + 1] - a.cu_rows[s] + kPiece - 1) / kPiece;
+  for (int s = 0; s < seg; ++s) first += (a.cu_rows[s + 1] - a.cu_rows[s] + piece_rows - 1) / piece_rows;
   const int rows = a.cu_rows[seg + 1] - a.cu_rows[seg];
-  const int pieces = (rows + kPiece - 1) / kPiece;
+  const int pieces = (rows + piece_rows - 1) / piece_rows;
   if (pieces < 2) return;
   const size_t plane = static_cast<size_t>(a.dim) * a.vdim;
-  float f = 1.f;
-  if (!GATED) {
-    const float p64 = a.decay_pow[h * kPowers + 64];
-    f = (p64 * p64) * (p64 * p64);
-  }
+  float constant = 1.f;
+  if (!GATED)
+    for (int i = 0; i < piece_rows; i += 64) constant *= a.decay_pow[h * kPowers + 64];
   const bool fresh = a.positions[a.cu_rows[seg]] == 0;
-  auto scan = [&](float* w, size_t stride, float run) {          // w: the first piece's entry
-    for (int i = 0; i < pieces; ++i, w += stride) {
-      const float own = i + 1 < pieces ? *w : 0.f;
-      *w = run;
-      if (GATED && i + 1 < pieces) f = expf(ws.log_decay[static_cast<size_t>(first + i) * a.heads + h]);
-      run = fmaf(run, f, own);
+  const size_t e = (static_cast<size_t>(blockIdx.z) * 256 + threadIdx.x) * 4;
+  const bool mine = e < plane;
+  float4* w = reinterpret_cast<float4*>(ws.state + (static_cast<size_t>(first) * a.heads + h) * plane + (mine ? e : 0));
+  const size_t stride = a.heads * plane / 4;
+  float4 run = make_float4(0.f, 0.f, 0.f, 0.f);
+  if (mine && !fresh) run = *reinterpret_cast<const float4*>(slot_state(a, seg, h) + e);
+  const bool norm = GATED && blockIdx.z == 0 && static_cast<int>(threadIdx.x) < a.dim;      // (dim <= 128)
+  float* wn = ws.normaliser + (static_cast<size_t>(first) * a.heads + h) * a.dim + threadIdx.x;
+  float run_n = norm && !fresh ? slot_normaliser(a, seg, h)[threadIdx.x] : 0.f;
+  for (int base = 0; base < pieces; base += 256) {
+    if (GATED) {
+      __syncthreads();
+      const int i = base + threadIdx.x;
+      if (i < pieces - 1) s_f[threadIdx.x] = expf(ws.log_decay[static_cast<size_t>(first + i) * a.heads + h]);
+      __syncthreads();
     }
-  };
-  const float* state = slot_state(a, seg, h);
-  for (size_t e = static_cast<size_t>(blockIdx.z) * 256 + threadIdx.x; e < plane; e += static_cast<size_t>(gridDim.z) * 256)
-    scan(ws.state + (static_cast<size_t>(first) * a.heads + h) * plane + e, a.heads * plane, fresh ? 0.f : state[e]);
-  if (GATED && blockIdx.z == 0)
-    for (int d = threadIdx.x; d < a.dim; d += 256)
-      scan(ws.normaliser + (static_cast<size_t>(first) * a.heads + h) * a.dim + d, static_cast<size_t>(a.heads) * a.dim,
-           fresh ? 0.f : slot_normaliser(a, seg, h)[d]);
+    const int stop = min(pieces, base + 256);
+    for (int i0 = base; i0 < stop; i0 += kAhead) {
+      float4 own[kAhead];
+      float own_n[kAhead];
+#pragma unroll
+      for (int u = 0; u < kAhead; ++u) {                 // (nobody needs the last piece's contribution: it has none)
+        const bool there = i0 + u < min(stop, pieces - 1);
+        own[u] = there && mine ? w[(i0 + u) * stride] : make_float4(0.f, 0.f, 0.f, 0.f);
+        own_n[u] = there && norm ? wn[static_cast<size_t>(i0 + u) * a.heads * a.dim] : 0.f;
+      }
+#pragma unroll
+      for (int u = 0; u < kAhead; ++u) {
+        if (i0 + u >= stop) break;
+        const float f = !GATED ? constant : i0 + u < pieces - 1 ? s_f[i0 + u - base] : 0.f;
+        if (mine) w[(i0 + u) * stride] = run;
+        run = make_float4(fmaf(run.x, f, own[u].x), fmaf(run.y, f, own[u].y), fmaf(run.z, f, own[u].z), fmaf(run.w, f, own[u].w));
+        if (norm) wn[static_cast<size_t>(i0 + u) * a.heads * a.dim] = run_n;
+        run_n = fmaf(run_n, f, own_n[u]);
+      }
+    }
+  }
 }
 
 // ---- matrix memory ---------------------------------------------------------------------------------------------------
@@ -524,31 +562,41 @@ __device__ __forceinline__ void log_gates(const Gates& g, int row, int heads, in
   *forget = log_sigmoid(g.cap * tanhf((z[heads + h] + g.forget_bias[h]) / g.cap));
 }
 
-// One block per (sequence, head), 256 tokens at a time. m_t = max(m_(t-1) + f_t, i_t) is a scan of pairs
+// One block per (sequence, head), 1024 tokens at a time. m_t = max(m_(t-1) + f_t, i_t) is a scan of pairs
 // (sum of f, maximum): (F1, M1) before (F2, M2) gives (F1 + F2, max(M1 + F2, M2)).
-__global__ void __launch_bounds__(256)
+constexpr int kGateThreads = 1024;
+__global__ void __launch_bounds__(kGateThreads)
 memory_gates_kernel(const Args a, const Gates g, float* __restrict__ log_decay, float* __restrict__ log_take, float* __restrict__ maximum) {
-  __shared__ float s_f[8], s_m[8], s_top[257];
+  __shared__ float s_f[32], s_m[32], s_top[kGateThreads + 1];
   const int seg = blockIdx.x, h = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int row0 = a.cu_rows[seg], row1 = a.cu_rows[seg + 1];
   if (row0 >= row1) return;
   float* slot = slot_maximum(a, seg, h);
   float before = a.positions[row0] == 0 ? 0.f : *slot;
-  for (int base = row0; base < row1; base += 256) {
+  for (int base = row0; base < row1; base += kGateThreads) {
     const int row = base + threadIdx.x;
     float in = -INFINITY, forget = 0.f;
     if (row < row1) log_gates(g, row, a.heads, h, &in, &forget);
-    float f = forget, m = in;
+    auto scan = [&](float& f, float& m) {   // inclusive, over a warp
 #pragma unroll
-    for (int off = 1; off < 32; off <<= 1) {
-      const float fu = __shfl_up_sync(0xffffffffu, f, off), mu = __shfl_up_sync(0xffffffffu, m, off);
-      if (lane >= off) { m = fmaxf(mu + f, m); f += fu; }
-    }
+      for (int off = 1; off < 32; off <<= 1) {
+        const float fu = __shfl_up_sync(0xffffffffu, f, off), mu = __shfl_up_sync(0xffffffffu, m, off);
+        if (lane >= off) { m = fmaxf(mu + f, m); f += fu; }
+      }
+    };
+    float f = forget, m = in;
+    scan(f, m);
     if (lane == 31) { s_f[warp] = f; s_m[warp] = m; }
     __syncthreads();
-    float top = before;                     // the maximum ahead of this warp's tokens
-    for (int w = 0; w < warp; ++w) top = fmaxf(top + s_f[w], s_m[w]);
-    top = fmaxf(top + f, m);
+    if (warp == 0) {
+      float wf = s_f[lane], wm = s_m[lane];
+      scan(wf, wm);
+      s_f[lane] = wf;
+      s_m[lane] = wm;
+    }
+    __syncthreads();
+    const float ahead = warp == 0 ? before : fmaxf(before + s_f[warp - 1], s_m[warp - 1]);      // of this warp's tokens
+    const float top = fmaxf(ahead + f, m);
     s_top[threadIdx.x + 1] = top;
     if (threadIdx.x == 0) s_top[0] = before;
     __syncthreads();
@@ -558,7 +606,7 @@ memory_gates_kernel(const Args a, const Gates g, float* __restrict__ log_decay, 
       log_take[at] = in - top;
       maximum[at] = top;
     }
-    before = s_top[min(row1 - base, 256)];
+    before = s_top[min(row1 - base, kGateThreads)];
     __syncthreads();
   }
   if (threadIdx.x == 0) *slot = before;
@@ -577,6 +625,38 @@ memory_norm_kernel(const T* __restrict__ o, const float* __restrict__ normaliser
   const int row = unit / heads, h = unit % heads;
   const float by = over_normaliser(normaliser[unit], maximum[unit]);
   const T* src = o + static_cast<size_t>(unit) * vdim;
+  const T* gsrc = gate + static_cast<size_t>(row) * gate_stride + static_cast<size_t>(h) * vdim;
+  const float* wsrc = w + static_cast<size_t>(h) * vdim;
+  T* dst = out + static_cast<size_t>(unit) * vdim;
+  constexpr int N = 2;                  // pieces per lane that stay in registers, everything requested before the sum
+  if (vdim <= 32 * VEC * N) {
+    float x[N][VEC], gt[N][VEC], wv[N][VEC], ss = 0.f;
+#pragma unroll
+    for (int k = 0; k < N; ++k) {
+      const int c = (k * 32 + lane) * VEC;
+      if (c < vdim) {
+        load_vec<T, VEC>(src + c, x[k]);
+        load_vec<T, VEC>(gsrc + c, gt[k]);
+        load_vec<float, VEC>(wsrc + c, wv[k]);
+      }
+    }
+#pragma unroll
+    for (int k = 0; k < N; ++k)
+      if ((k * 32 + lane) * VEC < vdim)
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) ss = fmaf(x[k][i] * by, x[k][i] * by, ss);
+    const float inv = by / sqrtf(warp_sum(ss) / static_cast<float>(vdim) + eps);
+#pragma unroll
+    for (int k = 0; k < N; ++k) {
+      const int c = (k * 32 + lane) * VEC;
+      if (c < vdim) {
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) x[k][i] = x[k][i] * inv * wv[k][i] * sigmoid_exact(gt[k][i]);
+        store_vec<T, VEC>(dst + c, x[k]);
+      }
+    }
+    return;
+  }
   float ss = 0.f;
   for (int c = lane * VEC; c < vdim; c += 32 * VEC) {
     float x[VEC];
@@ -588,16 +668,16 @@ memory_norm_kernel(const T* __restrict__ o, const float* __restrict__ normaliser
   for (int c = lane * VEC; c < vdim; c += 32 * VEC) {
     float x[VEC], gt[VEC], wv[VEC];
     load_vec<T, VEC>(src + c, x);
-    load_vec<T, VEC>(gate + static_cast<size_t>(row) * gate_stride + static_cast<size_t>(h) * vdim + c, gt);
-    load_vec<float, VEC>(w + static_cast<size_t>(h) * vdim + c, wv);
+    load_vec<T, VEC>(gsrc + c, gt);
+    load_vec<float, VEC>(wsrc + c, wv);
 #pragma unroll
     for (int i = 0; i < VEC; ++i) x[i] = x[i] * inv * wv[i] * sigmoid_exact(gt[i]);
-    store_vec<T, VEC>(out + static_cast<size_t>(unit) * vdim + c, x);
+    store_vec<T, VEC>(dst + c, x);
   }
 }
 
 template <typename T>
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(256, 4)
 memory_step_kernel(const Args a, const Gates g, const T* __restrict__ gate, long long gate_stride, const float* __restrict__ w, float eps) {
   __shared__ float4 s_red[256];
   __shared__ float scratch[32];
@@ -691,26 +771,35 @@ size_t chunk_smem(int dim) {
   return (static_cast<size_t>(2) * kChunk * (dim + 8) + static_cast<size_t>(3) * kChunk * kPitchV + static_cast<size_t>(2) * dim * kPitchV) * 2;
 }
 
+// Shorter pieces while all of them still run at once.
+int choose_piece(int rows, int segments, int heads, int vdim) {
+  int piece = kPiece;
+  const long long per_item = static_cast<long long>(heads) * ((vdim + kCols - 1) / kCols);
+  while (rows > kPiece && piece > kChunk && per_item * ragged_items(rows, segments, piece / 2) <= 2 * kNumSMs) piece /= 2;
+  return piece;
+}
+
 template <int MT, bool LOCAL, bool GATED>
-int launch_chunk(const Args& a, const PieceSpace& ws, cudaStream_t st) {
+int launch_chunk(const Args& a, const PieceSpace& ws, int piece, cudaStream_t st) {
   auto kern = recurrence_chunk_kernel<MT, LOCAL, GATED>;
   const size_t smem = chunk_smem(a.dim);
   cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
   if (e != cudaSuccess) return static_cast<int>(e);
-  kern<<<dim3(ragged_items(a.rows, a.segments, kPiece), a.heads, (a.vdim + kCols - 1) / kCols), 128, smem, st>>>(a, ws);
+  kern<<<dim3(ragged_items(a.rows, a.segments, piece), a.heads, (a.vdim + kCols - 1) / kCols), 128, smem, st>>>(a, ws, piece);
   return launch_status();
 }
 
 template <bool GATED>
 int launch_passes(const Args& a, float* workspace, bool pieces, cudaStream_t st) {
-  const PieceSpace ws = piece_space(a, workspace, ragged_items(a.rows, a.segments, kPiece));
+  const int piece = choose_piece(a.rows, a.segments, a.heads, a.vdim);
+  const PieceSpace ws = piece_space(a, workspace, ragged_items(a.rows, a.segments, piece));
   if (pieces) {
-    const int rc = a.dim <= 64 ? launch_chunk<1, true, GATED>(a, ws, st) : launch_chunk<2, true, GATED>(a, ws, st);
+    const int rc = a.dim <= 64 ? launch_chunk<1, true, GATED>(a, ws, piece, st) : launch_chunk<2, true, GATED>(a, ws, piece, st);
     if (rc != 0) return rc;
     const int z = (a.dim * a.vdim + 1023) / 1024;
-    recurrence_scan_kernel<GATED><<<dim3(a.segments, a.heads, z), 256, 0, st>>>(a, ws);
+    recurrence_scan_kernel<GATED><<<dim3(a.segments, a.heads, z), 256, 0, st>>>(a, ws, piece);
   }
-  return a.dim <= 64 ? launch_chunk<1, false, GATED>(a, ws, st) : launch_chunk<2, false, GATED>(a, ws, st);
+  return a.dim <= 64 ? launch_chunk<1, false, GATED>(a, ws, piece, st) : launch_chunk<2, false, GATED>(a, ws, piece, st);
 }
 
 template <typename T, bool GATED>
@@ -761,7 +850,7 @@ extern "C" int cacheir_b200_recurrence_chunked_supported(int dim, int vdim, int 
 
 extern "C" size_t cacheir_b200_recurrence_workspace_bytes(int rows, int segments, int heads, int dim, int vdim) {
   if (rows <= kPiece) return 0;
-  return static_cast<size_t>(ragged_items(rows, segments, kPiece)) * heads * (static_cast<size_t>(dim) * (vdim + 1) + 1) * 4;
+  return static_cast<size_t>(ragged_items(rows, segments, choose_piece(rows, segments, heads, vdim))) * heads * (static_cast<size_t>(dim) * (vdim + 1) + 1) * 4;
 }
 
 extern "C" int cacheir_b200_recurrence_chunked(const cacheir_b200_recurrence_args* a, void* workspace, size_t workspace_bytes, void* stream) {
@@ -784,7 +873,7 @@ extern "C" int cacheir_b200_memory_gates(const cacheir_b200_recurrence_args* a, 
   if (a->rows <= 0) return 0;
   const Gates g{logits, stride, in_bias, forget_bias, cap};
   if (!recurrence_args_ok(*a) || a->decay_pow || !gates_ok(g, a->heads) || !log_decay || !log_take || !maximum) return CACHEIR_B200_EINVAL;
-  memory_gates_kernel<<<dim3(a->segments, a->heads), 256, 0, as_stream(stream)>>>(*a, g, log_decay, log_take, maximum);
+  memory_gates_kernel<<<dim3(a->segments, a->heads), kGateThreads, 0, as_stream(stream)>>>(*a, g, log_decay, log_take, maximum);
   return launch_status();
 }
 

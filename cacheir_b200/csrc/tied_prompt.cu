@@ -421,17 +421,18 @@ tied_prompt_kernel(const __grid_constant__ CUtensorMap tmap_kv, const __grid_con
 }
 
 constexpr size_t kSmemLimit = 227 * 1024;
-int prompt_tiles(int dim) { return dim <= 128 ? 2 : 1; }
 int row_boxes(int width) { return (width + 63) / 64; }
-size_t prompt_fixed(int dim, int width, int key_from) {
-  const int tiles = prompt_tiles(dim);
+size_t prompt_fixed(int tiles, int width, int key_from) {
   return 1024 + static_cast<size_t>(tiles) * (row_boxes(width) - key_from / 64 + 2) * kTile * 128 + kMaxStages * kTiedPage * 4 + (2 * kMaxStages + 13) * 8 + 16;
 }
-int prompt_stages(int dim, int width, int key_from) {
-  const size_t fixed = prompt_fixed(dim, width, key_from), page = static_cast<size_t>(row_boxes(width)) * kTiedBox;
+int prompt_stages(int tiles, int width, int key_from) {
+  const size_t fixed = prompt_fixed(tiles, width, key_from), page = static_cast<size_t>(row_boxes(width)) * kTiedBox;
   const int s = fixed > kSmemLimit ? 0 : static_cast<int>((kSmemLimit - fixed) / page);
   return s > kMaxStages ? kMaxStages : (s >= 2 ? s : 0);
 }
+
+// Two tiles where tensor memory has room for their outputs and shared memory for their queries.
+int prompt_tiles(int dim, int width, int key_from) { return dim <= 128 && prompt_stages(2, width, key_from) > 0 ? 2 : 1; }
 
 // Odd polynomial for cap2 * tanh(reach * y) on [-1, 1]: y times the interpolant, at the Chebyshev nodes of [0, 1], of the
 // even quotient as a function of y^2. Double precision. Returns the number of terms: the quotient's poles lie at
@@ -460,7 +461,7 @@ int fit_tanh(double cap2, double reach, float (&coef)[kTerms]) {
 template <int TILES, bool FIXED, int TERMS>
 int launch_prompt(const PromptParams& p, const void* q, int items, cudaStream_t st) {
   const cacheir_b200_tied_args& a = p.a;
-  size_t smem = prompt_fixed(a.dim, a.width, a.key_from) + static_cast<size_t>(p.stages) * p.boxes * kTiedBox;
+  size_t smem = prompt_fixed(TILES, a.width, a.key_from) + static_cast<size_t>(p.stages) * p.boxes * kTiedBox;
   const size_t least = kSmemLimit / 2 + 1024;           // one CTA per SM: one that waited for tensor memory would be late
   if (smem < least) smem = least;
   CUtensorMap tkv, tq;
@@ -500,7 +501,7 @@ using namespace cb200;
 extern "C" int cacheir_b200_tied_prompt_supported(int heads, int kv_heads, int dim, int width, int key_from, int page_size, int dtype) {
   return dtype == CACHEIR_B200_BF16 && page_size == kTiedPage && kv_heads > 0 && heads % kv_heads == 0 && dim >= 8 && dim % 8 == 0 &&
          dim <= 256 && width >= dim && width % 8 == 0 && key_from >= 0 && key_from % 8 == 0 && key_from < width &&
-         prompt_stages(dim, width, key_from) > 0 ? 1 : 0;
+         prompt_stages(1, width, key_from) > 0 ? 1 : 0;
 }
 
 extern "C" int cacheir_b200_tied_attention_prompt(const cacheir_b200_tied_args* args, const void* q, const void* gate, long long gate_stride,
@@ -529,13 +530,13 @@ extern "C" int cacheir_b200_tied_attention_prompt(const cacheir_b200_tied_args* 
     p.pre = static_cast<float>((a.scale < 0.f ? -1.0 : 1.0) / most);
     terms = fit_tanh(static_cast<double>(a.cap) * kLog2e, reach / a.cap, p.coef);
   }
-  const int group = a.heads / a.kv_heads, tiles = prompt_tiles(a.dim);
+  const int group = a.heads / a.kv_heads, tiles = prompt_tiles(a.dim, a.width, a.key_from);
   p.subs = (group + kTile - 1) / kTile;
   p.heads_per_cta = (group + p.subs - 1) / p.subs;
   p.tokens_per_tile = kTile / p.heads_per_cta;
   p.boxes = row_boxes(a.width);
   p.lead_boxes = a.key_from / 64;
-  p.stages = prompt_stages(a.dim, a.width, a.key_from);
+  p.stages = prompt_stages(tiles, a.width, a.key_from);
   p.n_cols = (a.dim + 15) / 16 * 16;
   const int cols = tiles * (p.n_cols + 2 * kTiedPage);
   p.tmem_cols = cols <= 128 ? 128 : cols <= 256 ? 256 : 512;

@@ -30,11 +30,11 @@ def _want(name, tokens):
 
 
 def _oracle(name, tokens):
-    """(logits, positions up to which no router had a close call)"""
+    """(logits, positions at which no router had a close call)"""
     key = (name, tuple(tokens))
     if key not in _ORACLE:
         w = {k: a.astype(np.float64) for k, a in _weights(name).items()}
-        _ORACLE[key] = clear_choices(CONFIGS[name], w, tokens, 0.02)
+        _ORACLE[key] = clear_choices(CONFIGS[name], w, tokens, 0.01)
     return _ORACLE[key]
 
 
@@ -102,7 +102,7 @@ def test_portions_of_any_size_give_the_same_logits(name, portion, dtype):
 
 def _replay(rt, name, dtype, rng, requests, *, live, step_rows):
     """Random mixed steps: up to `live` requests at a time, each step some of them, portions and single tokens mixed."""
-    waiting, active, errors = list(requests), {}, []
+    waiting, active, errors, clear = list(requests), {}, [], []
     while waiting or active:
         while waiting and len(active) < live:
             tokens = waiting.pop(0)
@@ -115,6 +115,7 @@ def _replay(rt, name, dtype, rng, requests, *, live, step_rows):
         wanted = [sorted(set(int(p) for p in rng.integers(0, len(b), 3))) if rng.random() < 0.7 else [] for b in batches]
         logits = rt.run_step_batch([a[2] for a in chosen], batches, wanted)
         rows = [_want(name, a[0])[a[1] + p] for a, places in zip(chosen, wanted) for p in places]
+        clear += [_oracle(name, a[0])[1][a[1] + p] for a, places in zip(chosen, wanted) for p in places]
         assert logits.shape[0] == len(rows)
         if rows:
             errors.extend(row_errors(logits.float().cpu().numpy(), np.stack(rows)))
@@ -123,8 +124,9 @@ def _replay(rt, name, dtype, rng, requests, *, live, step_rows):
             if a[1] == len(a[0]):
                 a[2].kv_cache.clear()
                 del active[id(a[0])]
-    errors = np.array(errors)
-    assert np.isfinite(errors).all() and (errors > TOL[dtype]).sum() <= (0 if dtype == "float32" else len(errors) // 12), np.sort(errors)[-8:]
+    errors, over = np.array(errors), np.array(errors) > TOL[dtype]
+    assert np.isfinite(errors).all() and (over & clear).sum() <= (0 if dtype == "float32" else len(errors) // 20), np.sort(errors)[-8:]
+    assert dtype == "bfloat16" or not over.any()
     return len(errors)
 
 

@@ -303,9 +303,9 @@ def test_memory_token_by_token_kernel(shape, dtype):
 def test_memory_portions_and_decoding_carry_the_state(shape, dtype):
     chunked = dtype == "bfloat16" and shape[1] % 16 == 0 and shape[1] <= 128
     form = "chunked" if chunked else "simple"
-    m = Memory(*shape, (340, 9, 128), dtype=dtype, seed=shape[2])
+    m = Memory(*shape, (340, 10, 129), dtype=dtype, seed=shape[2])
     steps = [("step", (1, 1, 1))] * 4
-    m.check([(form, (2, 3, 64))] + steps + [(form, (270, 0, 2)), (form, (57, 2, 57))] + steps[:1] + [("simple", (2, 0, 0))] + steps[:0]
+    m.check([(form, (2, 3, 64))] + steps + [(form, (270, 0, 2)), (form, (57, 2, 57))] + steps[:1] + [("simple", (2, 0, 0))]
             + [(form, (340, 340, 340))], 1e-4 if dtype == "float32" else 1.5e-2)
 
 
@@ -417,7 +417,7 @@ def test_combine_with_identity_experts_and_a_gated_shared_one(rows, width, top, 
 
 # ---- residual rows and products --------------------------------------------------------------------------------------------
 @pytest.mark.parametrize("dtype", sorted(DTYPES))
-@pytest.mark.parametrize("rows,width", [(1, 1), (3, 90), (40, 2304)])
+@pytest.mark.parametrize("rows,width", [(1, 1), (3, 90), (40, 2304), (2, 4100)])
 def test_residual_rows(rows, width, dtype):
     from cacheir_b200 import hybrid_ops as H
 
