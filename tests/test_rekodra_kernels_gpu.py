@@ -166,7 +166,7 @@ def test_attention_with_one_norm_over_all_heads(shape, rot, kernel, portions):
 @pytest.mark.parametrize("splits", [1, 2, 5])
 def test_splits_of_rows_with_values_of_their_own(splits):
     rng = np.random.default_rng(splits)
-    got, want = _attend(rng, (4, 2, 48, 96), STEPS, dtype="bfloat16", kernel="step", own=True, whole=False, splits=splits)
+    got, want = _attend(rng, (4, 2, 56, 88), STEPS, dtype="bfloat16", kernel="step", own=True, whole=False, splits=splits)
     _rows_close(got, want, 2e-2)
 
 
@@ -282,7 +282,7 @@ class Memory:
         assert at == list(self.lengths)
 
 
-MEMORY_SHAPES = [(3, 48, 48), (2, 128, 64), (1, 16, 200), (4, 64, 8), (2, 112, 136)]
+MEMORY_SHAPES = [(3, 48, 40), (2, 128, 64), (1, 16, 200), (4, 64, 8), (2, 112, 136)]
 
 
 @pytest.mark.parametrize("shape", MEMORY_SHAPES, ids=str)
@@ -299,7 +299,7 @@ def test_memory_token_by_token_kernel(shape, dtype):
 
 
 @pytest.mark.parametrize("dtype", sorted(DTYPES))
-@pytest.mark.parametrize("shape", [(3, 48, 48), (2, 128, 64), (2, 17, 4), (1, 300, 1024), (1, 1, 12)], ids=str)
+@pytest.mark.parametrize("shape", [(3, 48, 40), (2, 128, 64), (2, 17, 4), (1, 300, 1024), (1, 1, 12)], ids=str)
 def test_memory_portions_and_decoding_carry_the_state(shape, dtype):
     chunked = dtype == "bfloat16" and shape[1] % 16 == 0 and shape[1] <= 128
     form = "chunked" if chunked else "simple"
