@@ -14,6 +14,7 @@ from .kv_cache import B200KVPageAllocator, B200PagedKVCache, KVPage
 from .models import load_model
 from .registry import B200_BACKEND, Backend, BackendRegistry, default_registry
 from .rekodra import RekodraConfig, build_rekodra_artifact
+from .zimorax import ZimoraxConfig, build_zimorax_artifact
 from .topunex import TopunexConfig, build_topunex_artifact
 
 __all__ = [
@@ -21,7 +22,7 @@ __all__ = [
     "B200KVPageAllocator", "B200PagedKVCache", "KVPage",
     "CompileArtifact", "Graph", "ModelConfig", "Node", "build_decoder_artifact", "build_decoder_graph",
     "GutoraxConfig", "build_gutorax_artifact", "TopunexConfig", "build_topunex_artifact", "RekodraConfig",
-    "build_rekodra_artifact", "load_model",
+    "build_rekodra_artifact", "ZimoraxConfig", "build_zimorax_artifact", "load_model",
     "B200_BACKEND", "Backend", "BackendRegistry", "default_registry",
 ]
 

@@ -1,5 +1,6 @@
 """ctypes binding of libcacheir_b200.so (the C ABI declared in include/cacheir_b200.h) and of the libraries of the
-ragged families: libcacheir_b200_ragged.so, _hybrid.so and _experts.so (headers of the same names).
+ragged families: libcacheir_b200_ragged.so, _hybrid.so, _recurrence.so, _experts.so, _talking.so and _delta.so (headers of the
+same names).
 
 There is no fallback: if the shared library is missing the import of any
 compute entry point raises, telling the user to build it.
@@ -11,7 +12,7 @@ from ctypes import c_char_p, c_float, c_int, c_longlong, c_size_t, c_void_p
 from pathlib import Path
 
 LIB_PATH = Path(__file__).resolve().parent / "lib" / "libcacheir_b200.so"
-GROUP_PATHS = {name: LIB_PATH.with_name(f"libcacheir_b200_{name}.so") for name in ("ragged", "hybrid", "recurrence", "experts")}
+GROUP_PATHS = {name: LIB_PATH.with_name(f"libcacheir_b200_{name}.so") for name in ("ragged", "hybrid", "recurrence", "experts", "talking", "delta")}
 
 # name -> (restype, argtypes); mirrors include/cacheir_b200.h one to one
 SIGNATURES: dict[str, tuple[object, list[object]]] = {
@@ -135,7 +136,35 @@ class RecurrenceArgs(ctypes.Structure):
                 ("heads", c_int), ("dim", c_int), ("vdim", c_int), ("q", c_void_p), ("k", c_void_p), ("v", c_void_p),
                 ("stride", c_longlong), ("decay_pow", c_void_p), ("state", c_void_p), ("num_slots", c_int), ("out", c_void_p),
                 ("dtype", c_int), ("slot_stride", c_longlong), ("log_decay", c_void_p), ("log_take", c_void_p),
-                ("normaliser", c_void_p), ("q_scale", c_float)]
+                ("normaliser", c_void_p), ("q_scale", c_float), ("key_heads", c_int), ("skip", c_void_p)]
+
+
+class ConvArgs(ctypes.Structure):
+    """cacheir_b200_conv_args"""
+
+    _fields_ = [("positions", c_void_p), ("cu_rows", c_void_p), ("slots", c_void_p),
+                ("rows", c_int), ("segments", c_int), ("channels", c_int), ("taps", c_int), ("x", c_void_p), ("stride", c_longlong),
+                ("w", c_void_p), ("bias", c_void_p), ("state", c_void_p), ("slot_stride", c_longlong), ("num_slots", c_int), ("dtype", c_int),
+                ("out", c_void_p), ("out_stride", c_longlong)]
+
+
+class DeltaArgs(ctypes.Structure):
+    """cacheir_b200_delta_args"""
+
+    _fields_ = [("positions", c_void_p), ("cu_rows", c_void_p), ("slots", c_void_p),
+                ("rows", c_int), ("segments", c_int), ("heads", c_int), ("key_heads", c_int), ("dim", c_int), ("vdim", c_int),
+                ("q", c_void_p), ("k", c_void_p), ("v", c_void_p), ("stride", c_longlong), ("z", c_void_p), ("z_stride", c_longlong),
+                ("bias", c_void_p), ("log_rate", c_void_p), ("state", c_void_p), ("slot_stride", c_longlong), ("num_slots", c_int),
+                ("dtype", c_int), ("out", c_void_p)]
+
+
+class TalkingArgs(ctypes.Structure):
+    """cacheir_b200_talking_args"""
+
+    _fields_ = [("positions", c_void_p), ("row_seg", c_void_p), ("cu_rows", c_void_p), ("page_table", c_void_p),
+                ("rows", c_int), ("segments", c_int), ("max_pages", c_int), ("page_size", c_int), ("num_slots", c_int),
+                ("heads", c_int), ("kv_heads", c_int), ("dim", c_int), ("vdim", c_int), ("window", c_int), ("scale", c_float),
+                ("talk", c_void_p), ("keys", c_void_p), ("values", c_void_p), ("dtype", c_int), ("decode", c_int)]
 
 
 class TiedArgs(ctypes.Structure):
@@ -165,13 +194,18 @@ GROUP_SIGNATURES: dict[str, dict[str, tuple[object, list[object]]]] = {
         "cacheir_b200_dyt_rows": (c_int, [c_void_p] * 4 + [c_float, c_void_p, c_int, c_int, c_int, c_void_p]),
         "cacheir_b200_rms_rows": (c_int, [c_void_p] * 3 + [c_float, c_void_p, c_int, c_int, c_int, c_void_p]),
         "cacheir_b200_residual_dyt": (c_int, [c_void_p] * 4 + [c_float, c_int, c_int] + _NEXT + [c_int, c_void_p]),
-        "cacheir_b200_residual_add": (c_int, [c_void_p] * 2 + [c_int, c_int] + _NEXT + [c_int, c_void_p]),
+        "cacheir_b200_layer_norm_rows": (c_int, [c_void_p] * 3 + [c_float, c_void_p, c_int, c_int, c_int, c_void_p]),
+        "cacheir_b200_join_embedding": (c_int, [c_void_p] * 4 + [c_int] * 4 + [c_void_p]),
+        "cacheir_b200_residual_add": (c_int, [c_void_p] * 3 + [c_int, c_int] + _NEXT + [c_int, c_void_p]),
         "cacheir_b200_residual_rms_pair": (c_int, [c_void_p] * 5 + [c_float, c_float, c_int, c_int] + _NEXT + [c_int, c_void_p]),
         "cacheir_b200_residual_rms": (c_int, [c_void_p] * 3 + [c_float, c_int, c_int] + _NEXT + [c_int, c_void_p]),
         "cacheir_b200_gated_rms": (c_int, [c_void_p, c_void_p, c_longlong, c_void_p, c_float, c_void_p, c_int, c_int, c_int, c_void_p]),
         "cacheir_b200_glu_pairs": (c_int, [c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_int, c_void_p]),
         "cacheir_b200_gelu_embed": (c_int, [c_void_p] * 3 + [c_longlong, c_int, c_void_p, c_int, c_int, c_int, c_int, c_void_p]),
         "cacheir_b200_silu_cols": (c_int, [c_void_p, c_int, c_longlong, c_int, c_int, c_void_p]),
+        "cacheir_b200_relu2_cols": (c_int, [c_void_p, c_int, c_longlong, c_int, c_int, c_void_p]),
+        "cacheir_b200_gated_parts_rms": (c_int, [c_void_p, c_void_p, c_longlong, c_void_p, c_int, c_int, c_float, c_void_p, c_int, c_int, c_int,
+                                                 c_int, c_void_p]),
         "cacheir_b200_ragged_device_status": (c_int, [c_int]),
     },
     "hybrid": {
@@ -195,7 +229,30 @@ GROUP_SIGNATURES: dict[str, dict[str, tuple[object, list[object]]]] = {
         "cacheir_b200_memory_norm": (c_int, [c_void_p] * 4 + [c_longlong, c_void_p, c_float, c_void_p, c_int, c_int, c_int, c_int, c_void_p]),
         "cacheir_b200_memory_step": (
             c_int, [c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_float, c_void_p, c_longlong, c_void_p, c_float, c_void_p]),
+        "cacheir_b200_state_space_gates": (c_int, [c_void_p, c_void_p, c_longlong] + [c_void_p] * 5),
+        "cacheir_b200_state_space_step": (c_int, [c_void_p, c_void_p, c_longlong] + [c_void_p] * 3),
         "cacheir_b200_recurrence_device_status": (c_int, [c_int]),
+    },
+    "talking": {
+        "cacheir_b200_talking_prepare": (
+            c_int, [c_void_p, c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_longlong, c_int, c_void_p, c_int, c_float, c_int, c_void_p,
+                    c_void_p]),
+        "cacheir_b200_talking_simple": (c_int, [c_void_p] * 4),
+        "cacheir_b200_talking_step_supported": (c_int, [c_int] * 6),
+        "cacheir_b200_talking_step_splits": (c_int, [c_int] * 8),
+        "cacheir_b200_talking_step": (c_int, [c_void_p] * 3 + [c_int, c_void_p]),
+        "cacheir_b200_talking_prompt_supported": (c_int, [c_int] * 6),
+        "cacheir_b200_talking_prompt": (c_int, [c_void_p] * 4),
+        "cacheir_b200_talking_device_status": (c_int, [c_int]),
+    },
+    "delta": {
+        "cacheir_b200_short_conv": (c_int, [c_void_p, c_void_p]),
+        "cacheir_b200_delta_simple": (c_int, [c_void_p, c_void_p]),
+        "cacheir_b200_delta_step": (c_int, [c_void_p, c_void_p, c_longlong, c_void_p, c_float, c_void_p]),
+        "cacheir_b200_delta_chunked_supported": (c_int, [c_int] * 3),
+        "cacheir_b200_delta_workspace_bytes": (c_size_t, [c_int] * 3),
+        "cacheir_b200_delta_chunked": (c_int, [c_void_p, c_void_p, c_size_t, c_void_p]),
+        "cacheir_b200_delta_device_status": (c_int, [c_int]),
     },
     "experts": {
         "cacheir_b200_tied_prepare": (

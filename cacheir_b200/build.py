@@ -6,8 +6,9 @@ Plain C-ABI shared objects (no torch, no pybind), each a group of the .cu files
 under csrc/ compiled with -gencode arch=compute_100a,code=sm_100a and linked
 with the static CUDA runtime: `core` (libcacheir_b200.so, Llama-shaped models),
 `ragged` (dense products and row operators of the families with ragged steps),
-`hybrid` (latent attention), `recurrence` (linear recurrences, matrix memory) and
-`experts` (tied attention, mixtures of experts). A model family names the groups it needs, so a fresh
+`hybrid` (latent attention), `recurrence` (linear recurrences, matrix memory, state
+spaces), `experts` (tied attention, mixtures of experts), `talking` (talking-heads
+attention) and `delta` (short convolutions, delta rule). A model family names the groups it needs, so a fresh
 checkout compiles only those. Objects are rebuilt only when their source or a
 header is newer.
 """
@@ -31,6 +32,8 @@ GROUP_FILES = {
     "ragged": ("dense_gemm", "hybrid_glue") + SHARED,
     "hybrid": ("latent_attention",),
     "recurrence": ("linear_recurrence",),
+    "talking": ("talking_attention", "talking_prompt"),
+    "delta": ("short_conv", "delta_rule"),
     "experts": ("tied_attention", "tied_prompt", "grouped_gemm", "expert_routing"),
 }
 LIB_PATHS = {"core": LIB_DIR / "libcacheir_b200.so", **{name: LIB_DIR / f"libcacheir_b200_{name}.so" for name in GROUP_FILES}}

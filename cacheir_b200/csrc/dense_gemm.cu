@@ -56,6 +56,7 @@ extern "C" int cacheir_b200_dense_gemm(const cacheir_b200_dense_args* args, void
     case CACHEIR_B200_DENSE_BF16: return p.y && tail_ok ? launch_mt<CACHEIR_B200_DENSE_BF16>(p, st) : CACHEIR_B200_EINVAL;
     case CACHEIR_B200_DENSE_F32: return p.y ? launch_mt<CACHEIR_B200_DENSE_F32>(p, st) : CACHEIR_B200_EINVAL;
     case CACHEIR_B200_DENSE_SILU: return p.y && tail_ok ? launch_mt<CACHEIR_B200_DENSE_SILU>(p, st) : CACHEIR_B200_EINVAL;
+    case CACHEIR_B200_DENSE_RELU2: return p.y ? launch_mt<CACHEIR_B200_DENSE_RELU2>(p, st) : CACHEIR_B200_EINVAL;
     case CACHEIR_B200_DENSE_GEGLU:
     case CACHEIR_B200_DENSE_SWIGLU:
     case CACHEIR_B200_DENSE_CLAMPED_GLU:

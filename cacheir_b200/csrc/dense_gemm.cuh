@@ -290,6 +290,8 @@ dense_gemm_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_const
             continue;
           } else if constexpr (EPI == CACHEIR_B200_DENSE_SILU) {
             if (n < p.act_cols) y = silu_exact(y);
+          } else if constexpr (EPI == CACHEIR_B200_DENSE_RELU2) {
+            y = relu_squared(y);
           } else if constexpr (EPI == CACHEIR_B200_DENSE_GATED) {
             y *= sigmoid_exact(f[j]);
           } else if constexpr (EPI == CACHEIR_B200_DENSE_GELU_EMBED) {

@@ -10,10 +10,13 @@ namespace cb200 {
 // (2 ulp) has no slow path to branch to, so that a thread's many elements overlap; past the exponential's range it is 0.
 __device__ __forceinline__ float sigmoid_exact(float z) { return __fdividef(1.f, 1.f + expf(-z)); }
 __device__ __forceinline__ float silu_exact(float z) { return z * sigmoid_exact(z); }
+__device__ __forceinline__ float relu_squared(float z) { return z > 0.f ? z * z : 0.f; }
 __device__ __forceinline__ float gelu_tanh(float z) {
   constexpr float kRoot2OverPi = 0.7978845608028654f;
   return 0.5f * z * (1.f + tanhf(kRoot2OverPi * fmaf(0.044715f * z * z, z, z)));
 }
+
+__device__ __forceinline__ float softplus(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
 
 __device__ __forceinline__ float clamped_glu(float gate, float up, float limit) {
   const float g = fminf(gate, limit), u = fminf(fmaxf(up, -limit), limit);

@@ -1,5 +1,5 @@
 // Row operators of the hybrid families that are not a GEMM epilogue: embedding into the 32-bit residual stream, Dynamic
-// Tanh, the RMS-normed residual add, the gated RMS norm behind a recurrence, and the stand-alone forms of the dense
+// Tanh, the (RMS-normed, scaled) residual add, layer norms, the gated RMS norms behind a recurrence, and the stand-alone forms of the dense
 // kernel's epilogues (used in 32-bit runs and for extents the tensor-core kernel does not take).
 #include "residual_rows.cuh"
 
@@ -132,17 +132,115 @@ embedding_rows_kernel(const T* __restrict__ table, const int64_t* __restrict__ i
   });
 }
 
-template <typename T, int VEC>
-__global__ void __launch_bounds__(kRowThreads)
-residual_add_kernel(float* x, const T* __restrict__ y, int width, RowNext nx) {
+// HELD: a thread's columns stay in registers from the first read to the last write
+constexpr int kAddThreads = 256, kAddPieces = 8;
+template <typename T, int VEC, bool HELD>
+__global__ void __launch_bounds__(kAddThreads)
+residual_add_kernel(float* x, const T* __restrict__ y, const float* __restrict__ scale, int width, RowNext nx) {
   __shared__ float scratch[32];
   const size_t row = blockIdx.x;
-  finish_row<T, VEC>(x + row * width, row, width, nx, scratch, [&](int c, float (&s)[VEC]) {
-    float v[VEC];
-    load_vec<T, VEC>(y + row * width + c, v);
+  x += row * width;
+  y += row * width;
+  auto added = [&](int c, float (&s)[VEC]) {
+    float v[VEC], f[VEC];
+    load_vec<T, VEC>(y + c, v);
+    if (scale) load_vec<float, VEC>(scale + c, f);
 #pragma unroll
-    for (int i = 0; i < VEC; ++i) s[i] += v[i];
-  });
+    for (int i = 0; i < VEC; ++i) s[i] = scale ? fmaf(v[i], f[i], s[i]) : s[i] + v[i];
+  };
+  if constexpr (HELD) {
+    float s[kAddPieces][VEC], sum = 0.f;
+    const bool centred = nx.mode == CACHEIR_B200_NEXT_LAYER;
+    const auto column = [](int k) { return (k * kAddThreads + static_cast<int>(threadIdx.x)) * VEC; };
+#pragma unroll
+    for (int k = 0; k < kAddPieces; ++k)
+      if (column(k) < width) load_vec<float, VEC>(x + column(k), s[k]);
+#pragma unroll
+    for (int k = 0; k < kAddPieces; ++k)
+      if (column(k) < width) {
+        added(column(k), s[k]);
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) sum = centred ? sum + s[k][i] : fmaf(s[k][i], s[k][i], sum);
+      }
+    T* out = static_cast<T*>(nx.out) + row * width;
+#pragma unroll
+    for (int k = 0; k < kAddPieces; ++k)
+      if (column(k) < width) {
+        store_vec<float, VEC>(x + column(k), s[k]);
+        if (nx.mode == CACHEIR_B200_NEXT_COPY) store_vec<T, VEC>(out + column(k), s[k]);
+      }
+    if (nx.mode != CACHEIR_B200_NEXT_RMS && !centred) return;
+    float mean = 0.f;
+    if (centred) {
+      mean = block_sum_all(sum, scratch) / static_cast<float>(width);
+      sum = 0.f;
+#pragma unroll
+      for (int k = 0; k < kAddPieces; ++k)
+        if (column(k) < width)
+#pragma unroll
+          for (int i = 0; i < VEC; ++i) sum = fmaf(s[k][i] - mean, s[k][i] - mean, sum);
+    }
+    const float inv = 1.f / sqrtf(block_sum_all(sum, scratch) / static_cast<float>(width) + nx.eps);
+#pragma unroll
+    for (int k = 0; k < kAddPieces; ++k)
+      if (column(k) < width) {
+        float w[VEC];
+        load_vec<float, VEC>(nx.w + column(k), w);
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) w[i] = (s[k][i] - mean) * inv * w[i];
+        store_vec<T, VEC>(out + column(k), w);
+      }
+  } else {
+    finish_row<T, VEC>(x, row, width, nx, scratch, added);
+  }
+}
+
+// out[j] = layer norm of residual row row_index[j]
+template <typename T, int VEC>
+__global__ void __launch_bounds__(512)
+layer_norm_rows_kernel(const float* __restrict__ x, const int32_t* __restrict__ row_index, const float* __restrict__ w, float eps,
+                       T* __restrict__ out, int width) {
+  __shared__ float scratch[32];
+  const size_t row = blockIdx.x;
+  const float* xr = x + (row_index ? static_cast<size_t>(max(row_index[row], 0)) : row) * width;
+  float sum = 0.f, ss = 0.f;
+  for (int c = threadIdx.x * VEC; c < width; c += 512 * VEC) {
+    float v[VEC];
+    load_vec<float, VEC>(xr + c, v);
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) sum += v[i];
+  }
+  const float mean = block_sum_all(sum, scratch) / static_cast<float>(width);
+  for (int c = threadIdx.x * VEC; c < width; c += 512 * VEC) {
+    float v[VEC];
+    load_vec<float, VEC>(xr + c, v);
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) ss = fmaf(v[i] - mean, v[i] - mean, ss);
+  }
+  const float inv = 1.f / sqrtf(block_sum_all(ss, scratch) / static_cast<float>(width) + eps);
+  for (int c = threadIdx.x * VEC; c < width; c += 512 * VEC) {
+    float v[VEC], wv[VEC];
+    load_vec<float, VEC>(xr + c, v);
+    load_vec<float, VEC>(w + c, wv);
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) v[i] = (v[i] - mean) * inv * wv[i];
+    store_vec<T, VEC>(out + row * width + c, v);
+  }
+}
+
+template <typename T, int VEC>
+__global__ void __launch_bounds__(256)
+join_embedding_kernel(const float* __restrict__ x, const T* __restrict__ table, const int64_t* __restrict__ ids, T* __restrict__ out, int width,
+                      int vocab) {
+  const size_t row = blockIdx.x;
+  const T* src = table + min(max(ids[row], static_cast<int64_t>(0)), static_cast<int64_t>(vocab - 1)) * width;
+  for (int c = (blockIdx.y * 256 + threadIdx.x) * VEC; c < width; c += gridDim.y * 256 * VEC) {
+    float v[VEC];
+    load_vec<float, VEC>(x + row * width + c, v);
+    store_vec<T, VEC>(out + row * 2 * width + c, v);
+    load_vec<T, VEC>(src + c, v);
+    store_vec<T, VEC>(out + row * 2 * width + width + c, v);
+  }
 }
 
 // HELD: a thread's columns (PIECES vectors at most) stay in registers from the first read to the last write, and what a later
@@ -265,6 +363,77 @@ gated_rms_kernel(const T* __restrict__ o, const T* __restrict__ gate, long long 
   }
 }
 
+// A unit is one part of one row; WARPS warps share it.
+template <typename T, int VEC, int WARPS>
+__global__ void __launch_bounds__(256)
+gated_parts_rms_kernel(const T* __restrict__ o, const T* __restrict__ gate, long long gate_stride, const float* __restrict__ w, int shared_weight,
+                       int gate_first, float eps, T* __restrict__ out, int units, int parts, int size) {
+  __shared__ float scratch[32];
+  const int unit = WARPS == 1 ? blockIdx.x * 8 + static_cast<int>(threadIdx.x >> 5) : static_cast<int>(blockIdx.x);
+  const int at = WARPS == 1 ? static_cast<int>(threadIdx.x & 31) : static_cast<int>(threadIdx.x);
+  if (unit >= units) return;
+  const int row = unit / parts, part = unit % parts;
+  const T* src = o + static_cast<size_t>(unit) * size;
+  const T* g = gate + static_cast<size_t>(row) * gate_stride + static_cast<size_t>(part) * size;
+  const float* weight = w + (shared_weight ? 0 : static_cast<size_t>(part) * size);
+  T* dst = out + static_cast<size_t>(unit) * size;
+  constexpr int kStep = 32 * WARPS * VEC, N = 4;         // pieces that stay in registers, everything requested before the sum
+  auto total = [&](float ss) { return WARPS == 1 ? warp_sum(ss) : block_sum_all(ss, scratch); };
+  auto gated = [&](float (&x)[VEC], const float (&gt)[VEC], float& ss) {
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) {
+      if (gate_first) x[i] *= silu_exact(gt[i]);
+      ss = fmaf(x[i], x[i], ss);
+    }
+  };
+  auto finish = [&](float (&x)[VEC], const float (&gt)[VEC], const float (&wv)[VEC], float inv) {
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) x[i] = x[i] * inv * wv[i] * (gate_first ? 1.f : silu_exact(gt[i]));
+  };
+  float ss = 0.f;
+  if (size <= kStep * N) {
+    float x[N][VEC], gt[N][VEC], wv[N][VEC];
+#pragma unroll
+    for (int k = 0; k < N; ++k) {
+      const int c = k * kStep + at * VEC;
+      if (c < size) {
+        load_vec<T, VEC>(src + c, x[k]);
+        load_vec<T, VEC>(g + c, gt[k]);
+        load_vec<float, VEC>(weight + c, wv[k]);
+      }
+    }
+#pragma unroll
+    for (int k = 0; k < N; ++k)
+      if (k * kStep + at * VEC < size) gated(x[k], gt[k], ss);
+    const float inv = 1.f / sqrtf(total(ss) / static_cast<float>(size) + eps);
+#pragma unroll
+    for (int k = 0; k < N; ++k) {
+      const int c = k * kStep + at * VEC;
+      if (c < size) {
+        finish(x[k], gt[k], wv[k], inv);
+        store_vec<T, VEC>(dst + c, x[k]);
+      }
+    }
+    return;
+  }
+  for (int c = at * VEC; c < size; c += kStep) {
+    float x[VEC], gt[VEC];
+    load_vec<T, VEC>(src + c, x);
+    load_vec<T, VEC>(g + c, gt);
+    gated(x, gt, ss);
+  }
+  const float inv = 1.f / sqrtf(total(ss) / static_cast<float>(size) + eps);
+  for (int c = at * VEC; c < size; c += kStep) {
+    float x[VEC], gt[VEC], wv[VEC], unused = 0.f;
+    load_vec<T, VEC>(src + c, x);
+    load_vec<T, VEC>(g + c, gt);
+    load_vec<float, VEC>(weight + c, wv);
+    gated(x, gt, unused);
+    finish(x, gt, wv, inv);
+    store_vec<T, VEC>(dst + c, x);
+  }
+}
+
 template <typename T>
 __global__ void __launch_bounds__(256)
 glu_pairs_kernel(const T* __restrict__ y, T* __restrict__ out, int ff, int epilogue, float limit) {
@@ -287,11 +456,14 @@ gelu_embed_kernel(const T* __restrict__ g, const int64_t* __restrict__ ids, cons
     Elem<T>::st(out + row * dim + c, gelu_tanh(Elem<T>::ld(g + row * dim + c)) * Elem<T>::ld(table + id * table_stride + table_col + c));
 }
 
-template <typename T>
+template <typename T, bool RELU2>
 __global__ void __launch_bounds__(256)
-silu_cols_kernel(T* __restrict__ y, long long stride, int cols) {
+activate_cols_kernel(T* __restrict__ y, long long stride, int cols) {
   T* yr = y + static_cast<size_t>(blockIdx.x) * stride;
-  for (int c = blockIdx.y * 256 + threadIdx.x; c < cols; c += gridDim.y * 256) Elem<T>::st(yr + c, silu_exact(Elem<T>::ld(yr + c)));
+  for (int c = blockIdx.y * 256 + threadIdx.x; c < cols; c += gridDim.y * 256) {
+    const float z = Elem<T>::ld(yr + c);
+    Elem<T>::st(yr + c, RELU2 ? relu_squared(z) : silu_exact(z));
+  }
 }
 
 // ---- plain tiled GEMM, float32 arithmetic: 64 tokens x 64 columns per CTA, 16 k at a time ---------------------------
@@ -358,7 +530,7 @@ extern "C" int cacheir_b200_scaled_embedding(const void* table, const int64_t* i
                                              void* next_out, int dtype, void* stream) {
   if (rows <= 0 || width <= 0) return 0;
   if (!table || !ids || !residual || vocab <= 0) return CACHEIR_B200_EINVAL;
-  if (accumulate || next_mode == CACHEIR_B200_NEXT_RMS) {
+  if (accumulate || row_next_norms(next_mode)) {
     if (!row_next_ok(next_mode, next_w, next_out)) return CACHEIR_B200_EINVAL;
     const RowNext rn{next_mode, next_w, next_alpha, next_out};
     const bool vec = width % 4 == 0 && aligned_to(table, 16) && aligned_to(residual, 16) && row_next_aligned(next_mode, next_w, next_out);
@@ -412,16 +584,47 @@ extern "C" int cacheir_b200_residual_dyt(float* residual, const void* y, const f
   return launch_status();
 }
 
-extern "C" int cacheir_b200_residual_add(float* residual, const void* y, int rows, int width, int next_mode, const float* next_w,
+extern "C" int cacheir_b200_layer_norm_rows(const float* residual, const int32_t* row_index, const float* w, float eps, void* out, int rows,
+                                            int width, int dtype, void* stream) {
+  if (rows <= 0 || width <= 0) return 0;
+  if (!residual || !w || !out) return CACHEIR_B200_EINVAL;
+  const bool vec = width % 4 == 0 && aligned_to(residual, 16) && aligned_to(w, 16) && aligned_to(out, 16);
+  CB200_HYBRID_DTYPE(dtype, {
+    if (vec) layer_norm_rows_kernel<T, 4><<<rows, 512, 0, as_stream(stream)>>>(residual, row_index, w, eps, static_cast<T*>(out), width);
+    else layer_norm_rows_kernel<T, 1><<<rows, 512, 0, as_stream(stream)>>>(residual, row_index, w, eps, static_cast<T*>(out), width);
+  });
+  return launch_status();
+}
+
+extern "C" int cacheir_b200_join_embedding(const float* residual, const void* table, const int64_t* ids, void* out, int rows, int width, int vocab,
+                                           int dtype, void* stream) {
+  if (rows <= 0 || width <= 0) return 0;
+  if (!residual || !table || !ids || !out || vocab <= 0) return CACHEIR_B200_EINVAL;
+  const bool vec = width % 4 == 0 && aligned_to(residual, 16) && aligned_to(table, 16) && aligned_to(out, 16);
+  CB200_HYBRID_DTYPE(dtype, {
+    if (vec) join_embedding_kernel<T, 4><<<row_grid(rows, width / 4), 256, 0, as_stream(stream)>>>(
+        residual, static_cast<const T*>(table), ids, static_cast<T*>(out), width, vocab);
+    else join_embedding_kernel<T, 1><<<row_grid(rows, width), 256, 0, as_stream(stream)>>>(
+        residual, static_cast<const T*>(table), ids, static_cast<T*>(out), width, vocab);
+  });
+  return launch_status();
+}
+
+extern "C" int cacheir_b200_residual_add(float* residual, const void* y, const float* scale, int rows, int width, int next_mode, const float* next_w,
                                          const float* next_b, float next_alpha, void* next_out, int dtype, void* stream) {
   if (rows <= 0 || width <= 0) return 0;
   if (!residual || !y || next_b || !row_next_ok(next_mode, next_w, next_out)) return CACHEIR_B200_EINVAL;
   const RowNext nx{next_mode, next_w, next_alpha, next_out};
-  const bool vec = width % 4 == 0 && aligned_to(residual, 16) && aligned_to(y, 16) && row_next_aligned(next_mode, next_w, next_out);
+  const bool vec = width % 4 == 0 && aligned_to(residual, 16) && aligned_to(y, 16) && (!scale || aligned_to(scale, 16)) &&
+                   row_next_aligned(next_mode, next_w, next_out);
+#define CB200_ADD(VEC, HELD) \
+  residual_add_kernel<T, VEC, HELD><<<rows, kAddThreads, 0, as_stream(stream)>>>(residual, static_cast<const T*>(y), scale, width, nx)
   CB200_HYBRID_DTYPE(dtype, {
-    if (vec) residual_add_kernel<T, 4><<<rows, kRowThreads, 0, as_stream(stream)>>>(residual, static_cast<const T*>(y), width, nx);
-    else residual_add_kernel<T, 1><<<rows, kRowThreads, 0, as_stream(stream)>>>(residual, static_cast<const T*>(y), width, nx);
+    if (vec && width <= 4 * kAddThreads * kAddPieces) CB200_ADD(4, true);
+    else if (vec) CB200_ADD(4, false);
+    else CB200_ADD(1, false);
   });
+#undef CB200_ADD
   return launch_status();
 }
 
@@ -437,7 +640,7 @@ extern "C" int cacheir_b200_residual_rms_pair(float* residual, const void* y1, c
   residual_rms_pair_kernel<T, VEC, HELD><<<rows, kPairThreads, 0, as_stream(stream)>>>(residual, static_cast<const T*>(y1), w1,        \
                                                                                       static_cast<const T*>(y2), w2, factor, eps, width, nx)
   CB200_HYBRID_DTYPE(dtype, {
-    if (vec && width <= 4 * kPairThreads * kPairPieces) CB200_PAIR(4, true);
+    if (vec && width <= 4 * kPairThreads * kPairPieces && next_mode != CACHEIR_B200_NEXT_LAYER) CB200_PAIR(4, true);
     else if (vec) CB200_PAIR(4, false);
     else CB200_PAIR(1, false);
   });
@@ -497,7 +700,34 @@ extern "C" int cacheir_b200_gelu_embed(const void* g, const int64_t* ids, const 
 extern "C" int cacheir_b200_silu_cols(void* y, int rows, long long stride, int cols, int dtype, void* stream) {
   if (rows <= 0 || cols <= 0) return 0;
   if (!y) return CACHEIR_B200_EINVAL;
-  CB200_HYBRID_DTYPE(dtype, (silu_cols_kernel<T><<<row_grid(rows, cols), 256, 0, as_stream(stream)>>>(static_cast<T*>(y), stride, cols)));
+  CB200_HYBRID_DTYPE(dtype, (activate_cols_kernel<T, false><<<row_grid(rows, cols), 256, 0, as_stream(stream)>>>(static_cast<T*>(y), stride, cols)));
+  return launch_status();
+}
+
+extern "C" int cacheir_b200_relu2_cols(void* y, int rows, long long stride, int cols, int dtype, void* stream) {
+  if (rows <= 0 || cols <= 0) return 0;
+  if (!y) return CACHEIR_B200_EINVAL;
+  CB200_HYBRID_DTYPE(dtype, (activate_cols_kernel<T, true><<<row_grid(rows, cols), 256, 0, as_stream(stream)>>>(static_cast<T*>(y), stride, cols)));
+  return launch_status();
+}
+
+extern "C" int cacheir_b200_gated_parts_rms(const void* o, const void* gate, long long gate_stride, const float* w, int shared_weight,
+                                            int gate_first, float eps, void* out, int rows, int cols, int parts, int dtype, void* stream) {
+  if (rows <= 0 || cols <= 0) return 0;
+  if (!o || !gate || !w || !out || parts <= 0 || cols % parts != 0) return CACHEIR_B200_EINVAL;
+  const int size = cols / parts, units = rows * parts, quad = 4 * (dtype == CACHEIR_B200_F32 ? 4 : 2);
+  const bool vec = size % 4 == 0 && gate_stride % 4 == 0 && aligned_to(o, quad) && aligned_to(gate, quad) && aligned_to(w, 16) && aligned_to(out, quad);
+  const bool wide = size > 512;
+#define CB200_PARTS(VEC, WARPS)                                                                                                         \
+  gated_parts_rms_kernel<T, VEC, WARPS><<<WARPS == 1 ? (units + 7) / 8 : units, 256, 0, as_stream(stream)>>>(                             \
+      static_cast<const T*>(o), static_cast<const T*>(gate), gate_stride, w, shared_weight, gate_first, eps, static_cast<T*>(out), units, parts, size)
+  CB200_HYBRID_DTYPE(dtype, {
+    if (vec && wide) CB200_PARTS(4, 8);
+    else if (vec) CB200_PARTS(4, 1);
+    else if (wide) CB200_PARTS(1, 8);
+    else CB200_PARTS(1, 1);
+  });
+#undef CB200_PARTS
   return launch_status();
 }
 

@@ -1,6 +1,7 @@
 // Linear recurrence S <- decay S + take k v^T, o = S^T q per head, float32 state carried per sequence slot, sm_100a.
-// decay is a constant per head and take one; or (GATED) both belong to the token and the head, given as logarithms, and a
-// vector n <- decay n + take k runs along, of which q . n is kept for whoever normalises o.
+// decay is a constant per head and take one; or (GATED) both belong to the token and the head, given as logarithms, and where
+// somebody normalises o a vector n <- decay n + take k runs along, of which q . n is kept. Neighbouring heads may share q and k,
+// and a multiple of v may be added to o.
 //
 // simple   any extents and types: one CTA per (sequence, head, 32 value columns) walks the tokens, state in shared memory
 // step     decode: one CTA per (sequence, head) streams the state once (16-byte accesses), HBM bound
@@ -13,6 +14,7 @@
 //          chunk, decay^(i-j) becomes exp(c_i - c_j + log take_j), and so on; n rides with the first value columns.
 // gates    matrix memory: log decay and log take from gate logits, relative to a running maximum (a scan over the tokens)
 // memory   matrix memory, decode: gates, state, normaliser, the head's norm and the output gate in one pass over the state
+// space    state space: its gates for prompts, and one decoded token (gates and recurrence in one pass over the state)
 #include "cacheir_b200_recurrence.h"
 #include "hybrid_common.cuh"
 #include "ragged.cuh"
@@ -43,6 +45,8 @@ __device__ __forceinline__ float* slot_maximum(const Args& a, int seg, int h) {
   return slot_base(a, seg) + static_cast<size_t>(a.heads) * a.dim * (a.vdim + 1) + h;
 }
 
+__device__ __forceinline__ int key_head(const Args& a, int h) { return a.key_heads > 0 ? h / (a.heads / a.key_heads) : h; }
+
 template <typename T, bool GATED>
 __global__ void __launch_bounds__(256)
 recurrence_simple_kernel(const Args a) {
@@ -62,7 +66,9 @@ recurrence_simple_kernel(const Args a) {
   const bool fresh = a.positions[row0] == 0;
   for (int d = group; d < a.dim; d += 8)
     s_state[d * 32 + lane] = (fresh || !col_ok) ? 0.f : state[static_cast<size_t>(d) * a.vdim + col];
-  const bool first = GATED && blockIdx.z == 0;        // this block also has the normaliser
+  const bool first = GATED && a.normaliser && blockIdx.z == 0;        // this block also has the normaliser
+  const int kh = key_head(a, h);
+  const float skip = a.skip ? a.skip[h] : 0.f;
   if (first)
     for (int d = threadIdx.x; d < a.dim; d += 256) s_n[d] = fresh ? 0.f : slot_normaliser(a, seg, h)[d];
   float decay = GATED ? 0.f : a.decay_pow[h * kPowers + 1], take = 1.f;
@@ -74,8 +80,8 @@ recurrence_simple_kernel(const Args a) {
     }
     const size_t off = static_cast<size_t>(row) * a.stride;
     for (int d = threadIdx.x; d < a.dim; d += 256) {
-      s_k[d] = Elem<T>::ld(static_cast<const T*>(a.k) + off + static_cast<size_t>(h) * a.dim + d) * take;
-      s_q[d] = Elem<T>::ld(static_cast<const T*>(a.q) + off + static_cast<size_t>(h) * a.dim + d) * (GATED ? a.q_scale : 1.f);
+      s_k[d] = Elem<T>::ld(static_cast<const T*>(a.k) + off + static_cast<size_t>(kh) * a.dim + d) * take;
+      s_q[d] = Elem<T>::ld(static_cast<const T*>(a.q) + off + static_cast<size_t>(kh) * a.dim + d) * (GATED ? a.q_scale : 1.f);
     }
     const float v = col_ok ? Elem<T>::ld(static_cast<const T*>(a.v) + off + static_cast<size_t>(h) * a.vdim + col) : 0.f;
     __syncthreads();
@@ -88,7 +94,7 @@ recurrence_simple_kernel(const Args a) {
     s_red[group * 32 + lane] = o;
     __syncthreads();
     if (group == 0 && col_ok) {
-      float t = 0.f;
+      float t = skip * v;
 #pragma unroll
       for (int g = 0; g < 8; ++g) t += s_red[g * 32 + lane];
       Elem<T>::st(static_cast<T*>(a.out) + (static_cast<size_t>(row) * a.heads + h) * a.vdim + col, t);
@@ -211,7 +217,9 @@ recurrence_chunk_kernel(const Args a, const PieceSpace ws, int piece_rows) {
   const float* init = alone ? state : piece;
   const bool zero = LOCAL || (alone && a.positions[it.row0] == 0);
   const int cols = min(kCols, a.vdim - v0);
-  const bool first = GATED && blockIdx.z == 0;        // this block also has the normaliser
+  const bool first = GATED && a.normaliser && blockIdx.z == 0;        // this block also has the normaliser
+  const int kh = key_head(a, h);
+  const float skip = a.skip ? a.skip[h] : 0.f;
   float sum = 0.f;                                    // of the piece's log decays
   if (first && static_cast<int>(threadIdx.x) < dim)
     s_n[0][threadIdx.x] = zero ? 0.f : (alone ? slot_normaliser(a, it.seg, h) : piece_n)[threadIdx.x];
@@ -275,7 +283,7 @@ recurrence_chunk_kernel(const Args a, const PieceSpace ws, int piece_rows) {
       const int r = i / kc, c = i % kc;
       uint4 q = make_uint4(0u, 0u, 0u, 0u), k = q;
       if (r < n) {
-        const size_t off = (base + r) * a.stride + static_cast<size_t>(h) * dim + c * 8;
+        const size_t off = (base + r) * a.stride + static_cast<size_t>(kh) * dim + c * 8;
         if (!LOCAL) q = *reinterpret_cast<const uint4*>(static_cast<const __nv_bfloat16*>(a.q) + off);
         k = *reinterpret_cast<const uint4*>(static_cast<const __nv_bfloat16*>(a.k) + off);
       }
@@ -418,6 +426,14 @@ recurrence_chunk_kernel(const Args a, const PieceSpace ws, int piece_rows) {
           nq[e] += __shfl_xor_sync(0xffffffffu, nq[e], 2);
           if ((lane & 3) == 0 && i < n) a.normaliser[(base + i) * a.heads + h] = nq[e];
         }
+        if (i < n && a.skip) {
+#pragma unroll
+          for (int nn = 0; nn < 8; ++nn) {
+            const uint32_t v2 = *reinterpret_cast<const uint32_t*>(s_v + i * kPitchV + nn * 8 + (lane & 3) * 2);
+            o[nn][e * 2] = fmaf(skip, __uint_as_float(v2 << 16), o[nn][e * 2]);
+            o[nn][e * 2 + 1] = fmaf(skip, __uint_as_float(v2 & 0xffff0000u), o[nn][e * 2 + 1]);
+          }
+        }
         if (i < n) {
           __nv_bfloat16* dst = out + ((base + i) * a.heads + h) * a.vdim + v0;
 #pragma unroll
@@ -475,7 +491,7 @@ recurrence_chunk_kernel(const Args a, const PieceSpace ws, int piece_rows) {
   float* dst = LOCAL ? piece : state;
   if (LOCAL || it.last) {
     if (first && static_cast<int>(threadIdx.x) < dim) (LOCAL ? piece_n : slot_normaliser(a, it.seg, h))[threadIdx.x] = s_n[now][threadIdx.x];
-    if (LOCAL && first && threadIdx.x == 0) ws.log_decay[static_cast<size_t>(blockIdx.x) * a.heads + h] = sum;
+    if (LOCAL && GATED && blockIdx.z == 0 && threadIdx.x == 0) ws.log_decay[static_cast<size_t>(blockIdx.x) * a.heads + h] = sum;
 #pragma unroll
     for (int t = 0; t < MT; ++t)
 #pragma unroll
@@ -513,7 +529,7 @@ recurrence_scan_kernel(const Args a, const PieceSpace ws, int piece_rows) {
   const size_t stride = a.heads * plane / 4;
   float4 run = make_float4(0.f, 0.f, 0.f, 0.f);
   if (mine && !fresh) run = *reinterpret_cast<const float4*>(slot_state(a, seg, h) + e);
-  const bool norm = GATED && blockIdx.z == 0 && static_cast<int>(threadIdx.x) < a.dim;      // (dim <= 128)
+  const bool norm = GATED && a.normaliser && blockIdx.z == 0 && static_cast<int>(threadIdx.x) < a.dim;      // (dim <= 128)
   float* wn = ws.normaliser + (static_cast<size_t>(first) * a.heads + h) * a.dim + threadIdx.x;
   float run_n = norm && !fresh ? slot_normaliser(a, seg, h)[threadIdx.x] : 0.f;
   for (int base = 0; base < pieces; base += 256) {
@@ -761,10 +777,100 @@ memory_step_kernel(const Args a, const Gates g, const T* __restrict__ gate, long
   }
 }
 
+// ---- state space -----------------------------------------------------------------------------------------------------
+struct Steps {
+  const float* z;               // [rows, stride], a column per head
+  long long stride;
+  const float* bias;
+  const float* log_rate;
+};
+__device__ __forceinline__ void step_gates(const Steps& s, int row, int h, float* dt, float* log_decay) {
+  *dt = softplus(s.z[static_cast<long long>(row) * s.stride + h] + s.bias[h]);
+  *log_decay = -expf(s.log_rate[h]) * *dt;
+}
+
+__global__ void __launch_bounds__(256)
+state_space_gates_kernel(const Steps s, int units, int heads, float* __restrict__ log_decay, float* __restrict__ log_take) {
+  const int unit = blockIdx.x * 256 + threadIdx.x;
+  if (unit >= units) return;
+  float dt, decay;
+  step_gates(s, unit / heads, unit % heads, &dt, &decay);
+  log_decay[unit] = decay;
+  log_take[unit] = logf(dt);
+}
+
+template <typename T>
+__global__ void __launch_bounds__(256, 4)
+state_space_step_kernel(const Args a, const Steps s) {
+  __shared__ float4 s_red[256];
+  extern __shared__ float s_kq[];           // [2][dim]
+  const int seg = blockIdx.x, h = blockIdx.y, kh = key_head(a, h);
+  const int row = a.cu_rows[seg];
+  const int groups_per_row = a.vdim / 4;                 // float4 columns
+  const int lanes_rows = 256 / groups_per_row;           // state rows per pass
+  const int cg = threadIdx.x % groups_per_row, rg = threadIdx.x / groups_per_row;
+  const bool active = rg < lanes_rows;
+  const size_t off = static_cast<size_t>(row) * a.stride;
+  const bool fresh = a.positions[row] == 0;
+  float4* state = reinterpret_cast<float4*>(slot_state(a, seg, h));
+  constexpr int U = 8;                                   // loads in flight per thread
+  float4 x[U];
+  auto fetch = [&](int d0) {
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      const int d = d0 + u * lanes_rows;
+      x[u] = (d < a.dim && !fresh) ? state[static_cast<size_t>(d) * groups_per_row + cg] : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+  };
+  if (active) fetch(rg);                                 // (the state travels while the gates are worked out)
+  float dt, decay;
+  step_gates(s, row, h, &dt, &decay);
+  decay = fresh ? 0.f : expf(decay);
+  for (int d = threadIdx.x; d < a.dim; d += 256) {
+    s_kq[d] = Elem<T>::ld(static_cast<const T*>(a.k) + off + static_cast<size_t>(kh) * a.dim + d) * dt;
+    s_kq[a.dim + d] = Elem<T>::ld(static_cast<const T*>(a.q) + off + static_cast<size_t>(kh) * a.dim + d) * a.q_scale;
+  }
+  float v[4];
+#pragma unroll
+  for (int i = 0; i < 4; ++i)
+    v[i] = active ? Elem<T>::ld(static_cast<const T*>(a.v) + off + static_cast<size_t>(h) * a.vdim + cg * 4 + i) : 0.f;
+  __syncthreads();
+  float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
+  for (int d0 = rg; active && d0 < a.dim; d0 += U * lanes_rows) {
+    if (d0 != rg) fetch(d0);
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      const int d = d0 + u * lanes_rows;
+      if (d >= a.dim) break;
+      const float k = s_kq[d], q = s_kq[a.dim + d];
+      x[u].x = fmaf(x[u].x, decay, k * v[0]); x[u].y = fmaf(x[u].y, decay, k * v[1]);
+      x[u].z = fmaf(x[u].z, decay, k * v[2]); x[u].w = fmaf(x[u].w, decay, k * v[3]);
+      state[static_cast<size_t>(d) * groups_per_row + cg] = x[u];
+      o.x = fmaf(x[u].x, q, o.x); o.y = fmaf(x[u].y, q, o.y); o.z = fmaf(x[u].z, q, o.z); o.w = fmaf(x[u].w, q, o.w);
+    }
+  }
+  s_red[threadIdx.x] = o;
+  __syncthreads();
+  if (rg == 0) {
+    for (int r = 1; r < lanes_rows; ++r) {
+      const float4 t = s_red[r * groups_per_row + cg];
+      o.x += t.x; o.y += t.y; o.z += t.z; o.w += t.w;
+    }
+    const float skip = a.skip ? a.skip[h] : 0.f;
+    T* dst = static_cast<T*>(a.out) + (static_cast<size_t>(row) * a.heads + h) * a.vdim + cg * 4;
+    const float y[4] = {o.x, o.y, o.z, o.w};
+#pragma unroll
+    for (int i = 0; i < 4; ++i) Elem<T>::st(dst + i, fmaf(skip, v[i], y[i]));
+  }
+}
+
 bool recurrence_args_ok(const Args& a) {
   return a.positions && a.cu_rows && a.slots && a.q && a.k && a.v && a.state && a.out &&
-         a.slot_stride >= static_cast<long long>(a.heads) * a.dim * a.vdim + (a.decay_pow ? 0 : static_cast<long long>(a.heads) * (a.dim + 1)) && a.segments > 0 && a.heads > 0 &&
-         a.heads <= 65535 && a.dim > 0 && a.vdim > 0 && a.num_slots > 0;
+         a.slot_stride >= static_cast<long long>(a.heads) * a.dim * a.vdim + (a.normaliser ? static_cast<long long>(a.heads) * (a.dim + 1) : 0) && a.segments > 0 && a.heads > 0 &&
+         a.heads <= 65535 && a.dim > 0 && a.vdim > 0 && a.num_slots > 0 && a.key_heads >= 0 && (a.key_heads == 0 || a.heads % a.key_heads == 0);
+}
+bool memory_slots_ok(const Args& a) {        // normalisers and maxima behind the state
+  return a.slot_stride >= static_cast<long long>(a.heads) * a.dim * a.vdim + static_cast<long long>(a.heads) * (a.dim + 1);
 }
 
 size_t chunk_smem(int dim) {
@@ -813,7 +919,7 @@ int launch_simple(const Args& a, cudaStream_t st) {
   return launch_status();
 }
 
-bool decay_ok(const Args& a) { return a.decay_pow || (a.log_decay && a.log_take && a.normaliser); }
+bool decay_ok(const Args& a) { return a.decay_pow || (a.log_decay && a.log_take); }
 bool gates_ok(const Gates& g, int heads) { return g.logits && g.in_bias && g.forget_bias && g.cap > 0.f && g.stride >= 2ll * heads; }
 
 }  // namespace
@@ -833,7 +939,7 @@ extern "C" int cacheir_b200_recurrence_simple(const cacheir_b200_recurrence_args
 extern "C" int cacheir_b200_recurrence_step(const cacheir_b200_recurrence_args* a, void* stream) {
   if (!a) return CACHEIR_B200_EINVAL;
   if (a->rows <= 0) return 0;
-  if (!recurrence_args_ok(*a) || !a->decay_pow || a->rows != a->segments) return CACHEIR_B200_EINVAL;
+  if (!recurrence_args_ok(*a) || !a->decay_pow || a->key_heads != 0 || a->skip || a->rows != a->segments) return CACHEIR_B200_EINVAL;
   if (a->vdim % 4 != 0 || a->vdim > 1024 || a->dim > 4096) return CACHEIR_B200_EUNSUPPORTED;
   if (!aligned_to(a->state, 16) || a->slot_stride % 4 != 0) return CACHEIR_B200_EALIGN;
   const dim3 grid(a->segments, a->heads);
@@ -872,7 +978,7 @@ extern "C" int cacheir_b200_memory_gates(const cacheir_b200_recurrence_args* a, 
   if (!a) return CACHEIR_B200_EINVAL;
   if (a->rows <= 0) return 0;
   const Gates g{logits, stride, in_bias, forget_bias, cap};
-  if (!recurrence_args_ok(*a) || a->decay_pow || !gates_ok(g, a->heads) || !log_decay || !log_take || !maximum) return CACHEIR_B200_EINVAL;
+  if (!recurrence_args_ok(*a) || !memory_slots_ok(*a) || a->decay_pow || !gates_ok(g, a->heads) || !log_decay || !log_take || !maximum) return CACHEIR_B200_EINVAL;
   memory_gates_kernel<<<dim3(a->segments, a->heads), kGateThreads, 0, as_stream(stream)>>>(*a, g, log_decay, log_take, maximum);
   return launch_status();
 }
@@ -901,12 +1007,36 @@ extern "C" int cacheir_b200_memory_step(const cacheir_b200_recurrence_args* a, c
   if (!a) return CACHEIR_B200_EINVAL;
   if (a->rows <= 0) return 0;
   const Gates g{logits, stride, in_bias, forget_bias, cap};
-  if (!recurrence_args_ok(*a) || a->decay_pow || !gates_ok(g, a->heads) || !gate || !w || a->rows != a->segments) return CACHEIR_B200_EINVAL;
+  if (!recurrence_args_ok(*a) || !memory_slots_ok(*a) || a->decay_pow || a->key_heads != 0 || a->skip || !gates_ok(g, a->heads) || !gate || !w ||
+      a->rows != a->segments)
+    return CACHEIR_B200_EINVAL;
   if (a->vdim % 4 != 0 || a->vdim > 1024 || a->dim > 4096) return CACHEIR_B200_EUNSUPPORTED;
   if (!aligned_to(a->state, 16) || a->slot_stride % 4 != 0) return CACHEIR_B200_EALIGN;
   const dim3 grid(a->segments, a->heads);
   const size_t smem = static_cast<size_t>(a->dim) * 8;
   CB200_HYBRID_DTYPE(a->dtype, (memory_step_kernel<T><<<grid, 256, smem, as_stream(stream)>>>(*a, g, static_cast<const T*>(gate), gate_stride, w, eps)));
+  return launch_status();
+}
+
+extern "C" int cacheir_b200_state_space_gates(const cacheir_b200_recurrence_args* a, const float* z, long long stride, const float* bias,
+                                              const float* log_rate, float* log_decay, float* log_take, void* stream) {
+  if (!a) return CACHEIR_B200_EINVAL;
+  if (a->rows <= 0) return 0;
+  if (a->heads <= 0 || !z || stride < a->heads || !bias || !log_rate || !log_decay || !log_take) return CACHEIR_B200_EINVAL;
+  const int units = a->rows * a->heads;
+  state_space_gates_kernel<<<(units + 255) / 256, 256, 0, as_stream(stream)>>>(Steps{z, stride, bias, log_rate}, units, a->heads, log_decay, log_take);
+  return launch_status();
+}
+
+extern "C" int cacheir_b200_state_space_step(const cacheir_b200_recurrence_args* a, const float* z, long long stride, const float* bias,
+                                             const float* log_rate, void* stream) {
+  if (!a) return CACHEIR_B200_EINVAL;
+  if (a->rows <= 0) return 0;
+  if (!recurrence_args_ok(*a) || a->decay_pow || a->rows != a->segments || !z || stride < a->heads || !bias || !log_rate) return CACHEIR_B200_EINVAL;
+  if (a->vdim % 4 != 0 || a->vdim > 1024 || a->dim > 4096) return CACHEIR_B200_EUNSUPPORTED;
+  if (!aligned_to(a->state, 16) || a->slot_stride % 4 != 0) return CACHEIR_B200_EALIGN;
+  const size_t smem = static_cast<size_t>(a->dim) * 8;
+  CB200_HYBRID_DTYPE(a->dtype, (state_space_step_kernel<T><<<dim3(a->segments, a->heads), 256, smem, as_stream(stream)>>>(*a, Steps{z, stride, bias, log_rate})));
   return launch_status();
 }
 

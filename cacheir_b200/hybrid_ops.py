@@ -15,9 +15,9 @@ from . import _lib
 from ._lib import DenseArgs, LatentArgs, RecurrenceArgs, check
 from .ops import _ptr, _require_cuda, _stream, dtype_code
 
-NEXT_NONE, NEXT_COPY, NEXT_DYT, NEXT_RMS = range(4)
+NEXT_NONE, NEXT_COPY, NEXT_DYT, NEXT_RMS, NEXT_LAYER = range(5)
 (DENSE_PLAIN, DENSE_F32, DENSE_SILU, DENSE_GEGLU, DENSE_GATED, DENSE_RESIDUAL, DENSE_GELU_EMBED, DENSE_SWIGLU,
- DENSE_CLAMPED_GLU) = range(9)
+ DENSE_CLAMPED_GLU, DENSE_RELU2) = range(10)
 GLU_EPILOGUES = {"gelu_tanh": DENSE_GEGLU, "silu": DENSE_SWIGLU, "clamped": DENSE_CLAMPED_GLU}
 RECURRENCE_POWERS = 65
 
@@ -40,11 +40,19 @@ class RmsNorm:
 
 
 @dataclass
+class LayerNorm:
+    """(x - mean) / sqrt(variance + eps) * weight; weight float32 on the device."""
+
+    weight: torch.Tensor
+    eps: float
+
+
+@dataclass
 class Next:
-    """What a kernel that finishes the residual leaves in `out`: the residual itself, its Dynamic Tanh, or its RMS norm."""
+    """What a kernel that finishes the residual leaves in `out`: the residual itself or a norm of it."""
 
     out: torch.Tensor
-    norm: DynamicTanh | RmsNorm | None = None
+    norm: DynamicTanh | RmsNorm | LayerNorm | None = None
 
 
 @dataclass
@@ -72,9 +80,9 @@ def _next(nx: Next | None) -> tuple:
         return (NEXT_NONE, None, None, 0.0, None)
     if nx.norm is None:
         return (NEXT_COPY, None, None, 0.0, nx.out.data_ptr())
-    if isinstance(nx.norm, RmsNorm):
+    if isinstance(nx.norm, (RmsNorm, LayerNorm)):
         _f32(nx.norm.weight)
-        return (NEXT_RMS, nx.norm.weight.data_ptr(), None, float(nx.norm.eps), nx.out.data_ptr())
+        return (NEXT_RMS if isinstance(nx.norm, RmsNorm) else NEXT_LAYER, nx.norm.weight.data_ptr(), None, float(nx.norm.eps), nx.out.data_ptr())
     return (NEXT_DYT, nx.norm.weight.data_ptr(), nx.norm.bias.data_ptr(), float(nx.norm.alpha), nx.out.data_ptr())
 
 
@@ -196,14 +204,37 @@ def residual_dyt(residual: torch.Tensor, y: torch.Tensor, norm: DynamicTanh, nx:
         int(y.shape[1]), *_next(nx), dtype_code(y.dtype), _stream()), "residual_dyt")
 
 
-def residual_add(residual: torch.Tensor, y: torch.Tensor, nx: Next | None = None) -> None:
-    """residual += y"""
-    _require_cuda(residual, y)
+def layer_norm_rows(residual: torch.Tensor, weight: torch.Tensor, eps: float, out: torch.Tensor, row_index: torch.Tensor | None = None) -> torch.Tensor:
+    """out[j] = layer norm of residual row row_index[j] (row j without an index) * weight."""
+    _require_cuda(residual, weight, out, row_index)
+    _f32(residual, weight)
+    check(_lib.load_group("ragged").cacheir_b200_layer_norm_rows(
+        residual.data_ptr(), _ptr(row_index), weight.data_ptr(), float(eps), out.data_ptr(), int(out.shape[0]), int(out.shape[1]),
+        dtype_code(out.dtype), _stream()), "layer_norm_rows")
+    return out
+
+
+def join_embedding(residual: torch.Tensor, table: torch.Tensor, ids: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
+    """out [rows, 2*width] = (residual | table[ids])"""
+    _require_cuda(residual, table, ids, out)
     _f32(residual)
-    if y.shape != residual.shape or not y.is_contiguous():
-        raise ValueError("y must be a contiguous tensor of the residual's shape")
+    if ids.dtype != torch.int64 or not table.is_contiguous() or residual.shape[1] != table.shape[1] or table.dtype != out.dtype \
+            or tuple(out.shape) != (residual.shape[0], 2 * residual.shape[1]) or not out.is_contiguous():
+        raise ValueError("join_embedding expects int64 ids, a contiguous [vocab, width] table and a contiguous [rows, 2*width] output")
+    check(_lib.load_group("ragged").cacheir_b200_join_embedding(
+        residual.data_ptr(), table.data_ptr(), ids.data_ptr(), out.data_ptr(), int(residual.shape[0]), int(table.shape[1]), int(table.shape[0]),
+        dtype_code(out.dtype), _stream()), "join_embedding")
+    return out
+
+
+def residual_add(residual: torch.Tensor, y: torch.Tensor, nx: Next | None = None, scale: torch.Tensor | None = None) -> None:
+    """residual += y, or y * scale column by column"""
+    _require_cuda(residual, y, scale)
+    _f32(residual, *([] if scale is None else [scale]))
+    if y.shape != residual.shape or not y.is_contiguous() or (scale is not None and scale.numel() != residual.shape[1]):
+        raise ValueError("y must be a contiguous tensor of the residual's shape, scale have an entry per column")
     check(_lib.load_group("ragged").cacheir_b200_residual_add(
-        residual.data_ptr(), y.data_ptr(), int(y.shape[0]), int(y.shape[1]), *_next(nx), dtype_code(y.dtype), _stream()), "residual_add")
+        residual.data_ptr(), y.data_ptr(), _ptr(scale), int(y.shape[0]), int(y.shape[1]), *_next(nx), dtype_code(y.dtype), _stream()), "residual_add")
 
 
 def residual_rms_pair(residual: torch.Tensor, y1: torch.Tensor, w1: torch.Tensor, y2: torch.Tensor, w2: torch.Tensor, factor: float, eps: float,
@@ -241,6 +272,22 @@ def gated_rms(o: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, eps: fl
     return out
 
 
+def gated_parts_rms(o: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, eps: float, out: torch.Tensor, *, parts: int,
+                    gate_first: bool) -> torch.Tensor:
+    """Norm in equal parts with a silu gate, before the norm or behind it; weight per column of a row, or of a part."""
+    _require_cuda(o, gate, weight, out)
+    _f32(weight)
+    cols = int(o.shape[1])
+    if not o.is_contiguous() or not out.is_contiguous() or gate.stride(1) != 1 or gate.shape != o.shape or out.shape != o.shape or cols % parts:
+        raise ValueError("gated_parts_rms expects contiguous o and out, a gate of their shape and equal parts")
+    if weight.numel() not in (cols, cols // parts):
+        raise ValueError("the weight has an entry per column of a row or of a part")
+    check(_lib.load_group("ragged").cacheir_b200_gated_parts_rms(
+        o.data_ptr(), gate.data_ptr(), gate.stride(0), weight.data_ptr(), int(weight.numel() != cols), int(gate_first), float(eps), out.data_ptr(),
+        int(o.shape[0]), cols, int(parts), dtype_code(o.dtype), _stream()), "gated_parts_rms")
+    return out
+
+
 def glu_pairs(y: torch.Tensor, out: torch.Tensor, epilogue: int = DENSE_GEGLU, limit: float = 0.0) -> torch.Tensor:
     """y [T, 2*ff] with columns alternating gate, up; out as the paired epilogue leaves it."""
     _require_cuda(y, out)
@@ -265,6 +312,13 @@ def silu_cols(y: torch.Tensor, cols: int) -> torch.Tensor:
     _require_cuda(y)
     check(_lib.load_group("ragged").cacheir_b200_silu_cols(y.data_ptr(), int(y.shape[0]), y.stride(0), int(cols), dtype_code(y.dtype), _stream()),
           "silu_cols")
+    return y
+
+
+def relu2_cols(y: torch.Tensor, cols: int) -> torch.Tensor:
+    _require_cuda(y)
+    check(_lib.load_group("ragged").cacheir_b200_relu2_cols(y.data_ptr(), int(y.shape[0]), y.stride(0), int(cols), dtype_code(y.dtype), _stream()),
+          "relu2_cols")
     return y
 
 
@@ -332,29 +386,34 @@ def decay_powers(decay, device: torch.device | str) -> torch.Tensor:
 
 
 def recurrence_args(rows: Rows, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, powers: torch.Tensor | None, state: torch.Tensor,
-                    out: torch.Tensor, *, heads: int, dim: int, vdim: int, gated: tuple[torch.Tensor, torch.Tensor, torch.Tensor] | None = None,
-                    q_scale: float = 1.0) -> RecurrenceArgs:
-    """q, k [T, heads*dim] and v [T, heads*vdim] with one common row stride. Constant decays: state [slots, heads, dim, vdim]
-    float32. Without `powers` the recurrence is gated: state [slots, memory_state_size(...)], and `gated` = (log_decay,
-    log_take, normaliser), [T, heads] float32 each (not needed by memory_step)."""
-    _require_cuda(q, k, v, powers, state, out)
-    _f32(state, *([] if powers is None else [powers]), *(gated or ()))
+                    out: torch.Tensor, *, heads: int, dim: int, vdim: int,
+                    gated: tuple[torch.Tensor, torch.Tensor, torch.Tensor | None] | None = None, q_scale: float = 1.0, key_heads: int | None = None,
+                    skip: torch.Tensor | None = None, memory: bool = True) -> RecurrenceArgs:
+    """q, k [T, key_heads*dim] (by default as many heads as v) and v [T, heads*vdim] with one common row stride. Constant decays:
+    state [slots, heads, dim, vdim] float32. Without `powers` the recurrence is gated: `gated` = (log_decay, log_take, normaliser),
+    [T, heads] float32 each (not needed by the step forms), and state [slots, memory_state_size(...)], or without `memory` (no
+    normaliser) rows of any length that begin with [heads, dim, vdim]. `skip` [heads]: o += skip * v."""
+    _require_cuda(q, k, v, powers, state, out, skip)
+    given = [] if gated is None else [t for t in gated if t is not None]
+    _f32(state, *([] if powers is None else [powers]), *given, *([] if skip is None else [skip]))
     if not (q.stride(0) == k.stride(0) == v.stride(0)) or q.stride(1) != 1 or k.stride(1) != 1 or v.stride(1) != 1:
         raise ValueError("q, k and v must share one row stride and have dense rows")
     if not out.is_contiguous() or (powers is not None and (tuple(state.shape[1:]) != (heads, dim, vdim) or tuple(powers.shape) != (heads, RECURRENCE_POWERS))):
         raise ValueError("state must be [slots, heads, dim, vdim], powers [heads, 65] and out contiguous")
-    if powers is None and tuple(state.shape[1:]) != (memory_state_size(heads, dim, vdim),):
+    if powers is None and memory and tuple(state.shape[1:]) != (memory_state_size(heads, dim, vdim),):
         raise ValueError("a gated recurrence's state must be [slots, memory_state_size]")
-    if gated is not None and any(tuple(t.shape) != (rows.rows, heads) for t in gated):
+    if state.stride(0) < heads * dim * vdim or (key_heads is not None and heads % key_heads) or (skip is not None and skip.numel() != heads):
+        raise ValueError("a state slot must hold [heads, dim, vdim], key heads divide the heads, skip has an entry per head")
+    if any(tuple(t.shape) != (rows.rows, heads) for t in given):
         raise ValueError("log_decay, log_take and normaliser are [rows, heads]")
     a = RecurrenceArgs()
     a.positions, a.cu_rows, a.slots = rows.positions.data_ptr(), rows.cu_rows.data_ptr(), rows.slots.data_ptr()
     a.rows, a.segments, a.heads, a.dim, a.vdim = rows.rows, rows.segments, heads, dim, vdim
     a.q, a.k, a.v, a.stride = q.data_ptr(), k.data_ptr(), v.data_ptr(), q.stride(0)
     a.decay_pow, a.state, a.num_slots, a.out, a.dtype = _ptr(powers), state.data_ptr(), int(state.shape[0]), out.data_ptr(), dtype_code(q.dtype)
-    a.slot_stride, a.q_scale = state.stride(0), float(q_scale)
+    a.slot_stride, a.q_scale, a.key_heads, a.skip = state.stride(0), float(q_scale), 0 if key_heads is None else key_heads, _ptr(skip)
     if gated is not None:
-        a.log_decay, a.log_take, a.normaliser = (t.data_ptr() for t in gated)
+        a.log_decay, a.log_take, a.normaliser = (_ptr(t) for t in gated)
     return a
 
 
@@ -433,6 +492,33 @@ def memory_step(a: RecurrenceArgs, gates: MemoryGates, gate: torch.Tensor, weigh
     _memory_gate(gate, weight, a.heads * a.vdim)
     check(_lib.load_group("recurrence").cacheir_b200_memory_step(
         ctypes.byref(a), *gates.args(), gate.data_ptr(), gate.stride(0), weight.data_ptr(), float(eps), _stream()), "memory_step")
+
+
+# ---- state space -----------------------------------------------------------------------------------------------------------
+@dataclass
+class StepSizes:
+    """Step size logits [T, heads] float32 (a view with dense rows), their bias and the logarithm of the decay rate [heads]."""
+
+    logits: torch.Tensor
+    bias: torch.Tensor
+    log_rate: torch.Tensor
+
+    def args(self) -> tuple:
+        _require_cuda(self.logits, self.bias, self.log_rate)
+        _f32(self.bias, self.log_rate)
+        if self.logits.dtype != torch.float32 or self.logits.stride(1) != 1 or not int(self.logits.shape[1]) == self.bias.numel() == self.log_rate.numel():
+            raise ValueError("step size logits are float32 [T, heads] with dense rows")
+        return (self.logits.data_ptr(), self.logits.stride(0), self.bias.data_ptr(), self.log_rate.data_ptr())
+
+
+def state_space_gates(a: RecurrenceArgs, steps: StepSizes, log_decay: torch.Tensor, log_take: torch.Tensor) -> None:
+    _require_cuda(log_decay, log_take)
+    check(_lib.load_group("recurrence").cacheir_b200_state_space_gates(
+        ctypes.byref(a), *steps.args(), log_decay.data_ptr(), log_take.data_ptr(), _stream()), "state_space_gates")
+
+
+def state_space_step(a: RecurrenceArgs, steps: StepSizes) -> None:
+    check(_lib.load_group("recurrence").cacheir_b200_state_space_step(ctypes.byref(a), *steps.args(), _stream()), "state_space_step")
 
 
 def device_status(reset: bool = True) -> int:

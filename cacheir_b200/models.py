@@ -6,7 +6,7 @@ from dataclasses import dataclass
 from pathlib import Path
 from typing import Any, Callable
 
-from . import gutorax, rekodra, topunex
+from . import gutorax, rekodra, topunex, zimorax
 from .artifact import CompileArtifact, ModelConfig, build_decoder_artifact
 
 
@@ -52,3 +52,5 @@ register_family(gutorax.ARCHITECTURE, ModelFamily("gutorax", gutorax.GutoraxConf
 register_family(topunex.ARCHITECTURE, ModelFamily("topunex", topunex.TopunexConfig.from_dict, topunex.build_topunex_artifact, ("ragged", "experts")))
 register_family(rekodra.ARCHITECTURE, ModelFamily("rekodra", rekodra.RekodraConfig.from_dict, rekodra.build_rekodra_artifact,
                                                   ("ragged", "recurrence", "experts")))
+register_family(zimorax.ARCHITECTURE, ModelFamily("zimorax", zimorax.ZimoraxConfig.from_dict, zimorax.build_zimorax_artifact,
+                                                  ("ragged", "recurrence", "talking", "delta")))

@@ -16,6 +16,7 @@ import torch
 
 from . import expert_ops as X
 from . import hybrid_ops as H
+from . import mixer_ops as M
 from . import ops
 
 # rows a portion plan is made for: one plan (and one CUDA graph) per bucket, not per portion length
@@ -53,6 +54,26 @@ def rotate_half_table(positions: int, dims: int, base: float, scaling: tuple[flo
     freq = rotary_frequencies(dims, base, scaling)
     angle = np.arange(positions, dtype=np.float64)[:, None] * freq[None, :]
     return np.stack([np.cos(angle), np.sin(angle)], axis=-1).astype(np.float32)
+
+
+def yarn_frequencies(dims: int, base: float, factor: float, original: float, fast: float, slow: float) -> tuple[np.ndarray, float]:
+    """(frequencies in double precision, factor of cosine and sine): pairs that turn more than `fast` times within `original`
+    positions keep their frequency, those that turn less than `slow` times have it divided by `factor`, with a linear ramp over the
+    pairs between."""
+    freq = rotary_frequencies(dims, base)
+
+    def pair(turns: float) -> float:
+        return dims * np.log(original / (2.0 * np.pi * turns)) / (2.0 * np.log(base))
+    lo, hi = max(np.floor(pair(fast)), 0.0), min(np.ceil(pair(slow)), dims - 1.0)
+    ramp = np.clip((np.arange(dims // 2, dtype=np.float64) - lo) / max(hi - lo, 0.001), 0.0, 1.0)
+    return freq / factor * ramp + freq * (1.0 - ramp), 0.1 * float(np.log(factor)) + 1.0
+
+
+def yarn_table(positions: int, dims: int, base: float, yarn: tuple[float, float, float, float]) -> np.ndarray:
+    """`rotate_half_table` of `yarn_frequencies`, cosine and sine with their factor."""
+    freq, factor = yarn_frequencies(dims, base, *yarn)
+    angle = np.arange(positions, dtype=np.float64)[:, None] * freq[None, :]
+    return (np.stack([np.cos(angle), np.sin(angle)], axis=-1) * factor).astype(np.float32)
 
 
 def make_plan_class(base: type) -> type:
@@ -164,6 +185,9 @@ def make_plan_class(base: type) -> type:
             if nxt.op == "rms_norm" and nxt.attrs.get("rows") != "logits" and nxt.inputs[0] == self._nodes[idx].outputs[0]:
                 norm = H.RmsNorm(self.engine.weights.get_f32(nxt.inputs[1]), float(nxt.attrs["eps"]))
                 return H.Next(self._scratch("normed", width), norm), nxt.outputs[0]
+            if nxt.op == "layer_norm" and nxt.attrs.get("rows") != "logits" and nxt.inputs[0] == self._nodes[idx].outputs[0]:
+                norm = H.LayerNorm(self.engine.weights.get_f32(nxt.inputs[1]), float(nxt.attrs["eps"]))
+                return H.Next(self._scratch("normed", width), norm), nxt.outputs[0]
             if nxt.op in READS_RESIDUAL and nxt.inputs[0] == self._nodes[idx].outputs[0]:
                 return H.Next(self._scratch("copied", width)), None
             return None, None
@@ -200,13 +224,16 @@ def make_plan_class(base: type) -> type:
             self.logits = logits
             self.feedback_tail = lambda: ops.argmax_rows(logits, self.ids)
 
-        def _dense(self, x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, bias: torch.Tensor | None = None, label: str = "") -> None:
-            """Plain product into `out` (float32 for logits): tensor cores where they take it, else CUDA cores."""
+        def _dense(self, x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, bias: torch.Tensor | None = None, label: str = "",
+                   relu2: bool = False) -> None:
+            """Plain product into `out` (float32 for logits), or its squared ReLU: tensor cores where they take it, else CUDA cores."""
             if H.dense_supported(int(w.shape[1]), w.stride(0), x.stride(0), dtype=x.dtype):
-                epilogue = H.DENSE_F32 if out.dtype == torch.float32 else H.DENSE_PLAIN
+                epilogue = H.DENSE_RELU2 if relu2 else H.DENSE_F32 if out.dtype == torch.float32 else H.DENSE_PLAIN
                 self._emit(lambda: H.dense_gemm(x, w, out, epilogue=epilogue, bias=bias), "b200.dense_gemm" + label)
             else:
                 self._emit(lambda: H.dense_simple(x, w, out, bias=bias), "b200.dense_simple")
+                if relu2:
+                    self._emit(lambda: H.relu2_cols(out, int(w.shape[0])), "b200.relu2_cols")
 
         def _input(self, name: str) -> torch.Tensor:
             """A product's input: an activation, or the residual's copy."""
@@ -224,6 +251,16 @@ def make_plan_class(base: type) -> type:
             self._finish_residual(idx, lambda nx: self._emit(lambda: H.scaled_embedding(table, self.ids, x, scale, nx, accumulate=True),
                                                              "b200.add_embedding"))
 
+        def _lower_join_embedding(self, idx: int, node: Any) -> None:
+            """residual = product of (residual, embedding output) + one row of the last input."""
+            eng, x = self.engine, self._residual
+            table, w = eng.weights.get_checked(node.inputs[2]), eng.weights.get_checked(node.inputs[3])
+            step = eng.weights.get_f32(node.inputs[4])[int(node.attrs["step"])]
+            joined = self._scratch("joined", int(w.shape[1]))
+            self._emit(lambda: H.join_embedding(x, table, self.ids, joined), "b200.join_embedding")
+            self._dense(joined, w, x, step, ".join")
+            self._env[node.outputs[0]] = x
+
         def _lower_dynamic_tanh(self, idx: int, node: Any) -> None:
             norm = self._dyt(node.inputs[1:4])
             width = int(self.engine.config.hidden_size)
@@ -239,9 +276,9 @@ def make_plan_class(base: type) -> type:
             eng, x = self.engine, self._input(node.inputs[0])
             names = tuple(node.inputs[1:])
             bias = eng.concat_bias(tuple(node.attrs["bias"]), names) if node.attrs.get("bias") else None
-            sizes = [int(eng.graph.weights[n].shape[0]) for n in names]
+            sizes = list(node.attrs.get("sizes") or [int(eng.graph.weights[n].shape[0]) for n in names])      # outputs, by default one per weight
             w = eng.concat_weight(names)
-            floats = sum(sizes[len(sizes) - int(node.attrs.get("float_tail", 0)):])     # columns of the last weights: float32, one output
+            floats = sum(sizes[len(sizes) - int(node.attrs.get("float_tail", 0)):])     # the last columns: float32, one output
             total = int(w.shape[0]) - floats
             out = self._scratch("projected", (total + 7) // 8 * 8)
             tail = self._scratch("projected_float", floats, torch.float32) if floats else None
@@ -348,6 +385,82 @@ def make_plan_class(base: type) -> type:
                 self._emit(lambda: H.recurrence_simple(args), "b200.recurrence_simple")
             self._emit(lambda: H.memory_norm(out, normaliser, maximum, gate, norm, eps, mixed, heads=heads, vdim=vdim), "b200.memory_norm")
 
+        def _lower_short_conv(self, idx: int, node: Any) -> None:
+            """Inputs: x, bias by name or "", convolution weights of neighbouring channels. One output per attrs["sizes"]."""
+            eng, x = self.engine, self._env[node.inputs[0]]
+            w = eng.concat_f32(tuple(node.inputs[2:]))
+            bias = eng.weights.get_f32(node.inputs[1]) if node.inputs[1] else None
+            state, offset = eng.allocator.state_for_layer(int(node.attrs["layer"])), int(node.attrs["offset"])
+            channels = int(w.shape[0])
+            out = self._scratch("convolved", (channels + 7) // 8 * 8)[:, :channels]
+            self._emit(lambda: M.short_conv(self.rows, x, w, bias, state, offset, out), "b200.short_conv")
+            col = 0
+            for name, n in zip(node.outputs, node.attrs["sizes"]):
+                self._env[name] = out[:, col:col + n]
+                col += n
+
+        def _lower_state_space(self, idx: int, node: Any) -> None:
+            eng, at = self.engine, node.attrs
+            q, k, v, logits = (self._env[n] for n in node.inputs[:4])
+            bias, log_rate, skip = (eng.weights.get_f32(n) for n in node.inputs[4:7])
+            heads, key_heads, dim, vdim = (int(at[n]) for n in ("heads", "key_heads", "dim", "vdim"))
+            state = eng.allocator.state_for_layer(int(at["layer"]))
+            steps = H.StepSizes(logits, bias, log_rate)
+            out = self._scratch("recurrence", heads * vdim)
+            self._env[node.outputs[0]] = out
+
+            def args(gated: tuple | None) -> Any:
+                return H.recurrence_args(self.rows, q, k, v, None, state, out, heads=heads, dim=dim, vdim=vdim, gated=gated, key_heads=key_heads,
+                                         skip=skip, memory=False)
+            if self.decode and vdim % 4 == 0 and vdim <= 1024 and dim <= 4096:
+                a = args(None)
+                self._emit(lambda: H.state_space_step(a, steps), "b200.state_space_step")
+                return
+            log_decay, log_take = (self._scratch("space_" + role, heads, torch.float32) for role in ("decay", "take"))
+            a = args((log_decay, log_take, None))
+            self._emit(lambda: H.state_space_gates(a, steps, log_decay, log_take), "b200.state_space_gates")
+            aligned = q.stride(0) % 8 == 0 and not any(t.data_ptr() % 16 for t in (q, k, v))
+            if H.recurrence_chunked_supported(dim, vdim, eng.dtype) and aligned:
+                need = H.recurrence_workspace_bytes(self.batch, self.segments, heads, dim, vdim)
+                ws = eng.scratch("recurrence_ws", need) if need else None
+                self._emit(lambda: H.recurrence_chunked(a, ws), "b200.recurrence_chunked", launches=3 if need else 1)
+            else:
+                self._emit(lambda: H.recurrence_simple(a), "b200.recurrence_simple")
+
+        def _lower_delta_rule(self, idx: int, node: Any) -> None:
+            """Inputs: q, k, v, gate logits, output gate, then bias and log rate of the decay and the head's norm weight."""
+            eng, at = self.engine, node.attrs
+            q, k, v, logits, gate = (self._env[n] for n in node.inputs[:5])
+            bias, log_rate, norm = (eng.weights.get_f32(n) for n in node.inputs[5:8])
+            heads, key_heads, dim, vdim, eps = int(at["heads"]), int(at["key_heads"]), int(at["dim"]), int(at["vdim"]), float(at["eps"])
+            state = eng.allocator.state_for_layer(int(at["layer"]))
+            mixed = self._scratch("mixed", heads * vdim)
+            self._env[node.outputs[0]] = mixed
+
+            def args(out: torch.Tensor) -> Any:
+                return M.delta_args(self.rows, q, k, v, logits, bias, log_rate, state, out, heads=heads, key_heads=key_heads, dim=dim, vdim=vdim)
+            if self.decode and vdim % 4 == 0 and vdim <= 1024 and dim <= 4096:
+                a = args(mixed)
+                self._emit(lambda: M.delta_step(a, gate, norm, eps), "b200.delta_step")
+                return
+            out = self._scratch("recurrence", heads * vdim)
+            a = args(out)
+            aligned = q.stride(0) % 8 == 0 and not any(t.data_ptr() % 16 for t in (q, k, v))
+            if M.delta_chunked_supported(dim, vdim, eng.dtype) and aligned:
+                ws = eng.scratch("delta_ws", M.delta_workspace_bytes(self.batch, self.segments, heads))
+                self._emit(lambda: M.delta_chunked(a, ws), "b200.delta_chunked", launches=2)
+            else:
+                self._emit(lambda: M.delta_simple(a), "b200.delta_simple")
+            self._emit(lambda: H.gated_parts_rms(out, gate, norm, eps, mixed, parts=heads, gate_first=False), "b200.gated_parts_rms")
+
+        def _lower_gated_parts_rms(self, idx: int, node: Any) -> None:
+            o, gate = self._env[node.inputs[0]], self._env[node.inputs[1]]
+            w, eps = self.engine.weights.get_f32(node.inputs[2]), float(node.attrs["eps"])
+            parts, first = int(node.attrs["parts"]), bool(node.attrs["gate_first"])
+            out = self._scratch("mixed", int(o.shape[1]))
+            self._emit(lambda: H.gated_parts_rms(o, gate, w, eps, out, parts=parts, gate_first=first), "b200.gated_parts_rms")
+            self._env[node.outputs[0]] = out
+
         def _lower_gated_rms_norm(self, idx: int, node: Any) -> None:
             o, gate = self._env[node.inputs[0]], self._env[node.inputs[1]]
             w, eps = self.engine.weights.get_f32(node.inputs[2]), float(node.attrs["eps"])
@@ -371,7 +484,8 @@ def make_plan_class(base: type) -> type:
             else:
                 out = self._scratch(str(node.attrs.get("role", "sublayer")), int(w.shape[0]))      # (a shared expert's lives until the combine)
             bias = node.attrs.get("bias")
-            self._dense(x, w, out, None if bias is None else eng.weights.get_f32(bias), "." + str(node.attrs["projection"]))
+            self._dense(x, w, out, None if bias is None else eng.weights.get_f32(bias), "." + str(node.attrs["projection"]),
+                        relu2=node.attrs.get("activation") == "relu2")
             self._env[node.outputs[0]] = out
 
         def _lower_residual_dynamic_tanh(self, idx: int, node: Any) -> None:
@@ -425,7 +539,8 @@ def make_plan_class(base: type) -> type:
 
         def _lower_residual_add(self, idx: int, node: Any) -> None:
             y, res = self._env[node.inputs[1]], self._residual
-            self._finish_residual(idx, lambda nx: self._emit(lambda: H.residual_add(res, y, nx), "b200.residual_add"))
+            scale = self.engine.weights.get_f32(node.inputs[2]) if len(node.inputs) > 2 else None
+            self._finish_residual(idx, lambda nx: self._emit(lambda: H.residual_add(res, y, nx, scale), "b200.residual_add"))
 
         def _lower_residual_rms_pair(self, idx: int, node: Any) -> None:
             y1, y2, res = self._env[node.inputs[1]], self._env[node.inputs[3]], self._residual
@@ -440,6 +555,40 @@ def make_plan_class(base: type) -> type:
             out = self._scratch("final" if logits else "normed", int(w.numel()), rows=self.logit_rows if logits else None)
             index = self.logit_index if logits else None
             self._emit(lambda: H.rms_rows(self._residual, w, eps, out, index), "b200.rms_rows")
+            self._env[node.outputs[0]] = out
+
+        def _lower_layer_norm(self, idx: int, node: Any) -> None:
+            w, eps = self.engine.weights.get_f32(node.inputs[1]), float(node.attrs["eps"])
+            logits = node.attrs.get("rows") == "logits"
+            out = self._scratch("final" if logits else "normed", int(w.numel()), rows=self.logit_rows if logits else None)
+            index = self.logit_index if logits else None
+            self._emit(lambda: H.layer_norm_rows(self._residual, w, eps, out, index), "b200.layer_norm_rows")
+            self._env[node.outputs[0]] = out
+
+        def _lower_talking_attention(self, idx: int, node: Any) -> None:
+            eng, at = self.engine, node.attrs
+            q, k, v = (self._env[n] for n in node.inputs[:3])
+            heads, kv_heads, dim, vdim, rot = (int(at[n]) for n in ("heads", "kv_heads", "dim", "vdim", "rot_dims"))
+            pool = eng.allocator.pool_for_layer(int(at["layer"]))
+            yarn = at.get("yarn")
+            table = None
+            if rot:
+                table = eng.rotate_half_table(rot, float(at["rot_base"])) if yarn is None else eng.yarn_table(rot, float(at["rot_base"]), tuple(map(float, yarn)))
+            args = M.talking_args(self.rows, pool["keys"], pool["values"], eng.weights.get_f32(node.inputs[3]), heads=heads, kv_heads=kv_heads, dim=dim,
+                                  vdim=vdim, window=int(at["window"]), scale=float(at["scale"]))
+            shape = (heads, kv_heads, dim, vdim, eng.page_size, eng.dtype)
+            step = self.decode and M.talking_step_supported(*shape)
+            mixed = not step and M.talking_prompt_supported(*shape)
+            prepared = self._scratch("prepared_q", heads * dim * (kv_heads if mixed else 1))
+            out = self._scratch("mixed", heads * vdim)
+            self._emit(lambda: M.talking_prepare(args, q, k, v, prepared, eps=float(at["eps"]), table=table, mixed=mixed), "b200.talking_prepare")
+            if step:
+                splits = M.talking_step_splits(self.batch, heads, kv_heads, dim, vdim, int(at["window"]), self.width, eng.page_size)
+                self._emit(lambda: M.talking_step(args, prepared, out, splits=splits), "b200.talking_step")
+            elif mixed:
+                self._emit(lambda: M.talking_prompt(args, prepared, out), "b200.talking_prompt")
+            else:
+                self._emit(lambda: M.talking_simple(args, prepared, out), "b200.talking_simple")
             self._env[node.outputs[0]] = out
 
         def _lower_tied_attention(self, idx: int, node: Any) -> None:

@@ -57,7 +57,7 @@ HYBRID_KERNELS_FOR_OP: dict[str, tuple[str, ...]] = {
     "scaled_token_embedding": ("cacheir_b200_scaled_embedding",),
     "dynamic_tanh": ("cacheir_b200_dyt_rows",),
     "concat_matmul": ("cacheir_b200_dense_gemm", "cacheir_b200_dense_simple", "cacheir_b200_silu_cols"),
-    "matmul": ("cacheir_b200_dense_gemm", "cacheir_b200_dense_simple"),
+    "matmul": ("cacheir_b200_dense_gemm", "cacheir_b200_dense_simple", "cacheir_b200_relu2_cols"),
     "latent_attention": ("cacheir_b200_latent_prepare", "cacheir_b200_dense_gemm", "cacheir_b200_latent_attention",
                          "cacheir_b200_latent_attention_simple"),
     "linear_recurrence": ("cacheir_b200_recurrence_step", "cacheir_b200_recurrence_chunked", "cacheir_b200_recurrence_simple"),
@@ -77,6 +77,13 @@ HYBRID_KERNELS_FOR_OP: dict[str, tuple[str, ...]] = {
     "matrix_memory": ("cacheir_b200_memory_step", "cacheir_b200_memory_gates", "cacheir_b200_recurrence_chunked", "cacheir_b200_recurrence_simple",
                       "cacheir_b200_memory_norm"),
     "residual_add": ("cacheir_b200_residual_add",),
+    "join_embedding": ("cacheir_b200_join_embedding", "cacheir_b200_dense_gemm", "cacheir_b200_dense_simple"),
+    "layer_norm": ("cacheir_b200_layer_norm_rows",),
+    "talking_attention": ("cacheir_b200_talking_prepare", "cacheir_b200_talking_step", "cacheir_b200_talking_prompt", "cacheir_b200_talking_simple"),
+    "short_conv": ("cacheir_b200_short_conv",),
+    "state_space": ("cacheir_b200_state_space_step", "cacheir_b200_state_space_gates", "cacheir_b200_recurrence_chunked", "cacheir_b200_recurrence_simple"),
+    "delta_rule": ("cacheir_b200_delta_step", "cacheir_b200_delta_chunked", "cacheir_b200_delta_simple", "cacheir_b200_gated_parts_rms"),
+    "gated_parts_rms": ("cacheir_b200_gated_parts_rms",),
     "residual_rms_pair": ("cacheir_b200_residual_rms_pair",),
     "combine_residual": ("cacheir_b200_combine_residual",),
 }
@@ -106,6 +113,10 @@ B200_BACKEND = Backend(
         "linear_recurrence",
         "tied_attention",
         "matrix_memory",
+        "talking_attention",
+        "state_space",
+        "delta_rule",
+        "short_conv",
         "grouped_gemm_bf16",
         "expert_routing",
     ),

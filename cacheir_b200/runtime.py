@@ -35,7 +35,7 @@ from . import hybrid_ops, ops
 from .artifact import CompileArtifact
 from .kv_cache import B200KVPageAllocator, B200PagedKVCache, KVPoolExhausted
 from .quantization import B200PackedWeight, concat_rows, quant_bits, to_tiled
-from .ragged import bucket, make_plan_class, rotate_half_table
+from .ragged import bucket, make_plan_class, rotate_half_table, yarn_table
 from .tensor_parallel import PeerCollectives, TensorParallel, shard_columns, shard_rows
 from .weights import B200WeightStore, TensorSource
 
@@ -270,6 +270,12 @@ class _Engine:
         """Several weights of one input, row after row."""
         return self._derive(("concat",) + names, lambda: torch.cat([self.weights.get_checked(n) for n in names]).contiguous(), names)
 
+    def concat_f32(self, names: tuple[str, ...]) -> torch.Tensor:
+        """Several float32 parameters, row after row."""
+        if len(names) == 1:
+            return self.weights.get_f32(names[0])
+        return self._derive(("concat_f32",) + names, lambda: torch.cat([self.weights.get_f32(n) for n in names]).contiguous(), names)
+
     def concat_bias(self, biases: tuple[str | None, ...], names: tuple[str, ...]) -> torch.Tensor:
         """float32 biases of `concat_weight(names)`, zeros where a weight has none."""
         return self._derive(("concat_bias",) + biases + names, lambda: torch.cat([
@@ -318,6 +324,9 @@ class _Engine:
     def rotate_half_table(self, dims: int, base: float, scaling: tuple[float, ...] | None = None) -> torch.Tensor:
         return self._derive(("rotate_half", dims, base, scaling),
                             lambda: torch.from_numpy(rotate_half_table(self.max_seq_len, dims, base, scaling)).to(self.device))
+
+    def yarn_table(self, dims: int, base: float, yarn: tuple[float, float, float, float]) -> torch.Tensor:
+        return self._derive(("yarn", dims, base, yarn), lambda: torch.from_numpy(yarn_table(self.max_seq_len, dims, base, yarn)).to(self.device))
 
     def decay_powers(self, decay: tuple[float, ...]) -> torch.Tensor:
         return self._derive(("decay",) + decay, lambda: hybrid_ops.decay_powers(decay, self.device))

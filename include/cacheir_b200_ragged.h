@@ -25,6 +25,7 @@ extern "C" {
 #define CACHEIR_B200_NEXT_COPY 1   /* the residual itself, rounded to the activation type */
 #define CACHEIR_B200_NEXT_DYT 2    /* tanh(alpha * residual) * w + b                      */
 #define CACHEIR_B200_NEXT_RMS 3    /* residual / sqrt(mean(residual^2) + alpha) * w       */
+#define CACHEIR_B200_NEXT_LAYER 4  /* (residual - mean) / sqrt(variance + alpha) * w      */
 
 /* Epilogues of cacheir_b200_dense_gemm */
 #define CACHEIR_B200_DENSE_BF16 0        /* y                                                        */
@@ -36,6 +37,7 @@ extern "C" {
 #define CACHEIR_B200_DENSE_GELU_EMBED 6  /* gelu_tanh(y) * table[ids[t], table_col + column]         */
 #define CACHEIR_B200_DENSE_SWIGLU 7      /* as GEGLU with silu(gate) * up                            */
 #define CACHEIR_B200_DENSE_CLAMPED_GLU 8 /* as GEGLU with g sigmoid(1.702 g) (u + 1), g = min(gate, limit), u = up in [-limit, limit] */
+#define CACHEIR_B200_DENSE_RELU2 9       /* max(y, 0)^2 */
 
 typedef struct {
   const void* x;            /* bf16 [T, x_stride]                                        */
@@ -83,8 +85,14 @@ int cacheir_b200_dyt_rows(const float* residual, const int32_t* row_index, const
 /* out[j] = x / sqrt(mean(x^2) + eps) * w, x = residual[row_index ? row_index[j] : j] */
 int cacheir_b200_rms_rows(const float* residual, const int32_t* row_index, const float* w, float eps, void* out, int rows, int width,
                           int dtype, void* stream);
-/* residual += y, then next_mode (NONE, COPY or RMS) */
-int cacheir_b200_residual_add(float* residual, const void* y, int rows, int width, int next_mode, const float* next_w, const float* next_b,
+/* out[j] = (x - mean) / sqrt(variance + eps) * w, x = residual[row_index ? row_index[j] : j] */
+int cacheir_b200_layer_norm_rows(const float* residual, const int32_t* row_index, const float* w, float eps, void* out, int rows,
+                                 int width, int dtype, void* stream);
+/* out [rows, 2*width] = (residual | table[ids]), the input of a product that meets the embedding output again */
+int cacheir_b200_join_embedding(const float* residual, const void* table, const int64_t* ids, void* out, int rows, int width, int vocab,
+                                int dtype, void* stream);
+/* residual += y * scale (scale [width], NULL: ones), then next_mode (NONE, COPY, RMS or LAYER) */
+int cacheir_b200_residual_add(float* residual, const void* y, const float* scale, int rows, int width, int next_mode, const float* next_w, const float* next_b,
                               float next_alpha, void* next_out, int dtype, void* stream);
 /* residual += factor * (rms(y1) * w1 + rms(y2) * w2) with rms(y) = y / sqrt(mean(y^2) + eps), then next_mode (NONE, COPY or RMS) */
 int cacheir_b200_residual_rms_pair(float* residual, const void* y1, const float* w1, const void* y2, const float* w2, float factor, float eps,
@@ -105,8 +113,14 @@ int cacheir_b200_glu_pairs(const void* y, void* out, int rows, int ff, int epilo
 /* out = gelu_tanh(g) * table[ids, table_col + column] */
 int cacheir_b200_gelu_embed(const void* g, const int64_t* ids, const void* table, long long table_stride, int table_col, void* out,
                             int rows, int dim, int vocab, int dtype, void* stream);
-/* silu in place on columns [0, cols) of y [rows, stride] */
+/* silu in place on columns [0, cols) of y [rows, stride]; likewise max(y, 0)^2 */
 int cacheir_b200_silu_cols(void* y, int rows, long long stride, int cols, int dtype, void* stream);
+int cacheir_b200_relu2_cols(void* y, int rows, long long stride, int cols, int dtype, void* stream);
+/* Norm in `parts` equal parts of a row, each by its own root mean square, with a gate [rows, gate_stride] and a weight w (one entry
+ * per column, or with shared_weight per column of a part):
+ *   gate_first:  y = o * silu(gate), out = y / sqrt(mean(y^2) + eps) * w        else  out = o / sqrt(mean(o^2) + eps) * w * silu(gate) */
+int cacheir_b200_gated_parts_rms(const void* o, const void* gate, long long gate_stride, const float* w, int shared_weight, int gate_first,
+                                 float eps, void* out, int rows, int cols, int parts, int dtype, void* stream);
 
 /* First bounded wait of this library's kernels that gave up since the last reset (0: none). Synchronises. */
 int cacheir_b200_ragged_device_status(int reset);

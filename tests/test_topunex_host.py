@@ -54,10 +54,13 @@ def test_every_graph_op_has_kernels_in_the_registry():
     from cacheir_b200.topunex import build_topunex_graph
     from gutorax_models import CONFIGS as OTHERS
     from rekodra_models import CONFIGS as THIRD
+    from cacheir_b200.zimorax import ZimoraxConfig, build_zimorax_graph
+    from zimorax_models import CONFIGS as FOURTH
 
     used = {n.op for name in CONFIGS for n in build_topunex_graph(_config(name)).nodes}
     used |= {n.op for cfg in OTHERS.values() for n in build_gutorax_graph(GutoraxConfig.from_dict(cfg)).nodes}
     used |= {n.op for cfg in THIRD.values() for n in build_rekodra_graph(RekodraConfig.from_dict(cfg)).nodes}
+    used |= {n.op for cfg in FOURTH.values() for n in build_zimorax_graph(ZimoraxConfig.from_dict(cfg)).nodes}
     assert used == set(registry.HYBRID_KERNELS_FOR_OP)
     exported = {name for table in _lib.GROUP_SIGNATURES.values() for name in table}
     assert {k for names in registry.HYBRID_KERNELS_FOR_OP.values() for k in names} <= exported
