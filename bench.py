@@ -859,8 +859,8 @@ def main() -> None:
     parser.add_argument("--separate-attention-prepass", action="store_true",
                         help="diagnostic: run the o projection's activation pre-pass as its own launch instead of inside the attention kernel")
     parser.add_argument("--no-tp-leg", action="store_true", help="with --gpus N > 1: skip the tensor-parallel leg attached to the line")
-    parser.add_argument("--family", choices=["gutorax", "topunex", "rekodra"], help="throughput and per-kernel rooflines of this model family "
-                        "beside the Llama-shaped one (topunex: and beside gutorax; rekodra: beside topunex and gutorax) at equal size (bench_hybrid.py); one JSON line per size")
+    parser.add_argument("--family", choices=["gutorax", "topunex", "rekodra", "zimorax"], help="throughput and per-kernel rooflines of this model family "
+                        "beside the Llama-shaped one (topunex: and beside gutorax; rekodra: beside topunex and gutorax; zimorax: beside rekodra and gutorax) at equal size (bench_hybrid.py); one JSON line per size")
     parser.add_argument("--family-sizes", default="4096,2048")
     parser.add_argument("--prompt", type=int, default=2048, help="--family: prompt tokens of the prefill measurement")
     parser.add_argument("--ctx", type=int, default=2048, help="--family: cached tokens per sequence when decoding")
@@ -899,7 +899,8 @@ def main() -> None:
             clocks = ClockSampler(0)
             clocks.start()
             line = bench_hybrid.run(size, batch, args.ctx, args.prompt, min(args.steps, 32), peaks,
-                                    {"topunex": ("topunex", "gutorax"), "rekodra": ("rekodra", "topunex", "gutorax")}.get(args.family, (args.family,)))
+                                    {"topunex": ("topunex", "gutorax"), "rekodra": ("rekodra", "topunex", "gutorax"),
+                                     "zimorax": ("zimorax", "rekodra", "gutorax")}.get(args.family, (args.family,)))
             emit(dict(line, clocks=clocks.stop(), peaks="measured" if peaks_path.exists() else "fallback"))
         return
     cfg = dict(WORKLOADS[args.workload])

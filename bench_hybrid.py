@@ -1,4 +1,4 @@
-"""`bench.py --family gutorax|topunex|rekodra`: prefill and decode throughput of a ragged family beside the other ones at equal
+"""`bench.py --family gutorax|topunex|rekodra|zimorax`: prefill and decode throughput of a ragged family beside the other ones at equal
 width, (active) feed-forward, heads and layer count (random weights), and every kernel's distance from its roofline.
 
 Throughput: decode is `decode_greedy_batch` (CUDA-graph replay, argmax fed back on the device) over `batch` sequences
@@ -64,6 +64,28 @@ def rekodra_config(s: dict) -> dict:
                        for i in range(s["layers"])]}
 
 
+def zimorax_shape(s: dict, i: int) -> dict:
+    """Mixer sizes of layer i: talking-heads attention, a state space of twice the width, a delta rule with a key head per two heads,
+    in turn."""
+    if i % 3 == 0:
+        return {"heads": s["heads"], "kv_heads": s["kv_heads"], "dim": s["dim"], "vdim": s["dim"]}
+    if i % 3 == 1:
+        return {"heads": 2 * s["width"] // 64, "vdim": 64, "state": 128, "groups": 8, "norm_groups": 8, "conv": 4}
+    return {"heads": s["heads"], "kv_heads": s["heads"] // 2, "dim": s["dim"], "vdim": s["dim"], "conv": 4}
+
+
+def zimorax_config(s: dict) -> dict:
+    """Feed-forward layers without a gate have 3/2 of the width, so that their weights are as many."""
+    layers = []
+    for i in range(s["layers"]):
+        m = zimorax_shape(s, i)
+        if i % 3 == 0:
+            m.update(scale=s["dim"] ** -0.5, mask={"size": s["window"]},
+                     rot={"base": 500000.0, "dims": s["rot"], "scaling": {"factor": 8.0, "original": 8192, "fast": 32.0, "slow": 1.0}})
+        layers.append({"type": ("attention", "mamba2", "delta")[i % 3], "mixer": m, "mlp": {"kind": "dense", "ff": s["ff"] * 3 // 2}})
+    return {"architecture": "Zimorax", "width": s["width"], "vocab": s["vocab"], "norm": {"eps": 1e-6}, "layers": layers}
+
+
 def synthetic(device):
     import zlib
 
@@ -77,6 +99,10 @@ def synthetic(device):
             return torch.zeros(shape, device=device)
         if key.endswith("mix.right.f.b"):
             return torch.full(shape, 4.0, device=device)
+        if key.endswith(".talk"):
+            return torch.eye(shape[0], device=device) + 0.02
+        if key.endswith(("dt_bias", "A_log")):
+            return torch.full(shape, -2.0, device=device)
         if len(shape) <= 1:
             return torch.full(shape, 0.6 if key.endswith("alpha") else 1.0, device=device)
         gen.manual_seed(zlib.crc32(key.encode()))
@@ -88,7 +114,8 @@ def build(family: str, s: dict, *, batch: int, positions: int):
     import torch
 
     from cacheir_b200 import (B200DecodeRuntime, B200KVPageAllocator, GutoraxConfig, ModelConfig, build_decoder_artifact,
-                              RekodraConfig, TopunexConfig, build_gutorax_artifact, build_rekodra_artifact, build_topunex_artifact)
+                              RekodraConfig, TopunexConfig, ZimoraxConfig, build_gutorax_artifact, build_rekodra_artifact, build_topunex_artifact,
+                              build_zimorax_artifact)
     dev = torch.device("cuda", torch.cuda.current_device())
     if family == "gutorax":
         art, page = build_gutorax_artifact(GutoraxConfig.from_dict(gutorax_config(s))), 64
@@ -97,6 +124,8 @@ def build(family: str, s: dict, *, batch: int, positions: int):
         art, page, dtype = build_topunex_artifact(TopunexConfig.from_dict(topunex_config(s))), 64, "bfloat16"
     elif family == "rekodra":
         art, page, dtype = build_rekodra_artifact(RekodraConfig.from_dict(rekodra_config(s))), 64, "bfloat16"
+    elif family == "zimorax":
+        art, page, dtype = build_zimorax_artifact(ZimoraxConfig.from_dict(zimorax_config(s))), 64, "bfloat16"
     else:
         art = build_decoder_artifact(ModelConfig(
             architecture="LlamaForCausalLM", hidden_size=s["width"], intermediate_size=s["ff"], num_layers=s["layers"],
@@ -278,6 +307,52 @@ def rekodra_work(s: dict, rows: int, logit_rows: int, span: int, decode: bool, t
     return work
 
 
+def zimorax_work(s: dict, rows: int, logit_rows: int, keys_per_row: float, cached_rows: float, decode: bool) -> dict[str, list[tuple[float, float]]]:
+    """Talking heads: the mixture of scores counts as heads^2 multiplications per key, whatever form a kernel gives it."""
+    w, ff = s["width"], s["ff"] * 3 // 2
+    work: dict[str, list[tuple[float, float]]] = defaultdict(list)
+
+    def gemm(kind, n, k, n_out, t=rows):
+        work["b200.dense_gemm" + kind].append((2.0 * (n * k + t * k + t * n_out), 2.0 * t * n * k))
+
+    for i in range(s["layers"]):
+        m = zimorax_shape(s, i)
+        h, e = m["heads"], m["vdim"]
+        io = rows * h * e * 2.0
+        if i % 3 == 0:
+            g, d = m["kv_heads"], m["dim"]
+            n = h * d + g * (d + e)
+            gemm("", n, w, n)
+            work["b200.talking_prepare"].append((2.0 * rows * 2 * n, 0.0))
+            work["b200.talking_step" if decode else "b200.talking_prompt"].append(
+                (2.0 * (cached_rows * g * (d + e) + rows * h * (d + e)), 2.0 * rows * h * keys_per_row * (d + h + e)))
+        else:
+            d = m["state"] if i % 3 == 1 else m["dim"]
+            channels = h * e + 2 * d * (m["groups"] if i % 3 == 1 else m["kv_heads"])
+            state = h * d * e * 8.0 * (rows if decode else 1)
+            n = channels + h * e + h * (1 if i % 3 == 1 else 2)
+            gemm("", n, w, n)
+            work["b200.short_conv"].append((rows * channels * 4.0 + (rows * (m["conv"] - 1) * channels * 8.0 if decode else 0.0), 0.0))
+            inputs = rows * (channels * 2.0 + h * 4)
+            if i % 3 == 1:
+                if not decode:
+                    work["b200.state_space_gates"].append((rows * h * 12.0, 0.0))
+                work["b200.state_space_step" if decode else "b200.recurrence_chunked"].append((state + inputs + io, rows * h * 4.0 * d * e))
+                work["b200.gated_parts_rms"].append((3 * io, 0.0))
+            else:
+                work["b200.delta_step" if decode else "b200.delta_chunked"].append((state + inputs + (2 if decode else 1) * io, rows * h * 6.0 * d * e))
+                if not decode:
+                    work["b200.gated_parts_rms"].append((3 * io, 0.0))
+        gemm(".o", w, h * e, w)
+        gemm(".up", ff, w, ff)
+        gemm(".down", w, ff, w)
+        work["b200.residual_add"] += [(rows * w * (2 + 8 + 2.0), 0.0)] * 2
+    work["b200.scaled_embedding"].append((rows * w * (2 + 4 + 2.0), 0.0))
+    work["b200.layer_norm_rows"].append((logit_rows * w * 6.0, 0.0))
+    gemm(".lm_head", s["vocab"], w, 2 * s["vocab"], t=logit_rows)
+    return work
+
+
 def llama_work(s: dict, rows: int, keys_per_row: float, cached_rows: float) -> dict[str, list[tuple[float, float]]]:
     w, ff, d = s["width"], s["ff"], s["width"] // s["heads"]
     kv = s["kv_heads"] * d
@@ -309,7 +384,7 @@ def against_roofline(times: dict[str, tuple[int, float]], work: dict, hbm_gbs: f
     return out
 
 
-RAGGED = ("gutorax", "topunex", "rekodra")
+RAGGED = ("gutorax", "topunex", "rekodra", "zimorax")
 
 
 def ragged_kernels(family: str, rt, plan, s: dict, rows: int, logit_rows: int, keys: float, cached: float, span: int, decode: bool, hbm: float,
@@ -318,6 +393,8 @@ def ragged_kernels(family: str, rt, plan, s: dict, rows: int, logit_rows: int, k
     times = kind_times(plan)
     if family == "gutorax":
         return against_roofline(times, gutorax_work(s, rows, logit_rows, keys, cached, decode), hbm, tf)
+    if family == "zimorax":
+        return against_roofline(times, zimorax_work(s, rows, logit_rows, keys, cached, decode), hbm, tf)
     if family == "rekodra":
         cu = rt._engine.scratch("route_cu", 0).view(torch.int32)[: s["experts"] * 7 // 8 + 1]
         return against_roofline(times, rekodra_work(s, rows, logit_rows, span, decode, int((cu.diff() > 0).sum()), int(cu[-1])), hbm, tf)

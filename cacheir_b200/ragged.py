@@ -574,7 +574,7 @@ def make_plan_class(base: type) -> type:
             table = None
             if rot:
                 table = eng.rotate_half_table(rot, float(at["rot_base"])) if yarn is None else eng.yarn_table(rot, float(at["rot_base"]), tuple(map(float, yarn)))
-            args = M.talking_args(self.rows, pool["keys"], pool["values"], eng.weights.get_f32(node.inputs[3]), heads=heads, kv_heads=kv_heads, dim=dim,
+            args = M.talking_args(self.rows, pool["key_rows"], pool["value_rows"], eng.weights.get_f32(node.inputs[3]), heads=heads, kv_heads=kv_heads, dim=dim,
                                   vdim=vdim, window=int(at["window"]), scale=float(at["scale"]))
             shape = (heads, kv_heads, dim, vdim, eng.page_size, eng.dtype)
             step = self.decode and M.talking_step_supported(*shape)

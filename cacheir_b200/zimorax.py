@@ -188,7 +188,7 @@ class ZimoraxConfig:
         for run, at in enumerate(self.runs):
             m = self.layers[at.layer].mixer
             if isinstance(m, TalkingMixer):
-                pools[run] = {"keys": ((page_size, m.kv_heads * m.dim), dtype), "values": ((page_size, m.kv_heads * m.vdim), dtype)}
+                pools[run] = {"key_rows": ((page_size, m.kv_heads * m.dim), dtype), "value_rows": ((page_size, m.kv_heads * m.vdim), dtype)}
             else:
                 states[run] = (state_floats(m)[1],)
         return pools, states

@@ -156,7 +156,7 @@ def test_step_attention(shape, splits):
 def test_simple_attention(shape, dtype):
     for mask in (dict(size=37, rot=2, yarn=(3.0, 20.0, 2.0, 0.1)), dict(size=None), dict(size=1), dict(size=64, rot=2)):
         got, want = _attend(np.random.default_rng(3), shape, PORTIONS, dtype=dtype, kernel="simple", **mask)
-        _rows_close(got, want, 2e-5 if dtype == "float32" else 1.5e-2)
+        _rows_close(got, want, 2e-5 if dtype == "float32" else 2.5e-2)
 
 
 @pytest.mark.parametrize("kernel", ["prompt", "step", "simple"])

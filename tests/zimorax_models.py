@@ -46,8 +46,8 @@ CONFIGS = {
                              (attention(8, 8, 64, 200, window=130, yarn=None), None), (delta(2, 2, 112, 8, conv=1), 24), (attention(2, 2, 256, 256, window=1), None)],
                    loop=(0, 2, 3)),
     "odd": config(90, 77, [(delta(3, 1, 10, 7, conv=5), 11), (attention(4, 2, 7, 11, window=13, rot=6, yarn=(2.0, 16.0, 2.0, 0.25)), 13),
-                           (mamba2(5, 6, 12, groups=5, norm_groups=3, conv=3), 90), (attention(3, 3, 25, 3, window=50, rot=0), None),
-                           (mamba2(2, 9, 20, groups=2, norm_groups=2, conv=6), None)], loop=(2, 5, 2)),
+                           (mamba2(5, 6, 12, groups=5, norm_groups=3, conv=3), 90), (attention(3, 3, 25, 9, window=50, rot=0), None),
+                           (mamba2(2, 9, 20, groups=2, conv=6), None)], loop=(2, 5, 2)),
     "ones": config(16, 40, [(attention(1, 1, 2, 1, window=2, rot=2), 1), (mamba2(1, 1, 1, conv=1), 8), (delta(1, 1, 1, 1, conv=1), 1),
                             (mamba2(2, 8, 16, groups=2, conv=2), None), (delta(2, 1, 16, 8, conv=2), 16)], loop=(3, 4, 1)),
 }
