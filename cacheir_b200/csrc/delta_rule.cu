@@ -217,21 +217,20 @@ __device__ __forceinline__ void split_pair(float x, float y, uint32_t* hi, uint3
 __global__ void __launch_bounds__(128)
 delta_local_kernel(const Args a, const ChunkSpace ws) {
   extern __shared__ __align__(16) uint8_t raw[];
-  constexpr int kPitch = kChunk + 1;
+  constexpr int kPitch = kChunk + 4;
   const int dim = a.dim, pitch = dim + 8;
   __nv_bfloat16* s_q = reinterpret_cast<__nv_bfloat16*>(raw);        // [64][pitch]
   __nv_bfloat16* s_k = s_q + kChunk * pitch;                         // [64][pitch]
-  float* s_a = reinterpret_cast<float*>(s_k + kChunk * pitch);       // [64][65] A
-  float* s_m = s_a + kChunk * kPitch;                                // [64][65] its inverse
-  float* s_t = s_m + kChunk * kPitch;                                // [32][33]
+  float* s_a = reinterpret_cast<float*>(s_k + kChunk * pitch);       // [64][kPitch] A
+  float* s_m = s_a + kChunk * kPitch;                                // [64][kPitch] (I + A)^-1
+  float* s_t = s_m + kChunk * kPitch;                                // [32][36]
   __shared__ float4 s_row[kChunk];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, h = blockIdx.y, kh = key_head(a, h);
   const RaggedItem it = find_item(a.cu_rows, a.segments, kChunk, blockIdx.x);
   if (it.seg < 0) return;
   const size_t unit = static_cast<size_t>(blockIdx.x) * a.heads + h;
-  const int n = it.count, kc = dim / 8;
-  for (int i = threadIdx.x; i < kChunk * kc; i += 128) {
-    const int r = i / kc, c = i % kc;
+  const int n = it.count, kc = dim / 8, r_step = 128 / kc, c_step = 128 % kc;
+  for (int r = static_cast<int>(threadIdx.x) / kc, c = static_cast<int>(threadIdx.x) % kc; r < kChunk;) {
     uint4 q = make_uint4(0u, 0u, 0u, 0u), k = q;
     if (r < n) {
       const size_t off = static_cast<size_t>(it.row0 + r) * a.stride + static_cast<size_t>(kh) * dim + c * 8;
@@ -240,7 +239,11 @@ delta_local_kernel(const Args a, const ChunkSpace ws) {
     }
     *reinterpret_cast<uint4*>(s_q + r * pitch + c * 8) = q;
     *reinterpret_cast<uint4*>(s_k + r * pitch + c * 8) = k;
+    r += r_step;
+    c += c_step;
+    if (c >= kc) { c -= kc; ++r; }
   }
+  for (int i = threadIdx.x; i < kChunk * kPitch; i += 128) s_m[i] = 0.f;
   if (warp == 0) {                     // gates and the running sum of log decays
     float last = 0.f;
 #pragma unroll
@@ -316,7 +319,7 @@ delta_local_kernel(const Args a, const ChunkSpace ws) {
       for (int e = 0; e < 4; ++e) {
         const int i = i0 + (e >> 1) * 8, j = kt * 16 + u * 8 + (lane & 3) * 2 + (e & 1);
         const float4 ri = s_row[i], rj = s_row[j];
-        const float d = j <= i ? expf(ri.x - rj.x) * rj.z : 0.f;
+        const float d = j <= i ? __expf(ri.x - rj.x) * rj.z : 0.f;
         p[u][e] = qk[2 * kt + u][e] * d * ri.w;
         s_a[i * kPitch + j] = j < i ? kk[2 * kt + u][e] * d * ri.z * ri.y : 0.f;
       }
@@ -348,33 +351,44 @@ delta_local_kernel(const Args a, const ChunkSpace ws) {
     }
   }
   __syncthreads();
-  // lower left blocks of size m from the diagonal ones: -M22 (A21 M11)
+  // lower left blocks of size m from the diagonal ones: -M22 (A21 M11); a thread has ROWS rows of four columns
+  auto lower_left = [&](auto size, auto count) {
+    constexpr int m = decltype(size)::value, ROWS = decltype(count)::value, kPitchT = 36;
+    const int unit_rows = m / ROWS, units = unit_rows * (m / 4), pair = static_cast<int>(threadIdx.x) / units, at = static_cast<int>(threadIdx.x) % units;
+    const int r0 = at / (m / 4) * ROWS, c0 = at % (m / 4) * 4, b = pair * 2 * m;
+    float* t = s_t + pair * m * kPitchT;
+    auto product = [&](const float* x, const float* y, int y_pitch, int from, int to, float (&out)[ROWS][4]) {
 #pragma unroll
-  for (int m = 16; m <= 32; m *= 2) {
-    const int pairs = 32 / m, cells = m * m;      // two pairs of 16, one of 32
-    for (int i = threadIdx.x; i < pairs * cells; i += 128) {
-      const int p = i / cells, r = i % cells / m, c = i % m, b = p * 2 * m;
-      float t = 0.f;
-      for (int j = c; j < m; ++j) t = fmaf(s_a[(b + m + r) * kPitch + b + j], s_m[(b + j) * kPitch + b + c], t);
-      s_t[p * 16 * 33 + r * 33 + c] = t;
-    }
+      for (int r = 0; r < ROWS; ++r)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) out[r][e] = 0.f;
+      for (int j = from; j < to; ++j) {
+        const float4 v = *reinterpret_cast<const float4*>(y + j * y_pitch);
+#pragma unroll
+        for (int r = 0; r < ROWS; ++r) {
+          const float f = x[r * kPitch + j];
+          out[r][0] = fmaf(f, v.x, out[r][0]); out[r][1] = fmaf(f, v.y, out[r][1]); out[r][2] = fmaf(f, v.z, out[r][2]); out[r][3] = fmaf(f, v.w, out[r][3]);
+        }
+      }
+    };
+    float out[ROWS][4];
+    product(s_a + (b + m + r0) * kPitch + b, s_m + b * kPitch + b + c0, kPitch, c0, m, out);
+#pragma unroll
+    for (int r = 0; r < ROWS; ++r) *reinterpret_cast<float4*>(t + (r0 + r) * kPitchT + c0) = make_float4(out[r][0], out[r][1], out[r][2], out[r][3]);
     __syncthreads();
-    for (int i = threadIdx.x; i < pairs * cells; i += 128) {
-      const int p = i / cells, r = i % cells / m, c = i % m, b = p * 2 * m;
-      float t = 0.f;
-      for (int j = 0; j <= r; ++j) t = fmaf(s_m[(b + m + r) * kPitch + b + m + j], s_t[p * 16 * 33 + j * 33 + c], t);
-      s_m[(b + m + r) * kPitch + b + c] = -t;
-    }
+    product(s_m + (b + m + r0) * kPitch + b + m, t + c0, kPitchT, 0, r0 + ROWS, out);
+#pragma unroll
+    for (int r = 0; r < ROWS; ++r)
+      *reinterpret_cast<float4*>(s_m + (b + m + r0 + r) * kPitch + b + c0) = make_float4(-out[r][0], -out[r][1], -out[r][2], -out[r][3]);
     __syncthreads();
-  }
+  };
+  lower_left(std::integral_constant<int, 16>{}, std::integral_constant<int, 1>{});
+  lower_left(std::integral_constant<int, 32>{}, std::integral_constant<int, 2>{});
 #pragma unroll
   for (int kt = 0; kt < 4; ++kt) {
     if (kt > warp) continue;
     const float* m0 = s_m + i0 * kPitch + kt * 16 + (lane & 3) * 2;
-    const bool diagonal = kt == warp;
-    auto entry = [&](int dr, int dc) {             // (above the diagonal nothing was written)
-      return diagonal && (lane & 3) * 2 + dc > (lane >> 2) + dr ? 0.f : m0[dr * kPitch + dc];
-    };
+    auto entry = [&](int dr, int dc) { return m0[dr * kPitch + dc]; };
     uint4 hi, lo;
     split_pair(entry(0, 0), entry(0, 1), &hi.x, &lo.x);
     split_pair(entry(8, 0), entry(8, 1), &hi.y, &lo.y);
@@ -386,20 +400,24 @@ delta_local_kernel(const Args a, const ChunkSpace ws) {
   }
 }
 
-// Four warps with 16 tokens (or 16-row state tiles warp, warp + 4) each; NT 8-column tiles of the values per CTA.
-template <int MT, int NT>
-__global__ void __launch_bounds__(128)
+// Warps 0..3 have the keys' side (16 tokens each: K S, the right-hand sides, the writes U), warps 4..7 the queries' (Q S, P U, the
+// output); all eight have a 16-row tile of the state. NT 8-column tiles of the values per CTA.
+constexpr int kChainThreads = 256;
+template <int NT>
+__global__ void __launch_bounds__(kChainThreads)
 delta_chain_kernel(const Args a, const ChunkSpace ws) {
   constexpr int kCols = NT * 8, kPitchC = kCols + 8;
   extern __shared__ __align__(16) uint8_t raw[];
   const int dim = a.dim, pitch = dim + 8;
   __nv_bfloat16* s_q = reinterpret_cast<__nv_bfloat16*>(raw);        // [2][64][pitch]
   __nv_bfloat16* s_k = s_q + 2 * kChunk * pitch;                     // [2][64][pitch]
-  __nv_bfloat16* s_s = s_k + 2 * kChunk * pitch;                     // [2][dim][kPitchC] state, hi | lo
-  __nv_bfloat16* s_r = s_s + 2 * dim * kPitchC;                      // [2][64][kPitchC] right-hand sides, then decayed writes
-  __nv_bfloat16* s_u = s_r + 2 * kChunk * kPitchC;                   // [2][64][kPitchC] writes
-  float4* s_row = reinterpret_cast<float4*>(s_u + 2 * kChunk * kPitchC);      // [2][64]
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  __nv_bfloat16* s_s = s_k + 2 * kChunk * pitch;                     // [hi, lo][dim][kPitchC] state
+  __nv_bfloat16* s_r = s_s + 2 * dim * kPitchC;                      // [hi, lo][64][kPitchC] right-hand sides
+  __nv_bfloat16* s_u = s_r + 2 * kChunk * kPitchC;                   // [hi, lo][64][kPitchC] writes
+  __nv_bfloat16* s_d = s_u + 2 * kChunk * kPitchC;                   // [hi, lo][64][kPitchC] writes, decayed to the chunk's end
+  float4* s_row = reinterpret_cast<float4*>(s_d + 2 * kChunk * kPitchC);      // [2][64]
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, band = warp & 3;
+  const bool keys = warp < 4;
   const int seg = blockIdx.x, h = blockIdx.y, kh = key_head(a, h), v0 = blockIdx.z * kCols;
   const int row0 = a.cu_rows[seg], rows = a.cu_rows[seg + 1] - row0;
   if (rows <= 0) return;
@@ -407,32 +425,19 @@ delta_chain_kernel(const Args a, const ChunkSpace ws) {
   for (int s = 0; s < seg; ++s) first += (a.cu_rows[s + 1] - a.cu_rows[s] + kChunk - 1) / kChunk;
   const int chunks = (rows + kChunk - 1) / kChunk, cols = min(kCols, a.vdim - v0), kc = dim / 8;
 
-  float* state = slot_state(a, seg, h) + v0;
-  const bool fresh = a.positions[row0] == 0;
-  float st[MT][NT][4];
-#pragma unroll
-  for (int t = 0; t < MT; ++t)
-#pragma unroll
-    for (int nn = 0; nn < NT; ++nn)
-#pragma unroll
-      for (int e = 0; e < 2; ++e) {
-        const int d = (warp + 4 * t) * 16 + (lane >> 2) + e * 8, c = nn * 8 + (lane & 3) * 2;
-        float2 x = make_float2(0.f, 0.f);
-        if (!fresh && d < dim && c < cols) x = *reinterpret_cast<const float2*>(state + static_cast<size_t>(d) * a.vdim + c);
-        st[t][nn][e * 2] = x.x;
-        st[t][nn][e * 2 + 1] = x.y;
-      }
-
+  const int r_first = static_cast<int>(threadIdx.x) / kc, c_first = static_cast<int>(threadIdx.x) % kc, r_step = kChainThreads / kc, c_step = kChainThreads % kc;
   auto fetch = [&](int chunk) {        // q, k and the rows' numbers of a chunk, asynchronously
     const int buf = chunk & 1, n = min(kChunk, rows - chunk * kChunk);
-    for (int i = threadIdx.x; i < kChunk * kc; i += 128) {
-      const int r = i / kc, c = i % kc;
+    for (int r = r_first, c = c_first; r < kChunk;) {
       const size_t off = static_cast<size_t>(row0 + chunk * kChunk + min(r, n - 1)) * a.stride + static_cast<size_t>(kh) * dim + c * 8;
       const int bytes = r < n ? 16 : 0;      // (rows behind the last are zero)
       asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_addr(s_q + (buf * kChunk + r) * pitch + c * 8)),
                    "l"(static_cast<const __nv_bfloat16*>(a.q) + off), "r"(bytes) : "memory");
       asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_addr(s_k + (buf * kChunk + r) * pitch + c * 8)),
                    "l"(static_cast<const __nv_bfloat16*>(a.k) + off), "r"(bytes) : "memory");
+      r += r_step;
+      c += c_step;
+      if (c >= kc) { c -= kc; ++r; }
     }
     if (threadIdx.x < kChunk) {
       const float4* src = ws.rows + (static_cast<size_t>(first + chunk) * a.heads + h) * kChunk + threadIdx.x;
@@ -442,8 +447,23 @@ delta_chain_kernel(const Args a, const ChunkSpace ws) {
   };
   fetch(0);
 
-  const int i0 = warp * 16 + (lane >> 2);
-  const uint32_t frag_row = ((warp * 16 + (lane & 15)) * pitch + (lane >> 4) * 8) * 2;
+  float* state = slot_state(a, seg, h) + v0;
+  const bool fresh = a.positions[row0] == 0;
+  const int m0 = warp * 16;            // this warp's rows of the state
+  float st[NT][4];
+#pragma unroll
+  for (int nn = 0; nn < NT; ++nn)
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      const int d = m0 + (lane >> 2) + e * 8, c = nn * 8 + (lane & 3) * 2;
+      float2 x = make_float2(0.f, 0.f);
+      if (!fresh && d < dim && c < cols) x = *reinterpret_cast<const float2*>(state + static_cast<size_t>(d) * a.vdim + c);
+      st[nn][e * 2] = x.x;
+      st[nn][e * 2 + 1] = x.y;
+    }
+
+  const int i0 = band * 16 + (lane >> 2);
+  const uint32_t frag_row = ((band * 16 + (lane & 15)) * pitch + (lane >> 4) * 8) * 2;
   const uint32_t frag_b = (((lane & 7) + ((lane >> 3) & 1) * 8) * kPitchC + (lane >> 4) * 8) * 2;
   const uint32_t frag_kt = (((lane & 7) + ((lane >> 4) & 1) * 8) * pitch + ((lane >> 3) & 1) * 8) * 2;
   // C fragments of rows i0, i0 + 8 as two bf16 planes
@@ -461,11 +481,12 @@ delta_chain_kernel(const Args a, const ChunkSpace ws) {
       }
   };
   // y += (hi + lo)[64 rows of a triangle's row tile] x [64][columns], the product of the two small parts left out
-  auto triangle = [&](const uint4 (&hi)[4], const uint4 (&lo)[4], const __nv_bfloat16* x, float (&y)[NT][4]) {
+  uint4 hi[4], lo[4];                  // this warp's row tile of M (keys) or P (queries)
+  auto triangle = [&](const __nv_bfloat16* x, float (&y)[NT][4]) {
     const uint32_t xb = smem_addr(x) + frag_b;
 #pragma unroll
     for (int kt = 0; kt < 4; ++kt) {
-      if (kt > warp) continue;
+      if (kt > band) continue;
       const uint32_t ah[4] = {hi[kt].x, hi[kt].y, hi[kt].z, hi[kt].w}, al[4] = {lo[kt].x, lo[kt].y, lo[kt].z, lo[kt].w};
 #pragma unroll
       for (int nn = 0; nn < NT; nn += 2) {
@@ -487,14 +508,12 @@ delta_chain_kernel(const Args a, const ChunkSpace ws) {
     const size_t unit = static_cast<size_t>(first + chunk) * a.heads + h;
     const size_t base = static_cast<size_t>(row0) + chunk * kChunk;
     // operands of this chunk that wait for nothing
-    uint4 mh[4], ml[4], ph[4], pl[4];
 #pragma unroll
     for (int kt = 0; kt < 4; ++kt)
-      if (kt <= warp) {
-        const uint4* m = tile_at(ws, unit, 0, warp, kt);
-        const uint4* p = tile_at(ws, unit, 1, warp, kt);
-        mh[kt] = m[lane]; ml[kt] = m[32 + lane];
-        ph[kt] = p[lane]; pl[kt] = p[32 + lane];
+      if (kt <= band) {
+        const uint4* m = tile_at(ws, unit, keys ? 0 : 1, band, kt);
+        hi[kt] = m[lane];
+        lo[kt] = m[32 + lane];
       }
     uint32_t v[NT][2];
 #pragma unroll
@@ -502,96 +521,84 @@ delta_chain_kernel(const Args a, const ChunkSpace ws) {
 #pragma unroll
       for (int e = 0; e < 2; ++e) {
         const int r = i0 + e * 8, c = nn * 8 + (lane & 3) * 2;
-        v[nn][e] = r < n && c < cols ? *reinterpret_cast<const uint32_t*>(static_cast<const __nv_bfloat16*>(a.v) + (base + r) * a.stride +
-                                                                         static_cast<size_t>(h) * a.vdim + v0 + c) : 0u;
+        v[nn][e] = keys && r < n && c < cols ? *reinterpret_cast<const uint32_t*>(static_cast<const __nv_bfloat16*>(a.v) + (base + r) * a.stride +
+                                                                                 static_cast<size_t>(h) * a.vdim + v0 + c) : 0u;
       }
-#pragma unroll
-    for (int t = 0; t < MT; ++t)
-#pragma unroll
-      for (int nn = 0; nn < NT; ++nn)
-#pragma unroll
-        for (int e = 0; e < 2; ++e) {
-          const int d = (warp + 4 * t) * 16 + (lane >> 2) + e * 8, c = nn * 8 + (lane & 3) * 2;
-          if (d < dim) {
-            uint32_t hi, lo;
-            split_pair(st[t][nn][e * 2], st[t][nn][e * 2 + 1], &hi, &lo);
-            *reinterpret_cast<uint32_t*>(s_s + d * kPitchC + c) = hi;
-            *reinterpret_cast<uint32_t*>(s_s + (dim + d) * kPitchC + c) = lo;
-          }
-        }
-    asm volatile("cp.async.wait_group 0;" ::: "memory");
-    __syncthreads();                   // this chunk's rows and state are there, the other buffer is free
-    if (chunk + 1 < chunks) fetch(chunk + 1);
-
-    float ks[NT][4], o[NT][4];
 #pragma unroll
     for (int nn = 0; nn < NT; ++nn)
 #pragma unroll
-      for (int e = 0; e < 4; ++e) ks[nn][e] = o[nn][e] = 0.f;
-    const uint32_t qa = smem_addr(s_q + buf * kChunk * pitch), ka = smem_addr(s_k + buf * kChunk * pitch), sb = smem_addr(s_s) + frag_b;
+      for (int e = 0; e < 2; ++e) {
+        const int d = m0 + (lane >> 2) + e * 8, c = nn * 8 + (lane & 3) * 2;
+        if (d < dim) {
+          uint32_t sh, sl;
+          split_pair(st[nn][e * 2], st[nn][e * 2 + 1], &sh, &sl);
+          *reinterpret_cast<uint32_t*>(s_s + d * kPitchC + c) = sh;
+          *reinterpret_cast<uint32_t*>(s_s + (dim + d) * kPitchC + c) = sl;
+        }
+      }
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    __syncthreads();                   // this chunk's rows and state are there, the other buffer and the writes are free
+    if (chunk + 1 < chunks) fetch(chunk + 1);
+
+    float x[2][NT][4];                 // K S or Q S, the state's two parts in sums of their own
+#pragma unroll
+    for (int part = 0; part < 2; ++part)
+#pragma unroll
+      for (int nn = 0; nn < NT; ++nn)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) x[part][nn][e] = 0.f;
+    const uint32_t ka = smem_addr(s_k + buf * kChunk * pitch), own = (keys ? ka : smem_addr(s_q + buf * kChunk * pitch)) + frag_row;
+    const uint32_t sb = smem_addr(s_s) + frag_b;
+#pragma unroll 4
     for (int k = 0; k < dim / 16; ++k) {
-      uint32_t fk[4], fq[4];
-      ldsm_x4(ka + frag_row + k * 32, fk);
-      ldsm_x4(qa + frag_row + k * 32, fq);
+      uint32_t f[4];
+      ldsm_x4(own + k * 32, f);
 #pragma unroll
       for (int part = 0; part < 2; ++part)
 #pragma unroll
         for (int nn = 0; nn < NT; nn += 2) {
           uint32_t b[4];
           ldsm_x4_t(sb + ((part * dim + k * 16) * kPitchC + nn * 8) * 2, b);
-          mma_bf16(ks[nn], fk, b[0], b[1]);
-          mma_bf16(ks[nn + 1], fk, b[2], b[3]);
-          mma_bf16(o[nn], fq, b[0], b[1]);
-          mma_bf16(o[nn + 1], fq, b[2], b[3]);
+          mma_bf16(x[part][nn], f, b[0], b[1]);
+          mma_bf16(x[part][nn + 1], f, b[2], b[3]);
         }
     }
     const float4 ra = s_row[buf * kChunk + i0], rb = s_row[buf * kChunk + i0 + 8];      // (c, beta, 1/|k|, 1/|q|)
     const float end = s_row[buf * kChunk + kChunk - 1].x;
-    const float ea = expf(ra.x), eb = expf(rb.x), fa = ea * ra.z, fb = eb * rb.z, ga = ea * ra.w, gb = eb * rb.w;
+    const float ea = __expf(ra.x) * (keys ? ra.z : ra.w), eb = __expf(rb.x) * (keys ? rb.z : rb.w);
+    float y[NT][4];
+    if (keys) {
 #pragma unroll
-    for (int nn = 0; nn < NT; ++nn) {
-      ks[nn][0] = ra.y * (__uint_as_float(v[nn][0] << 16) - fa * ks[nn][0]);
-      ks[nn][1] = ra.y * (__uint_as_float(v[nn][0] & 0xffff0000u) - fa * ks[nn][1]);
-      ks[nn][2] = rb.y * (__uint_as_float(v[nn][1] << 16) - fb * ks[nn][2]);
-      ks[nn][3] = rb.y * (__uint_as_float(v[nn][1] & 0xffff0000u) - fb * ks[nn][3]);
-      o[nn][0] *= ga; o[nn][1] *= ga; o[nn][2] *= gb; o[nn][3] *= gb;
-    }
-    leave(s_r, ks, 1.f, 1.f);
-    __syncthreads();
-    float u[NT][4];
-#pragma unroll
-    for (int nn = 0; nn < NT; ++nn)
-#pragma unroll
-      for (int e = 0; e < 4; ++e) u[nn][e] = 0.f;
-    triangle(mh, ml, s_r, u);
-    leave(s_u, u, 1.f, 1.f);
-    __syncthreads();                   // (everyone is done with the right-hand sides)
-    leave(s_r, u, expf(end - ra.x) * ra.z, expf(end - rb.x) * rb.z);
-    triangle(ph, pl, s_u, o);
-    __nv_bfloat16* out = static_cast<__nv_bfloat16*>(a.out);
-#pragma unroll
-    for (int e = 0; e < 2; ++e) {
-      const int i = i0 + e * 8;
-      if (i < n) {
-        __nv_bfloat16* dst = out + ((base + i) * a.heads + h) * a.vdim + v0;
-#pragma unroll
-        for (int nn = 0; nn < NT; ++nn) {
-          const int c = nn * 8 + (lane & 3) * 2;
-          if (c < cols) *reinterpret_cast<uint32_t*>(dst + c) = pack_bf16(o[nn][e * 2], o[nn][e * 2 + 1]);
-        }
+      for (int nn = 0; nn < NT; ++nn) {
+        y[nn][0] = ra.y * (__uint_as_float(v[nn][0] << 16) - ea * (x[0][nn][0] + x[1][nn][0]));
+        y[nn][1] = ra.y * (__uint_as_float(v[nn][0] & 0xffff0000u) - ea * (x[0][nn][1] + x[1][nn][1]));
+        y[nn][2] = rb.y * (__uint_as_float(v[nn][1] << 16) - eb * (x[0][nn][2] + x[1][nn][2]));
+        y[nn][3] = rb.y * (__uint_as_float(v[nn][1] & 0xffff0000u) - eb * (x[0][nn][3] + x[1][nn][3]));
       }
-    }
-    __syncthreads();
-    const float keep = expf(end);
-    const uint32_t rb_at = smem_addr(s_r) + frag_b;
-#pragma unroll
-    for (int t = 0; t < MT; ++t) {
-      const int m0 = (warp + 4 * t) * 16;
-      if (m0 >= dim) continue;
+      leave(s_r, y, 1.f, 1.f);
+      asm volatile("barrier.cta.sync 1, 128;" ::: "memory");
 #pragma unroll
       for (int nn = 0; nn < NT; ++nn)
 #pragma unroll
-        for (int e = 0; e < 4; ++e) st[t][nn][e] *= keep;
+        for (int e = 0; e < 4; ++e) y[nn][e] = 0.f;
+      triangle(s_r, y);
+      leave(s_u, y, 1.f, 1.f);
+      leave(s_d, y, __expf(end - ra.x) * ra.z, __expf(end - rb.x) * rb.z);
+    } else {
+#pragma unroll
+      for (int nn = 0; nn < NT; ++nn) {
+        y[nn][0] = ea * (x[0][nn][0] + x[1][nn][0]); y[nn][1] = ea * (x[0][nn][1] + x[1][nn][1]);
+        y[nn][2] = eb * (x[0][nn][2] + x[1][nn][2]); y[nn][3] = eb * (x[0][nn][3] + x[1][nn][3]);
+      }
+    }
+    __syncthreads();                   // the writes are there
+    const float keep = __expf(end);
+    if (m0 < dim) {
+      const uint32_t db = smem_addr(s_d) + frag_b;
+#pragma unroll
+      for (int nn = 0; nn < NT; ++nn)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) st[nn][e] *= keep;
 #pragma unroll
       for (int k = 0; k < kChunk / 16; ++k) {
         uint32_t af[4];
@@ -601,23 +608,36 @@ delta_chain_kernel(const Args a, const ChunkSpace ws) {
 #pragma unroll
           for (int nn = 0; nn < NT; nn += 2) {
             uint32_t b[4];
-            ldsm_x4_t(rb_at + ((part * kChunk + k * 16) * kPitchC + nn * 8) * 2, b);
-            mma_bf16(st[t][nn], af, b[0], b[1]);
-            mma_bf16(st[t][nn + 1], af, b[2], b[3]);
+            ldsm_x4_t(db + ((part * kChunk + k * 16) * kPitchC + nn * 8) * 2, b);
+            mma_bf16(st[nn], af, b[0], b[1]);
+            mma_bf16(st[nn + 1], af, b[2], b[3]);
           }
+      }
+    }
+    if (!keys) {
+      triangle(s_u, y);
+      __nv_bfloat16* out = static_cast<__nv_bfloat16*>(a.out);
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        const int i = i0 + e * 8;
+        if (i < n) {
+          __nv_bfloat16* dst = out + ((base + i) * a.heads + h) * a.vdim + v0;
+#pragma unroll
+          for (int nn = 0; nn < NT; ++nn) {
+            const int c = nn * 8 + (lane & 3) * 2;
+            if (c < cols) *reinterpret_cast<uint32_t*>(dst + c) = pack_bf16(y[nn][e * 2], y[nn][e * 2 + 1]);
+          }
+        }
       }
     }
   }
 #pragma unroll
-  for (int t = 0; t < MT; ++t)
+  for (int nn = 0; nn < NT; ++nn)
 #pragma unroll
-    for (int nn = 0; nn < NT; ++nn)
-#pragma unroll
-      for (int e = 0; e < 2; ++e) {
-        const int d = (warp + 4 * t) * 16 + (lane >> 2) + e * 8, c = nn * 8 + (lane & 3) * 2;
-        if (d < dim && c < cols)
-          *reinterpret_cast<float2*>(state + static_cast<size_t>(d) * a.vdim + c) = make_float2(st[t][nn][e * 2], st[t][nn][e * 2 + 1]);
-      }
+    for (int e = 0; e < 2; ++e) {
+      const int d = m0 + (lane >> 2) + e * 8, c = nn * 8 + (lane & 3) * 2;
+      if (d < dim && c < cols) *reinterpret_cast<float2*>(state + static_cast<size_t>(d) * a.vdim + c) = make_float2(st[nn][e * 2], st[nn][e * 2 + 1]);
+    }
 }
 
 bool delta_args_ok(const Args& a) {
@@ -650,14 +670,14 @@ int launch_step(const Args& a, const void* gate, long long gate_stride, const fl
   return launch_status();
 }
 
-template <int MT, int NT>
+template <int NT>
 int launch_chain(const Args& a, const ChunkSpace& ws, cudaStream_t st) {
   constexpr int kCols = NT * 8, kPitchC = kCols + 8;
-  auto kern = delta_chain_kernel<MT, NT>;
-  const size_t smem = (static_cast<size_t>(4) * kChunk * (a.dim + 8) + static_cast<size_t>(2) * (a.dim + 2 * kChunk) * kPitchC) * 2 + 2 * kChunk * 16;
+  auto kern = delta_chain_kernel<NT>;
+  const size_t smem = (static_cast<size_t>(4) * kChunk * (a.dim + 8) + static_cast<size_t>(2) * (a.dim + 3 * kChunk) * kPitchC) * 2 + 2 * kChunk * 16;
   const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
   if (e != cudaSuccess) return static_cast<int>(e);
-  kern<<<dim3(a.segments, a.heads, (a.vdim + kCols - 1) / kCols), 128, smem, st>>>(a, ws);
+  kern<<<dim3(a.segments, a.heads, (a.vdim + kCols - 1) / kCols), kChainThreads, smem, st>>>(a, ws);
   return launch_status();
 }
 
@@ -711,7 +731,7 @@ extern "C" int cacheir_b200_delta_chunked(const cacheir_b200_delta_args* args, v
   ws.tiles = static_cast<uint4*>(workspace);
   ws.rows = reinterpret_cast<float4*>(ws.tiles + units * 2 * kTri * 64);
   cudaStream_t st = as_stream(stream);
-  const size_t smem = static_cast<size_t>(2) * kChunk * (a.dim + 8) * 2 + (static_cast<size_t>(2) * kChunk * (kChunk + 1) + 32 * 33) * 4;
+  const size_t smem = static_cast<size_t>(2) * kChunk * (a.dim + 8) * 2 + (static_cast<size_t>(2) * kChunk * (kChunk + 4) + 32 * 36) * 4;
   const cudaError_t e = cudaFuncSetAttribute(delta_local_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
   if (e != cudaSuccess) return static_cast<int>(e);
   delta_local_kernel<<<dim3(items, a.heads), 128, smem, st>>>(a, ws);
@@ -719,8 +739,7 @@ extern "C" int cacheir_b200_delta_chunked(const cacheir_b200_delta_args* args, v
   if (rc != 0) return rc;
   // narrow column blocks while all of them still run at once
   const bool narrow = static_cast<long long>(a.segments) * a.heads * ((a.vdim + 15) / 16) <= kNumSMs;
-  if (a.dim <= 64) return narrow ? launch_chain<1, 2>(a, ws, st) : launch_chain<1, 4>(a, ws, st);
-  return narrow ? launch_chain<2, 2>(a, ws, st) : launch_chain<2, 4>(a, ws, st);
+  return narrow ? launch_chain<2>(a, ws, st) : launch_chain<4>(a, ws, st);
 }
 
 extern "C" int cacheir_b200_delta_device_status(int) { return 0; }

@@ -363,9 +363,9 @@ gated_rms_kernel(const T* __restrict__ o, const T* __restrict__ gate, long long 
   }
 }
 
-// A unit is one part of one row; WARPS warps share it.
+// A unit is one part of one row; WARPS warps share it (one: eight units per block).
 template <typename T, int VEC, int WARPS>
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(WARPS == 1 ? 256 : WARPS * 32)
 gated_parts_rms_kernel(const T* __restrict__ o, const T* __restrict__ gate, long long gate_stride, const float* __restrict__ w, int shared_weight,
                        int gate_first, float eps, T* __restrict__ out, int units, int parts, int size) {
   __shared__ float scratch[32];
@@ -377,7 +377,7 @@ gated_parts_rms_kernel(const T* __restrict__ o, const T* __restrict__ gate, long
   const T* g = gate + static_cast<size_t>(row) * gate_stride + static_cast<size_t>(part) * size;
   const float* weight = w + (shared_weight ? 0 : static_cast<size_t>(part) * size);
   T* dst = out + static_cast<size_t>(unit) * size;
-  constexpr int kStep = 32 * WARPS * VEC, N = 4;         // pieces that stay in registers, everything requested before the sum
+  constexpr int kStep = 32 * WARPS * VEC, N = 4;      // pieces that stay in registers, requested before the sum
   auto total = [&](float ss) { return WARPS == 1 ? warp_sum(ss) : block_sum_all(ss, scratch); };
   auto gated = [&](float (&x)[VEC], const float (&gt)[VEC], float& ss) {
 #pragma unroll
@@ -392,14 +392,13 @@ gated_parts_rms_kernel(const T* __restrict__ o, const T* __restrict__ gate, long
   };
   float ss = 0.f;
   if (size <= kStep * N) {
-    float x[N][VEC], gt[N][VEC], wv[N][VEC];
+    float x[N][VEC], gt[N][VEC];
 #pragma unroll
     for (int k = 0; k < N; ++k) {
       const int c = k * kStep + at * VEC;
       if (c < size) {
         load_vec<T, VEC>(src + c, x[k]);
         load_vec<T, VEC>(g + c, gt[k]);
-        load_vec<float, VEC>(weight + c, wv[k]);
       }
     }
 #pragma unroll
@@ -410,7 +409,9 @@ gated_parts_rms_kernel(const T* __restrict__ o, const T* __restrict__ gate, long
     for (int k = 0; k < N; ++k) {
       const int c = k * kStep + at * VEC;
       if (c < size) {
-        finish(x[k], gt[k], wv[k], inv);
+        float wv[VEC];
+        load_vec<float, VEC>(weight + c, wv);
+        finish(x[k], gt[k], wv, inv);
         store_vec<T, VEC>(dst + c, x[k]);
       }
     }
@@ -717,15 +718,15 @@ extern "C" int cacheir_b200_gated_parts_rms(const void* o, const void* gate, lon
   if (!o || !gate || !w || !out || parts <= 0 || cols % parts != 0) return CACHEIR_B200_EINVAL;
   const int size = cols / parts, units = rows * parts, quad = 4 * (dtype == CACHEIR_B200_F32 ? 4 : 2);
   const bool vec = size % 4 == 0 && gate_stride % 4 == 0 && aligned_to(o, quad) && aligned_to(gate, quad) && aligned_to(w, 16) && aligned_to(out, quad);
-  const bool wide = size > 512;
 #define CB200_PARTS(VEC, WARPS)                                                                                                         \
-  gated_parts_rms_kernel<T, VEC, WARPS><<<WARPS == 1 ? (units + 7) / 8 : units, 256, 0, as_stream(stream)>>>(                             \
+  gated_parts_rms_kernel<T, VEC, WARPS><<<WARPS == 1 ? (units + 7) / 8 : units, WARPS == 1 ? 256 : WARPS * 32, 0, as_stream(stream)>>>(                             \
       static_cast<const T*>(o), static_cast<const T*>(gate), gate_stride, w, shared_weight, gate_first, eps, static_cast<T*>(out), units, parts, size)
   CB200_HYBRID_DTYPE(dtype, {
-    if (vec && wide) CB200_PARTS(4, 8);
-    else if (vec) CB200_PARTS(4, 1);
-    else if (wide) CB200_PARTS(1, 8);
-    else CB200_PARTS(1, 1);
+    if (vec && size <= 512) CB200_PARTS(4, 1);
+    else if (vec && size <= 1024) CB200_PARTS(4, 2);
+    else if (vec) CB200_PARTS(4, 8);
+    else if (size <= 512) CB200_PARTS(1, 1);
+    else CB200_PARTS(1, 8);
   });
 #undef CB200_PARTS
   return launch_status();

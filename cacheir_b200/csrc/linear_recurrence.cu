@@ -8,7 +8,8 @@
 // chunked  prompts, bf16 operands on the tensor cores, 64 tokens at a time. With D_ij = decay^(i-j) for j <= i:
 //            O = diag(decay^(i+1)) Q S + ((Q K^T) o D) V        S' = decay^n S + K^T diag(decay^(n-1-j)) V
 //          The state stays in float32 registers; whatever is float32 by nature and has to enter an MMA (the state, the
-//          decayed scores, the decayed values) goes in as a sum of two bf16 numbers. Sequences are cut into pieces of
+//          decayed scores, the decayed values) goes in as a sum of two bf16 numbers. With many heads a CTA runs through its whole
+//          sequence, the next chunk's inputs travelling ahead; with few, sequences are cut into pieces of
 //          64 to 256 tokens that run in parallel: a first pass finds every piece's own contribution, a scan turns these into the
 //          pieces' initial states, and the main pass starts from them. GATED: with c the running sum of log decays in a
 //          chunk, decay^(i-j) becomes exp(c_i - c_j + log take_j), and so on; n rides with the first value columns.
@@ -25,8 +26,7 @@ namespace {
 constexpr int kPowers = 65;
 constexpr int kChunk = 64;
 constexpr int kPiece = 256;        // tokens of a piece at most, and of a step that is not cut
-constexpr int kCols = 64;          // value columns per CTA of the chunked form
-constexpr int kPitchV = kCols + 8; // bf16 elements per shared-memory row (16 bytes over a multiple of 128: conflict-free)
+constexpr int kWide = 8, kNarrow = 4;      // 8-column tiles of the values per CTA of the chunked form: in pieces, whole sequences
 
 using Args = cacheir_b200_recurrence_args;
 
@@ -185,18 +185,21 @@ PieceSpace piece_space(const Args& a, float* ws, int items) {
   return {ws, n, n + static_cast<size_t>(items) * a.heads * a.dim};
 }
 
-// MT = 16-row state tiles per warp (dim <= 64 MT)
-template <int MT, bool LOCAL, bool GATED>
+// MT = 16-row state tiles per warp (dim <= 64 MT), NC = 8-column tiles. AHEAD: two buffers of inputs, the next chunk's travel while
+// this one's products run.
+template <int MT, int NC, bool LOCAL, bool GATED, bool AHEAD>
 __global__ void __launch_bounds__(128)
 recurrence_chunk_kernel(const Args a, const PieceSpace ws, int piece_rows) {
+  constexpr int kCols = NC * 8, kPitchV = kCols + 8;      // (rows 16 bytes over a multiple of 32: conflict-free)
+  constexpr int kBuffers = AHEAD ? 2 : 1;
   extern __shared__ __align__(16) uint8_t raw[];
   const int dim = a.dim;
   const int pitch = dim + 8;
-  __nv_bfloat16* s_q = reinterpret_cast<__nv_bfloat16*>(raw);        // [64][pitch]
-  __nv_bfloat16* s_k = s_q + kChunk * pitch;                         // [64][pitch]
-  __nv_bfloat16* s_v = s_k + kChunk * pitch;                         // [64][72]
-  __nv_bfloat16* s_dv = s_v + kChunk * kPitchV;                      // [2][64][72] decayed values, hi | lo
-  __nv_bfloat16* s_s = s_dv + 2 * kChunk * kPitchV;                  // [2][dim][72] state, hi | lo
+  __nv_bfloat16* q_bufs = reinterpret_cast<__nv_bfloat16*>(raw);     // [buffers][64][pitch]
+  __nv_bfloat16* k_bufs = q_bufs + kBuffers * kChunk * pitch;        // [buffers][64][pitch]
+  __nv_bfloat16* v_bufs = k_bufs + kBuffers * kChunk * pitch;        // [buffers][64][kPitchV]
+  __nv_bfloat16* s_dv = v_bufs + kBuffers * kChunk * kPitchV;        // [2][64][kPitchV] decayed values, hi | lo
+  __nv_bfloat16* s_s = s_dv + 2 * kChunk * kPitchV;                  // [2][dim][kPitchV] state, hi | lo
   __shared__ float s_pow[kPowers];
   __shared__ float s_cum[kChunk], s_take[kChunk], s_left[kChunk];      // log decays summed, log take, weight in the chunk's last state
   __shared__ float s_n[2][128];                       // the normaliser before and after a chunk
@@ -210,7 +213,7 @@ recurrence_chunk_kernel(const Args a, const PieceSpace ws, int piece_rows) {
   if (!GATED)
     for (int i = threadIdx.x; i < kPowers; i += 128) s_pow[i] = a.decay_pow[h * kPowers + i];
 
-  float st[MT][8][4];          // state rows (warp + 4 t)*16 .. +15, columns v0 .. v0+63
+  float st[MT][NC][4];         // state rows (warp + 4 t)*16 .. +15, columns v0 .. v0 + kCols - 1
   float* state = slot_state(a, it.seg, h);
   float* piece = ws.state + (static_cast<size_t>(blockIdx.x) * a.heads + h) * dim * a.vdim;
   float* piece_n = ws.normaliser + (static_cast<size_t>(blockIdx.x) * a.heads + h) * dim;
@@ -226,7 +229,7 @@ recurrence_chunk_kernel(const Args a, const PieceSpace ws, int piece_rows) {
 #pragma unroll
   for (int t = 0; t < MT; ++t)
 #pragma unroll
-    for (int n = 0; n < 8; ++n)
+    for (int n = 0; n < NC; ++n)
 #pragma unroll
       for (int e = 0; e < 2; ++e) {
         const int d = (warp + 4 * t) * 16 + (lane >> 2) + e * 8, c = n * 8 + (lane & 3) * 2;
@@ -238,6 +241,12 @@ recurrence_chunk_kernel(const Args a, const PieceSpace ws, int piece_rows) {
   __syncthreads();
 
   const int kc = dim / 8;      // 16-byte pieces per q / k row
+  const int r_first = static_cast<int>(threadIdx.x) / kc, c_first = static_cast<int>(threadIdx.x) % kc, r_step = 128 / kc, c_step = 128 % kc;
+  auto next_piece = [&](int& r, int& c) {      // 128 pieces further
+    r += r_step;
+    c += c_step;
+    if (c >= kc) { c -= kc; ++r; }
+  };
   int now = 0;                 // which of s_n is the current one
   float ahead[4] = {};         // warp 0: the next chunk's log decays and log takes, two rows per lane
   auto fetch_gates = [&](int r0) {
@@ -250,9 +259,34 @@ recurrence_chunk_kernel(const Args a, const PieceSpace ws, int piece_rows) {
     }
   };
   if (GATED && warp == 0) fetch_gates(0);
+  // AHEAD: a chunk's inputs, asynchronously; a thread copies the values that it decays
+  auto fetch = [&](int r0) {
+    const int buf = (r0 / kChunk) & 1, n = min(kChunk, it.count - r0);
+    const size_t base = static_cast<size_t>(it.row0 + r0);
+    auto copy = [&](__nv_bfloat16* dst, const void* src, size_t off, bool there) {      // (what lies behind the end is zero)
+      asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_addr(dst)), "l"(static_cast<const __nv_bfloat16*>(src) + off),
+                   "r"(there ? 16 : 0) : "memory");
+    };
+    for (int r = r_first, c = c_first; r < kChunk; next_piece(r, c)) {
+      const size_t off = (base + min(r, n - 1)) * a.stride + static_cast<size_t>(kh) * dim + c * 8;
+      copy(q_bufs + (buf * kChunk + r) * pitch + c * 8, a.q, off, r < n);
+      copy(k_bufs + (buf * kChunk + r) * pitch + c * 8, a.k, off, r < n);
+    }
+    for (int i = threadIdx.x; i < kChunk * NC; i += 128) {
+      const int r = i / NC, c = i % NC;
+      const bool there = r < n && c * 8 < cols;
+      copy(v_bufs + (buf * kChunk + r) * kPitchV + c * 8, a.v, (base + min(r, n - 1)) * a.stride + static_cast<size_t>(h) * a.vdim + v0 + (there ? c * 8 : 0), there);
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  if (AHEAD) fetch(0);
   for (int r0 = 0; r0 < it.count; r0 += kChunk) {
     const int n = min(kChunk, it.count - r0);
     const size_t base = static_cast<size_t>(it.row0 + r0);
+    const int buf = AHEAD ? (r0 / kChunk) & 1 : 0;
+    __nv_bfloat16* s_q = q_bufs + buf * kChunk * pitch;
+    __nv_bfloat16* s_k = k_bufs + buf * kChunk * pitch;
+    __nv_bfloat16* s_v = v_bufs + buf * kChunk * kPitchV;
     if (GATED) {
       if (warp == 0) {
         float c[2], take[2], last = 0.f;
@@ -279,8 +313,8 @@ recurrence_chunk_kernel(const Args a, const PieceSpace ws, int piece_rows) {
       }
       __syncthreads();
     }
-    for (int i = threadIdx.x; i < kChunk * kc; i += 128) {
-      const int r = i / kc, c = i % kc;
+    if (AHEAD) asm volatile("cp.async.wait_group 0;" ::: "memory");
+    for (int r = AHEAD ? kChunk : r_first, c = c_first; r < kChunk; next_piece(r, c)) {
       uint4 q = make_uint4(0u, 0u, 0u, 0u), k = q;
       if (r < n) {
         const size_t off = (base + r) * a.stride + static_cast<size_t>(kh) * dim + c * 8;
@@ -290,12 +324,13 @@ recurrence_chunk_kernel(const Args a, const PieceSpace ws, int piece_rows) {
       if (!LOCAL) *reinterpret_cast<uint4*>(s_q + r * pitch + c * 8) = q;
       *reinterpret_cast<uint4*>(s_k + r * pitch + c * 8) = k;
     }
-    for (int i = threadIdx.x; i < kChunk * (kCols / 8); i += 128) {
-      const int r = i / (kCols / 8), c = i % (kCols / 8);
+    for (int i = threadIdx.x; i < kChunk * NC; i += 128) {
+      const int r = i / NC, c = i % NC;
       uint4 v = make_uint4(0u, 0u, 0u, 0u);
-      if (r < n && c * 8 < cols)
+      if (AHEAD) v = *reinterpret_cast<const uint4*>(s_v + r * kPitchV + c * 8);
+      else if (r < n && c * 8 < cols)
         v = *reinterpret_cast<const uint4*>(static_cast<const __nv_bfloat16*>(a.v) + (base + r) * a.stride + static_cast<size_t>(h) * a.vdim + v0 + c * 8);
-      if (!LOCAL) *reinterpret_cast<uint4*>(s_v + r * kPitchV + c * 8) = v;
+      if (!LOCAL && !AHEAD) *reinterpret_cast<uint4*>(s_v + r * kPitchV + c * 8) = v;
       const float f = GATED ? s_left[r] : s_pow[max(n - 1 - r, 0)];
       const uint32_t* w = reinterpret_cast<const uint32_t*>(&v);
       uint4 hi, lo;
@@ -316,7 +351,7 @@ recurrence_chunk_kernel(const Args a, const PieceSpace ws, int piece_rows) {
 #pragma unroll
       for (int t = 0; t < MT; ++t)
 #pragma unroll
-        for (int nn = 0; nn < 8; ++nn)
+        for (int nn = 0; nn < NC; ++nn)
 #pragma unroll
           for (int e = 0; e < 2; ++e) {
             const int d = (warp + 4 * t) * 16 + (lane >> 2) + e * 8, c = nn * 8 + (lane & 3) * 2;
@@ -330,11 +365,12 @@ recurrence_chunk_kernel(const Args a, const PieceSpace ws, int piece_rows) {
           }
     }
     __syncthreads();
+    if (AHEAD && r0 + kChunk < it.count) fetch(r0 + kChunk);
 
     if (!LOCAL && warp * 16 < n) {
-      float o[8][4];
+      float o[NC][4];
 #pragma unroll
-      for (int nn = 0; nn < 8; ++nn)
+      for (int nn = 0; nn < NC; ++nn)
 #pragma unroll
         for (int e = 0; e < 4; ++e) o[nn][e] = 0.f;
       float sc[8][4];
@@ -360,7 +396,7 @@ recurrence_chunk_kernel(const Args a, const PieceSpace ws, int piece_rows) {
 #pragma unroll
         for (int part = 0; part < 2; ++part)
 #pragma unroll
-          for (int nn = 0; nn < 8; nn += 2) {
+          for (int nn = 0; nn < NC; nn += 2) {
             uint32_t bf[4];
             ldsm_x4_t(sa + ((part * dim + k * 16) * kPitchV + nn * 8) * 2, bf);
             mma_bf16(o[nn], af, bf[0], bf[1]);
@@ -379,7 +415,7 @@ recurrence_chunk_kernel(const Args a, const PieceSpace ws, int piece_rows) {
         nq[1] *= f1;
       }
 #pragma unroll
-      for (int nn = 0; nn < 8; ++nn) {
+      for (int nn = 0; nn < NC; ++nn) {
         o[nn][0] *= f0; o[nn][1] *= f0; o[nn][2] *= f1; o[nn][3] *= f1;
       }
       const uint32_t va = smem_addr(s_v) + (((lane & 7) + ((lane >> 3) & 1) * 8) * kPitchV + (lane >> 4) * 8) * 2;
@@ -408,7 +444,7 @@ recurrence_chunk_kernel(const Args a, const PieceSpace ws, int piece_rows) {
             lo[u * 2 + e] = pack_bf16(l0, l1);
           }
 #pragma unroll
-        for (int nn = 0; nn < 8; nn += 2) {
+        for (int nn = 0; nn < NC; nn += 2) {
           uint32_t bf[4];
           ldsm_x4_t(va + (kk * 16 * kPitchV + nn * 8) * 2, bf);
           mma_bf16(o[nn], hi, bf[0], bf[1]);
@@ -428,7 +464,7 @@ recurrence_chunk_kernel(const Args a, const PieceSpace ws, int piece_rows) {
         }
         if (i < n && a.skip) {
 #pragma unroll
-          for (int nn = 0; nn < 8; ++nn) {
+          for (int nn = 0; nn < NC; ++nn) {
             const uint32_t v2 = *reinterpret_cast<const uint32_t*>(s_v + i * kPitchV + nn * 8 + (lane & 3) * 2);
             o[nn][e * 2] = fmaf(skip, __uint_as_float(v2 << 16), o[nn][e * 2]);
             o[nn][e * 2 + 1] = fmaf(skip, __uint_as_float(v2 & 0xffff0000u), o[nn][e * 2 + 1]);
@@ -437,7 +473,7 @@ recurrence_chunk_kernel(const Args a, const PieceSpace ws, int piece_rows) {
         if (i < n) {
           __nv_bfloat16* dst = out + ((base + i) * a.heads + h) * a.vdim + v0;
 #pragma unroll
-          for (int nn = 0; nn < 8; ++nn) {
+          for (int nn = 0; nn < NC; ++nn) {
             const int c = nn * 8 + (lane & 3) * 2;
             if (c < cols) *reinterpret_cast<uint32_t*>(dst + c) = pack_bf16(o[nn][e * 2], o[nn][e * 2 + 1]);
           }
@@ -455,7 +491,7 @@ recurrence_chunk_kernel(const Args a, const PieceSpace ws, int piece_rows) {
       const int m0 = (warp + 4 * t) * 16;
       if (m0 >= dim) continue;
 #pragma unroll
-      for (int nn = 0; nn < 8; ++nn)
+      for (int nn = 0; nn < NC; ++nn)
 #pragma unroll
         for (int e = 0; e < 4; ++e) st[t][nn][e] *= fn;
 #pragma unroll
@@ -465,7 +501,7 @@ recurrence_chunk_kernel(const Args a, const PieceSpace ws, int piece_rows) {
 #pragma unroll
         for (int part = 0; part < 2; ++part)
 #pragma unroll
-          for (int nn = 0; nn < 8; nn += 2) {
+          for (int nn = 0; nn < NC; nn += 2) {
             uint32_t bf[4];
             ldsm_x4_t(dv + ((part * kChunk + k * 16) * kPitchV + nn * 8) * 2, bf);
             mma_bf16(st[t][nn], af, bf[0], bf[1]);
@@ -495,7 +531,7 @@ recurrence_chunk_kernel(const Args a, const PieceSpace ws, int piece_rows) {
 #pragma unroll
     for (int t = 0; t < MT; ++t)
 #pragma unroll
-      for (int n = 0; n < 8; ++n)
+      for (int n = 0; n < NC; ++n)
 #pragma unroll
         for (int e = 0; e < 2; ++e) {
           const int d = (warp + 4 * t) * 16 + (lane >> 2) + e * 8, c = n * 8 + (lane & 3) * 2;
@@ -873,39 +909,48 @@ bool memory_slots_ok(const Args& a) {        // normalisers and maxima behind th
   return a.slot_stride >= static_cast<long long>(a.heads) * a.dim * a.vdim + static_cast<long long>(a.heads) * (a.dim + 1);
 }
 
-size_t chunk_smem(int dim) {
-  return (static_cast<size_t>(2) * kChunk * (dim + 8) + static_cast<size_t>(3) * kChunk * kPitchV + static_cast<size_t>(2) * dim * kPitchV) * 2;
+size_t chunk_smem(int dim, int tiles, bool ahead) {
+  const int buffers = ahead ? 2 : 1, pitch_v = tiles * 8 + 8;
+  return (static_cast<size_t>(2) * buffers * kChunk * (dim + 8) + static_cast<size_t>(buffers + 2) * kChunk * pitch_v + static_cast<size_t>(2) * dim * pitch_v) * 2;
 }
+
+// Heads and value columns alone keep the machine busy (two CTAs on most SMs): every sequence in one go.
+bool whole_sequences(int heads, int vdim) { return static_cast<long long>(heads) * ((vdim + 8 * kNarrow - 1) / (8 * kNarrow)) >= kNumSMs * 3 / 2; }
 
 // Shorter pieces while all of them still run at once.
 int choose_piece(int rows, int segments, int heads, int vdim) {
   int piece = kPiece;
-  const long long per_item = static_cast<long long>(heads) * ((vdim + kCols - 1) / kCols);
+  const long long per_item = static_cast<long long>(heads) * ((vdim + 8 * kWide - 1) / (8 * kWide));
   while (rows > kPiece && piece > kChunk && per_item * ragged_items(rows, segments, piece / 2) <= 2 * kNumSMs) piece /= 2;
   return piece;
 }
 
-template <int MT, bool LOCAL, bool GATED>
+template <int MT, int NC, bool LOCAL, bool GATED, bool AHEAD>
 int launch_chunk(const Args& a, const PieceSpace& ws, int piece, cudaStream_t st) {
-  auto kern = recurrence_chunk_kernel<MT, LOCAL, GATED>;
-  const size_t smem = chunk_smem(a.dim);
+  auto kern = recurrence_chunk_kernel<MT, NC, LOCAL, GATED, AHEAD>;
+  const size_t smem = chunk_smem(a.dim, NC, AHEAD);
   cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
   if (e != cudaSuccess) return static_cast<int>(e);
-  kern<<<dim3(ragged_items(a.rows, a.segments, piece), a.heads, (a.vdim + kCols - 1) / kCols), 128, smem, st>>>(a, ws, piece);
+  kern<<<dim3(ragged_items(a.rows, a.segments, piece), a.heads, (a.vdim + NC * 8 - 1) / (NC * 8)), 128, smem, st>>>(a, ws, piece);
   return launch_status();
 }
 
 template <bool GATED>
 int launch_passes(const Args& a, float* workspace, bool pieces, cudaStream_t st) {
+  if (whole_sequences(a.heads, a.vdim)) {
+    constexpr int kAll = 1 << 30;
+    const PieceSpace none{};
+    return a.dim <= 64 ? launch_chunk<1, kNarrow, false, GATED, true>(a, none, kAll, st) : launch_chunk<2, kNarrow, false, GATED, true>(a, none, kAll, st);
+  }
   const int piece = choose_piece(a.rows, a.segments, a.heads, a.vdim);
   const PieceSpace ws = piece_space(a, workspace, ragged_items(a.rows, a.segments, piece));
   if (pieces) {
-    const int rc = a.dim <= 64 ? launch_chunk<1, true, GATED>(a, ws, piece, st) : launch_chunk<2, true, GATED>(a, ws, piece, st);
+    const int rc = a.dim <= 64 ? launch_chunk<1, kWide, true, GATED, false>(a, ws, piece, st) : launch_chunk<2, kWide, true, GATED, false>(a, ws, piece, st);
     if (rc != 0) return rc;
     const int z = (a.dim * a.vdim + 1023) / 1024;
     recurrence_scan_kernel<GATED><<<dim3(a.segments, a.heads, z), 256, 0, st>>>(a, ws, piece);
   }
-  return a.dim <= 64 ? launch_chunk<1, false, GATED>(a, ws, piece, st) : launch_chunk<2, false, GATED>(a, ws, piece, st);
+  return a.dim <= 64 ? launch_chunk<1, kWide, false, GATED, false>(a, ws, piece, st) : launch_chunk<2, kWide, false, GATED, false>(a, ws, piece, st);
 }
 
 template <typename T, bool GATED>
@@ -955,7 +1000,7 @@ extern "C" int cacheir_b200_recurrence_chunked_supported(int dim, int vdim, int 
 }
 
 extern "C" size_t cacheir_b200_recurrence_workspace_bytes(int rows, int segments, int heads, int dim, int vdim) {
-  if (rows <= kPiece) return 0;
+  if (rows <= kPiece || whole_sequences(heads, vdim)) return 0;
   return static_cast<size_t>(ragged_items(rows, segments, choose_piece(rows, segments, heads, vdim))) * heads * (static_cast<size_t>(dim) * (vdim + 1) + 1) * 4;
 }
 

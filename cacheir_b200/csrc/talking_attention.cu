@@ -4,9 +4,10 @@
 //           is one product of a whole cached key row with a query that holds, per key/value head, sum_g talk[h, g] q_g.
 // simple    any extents, float32 arithmetic: one CTA per row, all heads.
 // step      one CTA per (sequence, split, set of key/value heads). Tiles of 16 or 32 cached tokens land in a ring as TMA boxes of 64
-//           columns. Eight warps: raw scores of all heads with warp MMAs (the heads of a key/value head being the 16-row operand),
-//           their mixture and the running softmax in float32, then the values of the set's heads. Splits meet in distributed shared
-//           memory. Sets read all keys and their own values; there is one unless the output would not fit the registers.
+//           columns. Eight warps with warp MMAs: raw scores of all heads (up to 16 heads of a key/value head, a band, being the 16-row
+//           operand) go to shared memory as sums of two bf16 numbers; then a band's warp has its mixed scores as one more product,
+//           its softmax and its values in registers. One barrier per tile. Splits meet in distributed shared memory. Sets read all
+//           keys and their own values; there is one unless the output would not fit the registers.
 #include "talking_attention.cuh"
 
 namespace cb200 {
@@ -56,7 +57,7 @@ talking_prepare_kernel(const PrepareParams p, const T* __restrict__ q, const T* 
       const T* src = q + static_cast<size_t>(row) * p.q_stride + static_cast<size_t>(u) * a.dim;
       for (int c = lane; c < a.dim; c += 32) {
         const float x = rotated(src, c, half, cs);
-        if (MIXED > 0) sm[u * a.dim + c] = x;
+        if (MIXED > 0) sm[u * a.dim + c] = a.scale < 0.f ? -x : x;
         else Elem<T>::st(q_out + (static_cast<size_t>(row) * a.heads + u) * a.dim + c, x);
       }
     } else if (!cached) {
@@ -199,12 +200,14 @@ constexpr int kConsumers = kWarps * 32;
 constexpr int kStepThreads = kConsumers + 32;
 constexpr int kMaxStages = 6;
 constexpr int kMaxSplits = 8;                    // CTAs of a cluster
-constexpr int kMaxUnits = 16;                    // 16 x 16 output tiles per warp
+constexpr int kMaxTiles = 16;                    // 16 x 16 output tiles per warp
 
 struct StepShape {
   int sets, tile, stages;                        // sets of key/value heads, cached tokens per tile
   int k_boxes, v_boxes;
-  int kv_per_set, units;                         // key/value heads of a set at most; output tiles per warp
+  int bands;                                     // of a set at most: a band is up to 16 heads of one key/value head
+  int shares;                                    // warps that share a band's value columns
+  int bands_per_warp, pairs_per_warp;            // pairs of 8-column tiles
   size_t ring, smem;
 };
 struct StepParams {
@@ -216,11 +219,22 @@ struct StepParams {
 };
 
 __host__ __device__ inline int round_to(int n, int m) { return (n + m - 1) / m * m; }
-// floats of the parts behind the ring: talk [set's heads][heads], raw scores [heads][tile], (m, l, factor) [set's heads]
-__host__ __device__ inline int step_floats(int set_heads, int heads, int tile) {
-  const int h4 = round_to(heads, 4);
-  return round_to(set_heads, 4) * h4 + h4 * (tile + 1) + 3 * round_to(set_heads, 4);
-}
+// Parts behind the ring, in bytes: barriers; talk [bands][16][heads], scores [2][hi, lo][heads][tile], queries [heads][dim] as bf16
+// with rows 16 bytes over a multiple of 16 entries; reference and sum of a set's heads.
+struct StepSpace {
+  int talk_pitch, score_pitch, q_pitch, talk, scores, q, meet, total;
+  __host__ __device__ StepSpace(int heads, int dim, int bands, int set_heads, int tile) {
+    const int h16 = round_to(heads, 16);
+    talk_pitch = h16 + 8;
+    score_pitch = tile + 8;
+    q_pitch = round_to(dim, 16) + 8;
+    talk = 2 * kMaxStages * 8;
+    scores = talk + bands * 16 * talk_pitch * 2;
+    q = scores + 4 * h16 * score_pitch * 2;
+    meet = q + heads * q_pitch * 2;
+    total = meet + 2 * round_to(set_heads, 4) * 4;
+  }
+};
 
 __device__ __forceinline__ float ld_peer_f32(const float* local, uint32_t rank) {
   uint32_t remote;
@@ -235,28 +249,29 @@ __device__ __forceinline__ void cluster_sync_all() {
 }
 __device__ __forceinline__ void consumers_sync() { asm volatile("barrier.cta.sync 1, %0;" ::"n"(kConsumers) : "memory"); }
 
-template <int UNITS, int TILE>
+// BANDS, PAIRS: what a warp has of the output at most
+template <int BANDS, int PAIRS, int TILE>
 __global__ void __launch_bounds__(kStepThreads, 1)
 talking_step_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_constant__ CUtensorMap tmap_v, const StepParams p) {
-  constexpr int kBox = TILE * 128;
-  constexpr int kPitchP = TILE + 8;
+  constexpr int kBox = TILE * 128, kBlocks = TILE / 16;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~static_cast<uintptr_t>(1023));
   const Args& a = p.a;
   const int group = a.heads / a.kv_heads, subs = (group + 15) / 16;
   const int split = blockIdx.x, seg = blockIdx.z;          // (the cluster spans the whole x extent)
   const int kv0 = a.kv_heads * static_cast<int>(blockIdx.y) / p.s.sets, kv1 = a.kv_heads * (static_cast<int>(blockIdx.y) + 1) / p.s.sets;
-  const int head0 = kv0 * group, set_heads = (kv1 - kv0) * group, h4 = round_to(a.heads, 4);
-  const int stage_bytes = (p.s.k_boxes + p.s.v_boxes) * kBox, q_pitch = round_to(a.dim, 16) + 8;
-  uint64_t* full = reinterpret_cast<uint64_t*>(smem + p.s.ring);
+  const int head0 = kv0 * group, set_heads = (kv1 - kv0) * group, bands = (kv1 - kv0) * subs, h16 = round_to(a.heads, 16);
+  const int stage_bytes = (p.s.k_boxes + p.s.v_boxes) * kBox;
+  const StepSpace space(a.heads, a.dim, p.s.bands, p.s.bands / subs * group, TILE);
+  uint8_t* rest = smem + p.s.ring;
+  uint64_t* full = reinterpret_cast<uint64_t*>(rest);
   uint64_t* empty = full + kMaxStages;
-  float* s_talk = reinterpret_cast<float*>(empty + kMaxStages);                       // [set_heads][h4]
-  float* s_rawscore = s_talk + round_to(p.s.kv_per_set * group, 4) * h4;              // [h4][TILE + 1]
-  float* s_m = s_rawscore + h4 * (TILE + 1);                                          // [set_heads], likewise behind it
-  float* s_l = s_m + round_to(p.s.kv_per_set * group, 4);
-  float* s_f = s_l + round_to(p.s.kv_per_set * group, 4);
-  __nv_bfloat16* s_q = reinterpret_cast<__nv_bfloat16*>(s_f + round_to(p.s.kv_per_set * group, 4));      // [heads][q_pitch]
-  __nv_bfloat16* s_p = s_q + round_to(a.heads * q_pitch, 8);                          // [set_heads][kPitchP]
+  __nv_bfloat16* s_talk = reinterpret_cast<__nv_bfloat16*>(rest + space.talk);
+  __nv_bfloat16* s_score = reinterpret_cast<__nv_bfloat16*>(rest + space.scores);
+  __nv_bfloat16* s_q = reinterpret_cast<__nv_bfloat16*>(rest + space.q);
+  float* s_m = reinterpret_cast<float*>(rest + space.meet);
+  float* s_l = s_m + round_to(p.s.bands / subs * group, 4);
+  const int plane = h16 * space.score_pitch;               // of s_score: [buffer][hi, lo]
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   if (a.row_seg[seg] < 0) return;                          // (a padding row: the whole cluster leaves)
@@ -268,48 +283,60 @@ talking_step_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_con
     for (int s = 0; s < p.s.stages; ++s) { ptx::mbar_init(smem_addr(&full[s]), 1); ptx::mbar_init(smem_addr(&empty[s]), kWarps); }
     ptx::mbar_fence_init();
   }
-  for (int i = threadIdx.x; i < a.heads * q_pitch; i += kStepThreads) {
-    const int h = i / q_pitch, c = i % q_pitch;
-    s_q[i] = c < a.dim ? p.q[(static_cast<size_t>(seg) * a.heads + h) * a.dim + c] : __float2bfloat16_rn(0.f);
-  }
-  for (int i = threadIdx.x; i < set_heads * h4; i += kStepThreads) {
-    const int h = i / h4, g = i % h4;
-    s_talk[i] = g < a.heads ? a.talk[static_cast<size_t>(head0 + h) * a.heads + g] * kTalkLog2e : 0.f;
-  }
-  for (int i = threadIdx.x; i < h4 * (TILE + 1); i += kStepThreads) s_rawscore[i] = 0.f;
-  for (int i = threadIdx.x; i < set_heads; i += kStepThreads) { s_m[i] = -1e30f; s_l[i] = 0.f; }
   __syncthreads();
 
-  const int pairs = (a.vdim + 15) / 16, all_units = (kv1 - kv0) * subs * pairs;
-  float o[UNITS][2][4];
+  const int g4 = lane >> 2, t4 = lane & 3, lrow = lane & 7, lmat = lane >> 3;
+  const int pairs = (a.vdim + 15) / 16, share = warp % p.s.shares, band0 = warp / p.s.shares;
+  float o[BANDS][PAIRS][2][4], m_run[BANDS][2], l_run[BANDS][2];
 #pragma unroll
-  for (int i = 0; i < UNITS; ++i)
+  for (int i = 0; i < BANDS; ++i) {
+    m_run[i][0] = m_run[i][1] = -1e30f;
+    l_run[i][0] = l_run[i][1] = 0.f;
 #pragma unroll
-    for (int t = 0; t < 2; ++t)
+    for (int j = 0; j < PAIRS; ++j)
 #pragma unroll
-      for (int e = 0; e < 4; ++e) o[i][t][e] = 0.f;
+      for (int t = 0; t < 2; ++t)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) o[i][j][t][e] = 0.f;
+  }
 
   if (warp == kWarps) {
-    // ---------------- copies ----------------
+    // ---------------- copies: a lane per box ----------------
+    const int boxes = p.s.k_boxes + p.s.v_boxes;
     int issued = 0;
-    if (lane == 0) {
-      for (int it = 0; it < n; ++it) {
-        const int s = it % p.s.stages, key0 = (tile_lo + begin + it) * TILE;
-        if (it >= p.s.stages && !ptx::mbar_wait(smem_addr(&empty[s]), ((it / p.s.stages) & 1) ^ 1, &g_talking_status, (10 << 8) | 1)) break;
-        const uint32_t bar = smem_addr(&full[s]), dst = smem_addr(smem + s * stage_bytes);
-        const int row = talk_slot(a, seg, key0 / kTalkPage) * kTalkPage + key0 % kTalkPage;
-        ptx::mbar_expect_tx(bar, stage_bytes);
-        for (int b = 0; b < p.s.k_boxes; ++b) ptx::tma_load_2d(dst + b * kBox, &tmap_k, bar, b * 64, row);
-        for (int b = 0; b < p.s.v_boxes; ++b) ptx::tma_load_2d(dst + (p.s.k_boxes + b) * kBox, &tmap_v, bar, kv0 * a.vdim + b * 64, row);
-        issued = it + 1;
+    bool ok = true;
+    for (int it = 0; it < n && ok; ++it) {
+      const int s = it % p.s.stages, key0 = (tile_lo + begin + it) * TILE;
+      if (it >= p.s.stages) ok = ptx::mbar_wait(smem_addr(&empty[s]), ((it / p.s.stages) & 1) ^ 1, &g_talking_status, (10 << 8) | 1);
+      ok = __all_sync(0xffffffffu, ok);
+      if (!ok) break;
+      const uint32_t bar = smem_addr(&full[s]), dst = smem_addr(smem + s * stage_bytes);
+      const int row = talk_slot(a, seg, key0 / kTalkPage) * kTalkPage + key0 % kTalkPage;
+      if (lane == 0) ptx::mbar_expect_tx(bar, stage_bytes);
+      __syncwarp();
+      for (int b = lane; b < boxes; b += 32) {
+        if (b < p.s.k_boxes) ptx::tma_load_2d(dst + b * kBox, &tmap_k, bar, b * 64, row);
+        else ptx::tma_load_2d(dst + b * kBox, &tmap_v, bar, kv0 * a.vdim + (b - p.s.k_boxes) * 64, row);
       }
-      if (issued < n)                    // a wait gave up: nothing may still be on its way when the block ends
-        for (int it = max(0, issued - p.s.stages); it < issued; ++it)
-          ptx::mbar_wait(smem_addr(&full[it % p.s.stages]), (it / p.s.stages) & 1, &g_talking_status, (10 << 8) | 2);
+      issued = it + 1;
     }
+    if (issued < n)                      // a wait gave up: nothing may still be on its way when the block ends
+      for (int it = max(0, issued - p.s.stages); it < issued; ++it)
+        ptx::mbar_wait(smem_addr(&full[it % p.s.stages]), (it / p.s.stages) & 1, &g_talking_status, (10 << 8) | 2);
     __syncwarp();
   } else {
-    const int g4 = lane >> 2, t4 = lane & 3, lrow = lane & 7, lmat = lane >> 3;
+    // queries and talk, while the first tiles travel
+    for (int h = warp; h < a.heads; h += kWarps)
+      for (int c = lane; c < space.q_pitch; c += 32)
+        s_q[h * space.q_pitch + c] = c < a.dim ? p.q[(static_cast<size_t>(seg) * a.heads + h) * a.dim + c] : __float2bfloat16_rn(0.f);
+    for (int r = warp; r < bands * 16; r += kWarps) {
+      const int h = (r >> 4) % subs * 16 + (r & 15), head = head0 + (r >> 4) / subs * group + h;
+      for (int g = lane; g < h16; g += 32)
+        s_talk[r * space.talk_pitch + g] = __float2bfloat16_rn(h < group && g < a.heads ? a.talk[static_cast<size_t>(head) * a.heads + g] : 0.f);
+    }
+    for (int i = threadIdx.x; i < 4 * plane; i += kConsumers) s_score[i] = __float2bfloat16_rn(0.f);      // (rows behind the last head stay zero)
+    consumers_sync();
+
     for (int it = 0; it < n; ++it) {
       const int s = it % p.s.stages, key0 = (tile_lo + begin + it) * TILE;
       // (a wait that gave up is on record; everyone goes on, so that the barriers below still meet)
@@ -318,6 +345,7 @@ talking_step_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_con
       uint8_t* k_tile = smem + s * stage_bytes;
       uint8_t* v_tile = k_tile + p.s.k_boxes * kBox;
       const uint32_t k_at = smem_addr(k_tile), v_at = smem_addr(v_tile);
+      __nv_bfloat16* score = s_score + (it & 1) * 2 * plane;
       // values behind the last token may be anything: zero, so that 0 * value stays 0
       if (key0 + TILE - 1 > pos) {
         const int valid = pos + 1 - key0;
@@ -326,104 +354,127 @@ talking_step_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_con
           *reinterpret_cast<uint4*>(v_tile + (c >> 3) * kBox + r * 128 + (c & 7) * 16) = make_uint4(0u, 0u, 0u, 0u);
         }
       }
-      // raw scores: (key/value head, 16 of its heads, 16 keys)
-      for (int u = warp; u < a.kv_heads * subs * (TILE / 16); u += kWarps) {
-        const int kb = u % (TILE / 16), sub = u / (TILE / 16) % subs, g = u / (TILE / 16) / subs;
+      // raw scores of all heads: a band and 16 keys at a time
+      for (int u = warp; u < a.kv_heads * subs * kBlocks; u += kWarps) {
+        const int kb = u % kBlocks, band = u / kBlocks, g = subs == 1 ? band : band / subs, sub = subs == 1 ? 0 : band % subs;
         const int h0 = g * group + sub * 16, count = min(16, group - sub * 16);
         float sc[2][4], sd[2][4];        // even and odd steps in sums of their own (shorter dependent chains)
 #pragma unroll
         for (int t = 0; t < 2; ++t)
 #pragma unroll
           for (int e = 0; e < 4; ++e) sc[t][e] = sd[t][e] = 0.f;
-        const uint32_t qa = smem_addr(s_q) + (min(h0 + (lane & 15), a.heads - 1) * q_pitch + (lane >> 4) * 8) * 2;
-        const int key = kb * 16 + (lmat >> 1) * 8 + lrow, last_piece = p.s.k_boxes * 8 - 1;
+        const uint32_t qa = smem_addr(s_q) + (min(h0 + (lane & 15), a.heads - 1) * space.q_pitch + (lane >> 4) * 8) * 2;
+        const int key = kb * 16 + (lmat >> 1) * 8 + lrow, last_piece = p.s.k_boxes * 8 - 1, piece0 = g * a.dim / 8 + (lmat & 1);
+        const uint32_t row_at = k_at + key * 128;
         auto step = [&](int k, float (&x)[2][4]) {
           uint32_t af[4], bf[4];
           ldsm_x4(qa + k * 32, af);
-          const int c = min(g * a.dim / 8 + 2 * k + (lmat & 1), last_piece);      // (a piece behind the head meets zero queries)
-          ldsm_x4(k_at + (c >> 3) * kBox + key * 128 + (((c & 7) ^ (key & 7)) << 4), bf);
+          const int c = min(piece0 + 2 * k, last_piece);      // (a piece behind the head meets zero queries)
+          ldsm_x4(row_at + (c >> 3) * kBox + (((c & 7) ^ lrow) << 4), bf);
           mma_bf16(x[0], af, bf[0], bf[1]);
           mma_bf16(x[1], af, bf[2], bf[3]);
         };
         const int steps = (a.dim + 15) / 16;
         int k = 0;
+#pragma unroll 2
         for (; k + 1 < steps; k += 2) { step(k, sc); step(k + 1, sd); }
         if (k < steps) step(k, sc);
 #pragma unroll
-        for (int t = 0; t < 2; ++t)
+        for (int r = 0; r < 2; ++r)
+          if (g4 + r * 8 < count)
 #pragma unroll
-          for (int e = 0; e < 4; ++e) {
-            const int r = g4 + (e >> 1) * 8;
-            if (r < count) s_rawscore[(h0 + r) * (TILE + 1) + kb * 16 + t * 8 + 2 * t4 + (e & 1)] = (sc[t][e] + sd[t][e]) * a.scale;
-          }
+            for (int t = 0; t < 2; ++t) {
+              const float x = (sc[t][2 * r] + sd[t][2 * r]) * a.scale, y = (sc[t][2 * r + 1] + sd[t][2 * r + 1]) * a.scale;
+              float xh, xl, yh, yl;
+              split_bf16(x, &xh, &xl);
+              split_bf16(y, &yh, &yl);
+              __nv_bfloat16* dst = score + (h0 + g4 + r * 8) * space.score_pitch + kb * 16 + t * 8 + 2 * t4;
+              *reinterpret_cast<uint32_t*>(dst) = pack_bf16(xh, yh);
+              *reinterpret_cast<uint32_t*>(dst + plane) = pack_bf16(xl, yl);
+            }
       }
       consumers_sync();
-      // mixture and running softmax: TILE neighbouring lanes have a head
-      {
-        constexpr int kLanes = TILE, kGroups = kConsumers / TILE, kAtOnce = 4;
-        const int j = threadIdx.x % kLanes, key = key0 + j;
-        const bool seen = key <= pos && key > pos - a.window;
-        for (int hb = threadIdx.x / kLanes; hb < set_heads; hb += kGroups * kAtOnce) {
-          float x[kAtOnce] = {};
-          for (int g = 0; g < h4; g += 4) {
-            float r[4];
 #pragma unroll
-            for (int e = 0; e < 4; ++e) r[e] = s_rawscore[(g + e) * (TILE + 1) + j];
+      for (int i = 0; i < BANDS; ++i) {
+        const int band = band0 + i * kWarps;
+        if (band >= bands) break;
+        // the band's mixed scores: talk (exact in bf16) times both halves of the raw ones
+        float x[kBlocks][2][4];
 #pragma unroll
-            for (int i = 0; i < kAtOnce; ++i) {
-              if (hb + i * kGroups < set_heads) {
-                const float4 t = *reinterpret_cast<const float4*>(s_talk + (hb + i * kGroups) * h4 + g);
-                x[i] = fmaf(t.x, r[0], fmaf(t.y, r[1], fmaf(t.z, r[2], fmaf(t.w, r[3], x[i]))));
-              }
+        for (int kb = 0; kb < kBlocks; ++kb)
+#pragma unroll
+          for (int t = 0; t < 2; ++t)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) x[kb][t][e] = 0.f;
+        const uint32_t ta = smem_addr(s_talk) + ((band * 16 + (lane & 15)) * space.talk_pitch + (lane >> 4) * 8) * 2;
+        const uint32_t sa = smem_addr(score) + (((lmat & 1) * 8 + lrow) * space.score_pitch + (lmat >> 1) * 8) * 2;
+#pragma unroll 2
+        for (int k = 0; k < h16; k += 16) {
+          uint32_t af[4];
+          ldsm_x4(ta + k * 2, af);
+#pragma unroll
+          for (int kb = 0; kb < kBlocks; ++kb)
+#pragma unroll
+            for (int part = 0; part < 2; ++part) {
+              uint32_t bf[4];
+              ldsm_x4_t(sa + (part * plane + k * space.score_pitch + kb * 16) * 2, bf);
+              mma_bf16(x[kb][0], af, bf[0], bf[1]);
+              mma_bf16(x[kb][1], af, bf[2], bf[3]);
             }
-          }
-          // (a half warp may have no head where the other has one: shuffles stay among a head's own lanes)
-          const uint32_t mates = TILE == 32 ? 0xffffffffu : 0xffffu << (lane & 16);
-#pragma unroll
-          for (int i = 0; i < kAtOnce; ++i) {
-            const int h = hb + i * kGroups;
-            if (h >= set_heads) break;
-            const float z = seen ? x[i] : -INFINITY;
-            float top = z;
-#pragma unroll
-            for (int off = TILE / 2; off > 0; off >>= 1) top = fmaxf(top, __shfl_xor_sync(mates, top, off));
-            const float before = s_m[h];
-            top = fmaxf(before, top);
-            const float e = talk_ex2(z - top);
-            float sum = e;
-#pragma unroll
-            for (int off = TILE / 2; off > 0; off >>= 1) sum += __shfl_xor_sync(mates, sum, off);
-            s_p[h * kPitchP + j] = __float2bfloat16_rn(e);
-            if (j == 0) {                          // (everyone has read the maximum: the sums came later)
-              const float f = talk_ex2(before - top);
-              s_f[h] = f;
-              s_m[h] = top;
-              s_l[h] = s_l[h] * f + sum;
-            }
-          }
         }
-      }
-      consumers_sync();
-      // values: (key/value head, 16 of its heads, 16 columns)
+        const int base = key0 + 2 * t4;
+        float top[2] = {m_run[i][0], m_run[i][1]}, corr[2];
 #pragma unroll
-      for (int i = 0; i < UNITS; ++i) {
-        const int u = warp + i * kWarps;
-        if (u >= all_units) break;
-        const int c16 = u % pairs, sub = u / pairs % subs, g = u / pairs / subs;
-        const int h0 = g * group + sub * 16;
-        const float f0 = s_f[min(h0 + g4, set_heads - 1)], f1 = s_f[min(h0 + g4 + 8, set_heads - 1)];
+        for (int kb = 0; kb < kBlocks; ++kb)
 #pragma unroll
-        for (int t = 0; t < 2; ++t) { o[i][t][0] *= f0; o[i][t][1] *= f0; o[i][t][2] *= f1; o[i][t][3] *= f1; }
-        const uint32_t pa = smem_addr(s_p) + (min(h0 + (lane & 15), set_heads - 1) * kPitchP + (lane >> 4) * 8) * 2;
-        const int c = min((g * a.vdim + c16 * 16) / 8 + (lmat >> 1), p.s.v_boxes * 8 - 1);      // (columns behind the head are not kept)
+          for (int t = 0; t < 2; ++t)
 #pragma unroll
-        for (int kk = 0; kk < TILE / 16; ++kk) {
-          uint32_t af[4], bf[4];
-          ldsm_x4(pa + kk * 32, af);
-          const int key = kk * 16 + (lmat & 1) * 8 + lrow;
-          ldsm_x4_t(v_at + (c >> 3) * kBox + key * 128 + (((c & 7) ^ (key & 7)) << 4), bf);
-          mma_bf16(o[i][0], af, bf[0], bf[1]);
-          mma_bf16(o[i][1], af, bf[2], bf[3]);
+            for (int e = 0; e < 4; ++e) {
+              const int key = base + kb * 16 + t * 8 + (e & 1);
+              x[kb][t][e] = key <= pos && key > pos - a.window ? x[kb][t][e] * kTalkLog2e : -INFINITY;
+              top[e >> 1] = fmaxf(top[e >> 1], x[kb][t][e]);
+            }
+#pragma unroll
+        for (int r = 0; r < 2; ++r) {
+          top[r] = fmaxf(top[r], __shfl_xor_sync(0xffffffffu, top[r], 1));
+          top[r] = fmaxf(top[r], __shfl_xor_sync(0xffffffffu, top[r], 2));
+          corr[r] = talk_ex2(m_run[i][r] - top[r]);
+          m_run[i][r] = top[r];
+          l_run[i][r] *= corr[r];
+        }
+        uint32_t pa[kBlocks][4];
+#pragma unroll
+        for (int kb = 0; kb < kBlocks; ++kb)
+#pragma unroll
+          for (int t = 0; t < 2; ++t)
+#pragma unroll
+            for (int r = 0; r < 2; ++r) {
+              const float u = talk_ex2(x[kb][t][2 * r] - top[r]), v = talk_ex2(x[kb][t][2 * r + 1] - top[r]);
+              l_run[i][r] += u + v;
+              pa[kb][t * 2 + r] = pack_bf16(u, v);
+            }
+        if (__any_sync(0xffffffffu, corr[0] != 1.f || corr[1] != 1.f)) {
+#pragma unroll
+          for (int j = 0; j < PAIRS; ++j)
+#pragma unroll
+            for (int t = 0; t < 2; ++t) { o[i][j][t][0] *= corr[0]; o[i][j][t][1] *= corr[0]; o[i][j][t][2] *= corr[1]; o[i][j][t][3] *= corr[1]; }
+        }
+        const int piece0 = (subs == 1 ? band : band / subs) * a.vdim / 8 + (lmat >> 1), last_piece = p.s.v_boxes * 8 - 1;
+        const uint32_t row_at = v_at + ((lmat & 1) * 8 + lrow) * 128;
+#pragma unroll
+        for (int j = 0; j < PAIRS; ++j) {
+          const int pair = share + j * p.s.shares;
+          if (pair < pairs) {
+            const int c = min(piece0 + 2 * pair, last_piece);      // (columns behind the head are not kept)
+            const uint32_t at = row_at + (c >> 3) * kBox + (((c & 7) ^ lrow) << 4);
+#pragma unroll
+            for (int kb = 0; kb < kBlocks; ++kb) {
+              uint32_t bf[4];
+              ldsm_x4_t(at + kb * 16 * 128, bf);
+              mma_bf16(o[i][j][0], pa[kb], bf[0], bf[1]);
+              mma_bf16(o[i][j][1], pa[kb], bf[2], bf[3]);
+            }
+          }
         }
       }
       __syncwarp();
@@ -436,15 +487,28 @@ talking_step_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_con
   float* s_o = reinterpret_cast<float*>(smem);                  // [set_heads][vdim]
   if (warp < kWarps) {
 #pragma unroll
-    for (int i = 0; i < UNITS; ++i) {
-      const int u = warp + i * kWarps;
-      if (u >= all_units) break;
-      const int c16 = u % pairs, sub = u / pairs % subs, g = u / pairs / subs;
+    for (int i = 0; i < BANDS; ++i) {
+      const int band = band0 + i * kWarps;
+      if (band >= bands) break;
+      const int sub = band % subs, h0 = band / subs * group + sub * 16, count = min(16, group - sub * 16);
 #pragma unroll
-      for (int e = 0; e < 8; ++e) {
-        const int r = sub * 16 + (lane >> 2) + ((e >> 1) & 1) * 8, c = c16 * 16 + (e >> 2) * 8 + (lane & 3) * 2 + (e & 1);
-        if (r < group && c < a.vdim) s_o[(g * group + r) * a.vdim + c] = o[i][e >> 2][e & 3];
+      for (int r = 0; r < 2; ++r) {
+        l_run[i][r] += __shfl_xor_sync(0xffffffffu, l_run[i][r], 1);
+        l_run[i][r] += __shfl_xor_sync(0xffffffffu, l_run[i][r], 2);
+        if (share == 0 && t4 == 0 && g4 + r * 8 < count) {
+          s_m[h0 + g4 + r * 8] = m_run[i][r];
+          s_l[h0 + g4 + r * 8] = l_run[i][r];
+        }
       }
+#pragma unroll
+      for (int j = 0; j < PAIRS; ++j)
+#pragma unroll
+        for (int t = 0; t < 2; ++t)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) {
+            const int r = g4 + (e >> 1) * 8, c = (share + j * p.s.shares) * 16 + t * 8 + 2 * t4 + (e & 1);
+            if (r < count && c < a.vdim) s_o[(h0 + r) * a.vdim + c] = o[i][j][t][e];
+          }
     }
   }
   __syncthreads();
@@ -485,25 +549,26 @@ constexpr size_t kSmemLimit = 227 * 1024;
 // Everything a launch needs to know about its shared memory; stages == 0: these extents do not fit.
 StepShape step_shape(int heads, int kv_heads, int dim, int vdim) {
   StepShape s{};
-  const int group = heads / kv_heads, subs = (group + 15) / 16;
+  const int group = heads / kv_heads, subs = (group + 15) / 16, pairs = (vdim + 15) / 16;
   for (int sets = 1; sets <= kv_heads; ++sets) {
+    const int kv_per_set = (kv_heads + sets - 1) / sets;
     s.sets = sets;
-    s.kv_per_set = (kv_heads + sets - 1) / sets;
-    s.units = (s.kv_per_set * subs * ((vdim + 15) / 16) + kWarps - 1) / kWarps;
-    if (s.units > kMaxUnits) continue;
+    s.bands = kv_per_set * subs;
+    s.shares = s.bands < kWarps ? kWarps / s.bands : 1;
+    s.bands_per_warp = (s.bands + kWarps - 1) / kWarps;
+    s.pairs_per_warp = (pairs + s.shares - 1) / s.shares;
+    if (s.bands_per_warp > 2 || s.bands_per_warp * s.pairs_per_warp > kMaxTiles) continue;
     s.k_boxes = (kv_heads * dim + 63) / 64;
-    s.v_boxes = (s.kv_per_set * vdim + 63) / 64;
-    const int set_heads = s.kv_per_set * group;
+    s.v_boxes = (kv_per_set * vdim + 63) / 64;
     for (int tile : {32, 16}) {
       s.tile = tile;
-      const size_t rest = 1024 + 2 * kMaxStages * 8 + static_cast<size_t>(step_floats(set_heads, heads, tile)) * 4 +
-                          static_cast<size_t>(round_to(heads * (round_to(dim, 16) + 8), 8)) * 2 + static_cast<size_t>(set_heads) * (tile + 8) * 2 + 64;
+      const size_t rest = 1024 + StepSpace(heads, dim, s.bands, kv_per_set * group, tile).total;
       const size_t stage = static_cast<size_t>(s.k_boxes + s.v_boxes) * tile * 128;
       if (rest + 2 * stage > kSmemLimit) continue;
       size_t stages = (kSmemLimit - rest) / stage;
       if (stages > kMaxStages) stages = kMaxStages;
       if (tile == 32 && stages < 3) continue;
-      if (static_cast<size_t>(set_heads) * vdim * 4 > stages * stage) continue;      // the outputs meet in the ring
+      if (static_cast<size_t>(kv_per_set) * group * vdim * 4 > stages * stage) continue;      // the outputs meet in the ring
       s.stages = static_cast<int>(stages);
       s.ring = stages * stage;
       s.smem = rest + s.ring;
@@ -514,7 +579,7 @@ StepShape step_shape(int heads, int kv_heads, int dim, int vdim) {
   return s;
 }
 
-template <int UNITS, int TILE>
+template <int BANDS, int PAIRS, int TILE>
 int launch_step(const StepParams& p, cudaStream_t st) {
   const Args& a = p.a;
   CUtensorMap tk, tv;
@@ -522,7 +587,7 @@ int launch_step(const StepParams& p, cudaStream_t st) {
   if (!talk_encode(&tk, a.keys, static_cast<uint64_t>(a.kv_heads) * a.dim, rows, TILE) ||
       !talk_encode(&tv, a.values, static_cast<uint64_t>(a.kv_heads) * a.vdim, rows, TILE))
     return CACHEIR_B200_EUNSUPPORTED;
-  auto kern = talking_step_kernel<UNITS, TILE>;
+  auto kern = talking_step_kernel<BANDS, PAIRS, TILE>;
   cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(p.s.smem));
   if (e != cudaSuccess) return static_cast<int>(e);
   cudaLaunchConfig_t cfg{};
@@ -542,9 +607,9 @@ int launch_step(const StepParams& p, cudaStream_t st) {
   return launch_status();
 }
 
-template <int UNITS>
+template <int BANDS, int PAIRS>
 int launch_tile(const StepParams& p, cudaStream_t st) {
-  return p.s.tile == 32 ? launch_step<UNITS, 32>(p, st) : launch_step<UNITS, 16>(p, st);
+  return p.s.tile == 32 ? launch_step<BANDS, PAIRS, 32>(p, st) : launch_step<BANDS, PAIRS, 16>(p, st);
 }
 
 }  // namespace
@@ -633,7 +698,9 @@ extern "C" int cacheir_b200_talking_step(const cacheir_b200_talking_args* args, 
   if (splits > kMaxSplits || a.rows > 65535) return CACHEIR_B200_ELIMIT;
   const StepParams p{a, static_cast<const __nv_bfloat16*>(q), static_cast<__nv_bfloat16*>(out), step_shape(a.heads, a.kv_heads, a.dim, a.vdim), splits};
   cudaStream_t st = as_stream(stream);
-  return p.s.units <= 2 ? launch_tile<2>(p, st) : p.s.units <= 4 ? launch_tile<4>(p, st) : p.s.units <= 8 ? launch_tile<8>(p, st) : launch_tile<kMaxUnits>(p, st);
+  const int pairs = p.s.pairs_per_warp;
+  if (p.s.bands_per_warp == 2) return pairs <= 4 ? launch_tile<2, 4>(p, st) : launch_tile<2, 8>(p, st);
+  return pairs <= 2 ? launch_tile<1, 2>(p, st) : pairs <= 4 ? launch_tile<1, 4>(p, st) : pairs <= 8 ? launch_tile<1, 8>(p, st) : launch_tile<1, 16>(p, st);
 }
 
 extern "C" int cacheir_b200_talking_device_status(int reset) {

@@ -72,9 +72,8 @@ __device__ __forceinline__ void tmem_ld_x32(uint32_t taddr, float (&v)[32]) {
         "=r"(r[20]), "=r"(r[21]), "=r"(r[22]), "=r"(r[23]), "=r"(r[24]), "=r"(r[25]), "=r"(r[26]), "=r"(r[27]), "=r"(r[28]), "=r"(r[29]),
         "=r"(r[30]), "=r"(r[31])
       : "r"(taddr) : "memory");
-  ptx::tc_wait_ld();
 #pragma unroll
-  for (int i = 0; i < 32; ++i) v[i] = __uint_as_float(r[i]);
+  for (int i = 0; i < 32; ++i) v[i] = __uint_as_float(r[i]);      // (nobody reads them before a tc_wait_ld)
 }
 __device__ __forceinline__ void tmem_ld_x16(uint32_t taddr, float (&v)[16]) {
   uint32_t r[16];
@@ -94,6 +93,25 @@ __device__ __forceinline__ void tmem_st_x16(uint32_t taddr, const uint32_t (&v)[
       "r"(v[11]), "r"(v[12]), "r"(v[13]), "r"(v[14]), "r"(v[15]) : "memory");
 }
 __device__ __forceinline__ void tmem_wait_st() { asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory"); }
+
+// pairs of float32 in one instruction
+using f32x2 = unsigned long long;
+__device__ __forceinline__ f32x2 pair(float lo, float hi) {
+  f32x2 d;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(d) : "f"(lo), "f"(hi));
+  return d;
+}
+__device__ __forceinline__ void unpair(f32x2 a, float& lo, float& hi) { asm("mov.b64 {%0, %1}, %2;" : "=f"(lo), "=f"(hi) : "l"(a)); }
+__device__ __forceinline__ f32x2 add2(f32x2 a, f32x2 b) {
+  f32x2 d;
+  asm("add.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+  return d;
+}
+__device__ __forceinline__ f32x2 fma2(f32x2 a, f32x2 b, f32x2 c) {
+  f32x2 d;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+  return d;
+}
 
 // Out of line: most waits find their barrier complete, and the loop's code would crowd theirs.
 __device__ __noinline__ bool wait_long(uint32_t bar, uint32_t parity, int code) { return ptx::mbar_wait(bar, parity, &g_prompt_status, code); }
@@ -229,30 +247,34 @@ talking_prompt_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_c
     const int tile_pos = pos0 + t * p.tokens_per_tile, rp = real ? tile_pos + tok : -1;
     const uint32_t lanes = static_cast<uint32_t>((warp & 3) * 32) << 16;
     const uint32_t scores = tmem_s + t * kKeys + lanes, outputs = tmem + t * p.n_cols + lanes;
-    const float scale = a.scale * kTalkLog2e;
+    const float scale = fabsf(a.scale) * kTalkLog2e;      // (its sign is the queries')
     float m_ref = 0.f, l = 1.f;                    // the score 0 that has no value
     for (int it = 0; it < n; ++it) {
       const int base = (page_lo + 2 * it) * kTalkPage;
       // (rows without a token may hold anything: a row of P reaches its own row of O only, which is not stored)
       const bool whole = base + kKeys - 1 <= tile_pos && base > tile_pos + count - 1 - a.window;
       const int hi = rp - base, lo = rp - a.window - base;      // seen: lo < key <= hi
+      auto mask = [&](int c, float (&v)[2][32]) {
+#pragma unroll
+        for (int j = 0; j < 64; ++j)
+          if (!(c + j <= hi && c + j > lo)) v[j >> 5][j & 31] = -INFINITY;
+      };
       wait(smem_addr(bar_s), it & 1, (11 << 8) | 9);
       __syncwarp();
       ptx::tc_fence_after();
       float mx = -INFINITY;
 #pragma unroll 1
-      for (int c = 0; c < kKeys; c += 32) {
-        float v[32];
-        tmem_ld_x32(scores + c, v);
-        if (!whole) {
+      for (int c = 0; c < kKeys; c += 64) {
+        float v[2][32], m[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
+        tmem_ld_x32(scores + c, v[0]);
+        tmem_ld_x32(scores + c + 32, v[1]);
+        ptx::tc_wait_ld();
+        if (!whole) mask(c, v);
 #pragma unroll
-          for (int j = 0; j < 32; ++j)
-            if (!(c + j <= hi && c + j > lo)) v[j] = -INFINITY;
-        }
-        // (with a negative scale the largest score is the smallest product)
-#pragma unroll
-        for (int j = 0; j < 32; ++j) mx = fmaxf(mx, v[j] == -INFINITY ? -INFINITY : v[j] * scale);
+        for (int j = 0; j < 64; ++j) m[j & 3] = fmaxf(m[j & 3], v[j >> 5][j & 31]);
+        mx = fmaxf(mx, fmaxf(fmaxf(m[0], m[1]), fmaxf(m[2], m[3])));
       }
+      mx *= scale;
       float alpha = 1.f;
       if (mx > m_ref + kStale) {
         alpha = talk_ex2(m_ref - mx);
@@ -270,26 +292,32 @@ talking_prompt_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_c
           tmem_st_x16(outputs + c, bits);
         }
       }
-      float sum[2] = {0.f, 0.f};
+      const f32x2 factor = pair(scale, scale), minus_ref = pair(-m_ref, -m_ref);
+      f32x2 sum[2] = {pair(0.f, 0.f), pair(0.f, 0.f)};
 #pragma unroll 1
-      for (int c = 0; c < kKeys; c += 32) {
-        float v[32];
-        tmem_ld_x32(scores + c, v);
-        uint32_t packed[16];
+      for (int c = 0; c < kKeys; c += 64) {
+        float v[2][32];
+        tmem_ld_x32(scores + c, v[0]);
+        tmem_ld_x32(scores + c + 32, v[1]);
+        ptx::tc_wait_ld();
+        if (!whole) mask(c, v);
+        uint32_t packed[2][16];
 #pragma unroll
-        for (int j = 0; j < 32; j += 2) {
-          float x = talk_ex2(fmaf(v[j], scale, -m_ref)), y = talk_ex2(fmaf(v[j + 1], scale, -m_ref));
-          if (!whole) {
-            if (!(c + j <= hi && c + j > lo)) x = 0.f;
-            if (!(c + j + 1 <= hi && c + j + 1 > lo)) y = 0.f;
-          }
-          sum[0] += x;
-          sum[1] += y;
-          packed[j / 2] = pack_bf16(x, y);
+        for (int j = 0; j < 64; j += 2) {
+          float x, y;
+          unpair(fma2(pair(v[j >> 5][j & 31], v[j >> 5][(j & 31) + 1]), factor, minus_ref), x, y);
+          x = talk_ex2(x);
+          y = talk_ex2(y);
+          sum[(j >> 1) & 1] = add2(sum[(j >> 1) & 1], pair(x, y));
+          packed[j >> 5][(j & 31) / 2] = pack_bf16(x, y);
         }
-        tmem_st_x16(scores + c / 2, packed);       // (behind what this thread has read)
+        tmem_st_x16(scores + c / 2, packed[0]);       // (behind what this thread has read)
+        tmem_st_x16(scores + c / 2 + 16, packed[1]);
       }
-      l += sum[0] + sum[1];
+      float part[4];
+      unpair(sum[0], part[0], part[1]);
+      unpair(sum[1], part[2], part[3]);
+      l += (part[0] + part[1]) + (part[2] + part[3]);
       tmem_wait_st();
       const int tail = pos_last + 1 - base;
       if (tail < kKeys && t == 0) {                // values behind the last token may be anything: zero, so that 0 * value stays 0

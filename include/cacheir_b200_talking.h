@@ -35,7 +35,7 @@ typedef struct {
 /* q, k, v as projected. Queries and keys are rotated (rotate-half pairs on the first rot_dims entries of a head; rope_table: float2
  * (cos, sin) [rope_positions, rot_dims / 2]), values divided by their root mean square per head; keys and values go to the cache.
  * q_out [rows, heads, dim]: rotated queries. With `mixed`, [rows, heads, kv_heads*dim]: what head h multiplies a whole cached key
- * row with to get its mixed score, for every key/value head the sum of talk[h, g] q_g over its heads g (dim % 8 == 0). */
+ * row with to get its mixed score, for every key/value head the sum of talk[h, g] q_g over its heads g, with the sign of the scale (dim % 8 == 0). */
 int cacheir_b200_talking_prepare(const cacheir_b200_talking_args* a, const void* q, long long q_stride, const void* k, long long k_stride,
                                  const void* v, long long v_stride, int rot_dims, const float* rope_table, int rope_positions, float eps,
                                  int mixed, void* q_out, void* stream);
